@@ -73,19 +73,62 @@ def kernel_sources() -> list[Path]:
     return sorted(CSRC.glob("*.cu"))
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
-    """Compile ``csrc/*.cu`` for sm_100a and link ``_kernels.so``. Needs no GPU."""
-    srcs = kernel_sources()
+# What the models of one architecture launch, for a process that serves only that: the first
+# use in a fresh checkout then compiles these files and leaves the others alone.
+KERNEL_SETS = {
+    "Taralix": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm",
+                "latent_attention", "moe", "sampling", "stream"),
+}
+_kernel_set: str | None = None
+
+
+def select_kernel_set(architecture: str) -> None:
+    """Called before the first kernel is loaded: this process serves ``architecture``."""
+    global _kernel_set
+    _kernel_set = architecture if architecture in KERNEL_SETS else None
+
+
+def load_kernel_set() -> ctypes.CDLL | None:
+    """The selected architecture's kernels as a library of their own, built if needed; None when
+    no set is selected or the whole library is there already."""
+    if _kernel_set is None or _kernel_lib is not None:
+        return None
+    if os.environ.get("ARCTIC_B200_NO_AUTOBUILD") or not _stale_sources(kernel_sources()) and \
+            KERNEL_LIB.exists():
+        return None
+    with _lock:
+        stems = KERNEL_SETS[_kernel_set]
+        out = PKG_DIR / ("_kernels_%s.so" % _kernel_set.lower())
+        build_kernels(sources=[s for s in kernel_sources() if s.stem in stems], out=out)
+        return ctypes.CDLL(str(out), mode=ctypes.RTLD_LOCAL)
+
+
+def _object_of(src: Path) -> Path:
+    return OBJ_DIR / (src.stem + ".o")
+
+
+def _stale_sources(srcs, hdr_time: float | None = None) -> list[Path]:
+    hdr_time = _newest(_headers()) if hdr_time is None else hdr_time
+    return [s for s in srcs if not _object_of(s).exists() or
+            _object_of(s).stat().st_mtime < max(s.stat().st_mtime, hdr_time)]
+
+
+def build_kernels(force: bool = False, verbose: bool = False, sources=None,
+                  out: Path | None = None) -> Path:
+    """Compile ``csrc/*.cu`` for sm_100a and link ``_kernels.so``. Needs no GPU. ``sources`` and
+    ``out``: a part of the library under another name."""
+    srcs = kernel_sources() if sources is None else sources
+    lib_path = KERNEL_LIB if out is None else out
     hdr_time = _newest(_headers())
     OBJ_DIR.mkdir(exist_ok=True)
     nvcc = _nvcc()
     jobs = []
     objs = []
+    stale = set(srcs if force else _stale_sources(srcs, hdr_time))
     for src in srcs:
-        obj = OBJ_DIR / (src.stem + ".o")
+        obj = _object_of(src)
         objs.append(obj)
-        stale = force or not obj.exists() or obj.stat().st_mtime < max(src.stat().st_mtime, hdr_time)
-        if stale:
+        if src in stale:
             cmd = [nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
             if verbose:
                 cmd.insert(1, "-Xptxas=-v")
@@ -93,11 +136,12 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
     if jobs:
         with ThreadPoolExecutor(max_workers=min(len(jobs), os.cpu_count() or 4)) as pool:
             list(pool.map(_run, jobs))
-    if jobs or force or not KERNEL_LIB.exists() or KERNEL_LIB.stat().st_mtime < _newest(objs):
-        tmp = KERNEL_LIB.with_suffix(".so.tmp%d" % os.getpid())
-        _run([nvcc, "-shared", "-o", str(tmp), *[str(o) for o in objs]])
-        os.replace(tmp, KERNEL_LIB)
-    return KERNEL_LIB
+    if jobs or force or not lib_path.exists() or lib_path.stat().st_mtime < _newest(objs):
+        tmp = lib_path.with_suffix(".so.tmp%d" % os.getpid())
+        # (-Bsymbolic: two libraries with the same kernels in one process keep to their own)
+        _run([nvcc, "-shared", "-Xlinker", "-Bsymbolic", "-o", str(tmp), *[str(o) for o in objs]])
+        os.replace(tmp, lib_path)
+    return lib_path
 
 
 def suffix_lib_path() -> Path:

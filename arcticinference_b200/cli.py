@@ -2,6 +2,7 @@
 
     serve MODEL [engine flags] [--host H --port P]     OpenAI-compatible server
     server [--host H --port P]                          replica-pool REST server
+    trace-run --model DIR --out DIR --max-tokens N      logits of given tokens (bin/trace_run)
     bench-embedding ...                                 see benchmarks/embedding_bench.py
 
 ``serve`` takes the flags the reference adds to ``vllm serve`` (README.md:98-124,
@@ -108,11 +109,17 @@ def make_parser() -> argparse.ArgumentParser:
     r.add_argument("--host", default="0.0.0.0")
     r.add_argument("--port", type=int, default=8000)
     r.set_defaults(fn=_server)
+    sub.add_parser("trace-run", help="replay token ids step by step and write logits "
+                                     "(the arguments of bin/trace_run)", add_help=False)
     return ap
 
 
 def main(argv=None) -> int:
     logging.basicConfig(level=logging.INFO)
+    args = list(sys.argv[1:] if argv is None else argv)
+    if args[:1] == ["trace-run"]:
+        from .entrypoints.trace_run import main as trace_run
+        return trace_run(args[1:])
     ns = make_parser().parse_args(argv)
     ns.argv = list(sys.argv[1:] if argv is None else argv)
     return ns.fn(ns)

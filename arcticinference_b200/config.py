@@ -30,10 +30,84 @@ logger = logging.getLogger(__name__)
 
 SHIFT_PARALLEL_THRESHOLD = 128
 
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Attention whose keys and values are linear maps of one latent vector per token: only the
+    latent (``kv_rank`` numbers) is cached. ``kv_from``: take the latents of that earlier layer
+    instead of projecting and caching some of one's own."""
+    heads: int
+    dim: int          # query / key dimensions per head
+    vdim: int         # value dimensions per head
+    kv_rank: int
+    scale: float      # factor of the scores
+    kv_from: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class FeedForwardSpec:
+    """A gated feed-forward layer, or ``experts`` of them of which every token uses ``top``."""
+    ff: int
+    act: str = "silu"     # silu | gelu_tanh
+    experts: int = 0      # 0: dense
+    top: int = 0
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One decoder layer of a model that lists its layers one by one."""
+    mixer: LatentAttentionSpec
+    mlp: Optional[FeedForwardSpec] = None
+
+
+def read_layer_specs(layers: list) -> tuple:
+    """The ``layers`` list of a layer-list checkpoint's config.json."""
+    out = []
+    for i, d in enumerate(layers):
+        if d.get("type") != "latent_attention":
+            raise NotImplementedError("layer %d: mixer type %r (supported: latent_attention)"
+                                      % (i, d.get("type")))
+        m = d["mixer"]
+        src = m.get("kv_from")
+        mixer = LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                    kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+                                    kv_from=None if src is None else int(src))
+        f, mlp = d.get("mlp"), None
+        if f is not None:
+            kind = f.get("kind")
+            if kind == "dense":
+                mlp = FeedForwardSpec(ff=int(f["ff"]), act="gelu_tanh")
+            elif kind == "moe":
+                mlp = FeedForwardSpec(ff=int(f["expert"]["ff"]), act="silu",
+                                      experts=int(f["router"]["experts"]),
+                                      top=int(f["router"]["top"]))
+            else:
+                raise NotImplementedError("layer %d: feed-forward kind %r (supported: dense, moe)"
+                                          % (i, kind))
+        out.append(LayerSpec(mixer, mlp))
+    return tuple(out)
+
+
+def validate_layer_specs(specs: tuple) -> None:
+    for i, l in enumerate(specs):
+        m, f = l.mixer, l.mlp
+        if min(m.heads, m.dim, m.vdim, m.kv_rank) < 1:
+            raise ValueError("layer %d: heads, dim, vdim and kv_rank must be positive" % i)
+        if m.kv_from is not None:
+            if not 0 <= m.kv_from < i:
+                raise ValueError("layer %d: kv_from must name an earlier layer" % i)
+            src = specs[m.kv_from].mixer
+            if src.kv_from is not None or src.kv_rank != m.kv_rank:
+                raise ValueError("layer %d: layer %d has no latents of this kv_rank of its own"
+                                 % (i, m.kv_from))
+        if f is not None and f.experts and not 1 <= f.top <= f.experts:
+            raise ValueError("layer %d: top must lie between 1 and the number of experts" % i)
+
+
 @dataclass
 class ModelConfig:
     """Architecture of a decoder (Llama, Mistral, Qwen2 and Qwen3 dense models, optionally
-    SwiftKV for Llama) or encoder (BERT)."""
+    SwiftKV for Llama; Taralix, which lists its layers one by one) or encoder (BERT)."""
 
     architecture: str = "LlamaForCausalLM"
     model_type: str = "llama"
@@ -61,6 +135,10 @@ class ModelConfig:
     sliding_window: Optional[int] = None
     # K/V heads of the checkpoint when ``num_key_value_heads`` was raised (see __post_init__)
     checkpoint_kv_heads: Optional[int] = None
+    # models that list their layers (each with its own mixer and feed-forward)
+    layer_specs: Optional[tuple] = None
+    # factor of the residual stream in "norm after the sum" layers: x <- norm(alpha * x + f(x))
+    postln_alpha: float = 1.0
     # encoder-only fields
     type_vocab_size: int = 2
     layer_norm_eps: float = 1e-12
@@ -88,7 +166,7 @@ class ModelConfig:
         function, the KV cache is r times larger. ``num_key_value_heads`` is the number of
         heads stored; ``checkpoint_kv_heads`` keeps the checkpoint's."""
         hq, hkv = self.num_attention_heads, self.num_key_value_heads
-        if self.is_encoder or hkv <= 0 or hq % hkv:
+        if self.is_encoder or self.layer_specs is not None or hkv <= 0 or hq % hkv:
             return
         g = hq // hkv
         if 128 % g == 0:
@@ -111,7 +189,18 @@ class ModelConfig:
     def is_encoder(self) -> bool:
         return self.model_type in ("bert",)
 
+    @property
+    def supports_float32(self) -> bool:
+        """Whether the model can be served with 32-bit weights, activations and cache."""
+        return self.layer_specs is not None
+
     def validate(self) -> None:
+        if self.layer_specs is not None:
+            validate_layer_specs(self.layer_specs)
+            if self.quantization is not None:
+                raise NotImplementedError("quantization=%r for %s" % (self.quantization,
+                                                                      self.architecture))
+            return
         if self.num_attention_heads % self.num_key_value_heads:
             raise ValueError("num_attention_heads must be a multiple of num_key_value_heads")
         if self.head_dim not in (64, 128):
@@ -177,11 +266,36 @@ class ModelConfig:
         return cfg
 
     @classmethod
+    def from_layer_list(cls, d: dict, name_or_path: str = "") -> "ModelConfig":
+        """config.json of a layer-list model (``architecture``, ``width``, ``vocab``, ``norm``,
+        ``postln_alpha`` and ``layers``). The head fields describe the cache as the engine sees
+        it: one latent "head" of ``kv_rank`` numbers (the largest, where layers differ)."""
+        specs = read_layer_specs(d["layers"])
+        if not specs:
+            raise ValueError("a model without layers")
+        eos = d.get("eos_token_id")
+        return cls(
+            architecture=d["architecture"], model_type=d["architecture"].lower(),
+            hidden_size=int(d["width"]), num_hidden_layers=len(specs),
+            num_attention_heads=max(l.mixer.heads for l in specs), num_key_value_heads=1,
+            head_dim=max(l.mixer.kv_rank for l in specs),
+            intermediate_size=max((l.mlp.ff for l in specs if l.mlp is not None), default=0),
+            vocab_size=int(d["vocab"]), rms_norm_eps=float(d["norm"]["eps"]),
+            postln_alpha=float(d["postln_alpha"]), layer_specs=specs,
+            # nothing in the model depends on a position's number, so nothing bounds it
+            max_position_embeddings=1 << 20, hidden_act="",
+            eos_token_id=int(eos) if isinstance(eos, int) else None, name_or_path=name_or_path)
+
+    @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
         if path in PRESETS:
             return dataclasses.replace(PRESETS[path], name_or_path=path)
         with open(os.path.join(path, "config.json")) as f:
-            cfg = cls.from_hf_dict(json.load(f), path)
+            d = json.load(f)
+        if d.get("architecture") in LAYER_LIST_ARCHITECTURES:
+            cfg = cls.from_layer_list(d, path)
+        else:
+            cfg = cls.from_hf_dict(d, path)
         gen = os.path.join(path, "generation_config.json")
         if os.path.exists(gen):
             with open(gen) as f:
@@ -198,6 +312,28 @@ class ModelConfig:
 # sliding window is off; Qwen2 adds a bias on the QKV projection; Qwen3 (dense) adds the
 # per-head query / key norms and a head_dim that is not hidden_size / heads
 DECODER_MODEL_TYPES = ("llama", "llama_swiftkv", "mistral", "qwen2", "qwen3")
+
+# models whose config.json lists the layers instead of giving one shape for all of them
+LAYER_LIST_ARCHITECTURES = ("Taralix",)
+
+
+def _taralix(width, vocab, layers, alpha, eps=1e-6) -> ModelConfig:
+    """``layers``: (heads, dim, vdim, kv_rank, kv_from, feed-forward) each; the feed-forward is
+    None, ff (dense) or (ff, experts, top)."""
+    out = []
+    for heads, dim, vdim, rank, src, f in layers:
+        m = {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": rank, "scale": dim ** -0.5}
+        if src is not None:
+            m["kv_from"] = src
+        mlp = None
+        if isinstance(f, int):
+            mlp = {"kind": "dense", "ff": f}
+        elif f is not None:
+            mlp = {"kind": "moe", "expert": {"ff": f[0]}, "router": {"experts": f[1], "top": f[2]}}
+        out.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+    return ModelConfig.from_layer_list({"architecture": "Taralix", "width": width, "vocab": vocab,
+                                        "norm": {"eps": eps}, "postln_alpha": alpha,
+                                        "layers": out})
 
 
 def _llama(layers, hidden, heads, kv, inter, **kw) -> ModelConfig:
@@ -266,6 +402,8 @@ PRESETS: dict[str, ModelConfig] = {
                              num_hidden_layers=2, num_attention_heads=2, num_key_value_heads=2,
                              head_dim=64, intermediate_size=256, vocab_size=1000,
                              max_position_embeddings=512, hidden_act="gelu"),
+    "taralix-tiny": _taralix(192, 1024, [(6, 32, 48, 96, None, 320), (4, 64, 32, 96, 0, (64, 8, 3)),
+                                         (5, 40, 64, 40, None, None)], alpha=1.7),
 }
 
 
@@ -482,6 +620,8 @@ class EngineConfig:
         m, p = self.model, self.parallel
         m.validate()
         ways = p.tp * p.sp
+        if m.layer_specs is not None:
+            self._validate_layer_list()
         if m.num_attention_heads % ways:
             raise ValueError("num_attention_heads (%d) must be divisible by TP*SP (%d)" %
                              (m.num_attention_heads, ways))
@@ -494,7 +634,7 @@ class EngineConfig:
                 "sliding-window attention: this checkpoint attends to the last %d tokens only; "
                 "contexts up to that length are served (max_model_len=%d asks for more)"
                 % (m.sliding_window, self.scheduler.max_model_len))
-        if not m.is_encoder:
+        if not m.is_encoder and m.layer_specs is None:
             per_rank = (m.num_attention_heads // ways) // max(1, m.num_key_value_heads // ways)
             if per_rank < 1 or 128 % per_rank:
                 raise NotImplementedError(
@@ -530,6 +670,15 @@ class EngineConfig:
             raise ValueError("suffix decoding is only available with the arctic or suffix methods")
         if self.scheduler.max_num_batched_tokens < p.sp:
             raise ValueError("max_num_batched_tokens must be >= the sequence-parallel size")
+
+    def _validate_layer_list(self) -> None:
+        """What layer-list models do not run with is refused here."""
+        m, p = self.model, self.parallel
+        if p.world_size > 1:
+            raise NotImplementedError("%s on more than one GPU (tensor, sequence or pipeline "
+                                      "parallelism)" % m.architecture)
+        if self.forest_cascade.enabled:
+            raise NotImplementedError("forest cascade attention with %s" % m.architecture)
 
     @property
     def kv_replication(self) -> int:
@@ -668,10 +817,14 @@ class EngineArgs:
             model.quantization = self.quantization
         if self.fp8_scheme is not None:
             model.fp8_scheme = self.fp8_scheme
-        if self.dtype not in ("auto", "bfloat16", "bf16"):
-            raise NotImplementedError("dtype=%r: weights, activations and the KV cache are "
-                                      "bfloat16 (the kernels accumulate in fp32)" % self.dtype)
-        model.dtype = "bfloat16"
+        if self.dtype in ("float32", "fp32", "float") and model.supports_float32:
+            model.dtype = "float32"
+        elif self.dtype in ("auto", "bfloat16", "bf16"):
+            model.dtype = "bfloat16"
+        else:
+            raise NotImplementedError("dtype=%r: weights, activations and the KV cache of %s are "
+                                      "bfloat16 (the kernels accumulate in fp32)"
+                                      % (self.dtype, model.architecture))
         max_len = self.max_model_len or min(model.max_position_embeddings, 8192,
                                             model.sliding_window or 8192)
         parallel = ParallelConfig(

@@ -107,6 +107,9 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
                     long long T, int Hq, int Hkv, int D, int causal, float scale, void* out,
                     long long ldo, void* o_part, void* lse_part, void* lse_out, int tile_keys,
                     int* status, cudaStream_t stream);
+int ab200_attention_merge(const void* o_part, const void* lse_part, const void* tok_splits,
+                          long long T, int Hq, int D, void* out, long long ldo,
+                          cudaStream_t stream);
 int ab200_attention_scatter(const void* q, long long ldq, const void* k, const void* v,
                             long long num_blocks, int block_size, const void* block_tables,
                             int max_blocks, const void* work, int num_work,
@@ -225,6 +228,52 @@ int ab200_argmax_exchange(const void* ids, const void* vals, int B, int max_rows
                           const void* const* slot_ptrs, const void* const* flag_ptrs, int my_rank,
                           int world, void* epoch_ctr, void* out_ids, void* out_vals, int* status,
                           cudaStream_t stream);
+
+// ---- stream.cu (dtype: 0 = bf16, 1 = fp32 elements; the residual stream is always fp32)
+int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, long long T,
+                           int W, long long vocab, int dtype, int* status, cudaStream_t stream);
+int ab200_stream_norm(const void* x, const void* rows, const void* y, long long ldy,
+                      const void* y_rows, const void* y_weights, int top, const void* weight,
+                      float alpha, float eps, void* x_out, void* act_out, long long T, int W,
+                      int dtype, cudaStream_t stream);
+int ab200_latent_norm_cache(const void* ckv, long long ld, const void* weight, int R, int Rp,
+                            float eps, const void* slots, void* cache, long long num_slots,
+                            long long T, int dtype, int* status, cudaStream_t stream);
+int ab200_gated_act(const void* gu, void* out, long long T, int ff, int act, int dtype,
+                    cudaStream_t stream);
+
+// ---- exact.cu
+int ab200_linear_exact(const void* x, long long ldx, long long x_gstride, const void* w,
+                       long long ldw, long long w_gstride, void* out, long long ldo,
+                       long long out_gstride, int M, int N, int K, int groups, const void* tiles,
+                       const void* num_tiles, int max_tiles, int dtype, cudaStream_t stream);
+int ab200_latent_attention_exact(const void* q, long long ldq, const void* cache, int num_blocks,
+                                 int block_size, const void* block_tables, int max_blocks,
+                                 const void* tok_seq, const void* positions, void* out,
+                                 long long ldo, long long T, int H, int R, float scale, int dtype,
+                                 int* status, cudaStream_t stream);
+
+// ---- moe.cu
+int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,
+                    void* ids, void* weights, int dtype, cudaStream_t stream);
+int ab200_moe_plan(const void* ids, long long n, int E, void* cursor, void* tiles, void* num_tiles,
+                   cudaStream_t stream);
+int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, void* xp,
+                      long long T, int W, int top, int dtype, cudaStream_t stream);
+
+// ---- grouped_gemm.cu
+int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long long x_rows,
+                       const void* w, long long ldw, long long w_gstride, void* out, long long ldo,
+                       long long out_gstride, int M, int N, int K, int groups, const void* tiles,
+                       const void* num_tiles, int max_tiles, int act, int* status,
+                       cudaStream_t stream);
+
+// ---- latent_attention.cu
+int ab200_latent_attention(const void* q, long long q_rows, const void* cache, int num_blocks,
+                           int block_size, const void* block_tables, int max_blocks,
+                           const void* work, int num_work, const void* tok_splits, int max_splits,
+                           long long T, int H, int R, int tile_rows, float scale, void* out,
+                           void* o_part, void* lse_part, int* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

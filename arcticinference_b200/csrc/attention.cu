@@ -57,7 +57,8 @@ struct AttnArgs {
   const int* block_tables;  // [num_seqs][max_blocks] (paged mode)
   int max_blocks;
   int block_size;  // 0 = contiguous K/V
-  int G;           // query heads per KV head
+  int G;           // query heads per KV head, rounded up to a power of two (rows per token)
+  int g_heads;     // query heads per KV head
   int Hq, Hkv;
   int causal;
   float scale_log2;  // softmax scale * log2(e)
@@ -340,7 +341,7 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     const int c_first = half * kLocalChunks;
     const int tok_local = row / p.G;
     const int g = row % p.G;
-    const bool valid_row = tok_local < n_q_tok;
+    const bool valid_row = tok_local < n_q_tok && g < p.g_heads;
     const int q_pos = q_pos0 + tok_local;
     const int limit = p.causal ? min(q_pos, kv_end - 1) : kv_end - 1;  // last visible key
     const uint32_t lane_off = (uint32_t)(quad * 32) << 16;
@@ -534,7 +535,7 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     if (ok && warp_active) {  // warp-uniform: every lane takes part in the TMEM reads
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
       const long long tok = (long long)q_tok0 + tok_local;
-      const int head = kvh * p.G + g;
+      const int head = kvh * p.g_heads + g;
       const float lse = l > 0.f ? m * p.scale + logf(l) : -INFINITY;
       __nv_bfloat16* dst16 = p.out + tok * p.ldo + (long long)head * D;
       if (p.peer_tokens > 0)
@@ -696,9 +697,11 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
                             float* lse_part, float* lse_out, int* status, cudaStream_t stream,
                             const void* const* peer_ptrs = nullptr, int world = 0,
                             int peer_tokens = 0, const Ab200PeerSync* sync = nullptr) {
-  const int G = Hq / Hkv;
+  const int heads = Hq / Hkv;
+  int G = 1;
+  while (G < heads) G *= 2;
   if (peer_tokens > 0 && (world < 1 || world > 16 || peer_ptrs == nullptr)) return -2;
-  if (G <= 0 || Hq % Hkv || 128 % G) return -2;
+  if (heads <= 0 || Hq % Hkv || G > 128) return -2;
   if (block_size > 0 && (TK % block_size || block_size < 8)) return -2;
   static bool attr_set[64] = {false};
   int dev = 0;
@@ -714,9 +717,9 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   }
   CUtensorMap tq, tk, tv;
   {
-    // q viewed as [T][Hkv][G][D]
-    const uint64_t dims[4] = {(uint64_t)D, (uint64_t)G, (uint64_t)Hkv, (uint64_t)T};
-    const uint64_t strides[3] = {(uint64_t)D * 2, (uint64_t)G * D * 2, (uint64_t)ldq * 2};
+    // q viewed as [T][Hkv][heads][D]; the box is G heads high, rows past `heads` read as zero
+    const uint64_t dims[4] = {(uint64_t)D, (uint64_t)heads, (uint64_t)Hkv, (uint64_t)T};
+    const uint64_t strides[3] = {(uint64_t)D * 2, (uint64_t)heads * D * 2, (uint64_t)ldq * 2};
     const uint32_t box[4] = {64, (uint32_t)G, 1, (uint32_t)(128 / G)};
     if (make_tmap_nd(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, dims, strides, box) != 0) return -4;
   }
@@ -745,6 +748,7 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   a.max_blocks = max_blocks;
   a.block_size = block_size;
   a.G = G;
+  a.g_heads = heads;
   a.Hq = Hq;
   a.Hkv = Hkv;
   a.causal = causal;
@@ -820,6 +824,26 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
                       reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, causal, scale,
                       out, ldo, reinterpret_cast<float*>(o_part), reinterpret_cast<float*>(lse_part),
                       reinterpret_cast<float*>(lse_out), status, stream);
+}
+
+// Folds split-KV partials of another attention kernel (same layouts as above): o_part fp32
+// [splits, T, Hq, D], D a multiple of 128 up to 512, out bf16.
+int ab200_attention_merge(const void* o_part, const void* lse_part, const void* tok_splits,
+                          long long T, int Hq, int D, void* out, long long ldo,
+                          cudaStream_t stream) {
+  AttnArgs a;
+  memset(&a, 0, sizeof(a));
+  auto k = D == 128   ? attention_merge_kernel<128>
+           : D == 256 ? attention_merge_kernel<256>
+           : D == 384 ? attention_merge_kernel<384>
+                      : attention_merge_kernel<512>;
+  if (D != 128 && D != 256 && D != 384 && D != 512) return -2;
+  return launch_pdl(k, dim3((unsigned)T), dim3(D >= 256 ? 256 : 128), 0, stream,
+                    reinterpret_cast<const float*>(o_part), reinterpret_cast<const float*>(lse_part),
+                    reinterpret_cast<const int*>(tok_splits), T, Hq,
+                    reinterpret_cast<__nv_bfloat16*>(out), ldo, (float*)nullptr, a) == cudaSuccess
+             ? 0
+             : -5;
 }
 
 // Paged attention whose output rows are scattered to `world` peer buffers (see AttnArgs):

@@ -1,0 +1,561 @@
+// Attention in latent space for sm_100a: queries [T, H, R] against a paged cache of one latent
+// vector of R = 128 .. 512 numbers per token, which is key and value of every head at once.
+// Decode and short chunks; softmax over every key up to the token itself.
+//
+// The keys are the tensor core's M side. Per tile of 128 keys
+//     S^T [128 keys x n]   = C Q^T       (tcgen05.mma, A = the latents K-major as they lie)
+//     O^T [R x n]         += C^T P^T     (A = the same shared-memory tile read MN-major)
+// with n = 16 .. 64 query rows. A row is one (token, head) pair and rows of a sequence are simply
+// consecutive rows of the query matrix, so any number of heads packs without padding and a
+// decode tile of 16 heads is 16 columns wide instead of 16 of 128 padded rows. Every latent is
+// fetched once per tile and used twice. O^T takes R/128 * n TMEM columns (n = 48, R = 512: 192),
+// which is what lets one CTA own the whole latent width.
+//
+// Latents arrive as 128 x 64 pieces (one 128-byte swizzle atom wide) in a ring; a piece is free
+// again when its share of O^T has been accumulated. While the tensor core works on tile j, the
+// pieces of tile j + 1 are loading (R <= 256: whole tiles ahead, and S of tile j + 1 is issued
+// before O of tile j).
+//
+// Softmax: four warps, a thread per key. A column's maximum over the keys is a butterfly over
+// the warp's lanes (16 columns in 16 shuffles) and four words of shared memory; sums stay
+// per-thread until the end. O is rescaled only in tiles where a maximum moved.
+//
+// With several pieces of the keys per sequence a CTA writes normalised fp32 partials and their
+// log-sum-exp, folded by the merge kernel of attention.cu.
+
+#include <math.h>
+#include <string.h>
+
+#include "api.h"
+#include "common/pdl.cuh"
+#include "common/ptx.cuh"
+#include "common/tensormap.h"
+
+namespace ab200 {
+
+constexpr int kLatThreads = 192;      // 4 softmax warps, the TMA warp, the MMA warp
+constexpr int kLatKeys = 128;
+constexpr uint32_t kPieceBytes = kLatKeys * 64 * 2;
+constexpr int kLatMaxSlots = 12;
+
+struct LatentArgs {
+  const int* work;   // [num_work][8]: sequence, first row, rows (0 = no-op), position of row r's
+                     // token minus r / H, first key, last key + 1, piece, pieces
+  const int* block_tables;
+  int max_blocks, block_size;
+  int H, pieces;           // pieces: R / 64 per tile
+  int slots, p_bufs, overlap;
+  float scale, scale_log2;
+  uint32_t tmem_cols;
+  __nv_bfloat16* out;      // [T * H][R]
+  float* o_part;           // [pieces of keys][T * H][R]
+  float* lse_part;         // [pieces of keys][T * H]
+  long long rows_total;    // T * H
+  int* status;
+};
+
+__device__ __forceinline__ void bar_softmax() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+
+__device__ __forceinline__ void tmem_ld_wait_dep16(uint32_t (&r)[16]) {
+  asm volatile("tcgen05.wait::ld.sync.aligned;"
+               : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]),
+                 "+r"(r[7]), "+r"(r[8]), "+r"(r[9]), "+r"(r[10]), "+r"(r[11]), "+r"(r[12]),
+                 "+r"(r[13]), "+r"(r[14]), "+r"(r[15])
+               :
+               : "memory");
+}
+__device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]),
+      "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]),
+      "r"(r[15])
+      : "memory");
+}
+
+// Reduces 16 values over the warp's lanes: lane l ends with the result of value
+// ((l >> 4) & 1) * 8 + ((l >> 3) & 1) * 4 + ((l >> 2) & 1) * 2 + ((l >> 1) & 1).
+template <bool MAX>
+__device__ __forceinline__ float reduce16(float (&v)[16], int lane) {
+#pragma unroll
+  for (int w = 8, o = 16; w >= 1; w >>= 1, o >>= 1) {
+    const bool hi = (lane & o) != 0;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (i < w) {
+        const float mine = hi ? v[i + w] : v[i];
+        const float send = hi ? v[i] : v[i + w];
+        const float got = __shfl_xor_sync(0xffffffffu, send, o);
+        v[i] = MAX ? fmaxf(mine, got) : mine + got;
+      }
+    }
+  }
+  const float other = __shfl_xor_sync(0xffffffffu, v[0], 1);
+  return MAX ? fmaxf(v[0], other) : v[0] + other;
+}
+__device__ __forceinline__ int reduce16_index(int lane) {
+  return ((lane >> 4) & 1) * 8 + ((lane >> 3) & 1) * 4 + ((lane >> 2) & 1) * 2 + ((lane >> 1) & 1);
+}
+
+template <int NR>
+__global__ void __launch_bounds__(kLatThreads, 1)
+latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
+                        const __grid_constant__ CUtensorMap tmap_c, const LatentArgs p) {
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
+                                             ~static_cast<uintptr_t>(1023));
+  __shared__ __align__(16) float wred[NR * 4];   // per column: the four warps' values
+  __shared__ __align__(16) float m_s[NR], neg_s[NR], alpha_s[NR], inv_s[NR];
+  __shared__ int lim_s[NR];                      // last visible key of each row
+  __shared__ int rescale_s[2];
+  __shared__ uint64_t bars[1 + 2 * kLatMaxSlots + 8];
+  __shared__ uint32_t tmem_slot;
+  __shared__ volatile int abort_s;
+
+  const int NC = p.pieces;
+  const uint32_t sQ = smem_u32(smem);
+  const uint32_t sC = sQ + (uint32_t)NC * NR * 128u;
+  const uint32_t sP = sC + (uint32_t)p.slots * kPieceBytes;
+  uint8_t* pC = smem + (size_t)NC * NR * 128;
+  uint8_t* pP = pC + (size_t)p.slots * kPieceBytes;
+  const uint32_t bb = smem_u32(bars);
+  const uint32_t q_full = bb;
+  auto c_full = [&](int s) { return bb + 8u * (1 + s); };
+  auto c_empty = [&](int s) { return bb + 8u * (1 + kLatMaxSlots + s); };
+  auto s_full = [&](int s) { return bb + 8u * (1 + 2 * kLatMaxSlots + s); };
+  auto s_empty = [&](int s) { return bb + 8u * (3 + 2 * kLatMaxSlots + s); };
+  auto p_full = [&](int s) { return bb + 8u * (5 + 2 * kLatMaxSlots + s); };
+  auto o_full = [&](int s) { return bb + 8u * (7 + 2 * kLatMaxSlots + s); };
+  const int warp = threadIdx.x >> 5;
+  const int lane = threadIdx.x & 31;
+
+  pdl_trigger();
+  const int* wk = p.work + (long long)blockIdx.x * 8;
+  const int n_rows = wk[2];
+  if (n_rows <= 0) {   // padding entry of a fixed-size work list
+    pdl_wait();
+    return;
+  }
+  const int seq = wk[0], row0 = wk[1], pos0 = wk[3], kv_start = wk[4], piece = wk[6], n_pieces = wk[7];
+  const int kv_end = min(wk[5], pos0 + (row0 + n_rows - 1) / p.H + 1);
+  const int n_tiles = kv_end > kv_start ? (kv_end - kv_start + kLatKeys - 1) / kLatKeys : 0;
+  const int bs = p.block_size;
+
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    for (int s = 0; s < p.slots; ++s) {
+      mbar_init(c_full(s), 1);
+      mbar_init(c_empty(s), 1);
+    }
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(s_full(s), 1);
+      mbar_init(s_empty(s), 4);
+      mbar_init(p_full(s), 4);
+      mbar_init(o_full(s), 1);
+      rescale_s[s] = 0;
+    }
+    abort_s = 0;
+    fence_barrier_init();
+    prefetch_tensormap(&tmap_q);
+    prefetch_tensormap(&tmap_c);
+  }
+  for (int i = threadIdx.x; i < NR; i += kLatThreads) {
+    m_s[i] = -INFINITY;
+    lim_s[i] = min(pos0 + (row0 + i) / p.H, kv_end - 1);
+  }
+  if (warp == 5) {
+    tmem_alloc(smem_u32(&tmem_slot), p.tmem_cols);
+    tmem_relinquish();
+  }
+  // Keys past the end of the last tile are never loaded and meet P = 0: what lies there must be
+  // finite. A slot that an earlier tile has filled is; the others are cleared.
+  if (n_tiles > 0) {
+    const int nkeys = kv_end - kv_start - (n_tiles - 1) * kLatKeys;
+    const int r_first = (nkeys + bs - 1) / bs * bs;
+    if (r_first < kLatKeys) {
+      const int vecs = (kLatKeys - r_first) * 8;
+      for (int c = 0; c < NC; ++c) {
+        const int idx = (n_tiles - 1) * NC + c;
+        if (idx >= p.slots) break;
+        uint4* z = reinterpret_cast<uint4*>(pC + (size_t)idx * kPieceBytes + (size_t)r_first * 128);
+        for (int i = threadIdx.x; i < vecs; i += kLatThreads) z[i] = make_uint4(0, 0, 0, 0);
+      }
+    }
+  }
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  pdl_wait();
+  const uint32_t tS = tmem_slot;                 // S buffers at columns 0, NR
+  const uint32_t tO = tmem_slot + 2 * NR;        // R / 128 blocks of NR columns
+
+  if (warp == 4) {
+    // ------------------------------ TMA producer ------------------------------
+    if (n_tiles > 0) {
+      if (lane == 0) {
+        mbar_arrive_expect_tx(q_full, (uint32_t)NC * NR * 128u);
+        for (int c = 0; c < NC; ++c)
+          tma_load_2d(sQ + (uint32_t)c * NR * 128u, &tmap_q, q_full, c * 64, row0);
+      }
+      const int* bt = p.block_tables + (long long)seq * p.max_blocks;
+      bool ok = true;
+      int slot = 0;
+      uint32_t ph = 0;
+      int issued = 0;
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        const int key0 = kv_start + j * kLatKeys;
+        const int nblk = (min(kLatKeys, kv_end - key0) + bs - 1) / bs;
+        const int bid = lane < nblk ? bt[key0 / bs + lane] : 0;
+        for (int c = 0; c < NC; ++c) {
+          if (!__all_sync(0xffffffffu, mbar_wait(c_empty(slot), ph ^ 1u, &abort_s, p.status,
+                                                 1500 + slot, j))) {
+            ok = false;
+            break;
+          }
+          if (lane == 0) mbar_arrive_expect_tx(c_full(slot), (uint32_t)(nblk * bs) * 128u);
+          __syncwarp();
+          if (lane < nblk)
+            tma_load_2d(sC + (uint32_t)slot * kPieceBytes + (uint32_t)(lane * bs) * 128u, &tmap_c,
+                        c_full(slot), c * 64, bid * bs);
+          __syncwarp();
+          ++issued;
+          if (++slot == p.slots) {
+            slot = 0;
+            ph ^= 1u;
+          }
+        }
+      }
+      if (!ok) {   // unwinding: give copies that were already issued a short time to land
+        for (int i = 0; i < min(issued, p.slots); ++i) {
+          if (--slot < 0) {
+            slot = p.slots - 1;
+            ph ^= 1u;
+          }
+          mbar_drain(c_full(slot), ph);
+        }
+        mbar_drain(q_full, 0);
+      }
+    }
+  } else if (warp == 5) {
+    // ------------------------------- MMA issuer -------------------------------
+    if (lane == 0 && n_tiles > 0) {
+      const uint32_t idesc_s = make_idesc(128, NR, 1, 1, 0, 0);
+      const uint32_t idesc_o = make_idesc(128, NR, 1, 1, 1, 0);
+      bool ok = mbar_wait(q_full, 0, &abort_s, p.status, 1600, 0);
+      auto issue_s = [&](int j) -> bool {
+        const int st = j & 1;
+        if (!mbar_wait(s_empty(st), ((uint32_t)(j >> 1) & 1u) ^ 1u, &abort_s, p.status, 1620 + st, j))
+          return false;
+        int idx = j * NC;
+        for (int c = 0; c < NC; ++c, ++idx) {
+          const int slot = idx % p.slots;
+          if (!mbar_wait(c_full(slot), (uint32_t)(idx / p.slots) & 1u, &abort_s, p.status,
+                         1610 + slot, j))
+            return false;
+          tc_fence_after();
+          const uint64_t cd = make_desc_kmajor_sw128(sC + (uint32_t)slot * kPieceBytes);
+          const uint64_t qd = make_desc_kmajor_sw128(sQ + (uint32_t)c * NR * 128u);
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            umma_f16_ss(tS + (uint32_t)st * NR, cd + (uint64_t)(2 * k), qd + (uint64_t)(2 * k),
+                        idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+        }
+        tc_commit(s_full(st));
+        return true;
+      };
+      auto issue_o = [&](int j) -> bool {
+        const int pb = p.p_bufs == 2 ? (j & 1) : 0;
+        const uint32_t pph = (uint32_t)(p.p_bufs == 2 ? (j >> 1) : j) & 1u;
+        if (!mbar_wait(p_full(pb), pph, &abort_s, p.status, 1640 + pb, j)) return false;
+        tc_fence_after();
+        const uint32_t pbase = sP + (uint32_t)pb * NR * 256u;
+        for (int rc = 0; rc < NC / 2; ++rc) {
+          // two neighbouring pieces (128 latent columns); a pair never wraps: slots is even
+          const int slot = (j * NC + 2 * rc) % p.slots;
+          const uint64_t cd =
+              make_desc_mnmajor_sw128(sC + (uint32_t)slot * kPieceBytes, kPieceBytes);
+#pragma unroll
+          for (int k = 0; k < kLatKeys / 16; ++k) {
+            const uint64_t pd = make_desc_kmajor_sw128(pbase + (uint32_t)(k / 4) * NR * 128u) +
+                                (uint64_t)(2 * (k % 4));
+            umma_f16_ss(tO + (uint32_t)(rc * NR), cd + (uint64_t)(128 * k), pd, idesc_o,
+                        (j > 0 || k > 0) ? 1u : 0u);
+          }
+          tc_commit(c_empty(slot));
+          tc_commit(c_empty(slot + 1));
+        }
+        tc_commit(o_full(j & 1));
+        return true;
+      };
+      if (ok) ok = issue_s(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        if (p.overlap && j + 1 < n_tiles) ok = issue_s(j + 1);
+        if (ok) ok = issue_o(j);
+        if (ok && !p.overlap && j + 1 < n_tiles) ok = issue_s(j + 1);
+      }
+    }
+  } else {
+    // ------------------------------ softmax warps ------------------------------
+    // A wait that runs out leaves `ok` false; the warp then only keeps the barriers going (every
+    // loop has the same trip count in all four warps), so that nobody waits for it.
+    const int tid = threadIdx.x;     // key of the tile, TMEM lane
+    const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
+    const float sc = p.scale_log2;
+    const int my_col = reduce16_index(lane);
+    float l[NR];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) l[i] = 0.f;
+    bool ok = true;
+    const int min_lim = pos0 + row0 / p.H;
+    for (int j = 0; j < n_tiles; ++j) {
+      const int st = j & 1;
+      const int key0 = kv_start + j * kLatKeys;
+      const int key = key0 + tid;
+      const bool need_mask = key0 + kLatKeys - 1 > min(min_lim, kv_end - 1);
+      ok = __all_sync(0xffffffffu, ok && mbar_wait(s_full(st), (uint32_t)(j >> 1) & 1u, &abort_s,
+                                                   p.status, 1700 + st, j));
+      tc_fence_after();
+      const uint32_t ts = tS + (uint32_t)st * NR + lane_off;
+      if (ok) {
+#pragma unroll
+        for (int g = 0; g < NR / 16; ++g) {
+          uint32_t r[16];
+          tmem_ld_x16(ts + 16u * g, r);
+          tmem_ld_wait_dep16(r);
+          float v[16];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            v[i] = __uint_as_float(r[i]);
+            if (need_mask && key > lim_s[16 * g + i]) v[i] = -INFINITY;
+          }
+          const float mx = reduce16<true>(v, lane);
+          if ((lane & 1) == 0) wred[(16 * g + my_col) * 4 + warp] = mx;
+        }
+      }
+      bar_softmax();
+      if (tid < NR) {
+        const float4 q = *reinterpret_cast<const float4*>(&wred[tid * 4]);
+        const float m_old = m_s[tid];
+        const float m_new = fmaxf(m_old, fmaxf(fmaxf(q.x, q.y), fmaxf(q.z, q.w)));
+        const float m_safe = m_new == -INFINITY ? 0.f : m_new;
+        // a row that has seen no key yet holds O = 0 and l = 0: nothing to rescale
+        const float alpha = m_old == -INFINITY ? 1.f : ex2_approx((m_old - m_safe) * sc);
+        m_s[tid] = m_new;
+        neg_s[tid] = -m_safe * sc;
+        alpha_s[tid] = alpha;
+        if (alpha != 1.f) rescale_s[st] = 1;
+      }
+      if (tid == 127) rescale_s[st ^ 1] = 0;
+      bar_softmax();
+      const bool rescale = j > 0 && *reinterpret_cast<volatile int*>(&rescale_s[st]) != 0;
+      // A rescale must not race with O(j-1) accumulating, and P(j) overwrites the buffer that
+      // O(j - p_bufs) reads
+      const int jw = (rescale || p.p_bufs == 1) ? j - 1 : j - 2;
+      if (jw >= 0)
+        ok = __all_sync(0xffffffffu, ok && mbar_wait(o_full(jw & 1), (uint32_t)(jw >> 1) & 1u,
+                                                     &abort_s, p.status, 1710, j));
+      if (rescale && ok) {
+        tc_fence_after();
+#pragma unroll
+        for (int i = 0; i < NR; i += 4) {
+          const float4 a = *reinterpret_cast<const float4*>(&alpha_s[i]);
+          l[i] *= a.x; l[i + 1] *= a.y; l[i + 2] *= a.z; l[i + 3] *= a.w;
+        }
+        for (int rc = 0; rc < NC / 2; ++rc) {
+#pragma unroll
+          for (int g = 0; g < NR / 16; ++g) {
+            uint32_t r[16];
+            const uint32_t to = tO + (uint32_t)(rc * NR + 16 * g) + lane_off;
+            tmem_ld_x16(to, r);
+            tmem_ld_wait_dep16(r);
+#pragma unroll
+            for (int i = 0; i < 16; ++i)
+              r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha_s[16 * g + i]);
+            tmem_st_x16(to, r);
+          }
+        }
+        tmem_st_wait();
+      }
+      if (ok) {
+        const int pb = p.p_bufs == 2 ? st : 0;
+        uint8_t* prow = pP + (size_t)pb * NR * 256 + (size_t)(tid >> 6) * NR * 128 + (tid & 7) * 2;
+        const int chunk = (tid & 63) >> 3;
+#pragma unroll
+        for (int g = 0; g < NR / 16; ++g) {
+          uint32_t r[16];
+          tmem_ld_x16(ts + 16u * g, r);
+          tmem_ld_wait_dep16(r);
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int n = 16 * g + i;
+            float e = ex2_approx(fmaf(__uint_as_float(r[i]), sc, neg_s[n]));
+            if (need_mask && key > lim_s[n]) e = 0.f;
+            l[n] += e;
+            *reinterpret_cast<__nv_bfloat16*>(prow + n * 128 + ((chunk ^ (n & 7)) << 4)) =
+                __float2bfloat16(e);
+          }
+        }
+      }
+      tc_fence_before();
+      fence_proxy_async_smem();
+      __syncwarp();
+      if (lane == 0) {
+        mbar_arrive(s_empty(st));
+        mbar_arrive(p_full(p.p_bufs == 2 ? st : 0));
+      }
+    }
+    // row sums over the keys, normalisation factors, log-sum-exp
+#pragma unroll
+    for (int g = 0; g < NR / 16; ++g) {
+      float v[16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) v[i] = l[16 * g + i];
+      const float s = reduce16<false>(v, lane);
+      if ((lane & 1) == 0) wred[(16 * g + my_col) * 4 + warp] = s;
+    }
+    bar_softmax();
+    if (tid < NR) {
+      const float4 q = *reinterpret_cast<const float4*>(&wred[tid * 4]);
+      const float sum = (q.x + q.y) + (q.z + q.w);
+      inv_s[tid] = sum > 0.f ? 1.f / sum : 0.f;
+      if (n_pieces > 1 && tid < n_rows)
+        p.lse_part[(long long)piece * p.rows_total + row0 + tid] =
+            sum > 0.f ? m_s[tid] * p.scale + logf(sum) : -INFINITY;
+    }
+    bar_softmax();
+    if (n_tiles > 0) {
+      const int jl = n_tiles - 1;
+      ok = __all_sync(0xffffffffu, ok && mbar_wait(o_full(jl & 1), (uint32_t)(jl >> 1) & 1u, &abort_s,
+                                                   p.status, 1720, jl));
+      tc_fence_after();
+    }
+    const int R = NC * 64;
+    if (ok) {
+      for (int rc = 0; rc < NC / 2; ++rc) {
+        const int col = rc * 128 + tid;
+#pragma unroll
+        for (int g = 0; g < NR / 16; ++g) {
+          uint32_t r[16];
+          if (n_tiles > 0) {
+            tmem_ld_x16(tO + (uint32_t)(rc * NR + 16 * g) + lane_off, r);
+            tmem_ld_wait_dep16(r);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) r[i] = 0u;
+          }
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int n = 16 * g + i;
+            if (n < n_rows) {
+              const float v = __uint_as_float(r[i]) * inv_s[n];
+              if (n_pieces > 1)
+                p.o_part[((long long)piece * p.rows_total + row0 + n) * R + col] = v;
+              else
+                p.out[(long long)(row0 + n) * R + col] = __float2bfloat16(v);
+            }
+          }
+        }
+      }
+    }
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 5) {
+    tc_fence_after();
+    tmem_dealloc(tmem_slot, p.tmem_cols);
+  }
+}
+
+template <int NR>
+static int launch_latent(const CUtensorMap& tq, const CUtensorMap& tc, LatentArgs a, int num_work,
+                         cudaStream_t stream) {
+  const int NC = a.pieces;
+  const size_t limit = 227 * 1024 - 4096;   // static shared memory and alignment aside
+  const size_t q_bytes = (size_t)NC * NR * 128;
+  a.p_bufs = 2;
+  auto fit = [&](int pb) {
+    int s = (int)((limit - q_bytes - (size_t)pb * NR * 256) / kPieceBytes) & ~1;
+    return s > kLatMaxSlots ? kLatMaxSlots : s;
+  };
+  a.slots = fit(2);
+  if (a.slots < NC + 2 && fit(1) > a.slots) {
+    a.p_bufs = 1;
+    a.slots = fit(1);
+  }
+  if (a.slots < NC) return -6;
+  a.overlap = a.slots >= 2 * NC;
+  a.tmem_cols = 32;
+  while (a.tmem_cols < (uint32_t)((2 + NC / 2) * NR)) a.tmem_cols <<= 1;
+  const size_t smem = q_bytes + (size_t)a.slots * kPieceBytes + (size_t)a.p_bufs * NR * 256 + 1024;
+  static bool attr_set[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return -3;
+  if (!attr_set[dev]) {
+    if (cudaFuncSetAttribute(latent_attention_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             224 * 1024) != cudaSuccess)
+      return -3;
+    attr_set[dev] = true;
+  }
+  return launch_pdl(latent_attention_kernel<NR>, dim3((unsigned)num_work), dim3(kLatThreads), smem,
+                    stream, tq, tc, a) == cudaSuccess
+             ? 0
+             : -5;
+}
+
+}  // namespace ab200
+
+using namespace ab200;
+
+extern "C" {
+
+// q and out: bf16 [T * H, R] contiguous; cache [num_blocks, block_size, R]; R a multiple of 128 up
+// to 512; tile_rows 16, 32, 48 or 64, the rows per work item.
+int ab200_latent_attention(const void* q, long long q_rows, const void* cache, int num_blocks,
+                           int block_size, const void* block_tables, int max_blocks,
+                           const void* work, int num_work, const void* tok_splits, int max_splits,
+                           long long T, int H, int R, int tile_rows, float scale, void* out,
+                           void* o_part, void* lse_part, int* status, cudaStream_t stream) {
+  if (num_work <= 0 || T <= 0) return 0;
+  if (R % 128 || R < 128 || R > 512 || H <= 0 || q_rows != T * H) return -2;
+  if (block_size < 8 || block_size > kLatKeys || kLatKeys % block_size) return -2;
+  if (T * H > 0x7fffffffll || (long long)num_blocks * block_size > 0x7fffffffll) return -6;
+  if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
+  CUtensorMap tq, tc;
+  if (make_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)q_rows, (uint64_t)R,
+                   (uint64_t)R * 2, (uint32_t)tile_rows, 64) != 0)
+    return -4;
+  if (make_tmap_2d(&tc, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)num_blocks * block_size,
+                   (uint64_t)R, (uint64_t)R * 2, (uint32_t)block_size, 64) != 0)
+    return -4;
+  LatentArgs a;
+  memset(&a, 0, sizeof(a));
+  a.work = reinterpret_cast<const int*>(work);
+  a.block_tables = reinterpret_cast<const int*>(block_tables);
+  a.max_blocks = max_blocks;
+  a.block_size = block_size;
+  a.H = H;
+  a.pieces = R / 64;
+  a.scale = scale;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.out = reinterpret_cast<__nv_bfloat16*>(out);
+  a.o_part = reinterpret_cast<float*>(o_part);
+  a.lse_part = reinterpret_cast<float*>(lse_part);
+  a.rows_total = q_rows;
+  a.status = status;
+  int rc;
+  switch (tile_rows) {
+    case 16: rc = launch_latent<16>(tq, tc, a, num_work, stream); break;
+    case 32: rc = launch_latent<32>(tq, tc, a, num_work, stream); break;
+    case 48: rc = launch_latent<48>(tq, tc, a, num_work, stream); break;
+    case 64: rc = launch_latent<64>(tq, tc, a, num_work, stream); break;
+    default: return -2;
+  }
+  if (rc != 0 || max_splits <= 1) return rc;
+  return ab200_attention_merge(o_part, lse_part, tok_splits, T, H, R, out, (long long)H * R, stream);
+}
+
+}  // extern "C"

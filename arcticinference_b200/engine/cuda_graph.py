@@ -6,8 +6,8 @@ launch-bound (about ten kernels per layer), so the whole forward pass + LM head 
 arg-max is captured once per (mode, padded token count) and replayed.
 
 Static shapes: token count padded to a bucket; block table ``[bucket,
-max_blocks_per_seq]``; attention work list ``[bucket * splits, 8]`` whose unused
-entries are no-ops; split-KV scratch sized for ``splits``. Per step only the
+max_blocks_per_seq]``; per kind of attention call a work list whose unused entries are
+no-ops and split-KV scratch (``ops.DecodePlan``, made by the model). Per step only the
 contents of those buffers change (two pinned-to-device copies).
 
 Bucket tables follow the reference's dual tables
@@ -45,35 +45,22 @@ class DecodeGraph:
         dev = runner.device
         cfg = runner.config
         self.max_blocks = (cfg.scheduler.max_model_len + runner.block_size - 1) // runner.block_size
-        hkv = m.hkv
-        # enough KV splits to occupy the GPU when the batch is small; for a large batch the
-        # sequences of the last, partly filled wave of CTAs are cut (ops.tail_split_plan)
         max_q = 1 + (cfg.speculative.max_draft_tokens if cfg.speculative else 0)
-        small_tiles = max_q * runner.G <= 32 and runner.block_size <= 64
-        self.splits = int(max(1, min(16, 148 // max(1, bucket * hkv))))
-        self.work_cap = bucket * self.splits + 1
-        n_cut, pieces = ops.tail_split_plan(bucket, hkv, 148 * (2 if small_tiles else 1))
-        if self.splits == 1 and n_cut > 0 and max_q == 1:
-            self.splits = pieces
-            self.work_cap = bucket + n_cut * (pieces - 1) + 1
+        self.plans = m.decode_plans(bucket, max_q, runner.block_size)
         n64 = 4 * bucket      # ids | positions | slots | source rows of run-ahead tokens
-        n32 = bucket * self.max_blocks + self.work_cap * 8 + bucket
+        n32 = bucket * self.max_blocks + sum(p.int32_words for p in self.plans)
         pin = dev.type == "cuda"
         self.h64 = torch.zeros(n64, dtype=torch.int64, pin_memory=pin)
         self.h32 = torch.zeros(n32, dtype=torch.int32, pin_memory=pin)
         self.d64 = torch.zeros(n64, dtype=torch.int64, device=dev)
         self.d32 = torch.zeros(n32, dtype=torch.int32, device=dev)
         B, MB = bucket, self.max_blocks
-        self.meta = ops.AttentionMetadata([], [], bucket)
-        self.meta.block_tables = self.d32[:B * MB].view(B, MB)
-        self.meta.work = self.d32[B * MB:B * MB + self.work_cap * 8].view(self.work_cap, 8)
-        self.meta.tok_splits = self.d32[B * MB + self.work_cap * 8:]
-        self.meta.num_work = self.work_cap
-        self.meta.max_splits = self.splits
-        self.meta.tile_keys = 64 if small_tiles else 128
-        if self.splits > 1:
-            self.meta.o_part = torch.empty(self.splits, B, m.h, m.D, dtype=torch.float32, device=dev)
-            self.meta.lse_part = torch.empty(self.splits, B, m.h, dtype=torch.float32, device=dev)
+        bt = self.d32[:B * MB].view(B, MB)
+        h32, off = self.h32.numpy(), B * MB
+        for p in self.plans:
+            p.bind(h32[off:off + p.int32_words], self.d32[off:off + p.int32_words], bt)
+            off += p.int32_words
+        self.meta = m.decode_attention(self.plans, bt)
         self.logits_indices = torch.arange(bucket, dtype=torch.int64, device=dev)
         self.batch = ForwardBatch(input_ids=self.d64[:B], positions=self.d64[B:2 * B],
                                   slots=self.d64[2 * B:3 * B], attn_meta=self.meta,
@@ -109,8 +96,6 @@ class DecodeGraph:
         if src_rows is not None:
             src[:len(src_rows)] = src_rows
         bt = h32[:B * MB].reshape(B, MB)
-        work = h32[B * MB:B * MB + self.work_cap * 8].reshape(self.work_cap, 8)
-        tok_splits = h32[B * MB + self.work_cap * 8:]
         from .model_runner import pack_tokens
         q_lens, kv_lens, offs = pack_tokens(out.scheduled, bs, ids, pos, slots, bt)
         rows = [[t] if n == 1 else list(range(t, t + n)) for t, n in zip(offs, q_lens)]
@@ -123,12 +108,8 @@ class DecodeGraph:
             bt[len(q_lens), :] = 0
             q_lens.append(B - N)
             kv_lens.append(B - N)
-        w, ts, _ = ops.plan_attention_work(q_lens, kv_lens, r.G, True, Hkv=r.model.hkv,
-                                           max_splits_cap=self.splits)
-        assert w.shape[0] <= self.work_cap
-        work[:w.shape[0]] = w
-        work[w.shape[0]:] = 0
-        tok_splits[:B] = ts[:B]
+        for p in self.plans:
+            p.fill(q_lens, kv_lens)
         return rows
 
     def upload(self) -> None:

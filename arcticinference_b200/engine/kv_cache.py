@@ -224,3 +224,26 @@ class KVCacheTensors:
     def free(self) -> None:
         self.k, self.v = [], []
         self._tables = {}
+
+
+class LatentCacheTensors:
+    """Device memory of a latent cache: one tensor ``[num_blocks, 1, block_size, width]`` per
+    layer that projects latents of its own. A layer that takes an earlier layer's latents has
+    that layer's tensor (``k[l]`` is the same object), so it costs no memory. The block tables,
+    prefix cache and scheduler above it are those of any other model."""
+
+    def __init__(self, owners: list, widths: list, num_blocks: int, block_size: int,
+                 dtype: torch.dtype, device):
+        """``owners[l]``: the layer whose latents layer l reads; ``widths[l]``: columns of a row."""
+        self.k = []
+        for l, o in enumerate(owners):
+            self.k.append(self.k[o] if o != l else torch.zeros(
+                (num_blocks, 1, block_size, widths[l]), dtype=dtype, device=device))
+
+    @staticmethod
+    def bytes_per_block(owners: list, widths: list, block_size: int, elem_bytes: int) -> int:
+        return sum(w for l, (o, w) in enumerate(zip(owners, widths)) if o == l) * \
+            block_size * elem_bytes
+
+    def free(self) -> None:
+        self.k = []

@@ -24,9 +24,9 @@ import torch
 
 from .. import ops
 from ..config import EngineConfig
-from ..models.llama import ForwardBatch, LlamaForCausalLM, ShardSpec
+from ..models.llama import ForwardBatch, ShardSpec
+from ..plugin import model_class
 from ..utils.tracing import trace_range
-from .kv_cache import KVCacheTensors
 from .sampler import row_seed
 from .scheduler import SchedulerOutput
 
@@ -118,12 +118,12 @@ class ModelRunner:
         self.comm = comm
         self.shard = shard or ShardSpec()
         mcfg = config.model
-        self.model = LlamaForCausalLM(mcfg, self.shard, self.device, torch.bfloat16, comm=comm)
+        self.model = model_class(mcfg)(mcfg, self.shard, self.device, comm=comm)
         # a pipeline stage (parallel/pipeline.py): the communicator is then the stage's handle
         self.pp = comm if getattr(comm, "stages", 1) > 1 else None
         if self.pp is not None:
             self.model.set_pipeline(self.pp)
-        self.kv: Optional[KVCacheTensors] = None
+        self.kv = None                # the model's cache tensors (engine/kv_cache.py)
         self.num_blocks = 0
         self.block_size = config.cache.block_size
         self.sp = config.parallel.sp
@@ -160,8 +160,7 @@ class ModelRunner:
                                                      fromlist=["PRESETS"]).PRESETS:
             self.model.init_random(cfg.seed)
         else:
-            from ..models.loader import load_llama_weights
-            load_llama_weights(self.model, cfg.model.name_or_path)
+            self.model.load_weights(cfg.model.name_or_path)
         if cfg.model.quantization == "fp8":
             from ..models.quant import quantize_model_fp8
             quantize_model_fp8(self.model, scheme=cfg.model.fp8_scheme)
@@ -171,9 +170,7 @@ class ModelRunner:
 
     def determine_num_blocks(self) -> int:
         cfg = self.config
-        m = self.model
-        per_block = KVCacheTensors.bytes_per_block(m.layer_hi - m.layer_lo, m.hkv,
-                                                   self.block_size, m.D)
+        per_block = self.model.kv_bytes_per_block(self.block_size)
         if cfg.cache.num_gpu_blocks is not None:
             return cfg.cache.num_gpu_blocks
         if self.device.type != "cuda":
@@ -191,11 +188,8 @@ class ModelRunner:
         return int(min(n, 1 << 22))
 
     def init_kv_cache(self, num_blocks: int) -> None:
-        m = self.model
         self.num_blocks = num_blocks
-        self.kv = KVCacheTensors(self.config.model.num_hidden_layers, num_blocks, m.hkv,
-                                 self.block_size, m.D, torch.bfloat16, self.device,
-                                 layers=range(m.layer_lo, m.layer_hi) if self.pp else None)
+        self.kv = self.model.new_kv_cache(num_blocks, self.block_size)
 
     # ------------------------------------------------------------- mode choice
     def choose_mode(self, total_tokens: int) -> str:
@@ -247,9 +241,15 @@ class ModelRunner:
                     sched = [sched[i] for i in plan.order]
                     out.scheduled = sched
                     self.cascade_steps += 1
+        order = self.model.batch_order([s.num_tokens for s in sched],
+                                       [s.start + s.num_tokens for s in sched])
+        if order is not None:
+            sched = [sched[i] for i in order]
+            out.scheduled = sched
         pad_to = self.sp if mode == "sp" else 1
         Np = (N + pad_to - 1) // pad_to * pad_to
-        n_smp = sum((s.num_draft + 1) if s.samples else 0 for s in sched)
+        n_smp = sum(len(s.want) if s.want is not None else
+                    (s.num_draft + 1) if s.samples else 0 for s in sched)
         # prompt log-probabilities: every prompt position of the chunk whose successor is a
         # prompt token is scored too; those rows follow the sampled rows
         prompt_spans = []       # (request, first position, count)
@@ -272,7 +272,14 @@ class ModelRunner:
         rows = []
         sel_q_lens = []
         for s, t in zip(sched, offs):
-            if s.samples:
+            if s.want is not None:
+                m = len(s.want)
+                at = np.asarray(s.want, dtype=np.int64)
+                sel[k:k + m], sel_pos[k:k + m] = t + at, s.start + at
+                rows.append(list(range(k, k + m)))
+                sel_q_lens.append(m)
+                k += m
+            elif s.samples:
                 m = s.num_draft + 1
                 last = t + s.num_tokens
                 if m == 1:
@@ -332,11 +339,10 @@ class ModelRunner:
             meta.o_part = torch.empty(max_splits, N, m.h, m.D, dtype=torch.float32, device=dev)
             meta.lse_part = torch.empty(max_splits, N, m.h, dtype=torch.float32, device=dev)
         else:
-            meta = ops.build_attention_metadata(q_lens_a, kv_lens_a, bt_t, self.G, m.h, m.D, dev,
-                                                Hkv=m.hkv)
+            meta = m.plan_attention(q_lens_a, kv_lens_a, bt_t,
+                                    [s.request.block_array() for s in sched], bs)
         # the attention work list and split table are uploaded too
-        extra = sum(t.numel() * t.element_size() for t in (meta.work, meta.tok_splits)
-                    if t is not None)
+        extra = meta.uploaded_bytes
         self.h2d_bytes += extra
         self.h2d_total += extra
         batch = ForwardBatch(input_ids=d[:Np], positions=d[Np:2 * Np], slots=d[2 * Np:3 * Np],
@@ -406,7 +412,8 @@ class ModelRunner:
 
     def _decode_graph(self, out: SchedulerOutput):
         """The captured graph for this step, or None when the step must run eagerly."""
-        if self.config.enforce_eager or self.device.type != "cuda" or self.pp is not None:
+        if self.config.enforce_eager or self.device.type != "cuda" or self.pp is not None or \
+                not self.model.supports_graphs:
             return None      # (a pipeline stage's step contains point-to-point transfers)
         fc = self.config.forest_cascade
         if fc.enabled and len(out.scheduled) >= fc.min_batch_size:
@@ -540,6 +547,32 @@ class ModelRunner:
             if prompt_lp is not None:
                 pend.prompt_logprobs = (prompt_lp, batch.prompt_rows)
         return self._after_launch(pend, out, rows, input_sel)
+
+    @torch.inference_mode()
+    def score(self, out: SchedulerOutput) -> Optional[torch.Tensor]:
+        """Run a step for its logits at the places ``ScheduledRequest.want`` names: [wanted, V] in
+        the order of ``out.scheduled`` as given, None when nothing is wanted. The batch, the
+        kernels and the captured decode steps are those of ``launch``."""
+        given = list(out.scheduled)
+        g = self._decode_graph(out)
+        if g is not None:
+            g.wait_uploaded()
+            rows = g.fill(out)
+            self.mode_counts[g.mode] += 1
+            self.graph_replays += 1
+            _, hidden = g.replay()
+            rows = [[rr[k] for k in s.want] for s, rr in zip(out.scheduled, rows)]
+        else:
+            batch, rows = self.prepare(out)
+            self.mode_counts[batch.mode] += 1
+            hidden = self.model.forward(batch, self.kv)
+        of = {id(s): rr for s, rr in zip(out.scheduled, rows)}
+        idx = [j for s in given for j in of[id(s)]]
+        if not idx:
+            return None
+        if idx != list(range(hidden.shape[0])):
+            hidden = hidden[ops.upload(np.asarray(idx, dtype=np.int64), self.device)]
+        return self.model.compute_logits(hidden, fp32=self.config.fp32_lm_head)
 
     def _after_launch(self, pend, out, rows, input_sel=None):
         """Start the step's tokens on their way to the host (and, with a speculator, verify

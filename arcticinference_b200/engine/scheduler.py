@@ -35,6 +35,8 @@ class ScheduledRequest:
     num_tokens: int       # tokens fed to the model (including draft tokens)
     num_draft: int        # trailing draft tokens among them
     samples: bool         # True if the step produces a new token for this request
+    # places among the step's tokens whose logits are asked for, instead of sampling
+    want: Optional[list] = None
 
 
 @dataclass

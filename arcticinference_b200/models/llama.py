@@ -216,6 +216,43 @@ class LlamaModel:
         from .loader import load_llama_state, random_llama_state
         load_llama_state(self, random_llama_state(self.cfg, seed, std, self.device, self.dtype))
 
+    def load_weights(self, path: str) -> None:
+        from .loader import load_llama_weights
+        load_llama_weights(self, path)
+
+    # ------------------------------------------------- cache and attention planning
+    supports_graphs = True
+
+    def kv_bytes_per_block(self, block_size: int) -> int:
+        from ..engine.kv_cache import KVCacheTensors
+        return KVCacheTensors.bytes_per_block(self.layer_hi - self.layer_lo, self.hkv, block_size,
+                                              self.D)
+
+    def new_kv_cache(self, num_blocks: int, block_size: int):
+        from ..engine.kv_cache import KVCacheTensors
+        return KVCacheTensors(self.cfg.num_hidden_layers, num_blocks, self.hkv, block_size, self.D,
+                              self.dtype, self.device,
+                              layers=range(self.layer_lo, self.layer_hi) if self.pp else None)
+
+    def batch_order(self, q_lens, kv_lens):
+        """The order in which a step's requests are laid out (None: as scheduled)."""
+        return None
+
+    def plan_attention(self, q_lens, kv_lens, block_tables, block_arrays, block_size):
+        """The step's attention description, ``ForwardBatch.attn_meta``."""
+        return ops.build_attention_metadata(q_lens, kv_lens, block_tables, self.h // self.hkv,
+                                            self.h, self.D, self.device, Hkv=self.hkv)
+
+    def decode_plans(self, bucket: int, max_q: int, block_size: int) -> list:
+        """What a captured decode step of ``bucket`` tokens plans per step: one entry per kind
+        of attention call (this family has one)."""
+        return [ops.DecodePlan(self.h // self.hkv, self.h, self.hkv, self.D, bucket, max_q,
+                               block_size)]
+
+    def decode_attention(self, plans: list, block_tables):
+        """``attn_meta`` over the fixed buffers of a captured step."""
+        return plans[0].meta
+
     def num_parameters(self) -> int:
         n = self.embed.numel() + self.norm.numel()
         if self.lm_head is not self.embed:

@@ -373,6 +373,10 @@ def linear(x: torch.Tensor, w, bias=None, residual=None, act=None, out=None,
         return y
     nat = _native()
     L = nat.lib()
+    if x.dtype == torch.float32 or x.shape[1] % 8 or w.shape[0] % 8:
+        # a 32-bit model, or rows that are no multiple of 16 bytes
+        assert bias is None and residual is None and act is None and sync is None
+        return _linear_exact(x, w, out)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     assert x.dim() == 2 and w.dim() == 2 and x.stride(1) == 1 and w.stride(1) == 1
     M, K = x.shape
@@ -398,6 +402,23 @@ def linear(x: torch.Tensor, w, bias=None, residual=None, act=None, out=None,
         ws.data_ptr(), ws.numel(), force_splits, nat.status_buffer(x.device).data_ptr(),
         nat.stream_ptr())
     nat.check(rc, "linear_bf16 M=%d N=%d K=%d" % (M, N, K))
+    launch_counter.add(1)
+    return out
+
+
+def _linear_exact(x: torch.Tensor, w: torch.Tensor, out=None) -> torch.Tensor:
+    nat = _native()
+    assert x.dtype == w.dtype and x.dtype in (torch.bfloat16, torch.float32)
+    assert x.stride(1) == 1 and w.stride(1) == 1
+    (M, K), N = x.shape, w.shape[0]
+    if out is None:
+        out = torch.empty(M, N, dtype=x.dtype, device=x.device)
+    if M == 0:
+        return out
+    rc = nat.lib().ab200_linear_exact(
+        x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(0), 0, out.data_ptr(), out.stride(0), 0,
+        M, N, K, 1, None, None, 0, 0 if x.dtype == torch.bfloat16 else 1, nat.stream_ptr())
+    nat.check(rc, "linear_exact M=%d N=%d K=%d" % (M, N, K))
     launch_counter.add(1)
     return out
 
@@ -793,6 +814,11 @@ class AttentionMetadata:
     tile_keys: int = 128     # 64 for decode-shaped calls (few query rows per sequence)
     extra: dict = field(default_factory=dict)
 
+    @property
+    def uploaded_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in (self.work, self.tok_splits)
+                   if t is not None)
+
 
 def plan_attention_work(q_lens, kv_lens, G: int, causal: bool = True, num_sms: int = 148,
                         Hkv: int = 1, seq_rows=None, allow_split: bool = True,
@@ -936,6 +962,55 @@ def build_attention_metadata(q_lens, kv_lens, block_tables, G, Hq, D, device, ca
         meta.o_part = torch.empty(max_splits, T, Hq, D, dtype=torch.float32, device=dev)
         meta.lse_part = torch.empty(max_splits, T, Hq, dtype=torch.float32, device=dev)
     return meta
+
+
+class DecodePlan:
+    """Attention work of a captured decode step: sizes of the fixed buffers, and the filling of
+    them from the step's lengths. ``bind`` gives it its slices of the step's int32 buffers."""
+
+    def __init__(self, G: int, Hq: int, Hkv: int, D: int, bucket: int, max_q: int,
+                 block_size: int):
+        self.G, self.Hq, self.Hkv, self.D, self.bucket = G, Hq, Hkv, D, bucket
+        # enough KV splits to occupy the GPU when the batch is small; for a large batch the
+        # sequences of the last, partly filled wave of CTAs are cut (tail_split_plan)
+        small_tiles = max_q * G <= 32 and block_size <= 64
+        self.splits = int(max(1, min(16, 148 // max(1, bucket * Hkv))))
+        self.work_cap = bucket * self.splits + 1
+        n_cut, pieces = tail_split_plan(bucket, Hkv, 148 * (2 if small_tiles else 1))
+        if self.splits == 1 and n_cut > 0 and max_q == 1:
+            self.splits = pieces
+            self.work_cap = bucket + n_cut * (pieces - 1) + 1
+        self.tile_keys = 64 if small_tiles else 128
+        self.meta = AttentionMetadata([], [], bucket)
+
+    @property
+    def int32_words(self) -> int:
+        return self.work_cap * 8 + self.bucket
+
+    def plan(self, q_lens, kv_lens):
+        return plan_attention_work(q_lens, kv_lens, self.G, True, Hkv=self.Hkv,
+                                   max_splits_cap=self.splits)
+
+    def bind(self, host, dev: torch.Tensor, block_tables: torch.Tensor) -> None:
+        """``host`` (numpy) and ``dev``: this plan's ``int32_words`` of the staging buffers."""
+        n = self.work_cap * 8
+        self._work, self._tok_splits = host[:n].reshape(self.work_cap, 8), host[n:]
+        m = self.meta
+        m.block_tables = block_tables
+        m.work, m.tok_splits = dev[:n].view(self.work_cap, 8), dev[n:]
+        m.num_work, m.max_splits, m.tile_keys = self.work_cap, self.splits, self.tile_keys
+        if self.splits > 1:
+            m.o_part = torch.empty(self.splits, self.bucket, self.Hq, self.D, dtype=torch.float32,
+                                   device=dev.device)
+            m.lse_part = torch.empty(self.splits, self.bucket, self.Hq, dtype=torch.float32,
+                                     device=dev.device)
+
+    def fill(self, q_lens, kv_lens) -> None:
+        w, ts, _ = self.plan(q_lens, kv_lens)
+        assert w.shape[0] <= self.work_cap
+        self._work[:w.shape[0]] = w
+        self._work[w.shape[0]:] = 0
+        self._tok_splits[:self.bucket] = ts[:self.bucket]
 
 
 def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,

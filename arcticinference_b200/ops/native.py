@@ -52,11 +52,36 @@ class KernelTimeout(KernelError):
     """A bounded device-side wait ran out (barrier or peer flag)."""
 
 
-def lib() -> ctypes.CDLL:
+class _PartialLibrary:
+    """The kernels of one model, loaded without the rest of the library. An entry point outside
+    that set (another model in the same process) brings in the whole library then."""
+
+    def __init__(self, part: ctypes.CDLL):
+        self._part = part
+        self._full = None
+
+    def __getattr__(self, name):
+        try:
+            fn = getattr(self._part, name)
+        except AttributeError:
+            if self._full is None:
+                self._full = _build.load_kernels()
+                _declare(self._full)
+            fn = getattr(self._full, name)
+        setattr(self, name, fn)
+        return fn
+
+
+def lib():
     global _lib
     if _lib is None:
-        _lib = _build.load_kernels()
-        _declare(_lib)
+        part = _build.load_kernel_set()
+        if part is not None:
+            _declare(part)
+            _lib = _PartialLibrary(part)
+        else:
+            _lib = _build.load_kernels()
+            _declare(_lib)
     return _lib
 
 
@@ -98,6 +123,19 @@ def _declare(L: ctypes.CDLL) -> None:
         "ab200_mlp_spec_step": (I, [P, LL, P, P, F, P, P, P, LL, LL, I, F, I, P]),
         "ab200_sum_lstm": (I, [P, LL, P, I, P, F, P, LL, P, P, P, P, P, P, LL, LL, I, F, I, P]),
         "ab200_verify_greedy": (I, [P, P, P, P, I, I, P, P, P, P, P]),
+        "ab200_stream_embedding": (I, [P, P, P, P, LL, I, LL, I, P, P]),
+        "ab200_stream_norm": (I, [P, P, P, LL, P, P, I, P, F, F, P, P, LL, I, I, P]),
+        "ab200_latent_norm_cache": (I, [P, LL, P, I, I, F, P, P, LL, LL, I, P, P]),
+        "ab200_gated_act": (I, [P, P, LL, I, I, I, P]),
+        "ab200_linear_exact": (I, [P, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P]),
+        "ab200_latent_attention_exact": (I, [P, LL, P, I, I, P, I, P, P, P, LL, LL, I, I, F, I, P,
+                                             P]),
+        "ab200_moe_route": (I, [P, P, P, LL, I, I, I, P, P, I, P]),
+        "ab200_moe_plan": (I, [P, LL, I, P, P, P, P]),
+        "ab200_moe_permute": (I, [P, P, P, P, P, LL, I, I, I, P]),
+        "ab200_grouped_gemm": (I, [P, LL, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P, P]),
+        "ab200_latent_attention": (I, [P, LL, P, I, I, P, I, P, I, P, I, LL, I, I, I, F, P, P, P, P,
+                                       P]),
         "ab200_attention": (I, [P, LL, P, P, LL, LL, I, P, I, P, I, P, I, LL, I, I, I, I, F, P,
                                 LL, P, P, P, I, P, P]),
     }

@@ -1,0 +1,294 @@
+"""Ops of decoders with a 32-bit residual stream and of mixture-of-experts feed-forwards.
+
+CUDA tensors run ``csrc/stream.cu``, ``csrc/moe.cu``, ``csrc/grouped_gemm.cu`` and, where the
+tensor-core kernels do not apply (32-bit models, rows that are no multiple of 16 bytes),
+``csrc/exact.cu``. CPU tensors run the PyTorch restatements below.
+
+The stream is a pair: ``x`` fp32 [T, W] and ``act``, its rounding to the model's element type,
+which the projections read (the same tensor for a 32-bit model).
+"""
+
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+import torch.nn.functional as F
+
+from . import launch_counter
+
+GATE_BLOCK = 16       # gate / up rows alternate in blocks of this many (csrc/common/elem.cuh)
+ACT_CODE = {"silu": 1, "gelu_tanh": 2}
+TILE_ROWS = 128       # rows per tile of a grouped product
+
+
+def _nat():
+    from . import native
+    return native
+
+
+def dtype_code(dt: torch.dtype) -> int:
+    if dt == torch.bfloat16:
+        return 0
+    if dt == torch.float32:
+        return 1
+    raise TypeError("element type %s" % dt)
+
+
+def activation(name: str, z: torch.Tensor) -> torch.Tensor:
+    return F.silu(z) if name == "silu" else F.gelu(z, approximate="tanh")
+
+
+# ------------------------------------------------------------------------ residual stream
+def stream_embedding(ids: torch.Tensor, table: torch.Tensor):
+    """(x, act) of the token embeddings."""
+    if not table.is_cuda:
+        act = table[ids]
+        x = act.float()
+        return (x, x) if table.dtype == torch.float32 else (x, act)
+    nat = _nat()
+    T, W = ids.numel(), table.shape[1]
+    x = torch.empty(T, W, dtype=torch.float32, device=table.device)
+    act = x if table.dtype == torch.float32 else torch.empty(T, W, dtype=table.dtype,
+                                                             device=table.device)
+    rc = nat.lib().ab200_stream_embedding(
+        ids.data_ptr(), table.data_ptr(), x.data_ptr(), None if act is x else act.data_ptr(), T, W,
+        table.shape[0], dtype_code(table.dtype), nat.status_buffer(table.device).data_ptr(),
+        nat.stream_ptr())
+    nat.check(rc, "stream_embedding")
+    launch_counter.add(1)
+    return x, act
+
+
+def _scaled_norm_ref(s, weight, eps):
+    return s / torch.sqrt(s.pow(2).mean(-1, keepdim=True) + eps) * (1.0 + weight)
+
+
+def stream_norm(x, act, y, weight, alpha: float, eps: float, experts: "Routing" = None) -> None:
+    """In place: ``x <- norm(alpha * x + y) * (1 + weight)``, ``act`` its rounding. With
+    ``experts`` (a :class:`Routing`) ``y`` holds the experts' output rows and the sublayer's
+    output is each token's weighted sum of its own."""
+    T, W = x.shape
+    if not x.is_cuda:
+        yf = y.float()
+        if experts is not None:
+            yf = (yf[experts.rows.long()] * experts.weights.unsqueeze(-1)).sum(1)
+        x.copy_(_scaled_norm_ref(alpha * x + yf, weight, eps))
+        if act is not x:
+            act.copy_(x)
+        return
+    nat = _nat()
+    assert x.is_contiguous() and act.is_contiguous() and y.stride(1) == 1
+    rc = nat.lib().ab200_stream_norm(
+        x.data_ptr(), None, y.data_ptr(), y.stride(0),
+        experts.rows.data_ptr() if experts is not None else None,
+        experts.weights.data_ptr() if experts is not None else None,
+        experts.top if experts is not None else 0, weight.data_ptr(), float(alpha), float(eps),
+        x.data_ptr(), None if act is x else act.data_ptr(), T, W, dtype_code(act.dtype),
+        nat.stream_ptr())
+    nat.check(rc, "stream_norm")
+    launch_counter.add(1)
+
+
+def stream_final_norm(x, rows, weight, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """norm(x[rows]) * (1 + weight), rounded to ``dtype``: the state the LM head reads."""
+    R, W = rows.numel(), x.shape[1]
+    if not x.is_cuda:
+        return _scaled_norm_ref(x[rows], weight, eps).to(dtype)
+    nat = _nat()
+    out = torch.empty(R, W, dtype=dtype, device=x.device)
+    rc = nat.lib().ab200_stream_norm(x.data_ptr(), rows.data_ptr(), None, 0, None, None, 0,
+                                     weight.data_ptr(), 1.0, float(eps), None, out.data_ptr(), R, W,
+                                     dtype_code(dtype), nat.stream_ptr())
+    nat.check(rc, "stream_final_norm")
+    launch_counter.add(1)
+    return out
+
+
+# ------------------------------------------------------------------------ gated feed-forward
+def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """[.., ff, W] gate and up matrices -> [.., 2 * ff', W] with rows alternating in blocks of
+    GATE_BLOCK; ff is padded with zero rows to a multiple of it (they produce zeros)."""
+    *lead, ff, W = gate.shape
+    pad = -ff % GATE_BLOCK
+    if pad:
+        z = torch.zeros(*lead, pad, W, dtype=gate.dtype, device=gate.device)
+        gate, up = torch.cat([gate, z], -2), torch.cat([up, z], -2)
+    n = gate.shape[-2] // GATE_BLOCK
+    g = gate.reshape(*lead, n, GATE_BLOCK, W)
+    u = up.reshape(*lead, n, GATE_BLOCK, W)
+    return torch.stack([g, u], -3).reshape(*lead, 2 * n * GATE_BLOCK, W).contiguous()
+
+
+def _gated_ref(gu, act):
+    T, n2 = gu.shape
+    v = gu.float().reshape(T, n2 // (2 * GATE_BLOCK), 2, GATE_BLOCK)
+    return (activation(act, v[:, :, 0]) * v[:, :, 1]).reshape(T, n2 // 2).to(gu.dtype)
+
+
+def gated_act(gu: torch.Tensor, act: str) -> torch.Tensor:
+    """act(gate) * up of the product with an interleaved gate / up matrix."""
+    if not gu.is_cuda:
+        return _gated_ref(gu, act)
+    nat = _nat()
+    assert gu.is_contiguous()
+    T, ff = gu.shape[0], gu.shape[1] // 2
+    out = torch.empty(T, ff, dtype=gu.dtype, device=gu.device)
+    rc = nat.lib().ab200_gated_act(gu.data_ptr(), out.data_ptr(), T, ff, ACT_CODE[act],
+                                   dtype_code(gu.dtype), nat.stream_ptr())
+    nat.check(rc, "gated_act")
+    launch_counter.add(1)
+    return out
+
+
+# ------------------------------------------------------------------------ grouped products
+@dataclass
+class Routing:
+    """Which experts each token uses and where its rows lie among the rows sorted by expert."""
+    ids: torch.Tensor         # int32 [T, top]
+    weights: torch.Tensor     # fp32 [T, top]
+    rows: torch.Tensor        # int32 [T, top]
+    top: int
+    num_experts: int
+    tiles: torch.Tensor = None        # int32 [max_tiles, 4]: expert, first row, rows
+    num_tiles: torch.Tensor = None    # int32 [1]
+    counts: list = None               # CPU path: rows per expert
+
+
+def route_ref(x, w, b, top: int):
+    z = x.float() @ w.float().t() + b
+    order = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :top]
+    return order, torch.softmax(z.gather(1, order), -1)
+
+
+def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, top: int):
+    """Router of a mixture of experts. ``x`` fp32 [T, W] stream, ``act`` its rounding (what the
+    experts read), ``w`` [E, W], ``b`` fp32 [E]. Returns (Routing, act rows sorted by expert)."""
+    T, W = x.shape
+    E = w.shape[0]
+    if not x.is_cuda:
+        ids, weights = route_ref(x, w, b, top)
+        order = torch.argsort(ids.reshape(-1), stable=True)
+        rows = torch.empty_like(order)
+        rows[order] = torch.arange(order.numel())
+        counts = torch.bincount(ids.reshape(-1), minlength=E).tolist()
+        r = Routing(ids.int(), weights, rows.reshape(T, top).int(), top, E, counts=counts)
+        return r, act[order // top]
+    nat = _nat()
+    L, dev, dc = nat.lib(), x.device, dtype_code(act.dtype)
+    assert x.is_contiguous() and act.is_contiguous() and w.is_contiguous() and w.dtype == act.dtype
+    i32 = torch.int32
+    ids = torch.empty(T, top, dtype=i32, device=dev)
+    weights = torch.empty(T, top, dtype=torch.float32, device=dev)
+    rc = L.ab200_moe_route(x.data_ptr(), w.data_ptr(), b.data_ptr(), T, W, E, top, ids.data_ptr(),
+                           weights.data_ptr(), dc, nat.stream_ptr())
+    nat.check(rc, "moe_route")
+    launch_counter.add(1)
+    max_tiles = min(T * top, T * top // TILE_ROWS + E)
+    plan = torch.empty(E + 4 * max_tiles + 4 + T * top, dtype=i32, device=dev)
+    tiles = plan[:4 * max_tiles].view(max_tiles, 4)
+    num_tiles = plan[4 * max_tiles:4 * max_tiles + 1]
+    cursor = plan[4 * max_tiles + 4:4 * max_tiles + 4 + E]
+    rows = plan[4 * max_tiles + 4 + E:].view(T, top)
+    rc = L.ab200_moe_plan(ids.data_ptr(), T * top, E, cursor.data_ptr(), tiles.data_ptr(),
+                          num_tiles.data_ptr(), nat.stream_ptr())
+    nat.check(rc, "moe_plan")
+    launch_counter.add(1)
+    xp = torch.empty(T * top, W, dtype=act.dtype, device=dev)
+    rc = L.ab200_moe_permute(act.data_ptr(), ids.data_ptr(), cursor.data_ptr(), rows.data_ptr(),
+                             xp.data_ptr(), T, W, top, dc, nat.stream_ptr())
+    nat.check(rc, "moe_permute")
+    launch_counter.add(1)
+    return Routing(ids, weights, rows, top, E, tiles, num_tiles), xp
+
+
+def _aligned(*ts) -> bool:
+    """Rows of 16-bit elements that the tensor-map copies can fetch."""
+    for t in ts:
+        if t.dtype != torch.bfloat16 or t.data_ptr() % 16:
+            return False
+        if t.stride(-1) != 1 or any(s % 8 for s in t.stride()[:-1]):
+            return False
+    return True
+
+
+def grouped_linear(x: torch.Tensor, w: torch.Tensor, routing: Routing, act: str = None):
+    """Rows sorted by expert [n, K] times each row's expert matrix of ``w`` [E, N, K]. With
+    ``act`` the matrices are interleaved gate / up ones and the result is act(gate) * up."""
+    n, K = x.shape
+    E, N, _ = w.shape
+    if not x.is_cuda:
+        out = torch.cat([xe.float() @ w[e].float().t()
+                         for e, xe in enumerate(x.split(routing.counts))]).to(x.dtype)
+        return _gated_ref(out, act) if act else out
+    nat = _nat()
+    fused = act is not None and _aligned(x, w) and K % 8 == 0
+    out = torch.empty(n, N // 2 if fused else N, dtype=x.dtype, device=x.device)
+    if _aligned(x, w, out) and K % 8 == 0:
+        rc = nat.lib().ab200_grouped_gemm(
+            x.data_ptr(), x.stride(0), 0, n, w.data_ptr(), w.stride(1), w.stride(0),
+            out.data_ptr(), out.stride(0), 0, 0, N, K, E, routing.tiles.data_ptr(),
+            routing.num_tiles.data_ptr(), routing.tiles.shape[0], ACT_CODE[act] if act else 0,
+            nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
+        nat.check(rc, "grouped_gemm n=%d N=%d K=%d" % (n, N, K))
+        launch_counter.add(1)
+        return out
+    rc = nat.lib().ab200_linear_exact(
+        x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(1), w.stride(0), out.data_ptr(),
+        out.stride(0), 0, 0, N, K, E, routing.tiles.data_ptr(), routing.num_tiles.data_ptr(),
+        routing.tiles.shape[0], dtype_code(x.dtype), nat.stream_ptr())
+    nat.check(rc, "linear_exact (experts)")
+    launch_counter.add(1)
+    return gated_act(out, act) if act else out
+
+
+def gated_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
+    """act(gate) * up of a dense feed-forward: ``w`` [2 * ff, W] is an interleaved gate / up
+    matrix. Long inputs run one tensor-core kernel with the activation in its epilogue; short
+    ones the framework's decode GEMM (split over K) and a separate activation."""
+    from . import linear
+    T = x.shape[0]
+    if not x.is_cuda or T <= FUSED_GATE_MIN_TOKENS or not _aligned(x, w) or x.shape[1] % 8:
+        return gated_act(linear(x, w), act)
+    nat = _nat()
+    N, K = w.shape
+    out = torch.empty(T, N // 2, dtype=x.dtype, device=x.device)
+    rc = nat.lib().ab200_grouped_gemm(
+        x.data_ptr(), x.stride(0), 0, T, w.data_ptr(), w.stride(0), 0, out.data_ptr(),
+        out.stride(0), 0, T, N, K, 1, None, None, 0, ACT_CODE[act],
+        nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
+    nat.check(rc, "gated_linear M=%d N=%d K=%d" % (T, N, K))
+    launch_counter.add(1)
+    return out
+
+
+FUSED_GATE_MIN_TOKENS = 256
+
+
+def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor = None) -> torch.Tensor:
+    """One matrix per head: x [T, H * K] (row stride free), w [H, N, K] -> [T, H * N] with head h's
+    columns ``x_h @ w[h].T``."""
+    H, N, K = w.shape
+    T = x.shape[0]
+    if out is None:
+        out = torch.empty(T, H * N, dtype=x.dtype, device=x.device)
+    if not x.is_cuda:
+        y = torch.einsum("thk,hnk->thn", x.reshape(T, H, K).float(), w.float())
+        out.copy_(y.reshape(T, H * N))
+        return out
+    if T == 0:
+        return out
+    nat = _nat()
+    if _aligned(x, w, out) and K % 8 == 0 and N % 8 == 0:
+        rc = nat.lib().ab200_grouped_gemm(
+            x.data_ptr(), x.stride(0), K, T, w.data_ptr(), w.stride(1), w.stride(0),
+            out.data_ptr(), out.stride(0), N, T, N, K, H, None, None, 0, 0,
+            nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
+        nat.check(rc, "head_linear T=%d H=%d N=%d K=%d" % (T, H, N, K))
+    else:
+        rc = nat.lib().ab200_linear_exact(
+            x.data_ptr(), x.stride(0), K, w.data_ptr(), w.stride(1), w.stride(0), out.data_ptr(),
+            out.stride(0), N, T, N, K, H, None, None, 0, dtype_code(x.dtype), nat.stream_ptr())
+        nat.check(rc, "linear_exact (heads)")
+    launch_counter.add(1)
+    return out

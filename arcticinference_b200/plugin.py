@@ -35,6 +35,15 @@ def resolve_model(architecture: str) -> Callable:
     return _MODEL_REGISTRY[architecture]
 
 
+def model_class(cfg) -> Callable:
+    """Factory of a decoder's model class: by architecture name, else (a checkpoint under another
+    class name whose ``model_type`` is served) the Llama family's."""
+    _ensure_registered()
+    if cfg.architecture not in _MODEL_REGISTRY and cfg.layer_specs is None:
+        return _MODEL_REGISTRY["LlamaForCausalLM"]
+    return resolve_model(cfg.architecture)
+
+
 def supported_architectures() -> list[str]:
     _ensure_registered()
     return sorted(_MODEL_REGISTRY)
@@ -48,6 +57,10 @@ def _ensure_registered() -> None:
         from .models.llama import LlamaForCausalLM
         return LlamaForCausalLM(*a, **k)
 
+    def _taralix(*a, **k):
+        from .models.taralix import TaralixForCausalLM
+        return TaralixForCausalLM(*a, **k)
+
     def _speculator(*a, **k):
         from .models.speculator import build_speculator
         return build_speculator(*a, **k)
@@ -60,6 +73,9 @@ def _ensure_registered() -> None:
     for arch in ("LlamaForCausalLM", "LlamaSwiftKVForCausalLM", "MistralForCausalLM",
                  "Qwen2ForCausalLM", "Qwen3ForCausalLM"):
         register_model(arch, _llama)
+    register_config("taralix", "layer list: latent attention with shared latents, dense and "
+                               "mixture-of-experts feed-forwards")
+    register_model("Taralix", _taralix)
     for arch in ("ArcticMLPSpeculatorPreTrainedModel", "ArcticLSTMSpeculatorPreTrainedModel",
                  "MLPVariantSpeculatorPreTrainedModel", "MLPSpeculatorPreTrainedModel"):
         register_model(arch, _speculator)

@@ -51,8 +51,15 @@ def chat_token_ids(tokenizer, messages, add_generation_prompt: bool = True, **kw
     return [int(t) for t in out]
 
 
+# a directory with none of these holds no tokenizer (and importing transformers takes seconds)
+_TOKENIZER_FILES = ("tokenizer.json", "tokenizer_config.json", "tokenizer.model", "vocab.json",
+                    "vocab.txt", "merges.txt", "spiece.model", "sentencepiece.bpe.model",
+                    "added_tokens.json", "special_tokens_map.json")
+
+
 def get_tokenizer(name_or_path: Optional[str], vocab_size: int = 1024):
-    if name_or_path and os.path.isdir(name_or_path):
+    if name_or_path and os.path.isdir(name_or_path) and \
+            any(os.path.exists(os.path.join(name_or_path, f)) for f in _TOKENIZER_FILES):
         try:
             from transformers import AutoTokenizer
             return AutoTokenizer.from_pretrained(name_or_path)
