@@ -27,7 +27,8 @@ stream_embedding_kernel(const long long* __restrict__ ids, const T* __restrict__
   const long long t = blockIdx.x;
   const long long id = ids[t];
   const bool ok = id >= 0 && id < vocab;
-  if (!ok && threadIdx.x == 0) report_error(status, kErrBounds, 40, (int)t);
+  // (-1 stands for a token that is not known yet, when a decode step is captured)
+  if (id >= vocab && threadIdx.x == 0) report_error(status, kErrBounds, 40, (int)t);
   const T* src = table + (ok ? id : 0) * W;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     const T v = ok ? src[i] : from_f32<T>(0.f);

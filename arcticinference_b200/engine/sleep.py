@@ -16,7 +16,8 @@ import torch
 
 def _model_tensors(engine):
     m = engine.runner.model
-    items = [(m, "embed"), (m, "norm"), (m, "lm_head"), (m, "norm_swiftkv"), (m, "wkv_swiftkv")]
+    items = [(m, n) for n in ("embed", "norm", "lm_head", "norm_swiftkv", "wkv_swiftkv")
+             if hasattr(m, n)]
     for lw in m.layers:
         if lw is None:
             continue

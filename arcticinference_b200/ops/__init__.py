@@ -1063,7 +1063,7 @@ def attention_contiguous(q, k, v, seq_lens, H: int, D: int, scale: float | None 
         out = torch.empty(T, H * D, dtype=q.dtype, device=q.device)
     assert k.stride(0) == v.stride(0)
     rc = nat.lib().ab200_attention(
-        q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), k.stride(0), T, 0, None, 0,
+        q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), k.stride(0), k.shape[0], 0, None, 0,
         meta.work.data_ptr(), meta.num_work, None, 1, T, H, H, D, 1 if causal else 0, float(scale),
         out.data_ptr(), out.stride(0), None, None, None, 128,
         nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
