@@ -54,6 +54,10 @@ def parse_args():
     ap.add_argument("--speculative-config", type=str, default=None)
     ap.add_argument("--enforce-eager", action="store_true")
     ap.add_argument("--no-clocks", action="store_true")
+    ap.add_argument("--workload", default="serving", choices=["serving", "layers"],
+                    help="serving: the headline benchmark; layers: prefill and decode of Taralix "
+                         "layers beside Llama layers of equal size (benchmarks/layer_bench.py)")
+    ap.add_argument("--layer-case", default=None)
     return ap.parse_args()
 
 
@@ -231,6 +235,9 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     n_gpus = args.gpus
 
+    if args.workload == "layers":
+        from benchmarks.layer_bench import main as layer_bench
+        return layer_bench(["--layer-case", args.layer_case] if args.layer_case else [])
     if args.impl == "reference":
         return run_reference(args, rank, local_rank) if rank == 0 else 0
 

@@ -1,0 +1,251 @@
+"""Prefill and decode throughput of Taralix layers beside Llama layers of equal size (random
+weights), with the device time of every op and the time its roofline allows.
+
+    python bench.py --workload layers [--layer-case NAME]       (or: python benchmarks/layer_bench.py)
+
+Cases (width, heads x (dim, vdim), kv_rank, feed-forward), every second layer sharing the latents
+of the one before it:
+
+    moe-2048     2048, 16 x (128, 128), 512, 64 experts of 1408, 6 per token
+    dense-2560   2560, 40 x (64, 64),   256, 6400
+    dense-4096   4096, 32 x (128, 128), 512, 14336
+
+The Llama beside each has the same width, query heads, head dimension and active feed-forward
+width, and 8 K/V heads. Prefill: four prompts of 2048 tokens in one step. Decode: 128 sequences at
+2000 tokens of context, captured step. Both are one forward pass without the LM head, timed with
+CUDA events; the weights of a pass exceed L2. The roofline of an op is the larger of its
+algorithmic bytes over the measured copy bandwidth and its flops over the measured bf16 rate.
+"""
+
+from __future__ import annotations
+
+import argparse
+import json
+import os
+import sys
+
+REPO = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+sys.path.insert(0, REPO)
+
+CASES = {
+    "moe-2048": dict(width=2048, heads=16, dim=128, rank=512, ff=1408, experts=64, top=6),
+    "dense-2560": dict(width=2560, heads=40, dim=64, rank=256, ff=6400, experts=0, top=1),
+    "dense-4096": dict(width=4096, heads=32, dim=128, rank=512, ff=14336, experts=0, top=1),
+}
+LAYERS, VOCAB, KV_HEADS = 4, 32000, 8
+PREFILL = [2048] * 4
+DECODE, CONTEXT = 128, 2000
+
+
+def model_configs(c):
+    from arcticinference_b200.config import ModelConfig
+    mlp = {"kind": "dense", "ff": c["ff"]} if not c["experts"] else \
+        {"kind": "moe", "expert": {"ff": c["ff"]},
+         "router": {"experts": c["experts"], "top": c["top"]}}
+    layers = []
+    for i in range(LAYERS):
+        m = {"heads": c["heads"], "dim": c["dim"], "vdim": c["dim"], "kv_rank": c["rank"],
+             "scale": c["dim"] ** -0.5}
+        if i % 2:
+            m["kv_from"] = i - 1
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+    tara = ModelConfig.from_layer_list({
+        "architecture": "Taralix", "width": c["width"], "vocab": VOCAB, "norm": {"eps": 1e-6},
+        "postln_alpha": 1.5, "layers": layers})
+    llama = ModelConfig(hidden_size=c["width"], num_hidden_layers=LAYERS,
+                        num_attention_heads=c["heads"], num_key_value_heads=KV_HEADS,
+                        head_dim=c["dim"], intermediate_size=c["ff"] * c["top"], vocab_size=VOCAB,
+                        max_position_embeddings=8192)
+    return {"taralix": tara, "llama": llama}
+
+
+def peaks():
+    try:
+        with open(os.path.join(REPO, "MEASURED_PEAKS.json")) as f:
+            d = json.load(f)
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "of measured"
+    except (OSError, KeyError, ValueError):
+        return 6.65e12, 1.59e15, "of fallback"
+
+
+def rooflines(cfg, q_lens, kv_lens):
+    """op -> seconds the layers' algorithmic bytes and flops allow (2 bytes per element)."""
+    hbm, flops, _ = peaks()
+    T = sum(q_lens)
+    pairs = sum(q * kl - q * (q - 1) / 2 for q, kl in zip(q_lens, kv_lens))
+    ctx = sum(kv_lens)
+    out: dict = {}
+
+    def add(op, nbytes, nflops=0.0):
+        out[op] = out.get(op, 0.0) + max(nbytes / hbm, nflops / flops)
+
+    def linear(n, k, rows=T, op="linear", weights=1):
+        add(op, 2.0 * (weights * n * k + rows * (n + k)), 2.0 * rows * n * k)
+
+    W = cfg.hidden_size
+    decode = max(q_lens) == 1
+    if cfg.layer_specs is None:
+        H, Hk, D, I = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim, cfg.intermediate_size
+        for _ in range(cfg.num_hidden_layers):
+            linear((H + 2 * Hk) * D, W)
+            add("rope_cache", 2.0 * T * (2 * (H + Hk) + 3 * Hk) * D)
+            add("attention", 2.0 * (2 * ctx * Hk * D + 2 * T * H * D), 4.0 * pairs * H * D)
+            linear(W, H * D)
+            linear(2 * I, W)
+            add("silu_mul_blocked", 2.0 * T * 3 * I)
+            linear(W, I)
+            add("rmsnorm", 2 * 2.0 * T * 4 * W)
+        return out
+    for l in cfg.layer_specs:
+        m, f = l.mixer, l.mlp
+        H, R, d = m.heads, m.kv_rank, m.dim
+        own = R if m.kv_from is None else 0
+        linear(H * d + own, W)
+        if own:
+            add("latent_norm_cache", 2.0 * T * 2 * R)
+        if decode:
+            add("head_linear", 2.0 * (H * R * d + T * H * (d + R)), 2.0 * T * H * R * d)
+            add("latent_attention", 2.0 * (ctx * R + 2 * T * H * R), 4.0 * pairs * H * R)
+            add("head_linear", 2.0 * (H * R * d + T * H * (d + R)), 2.0 * T * H * R * d)
+        else:
+            if own:
+                add("gather_rows", 2.0 * 2 * ctx * R)
+            linear(2 * H * d, R, rows=ctx)
+            add("attention_contiguous", 2.0 * (2 * ctx + 2 * T) * H * d, 4.0 * pairs * H * d)
+        linear(W, H * m.vdim)
+        add("stream_norm", T * W * 12.0)
+        if f.experts:
+            n = T * f.top
+            used = min(f.experts, n)
+            add("route", 4.0 * T * W + 2.0 * f.experts * W + 2.0 * (T + n) * W)
+            linear(2 * f.ff, W, rows=n, op="grouped_linear", weights=used)
+            linear(W, f.ff, rows=n, op="grouped_linear", weights=used)
+            add("stream_norm", T * W * 10.0 + 2.0 * n * W)
+        else:
+            linear(2 * f.ff, W, op="gated_linear" if T > 256 else "linear")
+            if T <= 256:
+                add("gated_act", 2.0 * T * 3 * f.ff)
+            linear(W, f.ff)
+            add("stream_norm", T * W * 12.0)
+    return out
+
+
+def build_runner(cfg):
+    from arcticinference_b200.config import (CacheConfig, EngineConfig, ParallelConfig,
+                                             SchedulerConfig)
+    from arcticinference_b200.engine.model_runner import ModelRunner
+    blocks = max(sum(-(-n // 64) for n in PREFILL), DECODE * (-(-(CONTEXT + 64) // 64))) + 1
+    ec = EngineConfig(model=cfg, parallel=ParallelConfig(),
+                      cache=CacheConfig(num_gpu_blocks=blocks, enable_prefix_caching=False),
+                      scheduler=SchedulerConfig(max_model_len=CONTEXT + 64), load_format="dummy")
+    ec.validate()
+    r = ModelRunner(ec, "cuda")
+    r.load_model()
+    r.init_kv_cache(blocks)
+    for c in r.kv.k + getattr(r.kv, "v", []):     # a cache that holds something
+        c.normal_()
+    return r
+
+
+def step_of(lens, new):
+    """A scheduler output in which request i has ``lens[i]`` tokens, the last ``new`` of them now."""
+    from arcticinference_b200.engine.request import Request
+    from arcticinference_b200.engine.sampling_params import SamplingParams
+    from arcticinference_b200.engine.scheduler import ScheduledRequest, SchedulerOutput
+    out, blk = SchedulerOutput(), 1
+    for i, n in enumerate(lens):
+        r = Request("r%d" % i, [(7 * i + 13 * j) % VOCAB for j in range(n)],
+                    SamplingParams(temperature=0.0))
+        k = -(-n // 64)
+        r.block_ids = list(range(blk, blk + k))
+        blk += k
+        q = n if new is None else new
+        out.scheduled.append(ScheduledRequest(r, n - q, q, 0, True))
+        out.total_tokens += q
+    return out
+
+
+def timed(fn, warmup=5, reps=20):
+    import torch
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    a, b = (torch.cuda.Event(enable_timing=True) for _ in range(2))
+    a.record()
+    for _ in range(reps):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / reps
+
+
+def measure(name, cfg):
+    import torch
+    from arcticinference_b200 import ops
+    from arcticinference_b200.engine.cuda_graph import DecodeGraph
+    r = build_runner(cfg)
+    res = {}
+    with torch.inference_mode():
+        for phase, lens, new in (("prefill", PREFILL, None), ("decode", [CONTEXT] * DECODE, 1)):
+            out = step_of(lens, new)
+            batch, _ = r.prepare(out)
+            fwd = lambda: r.model.forward(batch, r.kv)
+            if phase == "prefill":
+                ms = timed(fwd)
+            else:
+                g = DecodeGraph(r, "tp", DECODE)
+                g.fill(out)
+                g.upload()
+                torch.cuda.synchronize()
+                g._body = lambda: (fwd_graph(r, g), None)
+                g.capture()
+                ms = timed(g.graph.replay)
+            with ops.OpTimer() as t:
+                for _ in range(5):
+                    fwd()
+            q = [n if new is None else new for n in lens]
+            ideal = rooflines(cfg, q, lens)
+            table = {}
+            for op, (us, cnt) in t.summary().items():
+                if op == "_start":
+                    continue
+                row = {"us": round(us / 5, 1), "calls": cnt // 5}
+                if op in ideal:
+                    row["of_roofline"] = round(1e6 * ideal[op] / (us / 5), 3)
+                table[op] = row
+            tokens = sum(q)
+            res[phase] = {"ms": round(ms, 4), "tokens_per_s": round(tokens / ms * 1e3),
+                          "roofline_ms": round(1e3 * sum(ideal.values()), 4), "ops": table}
+    ops.check_status()
+    del r
+    torch.cuda.empty_cache()
+    return res
+
+
+def fwd_graph(r, g):
+    return r.model.forward(g.batch, r.kv)
+
+
+def main(argv=None) -> int:
+    ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
+    ap.add_argument("--layer-case", choices=sorted(CASES), default=None)
+    ap.add_argument("--model", choices=["taralix", "llama"], default=None)
+    ns = ap.parse_args(argv)
+    import torch
+    torch.cuda.set_device(0)
+    for name, c in CASES.items():
+        if ns.layer_case not in (None, name):
+            continue
+        line = {"workload": "layers", "case": name, "layers": LAYERS, **c,
+                "peaks": peaks()[2], "prefill_tokens": sum(PREFILL), "decode_batch": DECODE,
+                "context": CONTEXT, "data": "random weights and latents", "dtype": "bf16",
+                "l2": "weights and cache of a pass exceed L2"}
+        for kind, cfg in model_configs(c).items():
+            if ns.model in (None, kind):
+                line[kind] = measure(name, cfg)
+        print(json.dumps(line), flush=True)
+    return 0
+
+
+if __name__ == "__main__":
+    sys.exit(main())
