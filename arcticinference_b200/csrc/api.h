@@ -255,9 +255,8 @@ int ab200_latent_attention_exact(const void* q, long long ldq, const void* cache
 
 // ---- moe.cu
 int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,
-                    void* ids, void* weights, int dtype, cudaStream_t stream);
-int ab200_moe_plan(const void* ids, long long n, int E, void* cursor, void* tiles, void* num_tiles,
-                   cudaStream_t stream);
+                    void* ids, void* weights, void* state, void* cursor, void* tiles,
+                    void* num_tiles, int dtype, cudaStream_t stream);
 int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, void* xp,
                       long long T, int W, int top, int dtype, cudaStream_t stream);
 

@@ -12,9 +12,8 @@
 // which is what lets one CTA own the whole latent width.
 //
 // Latents arrive as 128 x 64 pieces (one 128-byte swizzle atom wide) in a ring; a piece is free
-// again when its share of O^T has been accumulated. While the tensor core works on tile j, the
-// pieces of tile j + 1 are loading (R <= 256: whole tiles ahead, and S of tile j + 1 is issued
-// before O of tile j).
+// again when its share of O^T has been accumulated.
+// S of tile j + 1 is issued before O of tile j where the ring holds two tiles (R <= 256).
 //
 // Softmax: four warps, a thread per key. A column's maximum over the keys is a butterfly over
 // the warp's lanes (16 columns in 16 shuffles) and four words of shared memory; sums stay
@@ -199,94 +198,127 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
         for (int c = 0; c < NC; ++c)
           tma_load_2d(sQ + (uint32_t)c * NR * 128u, &tmap_q, q_full, c * 64, row0);
       }
+      // A lane per (piece, cache block) box of the tile: it waits for the piece's slot itself and
+      // issues its copy, so a tile's copies leave as fast as their slots come free.
       const int* bt = p.block_tables + (long long)seq * p.max_blocks;
+      const int nb_max = kLatKeys / bs;
+      const int boxes = NC * nb_max;
       bool ok = true;
-      int slot = 0;
-      uint32_t ph = 0;
-      int issued = 0;
+      int bid_next = 0;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int key0 = kv_start + j * kLatKeys;
         const int nblk = (min(kLatKeys, kv_end - key0) + bs - 1) / bs;
-        const int bid = lane < nblk ? bt[key0 / bs + lane] : 0;
-        for (int c = 0; c < NC; ++c) {
-          if (!__all_sync(0xffffffffu, mbar_wait(c_empty(slot), ph ^ 1u, &abort_s, p.status,
-                                                 1500 + slot, j))) {
-            ok = false;
-            break;
+        for (int i0 = 0; i0 < boxes && ok; i0 += 32) {
+          const int i = i0 + lane;
+          const int c = i / nb_max, blk = i % nb_max;
+          const bool mine = i < boxes && blk < nblk;
+          const int bid = (j == 0 || boxes > 32) ? (mine ? bt[key0 / bs + blk] : 0) : bid_next;
+          const int idx = j * NC + c;
+          const int slot = idx % p.slots;
+          const uint32_t ph = (uint32_t)(idx / p.slots) & 1u;
+          if (boxes <= 32 && j + 1 < n_tiles) {   // the next tile's table entry is on its way
+            const int next0 = key0 + kLatKeys;
+            const int nn = (min(kLatKeys, kv_end - next0) + bs - 1) / bs;
+            bid_next = (i < boxes && blk < nn) ? bt[next0 / bs + blk] : 0;
           }
-          if (lane == 0) mbar_arrive_expect_tx(c_full(slot), (uint32_t)(nblk * bs) * 128u);
-          __syncwarp();
-          if (lane < nblk)
-            tma_load_2d(sC + (uint32_t)slot * kPieceBytes + (uint32_t)(lane * bs) * 128u, &tmap_c,
-                        c_full(slot), c * 64, bid * bs);
-          __syncwarp();
-          ++issued;
-          if (++slot == p.slots) {
-            slot = 0;
-            ph ^= 1u;
+          bool done = !mine;
+          unsigned long long t0 = 0;
+          uint32_t spins = 0;
+          while (!done) {
+            if (mbar_try_wait(c_empty(slot), ph ^ 1u)) {
+              if (blk == 0) mbar_arrive_expect_tx(c_full(slot), (uint32_t)(nblk * bs) * 128u);
+              tma_load_2d(sC + (uint32_t)slot * kPieceBytes + (uint32_t)(blk * bs) * 128u, &tmap_c,
+                          c_full(slot), c * 64, bid * bs);
+              done = true;
+            } else if ((++spins & 63u) == 0u) {
+              if (abort_s) {
+                ok = false;
+                break;
+              }
+              if (t0 == 0) t0 = globaltimer_ns();
+              else if (globaltimer_ns() - t0 > kWaitLimitNs) {
+                abort_s = 1;
+                report_error(p.status, kErrBarrierTimeout, 1500 + slot, j);
+                ok = false;
+                break;
+              }
+            }
           }
+          ok = __all_sync(0xffffffffu, ok);
         }
       }
       if (!ok) {   // unwinding: give copies that were already issued a short time to land
-        for (int i = 0; i < min(issued, p.slots); ++i) {
-          if (--slot < 0) {
-            slot = p.slots - 1;
-            ph ^= 1u;
-          }
-          mbar_drain(c_full(slot), ph);
+        const unsigned long long t0 = globaltimer_ns();
+        while (globaltimer_ns() - t0 < 5000000ull) {
         }
-        mbar_drain(q_full, 0);
       }
     }
   } else if (warp == 5) {
     // ------------------------------- MMA issuer -------------------------------
-    if (lane == 0 && n_tiles > 0) {
+    // The whole warp walks the loop with uniform values and one elected lane issues: descriptors
+    // then live in uniform registers, and an instruction goes out as fast as the tensor core
+    // takes it.
+    if (n_tiles > 0) {
       const uint32_t idesc_s = make_idesc(128, NR, 1, 1, 0, 0);
       const uint32_t idesc_o = make_idesc(128, NR, 1, 1, 1, 0);
-      bool ok = mbar_wait(q_full, 0, &abort_s, p.status, 1600, 0);
+      const uint32_t tm = __shfl_sync(0xffffffffu, tmem_slot, 0);
+      const uint32_t tS_u = tm, tO_u = tm + 2 * NR;
+      const uint64_t c_k = make_desc_kmajor_sw128(sC);                   // + 1024 per slot
+      const uint64_t c_mn = make_desc_mnmajor_sw128(sC, kPieceBytes);
+      const uint64_t q_k = make_desc_kmajor_sw128(sQ);                   // + NR * 8 per piece
+      const uint64_t p_k = make_desc_kmajor_sw128(sP);
+      int s_slot = 0, o_slot = 0;
+      uint32_t s_ph = 0;
+      auto wait = [&](uint32_t bar, uint32_t parity, int code, int j) -> bool {
+        return __all_sync(0xffffffffu, mbar_wait(bar, parity, &abort_s, p.status, code, j));
+      };
+      bool ok = wait(q_full, 0, 1600, 0);
       auto issue_s = [&](int j) -> bool {
         const int st = j & 1;
-        if (!mbar_wait(s_empty(st), ((uint32_t)(j >> 1) & 1u) ^ 1u, &abort_s, p.status, 1620 + st, j))
-          return false;
-        int idx = j * NC;
-        for (int c = 0; c < NC; ++c, ++idx) {
-          const int slot = idx % p.slots;
-          if (!mbar_wait(c_full(slot), (uint32_t)(idx / p.slots) & 1u, &abort_s, p.status,
-                         1610 + slot, j))
-            return false;
+        if (!wait(s_empty(st), ((uint32_t)(j >> 1) & 1u) ^ 1u, 1620 + st, j)) return false;
+        for (int c = 0; c < NC; ++c) {
+          if (!wait(c_full(s_slot), s_ph, 1610, j)) return false;
           tc_fence_after();
-          const uint64_t cd = make_desc_kmajor_sw128(sC + (uint32_t)slot * kPieceBytes);
-          const uint64_t qd = make_desc_kmajor_sw128(sQ + (uint32_t)c * NR * 128u);
+          const uint64_t cd = c_k + (uint64_t)(s_slot * (int)(kPieceBytes / 16));
+          const uint64_t qd = q_k + (uint64_t)(c * (NR * 8));
+          if (elect_one()) {
 #pragma unroll
-          for (int k = 0; k < 4; ++k)
-            umma_f16_ss(tS + (uint32_t)st * NR, cd + (uint64_t)(2 * k), qd + (uint64_t)(2 * k),
-                        idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+            for (int k = 0; k < 4; ++k)
+              umma_f16_ss(tS_u + (uint32_t)st * NR, cd + (uint64_t)(2 * k), qd + (uint64_t)(2 * k),
+                          idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+            if (c == NC - 1) tc_commit(s_full(st));
+          }
+          __syncwarp();
+          if (++s_slot == p.slots) {
+            s_slot = 0;
+            s_ph ^= 1u;
+          }
         }
-        tc_commit(s_full(st));
         return true;
       };
       auto issue_o = [&](int j) -> bool {
         const int pb = p.p_bufs == 2 ? (j & 1) : 0;
         const uint32_t pph = (uint32_t)(p.p_bufs == 2 ? (j >> 1) : j) & 1u;
-        if (!mbar_wait(p_full(pb), pph, &abort_s, p.status, 1640 + pb, j)) return false;
+        if (!wait(p_full(pb), pph, 1640 + pb, j)) return false;
         tc_fence_after();
-        const uint32_t pbase = sP + (uint32_t)pb * NR * 256u;
+        const uint64_t pd = p_k + (uint64_t)(pb * (NR * 16));
         for (int rc = 0; rc < NC / 2; ++rc) {
           // two neighbouring pieces (128 latent columns); a pair never wraps: slots is even
-          const int slot = (j * NC + 2 * rc) % p.slots;
-          const uint64_t cd =
-              make_desc_mnmajor_sw128(sC + (uint32_t)slot * kPieceBytes, kPieceBytes);
+          const uint64_t cd = c_mn + (uint64_t)(o_slot * (int)(kPieceBytes / 16));
+          if (elect_one()) {
 #pragma unroll
-          for (int k = 0; k < kLatKeys / 16; ++k) {
-            const uint64_t pd = make_desc_kmajor_sw128(pbase + (uint32_t)(k / 4) * NR * 128u) +
-                                (uint64_t)(2 * (k % 4));
-            umma_f16_ss(tO + (uint32_t)(rc * NR), cd + (uint64_t)(128 * k), pd, idesc_o,
-                        (j > 0 || k > 0) ? 1u : 0u);
+            for (int k = 0; k < kLatKeys / 16; ++k)
+              umma_f16_ss(tO_u + (uint32_t)(rc * NR), cd + (uint64_t)(128 * k),
+                          pd + (uint64_t)((k / 4) * (NR * 8) + 2 * (k % 4)), idesc_o,
+                          (j > 0 || k > 0) ? 1u : 0u);
+            tc_commit(c_empty(o_slot));
+            tc_commit(c_empty(o_slot + 1));
+            if (rc == NC / 2 - 1) tc_commit(o_full(j & 1));
           }
-          tc_commit(c_empty(slot));
-          tc_commit(c_empty(slot + 1));
+          __syncwarp();
+          o_slot += 2;
+          if (o_slot == p.slots) o_slot = 0;
         }
-        tc_commit(o_full(j & 1));
         return true;
       };
       if (ok) ok = issue_s(0);
@@ -318,18 +350,22 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
                                                    p.status, 1700 + st, j));
       tc_fence_after();
       const uint32_t ts = tS + (uint32_t)st * NR + lane_off;
+      uint32_t sr[NR / 16][16];   // this key's scores
       if (ok) {
 #pragma unroll
+        for (int g = 0; g < NR / 16; ++g) tmem_ld_x16(ts + 16u * g, sr[g]);
+#pragma unroll
+        for (int g = 0; g < NR / 16; ++g) tmem_ld_wait_dep16(sr[g]);
+        if (need_mask) {
+#pragma unroll
+          for (int i = 0; i < NR; ++i)
+            if (key > lim_s[i]) sr[i / 16][i % 16] = 0xff800000u;   // -inf
+        }
+#pragma unroll
         for (int g = 0; g < NR / 16; ++g) {
-          uint32_t r[16];
-          tmem_ld_x16(ts + 16u * g, r);
-          tmem_ld_wait_dep16(r);
           float v[16];
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            v[i] = __uint_as_float(r[i]);
-            if (need_mask && key > lim_s[16 * g + i]) v[i] = -INFINITY;
-          }
+          for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(sr[g][i]);
           const float mx = reduce16<true>(v, lane);
           if ((lane & 1) == 0) wred[(16 * g + my_col) * 4 + warp] = mx;
         }
@@ -338,7 +374,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
       if (tid < NR) {
         const float4 q = *reinterpret_cast<const float4*>(&wred[tid * 4]);
         const float m_old = m_s[tid];
-        const float m_new = fmaxf(m_old, fmaxf(fmaxf(q.x, q.y), fmaxf(q.z, q.w)));
+        // Any reference point near the maximum serves: it moves only when the maximum has grown by
+        // more than 2^8, so that O is rarely rescaled (weights stay below 2^8 in fp32 and bf16)
+        const float mx = fmaxf(fmaxf(q.x, q.y), fmaxf(q.z, q.w));
+        const float m_new = (m_old == -INFINITY || (mx - m_old) * sc > 8.f) ? fmaxf(m_old, mx) : m_old;
         const float m_safe = m_new == -INFINITY ? 0.f : m_new;
         // a row that has seen no key yet holds O = 0 and l = 0: nothing to rescale
         const float alpha = m_old == -INFINITY ? 1.f : ex2_approx((m_old - m_safe) * sc);
@@ -384,17 +423,21 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
         const int chunk = (tid & 63) >> 3;
 #pragma unroll
         for (int g = 0; g < NR / 16; ++g) {
-          uint32_t r[16];
-          tmem_ld_x16(ts + 16u * g, r);
-          tmem_ld_wait_dep16(r);
+          float e[16];
+#pragma unroll
+          for (int i = 0; i < 16; i += 4) {
+            const float4 ng = *reinterpret_cast<const float4*>(&neg_s[16 * g + i]);
+            e[i] = ex2_approx(fmaf(__uint_as_float(sr[g][i]), sc, ng.x));
+            e[i + 1] = ex2_approx(fmaf(__uint_as_float(sr[g][i + 1]), sc, ng.y));
+            e[i + 2] = ex2_approx(fmaf(__uint_as_float(sr[g][i + 2]), sc, ng.z));
+            e[i + 3] = ex2_approx(fmaf(__uint_as_float(sr[g][i + 3]), sc, ng.w));
+          }
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const int n = 16 * g + i;
-            float e = ex2_approx(fmaf(__uint_as_float(r[i]), sc, neg_s[n]));
-            if (need_mask && key > lim_s[n]) e = 0.f;
-            l[n] += e;
+            l[n] += e[i];
             *reinterpret_cast<__nv_bfloat16*>(prow + n * 128 + ((chunk ^ (n & 7)) << 4)) =
-                __float2bfloat16(e);
+                __float2bfloat16(e[i]);
           }
         }
       }

@@ -3,9 +3,10 @@
 //
 //   moe_route    fp32 router logits x * W^T + b (a block keeps a few tokens' rows in shared
 //                memory, so router weights are read once per block), the `top` largest per token
-//                and the softmax over those
-//   moe_plan     rows per expert, each expert's first row among the rows sorted by expert, and
-//                the list of 128-row tiles the grouped matrix products walk
+//                and the softmax over those; rows per expert are counted on the way, and the
+//                block that finishes last turns the counts into each expert's first row among
+//                the rows sorted by expert and into the list of 128-row tiles the grouped matrix
+//                products walk
 //   moe_permute  row of every (token, choice) and the copy of the token's activations there
 //
 // The weighted sum of the experts' outputs is taken by the norm kernel that follows (stream.cu).
@@ -18,24 +19,108 @@
 
 namespace ab200 {
 
-constexpr int kRouteThreads = 256;
 constexpr int kTileRows = 128;
 
-// Router weights of type T; TB tokens per block. Shared memory: x rows [TB][W], logits [TB][E].
-template <typename T, int TB>
-__global__ void __launch_bounds__(kRouteThreads)
-moe_route_kernel(const float* __restrict__ x, const T* __restrict__ w, const float* __restrict__ b,
-                 long long n, int W, int E, int top, int* __restrict__ ids,
-                 float* __restrict__ weights) {
+// Four elements as they lie in memory, widened when they are used.
+template <typename T>
+struct Raw4;
+template <>
+struct Raw4<float> {
+  float4 q;
+  __device__ __forceinline__ void load(const float* p) { q = load4(p); }
+  __device__ __forceinline__ float4 get() const { return q; }
+};
+template <>
+struct Raw4<__nv_bfloat16> {
+  uint2 q;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { q = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ float4 get() const {
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+};
+
+struct RouteArgs {
+  const float* x;
+  const void* w;       // [E][W]
+  const float* b;
+  long long n;
+  int W, E, top;
+  int* ids;            // [n][top]
+  float* weights;      // [n][top]
+  int* state;          // [E] counts and [1] finished blocks; zero before and after every launch
+  int* cursor;         // [E] first row of each expert
+  int4* tiles;
+  int* num_tiles;
+};
+
+// Run by the last block: counts -> first rows and tiles; leaves the counts at zero.
+__device__ void moe_plan(const RouteArgs& p, int* sh) {
+  const int E = p.E;
+  int* count = sh;            // [E]
+  int* first = sh + E;        // [E]
+  int* tile0 = sh + 2 * E;    // [E]
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    count[e] = __ldcg(p.state + e);
+    p.state[e] = 0;
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {
+    int row = 0, tile = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int c = e < E ? count[e] : 0;
+      const int k = (c + kTileRows - 1) / kTileRows;
+      int rs = c, ts = k;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, rs, o);
+        const int d = __shfl_up_sync(0xffffffffu, ts, o);
+        if ((int)threadIdx.x >= o) {
+          rs += a;
+          ts += d;
+        }
+      }
+      if (e < E) {
+        first[e] = row + rs - c;
+        tile0[e] = tile + ts - k;
+      }
+      row += __shfl_sync(0xffffffffu, rs, 31);
+      tile += __shfl_sync(0xffffffffu, ts, 31);
+    }
+    if (threadIdx.x == 0) *p.num_tiles = tile;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    p.cursor[e] = first[e];
+    for (int r = 0, k = 0; r < count[e]; r += kTileRows, ++k)
+      p.tiles[tile0[e] + k] = make_int4(e, first[e] + r, min(kTileRows, count[e] - r), 0);
+  }
+}
+
+// Router weights of type T; TB tokens per block. Shared memory: x rows [TB][W], logits [TB][E],
+// at least 3 * E words for the plan.
+template <typename T, int TB, int kRouteThreads>
+__global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArgs p) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) float sm[];
+  __shared__ int last;
+  const int W = p.W, E = p.E, top = p.top;
   float* xs = sm;
   float* z = sm + (size_t)TB * W;
+  const T* w = reinterpret_cast<const T*>(p.w);
   const long long t0 = (long long)blockIdx.x * TB;
-  const int nt = (int)min((long long)TB, n - t0);
-  for (int i = threadIdx.x; i < TB * W; i += kRouteThreads)
-    xs[i] = i / W < nt ? x[t0 * W + i] : 0.f;
+  const int nt = (int)min((long long)TB, p.n - t0);
+  const bool vec = W % 4 == 0;
+  if (vec) {
+    for (int i = threadIdx.x * 4; i < TB * W; i += kRouteThreads * 4)
+      store4(xs + i, i / W < nt ? load4(p.x + t0 * W + i) : make_float4(0.f, 0.f, 0.f, 0.f));
+  } else {
+    for (int i = threadIdx.x; i < TB * W; i += kRouteThreads)
+      xs[i] = i / W < nt ? p.x[t0 * W + i] : 0.f;
+  }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr int EB = 4;   // experts a warp takes at a time
@@ -45,16 +130,53 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ w, const flo
     for (int t = 0; t < TB; ++t)
 #pragma unroll
       for (int j = 0; j < EB; ++j) acc[t][j] = 0.f;
-    for (int i = lane; i < W; i += 32) {
-      float wv[EB];
+    if (vec) {
+      // Two pieces of four consecutive elements per lane and step (conflict-free in shared
+      // memory); the next step's weights are on their way while this one's are multiplied.
+      const T* we[EB];
 #pragma unroll
-      for (int j = 0; j < EB; ++j)
-        wv[j] = e0 + j < E ? to_f32<T>(w[(long long)(e0 + j) * W + i]) : 0.f;
+      for (int j = 0; j < EB; ++j) we[j] = w + (long long)min(e0 + j, E - 1) * W;
+      Raw4<T> nxt[EB][2];
+      auto fetch = [&](int i) {
 #pragma unroll
-      for (int t = 0; t < TB; ++t) {
-        const float xv = xs[t * W + i];
+        for (int h = 0; h < 2; ++h) {
+          const int k = min(i + 128 * h, W - 4);
 #pragma unroll
-        for (int j = 0; j < EB; ++j) acc[t][j] = fmaf(xv, wv[j], acc[t][j]);
+          for (int j = 0; j < EB; ++j) nxt[j][h].load(we[j] + k);
+        }
+      };
+      fetch(lane * 4);
+      for (int i = lane * 4; i < W; i += 256) {
+        float4 wv[2][EB];
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int j = 0; j < EB; ++j) wv[h][j] = nxt[j][h].get();
+        fetch(i + 256);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          if (i + 128 * h >= W) break;
+#pragma unroll
+          for (int t = 0; t < TB; ++t) {
+            const float4 xv = load4(xs + t * W + i + 128 * h);
+#pragma unroll
+            for (int j = 0; j < EB; ++j) {
+              acc[t][j] = fmaf(xv.x, wv[h][j].x, acc[t][j]);
+              acc[t][j] = fmaf(xv.y, wv[h][j].y, acc[t][j]);
+              acc[t][j] = fmaf(xv.z, wv[h][j].z, acc[t][j]);
+              acc[t][j] = fmaf(xv.w, wv[h][j].w, acc[t][j]);
+            }
+          }
+        }
+      }
+    } else {
+      for (int i = lane; i < W; i += 32) {
+#pragma unroll
+        for (int j = 0; j < EB; ++j) {
+          const float wv = to_f32<T>(w[(long long)min(e0 + j, E - 1) * W + i]);
+#pragma unroll
+          for (int t = 0; t < TB; ++t) acc[t][j] = fmaf(xs[t * W + i], wv, acc[t][j]);
+        }
       }
     }
 #pragma unroll
@@ -62,7 +184,7 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ w, const flo
 #pragma unroll
       for (int j = 0; j < EB; ++j) {
         const float s = warp_sum(acc[t][j]);
-        if (lane == 0 && e0 + j < E) z[t * E + e0 + j] = s + b[e0 + j];
+        if (lane == 0 && e0 + j < E) z[t * E + e0 + j] = s + p.b[e0 + j];
       }
   }
   __syncthreads();
@@ -70,8 +192,8 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ w, const flo
   for (int t = warp; t < nt; t += kRouteThreads / 32) {
     float* zt = z + t * E;
     float first = 0.f, sum = 0.f;
-    int* my_ids = ids + (t0 + t) * top;
-    float* my_w = weights + (t0 + t) * top;
+    int* my_ids = p.ids + (t0 + t) * top;
+    float* my_w = p.weights + (t0 + t) * top;
     for (int j = 0; j < top; ++j) {
       float best = -INFINITY;
       int bi = 0x7fffffff;
@@ -99,99 +221,69 @@ moe_route_kernel(const float* __restrict__ x, const T* __restrict__ w, const flo
         my_ids[j] = bi;
         my_w[j] = ex;
         zt[bi] = -INFINITY;
+        atomicAdd(p.state + bi, 1);
       }
       __syncwarp();
     }
     const float inv = 1.f / sum;
     for (int j = lane; j < top; j += 32) my_w[j] *= inv;
   }
-}
-
-// One block. Rows per expert -> first rows (cursor), 128-row tiles.
-__global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* __restrict__ ids, long long n, int E, int* __restrict__ cursor,
-                int4* __restrict__ tiles, int* __restrict__ num_tiles) {
-  pdl_wait();
-  pdl_trigger();
-  extern __shared__ int sh[];
-  int* count = sh;            // [E]
-  int* first = sh + E;        // [E]
-  int* tile0 = sh + 2 * E;    // [E]
-  for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
+  // every block counts itself done after its counts are visible; the last one plans
+  __threadfence();
   __syncthreads();
-  for (long long i = threadIdx.x; i < n; i += blockDim.x) atomicAdd(&count[ids[i]], 1);
-  __syncthreads();
-  if (threadIdx.x < 32) {
-    int row = 0, tile = 0;
-    for (int e0 = 0; e0 < E; e0 += 32) {
-      const int e = e0 + threadIdx.x;
-      const int c = e < E ? count[e] : 0;
-      const int k = (c + kTileRows - 1) / kTileRows;
-      int rs = c, ts = k;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const int a = __shfl_up_sync(0xffffffffu, rs, o);
-        const int d = __shfl_up_sync(0xffffffffu, ts, o);
-        if ((int)threadIdx.x >= o) {
-          rs += a;
-          ts += d;
-        }
-      }
-      if (e < E) {
-        first[e] = row + rs - c;
-        tile0[e] = tile + ts - k;
-      }
-      row += __shfl_sync(0xffffffffu, rs, 31);
-      tile += __shfl_sync(0xffffffffu, ts, 31);
-    }
-    if (threadIdx.x == 0) *num_tiles = tile;
+  if (threadIdx.x == 0) {
+    last = atomicAdd(p.state + E, 1) == (int)gridDim.x - 1;
+    if (last) p.state[E] = 0;
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < E; e += blockDim.x) {
-    cursor[e] = first[e];
-    for (int r = 0, k = 0; r < count[e]; r += kTileRows, ++k)
-      tiles[tile0[e] + k] = make_int4(e, first[e] + r, min(kTileRows, count[e] - r), 0);
+  if (last) {
+    __threadfence();
+    moe_plan(p, reinterpret_cast<int*>(sm));
   }
 }
 
-// A block per (token, choice): takes the next row of its expert and copies the activations.
+// A block per token: takes the next row of each of its experts and copies the activations there.
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 moe_permute_kernel(const T* __restrict__ x, const int* __restrict__ ids, int* __restrict__ cursor,
                    int* __restrict__ rows, T* __restrict__ xp, int W, int top) {
   pdl_wait();
   pdl_trigger();
-  __shared__ int row;
-  const long long i = blockIdx.x;
-  if (threadIdx.x == 0) {
-    row = atomicAdd(&cursor[ids[i]], 1);
-    rows[i] = row;
+  extern __shared__ int row[];
+  const long long t = blockIdx.x;
+  for (int j = threadIdx.x; j < top; j += blockDim.x) {
+    row[j] = atomicAdd(&cursor[ids[t * top + j]], 1);
+    rows[t * top + j] = row[j];
   }
   __syncthreads();
-  const T* src = x + (i / top) * W;
-  T* dst = xp + (long long)row * W;
+  const T* src = x + t * W;
   constexpr int V = 16 / sizeof(T);
   if (W % V == 0) {
-    for (int c = threadIdx.x; c < W / V; c += blockDim.x)
-      reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+    for (int c = threadIdx.x; c < W / V; c += blockDim.x) {
+      const uint4 v = reinterpret_cast<const uint4*>(src)[c];
+      for (int j = 0; j < top; ++j) reinterpret_cast<uint4*>(xp + (long long)row[j] * W)[c] = v;
+    }
   } else {
-    for (int c = threadIdx.x; c < W; c += blockDim.x) dst[c] = src[c];
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      const T v = src[c];
+      for (int j = 0; j < top; ++j) xp[(long long)row[j] * W + c] = v;
+    }
   }
 }
 
 template <typename T, int TB>
-static int launch_route(const void* x, const void* w, const void* b, long long n, int W, int E,
-                        int top, void* ids, void* weights, cudaStream_t stream) {
-  const size_t smem = ((size_t)TB * W + (size_t)TB * E) * sizeof(float);
+static int launch_route(const RouteArgs& a, cudaStream_t stream) {
+  size_t smem = ((size_t)TB * a.W + (size_t)TB * a.E) * sizeof(float);
+  if (smem < (size_t)3 * a.E * sizeof(int)) smem = (size_t)3 * a.E * sizeof(int);
   if (smem > 220 * 1024) return -6;
-  auto k = moe_route_kernel<T, TB>;
+  // few tokens: more warps per block, so that each has few experts to go through
+  constexpr int kRouteThreads = TB == 1 ? 512 : 256;
+  auto k = moe_route_kernel<T, TB, kRouteThreads>;
   if (smem > 48 * 1024 &&
       cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return -3;
-  return launch_pdl(k, dim3((unsigned)((n + TB - 1) / TB)), dim3(kRouteThreads), smem, stream,
-                    reinterpret_cast<const float*>(x), reinterpret_cast<const T*>(w),
-                    reinterpret_cast<const float*>(b), n, W, E, top, reinterpret_cast<int*>(ids),
-                    reinterpret_cast<float*>(weights)) == cudaSuccess
+  return launch_pdl(k, dim3((unsigned)((a.n + TB - 1) / TB)), dim3(kRouteThreads), smem, stream,
+                    a) == cudaSuccess
              ? 0
              : -5;
 }
@@ -203,42 +295,45 @@ typedef __nv_bfloat16 bf16;
 
 extern "C" {
 
-// x fp32 [T, W]; w [E, W] (dtype 0 = bf16, 1 = fp32); b fp32 [E]; ids int32 and weights fp32 [T, top]
+// x fp32 [T, W]; w [E, W] (dtype 0 = bf16, 1 = fp32); b fp32 [E]; ids int32 and weights fp32
+// [T, top]; state int32 [E + 1], zero; cursor int32 [E]; tiles int32 x 4 [T * top / 128 + E at
+// most]; num_tiles int32 [1]
 int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,
-                    void* ids, void* weights, int dtype, cudaStream_t stream) {
+                    void* ids, void* weights, void* state, void* cursor, void* tiles,
+                    void* num_tiles, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (top < 1 || top > E) return -2;
+  RouteArgs a;
+  a.x = reinterpret_cast<const float*>(x);
+  a.w = w;
+  a.b = reinterpret_cast<const float*>(b);
+  a.n = T;
+  a.W = W;
+  a.E = E;
+  a.top = top;
+  a.ids = reinterpret_cast<int*>(ids);
+  a.weights = reinterpret_cast<float*>(weights);
+  a.state = reinterpret_cast<int*>(state);
+  a.cursor = reinterpret_cast<int*>(cursor);
+  a.tiles = reinterpret_cast<int4*>(tiles);
+  a.num_tiles = reinterpret_cast<int*>(num_tiles);
   // many tokens: several per block, so that the router's weights are read less often
   const bool wide = T >= 148 * 8 && (size_t)8 * (W + E) * 4 <= 110 * 1024;
-  if (dtype == 0)
-    return wide ? launch_route<bf16, 8>(x, w, b, T, W, E, top, ids, weights, stream)
-                : launch_route<bf16, 1>(x, w, b, T, W, E, top, ids, weights, stream);
-  return wide ? launch_route<float, 8>(x, w, b, T, W, E, top, ids, weights, stream)
-              : launch_route<float, 1>(x, w, b, T, W, E, top, ids, weights, stream);
-}
-
-// ids int32 [n]; cursor int32 [E]; tiles int32 x 4 [n / 128 + E at most]; num_tiles int32 [1]
-int ab200_moe_plan(const void* ids, long long n, int E, void* cursor, void* tiles, void* num_tiles,
-                   cudaStream_t stream) {
-  if (E <= 0 || E > 4096) return -6;
-  return launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream,
-                    reinterpret_cast<const int*>(ids), n, E, reinterpret_cast<int*>(cursor),
-                    reinterpret_cast<int4*>(tiles), reinterpret_cast<int*>(num_tiles)) == cudaSuccess
-             ? 0
-             : -5;
+  if (dtype == 0) return wide ? launch_route<bf16, 8>(a, stream) : launch_route<bf16, 1>(a, stream);
+  return wide ? launch_route<float, 8>(a, stream) : launch_route<float, 1>(a, stream);
 }
 
 int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, void* xp,
                       long long T, int W, int top, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  const dim3 grid((unsigned)(T * top));
+  const size_t smem = (size_t)top * sizeof(int);
   const cudaError_t e =
       dtype == 0
-          ? launch_pdl(moe_permute_kernel<bf16>, grid, dim3(128), 0, stream,
+          ? launch_pdl(moe_permute_kernel<bf16>, dim3((unsigned)T), dim3(256), smem, stream,
                        reinterpret_cast<const bf16*>(x), reinterpret_cast<const int*>(ids),
                        reinterpret_cast<int*>(cursor), reinterpret_cast<int*>(rows),
                        reinterpret_cast<bf16*>(xp), W, top)
-          : launch_pdl(moe_permute_kernel<float>, grid, dim3(128), 0, stream,
+          : launch_pdl(moe_permute_kernel<float>, dim3((unsigned)T), dim3(256), smem, stream,
                        reinterpret_cast<const float*>(x), reinterpret_cast<const int*>(ids),
                        reinterpret_cast<int*>(cursor), reinterpret_cast<int*>(rows),
                        reinterpret_cast<float*>(xp), W, top);

@@ -49,7 +49,7 @@ def _up(n: int, m: int) -> int:
 class TaralixLayer:
     """Weights and shapes of one layer."""
 
-    __slots__ = LAYER_TENSORS + ("extra", "spec", "source", "shape", "dq", "dv", "rank", "expand",
+    __slots__ = LAYER_TENSORS + ("extra", "spec", "source", "shape", "scale", "dq", "dv", "rank", "expand",
                                  "ckv_cols")
 
     def __init__(self):
@@ -245,6 +245,10 @@ class TaralixForCausalLM:
         lw.shape, lw.dq, lw.dv, lw.expand = self._geometry[l]
         align = 8 if self.dtype == torch.bfloat16 else 1
         q = self._pad(self._expect(t["mix.q"], H * m.dim, W).view(H, m.dim, W), H, lw.dq)
+        # the attention kernels take a maximum of unscaled scores, i.e. a positive scale
+        lw.scale = m.scale
+        if m.scale <= 0:
+            q, lw.scale = (-q, -m.scale) if m.scale < 0 else (torch.zeros_like(q), 1.0)
         rows = [q.reshape(H * lw.dq, W)]
         lw.ckv_cols = 0
         if m.kv_from is None:
@@ -379,7 +383,7 @@ class TaralixForCausalLM:
         if n:
             q = st.head_linear(proj[:n, :nq], lw.wuk_t)
             o = lat.latent_attention(q, cache, step.absorbed[(lw.shape, n == T)], lw.shape,
-                                     m.scale, step.tok_seq, batch.positions)
+                                     lw.scale, step.tok_seq, batch.positions)
             st.head_linear(o, lw.wuv, out=out[:n])
         if n < T:
             c = contexts.get(lw.source)
@@ -387,7 +391,7 @@ class TaralixForCausalLM:
                 c = contexts[lw.source] = ops.gather_rows(cache.view(-1, lw.rank), step.ctx_slots)
             kvs = ops.linear(c, lw.wukv)
             lat.expanded_attention(proj[n:, :nq], kvs[:, :nq], kvs[:, nq:], step, H, lw.expand,
-                                   m.scale, out[n:])
+                                   lw.scale, out[n:])
         return ops.linear(out, lw.wo)
 
     def _feed_forward(self, lw: TaralixLayer, x, act):

@@ -130,8 +130,7 @@ def _declare(L: ctypes.CDLL) -> None:
         "ab200_linear_exact": (I, [P, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P]),
         "ab200_latent_attention_exact": (I, [P, LL, P, I, I, P, I, P, P, P, LL, LL, I, I, F, I, P,
                                              P]),
-        "ab200_moe_route": (I, [P, P, P, LL, I, I, I, P, P, I, P]),
-        "ab200_moe_plan": (I, [P, LL, I, P, P, P, P]),
+        "ab200_moe_route": (I, [P, P, P, LL, I, I, I, P, P, P, P, P, P, I, P]),
         "ab200_moe_permute": (I, [P, P, P, P, P, LL, I, I, I, P]),
         "ab200_grouped_gemm": (I, [P, LL, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P, P]),
         "ab200_latent_attention": (I, [P, LL, P, I, I, P, I, P, I, P, I, LL, I, I, I, F, P, P, P, P,

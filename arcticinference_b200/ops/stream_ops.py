@@ -161,6 +161,19 @@ def route_ref(x, w, b, top: int):
     return order, torch.softmax(z.gather(1, order), -1)
 
 
+_route_states: dict = {}
+
+
+def _route_state(E: int, device) -> torch.Tensor:
+    """Counters of the router kernel (zero between launches), one set per device and number of
+    experts."""
+    key = (torch.device(device).index, E)
+    t = _route_states.get(key)
+    if t is None:
+        t = _route_states[key] = torch.zeros(E + 1, dtype=torch.int32, device=device)
+    return t
+
+
 def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, top: int):
     """Router of a mixture of experts. ``x`` fp32 [T, W] stream, ``act`` its rounding (what the
     experts read), ``w`` [E, W], ``b`` fp32 [E]. Returns (Routing, act rows sorted by expert)."""
@@ -180,26 +193,31 @@ def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, 
     i32 = torch.int32
     ids = torch.empty(T, top, dtype=i32, device=dev)
     weights = torch.empty(T, top, dtype=torch.float32, device=dev)
-    rc = L.ab200_moe_route(x.data_ptr(), w.data_ptr(), b.data_ptr(), T, W, E, top, ids.data_ptr(),
-                           weights.data_ptr(), dc, nat.stream_ptr())
-    nat.check(rc, "moe_route")
-    launch_counter.add(1)
     max_tiles = min(T * top, T * top // TILE_ROWS + E)
     plan = torch.empty(E + 4 * max_tiles + 4 + T * top, dtype=i32, device=dev)
     tiles = plan[:4 * max_tiles].view(max_tiles, 4)
     num_tiles = plan[4 * max_tiles:4 * max_tiles + 1]
     cursor = plan[4 * max_tiles + 4:4 * max_tiles + 4 + E]
     rows = plan[4 * max_tiles + 4 + E:].view(T, top)
-    rc = L.ab200_moe_plan(ids.data_ptr(), T * top, E, cursor.data_ptr(), tiles.data_ptr(),
-                          num_tiles.data_ptr(), nat.stream_ptr())
-    nat.check(rc, "moe_plan")
+    rc = L.ab200_moe_route(x.data_ptr(), w.data_ptr(), b.data_ptr(), T, W, E, top, ids.data_ptr(),
+                           weights.data_ptr(), _route_state(E, dev).data_ptr(), cursor.data_ptr(),
+                           tiles.data_ptr(), num_tiles.data_ptr(), dc, nat.stream_ptr())
+    nat.check(rc, "moe_route")
     launch_counter.add(1)
-    xp = torch.empty(T * top, W, dtype=act.dtype, device=dev)
-    rc = L.ab200_moe_permute(act.data_ptr(), ids.data_ptr(), cursor.data_ptr(), rows.data_ptr(),
-                             xp.data_ptr(), T, W, top, dc, nat.stream_ptr())
+    r = Routing(ids, weights, rows, top, E, tiles, num_tiles)
+    return r, _permute(act, r, cursor)
+
+
+def _permute(act, r: Routing, cursor) -> torch.Tensor:
+    nat = _nat()
+    T, W = act.shape
+    xp = torch.empty(T * r.top, W, dtype=act.dtype, device=act.device)
+    rc = nat.lib().ab200_moe_permute(act.data_ptr(), r.ids.data_ptr(), cursor.data_ptr(),
+                                     r.rows.data_ptr(), xp.data_ptr(), T, W, r.top,
+                                     dtype_code(act.dtype), nat.stream_ptr())
     nat.check(rc, "moe_permute")
     launch_counter.add(1)
-    return Routing(ids, weights, rows, top, E, tiles, num_tiles), xp
+    return xp
 
 
 def _aligned(*ts) -> bool:

@@ -117,7 +117,8 @@ def rooflines(cfg, q_lens, kv_lens):
         if f.experts:
             n = T * f.top
             used = min(f.experts, n)
-            add("route", 4.0 * T * W + 2.0 * f.experts * W + 2.0 * (T + n) * W)
+            add("route", 4.0 * T * W + 2.0 * f.experts * W)
+            add("_permute", 2.0 * (T + n) * W)
             linear(2 * f.ff, W, rows=n, op="grouped_linear", weights=used)
             linear(W, f.ff, rows=n, op="grouped_linear", weights=used)
             add("stream_norm", T * W * 10.0 + 2.0 * n * W)
