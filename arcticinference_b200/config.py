@@ -659,8 +659,8 @@ class EngineConfig:
                 "per replica, or use the replica pool (python -m arcticinference_b200.server.cli), "
                 "which routes requests over them")
         if p.enable_expert_parallel:
-            raise NotImplementedError("enable_expert_parallel: no mixture-of-experts model is "
-                                      "implemented, so there is nothing to shard by expert")
+            raise NotImplementedError("enable_expert_parallel: experts are not sharded over GPUs "
+                                      "(mixture-of-experts models run on one GPU)")
         if self.cache.kv_cache_dtype not in SUPPORTED_KV_CACHE_DTYPES:
             raise NotImplementedError(
                 "kv_cache_dtype=%r: the attention kernels read %s caches only" %

@@ -168,39 +168,48 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
     }
   } else if (warp == 1) {
     // ------------------------------- MMA issuer -------------------------------
-    if (lane == 0) {
-      const uint32_t idesc = make_idesc(128, (uint32_t)p.bn, 1, 1, 0, 0);
-      int stage = 0, acc = 0;
-      uint32_t phase = 0, acc_phase = 0;
-      bool ok = true;
-      for (int w = blockIdx.x; w < total_work && ok; w += gridDim.x) {
-        if (!mbar_wait(tempty_bar(acc), acc_phase ^ 1u, abort_flag, p.status, 1200 + acc, w)) break;
+    // The warp walks the loop with uniform values and one elected lane issues, which keeps the
+    // descriptors in uniform registers: an instruction then costs what the tensor core takes,
+    // not what moving its operands there takes.
+    const uint32_t idesc = make_idesc(128, (uint32_t)p.bn, 1, 1, 0, 0);
+    const uint32_t tm = __shfl_sync(0xffffffffu, tmem_base, 0);
+    const uint64_t a0 = make_desc_kmajor_sw128(smem_base);
+    const uint64_t stage_step = stage_bytes / 16;
+    int stage = 0, acc = 0;
+    uint32_t phase = 0, acc_phase = 0;
+    bool ok = true;
+    for (int w = blockIdx.x; w < total_work && ok; w += gridDim.x) {
+      if (!__all_sync(0xffffffffu, mbar_wait(tempty_bar(acc), acc_phase ^ 1u, abort_flag, p.status,
+                                             1200 + acc, w)))
+        break;
+      tc_fence_after();
+      const uint32_t d_tmem = tm + (uint32_t)acc * acc_stride;
+      for (int kb = 0; kb < p.kblocks; ++kb) {
+        if (!__all_sync(0xffffffffu, mbar_wait(full_bar(stage), phase, abort_flag, p.status,
+                                               1300 + stage, kb))) {
+          ok = false;
+          break;
+        }
         tc_fence_after();
-        const uint32_t d_tmem = tmem_base + (uint32_t)acc * acc_stride;
-        for (int kb = 0; kb < p.kblocks; ++kb) {
-          if (!mbar_wait(full_bar(stage), phase, abort_flag, p.status, 1300 + stage, kb)) {
-            ok = false;
-            break;
-          }
-          tc_fence_after();
-          const uint32_t a_addr = smem_base + (uint32_t)stage * stage_bytes;
-          const uint64_t a_desc = make_desc_kmajor_sw128(a_addr);
-          const uint64_t b_desc = make_desc_kmajor_sw128(a_addr + kGgABytes);
+        const uint64_t a_desc = a0 + (uint64_t)stage * stage_step;
+        const uint64_t b_desc = a_desc + (uint64_t)(kGgABytes / 16);
+        if (elect_one()) {
 #pragma unroll
           for (int k = 0; k < kGgBlockK / 16; ++k)
             umma_f16_ss(d_tmem, a_desc + (uint64_t)(2 * k), b_desc + (uint64_t)(2 * k), idesc,
                         (kb > 0 || k > 0) ? 1u : 0u);
           tc_commit(empty_bar(stage));
-          if (++stage == p.stages) {
-            stage = 0;
-            phase ^= 1u;
-          }
+          if (kb == p.kblocks - 1) tc_commit(tfull_bar(acc));
         }
-        if (!ok) break;
-        tc_commit(tfull_bar(acc));
-        acc ^= 1;
-        if (acc == 0) acc_phase ^= 1u;
+        __syncwarp();
+        if (++stage == p.stages) {
+          stage = 0;
+          phase ^= 1u;
+        }
       }
+      if (!ok) break;
+      acc ^= 1;
+      if (acc == 0) acc_phase ^= 1u;
     }
   } else {
     // --------------------------------- epilogue --------------------------------

@@ -23,7 +23,7 @@ import torch
 
 from .engine import Alias, Channel, ack, receive_stream, send_stream
 from .schedule import TensorMeta, TransferSchedule, find_aliases
-from .utils import expected_llama_tensors, export_llama_state
+from .utils import expected_llama_tensors, export_llama_state, require_weight_sync
 
 
 def _rank(engine) -> int:
@@ -31,6 +31,7 @@ def _rank(engine) -> int:
 
 
 def engine_weights_info(engine) -> list:
+    require_weight_sync(engine)
     m = engine.runner.model
     return [asdict(t) for t in expected_llama_tensors(m.cfg, m.dtype)]
 
@@ -81,6 +82,8 @@ def engine_sync_weights(engine, kw: dict) -> dict:
     t0 = time.time()
     addr = kw.get("master_addr")
     target = kw.get("target", "model")
+    if target == "model":
+        require_weight_sync(engine)
     if isinstance(addr, str) and addr.startswith("ipc://"):
         from .ipc_engine import receive_ipc
         return receive_ipc(engine, addr[len("ipc://"):], target)

@@ -150,12 +150,19 @@ def assign_in_place(dst, src: torch.Tensor):
     return dst
 
 
+def require_weight_sync(engine) -> None:
+    """Live weight updates know the Llama family's checkpoint names only."""
+    cfg = engine.config.model
+    if cfg.layer_specs is not None:
+        raise NotImplementedError("weight sync for %s" % cfg.architecture)
+
+
 def engine_weight_norm(engine) -> float:
     """L2 norm over every weight this rank stores (fp8 weights are expanded): a cheap check
     that two replicas, or a replica and the trainer, hold the same parameters."""
     m = engine.runner.model
     acc = torch.zeros((), dtype=torch.float64, device=m.device)
-    ts = [m.embed, m.norm, m.norm_swiftkv, m.wkv_swiftkv]
+    ts = [m.embed, m.norm, getattr(m, "norm_swiftkv", None), getattr(m, "wkv_swiftkv", None)]
     if m.lm_head is not m.embed:
         ts.append(m.lm_head)
     for lw in m.layers:

@@ -83,6 +83,16 @@ def paged(q_lens, kv_lens, Hq=32, Hkv=8, D=128, bs=64):
 
 
 CASES = {
+    # decode in latent space: heads, latent width, sequences, cached tokens
+    "latent_512": ("latent", (16, 512, 128, 2000)),
+    "latent_256": ("latent", (40, 256, 128, 2000)),
+    "latent_128": ("latent", (16, 128, 128, 2000)),
+    # mixture of experts (gate / up with the activation): tokens, width, ff, experts, per token
+    "experts_prefill": ("experts", (8192, 2048, 1408, 64, 6)),
+    "experts_decode": ("experts", (128, 2048, 1408, 64, 6)),
+    "route_prefill": ("route", (8192, 2048, 64, 6)),
+    "route_decode": ("route", (128, 2048, 64, 6)),
+    "stream_norm": ("stream_norm", (8192, 4096)),
     # name: (kind, params)
     "gemm_prefill": ("gemm", (8192, 28672, 4096)),
     "gemm_prefill_qkv": ("gemm", (8192, 6144, 4096)),
@@ -192,6 +202,44 @@ def run_case(a, case):
                 st[3].tile_keys = a.tile_keys
         fn = lambda i=0: ops.attention(sets[i][0], sets[i][1], sets[i][2], sets[i][3], 32, 8, 128)
         flops = sum(4.0 * a_ * (b_ - a_ / 2.0) * 32 * 128 for a_, b_ in zip(ql, kl))
+    elif kind == "latent":
+        from arcticinference_b200.ops import latent_ops as lat
+        H, rank, n, kl = prm
+        byts = 2.0 * n * kl * rank + 4.0 * n * H * rank
+        nc = copies_for(byts)
+        nb = n * (-(-kl // 64)) + 1
+        bt = torch.arange(1, nb, dtype=torch.int32, device=DEV).view(n, -1)
+        shape = lat.LatentShape.of(H, rank, torch.bfloat16)
+        meta = lat.build_plan(shape, [1] * n, [kl] * n, bt, 64, DEV)
+        sets = [(R(n, H * rank), R(nb, 1, 64, rank)) for _ in range(nc)]
+        fn = lambda i=0: lat.latent_attention(sets[i][0], sets[i][1], meta, shape, 0.1)
+        flops = 4.0 * n * kl * H * rank
+    elif kind == "experts":
+        from arcticinference_b200.ops import stream_ops as st
+        T, W, ff, E, top = prm
+        x = torch.randn(T, W, device=DEV)
+        r, rows = st.route(x, x.to(torch.bfloat16), R(E, W), torch.zeros(E, device=DEV), top)
+        nc = copies_for(4 * E * W * ff)
+        ws = [R(E, 2 * ff, W) for _ in range(nc)]
+        fn = lambda i=0: st.grouped_linear(rows, ws[i], r, act="silu")
+        flops = 4.0 * T * top * W * ff
+        byts = 4.0 * E * W * ff + 2.0 * T * top * (W + ff)
+    elif kind == "route":
+        from arcticinference_b200.ops import stream_ops as st
+        T, W, E, top = prm
+        nc = copies_for(6 * T * W)
+        sets = [(torch.randn(T, W, device=DEV), R(T, W)) for _ in range(nc)]
+        w, b = R(E, W), torch.zeros(E, device=DEV)
+        fn = lambda i=0: st.route(sets[i][0], sets[i][1], w, b, top)
+        flops, byts = 2.0 * T * W * E, T * W * (6.0 + 2.0 * top)
+    elif kind == "stream_norm":
+        from arcticinference_b200.ops import stream_ops as st
+        T, W = prm
+        nc = copies_for(8 * T * W)
+        sets = [(torch.randn(T, W, device=DEV), R(T, W), R(T, W)) for _ in range(nc)]
+        w = torch.zeros(W, device=DEV)
+        fn = lambda i=0: st.stream_norm(sets[i][0], sets[i][1], sets[i][2], w, 1.5, 1e-6)
+        flops, byts = 0.0, 12.0 * T * W
     elif kind == "rmsnorm":
         T, H = prm
         nc = copies_for(4 * T * H)

@@ -195,6 +195,24 @@ def test_shared_latents_take_no_memory(tmp_path):
     assert m.kv_bytes_per_block(64) == (56 + 72) * 64 * 4
 
 
+def test_weight_sync_is_refused(tmp_path):
+    from arcticinference_b200.server.weight_sync.receiver import (engine_sync_weights,
+                                                                  engine_weights_info)
+    cfg = u.CONFIGS["single"]
+    engine = u.session(u.save(tmp_path, cfg, u.weights(cfg)), "float32", 64, "cpu").engine
+    with pytest.raises(NotImplementedError):
+        engine_weights_info(engine)
+    with pytest.raises(NotImplementedError):
+        engine_sync_weights(engine, {"master_addr": "ipc://nothing"})
+
+
+def test_kernel_set_names_existing_sources():
+    from arcticinference_b200 import build
+    stems = {p.stem for p in build.kernel_sources()}
+    for names in build.KERNEL_SETS.values():
+        assert set(names) <= stems
+
+
 # ---------------------------------------------------------------- planning of the latent kernel
 @pytest.mark.parametrize("heads,q_lens,kv_lens", [
     (16, [1] * 5, [1, 128, 129, 5000, 64]), (5, [3, 1, 130], [3, 700, 400]),
