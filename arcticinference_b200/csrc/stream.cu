@@ -134,14 +134,42 @@ latent_norm_cache_kernel(const T* __restrict__ ckv, long long ld, const float* _
     return;
   }
   const T* src = ckv + t * ld;
+  T* dst = cache + slot * Rp;
   float ss = 0.f;
+  if (((R | Rp) & 3) == 0 && (ld & 3) == 0 &&
+      ((reinterpret_cast<uintptr_t>(ckv) | reinterpret_cast<uintptr_t>(weight)) & 15) == 0) {
+    constexpr int kHeld = 4;   // of the row's four-element pieces, in registers
+    float4 v[kHeld];
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j) {
+      const int i = lane * 4 + 128 * j;
+      v[j] = i < R ? load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j)
+      ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    for (int i = lane * 4 + 128 * kHeld; i < R; i += 128) {
+      const float4 q = load4(src + i);
+      ss += q.x * q.x + q.y * q.y + q.z * q.z + q.w * q.w;
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / (float)R + eps);
+    auto put = [&](int i, const float4& q) {
+      const float4 w = load4(weight + i);
+      store4(dst + i, make_float4(q.x * inv * w.x, q.y * inv * w.y, q.z * inv * w.z, q.w * inv * w.w));
+    };
+#pragma unroll
+    for (int j = 0; j < kHeld; ++j)
+      if (lane * 4 + 128 * j < R) put(lane * 4 + 128 * j, v[j]);
+    for (int i = lane * 4 + 128 * kHeld; i < R; i += 128) put(i, load4(src + i));
+    return;
+  }
   for (int i = lane; i < R; i += 32) {
     const float v = to_f32<T>(src[i]);
     ss += v * v;
   }
   ss = warp_sum(ss);
   const float inv = 1.f / sqrtf(ss / (float)R + eps);
-  T* dst = cache + slot * Rp;
   for (int i = lane; i < R; i += 32) dst[i] = from_f32<T>(to_f32<T>(src[i]) * inv * weight[i]);
 }
 

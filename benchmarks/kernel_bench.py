@@ -93,6 +93,7 @@ CASES = {
     "route_prefill": ("route", (8192, 2048, 64, 6)),
     "route_decode": ("route", (128, 2048, 64, 6)),
     "stream_norm": ("stream_norm", (8192, 4096)),
+    "latent_norm_cache": ("latent_norm", (8192, 512)),
     # name: (kind, params)
     "gemm_prefill": ("gemm", (8192, 28672, 4096)),
     "gemm_prefill_qkv": ("gemm", (8192, 6144, 4096)),
@@ -232,6 +233,14 @@ def run_case(a, case):
         w, b = R(E, W), torch.zeros(E, device=DEV)
         fn = lambda i=0: st.route(sets[i][0], sets[i][1], w, b, top)
         flops, byts = 2.0 * T * W * E, T * W * (6.0 + 2.0 * top)
+    elif kind == "latent_norm":
+        from arcticinference_b200.ops import latent_ops as lat
+        T, rank = prm
+        nc = copies_for(4 * T * rank)
+        sets = [(R(T, rank), R(T // 64, 1, 64, rank)) for _ in range(nc)]
+        w, slots = torch.ones(rank, device=DEV), torch.arange(T, device=DEV)
+        fn = lambda i=0: lat.latent_norm_cache(sets[i][0], w, rank, 1e-6, slots, sets[i][1])
+        flops, byts = 0.0, 4.0 * T * rank
     elif kind == "stream_norm":
         from arcticinference_b200.ops import stream_ops as st
         T, W = prm

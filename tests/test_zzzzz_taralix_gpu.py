@@ -45,22 +45,24 @@ def test_stream_norm(T, W, dtype):
     close(out.cpu(), oracle.zero_centred_norm(x0.double().cpu(), w, 0.05)[rows.cpu()], dtype)
 
 
+@pytest.mark.parametrize("rank,ld", [(72, 300), (600, 800), (13, 77)])
 @pytest.mark.parametrize("dtype", [BF16, F32])
-def test_stream_embedding_and_latent_cache(dtype):
+def test_stream_embedding_and_latent_cache(dtype, rank, ld):
     torch.manual_seed(1)
     table, ids = rnd(50, 77, dtype=dtype), torch.tensor([3, 49, 0, 3], device=DEV)
     x, act = st.stream_embedding(ids, table)
     assert torch.equal(x, table[ids].float()) and torch.equal(act, table[ids])
-    buf, w = rnd(6, 300, dtype=dtype), rnd(72, dtype=F32)
-    cache = torch.zeros(3, 1, 16, 128, dtype=dtype, device=DEV)
+    buf, w = rnd(6, ld, dtype=dtype), rnd(rank, dtype=F32)
+    off, Rp = ld - rank - ld % 4, -(-rank // 128) * 128
+    cache = torch.zeros(3, 1, 16, Rp, dtype=dtype, device=DEV)
     slots = torch.tensor([47, -1, 0, 17, 16, 5], device=DEV)
-    lat.latent_norm_cache(buf[:, 200:], w, 72, 0.02, slots, cache)
-    want = torch.zeros(48, 128)
-    c = oracle.plain_norm(buf[:, 200:272].double().cpu(), w, 0.02).float()
+    lat.latent_norm_cache(buf[:, off:], w, rank, 0.02, slots, cache)
+    want = torch.zeros(48, Rp)
+    c = oracle.plain_norm(buf[:, off:off + rank].double().cpu(), w, 0.02).float()
     for i, s in enumerate(slots.tolist()):
         if s >= 0:
-            want[s, :72] = c[i]
-    close(cache.view(48, 128).cpu(), want, dtype)
+            want[s, :rank] = c[i]
+    close(cache.view(48, Rp).cpu(), want, dtype)
     ops.check_status()
 
 
