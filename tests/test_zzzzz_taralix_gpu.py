@@ -85,7 +85,7 @@ def test_gated_linear(T, W, ff, act, dtype):
 
 
 @pytest.mark.parametrize("dtype", [BF16, F32])
-@pytest.mark.parametrize("T,W,ff,E,top", [(1, 64, 24, 4, 2), (5, 101, 19, 3, 3), (9, 256, 96, 33, 1),
+@pytest.mark.parametrize("T,W,ff,E,top", [(1, 64, 24, 4, 2), (5, 101, 19, 3, 3), (9, 272, 112, 33, 1),
                                           (333, 264, 200, 7, 3), (1500, 128, 48, 40, 6)])
 def test_mixture_of_experts(T, W, ff, E, top, dtype):
     torch.manual_seed(E)
@@ -171,7 +171,7 @@ def _paged(c, lens, bs, R):
 
 @pytest.mark.parametrize("dtype", [BF16, F32])
 @pytest.mark.parametrize("H,R,bs,q_lens,kv_lens", [
-    (8, 64, 64, [1, 1, 1], [1, 64, 65]),
+    (9, 64, 64, [1, 1, 1], [1, 64, 65]),
     (5, 64, 16, [30, 1, 2], [30, 500, 129]),
     (12, 64, 64, [100], [300]),
     (1, 128, 16, [1, 3], [257, 128]),
@@ -220,7 +220,7 @@ def test_latent_attention(H, R, bs, q_lens, kv_lens, dtype):
 
 
 @pytest.mark.parametrize("splits", [1, 2, 5, 16])
-@pytest.mark.parametrize("H,R", [(8, 64), (16, 512), (24, 128)])
+@pytest.mark.parametrize("H,R", [(7, 64), (16, 512), (24, 128)])
 def test_latent_attention_does_not_depend_on_the_split(H, R, splits):
     torch.manual_seed(splits)
     lens = [1500, 130, 1]
