@@ -77,7 +77,9 @@ def kernel_sources() -> list[Path]:
 # use in a fresh checkout then compiles these files and leaves the others alone.
 KERNEL_SETS = {
     "Taralix": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm",
-                "latent_attention", "moe", "sampling", "stream"),
+                "latent_attention", "moe", "rotary", "sampling", "stream"),
+    "Zatirax": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm",
+                "latent_attention", "rotary", "sampling", "stream"),
 }
 _kernel_set: str | None = None
 

@@ -17,6 +17,7 @@ import argparse
 import dataclasses
 import json
 import logging
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Any, Optional
@@ -32,82 +33,238 @@ SHIFT_PARALLEL_THRESHOLD = 128
 
 
 @dataclass(frozen=True)
+class MaskSpec:
+    """Which earlier keys a token at position p sees, besides itself:
+
+    * ``causal``: all of them;
+    * ``window``: the ``size`` positions that end at p;
+    * ``chunk``: those with the same ``position // size``.
+    """
+    kind: str = "causal"
+    size: int = 0
+
+    @property
+    def code(self) -> int:
+        """The kernels' number of the kind (csrc/common/elem.cuh)."""
+        return {"causal": 0, "window": 1, "chunk": 2}[self.kind]
+
+    def first_key(self, pos):
+        """First position that ``pos`` (a number or an array) sees."""
+        if self.kind == "window":
+            return (pos - self.size + 1) * (pos >= self.size)
+        if self.kind == "chunk":
+            return pos // self.size * self.size
+        return pos * 0
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions over the first ``dims`` dimensions of a vector, dimension i paired with
+    i + dims / 2. ``scaling``: (factor, low, high, original), a context extension that divides the
+    frequencies whose wavelength exceeds original / low, keeps those below original / high and
+    interpolates between the two."""
+    base: float
+    dims: int
+    scaling: Optional[tuple] = None
+
+    def frequencies(self) -> list:
+        out = []
+        for i in range(self.dims // 2):
+            f = self.base ** (-2.0 * i / self.dims)
+            if self.scaling is not None:
+                factor, low, high, original = self.scaling
+                turns = original * f / (2.0 * math.pi)      # within the original context
+                if turns < low:
+                    f /= factor
+                elif turns <= high:
+                    s = (turns - low) / (high - low)
+                    f = (1.0 - s) * f / factor + s * f
+            out.append(f)
+        return out
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Attention whose keys and values are linear maps of one latent vector per token: only the
     latent (``kv_rank`` numbers) is cached. ``kv_from``: take the latents of that earlier layer
-    instead of projecting and caching some of one's own."""
+    instead of projecting and caching some of one's own. ``rot_dim`` > 0: every head has that many
+    further query dimensions, rotated by position, which meet one rotated key part that the heads
+    share and that is cached beside the latent."""
     heads: int
-    dim: int          # query / key dimensions per head
+    dim: int          # query / key dimensions per head (the unrotated ones)
     vdim: int         # value dimensions per head
     kv_rank: int
     scale: float      # factor of the scores
     kv_from: Optional[int] = None
+    rot_dim: int = 0
+    rotary: Optional[RotarySpec] = None
+    mask: MaskSpec = MaskSpec()
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Attention with cached keys and values, ``heads // kv_heads`` query heads to each of them."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rotary: Optional[RotarySpec] = None
+    mask: MaskSpec = MaskSpec()
+    qk_norm: bool = False       # RMS norm over dim of every query and key head, before rotation
+    sink: bool = False          # exp of a learned number per head in the softmax denominator
+    output_gate: bool = False   # heads' outputs times sigmoid of a projection of the layer's input
 
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
     """A gated feed-forward layer, or ``experts`` of them of which every token uses ``top``."""
     ff: int
-    act: str = "silu"     # silu | gelu_tanh
+    act: str = "silu"     # silu | gelu_tanh | clamped_swish (see ops.stream_ops.GATES)
     experts: int = 0      # 0: dense
     top: int = 0
+    limit: float = 0.0    # clamped_swish: bound of gate (above) and up (both sides)
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """One decoder layer of a model that lists its layers one by one."""
-    mixer: LatentAttentionSpec
+    mixer: Any            # LatentAttentionSpec | AttentionSpec
     mlp: Optional[FeedForwardSpec] = None
 
 
-def read_layer_specs(layers: list) -> tuple:
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers start .. stop - 1 run ``times`` times in a row with the same weights, each pass with
+    a cache of its own and a learned vector added to the stream before it."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayerListDesign:
+    """What the name of a layer-list architecture stands for, beyond the numbers of config.json.
+
+    ``residual``: where the norms are. "post": x <- norm(alpha * x + f(x)); "sandwich":
+    x <- x + norm_b(f(norm_a(x))). ``norm_offset``: added to the stored weights of the stream's
+    norms. ``masks``: kind of each mixer type's mask."""
+    residual: str
+    norm_offset: float
+    dense_act: str
+    mixers: tuple
+    feed_forwards: tuple
+    masks: dict = field(default_factory=dict)
+    qk_norm: bool = False
+    sink: bool = False
+    output_gate: bool = False
+
+
+LAYER_LIST_DESIGNS = {
+    "Taralix": LayerListDesign(residual="post", norm_offset=1.0, dense_act="gelu_tanh",
+                               mixers=("latent_attention",), feed_forwards=("dense", "moe")),
+    "Zatirax": LayerListDesign(residual="sandwich", norm_offset=0.0, dense_act="clamped_swish",
+                               mixers=("latent_attention", "attention"), feed_forwards=("dense",),
+                               masks={"latent_attention": "window", "attention": "chunk"},
+                               qk_norm=True, sink=True, output_gate=True),
+}
+
+
+def _read_rotary(d: Optional[dict]) -> Optional[RotarySpec]:
+    if d is None:
+        return None
+    s = d.get("scaling")
+    return RotarySpec(base=float(d["base"]), dims=int(d["dims"]),
+                      scaling=None if s is None else tuple(float(s[k]) for k in
+                                                           ("factor", "low", "high", "original")))
+
+
+def _read_mixer(kind: str, m: dict, design: LayerListDesign):
+    rotary, mask = _read_rotary(m.get("rot")), MaskSpec()
+    if m.get("mask") is not None:
+        mask = MaskSpec(design.masks[kind], int(m["mask"]["size"]))
+    shape = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                 scale=float(m["scale"]), rotary=rotary, mask=mask)
+    if kind == "attention":
+        return AttentionSpec(kv_heads=int(m["kv_heads"]), qk_norm=design.qk_norm,
+                             sink=design.sink, output_gate=design.output_gate, **shape)
+    src = m.get("kv_from")
+    return LatentAttentionSpec(kv_rank=int(m["kv_rank"]), rot_dim=int(m.get("rot_dim") or 0),
+                               kv_from=None if src is None else int(src), **shape)
+
+
+def read_layer_specs(layers: list, design: LayerListDesign) -> tuple:
     """The ``layers`` list of a layer-list checkpoint's config.json."""
     out = []
     for i, d in enumerate(layers):
-        if d.get("type") != "latent_attention":
-            raise NotImplementedError("layer %d: mixer type %r (supported: latent_attention)"
-                                      % (i, d.get("type")))
-        m = d["mixer"]
-        src = m.get("kv_from")
-        mixer = LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                                    kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
-                                    kv_from=None if src is None else int(src))
+        kind = d.get("type")
+        if kind not in design.mixers:
+            raise NotImplementedError("layer %d: mixer type %r (supported: %s)"
+                                      % (i, kind, ", ".join(design.mixers)))
+        mixer = _read_mixer(kind, d["mixer"], design)
         f, mlp = d.get("mlp"), None
         if f is not None:
             kind = f.get("kind")
+            if kind not in design.feed_forwards:
+                raise NotImplementedError("layer %d: feed-forward kind %r (supported: %s)"
+                                          % (i, kind, ", ".join(design.feed_forwards)))
             if kind == "dense":
-                mlp = FeedForwardSpec(ff=int(f["ff"]), act="gelu_tanh")
-            elif kind == "moe":
+                mlp = FeedForwardSpec(ff=int(f["ff"]), act=design.dense_act,
+                                      limit=float(f["limit"]) if "limit" in f else 0.0)
+            else:
                 mlp = FeedForwardSpec(ff=int(f["expert"]["ff"]), act="silu",
                                       experts=int(f["router"]["experts"]),
                                       top=int(f["router"]["top"]))
-            else:
-                raise NotImplementedError("layer %d: feed-forward kind %r (supported: dense, moe)"
-                                          % (i, kind))
         out.append(LayerSpec(mixer, mlp))
     return tuple(out)
 
 
-def validate_layer_specs(specs: tuple) -> None:
+def validate_layer_specs(specs: tuple, loop: Optional[LoopSpec] = None) -> None:
     for i, l in enumerate(specs):
         m, f = l.mixer, l.mlp
-        if min(m.heads, m.dim, m.vdim, m.kv_rank) < 1:
-            raise ValueError("layer %d: heads, dim, vdim and kv_rank must be positive" % i)
-        if m.kv_from is not None:
-            if not 0 <= m.kv_from < i:
-                raise ValueError("layer %d: kv_from must name an earlier layer" % i)
-            src = specs[m.kv_from].mixer
-            if src.kv_from is not None or src.kv_rank != m.kv_rank:
-                raise ValueError("layer %d: layer %d has no latents of this kv_rank of its own"
-                                 % (i, m.kv_from))
+        if min(m.heads, m.dim, m.vdim) < 1:
+            raise ValueError("layer %d: heads, dim and vdim must be positive" % i)
+        if m.mask.kind != "causal" and m.mask.size < 1:
+            raise ValueError("layer %d: a %s of %d positions" % (i, m.mask.kind, m.mask.size))
+        if m.rotary is not None and (m.rotary.dims % 2 or m.rotary.dims < 0):
+            raise ValueError("layer %d: rot.dims must be even" % i)
+        if isinstance(m, AttentionSpec):
+            if m.kv_heads < 1 or m.heads % m.kv_heads:
+                raise ValueError("layer %d: heads must be a multiple of kv_heads" % i)
+            if m.rotary is not None and m.rotary.dims > m.dim:
+                raise ValueError("layer %d: rot.dims exceeds dim" % i)
+        else:
+            if m.kv_rank < 1:
+                raise ValueError("layer %d: kv_rank must be positive" % i)
+            if m.rot_dim and (m.rotary is None or m.rotary.dims != m.rot_dim):
+                raise ValueError("layer %d: rot.dims must equal rot_dim" % i)
+            if m.kv_from is not None and m.rot_dim:
+                raise NotImplementedError("layer %d: shared latents with a rotated key part" % i)
+            if m.kv_from is not None:
+                if not 0 <= m.kv_from < i:
+                    raise ValueError("layer %d: kv_from must name an earlier layer" % i)
+                src = specs[m.kv_from].mixer
+                if getattr(src, "kv_rank", None) != m.kv_rank or src.kv_from is not None or \
+                        src.rot_dim:
+                    raise ValueError("layer %d: layer %d has no latents of this kv_rank of its own"
+                                     % (i, m.kv_from))
         if f is not None and f.experts and not 1 <= f.top <= f.experts:
             raise ValueError("layer %d: top must lie between 1 and the number of experts" % i)
+        if f is not None and f.act == "clamped_swish" and not f.limit > 0:
+            raise ValueError("layer %d: the feed-forward's limit must be positive" % i)
+    if loop is not None:
+        if not (0 <= loop.start < loop.stop <= len(specs) and loop.times >= 1):
+            raise ValueError("loop: 0 <= start < stop <= layers and times >= 1 are needed")
+        for i in range(len(specs)):
+            src = getattr(specs[i].mixer, "kv_from", None)
+            if src is not None and (loop.start <= src < loop.stop or loop.start <= i < loop.stop):
+                raise NotImplementedError("layer %d: shared latents inside a loop" % i)
 
 
 @dataclass
 class ModelConfig:
     """Architecture of a decoder (Llama, Mistral, Qwen2 and Qwen3 dense models, optionally
-    SwiftKV for Llama; Taralix, which lists its layers one by one) or encoder (BERT)."""
+    SwiftKV for Llama; Taralix and Zatirax, which list their layers one by one) or encoder (BERT)."""
 
     architecture: str = "LlamaForCausalLM"
     model_type: str = "llama"
@@ -139,6 +296,8 @@ class ModelConfig:
     layer_specs: Optional[tuple] = None
     # factor of the residual stream in "norm after the sum" layers: x <- norm(alpha * x + f(x))
     postln_alpha: float = 1.0
+    embedding_scale: float = 1.0
+    loop: Optional[LoopSpec] = None
     # encoder-only fields
     type_vocab_size: int = 2
     layer_norm_eps: float = 1e-12
@@ -196,7 +355,7 @@ class ModelConfig:
 
     def validate(self) -> None:
         if self.layer_specs is not None:
-            validate_layer_specs(self.layer_specs)
+            validate_layer_specs(self.layer_specs, self.loop)
             if self.quantization is not None:
                 raise NotImplementedError("quantization=%r for %s" % (self.quantization,
                                                                       self.architecture))
@@ -267,24 +426,47 @@ class ModelConfig:
 
     @classmethod
     def from_layer_list(cls, d: dict, name_or_path: str = "") -> "ModelConfig":
-        """config.json of a layer-list model (``architecture``, ``width``, ``vocab``, ``norm``,
-        ``postln_alpha`` and ``layers``). The head fields describe the cache as the engine sees
-        it: one latent "head" of ``kv_rank`` numbers (the largest, where layers differ)."""
-        specs = read_layer_specs(d["layers"])
+        """config.json of a layer-list model (``architecture``, ``width``, ``vocab``, ``norm`` and
+        ``layers``; by design ``postln_alpha``, ``embedding.scale``, ``loop``). The head fields
+        describe the cache as the engine sees it: one "head" of as many numbers as the widest
+        layer keeps per token."""
+        design = LAYER_LIST_DESIGNS[d["architecture"]]
+        specs = read_layer_specs(d["layers"], design)
         if not specs:
             raise ValueError("a model without layers")
-        eos = d.get("eos_token_id")
+        kept = lambda m: m.kv_heads * (m.dim + m.vdim) if isinstance(m, AttentionSpec) else \
+            m.kv_rank + m.rot_dim
+        eos, loop = d.get("eos_token_id"), d.get("loop")
         return cls(
             architecture=d["architecture"], model_type=d["architecture"].lower(),
             hidden_size=int(d["width"]), num_hidden_layers=len(specs),
             num_attention_heads=max(l.mixer.heads for l in specs), num_key_value_heads=1,
-            head_dim=max(l.mixer.kv_rank for l in specs),
+            head_dim=max(kept(l.mixer) for l in specs),
             intermediate_size=max((l.mlp.ff for l in specs if l.mlp is not None), default=0),
             vocab_size=int(d["vocab"]), rms_norm_eps=float(d["norm"]["eps"]),
-            postln_alpha=float(d["postln_alpha"]), layer_specs=specs,
-            # nothing in the model depends on a position's number, so nothing bounds it
+            postln_alpha=float(d["postln_alpha"]) if design.residual == "post" else 1.0,
+            embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+            loop=None if not loop else LoopSpec(int(loop["start"]), int(loop["stop"]),
+                                                int(loop["times"])),
+            layer_specs=specs,
+            # no table is indexed by position, so nothing bounds it
             max_position_embeddings=1 << 20, hidden_act="",
             eos_token_id=int(eos) if isinstance(eos, int) else None, name_or_path=name_or_path)
+
+    @property
+    def design(self) -> LayerListDesign:
+        return LAYER_LIST_DESIGNS[self.architecture]
+
+    @property
+    def layer_runs(self) -> list:
+        """(layer, pass of the loop or None) in the order of execution of a layer-list model; the
+        pass is named at its first layer only."""
+        order = list(range(len(self.layer_specs)))
+        if self.loop is None:
+            return [(l, None) for l in order]
+        lo, hi, n = self.loop.start, self.loop.stop, self.loop.times
+        body = [(l, t if l == lo else None) for t in range(n) for l in order[lo:hi]]
+        return [(l, None) for l in order[:lo]] + body + [(l, None) for l in order[hi:]]
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
@@ -314,7 +496,7 @@ class ModelConfig:
 DECODER_MODEL_TYPES = ("llama", "llama_swiftkv", "mistral", "qwen2", "qwen3")
 
 # models whose config.json lists the layers instead of giving one shape for all of them
-LAYER_LIST_ARCHITECTURES = ("Taralix",)
+LAYER_LIST_ARCHITECTURES = tuple(LAYER_LIST_DESIGNS)
 
 
 def _taralix(width, vocab, layers, alpha, eps=1e-6) -> ModelConfig:
@@ -334,6 +516,17 @@ def _taralix(width, vocab, layers, alpha, eps=1e-6) -> ModelConfig:
     return ModelConfig.from_layer_list({"architecture": "Taralix", "width": width, "vocab": vocab,
                                         "norm": {"eps": eps}, "postln_alpha": alpha,
                                         "layers": out})
+
+
+def _zatirax(width, vocab, layers, loop, scale=1.0, eps=1e-6) -> ModelConfig:
+    """``layers``: (mixer, ff) each; a mixer with ``kv_heads`` is ordinary attention."""
+    out = [{"type": "attention" if "kv_heads" in m else "latent_attention", "mixer": m,
+            "mlp": None if ff is None else {"kind": "dense", "ff": ff, "limit": 7.0}}
+           for m, ff in layers]
+    return ModelConfig.from_layer_list({
+        "architecture": "Zatirax", "width": width, "vocab": vocab, "norm": {"eps": eps},
+        "embedding": {"scale": scale}, "layers": out,
+        "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop))})
 
 
 def _llama(layers, hidden, heads, kv, inter, **kw) -> ModelConfig:
@@ -404,6 +597,14 @@ PRESETS: dict[str, ModelConfig] = {
                              max_position_embeddings=512, hidden_act="gelu"),
     "taralix-tiny": _taralix(192, 1024, [(6, 32, 48, 96, None, 320), (4, 64, 32, 96, 0, (64, 8, 3)),
                                          (5, 40, 64, 40, None, None)], alpha=1.7),
+    "zatirax-tiny": _zatirax(192, 1024, [
+        ({"heads": 5, "dim": 40, "vdim": 48, "kv_rank": 72, "rot_dim": 24, "scale": 0.15,
+          "mask": {"size": 90}, "rot": {"base": 10000.0, "dims": 24}}, 320),
+        ({"heads": 6, "kv_heads": 2, "dim": 64, "vdim": 48, "scale": 0.125, "mask": {"size": 150},
+          "rot": {"base": 10000.0, "dims": 48, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0,
+                                                           "original": 512}}}, 256),
+        ({"heads": 4, "dim": 32, "vdim": 32, "kv_rank": 48, "rot_dim": 16, "scale": 0.2,
+          "mask": {"size": 33}, "rot": {"base": 5000.0, "dims": 16}}, None)], loop=(1, 3, 2)),
 }
 
 

@@ -107,6 +107,13 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
                     long long T, int Hq, int Hkv, int D, int causal, float scale, void* out,
                     long long ldo, void* o_part, void* lse_part, void* lse_out, int tile_keys,
                     int* status, cudaStream_t stream);
+int ab200_attention_ext(const void* q, long long ldq, const void* k, const void* v, long long ld_kv,
+                        long long num_blocks, int block_size, const void* block_tables,
+                        int max_blocks, const void* work, int num_work, const void* tok_splits,
+                        int max_splits, long long T, int Hq, int Hkv, int D, int mask_kind,
+                        int mask_size, const void* sink, const void* gate, long long ldg,
+                        float scale, void* out, long long ldo, void* o_part, void* lse_part,
+                        int tile_keys, int* status, cudaStream_t stream);
 int ab200_attention_merge(const void* o_part, const void* lse_part, const void* tok_splits,
                           long long T, int Hq, int D, void* out, long long ldo,
                           cudaStream_t stream);
@@ -230,28 +237,44 @@ int ab200_argmax_exchange(const void* ids, const void* vals, int B, int max_rows
                           cudaStream_t stream);
 
 // ---- stream.cu (dtype: 0 = bf16, 1 = fp32 elements; the residual stream is always fp32)
-int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, long long T,
-                           int W, long long vocab, int dtype, int* status, cudaStream_t stream);
+int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, float scale,
+                           long long T, int W, long long vocab, int dtype, int* status, cudaStream_t stream);
 int ab200_stream_norm(const void* x, const void* rows, const void* y, long long ldy,
                       const void* y_rows, const void* y_weights, int top, const void* weight,
-                      float alpha, float eps, void* x_out, void* act_out, long long T, int W,
-                      int dtype, cudaStream_t stream);
+                      float alpha, float eps, float offset, void* x_out, void* act_out,
+                      long long T, int W, int dtype, cudaStream_t stream);
+int ab200_stream_sandwich(void* x, const void* y, long long ldy, const void* w_out, const void* step,
+                          const void* w_in, void* act, float eps, float offset, long long T, int W,
+                          int dtype, cudaStream_t stream);
 int ab200_latent_norm_cache(const void* ckv, long long ld, const void* weight, int R, int Rp,
                             float eps, const void* slots, void* cache, long long num_slots,
                             long long T, int dtype, int* status, cudaStream_t stream);
-int ab200_gated_act(const void* gu, void* out, long long T, int ff, int act, int dtype,
-                    cudaStream_t stream);
+int ab200_gated_act(const void* gu, void* out, long long T, int ff, int act, float limit,
+                    float alpha, int dtype, cudaStream_t stream);
 
 // ---- exact.cu
 int ab200_linear_exact(const void* x, long long ldx, long long x_gstride, const void* w,
                        long long ldw, long long w_gstride, void* out, long long ldo,
                        long long out_gstride, int M, int N, int K, int groups, const void* tiles,
                        const void* num_tiles, int max_tiles, int dtype, cudaStream_t stream);
-int ab200_latent_attention_exact(const void* q, long long ldq, const void* cache, int num_blocks,
-                                 int block_size, const void* block_tables, int max_blocks,
-                                 const void* tok_seq, const void* positions, void* out,
-                                 long long ldo, long long T, int H, int R, float scale, int dtype,
-                                 int* status, cudaStream_t stream);
+int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row, const void* v,
+                          int v_row, int num_blocks, int block_size, const void* block_tables,
+                          int max_blocks, const void* tok_seq, const void* positions,
+                          const void* sink, const void* gate, long long ldg, void* out,
+                          long long ldo, long long T, int H, int Hkv, int Dk, int Dv, int mask_kind,
+                          int mask_size, float scale, int dtype, int* status, cudaStream_t stream);
+
+// ---- rotary.cu
+int ab200_head_rope_cache(void* proj, long long ld, const void* positions, const void* slots,
+                          const void* wq, const void* wk, const void* freq, int half, void* k_cache,
+                          void* v_cache, long long T, int Hq, int Hkv, int D, int dim, int Dv,
+                          int block_size, long long num_slots, float eps, int dtype, int* status,
+                          cudaStream_t stream);
+int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* positions,
+                            const void* slots, const void* weight, const void* freq, int half,
+                            void* cache, long long T, int H, int dq, int dim, int R, int width,
+                            int rot_at, long long num_slots, float eps, int dtype, int* status,
+                            cudaStream_t stream);
 
 // ---- moe.cu
 int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,
@@ -264,15 +287,16 @@ int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, 
 int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long long x_rows,
                        const void* w, long long ldw, long long w_gstride, void* out, long long ldo,
                        long long out_gstride, int M, int N, int K, int groups, const void* tiles,
-                       const void* num_tiles, int max_tiles, int act, int* status,
-                       cudaStream_t stream);
+                       const void* num_tiles, int max_tiles, int act, float act_limit,
+                       float act_alpha, int* status, cudaStream_t stream);
 
 // ---- latent_attention.cu
 int ab200_latent_attention(const void* q, long long q_rows, const void* cache, int num_blocks,
                            int block_size, const void* block_tables, int max_blocks,
                            const void* work, int num_work, const void* tok_splits, int max_splits,
-                           long long T, int H, int R, int tile_rows, float scale, void* out,
-                           void* o_part, void* lse_part, int* status, cudaStream_t stream);
+                           long long T, int H, int R, int key_extra, int mask_kind, int mask_size,
+                           int tile_rows, float scale, void* out, void* o_part, void* lse_part,
+                           int* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -20,6 +20,12 @@
 // footprint (112 KB of shared memory, 256 TMEM columns, < 170 registers) lets two
 // CTAs share an SM and overlap one CTA's softmax with the other's loads.
 //
+// Instances with EXT also take a mask with a lower bound (a window, or chunks of positions: the
+// planner starts a tile's keys at the first one its rows see, the softmax masks the rest), a
+// learned sink per head in the denominator (added once, at the end) and an output gate (the
+// normalised rows times sigmoid of a projection, as they are stored). With split keys the merge
+// kernel adds the sink and applies the gate.
+//
 // K/V come either from a paged cache [num_blocks, Hkv, block_size, D] through a
 // block table (one TMA box per block) or from a contiguous [T, Hkv*D]-strided
 // tensor (encoder). With several KV splits per sequence each CTA writes a
@@ -34,6 +40,7 @@
 #include <string.h>
 
 #include "api.h"
+#include "common/elem.cuh"
 #include "common/pdl.cuh"
 #include "common/peer.cuh"
 #include "common/ptx.cuh"
@@ -75,6 +82,12 @@ struct AttnArgs {
   // row t % peer_tokens (the pointers already include this rank's column offset).
   int peer_tokens;
   __nv_bfloat16* peer_out[16];
+  // EXT instances: mask (first_visible), sink per query head [Hq] and output gate [T][ldg], the
+  // columns laid out like out's
+  int mask_kind, mask_size;
+  const float* sink;
+  const __nv_bfloat16* gate;
+  long long ldg;
   // completion signal to every rank once the last block has stored its rows (common/peer.cuh);
   // with split-KV the merge kernel sends it instead
   TailSignal sig;
@@ -86,7 +99,22 @@ struct AttnArgs {
 //  6 split index   7 number of splits of this sequence
 //  In contiguous mode field 0 is the row of the sequence's first key in the K/V tensor.
 
-template <int D, int TK>
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
+// eight bf16 values times the sigmoids of eight others
+__device__ __forceinline__ uint4 gate8(const uint4& v, const uint4& g) {
+  const uint32_t a[4] = {v.x, v.y, v.z, v.w}, b[4] = {g.x, g.y, g.z, g.w};
+  uint32_t r[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[i]));
+    const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&b[i]));
+    r[i] = pack_bf16x2(x.x * sigmoid_fast(y.x), x.y * sigmoid_fast(y.y));
+  }
+  return make_uint4(r[0], r[1], r[2], r[3]);
+}
+
+template <int D, int TK, bool EXT>
 __global__ void __launch_bounds__(AttnShape<TK>::kThreads, (TK == 64 ? 2 : 1))
 attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const AttnArgs p) {
@@ -344,6 +372,8 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     const bool valid_row = tok_local < n_q_tok && g < p.g_heads;
     const int q_pos = q_pos0 + tok_local;
     const int limit = p.causal ? min(q_pos, kv_end - 1) : kv_end - 1;  // last visible key
+    // first visible key (EXT only)
+    const int lower = EXT ? first_visible(p.mask_kind, p.mask_size, q_pos) : 0;
     const uint32_t lane_off = (uint32_t)(quad * 32) << 16;
     float m = -INFINITY;
     float l = 0.f;
@@ -379,7 +409,8 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
       }
       tc_fence_after();
       const uint32_t ts = tS + (uint32_t)st * TK + lane_off;
-      const bool need_mask = key0 + TK - 1 > limit;
+      const bool need_mask = key0 + TK - 1 > limit || (EXT && key0 < lower);
+      auto sees = [&](int k) { return k <= limit && (!EXT || k >= lower); };
       uint32_t ra[32], rb[32];
       // pass 1: row maximum (four independent chains; one warp per scheduler cannot hide a
       // long dependent chain). TMEM reads are software-pipelined.
@@ -397,10 +428,10 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
 #pragma unroll
           for (int t = 0; t < 32; t += 4) {
             const int k = key0 + c * 32 + t;
-            mx0 = fmaxf(mx0, k + 0 <= limit ? __uint_as_float(cur[t + 0]) : -INFINITY);
-            mx1 = fmaxf(mx1, k + 1 <= limit ? __uint_as_float(cur[t + 1]) : -INFINITY);
-            mx2 = fmaxf(mx2, k + 2 <= limit ? __uint_as_float(cur[t + 2]) : -INFINITY);
-            mx3 = fmaxf(mx3, k + 3 <= limit ? __uint_as_float(cur[t + 3]) : -INFINITY);
+            mx0 = fmaxf(mx0, sees(k + 0) ? __uint_as_float(cur[t + 0]) : -INFINITY);
+            mx1 = fmaxf(mx1, sees(k + 1) ? __uint_as_float(cur[t + 1]) : -INFINITY);
+            mx2 = fmaxf(mx2, sees(k + 2) ? __uint_as_float(cur[t + 2]) : -INFINITY);
+            mx3 = fmaxf(mx3, sees(k + 3) ? __uint_as_float(cur[t + 3]) : -INFINITY);
           }
         } else {
 #pragma unroll
@@ -481,10 +512,10 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
           float e3 = ex2_approx(fmaf(__uint_as_float(cur[t + 3]), sc, neg_ms));
           if (need_mask) {
             const int k = key0 + c * 32 + t;
-            e0 = k + 0 <= limit ? e0 : 0.f;
-            e1 = k + 1 <= limit ? e1 : 0.f;
-            e2 = k + 2 <= limit ? e2 : 0.f;
-            e3 = k + 3 <= limit ? e3 : 0.f;
+            e0 = sees(k + 0) ? e0 : 0.f;
+            e1 = sees(k + 1) ? e1 : 0.f;
+            e2 = sees(k + 2) ? e2 : 0.f;
+            e3 = sees(k + 3) ? e3 : 0.f;
           }
           s0 += e0;
           s1 += e1;
@@ -533,9 +564,12 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
       else l += *reinterpret_cast<volatile float*>(&sums[(half ^ 1) * 128 + row]);
     }
     if (ok && warp_active) {  // warp-uniform: every lane takes part in the TMEM reads
-      const float inv_l = l > 0.f ? 1.f / l : 0.f;
       const long long tok = (long long)q_tok0 + tok_local;
       const int head = kvh * p.g_heads + g;
+      // (split keys: the merge adds the sink, once)
+      if (EXT && p.sink != nullptr && num_splits <= 1 && valid_row && l > 0.f)
+        l += ex2_approx(p.sink[head] * 1.4426950408889634f - m * sc);
+      const float inv_l = l > 0.f ? 1.f / l : 0.f;
       const float lse = l > 0.f ? m * p.scale + logf(l) : -INFINITY;
       __nv_bfloat16* dst16 = p.out + tok * p.ldo + (long long)head * D;
       if (p.peer_tokens > 0)
@@ -581,8 +615,12 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
           const int rr = quad * 32 + rl;
           const unsigned long long d = __shfl_sync(0xffffffffu, my_dst, rl);
           if (d != 0ull) {
-            const uint4 q = *reinterpret_cast<const uint4*>(
+            uint4 q = *reinterpret_cast<const uint4*>(
                 smem + (size_t)(j >> 3) * 16384 + (size_t)rr * 128 + (((j & 7) ^ (rr & 7)) * 16));
+            if (EXT && p.gate != nullptr)
+              q = gate8(q, *reinterpret_cast<const uint4*>(
+                               p.gate + (long long)(q_tok0 + rr / p.G) * p.ldg +
+                               (long long)(kvh * p.g_heads + rr % p.G) * D + 8 * j));
             *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(d) + 8 * j) = q;
           }
         }
@@ -641,7 +679,7 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
 
 // Fold split-KV partials: out = sum_s w_s O_s / sum_s w_s, w_s = exp(lse_s - max lse).
 // tok_splits[t] = number of splits that cover token t (<= 1: nothing to do).
-template <int D>
+template <int D, bool EXT>
 __global__ void attention_merge_kernel(const float* __restrict__ o_part,
                                        const float* __restrict__ lse_part,
                                        const int* __restrict__ tok_splits, long long T, int Hq,
@@ -665,8 +703,13 @@ __global__ void attention_merge_kernel(const float* __restrict__ o_part,
     const int d4 = (idx % (D / 4)) * 4;
     float mx = -INFINITY;
     for (int s = 0; s < ns; ++s) mx = fmaxf(mx, lse_part[((long long)s * T + tok) * Hq + head]);
+    float sink = -INFINITY;
+    if (EXT && pa.sink != nullptr) {
+      sink = pa.sink[head];
+      mx = fmaxf(mx, sink);
+    }
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    float wsum = 0.f;
+    float wsum = (EXT && sink != -INFINITY) ? __expf(sink - mx) : 0.f;
     for (int s = 0; s < ns; ++s) {
       const float lse = lse_part[((long long)s * T + tok) * Hq + head];
       const float w = (lse == -INFINITY) ? 0.f : __expf(lse - mx);
@@ -679,6 +722,13 @@ __global__ void attention_merge_kernel(const float* __restrict__ o_part,
       wsum += w;
     }
     const float inv = wsum > 0.f ? 1.f / wsum : 0.f;
+    if (EXT && pa.gate != nullptr) {
+      const float4 g = load4(pa.gate + tok * pa.ldg + (long long)head * D + d4);
+      acc.x *= sigmoid_fast(g.x);
+      acc.y *= sigmoid_fast(g.y);
+      acc.z *= sigmoid_fast(g.z);
+      acc.w *= sigmoid_fast(g.w);
+    }
     uint2 q;
     q.x = pack_bf16x2(acc.x * inv, acc.y * inv);
     q.y = pack_bf16x2(acc.z * inv, acc.w * inv);
@@ -688,7 +738,14 @@ __global__ void attention_merge_kernel(const float* __restrict__ o_part,
   tail_signal(pa.sig, gridDim.x);
 }
 
-template <int D, int TK>
+struct AttnExt {
+  int mask_kind, mask_size;
+  const void* sink;
+  const void* gate;
+  long long ldg;
+};
+
+template <int D, int TK, bool EXT>
 static int launch_attention(const void* q, long long ldq, const void* k, const void* v,
                             long long ld_kv, long long num_blocks, int block_size,
                             const int* block_tables, int max_blocks, const int* work, int num_work,
@@ -696,7 +753,8 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
                             int causal, float scale, void* out, long long ldo, float* o_part,
                             float* lse_part, float* lse_out, int* status, cudaStream_t stream,
                             const void* const* peer_ptrs = nullptr, int world = 0,
-                            int peer_tokens = 0, const Ab200PeerSync* sync = nullptr) {
+                            int peer_tokens = 0, const Ab200PeerSync* sync = nullptr,
+                            const AttnExt* ext = nullptr) {
   const int heads = Hq / Hkv;
   int G = 1;
   while (G < heads) G *= 2;
@@ -710,7 +768,7 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   const size_t smem =
       128 * D * 2 + 4 * (size_t)TK * D * 2 + (TK == 128 ? 2 : 1) * (size_t)128 * TK * 2 + 256;
   if (!attr_set[dev]) {
-    if (cudaFuncSetAttribute(attention_kernel<D, TK>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attention_kernel<D, TK, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)smem) != cudaSuccess)
       return -3;
     attr_set[dev] = true;
@@ -761,6 +819,13 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   a.lse_out = lse_out;
   a.T = T;
   a.status = status;
+  if (EXT) {
+    a.mask_kind = ext->mask_kind;
+    a.mask_size = ext->mask_size;
+    a.sink = reinterpret_cast<const float*>(ext->sink);
+    a.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);
+    a.ldg = ext->ldg;
+  }
   TailSignal sig;
   memset(&sig, 0, sizeof(sig));
   if (sync != nullptr && sync->sig_world > 0) {
@@ -774,12 +839,12 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   }
   if (max_splits <= 1) a.sig = sig;
   dim3 grid((unsigned)num_work * (unsigned)Hkv);
-  (void)launch_pdl(attention_kernel<D, TK>, grid, dim3(AttnShape<TK>::kThreads), smem, stream, tq,
+  (void)launch_pdl(attention_kernel<D, TK, EXT>, grid, dim3(AttnShape<TK>::kThreads), smem, stream, tq,
                    tk, tv, a);
   if (cudaGetLastError() != cudaSuccess) return -5;
   a.sig = sig;
   if (max_splits > 1) {
-    (void)launch_pdl(attention_merge_kernel<D>, dim3((unsigned)T), dim3(128), 0, stream, o_part,
+    (void)launch_pdl(attention_merge_kernel<D, EXT>, dim3((unsigned)T), dim3(128), 0, stream, o_part,
                      lse_part, tok_splits, T, Hq, reinterpret_cast<__nv_bfloat16*>(out), ldo,
                      lse_out, a);
     if (cudaGetLastError() != cudaSuccess) return -5;
@@ -793,13 +858,13 @@ using namespace ab200;
 
 extern "C" {
 
-#define AB200_ATTN_DISPATCH(...)                                                       \
+#define AB200_ATTN_DISPATCH(EXT, ...)                                                     \
   do {                                                                                 \
     const bool small = tile_keys == 64 && (block_size == 0 || block_size <= 64);        \
-    if (D == 128) return small ? launch_attention<128, 64>(__VA_ARGS__)                \
-                               : launch_attention<128, 128>(__VA_ARGS__);              \
-    if (D == 64) return small ? launch_attention<64, 64>(__VA_ARGS__)                  \
-                              : launch_attention<64, 128>(__VA_ARGS__);                \
+    if (D == 128) return small ? launch_attention<128, 64, EXT>(__VA_ARGS__)                \
+                               : launch_attention<128, 128, EXT>(__VA_ARGS__);              \
+    if (D == 64) return small ? launch_attention<64, 64, EXT>(__VA_ARGS__)                  \
+                              : launch_attention<64, 128, EXT>(__VA_ARGS__);                \
     return -2;                                                                         \
   } while (0)
 
@@ -818,12 +883,37 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
   if (num_work <= 0 || T <= 0) return 0;
   if ((ldq % 8) || (ldo % 8) || (ld_kv % 8)) return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
-  AB200_ATTN_DISPATCH(q, ldq, k, v, ld_kv, num_blocks, block_size,
+  AB200_ATTN_DISPATCH(false, q, ldq, k, v, ld_kv, num_blocks, block_size,
                       reinterpret_cast<const int*>(block_tables), max_blocks,
                       reinterpret_cast<const int*>(work), num_work,
                       reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, causal, scale,
                       out, ldo, reinterpret_cast<float*>(o_part), reinterpret_cast<float*>(lse_part),
                       reinterpret_cast<float*>(lse_out), status, stream);
+}
+
+// The same with a mask (0 causal, 1 window, 2 chunk, see first_visible), an optional sink per query
+// head (fp32 [Hq]) and an optional output gate (bf16 rows of stride ldg, columns like out's).
+// Always causal; the work list's kv_start must not lie above the first key a tile's rows see.
+int ab200_attention_ext(const void* q, long long ldq, const void* k, const void* v, long long ld_kv,
+                        long long num_blocks, int block_size, const void* block_tables,
+                        int max_blocks, const void* work, int num_work, const void* tok_splits,
+                        int max_splits, long long T, int Hq, int Hkv, int D, int mask_kind,
+                        int mask_size, const void* sink, const void* gate, long long ldg,
+                        float scale, void* out, long long ldo, void* o_part, void* lse_part,
+                        int tile_keys, int* status, cudaStream_t stream) {
+  if (num_work <= 0 || T <= 0) return 0;
+  if ((ldq % 8) || (ldo % 8) || (ld_kv % 8)) return -2;
+  if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
+    return -2;
+  if (gate != nullptr && ((ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -2;
+  if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
+  const AttnExt ext = {mask_kind, mask_size, sink, gate, ldg};
+  AB200_ATTN_DISPATCH(true, q, ldq, k, v, ld_kv, num_blocks, block_size,
+                      reinterpret_cast<const int*>(block_tables), max_blocks,
+                      reinterpret_cast<const int*>(work), num_work,
+                      reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, 1, scale,
+                      out, ldo, reinterpret_cast<float*>(o_part), reinterpret_cast<float*>(lse_part),
+                      nullptr, status, stream, nullptr, 0, 0, nullptr, &ext);
 }
 
 // Folds split-KV partials of another attention kernel (same layouts as above): o_part fp32
@@ -833,10 +923,10 @@ int ab200_attention_merge(const void* o_part, const void* lse_part, const void* 
                           cudaStream_t stream) {
   AttnArgs a;
   memset(&a, 0, sizeof(a));
-  auto k = D == 128   ? attention_merge_kernel<128>
-           : D == 256 ? attention_merge_kernel<256>
-           : D == 384 ? attention_merge_kernel<384>
-                      : attention_merge_kernel<512>;
+  auto k = D == 128   ? attention_merge_kernel<128, false>
+           : D == 256 ? attention_merge_kernel<256, false>
+           : D == 384 ? attention_merge_kernel<384, false>
+                      : attention_merge_kernel<512, false>;
   if (D != 128 && D != 256 && D != 384 && D != 512) return -2;
   return launch_pdl(k, dim3((unsigned)T), dim3(D >= 256 ? 256 : 128), 0, stream,
                     reinterpret_cast<const float*>(o_part), reinterpret_cast<const float*>(lse_part),
@@ -874,7 +964,7 @@ int ab200_attention_scatter_sync(const void* q, long long ldq, const void* k, co
   if (num_work <= 0 || T <= 0) return 0;
   if ((ldq % 8) || (ldo % 8) || peer_tokens <= 0) return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
-  AB200_ATTN_DISPATCH(q, ldq, k, v, 0, num_blocks, block_size,
+  AB200_ATTN_DISPATCH(false, q, ldq, k, v, 0, num_blocks, block_size,
                       reinterpret_cast<const int*>(block_tables), max_blocks,
                       reinterpret_cast<const int*>(work), num_work,
                       reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, 1, scale,

@@ -55,15 +55,34 @@ __device__ __forceinline__ float block_max_all(float v, float* red) {
   return warp_max(lane < nwarps ? red[lane] : -INFINITY);
 }
 
-enum GatedAct : int { kActSilu = 1, kActGeluTanh = 2 };
+// Gated activations: silu(g) * u, gelu_tanh(g) * u, and the clamped swish
+// min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1).
+enum GatedAct : int { kActSilu = 1, kActGeluTanh = 2, kActClampedSwish = 3 };
+
+struct GateParams {
+  float limit, alpha;   // of the clamped swish
+};
 
 __device__ __forceinline__ float gate_silu(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float gate_gelu_tanh(float z) {
   const float k = 0.79788456080286535588f;   // sqrt(2 / pi)
   return 0.5f * z * (1.f + tanhf(k * (z + 0.044715f * z * z * z)));
 }
-__device__ __forceinline__ float gate_act(int act, float z) {
-  return act == kActSilu ? gate_silu(z) : gate_gelu_tanh(z);
+__device__ __forceinline__ float gated(int act, const GateParams& p, float g, float u) {
+  if (act == kActClampedSwish) {
+    g = fminf(g, p.limit);
+    return g / (1.f + expf(-p.alpha * g)) * (fminf(fmaxf(u, -p.limit), p.limit) + 1.f);
+  }
+  return (act == kActSilu ? gate_silu(g) : gate_gelu_tanh(g)) * u;
+}
+
+// Which keys a token at position `pos` sees: first_visible .. pos.
+enum MaskKind : int { kMaskCausal = 0, kMaskWindow = 1, kMaskChunk = 2 };
+
+__host__ __device__ __forceinline__ int first_visible(int kind, int size, int pos) {
+  if (kind == kMaskWindow) return pos >= size ? pos - size + 1 : 0;
+  if (kind == kMaskChunk) return pos / size * size;
+  return 0;
 }
 
 // Gate and up projections are stored as one matrix whose rows alternate in blocks of this many:

@@ -4,8 +4,9 @@
 //
 //   linear_exact            out[g] = x[g] * w[g]^T: one matrix, one per group (heads), or one per
 //                           expert over rows sorted by expert (a device-side tile list)
-//   latent_attention_exact  softmax attention over the paged latent cache, a block per
-//                           (token, head), keys in tiles with a running maximum
+//   attention_exact         softmax attention over a paged cache (keys and values, or one latent
+//                           row that is both), with a mask, a sink and an output gate, a block
+//                           per (token, head), keys in tiles with a running maximum
 //
 // Every product and sum is IEEE fp32 (FMA); no reduced-precision mode is involved.
 
@@ -96,23 +97,30 @@ __global__ void __launch_bounds__(256) linear_exact_kernel(const ExactArgs p) {
 constexpr int kAttnKeys = 128;
 
 struct ExactAttnArgs {
-  const void* q;
+  const void* q;            // [T][ldq], head h at column h * Dk
   long long ldq;
-  const void* cache;        // [num_blocks * block_size][R]
+  // cache row of (block, kv head, offset): ((block * Hkv + head) * block_size + offset) * row
+  const void* k;
+  const void* v;
+  int k_row, v_row;
   const int* block_tables;
   int max_blocks, block_size;
   const int* tok_seq;       // [T] sequence (row of block_tables) of each token
   const long long* positions;
-  void* out;
+  const float* sink;        // [H] or null
+  const void* gate;         // [T][ldg], head h at column h * Dv, or null
+  long long ldg;
+  void* out;                // [T][ldo], head h at column h * Dv
   long long ldo;
-  int H, R, num_blocks;
+  int H, Hkv, Dk, Dv, num_blocks;
+  int mask_kind, mask_size;
   float scale;
   int* status;
 };
 
-// Shared memory: q[R], the tile's cache rows' offsets, the tile's weights, the accumulator[R].
+// Shared memory: q[Dk], the accumulator[Dv]; the tile's cache rows and weights.
 template <typename T>
-__global__ void __launch_bounds__(kAttnKeys) latent_attention_exact_kernel(const ExactAttnArgs p) {
+__global__ void __launch_bounds__(kAttnKeys) attention_exact_kernel(const ExactAttnArgs p) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) float sm[];
@@ -120,20 +128,21 @@ __global__ void __launch_bounds__(kAttnKeys) latent_attention_exact_kernel(const
   __shared__ float pw[kAttnKeys];
   __shared__ long long rowp[kAttnKeys];
   float* q = sm;
-  float* acc = sm + p.R;
+  float* acc = sm + p.Dk;
   const long long t = blockIdx.x;
   const int h = blockIdx.y;
+  const int kvh = h / (p.H / p.Hkv);
   const int tid = threadIdx.x;
-  const T* qr = reinterpret_cast<const T*>(p.q) + t * p.ldq + (long long)h * p.R;
-  for (int i = tid; i < p.R; i += kAttnKeys) {
-    q[i] = to_f32<T>(qr[i]);
-    acc[i] = 0.f;
-  }
-  const long long n_keys = p.positions[t] + 1;   // causal: everything up to the token itself
+  const T* qr = reinterpret_cast<const T*>(p.q) + t * p.ldq + (long long)h * p.Dk;
+  for (int i = tid; i < p.Dk; i += kAttnKeys) q[i] = to_f32<T>(qr[i]);
+  for (int i = tid; i < p.Dv; i += kAttnKeys) acc[i] = 0.f;
+  const long long n_keys = p.positions[t] + 1;
   const int* bt = p.block_tables + (long long)p.tok_seq[t] * p.max_blocks;
-  const T* cache = reinterpret_cast<const T*>(p.cache);
+  const T* kc = reinterpret_cast<const T*>(p.k);
+  const T* vc = reinterpret_cast<const T*>(p.v);
   float m = -INFINITY, l = 0.f;
-  for (long long k0 = 0; k0 < n_keys; k0 += kAttnKeys) {
+  for (long long k0 = first_visible(p.mask_kind, p.mask_size, (int)(n_keys - 1)); k0 < n_keys;
+       k0 += kAttnKeys) {
     __syncthreads();   // q and acc are set; the last tile's weights have been read
     const long long key = k0 + tid;
     float s = -INFINITY;
@@ -141,10 +150,11 @@ __global__ void __launch_bounds__(kAttnKeys) latent_attention_exact_kernel(const
       const long long b = key / p.block_size;
       const int blk = b < p.max_blocks ? bt[b] : -1;
       if (blk >= 0 && blk < p.num_blocks) {
-        const long long row = ((long long)blk * p.block_size + key % p.block_size) * p.R;
-        rowp[tid] = row;
+        const long long row = ((long long)blk * p.Hkv + kvh) * p.block_size + key % p.block_size;
+        rowp[tid] = row * p.v_row;
+        const T* kr = kc + row * p.k_row;
         float d = 0.f;
-        for (int i = 0; i < p.R; ++i) d = fmaf(q[i], to_f32<T>(cache[row + i]), d);
+        for (int i = 0; i < p.Dk; ++i) d = fmaf(q[i], to_f32<T>(kr[i]), d);
         s = d * p.scale;
       } else {
         rowp[tid] = 0;
@@ -159,15 +169,21 @@ __global__ void __launch_bounds__(kAttnKeys) latent_attention_exact_kernel(const
     l = l * keep + sum;
     m = m_new;
     const int n = (int)min((long long)kAttnKeys, n_keys - k0);
-    for (int i = tid; i < p.R; i += kAttnKeys) {
+    for (int i = tid; i < p.Dv; i += kAttnKeys) {
       float a = acc[i] * keep;
-      for (int j = 0; j < n; ++j) a = fmaf(pw[j], to_f32<T>(cache[rowp[j] + i]), a);
+      for (int j = 0; j < n; ++j) a = fmaf(pw[j], to_f32<T>(vc[rowp[j] + i]), a);
       acc[i] = a;
     }
   }
-  T* o = reinterpret_cast<T*>(p.out) + t * p.ldo + (long long)h * p.R;
+  if (p.sink != nullptr && m != -INFINITY) l += expf(p.sink[h] - m);
+  T* o = reinterpret_cast<T*>(p.out) + t * p.ldo + (long long)h * p.Dv;
+  const T* gate = p.gate ? reinterpret_cast<const T*>(p.gate) + t * p.ldg + (long long)h * p.Dv : nullptr;
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int i = tid; i < p.R; i += kAttnKeys) o[i] = from_f32<T>(acc[i] * inv);   // own columns
+  for (int i = tid; i < p.Dv; i += kAttnKeys) {   // own columns
+    float v = acc[i] * inv;
+    if (gate != nullptr) v /= 1.f + expf(-to_f32<T>(gate[i]));
+    o[i] = from_f32<T>(v);
+  }
 }
 
 }  // namespace ab200
@@ -201,32 +217,42 @@ int ab200_linear_exact(const void* x, long long ldx, long long x_gstride, const 
   return e == cudaSuccess ? 0 : -5;
 }
 
-// q [T, H * R] in latent space; cache [num_blocks, block_size, R]; out [T, H * R].
-int ab200_latent_attention_exact(const void* q, long long ldq, const void* cache, int num_blocks,
-                                 int block_size, const void* block_tables, int max_blocks,
-                                 const void* tok_seq, const void* positions, void* out,
-                                 long long ldo, long long T, int H, int R, float scale, int dtype,
-                                 int* status, cudaStream_t stream) {
+// k: [num_blocks, Hkv, block_size, k_row] of which the first Dk columns count, v likewise (it may
+// be the same tensor); sink fp32 [H] and gate [T, ldg] may be null.
+int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row, const void* v,
+                          int v_row, int num_blocks, int block_size, const void* block_tables,
+                          int max_blocks, const void* tok_seq, const void* positions,
+                          const void* sink, const void* gate, long long ldg, void* out,
+                          long long ldo, long long T, int H, int Hkv, int Dk, int Dv, int mask_kind,
+                          int mask_size, float scale, int dtype, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
-  const size_t smem = 2 * (size_t)R * sizeof(float);
+  if (H < 1 || Hkv < 1 || H % Hkv || Dk > k_row || Dv > v_row || block_size < 1) return -2;
+  if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
+    return -2;
+  const size_t smem = ((size_t)Dk + Dv) * sizeof(float);
   if (H > 65535 || smem > 200 * 1024) return -6;
   ExactAttnArgs a;
   a.q = q; a.ldq = ldq;
-  a.cache = cache;
+  a.k = k; a.v = v;
+  a.k_row = k_row; a.v_row = v_row;
   a.block_tables = reinterpret_cast<const int*>(block_tables);
   a.max_blocks = max_blocks; a.block_size = block_size;
   a.tok_seq = reinterpret_cast<const int*>(tok_seq);
   a.positions = reinterpret_cast<const long long*>(positions);
+  a.sink = reinterpret_cast<const float*>(sink);
+  a.gate = gate; a.ldg = ldg;
   a.out = out; a.ldo = ldo;
-  a.H = H; a.R = R; a.num_blocks = num_blocks;
+  a.H = H; a.Hkv = Hkv; a.Dk = Dk; a.Dv = Dv;
+  a.num_blocks = num_blocks;
+  a.mask_kind = mask_kind; a.mask_size = mask_size;
   a.scale = scale;
   a.status = status;
   const dim3 grid((unsigned)T, (unsigned)H);
-  auto k = dtype == 0 ? latent_attention_exact_kernel<bf16> : latent_attention_exact_kernel<float>;
+  auto kern = dtype == 0 ? attention_exact_kernel<bf16> : attention_exact_kernel<float>;
   if (smem > 40 * 1024 &&
-      cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return -3;
-  return launch_pdl(k, grid, dim3(kAttnKeys), smem, stream, a) == cudaSuccess ? 0 : -5;
+  return launch_pdl(kern, grid, dim3(kAttnKeys), smem, stream, a) == cudaSuccess ? 0 : -5;
 }
 
 }  // extern "C"

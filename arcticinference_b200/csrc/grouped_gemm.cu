@@ -35,6 +35,7 @@ struct GroupedArgs {
   int x_by_group;           // the activations' map has a group dimension
   int m_fastest;            // work order: row tiles of one weight tile next to each other
   int act;
+  GateParams gate;
   uint32_t tmem_cols;
   const int4* tiles;
   const int* num_tiles;
@@ -72,9 +73,16 @@ __device__ __forceinline__ GgWork gg_work(const GroupedArgs& p, int w, int m_tot
 }
 
 // The activations' rounding to bf16 is far coarser than the fast exponential and division.
-__device__ __forceinline__ float gg_act(int act, float z) {
-  const float u = act == kActSilu ? z : 1.5957691216057308f * (z + 0.044715f * z * z * z);
-  return __fdividef(z, 1.f + __expf(-u));   // gelu_tanh(z) = z * sigmoid(2 sqrt(2/pi) (...))
+__device__ __forceinline__ float gg_gated(int act, const GateParams& p, float g, float u) {
+  float t;   // g * sigmoid(t)
+  if (act == kActClampedSwish) {
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit) + 1.f;
+    t = p.alpha * g;
+  } else {   // gelu_tanh(z) = z * sigmoid(2 sqrt(2/pi) (...))
+    t = act == kActSilu ? g : 1.5957691216057308f * (g + 0.044715f * g * g * g);
+  }
+  return __fdividef(g, 1.f + __expf(-t)) * u;
 }
 
 __global__ void __launch_bounds__(kGgThreads, 1)
@@ -238,9 +246,10 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x,
             uint32_t o[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i)
-              o[i] = pack_bf16x2(
-                  gg_act(p.act, __uint_as_float(r[2 * i])) * __uint_as_float(r[16 + 2 * i]),
-                  gg_act(p.act, __uint_as_float(r[2 * i + 1])) * __uint_as_float(r[17 + 2 * i]));
+              o[i] = pack_bf16x2(gg_gated(p.act, p.gate, __uint_as_float(r[2 * i]),
+                                          __uint_as_float(r[16 + 2 * i])),
+                                 gg_gated(p.act, p.gate, __uint_as_float(r[2 * i + 1]),
+                                          __uint_as_float(r[17 + 2 * i])));
             uint4* q = reinterpret_cast<uint4*>(dst + (n0 + c0) / 2);
             q[0] = make_uint4(o[0], o[1], o[2], o[3]);
             q[1] = make_uint4(o[4], o[5], o[6], o[7]);
@@ -282,17 +291,17 @@ extern "C" {
 // x [x_rows, K] with row stride ldx; x_gstride > 0: group g's activations start g * x_gstride
 // further. w[g] at w + g * w_gstride, rows ldw apart. With `tiles` (int32 x 4: group, first row,
 // rows; `num_tiles` of them, at most max_tiles) x and out hold the rows of all groups one after
-// the other; without, every group has M rows. act: 0, 1 (silu) or 2 (gelu_tanh): gated product,
-// out has N / 2 columns.
+// the other; without, every group has M rows. act: 0, 1 (silu), 2 (gelu_tanh) or 3 (clamped swish
+// with act_limit and act_alpha): gated product, out has N / 2 columns.
 int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long long x_rows,
                        const void* w, long long ldw, long long w_gstride, void* out, long long ldo,
                        long long out_gstride, int M, int N, int K, int groups, const void* tiles,
-                       const void* num_tiles, int max_tiles, int act, int* status,
-                       cudaStream_t stream) {
+                       const void* num_tiles, int max_tiles, int act, float act_limit,
+                       float act_alpha, int* status, cudaStream_t stream) {
   if (N <= 0 || K <= 0 || groups <= 0 || x_rows <= 0 || (tiles == nullptr ? M : max_tiles) <= 0)
     return 0;
   if ((K % 8) || (N % 8) || (ldx % 8) || (x_gstride % 8) || (ldw % 8) || (w_gstride % 8) ||
-      (ldo % 8) || (out_gstride % 8) || (act != 0 && N % 32) || act < 0 || act > 2 ||
+      (ldo % 8) || (out_gstride % 8) || (act != 0 && N % 32) || act < 0 || act > 3 ||
       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) |
         reinterpret_cast<uintptr_t>(out)) & 15))
     return -2;
@@ -322,6 +331,8 @@ int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long l
   a.groups = groups;
   a.x_by_group = x_gstride > 0;
   a.act = act;
+  a.gate.limit = act_limit;
+  a.gate.alpha = act_alpha;
   a.tiles = reinterpret_cast<const int4*>(tiles);
   a.num_tiles = reinterpret_cast<const int*>(num_tiles);
   a.out = reinterpret_cast<__nv_bfloat16*>(out);

@@ -1,6 +1,6 @@
 // Attention in latent space for sm_100a: queries [T, H, R] against a paged cache of one latent
 // vector of R = 128 .. 512 numbers per token, which is key and value of every head at once.
-// Decode and short chunks; softmax over every key up to the token itself.
+// Decode and short chunks; softmax over the keys up to the token itself that its mask shows.
 //
 // The keys are the tensor core's M side. Per tile of 128 keys
 //     S^T [128 keys x n]   = C Q^T       (tcgen05.mma, A = the latents K-major as they lie)
@@ -15,6 +15,10 @@
 // again when its share of O^T has been accumulated.
 // S of tile j + 1 is issued before O of tile j where the ring holds two tiles (R <= 256).
 //
+// A cache row may carry 64 more columns that belong to the key only (a rotated part that the heads
+// share, beside the latent): a piece outside the ring, in one or two buffers of its own, that is
+// free as soon as its share of S is done.
+//
 // Softmax: four warps, a thread per key. A column's maximum over the keys is a butterfly over
 // the warp's lanes (16 columns in 16 shuffles) and four words of shared memory; sums stay
 // per-thread until the end. O is rescaled only in tiles where a maximum moved.
@@ -26,6 +30,7 @@
 #include <string.h>
 
 #include "api.h"
+#include "common/elem.cuh"
 #include "common/pdl.cuh"
 #include "common/ptx.cuh"
 #include "common/tensormap.h"
@@ -44,6 +49,8 @@ struct LatentArgs {
   int max_blocks, block_size;
   int H, pieces;           // pieces: R / 64 per tile
   int slots, p_bufs, overlap;
+  int x_bufs;              // buffers of the key-only piece (0: none)
+  int mask_kind, mask_size;
   float scale, scale_log2;
   uint32_t tmem_cols;
   __nv_bfloat16* out;      // [T * H][R]
@@ -106,18 +113,20 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
                                              ~static_cast<uintptr_t>(1023));
   __shared__ __align__(16) float wred[NR * 4];   // per column: the four warps' values
   __shared__ __align__(16) float m_s[NR], neg_s[NR], alpha_s[NR], inv_s[NR];
-  __shared__ int lim_s[NR];                      // last visible key of each row
+  __shared__ int2 see_s[NR];                     // first and last visible key of each row
   __shared__ int rescale_s[2];
-  __shared__ uint64_t bars[1 + 2 * kLatMaxSlots + 8];
+  __shared__ uint64_t bars[1 + 2 * kLatMaxSlots + 12];
   __shared__ uint32_t tmem_slot;
   __shared__ volatile int abort_s;
 
   const int NC = p.pieces;
+  const int NX = p.x_bufs > 0 ? 1 : 0;
   const uint32_t sQ = smem_u32(smem);
-  const uint32_t sC = sQ + (uint32_t)NC * NR * 128u;
-  const uint32_t sP = sC + (uint32_t)p.slots * kPieceBytes;
-  uint8_t* pC = smem + (size_t)NC * NR * 128;
-  uint8_t* pP = pC + (size_t)p.slots * kPieceBytes;
+  const uint32_t sC = sQ + (uint32_t)(NC + NX) * NR * 128u;
+  const uint32_t sX = sC + (uint32_t)p.slots * kPieceBytes;
+  const uint32_t sP = sX + (uint32_t)p.x_bufs * kPieceBytes;
+  uint8_t* pC = smem + (size_t)(NC + NX) * NR * 128;
+  uint8_t* pP = pC + (size_t)(p.slots + p.x_bufs) * kPieceBytes;
   const uint32_t bb = smem_u32(bars);
   const uint32_t q_full = bb;
   auto c_full = [&](int s) { return bb + 8u * (1 + s); };
@@ -126,6 +135,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
   auto s_empty = [&](int s) { return bb + 8u * (3 + 2 * kLatMaxSlots + s); };
   auto p_full = [&](int s) { return bb + 8u * (5 + 2 * kLatMaxSlots + s); };
   auto o_full = [&](int s) { return bb + 8u * (7 + 2 * kLatMaxSlots + s); };
+  auto x_full = [&](int s) { return bb + 8u * (9 + 2 * kLatMaxSlots + s); };
+  auto x_empty = [&](int s) { return bb + 8u * (11 + 2 * kLatMaxSlots + s); };
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
 
@@ -152,6 +163,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
       mbar_init(s_empty(s), 4);
       mbar_init(p_full(s), 4);
       mbar_init(o_full(s), 1);
+      mbar_init(x_full(s), 1);
+      mbar_init(x_empty(s), 1);
       rescale_s[s] = 0;
     }
     abort_s = 0;
@@ -161,7 +174,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
   }
   for (int i = threadIdx.x; i < NR; i += kLatThreads) {
     m_s[i] = -INFINITY;
-    lim_s[i] = min(pos0 + (row0 + i) / p.H, kv_end - 1);
+    const int pos = pos0 + (row0 + i) / p.H;
+    see_s[i] = make_int2(first_visible(p.mask_kind, p.mask_size, pos), min(pos, kv_end - 1));
   }
   if (warp == 5) {
     tmem_alloc(smem_u32(&tmem_slot), p.tmem_cols);
@@ -194,15 +208,15 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
     // ------------------------------ TMA producer ------------------------------
     if (n_tiles > 0) {
       if (lane == 0) {
-        mbar_arrive_expect_tx(q_full, (uint32_t)NC * NR * 128u);
-        for (int c = 0; c < NC; ++c)
+        mbar_arrive_expect_tx(q_full, (uint32_t)(NC + NX) * NR * 128u);
+        for (int c = 0; c < NC + NX; ++c)
           tma_load_2d(sQ + (uint32_t)c * NR * 128u, &tmap_q, q_full, c * 64, row0);
       }
       // A lane per (piece, cache block) box of the tile: it waits for the piece's slot itself and
       // issues its copy, so a tile's copies leave as fast as their slots come free.
       const int* bt = p.block_tables + (long long)seq * p.max_blocks;
       const int nb_max = kLatKeys / bs;
-      const int boxes = NC * nb_max;
+      const int boxes = (NC + NX) * nb_max;
       bool ok = true;
       int bid_next = 0;
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -213,9 +227,15 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
           const int c = i / nb_max, blk = i % nb_max;
           const bool mine = i < boxes && blk < nblk;
           const int bid = (j == 0 || boxes > 32) ? (mine ? bt[key0 / bs + blk] : 0) : bid_next;
-          const int idx = j * NC + c;
-          const int slot = idx % p.slots;
-          const uint32_t ph = (uint32_t)(idx / p.slots) & 1u;
+          // a piece of the latent has a slot of the ring, the key-only piece one of its buffers
+          const bool kx = c >= NC;
+          const int idx = kx ? j : j * NC + c;
+          const int bufs = kx ? p.x_bufs : p.slots;
+          const int slot = idx % bufs;
+          const uint32_t ph = (uint32_t)(idx / bufs) & 1u;
+          const uint32_t full = kx ? x_full(slot) : c_full(slot);
+          const uint32_t empty = kx ? x_empty(slot) : c_empty(slot);
+          const uint32_t dst = (kx ? sX : sC) + (uint32_t)slot * kPieceBytes;
           if (boxes <= 32 && j + 1 < n_tiles) {   // the next tile's table entry is on its way
             const int next0 = key0 + kLatKeys;
             const int nn = (min(kLatKeys, kv_end - next0) + bs - 1) / bs;
@@ -225,10 +245,9 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
           unsigned long long t0 = 0;
           uint32_t spins = 0;
           while (!done) {
-            if (mbar_try_wait(c_empty(slot), ph ^ 1u)) {
-              if (blk == 0) mbar_arrive_expect_tx(c_full(slot), (uint32_t)(nblk * bs) * 128u);
-              tma_load_2d(sC + (uint32_t)slot * kPieceBytes + (uint32_t)(blk * bs) * 128u, &tmap_c,
-                          c_full(slot), c * 64, bid * bs);
+            if (mbar_try_wait(empty, ph ^ 1u)) {
+              if (blk == 0) mbar_arrive_expect_tx(full, (uint32_t)(nblk * bs) * 128u);
+              tma_load_2d(dst + (uint32_t)(blk * bs) * 128u, &tmap_c, full, c * 64, bid * bs);
               done = true;
             } else if ((++spins & 63u) == 0u) {
               if (abort_s) {
@@ -267,6 +286,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const uint64_t c_mn = make_desc_mnmajor_sw128(sC, kPieceBytes);
       const uint64_t q_k = make_desc_kmajor_sw128(sQ);                   // + NR * 8 per piece
       const uint64_t p_k = make_desc_kmajor_sw128(sP);
+      const uint64_t x_k = make_desc_kmajor_sw128(sX);
       int s_slot = 0, o_slot = 0;
       uint32_t s_ph = 0;
       auto wait = [&](uint32_t bar, uint32_t parity, int code, int j) -> bool {
@@ -286,13 +306,30 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
             for (int k = 0; k < 4; ++k)
               umma_f16_ss(tS_u + (uint32_t)st * NR, cd + (uint64_t)(2 * k), qd + (uint64_t)(2 * k),
                           idesc_s, (c > 0 || k > 0) ? 1u : 0u);
-            if (c == NC - 1) tc_commit(s_full(st));
+            if (c == NC - 1 && NX == 0) tc_commit(s_full(st));
           }
           __syncwarp();
           if (++s_slot == p.slots) {
             s_slot = 0;
             s_ph ^= 1u;
           }
+        }
+        if (NX) {
+          const int xb = p.x_bufs == 2 ? (j & 1) : 0;
+          const uint32_t xph = (uint32_t)(p.x_bufs == 2 ? (j >> 1) : j) & 1u;
+          if (!wait(x_full(xb), xph, 1630 + xb, j)) return false;
+          tc_fence_after();
+          const uint64_t xd = x_k + (uint64_t)(xb * (int)(kPieceBytes / 16));
+          const uint64_t qd = q_k + (uint64_t)(NC * (NR * 8));
+          if (elect_one()) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              umma_f16_ss(tS_u + (uint32_t)st * NR, xd + (uint64_t)(2 * k), qd + (uint64_t)(2 * k),
+                          idesc_s, 1u);
+            tc_commit(x_empty(xb));
+            tc_commit(s_full(st));
+          }
+          __syncwarp();
         }
         return true;
       };
@@ -341,11 +378,13 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
     for (int i = 0; i < NR; ++i) l[i] = 0.f;
     bool ok = true;
     const int min_lim = pos0 + row0 / p.H;
+    const int max_low =
+        first_visible(p.mask_kind, p.mask_size, pos0 + (row0 + n_rows - 1) / p.H);
     for (int j = 0; j < n_tiles; ++j) {
       const int st = j & 1;
       const int key0 = kv_start + j * kLatKeys;
       const int key = key0 + tid;
-      const bool need_mask = key0 + kLatKeys - 1 > min(min_lim, kv_end - 1);
+      const bool need_mask = key0 + kLatKeys - 1 > min(min_lim, kv_end - 1) || key0 < max_low;
       ok = __all_sync(0xffffffffu, ok && mbar_wait(s_full(st), (uint32_t)(j >> 1) & 1u, &abort_s,
                                                    p.status, 1700 + st, j));
       tc_fence_after();
@@ -358,8 +397,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
         for (int g = 0; g < NR / 16; ++g) tmem_ld_wait_dep16(sr[g]);
         if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < NR; ++i)
-            if (key > lim_s[i]) sr[i / 16][i % 16] = 0xff800000u;   // -inf
+          for (int i = 0; i < NR; ++i) {
+            const int2 seen = see_s[i];
+            if (key < seen.x || key > seen.y) sr[i / 16][i % 16] = 0xff800000u;   // -inf
+          }
         }
 #pragma unroll
         for (int g = 0; g < NR / 16; ++g) {
@@ -517,22 +558,32 @@ static int launch_latent(const CUtensorMap& tq, const CUtensorMap& tc, LatentArg
                          cudaStream_t stream) {
   const int NC = a.pieces;
   const size_t limit = 227 * 1024 - 4096;   // static shared memory and alignment aside
-  const size_t q_bytes = (size_t)NC * NR * 128;
+  const int NX = a.x_bufs;   // (wanted: 0 or 1)
+  const size_t q_bytes = (size_t)(NC + NX) * NR * 128;
+  const size_t room = limit - q_bytes;
   a.p_bufs = 2;
-  auto fit = [&](int pb) {
-    int s = (int)((limit - q_bytes - (size_t)pb * NR * 256) / kPieceBytes) & ~1;
+  auto fit = [&](int pb, int xb) {
+    const size_t other = (size_t)pb * NR * 256 + (size_t)xb * kPieceBytes;
+    if (other >= room) return 0;
+    int s = (int)((room - other) / kPieceBytes) & ~1;
     return s > kLatMaxSlots ? kLatMaxSlots : s;
   };
-  a.slots = fit(2);
-  if (a.slots < NC + 2 && fit(1) > a.slots) {
+  a.slots = fit(2, NX);
+  if (a.slots < NC + 2 && fit(1, NX) > a.slots) {
     a.p_bufs = 1;
-    a.slots = fit(1);
+    a.slots = fit(1, NX);
   }
   if (a.slots < NC) return -6;
+  // a second buffer of the key-only piece where it costs no slot that overlapping needs
+  if (NX && (fit(a.p_bufs, 2) >= a.slots || fit(a.p_bufs, 2) >= 2 * NC)) {
+    a.x_bufs = 2;
+    a.slots = fit(a.p_bufs, 2);
+  }
   a.overlap = a.slots >= 2 * NC;
   a.tmem_cols = 32;
   while (a.tmem_cols < (uint32_t)((2 + NC / 2) * NR)) a.tmem_cols <<= 1;
-  const size_t smem = q_bytes + (size_t)a.slots * kPieceBytes + (size_t)a.p_bufs * NR * 256 + 1024;
+  const size_t smem = q_bytes + (size_t)(a.slots + a.x_bufs) * kPieceBytes +
+                      (size_t)a.p_bufs * NR * 256 + 1024;
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -555,24 +606,30 @@ using namespace ab200;
 
 extern "C" {
 
-// q and out: bf16 [T * H, R] contiguous; cache [num_blocks, block_size, R]; R a multiple of 128 up
-// to 512; tile_rows 16, 32, 48 or 64, the rows per work item.
+// q bf16 [T * H, R + key_extra], out [T * H, R], both contiguous; cache [num_blocks, block_size,
+// R + key_extra]; R a multiple of 128 up to 512, key_extra 0 or 64 (columns of the key only);
+// tile_rows 16, 32, 48 or 64, the rows per work item (at most 48 with R = 512 and key_extra).
 int ab200_latent_attention(const void* q, long long q_rows, const void* cache, int num_blocks,
                            int block_size, const void* block_tables, int max_blocks,
                            const void* work, int num_work, const void* tok_splits, int max_splits,
-                           long long T, int H, int R, int tile_rows, float scale, void* out,
-                           void* o_part, void* lse_part, int* status, cudaStream_t stream) {
+                           long long T, int H, int R, int key_extra, int mask_kind, int mask_size,
+                           int tile_rows, float scale, void* out, void* o_part, void* lse_part,
+                           int* status, cudaStream_t stream) {
   if (num_work <= 0 || T <= 0) return 0;
   if (R % 128 || R < 128 || R > 512 || H <= 0 || q_rows != T * H) return -2;
+  if (key_extra != 0 && key_extra != 64) return -2;
+  if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
+    return -2;
   if (block_size < 8 || block_size > kLatKeys || kLatKeys % block_size) return -2;
   if (T * H > 0x7fffffffll || (long long)num_blocks * block_size > 0x7fffffffll) return -6;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
+  const int W = R + key_extra;
   CUtensorMap tq, tc;
-  if (make_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)q_rows, (uint64_t)R,
-                   (uint64_t)R * 2, (uint32_t)tile_rows, 64) != 0)
+  if (make_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)q_rows, (uint64_t)W,
+                   (uint64_t)W * 2, (uint32_t)tile_rows, 64) != 0)
     return -4;
   if (make_tmap_2d(&tc, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)num_blocks * block_size,
-                   (uint64_t)R, (uint64_t)R * 2, (uint32_t)block_size, 64) != 0)
+                   (uint64_t)W, (uint64_t)W * 2, (uint32_t)block_size, 64) != 0)
     return -4;
   LatentArgs a;
   memset(&a, 0, sizeof(a));
@@ -582,6 +639,9 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
   a.block_size = block_size;
   a.H = H;
   a.pieces = R / 64;
+  a.x_bufs = key_extra / 64;
+  a.mask_kind = mask_kind;
+  a.mask_size = mask_size;
   a.scale = scale;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);

@@ -1,0 +1,262 @@
+// What lies between an attention layer's input projection and its scores, for layers with
+// partial rotary positions:
+//
+//   head_rope_cache    per-head RMS norm of queries and keys (optional), rotation of their first
+//                      rot dimensions, queries in place, keys and values to the paged cache
+//   latent_rope_cache  RMS norm of a compressed K/V projection and rotation of the key part that
+//                      the heads share, both to the paged latent cache; rotation of every query
+//                      head's rotary part in place
+//
+// A block owns a token: its sines and cosines are computed once (angle = position * frequency in
+// fp32, as are the norms), and its warps walk the heads. Dimension i is paired with i + rot / 2.
+// T is the model's element type (bf16 or fp32).
+
+#include "api.h"
+#include "common/elem.cuh"
+#include "common/pdl.cuh"
+
+namespace ab200 {
+
+constexpr int kRopeThreads = 256;
+
+// cs[2 * i], cs[2 * i + 1]: cosine and sine of pair i
+__device__ __forceinline__ void angles(float* cs, const float* __restrict__ freq, int half,
+                                       long long pos) {
+  for (int i = threadIdx.x; i < half; i += blockDim.x)
+    sincosf((float)pos * freq[i], &cs[2 * i + 1], &cs[2 * i]);
+}
+
+__device__ __forceinline__ float rotated(const float* row, const float* cs, int half, int i) {
+  if (i < half) return row[i] * cs[2 * i] - row[i + half] * cs[2 * i + 1];
+  if (i < 2 * half) return row[i] * cs[2 * (i - half)] + row[i - half] * cs[2 * (i - half) + 1];
+  return row[i];
+}
+
+struct HeadRopeArgs {
+  void* proj;               // [T][ld]: Hq query heads, Hkv key heads of D, Hkv value heads of Dv
+  long long ld;
+  const long long* positions;
+  const long long* slots;
+  const float* wq;          // [D] or null: no norm
+  const float* wk;
+  const float* freq;        // [half]
+  void* k_cache;            // [num_blocks][Hkv][block_size][D]
+  void* v_cache;            // [num_blocks][Hkv][block_size][Dv]
+  long long num_slots;
+  int Hq, Hkv, D, Dv, half, block_size;
+  float rdim, eps;          // 1 / (dimensions the norm's mean is over; columns beyond are zero)
+  int* status;
+};
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const HeadRopeArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) float sm[];
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* cs = sm + (kRopeThreads / 32) * p.D;
+  float* row = sm + warp * p.D;
+  angles(cs, p.freq, p.half, p.positions[t]);
+  __syncthreads();
+  long long slot = p.slots[t];
+  if (slot >= p.num_slots) {
+    if (threadIdx.x == 0) report_error(p.status, kErrBounds, 43, (int)t);
+    slot = -1;
+  }
+  const long long blk = slot >= 0 ? slot / p.block_size : 0;
+  const long long off = slot >= 0 ? slot % p.block_size : 0;
+  T* base = reinterpret_cast<T*>(p.proj) + t * p.ld;
+  for (int j = warp; j < p.Hq + 2 * p.Hkv; j += kRopeThreads / 32) {
+    const bool is_q = j < p.Hq, is_v = j >= p.Hq + p.Hkv;
+    if (!is_q && slot < 0) continue;   // padding token: no key, no value
+    if (is_v) {
+      const int g = j - p.Hq - p.Hkv;
+      const T* src = base + (long long)(p.Hq + p.Hkv) * p.D + (long long)g * p.Dv;
+      T* dst = reinterpret_cast<T*>(p.v_cache) + ((blk * p.Hkv + g) * p.block_size + off) * p.Dv;
+      if (VEC) {
+        for (int i = lane * 4; i < p.Dv; i += 128) store4(dst + i, load4(src + i));
+      } else {
+        for (int i = lane; i < p.Dv; i += 32) dst[i] = src[i];
+      }
+      continue;
+    }
+    T* src = base + (long long)j * p.D;
+    const float* w = is_q ? p.wq : p.wk;
+    float inv = 1.f;
+    if (w != nullptr) {
+      float ss = 0.f;
+      if (VEC) {
+        for (int i = lane * 4; i < p.D; i += 128) {
+          const float4 v = load4(src + i);
+          ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+      } else {
+        for (int i = lane; i < p.D; i += 32) {
+          const float v = to_f32<T>(src[i]);
+          ss += v * v;
+        }
+      }
+      inv = 1.f / sqrtf(warp_sum(ss) * p.rdim + p.eps);
+    }
+    __syncwarp();   // the last head's row has been read
+    if (VEC) {
+      for (int i = lane * 4; i < p.D; i += 128) {
+        float4 v = load4(src + i);
+        if (w != nullptr) {
+          const float4 g = load4(w + i);
+          v = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+        }
+        store4(row + i, v);
+      }
+    } else {
+      for (int i = lane; i < p.D; i += 32)
+        row[i] = w != nullptr ? to_f32<T>(src[i]) * inv * w[i] : to_f32<T>(src[i]);
+    }
+    __syncwarp();
+    T* dst = src;
+    if (!is_q)
+      dst = reinterpret_cast<T*>(p.k_cache) +
+            ((blk * p.Hkv + (j - p.Hq)) * p.block_size + off) * p.D;
+    if (VEC) {
+      for (int i = lane * 4; i < p.D; i += 128)
+        store4(dst + i, make_float4(rotated(row, cs, p.half, i), rotated(row, cs, p.half, i + 1),
+                                    rotated(row, cs, p.half, i + 2), rotated(row, cs, p.half, i + 3)));
+    } else {
+      for (int i = lane; i < p.D; i += 32) dst[i] = from_f32<T>(rotated(row, cs, p.half, i));
+    }
+  }
+}
+
+struct LatentRopeArgs {
+  void* q;                  // [T][ld]: H heads of dq columns, the rotary part from column dim
+  const void* ckv;          // [T][ld]: R latent columns, then 2 * half rotary ones
+  long long ld;
+  const long long* positions;
+  const long long* slots;
+  const float* weight;      // [R]
+  const float* freq;        // [half]
+  void* cache;              // rows of `width` columns, the rotary key part from column rot_at
+  long long num_slots;
+  int H, dq, dim, R, half, width, rot_at;
+  float eps;
+  int* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kRopeThreads) latent_rope_cache_kernel(const LatentRopeArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) float cs[];
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  angles(cs, p.freq, p.half, p.positions[t]);
+  const T* c = reinterpret_cast<const T*>(p.ckv) + t * p.ld;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < p.R; i += blockDim.x) {
+    const float v = to_f32<T>(c[i]);
+    ss += v * v;
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, red) / (float)p.R + p.eps);   // (publishes cs)
+  const long long slot = p.slots[t];
+  if (slot >= p.num_slots) {
+    if (threadIdx.x == 0) report_error(p.status, kErrBounds, 44, (int)t);
+  } else if (slot >= 0) {
+    T* dst = reinterpret_cast<T*>(p.cache) + slot * p.width;
+    for (int i = threadIdx.x; i < p.R; i += blockDim.x)
+      dst[i] = from_f32<T>(to_f32<T>(c[i]) * inv * p.weight[i]);
+    for (int i = threadIdx.x; i < p.half; i += blockDim.x) {
+      const float u = to_f32<T>(c[p.R + i]), v = to_f32<T>(c[p.R + p.half + i]);
+      dst[p.rot_at + i] = from_f32<T>(u * cs[2 * i] - v * cs[2 * i + 1]);
+      dst[p.rot_at + p.half + i] = from_f32<T>(v * cs[2 * i] + u * cs[2 * i + 1]);
+    }
+  }
+  T* q = reinterpret_cast<T*>(p.q) + t * p.ld;
+  const int n = p.H * p.half;
+  for (int k = threadIdx.x; k < n; k += blockDim.x) {
+    const int h = k / p.half, i = k - h * p.half;
+    T* a = q + (long long)h * p.dq + p.dim + i;
+    const float u = to_f32<T>(a[0]), v = to_f32<T>(a[p.half]);
+    a[0] = from_f32<T>(u * cs[2 * i] - v * cs[2 * i + 1]);
+    a[p.half] = from_f32<T>(v * cs[2 * i] + u * cs[2 * i + 1]);
+  }
+}
+
+template <typename T>
+static int launch_head_rope(const HeadRopeArgs& a, long long n, cudaStream_t stream) {
+  const size_t smem = ((size_t)(kRopeThreads / 32) * a.D + 2 * (size_t)a.half) * sizeof(float);
+  if (smem > 200 * 1024) return -6;
+  const bool vec = a.D % 4 == 0 && a.Dv % 4 == 0 && a.ld % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.proj) | reinterpret_cast<uintptr_t>(a.wq) |
+                     reinterpret_cast<uintptr_t>(a.wk) | reinterpret_cast<uintptr_t>(a.k_cache) |
+                     reinterpret_cast<uintptr_t>(a.v_cache)) & 15) == 0;
+  auto k = vec ? head_rope_cache_kernel<T, true> : head_rope_cache_kernel<T, false>;
+  if (smem > 48 * 1024 &&
+      cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    return -3;
+  return launch_pdl(k, dim3((unsigned)n), dim3(kRopeThreads), smem, stream, a) == cudaSuccess ? 0 : -5;
+}
+
+}  // namespace ab200
+
+using namespace ab200;
+typedef __nv_bfloat16 bf16;
+
+extern "C" {
+
+// proj [T, ld] holds Hq query and Hkv key heads of D columns, then Hkv value heads of Dv, of which
+// the first `dim` (query, key) columns are in use and the others zero; wq, wk fp32 [D] or null;
+// freq fp32 [half]: rotary frequencies of the pairs (i, i + half).
+int ab200_head_rope_cache(void* proj, long long ld, const void* positions, const void* slots,
+                          const void* wq, const void* wk, const void* freq, int half, void* k_cache,
+                          void* v_cache, long long T, int Hq, int Hkv, int D, int dim, int Dv,
+                          int block_size, long long num_slots, float eps, int dtype, int* status,
+                          cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (dim < 1 || dim > D || 2 * half > D || half < 0 || block_size < 1 || Hq < 0 || Hkv < 0) return -2;
+  if (ld < (long long)(Hq + Hkv) * D + (long long)Hkv * Dv) return -2;
+  HeadRopeArgs a;
+  a.proj = proj; a.ld = ld;
+  a.positions = reinterpret_cast<const long long*>(positions);
+  a.slots = reinterpret_cast<const long long*>(slots);
+  a.wq = reinterpret_cast<const float*>(wq);
+  a.wk = reinterpret_cast<const float*>(wk);
+  a.freq = reinterpret_cast<const float*>(freq);
+  a.k_cache = k_cache; a.v_cache = v_cache;
+  a.num_slots = num_slots;
+  a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.Dv = Dv;
+  a.half = half; a.block_size = block_size;
+  a.rdim = 1.f / (float)dim;
+  a.eps = eps;
+  a.status = status;
+  return dtype == 0 ? launch_head_rope<bf16>(a, T, stream) : launch_head_rope<float>(a, T, stream);
+}
+
+// q [T, ld]: H heads of dq columns whose rotary part starts at column `dim`; ckv [T, ld]: R latent
+// columns and 2 * half rotary ones; cache rows of `width` columns, the rotary part at rot_at.
+int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* positions,
+                            const void* slots, const void* weight, const void* freq, int half,
+                            void* cache, long long T, int H, int dq, int dim, int R, int width,
+                            int rot_at, long long num_slots, float eps, int dtype, int* status,
+                            cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (half < 0 || dim + 2 * half > dq || R > rot_at || rot_at + 2 * half > width) return -2;
+  LatentRopeArgs a;
+  a.q = q; a.ckv = ckv; a.ld = ld;
+  a.positions = reinterpret_cast<const long long*>(positions);
+  a.slots = reinterpret_cast<const long long*>(slots);
+  a.weight = reinterpret_cast<const float*>(weight);
+  a.freq = reinterpret_cast<const float*>(freq);
+  a.cache = cache;
+  a.num_slots = num_slots;
+  a.H = H; a.dq = dq; a.dim = dim; a.R = R; a.half = half;
+  a.width = width; a.rot_at = rot_at;
+  a.eps = eps;
+  a.status = status;
+  const size_t smem = (2 * (size_t)half + 4) * sizeof(float);
+  if (smem > 48 * 1024) return -6;
+  auto k = dtype == 0 ? latent_rope_cache_kernel<bf16> : latent_rope_cache_kernel<float>;
+  return launch_pdl(k, dim3((unsigned)T), dim3(kRopeThreads), smem, stream, a) == cudaSuccess ? 0 : -5;
+}
+
+}  // extern "C"

@@ -1,10 +1,12 @@
-// Kernels around a 32-bit residual stream ("norm after the sum" decoders):
+// Kernels around a 32-bit residual stream (decoders that list their layers):
 //
-//   embedding          x (fp32) and its 16-bit copy that the projections read
+//   embedding          x (fp32, scaled) and its 16-bit copy that the projections read
 //   stream_norm        x <- norm(alpha * x + y) * (1 + w), in place, plus the 16-bit copy; y is a
 //                      sublayer's output or, for a mixture of experts, the weighted sum of the
 //                      chosen experts' rows, gathered here so that it never exists in memory;
 //                      with a row list it also serves the final norm of the sampled rows
+//   stream_sandwich    x <- x + norm(y) * w_out (+ a vector), in place, and the next sublayer's
+//                      input act = norm(x) * w_in, in one pass over the row
 //   latent_norm_cache  RMS norm of the compressed K/V projection and its write into the paged
 //                      latent cache
 //   gated_act          act(gate) * up on the interleaved gate / up layout
@@ -20,8 +22,8 @@ namespace ab200 {
 template <typename T>
 __global__ void __launch_bounds__(256)
 stream_embedding_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
-                        float* __restrict__ x, T* __restrict__ act, int W, long long vocab,
-                        int* status) {
+                        float* __restrict__ x, T* __restrict__ act, float scale, int W,
+                        long long vocab, int* status) {
   pdl_wait();
   pdl_trigger();
   const long long t = blockIdx.x;
@@ -31,9 +33,9 @@ stream_embedding_kernel(const long long* __restrict__ ids, const T* __restrict__
   if (id >= vocab && threadIdx.x == 0) report_error(status, kErrBounds, 40, (int)t);
   const T* src = table + (ok ? id : 0) * W;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
-    const T v = ok ? src[i] : from_f32<T>(0.f);
-    x[t * W + i] = to_f32<T>(v);
-    if (act != nullptr) act[t * W + i] = v;
+    const float v = ok ? to_f32<T>(src[i]) * scale : 0.f;
+    x[t * W + i] = v;
+    if (act != nullptr) act[t * W + i] = from_f32<T>(v);
   }
 }
 
@@ -46,7 +48,7 @@ struct StreamNormArgs {
   const float* y_weights;  // ... and their weights
   int top;
   const float* weight;
-  float alpha, eps;
+  float alpha, eps, offset;   // offset: added to the weight
   float* x_out;            // optional
   void* act_out;           // optional
   int W;
@@ -101,18 +103,131 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormArgs p
     for (int i = threadIdx.x * 4; i < p.W; i += blockDim.x * 4) {
       float4 s = load4(row + i);
       const float4 w = load4(p.weight + i);
-      s.x *= inv * (1.f + w.x); s.y *= inv * (1.f + w.y);
-      s.z *= inv * (1.f + w.z); s.w *= inv * (1.f + w.w);
+      s.x *= inv * (p.offset + w.x); s.y *= inv * (p.offset + w.y);
+      s.z *= inv * (p.offset + w.z); s.w *= inv * (p.offset + w.w);
       if (p.x_out) store4(p.x_out + t * p.W + i, s);
       if (act) store4(act + t * p.W + i, s);
     }
   } else {
     for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
-      const float s = row[i] * inv * (1.f + p.weight[i]);
+      const float s = row[i] * inv * (p.offset + p.weight[i]);
       if (p.x_out) p.x_out[t * p.W + i] = s;
       if (act) act[t * p.W + i] = from_f32<T>(s);
     }
   }
+}
+
+struct SandwichArgs {
+  float* x;                // updated in place when y or step is given
+  const void* y;           // optional sublayer output (element type T)
+  long long ldy;
+  const float* w_out;      // its norm's weight
+  const float* step;       // optional vector added to the stream after it
+  const float* w_in;       // optional: norm of the new stream, written to act
+  void* act;
+  float eps, offset;
+  int W;
+};
+
+// N4: four-element pieces of the row a thread holds in registers (0: any width, through memory)
+template <typename T, int N4>
+__global__ void __launch_bounds__(256) stream_sandwich_kernel(const SandwichArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  float* xr = p.x + t * p.W;
+  const T* yr = p.y ? reinterpret_cast<const T*>(p.y) + t * p.ldy : nullptr;
+  T* act = p.act ? reinterpret_cast<T*>(p.act) + t * p.W : nullptr;
+  const float rw = 1.f / (float)p.W;
+  if constexpr (N4 > 0) {
+    float4 x[N4], y[N4];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (threadIdx.x + j * blockDim.x) * 4;
+      x[j] = i < p.W ? load4(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      y[j] = (yr != nullptr && i < p.W) ? load4(yr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
+    }
+    if (yr != nullptr) {
+      const float inv = 1.f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+#pragma unroll
+      for (int j = 0; j < N4; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * 4;
+        if (i >= p.W) continue;
+        const float4 w = load4(p.w_out + i);
+        x[j].x += y[j].x * inv * (p.offset + w.x);
+        x[j].y += y[j].y * inv * (p.offset + w.y);
+        x[j].z += y[j].z * inv * (p.offset + w.z);
+        x[j].w += y[j].w * inv * (p.offset + w.w);
+      }
+    }
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (threadIdx.x + j * blockDim.x) * 4;
+      if (i >= p.W) continue;
+      if (p.step != nullptr) {
+        const float4 s = load4(p.step + i);
+        x[j].x += s.x; x[j].y += s.y; x[j].z += s.z; x[j].w += s.w;
+      }
+      if (yr != nullptr || p.step != nullptr) store4(xr + i, x[j]);
+      ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
+    }
+    if (act == nullptr) return;
+    const float inv = 1.f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (threadIdx.x + j * blockDim.x) * 4;
+      if (i >= p.W) continue;
+      const float4 w = load4(p.w_in + i);
+      store4(act + i, make_float4(x[j].x * inv * (p.offset + w.x), x[j].y * inv * (p.offset + w.y),
+                                  x[j].z * inv * (p.offset + w.z), x[j].w * inv * (p.offset + w.w)));
+    }
+  } else {
+    float inv = 0.f, ss = 0.f;
+    if (yr != nullptr) {
+      for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+        const float v = to_f32<T>(yr[i]);
+        ss += v * v;
+      }
+      inv = 1.f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+    }
+    ss = 0.f;
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x) {   // a thread re-reads only its own columns
+      float v = xr[i];
+      if (yr != nullptr) v += to_f32<T>(yr[i]) * inv * (p.offset + p.w_out[i]);
+      if (p.step != nullptr) v += p.step[i];
+      if (yr != nullptr || p.step != nullptr) xr[i] = v;
+      ss += v * v;
+    }
+    if (act == nullptr) return;
+    inv = 1.f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x)
+      act[i] = from_f32<T>(xr[i] * inv * (p.offset + p.w_in[i]));
+  }
+}
+
+template <typename T>
+static int launch_stream_sandwich(const SandwichArgs& a, long long T_rows, cudaStream_t stream) {
+  const bool vec = a.W % 4 == 0 && a.ldy % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.x) |
+                     reinterpret_cast<uintptr_t>(a.w_out) | reinterpret_cast<uintptr_t>(a.step) |
+                     reinterpret_cast<uintptr_t>(a.w_in) | reinterpret_cast<uintptr_t>(a.act)) & 15) == 0;
+  const int n4 = (a.W + 3) / 4;
+  auto k = stream_sandwich_kernel<T, 0>;
+  int threads = 256;
+  if (vec && n4 <= 256 * 8) {
+    // few enough pieces per thread to stay in registers, few enough threads to have work
+    while (threads > 64 && n4 <= threads) threads /= 2;
+    const int per = (n4 + threads - 1) / threads;
+    k = per <= 1   ? stream_sandwich_kernel<T, 1>
+        : per <= 2 ? stream_sandwich_kernel<T, 2>
+        : per <= 4 ? stream_sandwich_kernel<T, 4>
+                   : stream_sandwich_kernel<T, 8>;
+  }
+  return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), 0, stream, a) == cudaSuccess ? 0 : -5;
 }
 
 // c = ckv / rms(ckv) * w over R columns -> cache row `slot` of Rp columns (the rest stays zero).
@@ -175,7 +290,8 @@ latent_norm_cache_kernel(const T* __restrict__ ckv, long long ld, const float* _
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long n, int ff, int act) {
+gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long n, int ff, int act,
+                 const GateParams gp) {
   pdl_wait();
   pdl_trigger();
   // four outputs per thread: they share a block of kGateBlock
@@ -185,8 +301,8 @@ gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, long long n, int
     const int c = (int)(i - t * ff);
     const T* g = gu + t * 2 * ff + (c / kGateBlock) * (2 * kGateBlock) + c % kGateBlock;
     const float4 a = load4(g), b = load4(g + kGateBlock);
-    store4(out + i, make_float4(gate_act(act, a.x) * b.x, gate_act(act, a.y) * b.y,
-                                gate_act(act, a.z) * b.z, gate_act(act, a.w) * b.w));
+    store4(out + i, make_float4(gated(act, gp, a.x, b.x), gated(act, gp, a.y, b.y),
+                                gated(act, gp, a.z, b.z), gated(act, gp, a.w, b.w)));
   }
 }
 
@@ -212,27 +328,27 @@ typedef __nv_bfloat16 bf16;
 extern "C" {
 
 // dtype: 0 = bf16, 1 = fp32 (element type of weights, activations and caches)
-int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, long long T,
-                           int W, long long vocab, int dtype, int* status, cudaStream_t stream) {
+int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, float scale,
+                           long long T, int W, long long vocab, int dtype, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   cudaError_t e;
   if (dtype == 0)
     e = launch_pdl(stream_embedding_kernel<bf16>, dim3((unsigned)T), dim3(256), 0, stream,
                    reinterpret_cast<const long long*>(ids), reinterpret_cast<const bf16*>(table),
-                   reinterpret_cast<float*>(x), reinterpret_cast<bf16*>(act), W, vocab, status);
+                   reinterpret_cast<float*>(x), reinterpret_cast<bf16*>(act), scale, W, vocab, status);
   else
     e = launch_pdl(stream_embedding_kernel<float>, dim3((unsigned)T), dim3(256), 0, stream,
                    reinterpret_cast<const long long*>(ids), reinterpret_cast<const float*>(table),
-                   reinterpret_cast<float*>(x), reinterpret_cast<float*>(act), W, vocab, status);
+                   reinterpret_cast<float*>(x), reinterpret_cast<float*>(act), scale, W, vocab, status);
   return e == cudaSuccess ? 0 : -5;
 }
 
-// out rows t < T: norm(alpha * x[rows ? rows[t] : t] + y[t]) * (1 + weight). x_out may be x itself
+// out rows t < T: norm(alpha * x[rows ? rows[t] : t] + y[t]) * (offset + weight). x_out may be x itself
 // when rows is null (each block owns its row).
 int ab200_stream_norm(const void* x, const void* rows, const void* y, long long ldy,
                       const void* y_rows, const void* y_weights, int top, const void* weight,
-                      float alpha, float eps, void* x_out, void* act_out, long long T, int W,
-                      int dtype, cudaStream_t stream) {
+                      float alpha, float eps, float offset, void* x_out, void* act_out,
+                      long long T, int W, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   StreamNormArgs a;
   a.x = reinterpret_cast<const float*>(x);
@@ -245,10 +361,33 @@ int ab200_stream_norm(const void* x, const void* rows, const void* y, long long 
   a.weight = reinterpret_cast<const float*>(weight);
   a.alpha = alpha;
   a.eps = eps;
+  a.offset = offset;
   a.x_out = reinterpret_cast<float*>(x_out);
   a.act_out = act_out;
   a.W = W;
   return dtype == 0 ? launch_stream_norm<bf16>(a, T, stream) : launch_stream_norm<float>(a, T, stream);
+}
+
+// In place on x [T, W]: x += norm(y) * (offset + w_out) if y, += step if step; act = norm(x) *
+// (offset + w_in) if act.
+int ab200_stream_sandwich(void* x, const void* y, long long ldy, const void* w_out, const void* step,
+                          const void* w_in, void* act, float eps, float offset, long long T, int W,
+                          int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if ((y != nullptr && w_out == nullptr) || (act != nullptr && w_in == nullptr)) return -2;
+  SandwichArgs a;
+  a.x = reinterpret_cast<float*>(x);
+  a.y = y;
+  a.ldy = ldy;
+  a.w_out = reinterpret_cast<const float*>(w_out);
+  a.step = reinterpret_cast<const float*>(step);
+  a.w_in = reinterpret_cast<const float*>(w_in);
+  a.act = act;
+  a.eps = eps;
+  a.offset = offset;
+  a.W = W;
+  return dtype == 0 ? launch_stream_sandwich<bf16>(a, T, stream)
+                    : launch_stream_sandwich<float>(a, T, stream);
 }
 
 int ab200_latent_norm_cache(const void* ckv, long long ld, const void* weight, int R, int Rp,
@@ -272,20 +411,21 @@ int ab200_latent_norm_cache(const void* ckv, long long ld, const void* weight, i
 }
 
 // gu [T, 2 * ff] with gate and up columns alternating in blocks of 16 -> out [T, ff]
-int ab200_gated_act(const void* gu, void* out, long long T, int ff, int act, int dtype,
-                    cudaStream_t stream) {
+int ab200_gated_act(const void* gu, void* out, long long T, int ff, int act, float limit,
+                    float alpha, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (ff % kGateBlock || (act != kActSilu && act != kActGeluTanh)) return -2;
+  if (ff % kGateBlock || act < kActSilu || act > kActClampedSwish) return -2;
+  const GateParams gp = {limit, alpha};
   const long long n = T * ff;
   long long blocks = (n / 4 + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   cudaError_t e;
   if (dtype == 0)
     e = launch_pdl(gated_act_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, stream,
-                   reinterpret_cast<const bf16*>(gu), reinterpret_cast<bf16*>(out), n, ff, act);
+                   reinterpret_cast<const bf16*>(gu), reinterpret_cast<bf16*>(out), n, ff, act, gp);
   else
     e = launch_pdl(gated_act_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream,
-                   reinterpret_cast<const float*>(gu), reinterpret_cast<float*>(out), n, ff, act);
+                   reinterpret_cast<const float*>(gu), reinterpret_cast<float*>(out), n, ff, act, gp);
   return e == cudaSuccess ? 0 : -5;
 }
 

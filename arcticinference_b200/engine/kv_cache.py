@@ -226,24 +226,29 @@ class KVCacheTensors:
         self._tables = {}
 
 
-class LatentCacheTensors:
-    """Device memory of a latent cache: one tensor ``[num_blocks, 1, block_size, width]`` per
-    layer that projects latents of its own. A layer that takes an earlier layer's latents has
-    that layer's tensor (``k[l]`` is the same object), so it costs no memory. The block tables,
-    prefix cache and scheduler above it are those of any other model."""
+class RunCacheTensors:
+    """Device memory of a layer-list decoder's cache. Every run of a layer keeps one or two tensors
+    ``[num_blocks, heads, block_size, columns]``: keys and values, or latent rows. A run that takes
+    an earlier one's latents has that run's tensors (the same objects), so it costs no memory.
+    The block tables, prefix cache and scheduler above it are those of any other model."""
 
-    def __init__(self, owners: list, widths: list, num_blocks: int, block_size: int,
+    def __init__(self, owners: list, rows: list, num_blocks: int, block_size: int,
                  dtype: torch.dtype, device):
-        """``owners[l]``: the layer whose latents layer l reads; ``widths[l]``: columns of a row."""
-        self.k = []
-        for l, o in enumerate(owners):
-            self.k.append(self.k[o] if o != l else torch.zeros(
-                (num_blocks, 1, block_size, widths[l]), dtype=dtype, device=device))
+        """``owners[r]``: the run whose cache run r uses; ``rows[r]``: (heads, columns) of each of
+        its tensors."""
+        self.runs = []
+        for r, o in enumerate(owners):
+            self.runs.append(self.runs[o] if o != r else tuple(
+                torch.zeros((num_blocks, h, block_size, c), dtype=dtype, device=device)
+                for h, c in rows[r]))
+
+    def of(self, run: int) -> tuple:
+        return self.runs[run]
 
     @staticmethod
-    def bytes_per_block(owners: list, widths: list, block_size: int, elem_bytes: int) -> int:
-        return sum(w for l, (o, w) in enumerate(zip(owners, widths)) if o == l) * \
+    def bytes_per_block(owners: list, rows: list, block_size: int, elem_bytes: int) -> int:
+        return sum(h * c for r, (o, t) in enumerate(zip(owners, rows)) if o == r for h, c in t) * \
             block_size * elem_bytes
 
     def free(self) -> None:
-        self.k = []
+        self.runs = []

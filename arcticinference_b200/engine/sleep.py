@@ -16,7 +16,7 @@ import torch
 
 def _model_tensors(engine):
     m = engine.runner.model
-    items = [(m, n) for n in ("embed", "norm", "lm_head", "norm_swiftkv", "wkv_swiftkv")
+    items = [(m, n) for n in ("embed", "norm", "lm_head", "norm_swiftkv", "wkv_swiftkv", "loop_step")
              if hasattr(m, n)]
     for lw in m.layers:
         if lw is None:

@@ -822,8 +822,10 @@ class AttentionMetadata:
 
 def plan_attention_work(q_lens, kv_lens, G: int, causal: bool = True, num_sms: int = 148,
                         Hkv: int = 1, seq_rows=None, allow_split: bool = True,
-                        max_splits_cap: int = 16):
+                        max_splits_cap: int = 16, mask=None, align: int = 1):
     """Pure-host planner. Returns (work [n,8] int32 ndarray, tok_splits [T] int32, max_splits).
+    ``mask`` (a MaskSpec): a tile's keys start at the first one its rows see, rounded down to a
+    multiple of ``align`` (the cache's block size).
 
     Query tokens of a sequence are cut into tiles of 128/G tokens. When the call has too few
     tiles to occupy the GPU (decode), the keys of each sequence are cut into up to 16 splits
@@ -831,7 +833,9 @@ def plan_attention_work(q_lens, kv_lens, G: int, causal: bool = True, num_sms: i
     tpt = 128 // G
     if len(q_lens) >= 16 and max(q_lens) == 1 and min(q_lens) == 1:
         return _plan_decode_work(kv_lens, G, causal, num_sms, Hkv, seq_rows, allow_split,
-                                 max_splits_cap)
+                                 max_splits_cap, mask, align)
+    first = (lambda pos: 0) if mask is None else \
+        (lambda pos: int(mask.first_key(pos)) // align * align)
     rows = []
     T = int(sum(q_lens))
     tok_splits = np.ones(max(T, 1), dtype=np.int32)
@@ -844,7 +848,8 @@ def plan_attention_work(q_lens, kv_lens, G: int, causal: bool = True, num_sms: i
         if ql <= 0:
             continue
         seq_field = i if seq_rows is None else int(seq_rows[i])
-        key_tiles = (kl + TILE_KEYS - 1) // TILE_KEYS
+        lo = first(kl - ql)
+        key_tiles = (kl - lo + TILE_KEYS - 1) // TILE_KEYS
         ns = 1
         if allow_split and n_tiles_total * Hkv < num_sms and key_tiles > 4:
             want = max(1, num_sms // max(1, n_tiles_total * Hkv))
@@ -856,8 +861,10 @@ def plan_attention_work(q_lens, kv_lens, G: int, causal: bool = True, num_sms: i
             n = min(tpt, ql - a)
             q_pos0 = kl - ql + a
             for s in range(ns):
-                ks = s * tiles_per_split * TILE_KEYS
-                ke = min(kl, (s + 1) * tiles_per_split * TILE_KEYS)
+                ks = lo + s * tiles_per_split * TILE_KEYS
+                ke = min(kl, lo + (s + 1) * tiles_per_split * TILE_KEYS)
+                if ns == 1:
+                    ks = first(q_pos0)
                 rows.append((seq_field, t0 + a, n, q_pos0, ks, ke, s, ns))
         if ns > 1:
             tok_splits[t0:t0 + ql] = ns
@@ -885,14 +892,16 @@ def tail_split_plan(n_seqs: int, Hkv: int, slots: int, max_splits: int = 4):
     return -(-rem // Hkv), pieces
 
 
-def _plan_decode_work(kv_lens, G, causal, num_sms, Hkv, seq_rows, allow_split, max_splits_cap):
+def _plan_decode_work(kv_lens, G, causal, num_sms, Hkv, seq_rows, allow_split, max_splits_cap,
+                      mask=None, align=1):
     """The planner above for the one-token-per-sequence case, on arrays (same rows, same
     order): a serving step with a thousand sequences must not spend milliseconds here."""
     kl = np.asarray(kv_lens, dtype=np.int64)
     R = kl.size
     if G <= 32:
         num_sms *= 2
-    key_tiles = (kl + TILE_KEYS - 1) // TILE_KEYS
+    lo = np.zeros_like(kl) if mask is None else mask.first_key(kl - 1) // align * align
+    key_tiles = (kl - lo + TILE_KEYS - 1) // TILE_KEYS
     ns = np.ones(R, dtype=np.int64)
     if allow_split and R * Hkv < num_sms:
         want = max(1, num_sms // max(1, R * Hkv))
@@ -902,7 +911,7 @@ def _plan_decode_work(kv_lens, G, causal, num_sms, Hkv, seq_rows, allow_split, m
         n_cut, pieces = tail_split_plan(R, Hkv, num_sms, int(min(4, max_splits_cap)))
         if n_cut > 0:
             # the longest sequences are cut (at least 4 tiles per piece)
-            longest = np.argsort(-kl, kind="stable")[:n_cut]
+            longest = np.argsort(-(kl - lo), kind="stable")[:n_cut]
             longest = longest[key_tiles[longest] >= 4 * pieces]
             ns[longest] = pieces
     tps = (key_tiles + ns - 1) // ns
@@ -911,8 +920,8 @@ def _plan_decode_work(kv_lens, G, causal, num_sms, Hkv, seq_rows, allow_split, m
     rep = np.repeat(np.arange(R), ns)
     first = np.cumsum(ns) - ns
     sidx = np.arange(rep.size) - first[rep]                     # split index within its sequence
-    ks = sidx * tps[rep] * TILE_KEYS
-    ke = np.minimum(kl[rep], (sidx + 1) * tps[rep] * TILE_KEYS)
+    ks = lo[rep] + sidx * tps[rep] * TILE_KEYS
+    ke = np.minimum(kl[rep], lo[rep] + (sidx + 1) * tps[rep] * TILE_KEYS)
     work = np.stack([seq[rep], rep, np.ones_like(rep), kl[rep] - 1, ks, ke, sidx, ns[rep]], 1)
     if causal:
         order = np.argsort(-(np.minimum(ke, kl[rep]) - ks), kind="stable")
@@ -940,10 +949,12 @@ def pick_tile_keys(q_lens, G: int) -> int:
 
 def build_attention_metadata(q_lens, kv_lens, block_tables, G, Hq, D, device, causal=True,
                              Hkv=None, seq_rows=None, allow_split=True,
-                             work_capacity: int | None = None) -> AttentionMetadata:
+                             work_capacity: int | None = None, mask=None,
+                             align: int = 1) -> AttentionMetadata:
     Hkv = Hkv if Hkv is not None else Hq // G
     work, tok_splits, max_splits = plan_attention_work(q_lens, kv_lens, G, causal, Hkv=Hkv,
-                                                       seq_rows=seq_rows, allow_split=allow_split)
+                                                       seq_rows=seq_rows, allow_split=allow_split,
+                                                       mask=mask, align=align)
     T = int(sum(q_lens))
     n = work.shape[0]
     if work_capacity is not None:
@@ -969,7 +980,8 @@ class DecodePlan:
     them from the step's lengths. ``bind`` gives it its slices of the step's int32 buffers."""
 
     def __init__(self, G: int, Hq: int, Hkv: int, D: int, bucket: int, max_q: int,
-                 block_size: int):
+                 block_size: int, mask=None):
+        self.mask, self.block_size = mask, block_size
         self.G, self.Hq, self.Hkv, self.D, self.bucket = G, Hq, Hkv, D, bucket
         # enough KV splits to occupy the GPU when the batch is small; for a large batch the
         # sequences of the last, partly filled wave of CTAs are cut (tail_split_plan)
@@ -989,7 +1001,8 @@ class DecodePlan:
 
     def plan(self, q_lens, kv_lens):
         return plan_attention_work(q_lens, kv_lens, self.G, True, Hkv=self.Hkv,
-                                   max_splits_cap=self.splits)
+                                   max_splits_cap=self.splits, mask=self.mask,
+                                   align=self.block_size)
 
     def bind(self, host, dev: torch.Tensor, block_tables: torch.Tensor) -> None:
         """``host`` (numpy) and ``dev``: this plan's ``int32_words`` of the staging buffers."""
@@ -1042,6 +1055,36 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
         float(scale), out.data_ptr(), out.stride(0), nat.ptr(meta.o_part), nat.ptr(meta.lse_part),
         nat.ptr(lse_out), meta.tile_keys, nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "attention")
+    launch_counter.add(2 if meta.max_splits > 1 else 1)
+    return out
+
+
+def attention_masked(q, k, v, meta: AttentionMetadata, Hq: int, Hkv: int, D: int, scale: float, mask,
+                     sink=None, gate=None, out=None, paged: bool = True) -> torch.Tensor:
+    """Causal attention with a lower bound on the keys (``mask``, a MaskSpec), an optional sink
+    (fp32 [Hq]: a further term of the softmax denominator) and an optional output gate (rows
+    [T, Hq * D]; the output is multiplied by their sigmoid). CUDA tensors only. Keys and values:
+    caches [num_blocks, Hkv, block_size, D], or with ``paged`` false rows [n, Hkv * D]. ``meta``
+    must have been planned with the same mask."""
+    nat = _native()
+    T = q.shape[0]
+    if out is None:
+        out = torch.empty(T, Hq * D, dtype=q.dtype, device=q.device)
+    bt = meta.block_tables if paged else None
+    if paged:
+        assert bt.dtype == torch.int32 and bt.is_contiguous()
+        assert k.is_contiguous() and v.is_contiguous()
+    else:
+        assert k.stride(0) == v.stride(0)
+    rc = nat.lib().ab200_attention_ext(
+        q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), 0 if paged else k.stride(0),
+        k.shape[0], k.shape[2] if paged else 0, nat.ptr(bt), bt.shape[1] if paged else 0,
+        meta.work.data_ptr(), meta.num_work, nat.ptr(meta.tok_splits) if meta.max_splits > 1 else None,
+        meta.max_splits, T, Hq, Hkv, D, mask.code, mask.size, nat.ptr(sink), nat.ptr(gate),
+        gate.stride(0) if gate is not None else 0, float(scale), out.data_ptr(), out.stride(0),
+        nat.ptr(meta.o_part), nat.ptr(meta.lse_part), meta.tile_keys if paged else 128,
+        nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
+    nat.check(rc, "attention_masked")
     launch_counter.add(2 if meta.max_splits > 1 else 1)
     return out
 

@@ -4,8 +4,9 @@ CUDA tensors run ``csrc/stream.cu``, ``csrc/moe.cu``, ``csrc/grouped_gemm.cu`` a
 tensor-core kernels do not apply (32-bit models, rows that are no multiple of 16 bytes),
 ``csrc/exact.cu``. CPU tensors run the PyTorch restatements below.
 
-The stream is a pair: ``x`` fp32 [T, W] and ``act``, its rounding to the model's element type,
-which the projections read (the same tensor for a 32-bit model).
+The stream is ``x`` fp32 [T, W]; ``act`` is what the projections read, in the model's element
+type: the stream's rounding in decoders that normalise after the residual sum (the same tensor
+for a 32-bit model), its norm in those that normalise before the sublayer.
 """
 
 from __future__ import annotations
@@ -18,8 +19,31 @@ import torch.nn.functional as F
 from . import launch_counter
 
 GATE_BLOCK = 16       # gate / up rows alternate in blocks of this many (csrc/common/elem.cuh)
-ACT_CODE = {"silu": 1, "gelu_tanh": 2}
 TILE_ROWS = 128       # rows per tile of a grouped product
+
+
+@dataclass(frozen=True)
+class Gate:
+    """How a gated feed-forward joins its gate and up projections: silu(g) * u, gelu_tanh(g) * u or
+    clamped_swish: g' * sigmoid(alpha * g') * (u' + 1) with g' = min(g, limit) and u' clamped to
+    -limit .. limit. Functions that take a gate also take its name alone."""
+    name: str
+    limit: float = 0.0
+    alpha: float = 1.702
+
+    @staticmethod
+    def of(gate) -> "Gate":
+        return gate if isinstance(gate, Gate) else Gate(gate)
+
+    @property
+    def code(self) -> int:
+        return {"silu": 1, "gelu_tanh": 2, "clamped_swish": 3}[self.name]
+
+    def join(self, g: torch.Tensor, u: torch.Tensor) -> torch.Tensor:
+        if self.name == "clamped_swish":
+            g = g.clamp(max=self.limit)
+            return g * torch.sigmoid(self.alpha * g) * (u.clamp(-self.limit, self.limit) + 1.0)
+        return (F.silu(g) if self.name == "silu" else F.gelu(g, approximate="tanh")) * u
 
 
 def _nat():
@@ -35,33 +59,33 @@ def dtype_code(dt: torch.dtype) -> int:
     raise TypeError("element type %s" % dt)
 
 
-def activation(name: str, z: torch.Tensor) -> torch.Tensor:
-    return F.silu(z) if name == "silu" else F.gelu(z, approximate="tanh")
-
-
 # ------------------------------------------------------------------------ residual stream
-def stream_embedding(ids: torch.Tensor, table: torch.Tensor):
-    """(x, act) of the token embeddings."""
+def stream_embedding(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0,
+                     rounded: bool = True):
+    """(x, act) of the token embeddings times ``scale``; act is None unless ``rounded``."""
     if not table.is_cuda:
-        act = table[ids]
-        x = act.float()
-        return (x, x) if table.dtype == torch.float32 else (x, act)
+        x = table[ids].float() * scale
+        if not rounded:
+            return x, None
+        return (x, x) if table.dtype == torch.float32 else (x, x.to(table.dtype))
     nat = _nat()
     T, W = ids.numel(), table.shape[1]
     x = torch.empty(T, W, dtype=torch.float32, device=table.device)
-    act = x if table.dtype == torch.float32 else torch.empty(T, W, dtype=table.dtype,
-                                                             device=table.device)
+    act = None
+    if rounded:
+        act = x if table.dtype == torch.float32 else torch.empty(T, W, dtype=table.dtype,
+                                                                 device=table.device)
     rc = nat.lib().ab200_stream_embedding(
-        ids.data_ptr(), table.data_ptr(), x.data_ptr(), None if act is x else act.data_ptr(), T, W,
-        table.shape[0], dtype_code(table.dtype), nat.status_buffer(table.device).data_ptr(),
+        ids.data_ptr(), table.data_ptr(), x.data_ptr(), None if act is x else nat.ptr(act),
+        float(scale), T, W, table.shape[0], dtype_code(table.dtype), nat.status_buffer(table.device).data_ptr(),
         nat.stream_ptr())
     nat.check(rc, "stream_embedding")
     launch_counter.add(1)
     return x, act
 
 
-def _scaled_norm_ref(s, weight, eps):
-    return s / torch.sqrt(s.pow(2).mean(-1, keepdim=True) + eps) * (1.0 + weight)
+def _scaled_norm_ref(s, weight, eps, offset=1.0):
+    return s / torch.sqrt(s.pow(2).mean(-1, keepdim=True) + eps) * (offset + weight)
 
 
 def stream_norm(x, act, y, weight, alpha: float, eps: float, experts: "Routing" = None) -> None:
@@ -84,22 +108,49 @@ def stream_norm(x, act, y, weight, alpha: float, eps: float, experts: "Routing" 
         experts.rows.data_ptr() if experts is not None else None,
         experts.weights.data_ptr() if experts is not None else None,
         experts.top if experts is not None else 0, weight.data_ptr(), float(alpha), float(eps),
-        x.data_ptr(), None if act is x else act.data_ptr(), T, W, dtype_code(act.dtype),
+        1.0, x.data_ptr(), None if act is x else act.data_ptr(), T, W, dtype_code(act.dtype),
         nat.stream_ptr())
     nat.check(rc, "stream_norm")
     launch_counter.add(1)
 
 
-def stream_final_norm(x, rows, weight, eps: float, dtype: torch.dtype) -> torch.Tensor:
-    """norm(x[rows]) * (1 + weight), rounded to ``dtype``: the state the LM head reads."""
+def stream_sandwich(x, y=None, w_out=None, step=None, w_in=None, act=None, eps: float = 0.0,
+                    offset: float = 0.0) -> None:
+    """In place, in one pass over the rows of the stream: ``x += norm(y) * (offset + w_out)`` if a
+    sublayer's output ``y`` is given, ``x += step`` if a vector is; then ``act = norm(x) * (offset
+    + w_in)`` if ``act`` is given: what the next sublayer reads."""
+    T, W = x.shape
+    if not x.is_cuda:
+        if y is not None:
+            x += _scaled_norm_ref(y.float(), w_out, eps, offset)
+        if step is not None:
+            x += step
+        if act is not None:
+            act.copy_(_scaled_norm_ref(x, w_in, eps, offset))
+        return
+    nat = _nat()
+    dt = act.dtype if act is not None else y.dtype if y is not None else torch.float32
+    assert x.is_contiguous() and act is not x and (act is None or act.is_contiguous())
+    assert y is None or (y.stride(1) == 1 and y.dtype == dt)
+    rc = nat.lib().ab200_stream_sandwich(
+        x.data_ptr(), nat.ptr(y), y.stride(0) if y is not None else 0, nat.ptr(w_out),
+        nat.ptr(step), nat.ptr(w_in), nat.ptr(act), float(eps), float(offset), T, W,
+        dtype_code(dt), nat.stream_ptr())
+    nat.check(rc, "stream_sandwich")
+    launch_counter.add(1)
+
+
+def stream_final_norm(x, rows, weight, eps: float, dtype: torch.dtype,
+                      offset: float = 1.0) -> torch.Tensor:
+    """norm(x[rows]) * (offset + weight), rounded to ``dtype``: the state the LM head reads."""
     R, W = rows.numel(), x.shape[1]
     if not x.is_cuda:
-        return _scaled_norm_ref(x[rows], weight, eps).to(dtype)
+        return _scaled_norm_ref(x[rows], weight, eps, offset).to(dtype)
     nat = _nat()
     out = torch.empty(R, W, dtype=dtype, device=x.device)
     rc = nat.lib().ab200_stream_norm(x.data_ptr(), rows.data_ptr(), None, 0, None, None, 0,
-                                     weight.data_ptr(), 1.0, float(eps), None, out.data_ptr(), R, W,
-                                     dtype_code(dtype), nat.stream_ptr())
+                                     weight.data_ptr(), 1.0, float(eps), float(offset), None,
+                                     out.data_ptr(), R, W, dtype_code(dtype), nat.stream_ptr())
     nat.check(rc, "stream_final_norm")
     launch_counter.add(1)
     return out
@@ -123,19 +174,20 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 def _gated_ref(gu, act):
     T, n2 = gu.shape
     v = gu.float().reshape(T, n2 // (2 * GATE_BLOCK), 2, GATE_BLOCK)
-    return (activation(act, v[:, :, 0]) * v[:, :, 1]).reshape(T, n2 // 2).to(gu.dtype)
+    return Gate.of(act).join(v[:, :, 0], v[:, :, 1]).reshape(T, n2 // 2).to(gu.dtype)
 
 
-def gated_act(gu: torch.Tensor, act: str) -> torch.Tensor:
-    """act(gate) * up of the product with an interleaved gate / up matrix."""
+def gated_act(gu: torch.Tensor, act) -> torch.Tensor:
+    """``act`` (a Gate) of gate and up, from the product with an interleaved gate / up matrix."""
+    act = Gate.of(act)
     if not gu.is_cuda:
         return _gated_ref(gu, act)
     nat = _nat()
     assert gu.is_contiguous()
     T, ff = gu.shape[0], gu.shape[1] // 2
     out = torch.empty(T, ff, dtype=gu.dtype, device=gu.device)
-    rc = nat.lib().ab200_gated_act(gu.data_ptr(), out.data_ptr(), T, ff, ACT_CODE[act],
-                                   dtype_code(gu.dtype), nat.stream_ptr())
+    rc = nat.lib().ab200_gated_act(gu.data_ptr(), out.data_ptr(), T, ff, act.code, act.limit,
+                                   act.alpha, dtype_code(gu.dtype), nat.stream_ptr())
     nat.check(rc, "gated_act")
     launch_counter.add(1)
     return out
@@ -230,9 +282,10 @@ def _aligned(*ts) -> bool:
     return True
 
 
-def grouped_linear(x: torch.Tensor, w: torch.Tensor, routing: Routing, act: str = None):
+def grouped_linear(x: torch.Tensor, w: torch.Tensor, routing: Routing, act=None):
     """Rows sorted by expert [n, K] times each row's expert matrix of ``w`` [E, N, K]. With
-    ``act`` the matrices are interleaved gate / up ones and the result is act(gate) * up."""
+    ``act`` (a Gate) the matrices are interleaved gate / up ones, joined by it."""
+    act = None if act is None else Gate.of(act)
     n, K = x.shape
     E, N, _ = w.shape
     if not x.is_cuda:
@@ -246,8 +299,8 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, routing: Routing, act: str 
         rc = nat.lib().ab200_grouped_gemm(
             x.data_ptr(), x.stride(0), 0, n, w.data_ptr(), w.stride(1), w.stride(0),
             out.data_ptr(), out.stride(0), 0, 0, N, K, E, routing.tiles.data_ptr(),
-            routing.num_tiles.data_ptr(), routing.tiles.shape[0], ACT_CODE[act] if act else 0,
-            nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
+            routing.num_tiles.data_ptr(), routing.tiles.shape[0], act.code if act else 0,
+            act.limit if act else 0.0, act.alpha if act else 0.0, nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
         nat.check(rc, "grouped_gemm n=%d N=%d K=%d" % (n, N, K))
         launch_counter.add(1)
         return out
@@ -260,11 +313,12 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, routing: Routing, act: str 
     return gated_act(out, act) if act else out
 
 
-def gated_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
-    """act(gate) * up of a dense feed-forward: ``w`` [2 * ff, W] is an interleaved gate / up
-    matrix. Long inputs run one tensor-core kernel with the activation in its epilogue; short
+def gated_linear(x: torch.Tensor, w: torch.Tensor, act) -> torch.Tensor:
+    """Gate and up of a dense feed-forward joined by ``act`` (a Gate): ``w`` [2 * ff, W] is an
+    interleaved gate / up matrix. Long inputs run one tensor-core kernel with the activation in its epilogue; short
     ones the framework's decode GEMM (split over K) and a separate activation."""
     from . import linear
+    act = Gate.of(act)
     T = x.shape[0]
     if not x.is_cuda or T <= FUSED_GATE_MIN_TOKENS or not _aligned(x, w) or x.shape[1] % 8:
         return gated_act(linear(x, w), act)
@@ -273,7 +327,7 @@ def gated_linear(x: torch.Tensor, w: torch.Tensor, act: str) -> torch.Tensor:
     out = torch.empty(T, N // 2, dtype=x.dtype, device=x.device)
     rc = nat.lib().ab200_grouped_gemm(
         x.data_ptr(), x.stride(0), 0, T, w.data_ptr(), w.stride(0), 0, out.data_ptr(),
-        out.stride(0), 0, T, N, K, 1, None, None, 0, ACT_CODE[act],
+        out.stride(0), 0, T, N, K, 1, None, None, 0, act.code, act.limit, act.alpha,
         nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "gated_linear M=%d N=%d K=%d" % (T, N, K))
     launch_counter.add(1)
@@ -300,7 +354,7 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor = None) -> t
     if _aligned(x, w, out) and K % 8 == 0 and N % 8 == 0:
         rc = nat.lib().ab200_grouped_gemm(
             x.data_ptr(), x.stride(0), K, T, w.data_ptr(), w.stride(1), w.stride(0),
-            out.data_ptr(), out.stride(0), N, T, N, K, H, None, None, 0, 0,
+            out.data_ptr(), out.stride(0), N, T, N, K, H, None, None, 0, 0, 0.0, 0.0,
             nat.status_buffer(x.device).data_ptr(), nat.stream_ptr())
         nat.check(rc, "head_linear T=%d H=%d N=%d K=%d" % (T, H, N, K))
     else:

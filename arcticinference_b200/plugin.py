@@ -57,9 +57,9 @@ def _ensure_registered() -> None:
         from .models.llama import LlamaForCausalLM
         return LlamaForCausalLM(*a, **k)
 
-    def _taralix(*a, **k):
-        from .models.taralix import TaralixForCausalLM
-        return TaralixForCausalLM(*a, **k)
+    def _layer_list(*a, **k):
+        from .models.layer_list import LayerListForCausalLM
+        return LayerListForCausalLM(*a, **k)
 
     def _speculator(*a, **k):
         from .models.speculator import build_speculator
@@ -75,7 +75,10 @@ def _ensure_registered() -> None:
         register_model(arch, _llama)
     register_config("taralix", "layer list: latent attention with shared latents, dense and "
                                "mixture-of-experts feed-forwards")
-    register_model("Taralix", _taralix)
+    register_model("Taralix", _layer_list)
+    register_config("zatirax", "layer list: windowed latent attention with rotary keys, chunked "
+                               "attention with sinks and output gates, a loop over layers")
+    register_model("Zatirax", _layer_list)
     for arch in ("ArcticMLPSpeculatorPreTrainedModel", "ArcticLSTMSpeculatorPreTrainedModel",
                  "MLPVariantSpeculatorPreTrainedModel", "MLPSpeculatorPreTrainedModel"):
         register_model(arch, _speculator)

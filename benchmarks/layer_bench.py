@@ -143,8 +143,9 @@ def build_runner(cfg):
     r = ModelRunner(ec, "cuda")
     r.load_model()
     r.init_kv_cache(blocks)
-    for c in r.kv.k + getattr(r.kv, "v", []):     # a cache that holds something
-        c.normal_()
+    runs = getattr(r.kv, "runs", None)
+    for c in (r.kv.k + r.kv.v if runs is None else [t for run in runs for t in run]):
+        c.normal_()     # a cache that holds something
     return r
 
 

@@ -191,7 +191,7 @@ def test_shared_latents_take_no_memory(tmp_path):
     cfg = u.CONFIGS["mixed"]
     sess = u.session(u.save(tmp_path, cfg, u.weights(cfg)), "float32", 256, "cpu")
     kv, m = sess.engine.runner.kv, sess.engine.runner.model
-    assert kv.k[1] is kv.k[0] and kv.k[5] is kv.k[0] and kv.k[4] is kv.k[2]
+    assert kv.of(1) is kv.of(0) and kv.of(5) is kv.of(0) and kv.of(4) is kv.of(2)
     assert m.kv_bytes_per_block(64) == (56 + 72) * 64 * 4
 
 
