@@ -1,20 +1,23 @@
-"""Prefill and decode throughput of Taralix layers beside Llama layers of equal size (random
-weights), with the device time of every op and the time its roofline allows.
+"""Prefill and decode throughput of layer-list decoders (Taralix, Zatirax) beside Llama layers of
+equal size (random weights), with the device time of every op and the time its roofline allows.
 
     python bench.py --workload layers [--layer-case NAME]       (or: python benchmarks/layer_bench.py)
 
-Cases (width, heads x (dim, vdim), kv_rank, feed-forward), every second layer sharing the latents
-of the one before it:
+Cases (width, heads x (dim, vdim), kv_rank, feed-forward):
 
-    moe-2048     2048, 16 x (128, 128), 512, 64 experts of 1408, 6 per token
+    moe-2048     2048, 16 x (128, 128), 512, 64 experts of 1408, 6 per token   (Taralix)
     dense-2560   2560, 40 x (64, 64),   256, 6400
     dense-4096   4096, 32 x (128, 128), 512, 14336
+    masks-4096   dense-4096 with windows and chunks of 1024 positions          (Zatirax)
 
-The Llama beside each has the same width, query heads, head dimension and active feed-forward
-width, and 8 K/V heads. Prefill: four prompts of 2048 tokens in one step. Decode: 128 sequences at
-2000 tokens of context, captured step. Both are one forward pass without the LM head, timed with
-CUDA events; the weights of a pass exceed L2. The roofline of an op is the larger of its
-algorithmic bytes over the measured copy bandwidth and its flops over the measured bf16 rate.
+Taralix: every second layer shares the latents of the one before it. Zatirax: attention layers with
+8 K/V heads (a quarter of the dimensions rotated) alternate with latent layers that add a rotated
+key part of 64; windows and chunks of 4096 positions, which hold every context here, but in
+masks-4096. The Llama beside them has the same width, query heads, head dimension and active feed-forward width, and 8
+K/V heads. Prefill: four prompts of 2048 tokens in one step. Decode: 128 sequences at 2000 tokens of
+context, captured step. Both are one forward pass without the LM head, timed with CUDA events; the
+weights of a pass exceed L2. The roofline of an op is the larger of its algorithmic bytes over the
+measured copy bandwidth and its flops over the measured bf16 rate; only visible keys count.
 """
 
 from __future__ import annotations
@@ -31,13 +34,15 @@ CASES = {
     "moe-2048": dict(width=2048, heads=16, dim=128, rank=512, ff=1408, experts=64, top=6),
     "dense-2560": dict(width=2560, heads=40, dim=64, rank=256, ff=6400, experts=0, top=1),
     "dense-4096": dict(width=4096, heads=32, dim=128, rank=512, ff=14336, experts=0, top=1),
+    "masks-4096": dict(width=4096, heads=32, dim=128, rank=512, ff=14336, experts=0, top=1,
+                       mask=1024),
 }
-LAYERS, VOCAB, KV_HEADS = 4, 32000, 8
+LAYERS, VOCAB, KV_HEADS, ROT = 4, 32000, 8, 64
 PREFILL = [2048] * 4
 DECODE, CONTEXT = 128, 2000
 
 
-def model_configs(c):
+def taralix_config(c):
     from arcticinference_b200.config import ModelConfig
     mlp = {"kind": "dense", "ff": c["ff"]} if not c["experts"] else \
         {"kind": "moe", "expert": {"ff": c["ff"]},
@@ -49,14 +54,44 @@ def model_configs(c):
         if i % 2:
             m["kv_from"] = i - 1
         layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
-    tara = ModelConfig.from_layer_list({
+    return ModelConfig.from_layer_list({
         "architecture": "Taralix", "width": c["width"], "vocab": VOCAB, "norm": {"eps": 1e-6},
         "postln_alpha": 1.5, "layers": layers})
+
+
+def zatirax_config(c):
+    from arcticinference_b200.config import ModelConfig
+    H, d, size = c["heads"], c["dim"], c.get("mask", 4096)
+    rot = lambda n: {"base": 10000.0, "dims": n}
+    attn = {"type": "attention", "mixer": {
+        "heads": H, "kv_heads": KV_HEADS, "dim": d, "vdim": d, "scale": d ** -0.5,
+        "mask": {"size": size}, "rot": {**rot(d // 4), "scaling": {
+            "factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    latent = {"type": "latent_attention", "mixer": {
+        "heads": H, "dim": d, "rot_dim": ROT, "vdim": d, "kv_rank": c["rank"],
+        "scale": (d + ROT) ** -0.5, "mask": {"size": size}, "rot": rot(ROT)}}
+    mlp = {"kind": "dense", "ff": c["ff"], "limit": 7.0}
+    # runs: attention, latent, attention, latent
+    layers = [attn, latent, attn, latent][:LAYERS]
+    return ModelConfig.from_layer_list({
+        "architecture": "Zatirax", "width": c["width"], "vocab": VOCAB, "norm": {"eps": 1e-6},
+        "embedding": {"scale": 1.0}, "loop": None,
+        "layers": [{**l, "mlp": mlp} for l in layers]})
+
+
+def model_configs(c):
+    from arcticinference_b200.config import ModelConfig
     llama = ModelConfig(hidden_size=c["width"], num_hidden_layers=LAYERS,
                         num_attention_heads=c["heads"], num_key_value_heads=KV_HEADS,
                         head_dim=c["dim"], intermediate_size=c["ff"] * c["top"], vocab_size=VOCAB,
                         max_position_embeddings=8192)
-    return {"taralix": tara, "llama": llama}
+    out = {}
+    if not c["experts"]:
+        out["zatirax"] = zatirax_config(c)
+    if "mask" not in c:
+        out["taralix"] = taralix_config(c)
+        out["llama"] = llama
+    return out
 
 
 def peaks():
@@ -68,12 +103,23 @@ def peaks():
         return 6.65e12, 1.59e15, "of fallback"
 
 
-def rooflines(cfg, q_lens, kv_lens):
+def visible_pairs(mask, q_lens, kv_lens):
+    """(query, key) pairs that attend, and keys that any query of a sequence sees."""
+    import numpy as np
+    pairs = keys = 0
+    for q, kl in zip(q_lens, kv_lens):
+        pos = np.arange(kl - q, kl)
+        pairs += int((pos + 1 - mask.first_key(pos)).sum())
+        keys += kl - int(mask.first_key(kl - q))
+    return pairs, keys
+
+
+def rooflines(model, q_lens, kv_lens):
     """op -> seconds the layers' algorithmic bytes and flops allow (2 bytes per element)."""
+    from arcticinference_b200.config import AttentionSpec, MaskSpec
+    cfg = model.cfg
     hbm, flops, _ = peaks()
     T = sum(q_lens)
-    pairs = sum(q * kl - q * (q - 1) / 2 for q, kl in zip(q_lens, kv_lens))
-    ctx = sum(kv_lens)
     out: dict = {}
 
     def add(op, nbytes, nflops=0.0):
@@ -86,6 +132,7 @@ def rooflines(cfg, q_lens, kv_lens):
     decode = max(q_lens) == 1
     if cfg.layer_specs is None:
         H, Hk, D, I = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim, cfg.intermediate_size
+        pairs, ctx = visible_pairs(MaskSpec(), q_lens, kv_lens)
         for _ in range(cfg.num_hidden_layers):
             linear((H + 2 * Hk) * D, W)
             add("rope_cache", 2.0 * T * (2 * (H + Hk) + 3 * Hk) * D)
@@ -96,24 +143,42 @@ def rooflines(cfg, q_lens, kv_lens):
             linear(W, I)
             add("rmsnorm", 2 * 2.0 * T * 4 * W)
         return out
-    for l in cfg.layer_specs:
+    sandwich = cfg.design.residual == "sandwich"
+    for i, _ in cfg.layer_runs:
+        l = cfg.layer_specs[i]
         m, f = l.mixer, l.mlp
-        H, R, d = m.heads, m.kv_rank, m.dim
-        own = R if m.kv_from is None else 0
-        linear(H * d + own, W)
-        if own:
-            add("latent_norm_cache", 2.0 * T * 2 * R)
-        if decode:
-            add("head_linear", 2.0 * (H * R * d + T * H * (d + R)), 2.0 * T * H * R * d)
-            add("latent_attention", 2.0 * (ctx * R + 2 * T * H * R), 4.0 * pairs * H * R)
-            add("head_linear", 2.0 * (H * R * d + T * H * (d + R)), 2.0 * T * H * R * d)
+        H, d, dv = m.heads, m.dim, m.vdim
+        masked = m.mask.kind != "causal"
+        pairs, ctx = visible_pairs(m.mask, q_lens, kv_lens)
+        if isinstance(m, AttentionSpec):
+            G = m.kv_heads
+            linear(H * (d + dv) + G * (d + dv), W)
+            add("head_rope_cache", 2.0 * T * (2 * (H + G) * d + 2 * G * dv))
+            add("attention_masked", 2.0 * (ctx * G * (d + dv) + T * H * (d + 2 * dv)),
+                2.0 * pairs * H * (d + dv))
         else:
-            if own:
-                add("gather_rows", 2.0 * 2 * ctx * R)
-            linear(2 * H * d, R, rows=ctx)
-            add("attention_contiguous", 2.0 * (2 * ctx + 2 * T) * H * d, 4.0 * pairs * H * d)
-        linear(W, H * m.vdim)
-        add("stream_norm", T * W * 12.0)
+            R, rot = m.kv_rank, m.rot_dim
+            own = R + rot if m.kv_from is None else 0
+            dq = d + rot
+            linear(H * dq + own, W)
+            if rot:
+                add("latent_rope_cache", 2.0 * T * 2 * (R + rot + H * rot))
+            elif own:
+                add("latent_norm_cache", 2.0 * T * 2 * R)
+            if decode or not model.mixers[i].expand:
+                add("head_linear", 2.0 * (H * R * d + T * H * (dq + R + rot)), 2.0 * T * H * R * d)
+                add("latent_attention", 2.0 * (ctx * (R + rot) + T * H * (2 * R + rot)),
+                    2.0 * pairs * H * (2 * R + rot))
+                add("head_linear", 2.0 * (H * R * dv + T * H * (dv + R)), 2.0 * T * H * R * dv)
+            else:
+                if own:
+                    add("gather_rows", 2.0 * 2 * ctx * (R + rot))
+                linear(H * (d + dv), R, rows=ctx)
+                add("attention_masked" if masked else "attention_contiguous",
+                    2.0 * (ctx + T) * H * (dq + dv), 2.0 * pairs * H * (dq + dv))
+        linear(W, H * dv)
+        norm, per = ("stream_sandwich", 12.0) if sandwich else ("stream_norm", 12.0)
+        add(norm, T * W * per)
         if f.experts:
             n = T * f.top
             used = min(f.experts, n)
@@ -127,7 +192,7 @@ def rooflines(cfg, q_lens, kv_lens):
             if T <= 256:
                 add("gated_act", 2.0 * T * 3 * f.ff)
             linear(W, f.ff)
-            add("stream_norm", T * W * 12.0)
+            add(norm, T * W * per)
     return out
 
 
@@ -206,7 +271,7 @@ def measure(name, cfg):
                 for _ in range(5):
                     fwd()
             q = [n if new is None else new for n in lens]
-            ideal = rooflines(cfg, q, lens)
+            ideal = rooflines(r.model, q, lens)
             table = {}
             for op, (us, cnt) in t.summary().items():
                 if op == "_start":
@@ -231,7 +296,7 @@ def fwd_graph(r, g):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("--layer-case", choices=sorted(CASES), default=None)
-    ap.add_argument("--model", choices=["taralix", "llama"], default=None)
+    ap.add_argument("--model", choices=["zatirax", "taralix", "llama"], default=None)
     ns = ap.parse_args(argv)
     import torch
     torch.cuda.set_device(0)

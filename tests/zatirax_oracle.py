@@ -6,6 +6,7 @@ test.
 checkpoint's names.
 """
 
+import functools
 import math
 
 import torch
@@ -62,6 +63,7 @@ def in_chunk(i, j, size):
     return j <= i and i // size == j // size
 
 
+@functools.lru_cache(maxsize=64)
 def visible(seen, n, size):
     return torch.tensor([[seen(i, j, size) for j in range(n)] for i in range(n)], dtype=torch.bool)
 
