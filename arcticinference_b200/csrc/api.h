@@ -110,7 +110,7 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
 int ab200_attention_ext(const void* q, long long ldq, const void* k, const void* v, long long ld_kv,
                         long long num_blocks, int block_size, const void* block_tables,
                         int max_blocks, const void* work, int num_work, const void* tok_splits,
-                        int max_splits, long long T, int Hq, int Hkv, int D, int mask_kind,
+                        int max_splits, long long T, int Hq, int Hkv, int Dk, int D, int mask_kind,
                         int mask_size, const void* sink, const void* gate, long long ldg,
                         float scale, void* out, long long ldo, void* o_part, void* lse_part,
                         int tile_keys, int* status, cudaStream_t stream);

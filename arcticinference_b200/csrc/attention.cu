@@ -19,6 +19,10 @@
 // calls (a handful of query rows per sequence) use 64-wide tiles, whose smaller
 // footprint (112 KB of shared memory, 256 TMEM columns, < 170 registers) lets two
 // CTAs share an SM and overlap one CTA's softmax with the other's loads.
+// Queries and keys may be wider than values (DK = 192, DV = 128: an expanded latent attention with
+// a rotated part); those take 64-wide key tiles with the prefill arrangement of warps.
+// The MMA warp walks its loop with warp-uniform values and one elected lane issues: descriptors
+// then live in uniform registers and an instruction costs what the tensor core takes.
 //
 // Instances with EXT also take a mask with a lower bound (a window, or chunks of positions: the
 // planner starts a tile's keys at the first one its rows see, the softmax masks the rest), a
@@ -53,9 +57,10 @@ namespace ab200 {
 // latency of its TMEM reads and exponentials, and the softmax, not the tensor core, was the
 // longest stage of a prefill tile), four for the 64-key decode tiles, whose two CTAs per SM
 // already give every scheduler two softmax warps. Then the TMA warp and the MMA warp.
-template <int TK>
+template <int DK, int TK>
 struct AttnShape {
-  static constexpr int kSoftmaxWarps = (TK == 128) ? 8 : 4;
+  static constexpr bool kPrefill = TK == 128 || DK > 128;
+  static constexpr int kSoftmaxWarps = kPrefill ? 8 : 4;
   static constexpr int kThreads = (kSoftmaxWarps + 2) * 32;
 };
 
@@ -114,21 +119,21 @@ __device__ __forceinline__ uint4 gate8(const uint4& v, const uint4& g) {
   return make_uint4(r[0], r[1], r[2], r[3]);
 }
 
-template <int D, int TK, bool EXT>
-__global__ void __launch_bounds__(AttnShape<TK>::kThreads, (TK == 64 ? 2 : 1))
+template <int DK, int D, int TK, bool EXT>   // D: columns of values and outputs
+__global__ void __launch_bounds__(AttnShape<DK, TK>::kThreads, (AttnShape<DK, TK>::kPrefill ? 1 : 2))
 attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const AttnArgs p) {
-  constexpr int kHalves = D / 64;
-  constexpr uint32_t kQBytes = 128 * D * 2;
-  constexpr uint32_t kKVBytes = TK * D * 2;
+  constexpr bool kPrefill = AttnShape<DK, TK>::kPrefill;
+  constexpr uint32_t kQBytes = 128 * DK * 2;
+  constexpr uint32_t kKBytes = TK * DK * 2, kVBytes = TK * D * 2;
   constexpr uint32_t kPBytes = 128 * TK * 2;
   constexpr uint32_t kHalf = TK * 128;     // bytes of one 64-wide d half of a K/V stage
   constexpr int kChunks = TK / 32;         // 32-column chunks of a row of S
   constexpr uint32_t kTmemCols = (TK == 128) ? 512 : 256;  // 2 S buffers + O
-  constexpr int kPStages = (TK == 128) ? 2 : 1;  // decode tiles share the SM with a second CTA
-  constexpr int kSW = AttnShape<TK>::kSoftmaxWarps;
+  constexpr int kPStages = kPrefill ? 2 : 1;  // decode tiles share the SM with a second CTA
+  constexpr int kSW = AttnShape<DK, TK>::kSoftmaxWarps;
   constexpr int kHalves2 = kSW / 4;                // warps per lane quadrant
-  constexpr int kAttThreads = AttnShape<TK>::kThreads;
+  constexpr int kAttThreads = AttnShape<DK, TK>::kThreads;
   constexpr int kTmaWarp = kSW, kMmaWarp = kSW + 1;
   // per-row values the two warps of a quadrant hand each other: tile maxima (double-buffered
   // by tile parity) and, at the end, the partial row sums
@@ -153,10 +158,11 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
   }
   const uint32_t sQ = smem_u32(smem);
   const uint32_t sK = sQ + kQBytes;          // 2 stages
-  const uint32_t sV = sK + 2 * kKVBytes;     // 2 stages
-  const uint32_t sP = sV + 2 * kKVBytes;
-  uint8_t* pP = smem + kQBytes + 4 * kKVBytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kQBytes + 4 * kKVBytes + kPStages * kPBytes);
+  const uint32_t sV = sK + 2 * kKBytes;      // 2 stages
+  const uint32_t sP = sV + 2 * kVBytes;
+  uint8_t* pV = smem + kQBytes + 2 * kKBytes;
+  uint8_t* pP = pV + 2 * kVBytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(pP + kPStages * kPBytes);
   const uint32_t bb = smem_u32(bars);
   // barrier indices
   const uint32_t q_full = bb;
@@ -220,14 +226,20 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     tmem_alloc(smem_u32(tmem_slot), kTmemCols);
     tmem_relinquish();
   }
-  // Stale shared memory may hold non-finite bit patterns; keys that are never
-  // loaded (past the end of a sequence) are multiplied by P = 0 and must be finite.
   for (int i = threadIdx.x; i < 256; i += kAttThreads) (&pair_seq[0][0])[i] = 0;
   // (counts stay far below 32767: a sequence of 2^21 keys is 16384 tiles)
-  {
-    uint4* z = reinterpret_cast<uint4*>(smem + kQBytes);
-    const uint4 zero = make_uint4(0, 0, 0, 0);
-    for (int i = threadIdx.x; i < (int)(4 * kKVBytes / 16); i += kAttThreads) z[i] = zero;
+  // Stale shared memory may hold non-finite bit patterns; values that are never loaded (the last
+  // tile's, past the sequence's last block) meet P = 0 and must be finite. A stage that an
+  // earlier tile has filled is. (Scores of such keys are replaced before anything reads them.)
+  if (p.block_size > 0 && (n_tiles == 1 || n_tiles == 2)) {
+    const int last = kv_end - kv_start - (n_tiles - 1) * TK;
+    const int r_first = (last + p.block_size - 1) / p.block_size * p.block_size;
+    const int vecs = (TK - r_first) * 8;
+#pragma unroll
+    for (int h = 0; h < D / 64; ++h) {
+      uint4* z = reinterpret_cast<uint4*>(pV + (n_tiles - 1) * kVBytes + h * kHalf + r_first * 128);
+      for (int i = threadIdx.x; i < vecs; i += kAttThreads) z[i] = make_uint4(0, 0, 0, 0);
+    }
   }
   fence_proxy_async_smem();
   tc_fence_before();
@@ -242,7 +254,7 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     // ------------------------------ TMA producer ------------------------------
     if (lane == 0) {
       mbar_arrive_expect_tx(q_full, kQBytes);
-      for (int h = 0; h < kHalves; ++h)
+      for (int h = 0; h < DK / 64; ++h)
         tma_load_4d(sQ + h * 16384u, &tmap_q, q_full, h * 64, 0, kvh, q_tok0);
     }
     const int bs = p.block_size;
@@ -256,7 +268,8 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
       for (int kv = 0; kv < 2; ++kv) {
         const uint32_t full = kv == 0 ? k_full(st) : v_full(st);
         const uint32_t empty = kv == 0 ? k_empty(st) : v_empty(st);
-        const uint32_t dst = (kv == 0 ? sK : sV) + (uint32_t)st * kKVBytes;
+        const uint32_t dst = kv == 0 ? sK + (uint32_t)st * kKBytes : sV + (uint32_t)st * kVBytes;
+        const int halves = (kv == 0 ? DK : D) / 64;
         const CUtensorMap* tm = kv == 0 ? &tmap_k : &tmap_v;
         if (!mbar_wait(empty, ph ^ 1u, abort_flag, p.status, 500 + kv * 10 + st, j)) {
           ok = false;
@@ -264,18 +277,18 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         }
         if (bs > 0) {
           const int nblk = (nkeys + bs - 1) / bs;
-          if (lane == 0) mbar_arrive_expect_tx(full, (uint32_t)(nblk * bs * D * 2));
+          if (lane == 0) mbar_arrive_expect_tx(full, (uint32_t)(nblk * bs * halves * 128));
           __syncwarp();
           if (lane < nblk) {
             const int bid = bt[key0 / bs + lane];
-            for (int h = 0; h < kHalves; ++h)
+            for (int h = 0; h < halves; ++h)
               tma_load_4d(dst + h * kHalf + (uint32_t)(lane * bs) * 128u, tm, full, h * 64, 0, kvh,
                           bid);
           }
         } else {
           if (lane == 0) {
-            mbar_arrive_expect_tx(full, kKVBytes);
-            for (int h = 0; h < kHalves; ++h)
+            mbar_arrive_expect_tx(full, (uint32_t)(TK * halves * 128));
+            for (int h = 0; h < halves; ++h)
               tma_load_3d(dst + h * kHalf, tm, full, h * 64, kvh, seq + key0);
           }
         }
@@ -284,47 +297,57 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     }
   } else if (warp == kMmaWarp) {
     // ------------------------------- MMA issuer -------------------------------
-    if (lane == 0 && n_tiles > 0) {
+    if (n_tiles > 0) {
       const uint32_t idesc_s = make_idesc(128, TK, 1, 1, 0, 0);
       const uint32_t idesc_pv = make_idesc(128, D, 1, 1, 0, 1);
-      bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 600, 0);
+      const uint32_t tm = __shfl_sync(0xffffffffu, tmem_base, 0);
+      const uint32_t tS_u = tm, tO_u = tm + 2 * TK;
+      const uint64_t q_d = make_desc_kmajor_sw128(sQ), k_d = make_desc_kmajor_sw128(sK);
+      const uint64_t p_d = make_desc_kmajor_sw128(sP), v_d = make_desc_mnmajor_sw128(sV, kHalf);
+      auto wait = [&](uint32_t bar, uint32_t parity, int code, int j) -> bool {
+        return __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag, p.status, code, j));
+      };
+      bool ok = wait(q_full, 0, 600, 0);
       auto issue_s = [&](int j) -> bool {
         const int st = j & 1;
         const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-        if (!mbar_wait(k_full(st), ph, abort_flag, p.status, 610 + st, j)) return false;
-        if (!mbar_wait(s_empty(st), ph ^ 1u, abort_flag, p.status, 620 + st, j)) return false;
+        if (!wait(k_full(st), ph, 610 + st, j)) return false;
+        if (!wait(s_empty(st), ph ^ 1u, 620 + st, j)) return false;
         tc_fence_after();
-        const uint32_t kb = sK + (uint32_t)st * kKVBytes;
+        const uint64_t kd = k_d + (uint64_t)(st * (int)(kKBytes / 16));
+        if (elect_one()) {
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) {
-          const uint64_t qd = make_desc_kmajor_sw128(sQ + (uint32_t)(k / 4) * 16384u) + 2u * (k % 4);
-          const uint64_t kd = make_desc_kmajor_sw128(kb + (uint32_t)(k / 4) * kHalf) + 2u * (k % 4);
-          umma_f16_ss(tS + (uint32_t)st * TK, qd, kd, idesc_s, k > 0 ? 1u : 0u);
+          for (int k = 0; k < DK / 16; ++k)
+            umma_f16_ss(tS_u + (uint32_t)st * TK, q_d + (uint64_t)((k / 4) * 1024 + 2 * (k % 4)),
+                        kd + (uint64_t)((k / 4) * (int)(kHalf / 16) + 2 * (k % 4)), idesc_s,
+                        k > 0 ? 1u : 0u);
+          tc_commit(k_empty(st));
+          tc_commit(s_full(st));
         }
-        tc_commit(k_empty(st));
-        tc_commit(s_full(st));
+        __syncwarp();
         return true;
       };
       auto issue_pv = [&](int j) -> bool {
         const int st = j & 1;
         const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-        if (!mbar_wait(v_full(st), ph, abort_flag, p.status, 630 + st, j)) return false;
+        if (!wait(v_full(st), ph, 630 + st, j)) return false;
         // P(j) sits in buffer j % kPStages; its barrier completes once per use of that buffer
         const int pst = j % kPStages;
         const uint32_t pph = (uint32_t)(j / kPStages) & 1u;
-        if (!mbar_wait(p_full(pst), pph, abort_flag, p.status, 640, j)) return false;
+        if (!wait(p_full(pst), pph, 640, j)) return false;
         tc_fence_after();
-        const uint32_t vb = sV + (uint32_t)st * kKVBytes;
-        const uint32_t pb = sP + (uint32_t)pst * kPBytes;
-#pragma unroll
-        for (int k = 0; k < TK / 16; ++k) {
-          const uint64_t pd = make_desc_kmajor_sw128(pb + (uint32_t)(k / 4) * 16384u) + 2u * (k % 4);
-          const uint64_t vd = make_desc_mnmajor_sw128(vb, kHalf) + 128u * k;
+        const uint64_t vd = v_d + (uint64_t)(st * (int)(kVBytes / 16));
+        const uint64_t pd = p_d + (uint64_t)(pst * (int)(kPBytes / 16));
+        if (elect_one()) {
           // O accumulates in tensor memory across key tiles
-          umma_f16_ss(tO, pd, vd, idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
+#pragma unroll
+          for (int k = 0; k < TK / 16; ++k)
+            umma_f16_ss(tO_u, pd + (uint64_t)((k / 4) * 1024 + 2 * (k % 4)), vd + (uint64_t)(128 * k),
+                        idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
+          tc_commit(v_empty(st));
+          tc_commit(o_full(st));
         }
-        tc_commit(v_empty(st));
-        tc_commit(o_full(st));
+        __syncwarp();
         return true;
       };
       if (ok) ok = issue_s(0);
@@ -542,6 +565,22 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         mbar_arrive(p_full(j % kPStages));
       }
     }
+    // The gate's pieces that this lane will multiply at the end are on their way while the last
+    // product finishes (the wide arrangement only: a decode CTA has a second one beside it).
+    constexpr int kCh = D / 8;   // 16-byte chunks per row
+    constexpr int kHeld = (EXT && kPrefill) ? kCh / kHalves2 : 1;
+    uint4 gates[kHeld];
+    if (EXT && kPrefill && p.gate != nullptr && num_splits <= 1 && warp_active) {
+#pragma unroll
+      for (int i = 0; i < kHeld; ++i) {
+        const int rr = quad * 32 + (i * kHalves2 + half) * (32 / kCh) + lane / kCh;
+        gates[i] = make_uint4(0, 0, 0, 0);
+        if (rr / p.G < n_q_tok && rr % p.G < p.g_heads)
+          gates[i] = *reinterpret_cast<const uint4*>(
+              p.gate + (long long)(q_tok0 + rr / p.G) * p.ldg +
+              (long long)(kvh * p.g_heads + rr % p.G) * D + 8 * (lane % kCh));
+      }
+    }
     if (ok && n_tiles > 0 && warp_active) {
       const int jl = n_tiles - 1;
       if (!mbar_wait(o_full(jl & 1), (uint32_t)(jl >> 1) & 1u, abort_flag, p.status, 720, jl))
@@ -580,7 +619,6 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         // has completed; same 128-byte swizzle, so the writes are conflict-free) and leave as
         // whole rows: one store instruction covers 32 / (D / 8) complete rows of D bf16 instead
         // of 16-byte pieces of 32 different rows -- what a peer's memory over NVLink needs.
-        constexpr int kCh = D / 8;  // 16-byte chunks per row
         uint8_t* my_row = smem + (size_t)row * 128;
 #pragma unroll
         for (int cl = 0; cl < D / 32 / kHalves2; ++cl) {
@@ -617,10 +655,14 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
           if (d != 0ull) {
             uint4 q = *reinterpret_cast<const uint4*>(
                 smem + (size_t)(j >> 3) * 16384 + (size_t)rr * 128 + (((j & 7) ^ (rr & 7)) * 16));
-            if (EXT && p.gate != nullptr)
-              q = gate8(q, *reinterpret_cast<const uint4*>(
-                               p.gate + (long long)(q_tok0 + rr / p.G) * p.ldg +
-                               (long long)(kvh * p.g_heads + rr % p.G) * D + 8 * j));
+            if (EXT && p.gate != nullptr) {
+              if (kPrefill)
+                q = gate8(q, gates[it / kHalves2 % kHeld]);
+              else
+                q = gate8(q, *reinterpret_cast<const uint4*>(
+                                 p.gate + (long long)(q_tok0 + rr / p.G) * p.ldg +
+                                 (long long)(kvh * p.g_heads + rr % p.G) * D + 8 * j));
+            }
             *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(d) + 8 * j) = q;
           }
         }
@@ -745,7 +787,7 @@ struct AttnExt {
   long long ldg;
 };
 
-template <int D, int TK, bool EXT>
+template <int DK, int D, int TK, bool EXT>
 static int launch_attention(const void* q, long long ldq, const void* k, const void* v,
                             long long ld_kv, long long num_blocks, int block_size,
                             const int* block_tables, int max_blocks, const int* work, int num_work,
@@ -761,14 +803,16 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   if (peer_tokens > 0 && (world < 1 || world > 16 || peer_ptrs == nullptr)) return -2;
   if (heads <= 0 || Hq % Hkv || G > 128) return -2;
   if (block_size > 0 && (TK % block_size || block_size < 8)) return -2;
+  if (DK != D && block_size > 0) return -2;   // wider keys: contiguous rows only
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return -3;
   const size_t smem =
-      128 * D * 2 + 4 * (size_t)TK * D * 2 + (TK == 128 ? 2 : 1) * (size_t)128 * TK * 2 + 256;
+      128 * DK * 2 + 2 * (size_t)TK * (DK + D) * 2 +
+      (AttnShape<DK, TK>::kPrefill ? 2 : 1) * (size_t)128 * TK * 2 + 256;
   if (!attr_set[dev]) {
-    if (cudaFuncSetAttribute(attention_kernel<D, TK, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attention_kernel<DK, D, TK, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)smem) != cudaSuccess)
       return -3;
     attr_set[dev] = true;
@@ -776,8 +820,8 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   CUtensorMap tq, tk, tv;
   {
     // q viewed as [T][Hkv][heads][D]; the box is G heads high, rows past `heads` read as zero
-    const uint64_t dims[4] = {(uint64_t)D, (uint64_t)heads, (uint64_t)Hkv, (uint64_t)T};
-    const uint64_t strides[3] = {(uint64_t)D * 2, (uint64_t)heads * D * 2, (uint64_t)ldq * 2};
+    const uint64_t dims[4] = {(uint64_t)DK, (uint64_t)heads, (uint64_t)Hkv, (uint64_t)T};
+    const uint64_t strides[3] = {(uint64_t)DK * 2, (uint64_t)heads * DK * 2, (uint64_t)ldq * 2};
     const uint32_t box[4] = {64, (uint32_t)G, 1, (uint32_t)(128 / G)};
     if (make_tmap_nd(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, dims, strides, box) != 0) return -4;
   }
@@ -790,10 +834,12 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
     if (make_tmap_nd(&tv, v, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, dims, strides, box) != 0) return -4;
   } else {
     // contiguous: k/v rows are tokens with stride ld_kv, heads packed [Hkv][D]
-    const uint64_t dims[3] = {(uint64_t)D, (uint64_t)Hkv, (uint64_t)num_blocks /* = rows */};
-    const uint64_t strides[2] = {(uint64_t)D * 2, (uint64_t)ld_kv * 2};
+    uint64_t dims[3] = {(uint64_t)DK, (uint64_t)Hkv, (uint64_t)num_blocks /* = rows */};
+    uint64_t strides[2] = {(uint64_t)DK * 2, (uint64_t)ld_kv * 2};
     const uint32_t box[3] = {64, 1, (uint32_t)TK};
     if (make_tmap_nd(&tk, k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, strides, box) != 0) return -4;
+    dims[0] = (uint64_t)D;
+    strides[0] = (uint64_t)D * 2;
     if (make_tmap_nd(&tv, v, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, strides, box) != 0) return -4;
   }
   AttnArgs a;
@@ -839,7 +885,7 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   }
   if (max_splits <= 1) a.sig = sig;
   dim3 grid((unsigned)num_work * (unsigned)Hkv);
-  (void)launch_pdl(attention_kernel<D, TK, EXT>, grid, dim3(AttnShape<TK>::kThreads), smem, stream, tq,
+  (void)launch_pdl(attention_kernel<DK, D, TK, EXT>, grid, dim3(AttnShape<DK, TK>::kThreads), smem, stream, tq,
                    tk, tv, a);
   if (cudaGetLastError() != cudaSuccess) return -5;
   a.sig = sig;
@@ -858,14 +904,14 @@ using namespace ab200;
 
 extern "C" {
 
-#define AB200_ATTN_DISPATCH(EXT, ...)                                                     \
-  do {                                                                                 \
-    const bool small = tile_keys == 64 && (block_size == 0 || block_size <= 64);        \
-    if (D == 128) return small ? launch_attention<128, 64, EXT>(__VA_ARGS__)                \
-                               : launch_attention<128, 128, EXT>(__VA_ARGS__);              \
-    if (D == 64) return small ? launch_attention<64, 64, EXT>(__VA_ARGS__)                  \
-                              : launch_attention<64, 128, EXT>(__VA_ARGS__);                \
-    return -2;                                                                         \
+#define AB200_ATTN_DISPATCH(EXT, ...)                                                      \
+  do {                                                                                     \
+    const bool small = tile_keys == 64 && (block_size == 0 || block_size <= 64);           \
+    if (D == 128) return small ? launch_attention<128, 128, 64, EXT>(__VA_ARGS__)          \
+                               : launch_attention<128, 128, 128, EXT>(__VA_ARGS__);        \
+    if (D == 64) return small ? launch_attention<64, 64, 64, EXT>(__VA_ARGS__)             \
+                              : launch_attention<64, 64, 128, EXT>(__VA_ARGS__);           \
+    return -2;                                                                             \
   } while (0)
 
 // q: [T, Hq*D] rows with stride ldq. Paged mode (block_size > 0): k/v are caches
@@ -894,10 +940,12 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
 // The same with a mask (0 causal, 1 window, 2 chunk, see first_visible), an optional sink per query
 // head (fp32 [Hq]) and an optional output gate (bf16 rows of stride ldg, columns like out's).
 // Always causal; the work list's kv_start must not lie above the first key a tile's rows see.
+// Queries and keys have Dk columns per head, values and outputs D; they may differ (192, 128) with
+// contiguous keys and values.
 int ab200_attention_ext(const void* q, long long ldq, const void* k, const void* v, long long ld_kv,
                         long long num_blocks, int block_size, const void* block_tables,
                         int max_blocks, const void* work, int num_work, const void* tok_splits,
-                        int max_splits, long long T, int Hq, int Hkv, int D, int mask_kind,
+                        int max_splits, long long T, int Hq, int Hkv, int Dk, int D, int mask_kind,
                         int mask_size, const void* sink, const void* gate, long long ldg,
                         float scale, void* out, long long ldo, void* o_part, void* lse_part,
                         int tile_keys, int* status, cudaStream_t stream) {
@@ -908,6 +956,14 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
   if (gate != nullptr && ((ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
   const AttnExt ext = {mask_kind, mask_size, sink, gate, ldg};
+  if (Dk == 192 && D == 128)
+    return launch_attention<192, 128, 64, true>(
+        q, ldq, k, v, ld_kv, num_blocks, block_size, reinterpret_cast<const int*>(block_tables),
+        max_blocks, reinterpret_cast<const int*>(work), num_work,
+        reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, 1, scale, out, ldo,
+        reinterpret_cast<float*>(o_part), reinterpret_cast<float*>(lse_part), nullptr, status, stream,
+        nullptr, 0, 0, nullptr, &ext);
+  if (Dk != D) return -2;
   AB200_ATTN_DISPATCH(true, q, ldq, k, v, ld_kv, num_blocks, block_size,
                       reinterpret_cast<const int*>(block_tables), max_blocks,
                       reinterpret_cast<const int*>(work), num_work,

@@ -143,7 +143,7 @@ class LayerListForCausalLM:
         if exp:
             q = sum(m.cost for m in exp) / sum(m.gain for m in exp)
             self.expand_min_tokens = max(128, min(512, int(q)))
-        self._expand_row_bytes = max((2 * m.spec.heads * m.expand * 2 for m in exp), default=0)
+        self._expand_row_bytes = max((2 * m.spec.heads * sum(m.expand) for m in exp), default=0)
         # captured steps need a plan per shape; the "exact" kernels and 32-bit models run eagerly
         self.supports_graphs = self.dtype == torch.bfloat16 and all(m.capturable for m in self.mixers)
 
@@ -292,7 +292,7 @@ class LayerListForCausalLM:
         if key not in step.exp_plans:
             rows = np.asarray(kv_lens) - np.asarray(lo)
             step.exp_plans[key] = ops.build_attention_metadata(
-                q_lens, kv_lens, None, 1, H, m.expand, self.device, Hkv=H,
+                q_lens, kv_lens, None, 1, H, m.expand[1], self.device, Hkv=H,
                 seq_rows=np.cumsum(rows) - rows - np.asarray(lo), allow_split=False, mask=mask)
 
     def decode_plans(self, bucket: int, max_q: int, block_size: int) -> list:

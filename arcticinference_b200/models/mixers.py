@@ -83,21 +83,20 @@ class LatentMixer:
                                         spec.mask)
         self.freq = frequencies(spec.rotary if spec.rot_dim else None, device)
         self.dq0 = spec.dim + spec.rot_dim
-        # expanded form of long chunks: width of its keys and values, None where it does not pay.
+        # expanded form of long chunks: widths of its keys and values, None where it does not pay.
         # ``gain``: multiply-adds saved per query, key and head; ``cost``: spent per row of the
         # context and head. A bounded mask spreads a row's cost over fewer queries.
         self.expand = None
         self.gain = self.cost = 0.0
-        d = max(self.dq0, spec.vdim)
-        if bf16 and self.shape.kernel != "packed" and d <= 128:
-            d = 64 if d <= 64 else 128
-            gain = self.layout.width + self.layout.rank - 2 * d
-            cost = self.layout.width * 2 * d
+        wide = lat.expanded_widths(self.dq0, spec.vdim)
+        if bf16 and self.shape.kernel != "packed" and wide is not None:
+            gain = self.layout.width + self.layout.rank - sum(wide)
+            cost = self.layout.width * sum(wide)
             if spec.mask.kind != "causal":
                 gain -= cost / spec.mask.size
-            if d <= self.layout.rank and gain > 0:
-                self.expand, self.gain, self.cost = d, spec.heads * gain, spec.heads * cost
-        self.dq, self.dv = self.expand or self.dq0, self.expand or spec.vdim
+            if wide[1] <= self.layout.rank and gain > 0:
+                self.expand, self.gain, self.cost = wide, spec.heads * gain, spec.heads * cost
+        self.dq, self.dv = self.expand or (self.dq0, spec.vdim)
         if bf16:
             self.dq, self.dv = round_up(self.dq, 8), round_up(self.dv, 8)
 

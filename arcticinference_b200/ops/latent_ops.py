@@ -201,7 +201,7 @@ class AttentionStep:
     # mask -> (cache rows of the keys its expanded sequences see, one sequence after the other,
     # and how many of each sequence's first keys are left out)
     ctx: dict = field(default_factory=dict)
-    exp_plans: dict = field(default_factory=dict)   # (heads, D, mask) -> AttentionMetadata
+    exp_plans: dict = field(default_factory=dict)   # (heads, widths, mask) -> AttentionMetadata
 
     @property
     def uploaded_bytes(self) -> int:
@@ -353,22 +353,33 @@ def latent_attention(q: torch.Tensor, cache: torch.Tensor, meta: AttentionMetada
     return out
 
 
-def expanded_attention(q, k, v, step: AttentionStep, H: int, D: int, scale: float, out,
+def expanded_widths(dq: int, dv: int):
+    """(columns of keys, of values) the expanded form stores per head: what the attention kernel
+    has; None when it has nothing that wide."""
+    if max(dq, dv) <= 64:
+        return 64, 64
+    if max(dq, dv) <= 128:
+        return 128, 128
+    return (192, 128) if dq <= 192 and dv <= 128 else None
+
+
+def expanded_attention(q, k, v, step: AttentionStep, H: int, widths: tuple, scale: float, out,
                        mask: MaskSpec = CAUSAL) -> None:
     """Attention of the step's long chunks over expanded keys and values (rows of ``k`` and ``v``:
-    the keys those sequences see, one sequence after the other, as ``step.ctx[mask]`` names
-    them)."""
+    the keys those sequences see, one sequence after the other, as ``step.ctx[mask]`` names them;
+    ``widths``: columns of a head of each)."""
+    Dk, D = widths
     if q.is_cuda:
-        meta = step.exp_plans[(H, D, mask)]
-        if mask.kind == "causal":
+        meta = step.exp_plans[(H, widths, mask)]
+        if mask.kind == "causal" and Dk == D:
             attention_contiguous(q, k, v, None, H, D, scale, causal=True, meta=meta, out=out)
         else:
-            attention_masked(q, k, v, meta, H, H, D, scale, mask, out=out, paged=False)
+            attention_masked(q, k, v, meta, H, H, D, scale, mask, out=out, paged=False, Dk=Dk)
         return
     t = r = 0
     for n, kl, lo in zip(step.exp_q_lens, step.exp_kv_lens, step.ctx[mask][1]):
-        qs = q[t:t + n].reshape(n, H, D).float()
-        ks, vs = (z[r:r + kl - lo].reshape(kl - lo, H, D).float() for z in (k, v))
+        qs = q[t:t + n].reshape(n, H, Dk).float()
+        ks, vs = (z[r:r + kl - lo].reshape(kl - lo, H, d).float() for z, d in ((k, Dk), (v, D)))
         s = torch.einsum("thd,khd->htk", qs, ks) * scale
         at, pos = torch.arange(kl - n, kl).view(n, 1), torch.arange(lo, kl)
         s = s.masked_fill((pos > at) | (pos < mask.first_key(at)), float("-inf"))

@@ -141,7 +141,7 @@ def _declare(L: ctypes.CDLL) -> None:
                                    F, P, P]),
         "ab200_latent_attention": (I, [P, LL, P, I, I, P, I, P, I, P, I, LL, I, I, I, I, I, I, F, P,
                                        P, P, P, P]),
-        "ab200_attention_ext": (I, [P, LL, P, P, LL, LL, I, P, I, P, I, P, I, LL, I, I, I, I, I, P,
+        "ab200_attention_ext": (I, [P, LL, P, P, LL, LL, I, P, I, P, I, P, I, LL, I, I, I, I, I, I, P,
                                     P, LL, F, P, LL, P, P, I, P, P]),
         "ab200_attention": (I, [P, LL, P, P, LL, LL, I, P, I, P, I, P, I, LL, I, I, I, I, F, P,
                                 LL, P, P, P, I, P, P]),

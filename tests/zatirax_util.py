@@ -69,6 +69,15 @@ CONFIGS = {
 }
 
 
+# windows long enough that long chunks go through expanded keys and values, and one that is not
+EXPANDED = config(128, 90, [
+    (latent(5, 16, 16, 24, 200, 150), (48, 1.0)),
+    (latent(3, 96, 32, 128, 480, 200), None),
+    (latent(4, 128, 64, 128, 500, 250), (56, 2.0)),
+    (latent(2, 72, 64, 40, 300, 260), None),
+    (latent(6, 40, 24, 32, 160, 30), None),
+    (attention(4, 2, 64, 64, 120, rotary(32)), None)], eps=1e-3)
+
 # how far single keys stand out (heads of a few dimensions do by themselves, in 16 bits too far)
 PEAK = {"mixed": 1.0, "wide_latents": 1.0, "all_looped": 1.0, "odd": 0.0}
 
