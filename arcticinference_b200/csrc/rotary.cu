@@ -9,6 +9,8 @@
 //
 // A block owns a token: its sines and cosines are computed once (angle = position * frequency in
 // fp32, as are the norms), and its warps walk the heads. Dimension i is paired with i + rot / 2.
+// Heads of 64 or 128 bf16 columns stay in registers, four columns a lane and several heads in
+// flight; a pair's other half then comes from another lane.
 // T is the model's element type (bf16 or fp32).
 
 #include "api.h"
@@ -128,6 +130,80 @@ __global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const Hea
   }
 }
 
+// D = Dv = 64 or 128, half a multiple of 4
+template <int D>
+__global__ void __launch_bounds__(kRopeThreads) head_rope_cache_wide_kernel(const HeadRopeArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  constexpr int kLanes = D / 4;                 // per head
+  constexpr int kPer = 32 / kLanes;             // heads per warp
+  constexpr int kStep = kPer * kRopeThreads / 32;
+  constexpr int kFlight = 3;                    // heads per lane in flight
+  __shared__ float cs[D];
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int i0 = (lane % kLanes) * 4;           // this lane's columns
+  const int j0 = warp * kPer + lane / kLanes;   // its first head
+  const int heads = p.Hq + 2 * p.Hkv;
+  long long slot = p.slots[t];
+  if (slot >= p.num_slots) {
+    if (threadIdx.x == 0) report_error(p.status, kErrBounds, 43, (int)t);
+    slot = -1;
+  }
+  const long long blk = slot >= 0 ? slot / p.block_size : 0;
+  const long long off = slot >= 0 ? slot % p.block_size : 0;
+  __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(p.proj) + t * p.ld + i0;
+  const int side = i0 < p.half ? 0 : i0 < 2 * p.half ? 1 : 2;   // first, second of a pair, neither
+  const int other = side == 0 ? lane + p.half / 4 : side == 1 ? lane - p.half / 4 : lane;
+  float c[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int first = 0; first < heads; first += kStep * kFlight) {
+    float4 v[kFlight];
+#pragma unroll
+    for (int f = 0; f < kFlight; ++f) {
+      const int j = first + f * kStep + j0;
+      v[f] = j < heads ? load4(base + (long long)j * D) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (first == 0) {   // (the heads are on their way)
+      angles(cs, p.freq, p.half, p.positions[t]);
+      __syncthreads();
+      if (side < 2) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int k = 2 * (i0 - side * p.half + e);
+          c[e] = cs[k];
+          sn[e] = side == 0 ? -cs[k + 1] : cs[k + 1];
+        }
+      }
+    }
+#pragma unroll
+    for (int f = 0; f < kFlight; ++f) {
+      const int j = first + f * kStep + j0;
+      const bool is_v = j >= p.Hq + p.Hkv;
+      float4 x = v[f];
+      float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+#pragma unroll
+      for (int o = kLanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (p.wq != nullptr && !is_v) {
+        const float inv = 1.f / sqrtf(ss * p.rdim + p.eps);
+        const float4 w = load4((j < p.Hq ? p.wq : p.wk) + i0);
+        x = make_float4(x.x * inv * w.x, x.y * inv * w.y, x.z * inv * w.z, x.w * inv * w.w);
+      }
+      const float4 y = make_float4(__shfl_sync(0xffffffffu, x.x, other), __shfl_sync(0xffffffffu, x.y, other),
+                                   __shfl_sync(0xffffffffu, x.z, other), __shfl_sync(0xffffffffu, x.w, other));
+      if (!is_v)
+        x = make_float4(x.x * c[0] + y.x * sn[0], x.y * c[1] + y.y * sn[1], x.z * c[2] + y.z * sn[2],
+                        x.w * c[3] + y.w * sn[3]);
+      if (j < p.Hq) {
+        store4(base + (long long)j * D, x);
+      } else if (j < heads && slot >= 0) {
+        const int g = is_v ? j - p.Hq - p.Hkv : j - p.Hq;
+        __nv_bfloat16* cache = reinterpret_cast<__nv_bfloat16*>(is_v ? p.v_cache : p.k_cache);
+        store4(cache + ((blk * p.Hkv + g) * p.block_size + off) * D + i0, x);
+      }
+    }
+  }
+}
+
 struct LatentRopeArgs {
   void* q;                  // [T][ld]: H heads of dq columns, the rotary part from column dim
   const void* ckv;          // [T][ld]: R latent columns, then 2 * half rotary ones
@@ -190,6 +266,11 @@ static int launch_head_rope(const HeadRopeArgs& a, long long n, cudaStream_t str
                    ((reinterpret_cast<uintptr_t>(a.proj) | reinterpret_cast<uintptr_t>(a.wq) |
                      reinterpret_cast<uintptr_t>(a.wk) | reinterpret_cast<uintptr_t>(a.k_cache) |
                      reinterpret_cast<uintptr_t>(a.v_cache)) & 15) == 0;
+  if (sizeof(T) == 2 && vec && a.D == a.Dv && (a.D == 64 || a.D == 128) && a.half % 4 == 0)
+    return launch_pdl(a.D == 128 ? head_rope_cache_wide_kernel<128> : head_rope_cache_wide_kernel<64>,
+                      dim3((unsigned)n), dim3(kRopeThreads), 0, stream, a) == cudaSuccess
+               ? 0
+               : -5;
   auto k = vec ? head_rope_cache_kernel<T, true> : head_rope_cache_kernel<T, false>;
   if (smem > 48 * 1024 &&
       cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)

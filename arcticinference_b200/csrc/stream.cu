@@ -32,6 +32,16 @@ stream_embedding_kernel(const long long* __restrict__ ids, const T* __restrict__
   // (-1 stands for a token that is not known yet, when a decode step is captured)
   if (id >= vocab && threadIdx.x == 0) report_error(status, kErrBounds, 40, (int)t);
   const T* src = table + (ok ? id : 0) * W;
+  if (W % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(x) |
+                      reinterpret_cast<uintptr_t>(act)) & 15) == 0) {
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      float4 v = ok ? load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+      store4(x + t * W + i, v);
+      if (act != nullptr) store4(act + t * W + i, v);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     const float v = ok ? to_f32<T>(src[i]) * scale : 0.f;
     x[t * W + i] = v;
