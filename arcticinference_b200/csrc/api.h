@@ -265,16 +265,17 @@ int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row
                           int mask_size, float scale, int dtype, int* status, cudaStream_t stream);
 
 // ---- rotary.cu
-int ab200_head_rope_cache(void* proj, long long ld, const void* positions, const void* slots,
-                          const void* wq, const void* wk, const void* freq, int half, void* k_cache,
+int ab200_rotary_table(const void* positions, const void* freq, void* table, long long T, int half,
+                       cudaStream_t stream);
+int ab200_head_rope_cache(void* proj, long long ld, const void* table, int half,
+                          const void* slots, const void* wq, const void* wk, void* k_cache,
                           void* v_cache, long long T, int Hq, int Hkv, int D, int dim, int Dv,
                           int block_size, long long num_slots, float eps, int dtype, int* status,
                           cudaStream_t stream);
-int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* positions,
-                            const void* slots, const void* weight, const void* freq, int half,
-                            void* cache, long long T, int H, int dq, int dim, int R, int width,
-                            int rot_at, long long num_slots, float eps, int dtype, int* status,
-                            cudaStream_t stream);
+int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* table, int half,
+                            const void* slots, const void* weight, void* cache, long long T, int H,
+                            int dq, int dim, int R, int width, int rot_at, long long num_slots,
+                            float eps, int dtype, int* status, cudaStream_t stream);
 
 // ---- moe.cu
 int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,

@@ -1,16 +1,17 @@
 // What lies between an attention layer's input projection and its scores, for layers with
 // partial rotary positions:
 //
+//   rotary_table       cosine and sine of every token's angles (angle = position * frequency in
+//                      fp32), once per step for all layers with the same frequencies
 //   head_rope_cache    per-head RMS norm of queries and keys (optional), rotation of their first
 //                      rot dimensions, queries in place, keys and values to the paged cache
 //   latent_rope_cache  RMS norm of a compressed K/V projection and rotation of the key part that
 //                      the heads share, both to the paged latent cache; rotation of every query
 //                      head's rotary part in place
 //
-// A block owns a token: its sines and cosines are computed once (angle = position * frequency in
-// fp32, as are the norms), and its warps walk the heads. Dimension i is paired with i + rot / 2.
-// Heads of 64 or 128 bf16 columns stay in registers, four columns a lane and several heads in
-// flight; a pair's other half then comes from another lane.
+// A block owns a token and its warps walk the heads; norms and rotations are fp32. Dimension i is
+// paired with i + rot / 2. Heads of 64 or 128 bf16 columns stay in registers, four columns a lane
+// and several heads in flight; a pair's other half then comes from another lane.
 // T is the model's element type (bf16 or fp32).
 
 #include "api.h"
@@ -21,13 +22,20 @@ namespace ab200 {
 
 constexpr int kRopeThreads = 256;
 
-// cs[2 * i], cs[2 * i + 1]: cosine and sine of pair i
-__device__ __forceinline__ void angles(float* cs, const float* __restrict__ freq, int half,
-                                       long long pos) {
-  for (int i = threadIdx.x; i < half; i += blockDim.x)
-    sincosf((float)pos * freq[i], &cs[2 * i + 1], &cs[2 * i]);
+__global__ void __launch_bounds__(256)
+rotary_table_kernel(const long long* __restrict__ positions, const float* __restrict__ freq,
+                    float2* __restrict__ table, int half, long long n) {
+  pdl_wait();
+  pdl_trigger();
+  const long long k = blockIdx.x * (long long)blockDim.x + threadIdx.x;
+  if (k >= n) return;
+  const long long t = k / half;
+  float s, c;
+  sincosf((float)positions[t] * freq[k - t * half], &s, &c);
+  table[k] = make_float2(c, s);
 }
 
+// cs[2 * i], cs[2 * i + 1]: cosine and sine of pair i
 __device__ __forceinline__ float rotated(const float* row, const float* cs, int half, int i) {
   if (i < half) return row[i] * cs[2 * i] - row[i + half] * cs[2 * i + 1];
   if (i < 2 * half) return row[i] * cs[2 * (i - half)] + row[i - half] * cs[2 * (i - half) + 1];
@@ -37,11 +45,10 @@ __device__ __forceinline__ float rotated(const float* row, const float* cs, int 
 struct HeadRopeArgs {
   void* proj;               // [T][ld]: Hq query heads, Hkv key heads of D, Hkv value heads of Dv
   long long ld;
-  const long long* positions;
+  const float* table;       // [T][half][2]
   const long long* slots;
   const float* wq;          // [D] or null: no norm
   const float* wk;
-  const float* freq;        // [half]
   void* k_cache;            // [num_blocks][Hkv][block_size][D]
   void* v_cache;            // [num_blocks][Hkv][block_size][Dv]
   long long num_slots;
@@ -59,7 +66,7 @@ __global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const Hea
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* cs = sm + (kRopeThreads / 32) * p.D;
   float* row = sm + warp * p.D;
-  angles(cs, p.freq, p.half, p.positions[t]);
+  for (int i = threadIdx.x; i < 2 * p.half; i += blockDim.x) cs[i] = p.table[t * 2 * p.half + i];
   __syncthreads();
   long long slot = p.slots[t];
   if (slot >= p.num_slots) {
@@ -132,73 +139,82 @@ __global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const Hea
 
 // D = Dv = 64 or 128, half a multiple of 4
 template <int D>
-__global__ void __launch_bounds__(kRopeThreads) head_rope_cache_wide_kernel(const HeadRopeArgs p) {
+__global__ void __launch_bounds__(kRopeThreads, 4) head_rope_cache_wide_kernel(const HeadRopeArgs p) {
   pdl_wait();
   pdl_trigger();
   constexpr int kLanes = D / 4;                 // per head
   constexpr int kPer = 32 / kLanes;             // heads per warp
   constexpr int kStep = kPer * kRopeThreads / 32;
-  constexpr int kFlight = 3;                    // heads per lane in flight
-  __shared__ float cs[D];
+  constexpr int kFlight = 6;                    // heads per lane in flight
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int i0 = (lane % kLanes) * 4;           // this lane's columns
   const int j0 = warp * kPer + lane / kLanes;   // its first head
   const int heads = p.Hq + 2 * p.Hkv;
-  long long slot = p.slots[t];
-  if (slot >= p.num_slots) {
-    if (threadIdx.x == 0) report_error(p.status, kErrBounds, 43, (int)t);
-    slot = -1;
-  }
-  const long long blk = slot >= 0 ? slot / p.block_size : 0;
-  const long long off = slot >= 0 ? slot % p.block_size : 0;
   __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(p.proj) + t * p.ld + i0;
   const int side = i0 < p.half ? 0 : i0 < 2 * p.half ? 1 : 2;   // first, second of a pair, neither
   const int other = side == 0 ? lane + p.half / 4 : side == 1 ? lane - p.half / 4 : lane;
-  float c[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
-  for (int first = 0; first < heads; first += kStep * kFlight) {
-    float4 v[kFlight];
+  float4 v[kFlight];
+  auto load = [&](int first) {
 #pragma unroll
     for (int f = 0; f < kFlight; ++f) {
       const int j = first + f * kStep + j0;
       v[f] = j < heads ? load4(base + (long long)j * D) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    if (first == 0) {   // (the heads are on their way)
-      angles(cs, p.freq, p.half, p.positions[t]);
-      __syncthreads();
-      if (side < 2) {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int k = 2 * (i0 - side * p.half + e);
-          c[e] = cs[k];
-          sn[e] = side == 0 ? -cs[k + 1] : cs[k + 1];
-        }
-      }
-    }
+  };
+  load(0);
+  const long long slot = p.slots[t];
+  float4 c = make_float4(1.f, 1.f, 1.f, 1.f), sn = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (side < 2) {
+    const float* cs = p.table + (t * p.half + i0 - side * p.half) * 2;
+    const float4 a = load4(cs), b = load4(cs + 4);
+    const float sg = side == 0 ? -1.f : 1.f;
+    c = make_float4(a.x, a.z, b.x, b.z);
+    sn = make_float4(sg * a.y, sg * a.w, sg * b.y, sg * b.w);
+  }
+  float4 wq = make_float4(1.f, 1.f, 1.f, 1.f), wk = wq;
+  if (p.wq != nullptr) {
+    wq = load4(p.wq + i0);
+    wk = load4(p.wk + i0);
+  }
+  long long row0 = -1;   // cache row of K/V head 0 (-1: padding token)
+  if (slot >= p.num_slots) {
+    if (threadIdx.x == 0) report_error(p.status, kErrBounds, 43, (int)t);
+  } else if (slot >= 0) {   // (fewer than 2^31 slots)
+    const unsigned blk = (unsigned)slot / (unsigned)p.block_size;
+    row0 = (long long)blk * p.Hkv * p.block_size + ((unsigned)slot - blk * p.block_size);
+  }
+  for (int first = 0; first < heads; first += kStep * kFlight) {
+    if (first > 0) load(first);
 #pragma unroll
     for (int f = 0; f < kFlight; ++f) {
+      if (first + f * kStep >= heads) break;
       const int j = first + f * kStep + j0;
       const bool is_v = j >= p.Hq + p.Hkv;
       float4 x = v[f];
-      float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+      if (first + f * kStep + warp * kPer < p.Hq + p.Hkv) {   // (else all of the warp's are values)
+        float4 z = x;
+        if (p.wq != nullptr) {
+          float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
 #pragma unroll
-      for (int o = kLanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      if (p.wq != nullptr && !is_v) {
-        const float inv = 1.f / sqrtf(ss * p.rdim + p.eps);
-        const float4 w = load4((j < p.Hq ? p.wq : p.wk) + i0);
-        x = make_float4(x.x * inv * w.x, x.y * inv * w.y, x.z * inv * w.z, x.w * inv * w.w);
+          for (int o = kLanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+          const float inv = rsqrtf(ss * p.rdim + p.eps);
+          const float4 w = j < p.Hq ? wq : wk;
+          z = make_float4(x.x * inv * w.x, x.y * inv * w.y, x.z * inv * w.z, x.w * inv * w.w);
+        }
+        const float4 y = make_float4(
+            __shfl_sync(0xffffffffu, z.x, other), __shfl_sync(0xffffffffu, z.y, other),
+            __shfl_sync(0xffffffffu, z.z, other), __shfl_sync(0xffffffffu, z.w, other));
+        if (!is_v)
+          x = make_float4(z.x * c.x + y.x * sn.x, z.y * c.y + y.y * sn.y, z.z * c.z + y.z * sn.z,
+                          z.w * c.w + y.w * sn.w);
       }
-      const float4 y = make_float4(__shfl_sync(0xffffffffu, x.x, other), __shfl_sync(0xffffffffu, x.y, other),
-                                   __shfl_sync(0xffffffffu, x.z, other), __shfl_sync(0xffffffffu, x.w, other));
-      if (!is_v)
-        x = make_float4(x.x * c[0] + y.x * sn[0], x.y * c[1] + y.y * sn[1], x.z * c[2] + y.z * sn[2],
-                        x.w * c[3] + y.w * sn[3]);
       if (j < p.Hq) {
         store4(base + (long long)j * D, x);
-      } else if (j < heads && slot >= 0) {
+      } else if (j < heads && row0 >= 0) {
         const int g = is_v ? j - p.Hq - p.Hkv : j - p.Hq;
         __nv_bfloat16* cache = reinterpret_cast<__nv_bfloat16*>(is_v ? p.v_cache : p.k_cache);
-        store4(cache + ((blk * p.Hkv + g) * p.block_size + off) * D + i0, x);
+        store4(cache + (row0 + g * p.block_size) * D + i0, x);
       }
     }
   }
@@ -208,13 +224,13 @@ struct LatentRopeArgs {
   void* q;                  // [T][ld]: H heads of dq columns, the rotary part from column dim
   const void* ckv;          // [T][ld]: R latent columns, then 2 * half rotary ones
   long long ld;
-  const long long* positions;
+  const float* table;       // [T][half][2]
   const long long* slots;
   const float* weight;      // [R]
-  const float* freq;        // [half]
   void* cache;              // rows of `width` columns, the rotary key part from column rot_at
   long long num_slots;
   int H, dq, dim, R, half, width, rot_at;
+  int vec;                  // four columns at a time are aligned
   float eps;
   int* status;
 };
@@ -226,7 +242,7 @@ __global__ void __launch_bounds__(kRopeThreads) latent_rope_cache_kernel(const L
   extern __shared__ __align__(16) float cs[];
   __shared__ float red[32];
   const long long t = blockIdx.x;
-  angles(cs, p.freq, p.half, p.positions[t]);
+  for (int i = threadIdx.x; i < 2 * p.half; i += blockDim.x) cs[i] = p.table[t * 2 * p.half + i];
   const T* c = reinterpret_cast<const T*>(p.ckv) + t * p.ld;
   float ss = 0.f;
   for (int i = threadIdx.x; i < p.R; i += blockDim.x) {
@@ -248,6 +264,20 @@ __global__ void __launch_bounds__(kRopeThreads) latent_rope_cache_kernel(const L
     }
   }
   T* q = reinterpret_cast<T*>(p.q) + t * p.ld;
+  if (p.vec) {   // four pairs a thread
+    const int quads = p.half / 4, n = p.H * quads;
+    for (int k = threadIdx.x; k < n; k += blockDim.x) {
+      const int h = k / quads, i = (k - h * quads) * 4;
+      T* a = q + (long long)h * p.dq + p.dim + i;
+      const float4 u = load4(a), v = load4(a + p.half);
+      const float* g = cs + 2 * i;
+      store4(a, make_float4(u.x * g[0] - v.x * g[1], u.y * g[2] - v.y * g[3], u.z * g[4] - v.z * g[5],
+                            u.w * g[6] - v.w * g[7]));
+      store4(a + p.half, make_float4(v.x * g[0] + u.x * g[1], v.y * g[2] + u.y * g[3],
+                                     v.z * g[4] + u.z * g[5], v.w * g[6] + u.w * g[7]));
+    }
+    return;
+  }
   const int n = p.H * p.half;
   for (int k = threadIdx.x; k < n; k += blockDim.x) {
     const int h = k / p.half, i = k - h * p.half;
@@ -266,7 +296,8 @@ static int launch_head_rope(const HeadRopeArgs& a, long long n, cudaStream_t str
                    ((reinterpret_cast<uintptr_t>(a.proj) | reinterpret_cast<uintptr_t>(a.wq) |
                      reinterpret_cast<uintptr_t>(a.wk) | reinterpret_cast<uintptr_t>(a.k_cache) |
                      reinterpret_cast<uintptr_t>(a.v_cache)) & 15) == 0;
-  if (sizeof(T) == 2 && vec && a.D == a.Dv && (a.D == 64 || a.D == 128) && a.half % 4 == 0)
+  if (sizeof(T) == 2 && vec && a.D == a.Dv && (a.D == 64 || a.D == 128) && a.half % 4 == 0 &&
+      a.num_slots <= 0x7fffffffll && (a.wq == nullptr || a.wk != nullptr))
     return launch_pdl(a.D == 128 ? head_rope_cache_wide_kernel<128> : head_rope_cache_wide_kernel<64>,
                       dim3((unsigned)n), dim3(kRopeThreads), 0, stream, a) == cudaSuccess
                ? 0
@@ -285,11 +316,25 @@ typedef __nv_bfloat16 bf16;
 
 extern "C" {
 
+// positions int64 [T], freq fp32 [half] -> table fp32 [T, half, 2]: cosine, sine
+int ab200_rotary_table(const void* positions, const void* freq, void* table, long long T, int half,
+                       cudaStream_t stream) {
+  const long long n = T * half;
+  if (n <= 0) return 0;
+  if (n > (1ll << 38)) return -6;
+  return launch_pdl(rotary_table_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream,
+                    reinterpret_cast<const long long*>(positions),
+                    reinterpret_cast<const float*>(freq), reinterpret_cast<float2*>(table), half,
+                    n) == cudaSuccess
+             ? 0
+             : -5;
+}
+
 // proj [T, ld] holds Hq query and Hkv key heads of D columns, then Hkv value heads of Dv, of which
 // the first `dim` (query, key) columns are in use and the others zero; wq, wk fp32 [D] or null;
-// freq fp32 [half]: rotary frequencies of the pairs (i, i + half).
-int ab200_head_rope_cache(void* proj, long long ld, const void* positions, const void* slots,
-                          const void* wq, const void* wk, const void* freq, int half, void* k_cache,
+// table fp32 [T, half, 2]: cosines and sines of the pairs (i, i + half).
+int ab200_head_rope_cache(void* proj, long long ld, const void* table, int half,
+                          const void* slots, const void* wq, const void* wk, void* k_cache,
                           void* v_cache, long long T, int Hq, int Hkv, int D, int dim, int Dv,
                           int block_size, long long num_slots, float eps, int dtype, int* status,
                           cudaStream_t stream) {
@@ -298,11 +343,10 @@ int ab200_head_rope_cache(void* proj, long long ld, const void* positions, const
   if (ld < (long long)(Hq + Hkv) * D + (long long)Hkv * Dv) return -2;
   HeadRopeArgs a;
   a.proj = proj; a.ld = ld;
-  a.positions = reinterpret_cast<const long long*>(positions);
+  a.table = reinterpret_cast<const float*>(table);
   a.slots = reinterpret_cast<const long long*>(slots);
   a.wq = reinterpret_cast<const float*>(wq);
   a.wk = reinterpret_cast<const float*>(wk);
-  a.freq = reinterpret_cast<const float*>(freq);
   a.k_cache = k_cache; a.v_cache = v_cache;
   a.num_slots = num_slots;
   a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.Dv = Dv;
@@ -315,25 +359,25 @@ int ab200_head_rope_cache(void* proj, long long ld, const void* positions, const
 
 // q [T, ld]: H heads of dq columns whose rotary part starts at column `dim`; ckv [T, ld]: R latent
 // columns and 2 * half rotary ones; cache rows of `width` columns, the rotary part at rot_at.
-int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* positions,
-                            const void* slots, const void* weight, const void* freq, int half,
-                            void* cache, long long T, int H, int dq, int dim, int R, int width,
+int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* table, int half,
+                            const void* slots, const void* weight, void* cache, long long T, int H, int dq, int dim, int R, int width,
                             int rot_at, long long num_slots, float eps, int dtype, int* status,
                             cudaStream_t stream) {
   if (T <= 0) return 0;
   if (half < 0 || dim + 2 * half > dq || R > rot_at || rot_at + 2 * half > width) return -2;
   LatentRopeArgs a;
   a.q = q; a.ckv = ckv; a.ld = ld;
-  a.positions = reinterpret_cast<const long long*>(positions);
+  a.table = reinterpret_cast<const float*>(table);
   a.slots = reinterpret_cast<const long long*>(slots);
   a.weight = reinterpret_cast<const float*>(weight);
-  a.freq = reinterpret_cast<const float*>(freq);
   a.cache = cache;
   a.num_slots = num_slots;
   a.H = H; a.dq = dq; a.dim = dim; a.R = R; a.half = half;
   a.width = width; a.rot_at = rot_at;
   a.eps = eps;
   a.status = status;
+  a.vec = half > 0 && half % 4 == 0 && dim % 4 == 0 && dq % 4 == 0 && ld % 4 == 0 &&
+          (reinterpret_cast<uintptr_t>(q) & 15) == 0;
   const size_t smem = (2 * (size_t)half + 4) * sizeof(float);
   if (smem > 48 * 1024) return -6;
   auto k = dtype == 0 ? latent_rope_cache_kernel<bf16> : latent_rope_cache_kernel<float>;

@@ -321,10 +321,10 @@ class LayerListForCausalLM:
     def forward(self, batch: ForwardBatch, kv, layers_out: list = None) -> torch.Tensor:
         """Final-norm states of the sampled rows [B, W]. ``layers_out`` receives a copy of the
         residual stream after every run."""
-        contexts: dict = {}
+        shared: dict = {}
         step, eps = batch.attn_meta, self.cfg.rms_norm_eps
         mix = lambda r, l, act: self.mixers[l].run(act, self.layers[l], batch, kv.of(r), step,
-                                                   contexts, eps)
+                                                   shared, eps)
         body = self._post_norm_body if self.design.residual == "post" else self._sandwich_body
         x = body(batch, mix, layers_out)
         return st.stream_final_norm(x, batch.logits_indices, self.norm, eps, self.dtype,

@@ -73,6 +73,14 @@ def frequencies(rotary, device) -> torch.Tensor:
     return torch.tensor(f, dtype=torch.float64).float().to(device)
 
 
+def angles(rotary, freq, batch, shared: dict) -> torch.Tensor:
+    """The step's rotary table for these frequencies, made by the first run that needs it."""
+    table = shared.get(rotary)
+    if table is None:
+        table = shared[rotary] = heads.rotary_table(batch.positions, freq)
+    return table
+
+
 class LatentMixer:
     def __init__(self, spec: LatentAttentionSpec, heads_sharing: int, dtype: torch.dtype, device):
         """``heads_sharing``: the most heads among the layers that read these latents."""
@@ -164,17 +172,17 @@ class LatentMixer:
         return lat.LatentDecodePlan(self.shape, bucket, max_q, block_size)
 
     # ---- the layer's mixer
-    def run(self, act, lw: LayerWeights, batch, cache, step, contexts: dict, eps: float):
-        """``cache``: this run's tensors; ``contexts``: gathered latents of the expanded sequences,
-        by cache tensor and mask, reused by the layers that share them."""
+    def run(self, act, lw: LayerWeights, batch, cache, step, shared: dict, eps: float):
+        """``cache``: this run's tensors; ``shared``: what several runs of a step use, i.e. rotary
+        tables and, by cache tensor and mask, gathered latents of the expanded sequences."""
         m, T = self.spec, act.shape[0]
         H, nq = m.heads, m.heads * self.dq
         proj = ops.linear(act, lw.wq)
         cache = cache[0]
         if m.rot_dim:
             lat.latent_rope_cache(proj, proj[:, nq:], H, self.dq, m.dim, lw.ckv_norm, m.kv_rank,
-                                  self.freq, eps, batch.positions, batch.slots, cache,
-                                  self.layout.rot_at)
+                                  angles(m.rotary, self.freq, batch, shared), eps, batch.slots,
+                                  cache, self.layout.rot_at)
         elif m.kv_from is None:
             lat.latent_norm_cache(proj[:, nq:], lw.ckv_norm, m.kv_rank, eps, batch.slots, cache)
         n = T if self.expand is None else step.n_absorbed
@@ -186,9 +194,9 @@ class LatentMixer:
             st.head_linear(o, lw.wuv, out=out[:n])
         if n < T:
             key = (cache.data_ptr(), m.mask)
-            c = contexts.get(key)
+            c = shared.get(key)
             if c is None:
-                c = contexts[key] = ops.gather_rows(cache.view(-1, self.layout.width),
+                c = shared[key] = ops.gather_rows(cache.view(-1, self.layout.width),
                                                     step.ctx[m.mask][0])
             kvs = ops.linear(c, lw.wukv)
             lat.expanded_attention(proj[n:, :nq], kvs[:, :nq], kvs[:, nq:], step, H, self.expand,
@@ -266,12 +274,13 @@ class HeadMixer:
         return heads.HeadDecodePlan(self.shape, bucket, max_q, block_size)
 
     # ---- the layer's mixer
-    def run(self, act, lw: LayerWeights, batch, cache, step, contexts: dict, eps: float):
+    def run(self, act, lw: LayerWeights, batch, cache, step, shared: dict, eps: float):
         m, s = self.spec, self.shape
         proj = ops.linear(act, lw.wqkv)
         k, v = cache
         norm = (lw.q_norm, lw.k_norm) if m.qk_norm else (None, None)
-        heads.head_rope_cache(proj, s, m.dim, *norm, self.freq, eps, batch.positions, batch.slots, k, v)
+        heads.head_rope_cache(proj, s, m.dim, *norm, angles(m.rotary, self.freq, batch, shared), eps,
+                              batch.slots, k, v)
         gate = proj[:, (s.heads + s.kv_heads) * s.D + s.kv_heads * s.Dv:] if m.output_gate else None
         out = heads.head_attention(proj[:, :s.heads * s.D], k, v, step.heads[s], s, self.scale,
                                    lw.sink if m.sink else None, gate, step.tok_seq, batch.positions)

@@ -70,20 +70,36 @@ class HeadDecodePlan(DecodePlan):
 
 
 # ------------------------------------------------------------------------------ kernels
-def rotate_ref(x, positions, freq):
-    """x [T, heads, d] fp32: rotary positions over the first 2 * len(freq) dimensions."""
-    half = freq.numel()
-    a = (positions.float().unsqueeze(1) * freq).unsqueeze(1)
+def rotary_table(positions: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
+    """fp32 [T, len(freq), 2]: cosine and sine of every token's angles, position * frequency in
+    fp32. Layers with the same frequencies share it."""
+    T, half = positions.numel(), freq.numel()
+    if not positions.is_cuda:
+        a = positions.float().unsqueeze(1) * freq
+        return torch.stack([a.cos(), a.sin()], -1)
+    nat = _nat()
+    table = torch.empty(T, half, 2, dtype=torch.float32, device=positions.device)
+    assert positions.dtype == torch.int64 and positions.is_contiguous()
+    rc = nat.lib().ab200_rotary_table(positions.data_ptr(), freq.data_ptr(), table.data_ptr(), T,
+                                      half, nat.stream_ptr())
+    nat.check(rc, "rotary_table")
+    launch_counter.add(1)
+    return table
+
+
+def rotate_ref(x, table):
+    """x [T, heads, d] fp32, table [T, half, 2]: the first 2 * half dimensions rotated."""
+    half = table.shape[1]
     u, v = x[..., :half], x[..., half:2 * half]
-    c, s = a.cos(), a.sin()
+    c, s = table[:, None, :, 0], table[:, None, :, 1]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1)
 
 
-def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, freq, eps: float, positions, slots,
-                    k_cache, v_cache) -> None:
+def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, table, eps: float, slots, k_cache,
+                    v_cache) -> None:
     """``proj`` [T, ...] holds the query heads, key heads (``D`` columns each, ``dim`` in use) and
     value heads (``Dv``). RMS norm of every query and key head over its ``dim`` columns with the
-    weights ``wq`` / ``wk`` (fp32 [D], or None), rotation of the first 2 * len(freq), queries in
+    weights ``wq`` / ``wk`` (fp32 [D], or None), rotation by ``table`` (rotary_table), queries in
     place, keys and values to the rows ``slots`` of the caches; slot < 0: no write."""
     H, G, D, Dv = shape.heads, shape.kv_heads, shape.D, shape.Dv
     T, bs = proj.shape[0], k_cache.shape[2]
@@ -92,7 +108,7 @@ def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, freq, eps: float, 
         if wq is not None:
             w = torch.cat([wq.expand(H, D), wk.expand(G, D)])
             x = x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) / dim + eps) * w
-        x = rotate_ref(x, positions, freq).to(proj.dtype)
+        x = rotate_ref(x, table).to(proj.dtype)
         proj[:, :H * D] = x[:, :H].reshape(T, H * D)
         ok = slots >= 0
         blk, off = slots[ok] // bs, slots[ok] % bs
@@ -101,11 +117,11 @@ def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, freq, eps: float, 
         return
     nat = _nat()
     assert proj.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
-    assert slots.dtype == positions.dtype == torch.int64
+    assert slots.dtype == torch.int64 and table.is_contiguous()
     rc = nat.lib().ab200_head_rope_cache(
-        proj.data_ptr(), proj.stride(0), positions.data_ptr(), slots.data_ptr(), nat.ptr(wq),
-        nat.ptr(wk), freq.data_ptr(), freq.numel(), k_cache.data_ptr(), v_cache.data_ptr(), T, H, G, D,
-        dim, Dv, bs, k_cache.shape[0] * bs, float(eps), dtype_code(proj.dtype),
+        proj.data_ptr(), proj.stride(0), table.data_ptr(), table.shape[1], slots.data_ptr(),
+        nat.ptr(wq), nat.ptr(wk), k_cache.data_ptr(), v_cache.data_ptr(), T, H, G, D, dim, Dv, bs,
+        k_cache.shape[0] * bs, float(eps), dtype_code(proj.dtype),
         nat.status_buffer(proj.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "head_rope_cache")
     launch_counter.add(1)

@@ -272,31 +272,31 @@ def latent_norm_cache(ckv: torch.Tensor, weight: torch.Tensor, rank: int, eps: f
     launch_counter.add(1)
 
 
-def latent_rope_cache(q, ckv, heads: int, dq: int, dim: int, weight, rank: int, freq, eps: float,
-                      positions, slots, cache, rot_at: int) -> None:
+def latent_rope_cache(q, ckv, heads: int, dq: int, dim: int, weight, rank: int, table, eps: float,
+                      slots, cache, rot_at: int) -> None:
     """:func:`latent_norm_cache` for latents with a rotated key part: ``ckv`` [T, >= rank + rot]
     holds it behind the latent, the cache row from column ``rot_at``. ``q`` [T, >= heads * dq] (of
     the same row stride) is rotated in place: ``rot`` columns of every head from ``dim`` on.
-    ``freq`` fp32 [rot / 2]."""
+    ``table``: head_ops.rotary_table."""
     nb, _, bs, W = cache.shape
-    half = freq.numel()
+    half = table.shape[1]
     if not ckv.is_cuda:
         from .head_ops import rotate_ref
         x = q[:, :heads * dq].unflatten(1, (heads, dq))      # (a view)
-        part = rotate_ref(x[:, :, dim:dim + 2 * half].float(), positions, freq)
+        part = rotate_ref(x[:, :, dim:dim + 2 * half].float(), table)
         x[:, :, dim:dim + 2 * half] = part.to(q.dtype)
         latent_norm_cache(ckv, weight, rank, eps, slots, cache)
-        shared = rotate_ref(ckv[:, None, rank:rank + 2 * half].float(), positions, freq)[:, 0]
+        shared = rotate_ref(ckv[:, None, rank:rank + 2 * half].float(), table)[:, 0]
         ok = slots >= 0
         cache.view(nb * bs, W)[slots[ok], rot_at:rot_at + 2 * half] = shared[ok].to(cache.dtype)
         return
     nat = _nat()
     assert q.stride(0) == ckv.stride(0) and q.stride(1) == ckv.stride(1) == 1
-    assert cache.is_contiguous() and slots.dtype == positions.dtype == torch.int64
+    assert cache.is_contiguous() and slots.dtype == torch.int64 and table.is_contiguous()
     rc = nat.lib().ab200_latent_rope_cache(
-        q.data_ptr(), ckv.data_ptr(), q.stride(0), positions.data_ptr(), slots.data_ptr(),
-        weight.data_ptr(), freq.data_ptr(), half, cache.data_ptr(), q.shape[0], heads, dq, dim, rank,
-        W, rot_at, nb * bs, float(eps), dtype_code(q.dtype), nat.status_buffer(q.device).data_ptr(),
+        q.data_ptr(), ckv.data_ptr(), q.stride(0), table.data_ptr(), half, slots.data_ptr(),
+        weight.data_ptr(), cache.data_ptr(), q.shape[0], heads, dq, dim, rank, W, rot_at, nb * bs,
+        float(eps), dtype_code(q.dtype), nat.status_buffer(q.device).data_ptr(),
         nat.stream_ptr())
     nat.check(rc, "latent_rope_cache")
     launch_counter.add(1)

@@ -131,10 +131,11 @@ def _declare(L: ctypes.CDLL) -> None:
         "ab200_linear_exact": (I, [P, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P]),
         "ab200_attention_exact": (I, [P, LL, P, I, P, I, I, I, P, I, P, P, P, P, LL, P, LL, LL, I,
                                       I, I, I, I, I, F, I, P, P]),
-        "ab200_head_rope_cache": (I, [P, LL, P, P, P, P, P, I, P, P, LL, I, I, I, I, I, I, LL, F, I,
-                                      P, P]),
-        "ab200_latent_rope_cache": (I, [P, P, LL, P, P, P, P, I, P, LL, I, I, I, I, I, I, LL, F, I,
-                                        P, P]),
+        "ab200_rotary_table": (I, [P, P, P, LL, I, P]),
+        "ab200_head_rope_cache": (I, [P, LL, P, I, P, P, P, P, P, LL, I, I, I, I, I, I, LL, F, I, P,
+                                      P]),
+        "ab200_latent_rope_cache": (I, [P, P, LL, P, I, P, P, P, LL, I, I, I, I, I, I, LL, F, I, P,
+                                        P]),
         "ab200_moe_route": (I, [P, P, P, LL, I, I, I, P, P, P, P, P, P, I, P]),
         "ab200_moe_permute": (I, [P, P, P, P, P, LL, I, I, I, P]),
         "ab200_grouped_gemm": (I, [P, LL, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, F,

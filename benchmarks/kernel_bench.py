@@ -94,6 +94,21 @@ CASES = {
     "route_decode": ("route", (128, 2048, 64, 6)),
     "stream_norm": ("stream_norm", (8192, 4096)),
     "latent_norm_cache": ("latent_norm", (8192, 512)),
+    # attention with sink, output gate and a mask (kind, positions): query and cached lengths
+    "masked_prefill_4x2048": ("masked", ([2048] * 4, [2048] * 4, "chunk", 4096)),
+    "masked_prefill_chunks_1024": ("masked", ([2048] * 4, [2048] * 4, "chunk", 1024)),
+    "masked_decode_128": ("masked", ([1] * 128, [2000] * 128, "chunk", 4096)),
+    "masked_decode_window_128": ("masked", ([1] * 128, [2000] * 128, "window", 128)),
+    # expanded latents with a rotated part: keys of 192, values of 128
+    "expanded_192_4x2048": ("expanded", (32, [2048] * 4, 4096)),
+    # decode in latent space with 64 key-only columns under a window
+    "latent_rot_512": ("latent_rot", (32, 512, 128, 2000, 4096)),
+    "latent_rot_512_window_128": ("latent_rot", (32, 512, 128, 2000, 128)),
+    # query / key norms, rotation, cache write: tokens, heads, K/V heads, dimensions, rotated
+    "head_rope": ("head_rope", (8192, 32, 8, 128, 32)),
+    "head_rope_64": ("head_rope", (8192, 40, 8, 64, 16)),
+    "latent_rope": ("latent_rope", (8192, 32, 128, 64, 512)),
+    "stream_sandwich": ("sandwich", (8192, 4096)),
     # name: (kind, params)
     "gemm_prefill": ("gemm", (8192, 28672, 4096)),
     "gemm_prefill_qkv": ("gemm", (8192, 6144, 4096)),
@@ -129,6 +144,7 @@ CASES = {
     "attn_prefill_4x2048": ("attn", ([2048] * 4, [2048] * 4)),
     "attn_decode": ("attn", ([1] * 32, [2000] * 32)),
     "attn_decode_128": ("attn", ([1] * 128, [2000] * 128)),
+    "attn_decode_128_short": ("attn", ([1] * 128, [144] * 128)),
     "attn_decode_long": ("attn", ([1] * 8, [8000] * 8)),
     "attn_verify": ("attn", ([4] * 32, [2000] * 32)),
     "rmsnorm": ("rmsnorm", (8192, 4096)),
@@ -215,6 +231,81 @@ def run_case(a, case):
         sets = [(R(n, H * rank), R(nb, 1, 64, rank)) for _ in range(nc)]
         fn = lambda i=0: lat.latent_attention(sets[i][0], sets[i][1], meta, shape, 0.1)
         flops = 4.0 * n * kl * H * rank
+    elif kind == "masked":
+        from arcticinference_b200.config import MaskSpec
+        from arcticinference_b200.ops import head_ops as hd
+        ql, kl, name, size = prm
+        shape = hd.HeadShape.of(32, 8, 128, 128, torch.bfloat16, MaskSpec(name, size))
+        pairs = sum(p - shape.mask.first_key(p) + 1 for n, k in zip(ql, kl) for p in range(k - n, k))
+        keys = sum(k - shape.mask.first_key(k - n) for n, k in zip(ql, kl))
+        flops, byts = 4.0 * pairs * 32 * 128, 4.0 * keys * 8 * 128 + 6.0 * sum(ql) * 32 * 128
+        nc = copies_for(byts)
+        sink, sets = torch.zeros(32, device=DEV), []
+        for _ in range(nc):
+            q, kc, vc, meta = paged(ql, kl)
+            sets.append((q, kc, vc, hd.build_plan(shape, ql, kl, meta.block_tables, 64, DEV), R(*q.shape)))
+        fn = lambda i=0: hd.head_attention(*sets[i][:4], shape, 0.09, sink, sets[i][4])
+    elif kind == "expanded":
+        from arcticinference_b200.config import MaskSpec
+        H, ql, size = prm
+        mask, T = MaskSpec("window", size), sum(ql)
+        starts = [sum(ql[:i]) for i in range(len(ql))]
+        meta = ops.build_attention_metadata(ql, ql, None, 1, H, 128, DEV, Hkv=H, seq_rows=starts,
+                                            allow_split=False, mask=mask)
+        q, kv = R(T, H * 192), R(T, H * 320)
+        fn = lambda i=0: ops.attention_masked(q, kv[:, :H * 192], kv[:, H * 192:], meta, H, H, 128,
+                                              0.07, mask, paged=False, Dk=192)
+        nc = 1
+        pairs = sum(p - mask.first_key(p) + 1 for n in ql for p in range(n))
+        flops, byts = 2.0 * pairs * H * 320, 2.0 * T * H * (192 + 320 + 128)
+    elif kind == "latent_rot":
+        from arcticinference_b200.config import MaskSpec
+        from arcticinference_b200.ops import latent_ops as lat
+        H, rank, n, kl, size = prm
+        seen = min(kl, size)
+        byts = 2.0 * n * seen * (rank + 64) + 2.0 * n * H * (2 * rank + 64)
+        nc = copies_for(byts)
+        nb = n * (-(-kl // 64)) + 1
+        bt = torch.arange(1, nb, dtype=torch.int32, device=DEV).view(n, -1)
+        shape = lat.LatentShape.of(H, rank, torch.bfloat16, 64, MaskSpec("window", size))
+        meta = lat.build_plan(shape, [1] * n, [kl] * n, bt, 64, DEV)
+        sets = [(R(n, H * (rank + 64)), R(nb, 1, 64, rank + 64)) for _ in range(nc)]
+        fn = lambda i=0: lat.latent_attention(sets[i][0], sets[i][1], meta, shape, 0.1)
+        flops = 2.0 * n * seen * H * (2 * rank + 64)
+    elif kind == "head_rope":
+        from arcticinference_b200.ops import head_ops as hd
+        T, H, G, D, dims = prm
+        shape = hd.HeadShape.of(H, G, D, D, torch.bfloat16)
+        byts = 2.0 * T * D * (2 * (H + G) + 2 * G)
+        nc = copies_for(byts)
+        sets = [(R(T, (H + 2 * G) * D), *(R(T // 64, G, 64, D) for _ in range(2))) for _ in range(nc)]
+        w, freq = torch.ones(D, device=DEV), torch.rand(dims // 2, device=DEV)
+        at = torch.arange(T, device=DEV)
+        table = hd.rotary_table(at, freq)
+        fn = lambda i=0: hd.head_rope_cache(sets[i][0], shape, D, w, w, table, 1e-6, at, *sets[i][1:])
+        flops = 0.0
+    elif kind == "latent_rope":
+        from arcticinference_b200.ops import head_ops as hd
+        from arcticinference_b200.ops import latent_ops as lat
+        T, H, dim, rot, rank = prm
+        nq = H * (dim + rot)
+        byts = 4.0 * T * (H * rot + rank + rot)
+        nc = copies_for(byts)
+        sets = [(R(T, nq + rank + rot), R(T // 64, 1, 64, rank + rot)) for _ in range(nc)]
+        w, freq = torch.ones(rank, device=DEV), torch.rand(rot // 2, device=DEV)
+        at = torch.arange(T, device=DEV)
+        table = hd.rotary_table(at, freq)
+        fn = lambda i=0: lat.latent_rope_cache(sets[i][0], sets[i][0][:, nq:], H, dim + rot, dim, w,
+                                               rank, table, 1e-6, at, sets[i][1], rank)
+        flops = 0.0
+    elif kind == "sandwich":
+        from arcticinference_b200.ops import stream_ops as st
+        T, W = prm
+        nc = copies_for(8 * T * W)
+        sets = [(torch.randn(T, W, device=DEV), R(T, W), R(T, W)) for _ in range(nc)]
+        w = torch.ones(W, device=DEV)
+        fn = lambda i=0: st.stream_sandwich(sets[i][0], sets[i][1], w, None, w, sets[i][2], eps=1e-6)
+        flops, byts = 0.0, 12.0 * T * W
     elif kind == "experts":
         from arcticinference_b200.ops import stream_ops as st
         T, W, ff, E, top = prm

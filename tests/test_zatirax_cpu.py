@@ -105,7 +105,7 @@ def test_rotation(rot):
     assert np.allclose(spec.frequencies(), oracle.frequencies(rot), rtol=1e-12)
     pos = torch.tensor([0, 1, 77, 4000])
     x = torch.randn(4, 3, rot["dims"] + 5)
-    got = hd.rotate_ref(x, pos, torch.tensor(spec.frequencies()).float())
+    got = hd.rotate_ref(x, hd.rotary_table(pos, torch.tensor(spec.frequencies()).float()))
     for h in range(3):
         assert float((got[:, h] - oracle.rotate(x[:, h].double(), pos, rot)).abs().max()) < 2e-3
         assert torch.equal(got[:, h, rot["dims"]:], x[:, h, rot["dims"]:])

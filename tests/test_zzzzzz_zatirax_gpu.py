@@ -102,7 +102,7 @@ def test_head_rope_cache(H, G, dim, vdim, dims, normed, dtype):
     pos = torch.tensor([0, 1, 300, 7, 4000, 63], device=DEV)
     freq = torch.tensor(oracle.frequencies(rot)).float().to(DEV)
     hd.head_rope_cache(proj, shape, dim, pad(wq) if normed else None, pad(wk) if normed else None,
-                       freq, 0.02, pos, slots, k, vc)
+                       hd.rotary_table(pos, freq), 0.02, slots, k, vc)
     ops.check_status()
     for j in range(H + G):
         want = x[:, j].double().cpu()
@@ -138,8 +138,8 @@ def test_latent_rope_cache(H, dim, rot, rank, extra, dtype):
     slots = torch.tensor([31, 0, -1, 16, 9], device=DEV)
     pos = torch.tensor([0, 5000, 3, 64, 129], device=DEV)
     freq = torch.tensor(oracle.frequencies(r)).float().to(DEV)
-    lat.latent_rope_cache(buf, buf[:, H * dq:], H, dq, dim, weight, rank, freq, 0.02, pos, slots,
-                          cache, at)
+    lat.latent_rope_cache(buf, buf[:, H * dq:], H, dq, dim, weight, rank,
+                          hd.rotary_table(pos, freq), 0.02, slots, cache, at)
     ops.check_status()
     scale = 1.0 if dtype == BF16 else 10.0
     for h in range(H):
