@@ -20,7 +20,7 @@ from . import reference as ref
 __all__ = [
     "linear", "linear_fp8", "linear_fp8_row", "quant_fp8", "quant_fp8_row", "gemm_nn", "embedding", "rmsnorm", "layernorm", "silu_mul", "silu_mul_blocked", "rope_cache",
     "gather_rows", "argmax_sample", "AttentionMetadata", "build_attention_metadata", "pick_tile_keys", "plan_attention_work",
-    "attention", "attention_contiguous", "check_status", "count_launches", "launch_counter",
+    "attention", "attention_masked", "attention_contiguous", "check_status", "count_launches", "launch_counter",
 ]
 
 
