@@ -59,8 +59,8 @@ class MaskSpec:
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary positions over the first ``dims`` dimensions of a vector, dimension i paired with
-    i + dims / 2. ``scaling``: (factor, low, high, original), a context extension that divides the
+    """Rotary positions over the leading ``dims`` dimensions of a vector, whose two halves form the
+    pairs (i, i + dims / 2). ``scaling``: (factor, low, high, original), a context extension that divides the
     frequencies whose wavelength exceeds original / low, keeps those below original / high and
     interpolates between the two."""
     base: float
@@ -135,8 +135,9 @@ class LayerSpec:
 
 @dataclass(frozen=True)
 class LoopSpec:
-    """Layers start .. stop - 1 run ``times`` times in a row with the same weights, each pass with
-    a cache of its own and a learned vector added to the stream before it."""
+    """The slice ``[start, stop)`` of the layer list is executed ``times`` times before the layers
+    behind it. Passes share weights, not caches; a learned vector per pass is added to the stream as
+    the pass begins."""
     start: int
     stop: int
     times: int

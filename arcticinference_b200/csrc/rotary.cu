@@ -9,8 +9,8 @@
 //                      the heads share, both to the paged latent cache; rotation of every query
 //                      head's rotary part in place
 //
-// A block owns a token and its warps walk the heads; norms and rotations are fp32. Dimension i is
-// paired with i + rot / 2. Heads of 64 or 128 bf16 columns stay in registers, four columns a lane
+// A block owns a token and its warps walk the heads; norms and rotations are fp32. Pairs are
+// (i, i + rot / 2). Heads of 64 or 128 bf16 columns stay in registers, four columns a lane
 // and several heads in flight; a pair's other half then comes from another lane.
 // T is the model's element type (bf16 or fp32).
 

@@ -46,8 +46,8 @@ def frequencies(rot):
 
 
 def rotate(x, positions, rot):
-    """x [n, d]: the first rot.dims dimensions turned by their positions' angles, dimension i
-    with dimension i + dims / 2."""
+    """x [n, d]: the pairs (i, i + dims / 2) turned by their positions' angles, the dimensions
+    from rot.dims on left alone."""
     n, half = rot["dims"], rot["dims"] // 2
     a = positions.double().unsqueeze(1) * torch.tensor(frequencies(rot), dtype=torch.float64)
     u, v = x[:, :half], x[:, half:n]
