@@ -80,6 +80,8 @@ KERNEL_SETS = {
                 "latent_attention", "moe", "rotary", "sampling", "stream"),
     "Zatirax": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm",
                 "latent_attention", "rotary", "sampling", "stream"),
+    "Pererax": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm", "moe", "recurrent",
+                "rotary", "sampling", "stream"),
 }
 _kernel_set: str | None = None
 

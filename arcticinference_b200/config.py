@@ -111,9 +111,55 @@ class AttentionSpec:
     scale: float
     rotary: Optional[RotarySpec] = None
     mask: MaskSpec = MaskSpec()
-    qk_norm: bool = False       # RMS norm over dim of every query and key head, before rotation
-    sink: bool = False          # exp of a learned number per head in the softmax denominator
+    # RMS norm before rotation: "head" (over dim of every query and key head), "projection" (over
+    # all query, and all key, heads of a token at once) or None
+    qk_norm: Optional[str] = None
+    # a further term of the softmax denominator: exp of a "learned" number per head, exp(0)
+    # ("zero"), or None
+    sink: Optional[str] = None
     output_gate: bool = False   # heads' outputs times sigmoid of a projection of the layer's input
+    softcap: float = 0.0        # scores become softcap * tanh(score / softcap); 0: they do not
+    values_are_keys: bool = False   # the key projection (before norm and rotation) is the value
+
+
+@dataclass(frozen=True)
+class DeltaRuleSpec:
+    """Gated delta rule with a decay per key channel: a [dim, vdim] state per head. ``kv_heads``
+    query / key heads serve ``heads`` value heads; queries, keys and values pass a causal
+    convolution of ``conv`` taps. The ranks of the decay and gate projections come from the
+    tensors."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory with exponential gates (the mLSTM of xLSTM): a [dim, vdim] state, a [dim]
+    normaliser and a running maximum per head. ``gate_cap``: soft cap of both gates."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same input; the result is half the sum of their normed outputs."""
+    left: AttentionSpec
+    right: MatrixMemorySpec
+
+
+def mixer_parts(m) -> tuple:
+    """The elementary mixers of a layer's mixer."""
+    return (m.left, m.right) if isinstance(m, ParallelSpec) else (m,)
+
+
+def has_state(m) -> bool:
+    """Whether a mixer carries a state from token to token, which cannot be taken back."""
+    return any(isinstance(x, (DeltaRuleSpec, MatrixMemorySpec)) for x in mixer_parts(m))
 
 
 @dataclass(frozen=True)
@@ -124,13 +170,20 @@ class FeedForwardSpec:
     experts: int = 0      # 0: dense
     top: int = 0
     limit: float = 0.0    # clamped_swish: bound of gate (above) and up (both sides)
+    # router: "chosen" (largest logits plus bias, softmax over the chosen ones) or "all" (softmax
+    # over all; a correction enters the choice, not the weights; weights times ``router_scale``)
+    scoring: str = "chosen"
+    router_scale: float = 1.0
+    identity: int = 0     # further router outputs behind the experts' whose expert is the identity
+    shared: Optional["FeedForwardSpec"] = None   # runs for every token beside the chosen ones
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """One decoder layer of a model that lists its layers one by one."""
-    mixer: Any            # LatentAttentionSpec | AttentionSpec
+    mixer: Any            # AttentionSpec | LatentAttentionSpec | DeltaRuleSpec | ParallelSpec
     mlp: Optional[FeedForwardSpec] = None
+    weights_of: Optional[int] = None    # layer whose tensors this one uses (cache and state are its own)
 
 
 @dataclass(frozen=True)
@@ -148,17 +201,20 @@ class LayerListDesign:
     """What the name of a layer-list architecture stands for, beyond the numbers of config.json.
 
     ``residual``: where the norms are. "post": x <- norm(alpha * x + f(x)); "sandwich":
-    x <- x + norm_b(f(norm_a(x))). ``norm_offset``: added to the stored weights of the stream's
-    norms. ``masks``: kind of each mixer type's mask."""
+    x <- x + norm_b(f(norm_a(x))); "output": x <- x + norm(f(x)) * scale. ``norm_offset``: added to
+    the stored weights of the stream's norms. ``masks``: kind of each mixer type's mask.
+    ``attention``: options of :class:`AttentionSpec` by mixer type ("left": the attention side of
+    a parallel mixer). ``scoring``: the router's. ``tied``: the embedding is the output matrix."""
     residual: str
     norm_offset: float
     dense_act: str
     mixers: tuple
     feed_forwards: tuple
     masks: dict = field(default_factory=dict)
-    qk_norm: bool = False
-    sink: bool = False
-    output_gate: bool = False
+    attention: dict = field(default_factory=dict)
+    expert_act: str = "silu"
+    scoring: str = "chosen"
+    tied: bool = False
 
 
 LAYER_LIST_DESIGNS = {
@@ -167,7 +223,15 @@ LAYER_LIST_DESIGNS = {
     "Zatirax": LayerListDesign(residual="sandwich", norm_offset=0.0, dense_act="clamped_swish",
                                mixers=("latent_attention", "attention"), feed_forwards=("dense",),
                                masks={"latent_attention": "window", "attention": "chunk"},
-                               qk_norm=True, sink=True, output_gate=True),
+                               attention={"attention": dict(qk_norm="head", sink="learned",
+                                                            output_gate=True)}),
+    "Pererax": LayerListDesign(residual="output", norm_offset=0.0, dense_act="clamped_swish",
+                               mixers=("channel_delta", "parallel", "attention"),
+                               feed_forwards=("moe",), masks={"attention": "window"},
+                               attention={"attention": dict(qk_norm="projection",
+                                                            values_are_keys=True),
+                                          "left": dict(qk_norm="projection", sink="zero")},
+                               expert_act="clamped_swish", scoring="all", tied=True),
 }
 
 
@@ -181,17 +245,37 @@ def _read_rotary(d: Optional[dict]) -> Optional[RotarySpec]:
 
 
 def _read_mixer(kind: str, m: dict, design: LayerListDesign):
+    if kind == "parallel":
+        r = m["right"]
+        return ParallelSpec(_read_mixer("left", m["left"], design),
+                            MatrixMemorySpec(heads=int(r["heads"]), dim=int(r["dim"]),
+                                             vdim=int(r["vdim"]), gate_cap=float(r["gate_cap"])))
+    if kind == "channel_delta":
+        return DeltaRuleSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                             vdim=int(m["vdim"]), conv=int(m["conv"]))
     rotary, mask = _read_rotary(m.get("rot")), MaskSpec()
     if m.get("mask") is not None:
         mask = MaskSpec(design.masks[kind], int(m["mask"]["size"]))
-    shape = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                 scale=float(m["scale"]), rotary=rotary, mask=mask)
-    if kind == "attention":
-        return AttentionSpec(kv_heads=int(m["kv_heads"]), qk_norm=design.qk_norm,
-                             sink=design.sink, output_gate=design.output_gate, **shape)
+    options = design.attention.get(kind, {})
+    vdim = m["dim"] if options.get("values_are_keys") else m["vdim"]
+    shape = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(vdim), scale=float(m["scale"]),
+                 rotary=rotary, mask=mask)
+    if kind in ("attention", "left"):
+        return AttentionSpec(kv_heads=int(m["kv_heads"]), softcap=float(m.get("softcap") or 0.0),
+                             **options, **shape)
     src = m.get("kv_from")
     return LatentAttentionSpec(kv_rank=int(m["kv_rank"]), rot_dim=int(m.get("rot_dim") or 0),
                                kv_from=None if src is None else int(src), **shape)
+
+
+def _read_experts(f: dict, design: LayerListDesign) -> FeedForwardSpec:
+    gated = lambda d: dict(ff=int(d["ff"]), act=design.expert_act, limit=float(d.get("limit", 0.0)))
+    r, shared = f["router"], f.get("shared")
+    return FeedForwardSpec(experts=int(r["experts"]), top=int(r["top"]), scoring=design.scoring,
+                           router_scale=float(r.get("scale", 1.0)),
+                           identity=int(r.get("identity") or 0),
+                           shared=FeedForwardSpec(**gated(shared)) if shared else None,
+                           **gated(f["expert"]))
 
 
 def read_layer_specs(layers: list, design: LayerListDesign) -> tuple:
@@ -213,46 +297,75 @@ def read_layer_specs(layers: list, design: LayerListDesign) -> tuple:
                 mlp = FeedForwardSpec(ff=int(f["ff"]), act=design.dense_act,
                                       limit=float(f["limit"]) if "limit" in f else 0.0)
             else:
-                mlp = FeedForwardSpec(ff=int(f["expert"]["ff"]), act="silu",
-                                      experts=int(f["router"]["experts"]),
-                                      top=int(f["router"]["top"]))
-        out.append(LayerSpec(mixer, mlp))
+                mlp = _read_experts(f, design)
+        src = d.get("weights_of")
+        out.append(LayerSpec(mixer, mlp, None if src is None else int(src)))
     return tuple(out)
+
+
+def _validate_mixer(i: int, m, specs: tuple) -> None:
+    if min(m.heads, m.dim, m.vdim) < 1:
+        raise ValueError("layer %d: heads, dim and vdim must be positive" % i)
+    if isinstance(m, MatrixMemorySpec):
+        if not m.gate_cap > 0:
+            raise ValueError("layer %d: gate_cap must be positive" % i)
+        return
+    if isinstance(m, (AttentionSpec, DeltaRuleSpec)) and (m.kv_heads < 1 or m.heads % m.kv_heads):
+        raise ValueError("layer %d: heads must be a multiple of kv_heads" % i)
+    if isinstance(m, DeltaRuleSpec):
+        if m.conv < 1:
+            raise ValueError("layer %d: a convolution of %d taps" % (i, m.conv))
+        return
+    if m.mask.kind != "causal" and m.mask.size < 1:
+        raise ValueError("layer %d: a %s of %d positions" % (i, m.mask.kind, m.mask.size))
+    if m.rotary is not None and (m.rotary.dims % 2 or m.rotary.dims < 0):
+        raise ValueError("layer %d: rot.dims must be even" % i)
+    if isinstance(m, AttentionSpec):
+        if m.rotary is not None and m.rotary.dims > m.dim:
+            raise ValueError("layer %d: rot.dims exceeds dim" % i)
+        if m.softcap < 0:
+            raise ValueError("layer %d: softcap must not be negative" % i)
+        return
+    if m.kv_rank < 1:
+        raise ValueError("layer %d: kv_rank must be positive" % i)
+    if m.rot_dim and (m.rotary is None or m.rotary.dims != m.rot_dim):
+        raise ValueError("layer %d: rot.dims must equal rot_dim" % i)
+    if m.kv_from is not None and m.rot_dim:
+        raise NotImplementedError("layer %d: shared latents with a rotated key part" % i)
+    if m.kv_from is not None:
+        if not 0 <= m.kv_from < i:
+            raise ValueError("layer %d: kv_from must name an earlier layer" % i)
+        src = specs[m.kv_from].mixer
+        if getattr(src, "kv_rank", None) != m.kv_rank or src.kv_from is not None or src.rot_dim:
+            raise ValueError("layer %d: layer %d has no latents of this kv_rank of its own"
+                             % (i, m.kv_from))
+
+
+def _validate_feed_forward(i: int, f: FeedForwardSpec) -> None:
+    if f.experts and not 1 <= f.top <= f.experts + f.identity:
+        raise ValueError("layer %d: top must lie between 1 and the number of experts" % i)
+    if f.identity < 0:
+        raise ValueError("layer %d: router.identity must not be negative" % i)
+    if f.act == "clamped_swish" and not f.limit > 0:
+        raise ValueError("layer %d: the feed-forward's limit must be positive" % i)
+    if f.shared is not None:
+        _validate_feed_forward(i, f.shared)
 
 
 def validate_layer_specs(specs: tuple, loop: Optional[LoopSpec] = None) -> None:
     for i, l in enumerate(specs):
-        m, f = l.mixer, l.mlp
-        if min(m.heads, m.dim, m.vdim) < 1:
-            raise ValueError("layer %d: heads, dim and vdim must be positive" % i)
-        if m.mask.kind != "causal" and m.mask.size < 1:
-            raise ValueError("layer %d: a %s of %d positions" % (i, m.mask.kind, m.mask.size))
-        if m.rotary is not None and (m.rotary.dims % 2 or m.rotary.dims < 0):
-            raise ValueError("layer %d: rot.dims must be even" % i)
-        if isinstance(m, AttentionSpec):
-            if m.kv_heads < 1 or m.heads % m.kv_heads:
-                raise ValueError("layer %d: heads must be a multiple of kv_heads" % i)
-            if m.rotary is not None and m.rotary.dims > m.dim:
-                raise ValueError("layer %d: rot.dims exceeds dim" % i)
-        else:
-            if m.kv_rank < 1:
-                raise ValueError("layer %d: kv_rank must be positive" % i)
-            if m.rot_dim and (m.rotary is None or m.rotary.dims != m.rot_dim):
-                raise ValueError("layer %d: rot.dims must equal rot_dim" % i)
-            if m.kv_from is not None and m.rot_dim:
-                raise NotImplementedError("layer %d: shared latents with a rotated key part" % i)
-            if m.kv_from is not None:
-                if not 0 <= m.kv_from < i:
-                    raise ValueError("layer %d: kv_from must name an earlier layer" % i)
-                src = specs[m.kv_from].mixer
-                if getattr(src, "kv_rank", None) != m.kv_rank or src.kv_from is not None or \
-                        src.rot_dim:
-                    raise ValueError("layer %d: layer %d has no latents of this kv_rank of its own"
-                                     % (i, m.kv_from))
-        if f is not None and f.experts and not 1 <= f.top <= f.experts:
-            raise ValueError("layer %d: top must lie between 1 and the number of experts" % i)
-        if f is not None and f.act == "clamped_swish" and not f.limit > 0:
-            raise ValueError("layer %d: the feed-forward's limit must be positive" % i)
+        for m in mixer_parts(l.mixer):
+            _validate_mixer(i, m, specs)
+        if l.mlp is not None:
+            _validate_feed_forward(i, l.mlp)
+        if l.weights_of is not None:
+            j = l.weights_of
+            if not 0 <= j < len(specs) or j == i:
+                raise ValueError("layer %d: weights_of must name another layer" % i)
+            if specs[j].weights_of is not None and loops_back(specs, i):
+                raise ValueError("layer %d: weights_of leads back to itself" % i)
+            if specs[j].mixer != l.mixer or specs[j].mlp != l.mlp:
+                raise ValueError("layer %d: layer %d, whose weights it uses, differs" % (i, j))
     if loop is not None:
         if not (0 <= loop.start < loop.stop <= len(specs) and loop.times >= 1):
             raise ValueError("loop: 0 <= start < stop <= layers and times >= 1 are needed")
@@ -262,10 +375,26 @@ def validate_layer_specs(specs: tuple, loop: Optional[LoopSpec] = None) -> None:
                 raise NotImplementedError("layer %d: shared latents inside a loop" % i)
 
 
+def loops_back(specs: tuple, i: int) -> bool:
+    seen = set()
+    while i is not None and i not in seen:
+        seen.add(i)
+        i = specs[i].weights_of
+    return i is not None
+
+
+def weights_index(specs: tuple, i: int) -> int:
+    """The layer whose tensors layer i uses."""
+    while specs[i].weights_of is not None:
+        i = specs[i].weights_of
+    return i
+
+
 @dataclass
 class ModelConfig:
     """Architecture of a decoder (Llama, Mistral, Qwen2 and Qwen3 dense models, optionally
-    SwiftKV for Llama; Taralix and Zatirax, which list their layers one by one) or encoder (BERT)."""
+    SwiftKV for Llama; Taralix, Zatirax and Pererax, which list their layers one by one) or
+    encoder (BERT)."""
 
     architecture: str = "LlamaForCausalLM"
     model_type: str = "llama"
@@ -354,6 +483,11 @@ class ModelConfig:
         """Whether the model can be served with 32-bit weights, activations and cache."""
         return self.layer_specs is not None
 
+    @property
+    def has_state(self) -> bool:
+        """Whether layers carry a state from token to token beside, or instead of, a cache."""
+        return self.layer_specs is not None and any(has_state(l.mixer) for l in self.layer_specs)
+
     def validate(self) -> None:
         if self.layer_specs is not None:
             validate_layer_specs(self.layer_specs, self.loop)
@@ -435,21 +569,25 @@ class ModelConfig:
         specs = read_layer_specs(d["layers"], design)
         if not specs:
             raise ValueError("a model without layers")
-        kept = lambda m: m.kv_heads * (m.dim + m.vdim) if isinstance(m, AttentionSpec) else \
-            m.kv_rank + m.rot_dim
+        parts = [m for l in specs for m in mixer_parts(l.mixer)]
+
+        def kept(m):
+            if isinstance(m, AttentionSpec):
+                return m.kv_heads * (m.dim + m.vdim)
+            return m.kv_rank + m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim
         eos, loop = d.get("eos_token_id"), d.get("loop")
         return cls(
             architecture=d["architecture"], model_type=d["architecture"].lower(),
             hidden_size=int(d["width"]), num_hidden_layers=len(specs),
-            num_attention_heads=max(l.mixer.heads for l in specs), num_key_value_heads=1,
-            head_dim=max(kept(l.mixer) for l in specs),
+            num_attention_heads=max(m.heads for m in parts), num_key_value_heads=1,
+            head_dim=max(kept(m) for m in parts),
             intermediate_size=max((l.mlp.ff for l in specs if l.mlp is not None), default=0),
             vocab_size=int(d["vocab"]), rms_norm_eps=float(d["norm"]["eps"]),
             postln_alpha=float(d["postln_alpha"]) if design.residual == "post" else 1.0,
             embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
             loop=None if not loop else LoopSpec(int(loop["start"]), int(loop["stop"]),
                                                 int(loop["times"])),
-            layer_specs=specs,
+            layer_specs=specs, tie_word_embeddings=design.tied,
             # no table is indexed by position, so nothing bounds it
             max_position_embeddings=1 << 20, hidden_act="",
             eos_token_id=int(eos) if isinstance(eos, int) else None, name_or_path=name_or_path)
@@ -460,13 +598,13 @@ class ModelConfig:
 
     @property
     def layer_runs(self) -> list:
-        """(layer, pass of the loop or None) in the order of execution of a layer-list model; the
-        pass is named at its first layer only."""
-        order = list(range(len(self.layer_specs)))
+        """(layer whose weights run, pass of the loop or None) in the order of execution of a
+        layer-list model; the pass is named at its first layer only."""
+        order = [weights_index(self.layer_specs, i) for i in range(len(self.layer_specs))]
         if self.loop is None:
             return [(l, None) for l in order]
         lo, hi, n = self.loop.start, self.loop.stop, self.loop.times
-        body = [(l, t if l == lo else None) for t in range(n) for l in order[lo:hi]]
+        body = [(l, t if k == 0 else None) for t in range(n) for k, l in enumerate(order[lo:hi])]
         return [(l, None) for l in order[:lo]] + body + [(l, None) for l in order[hi:]]
 
     @classmethod
@@ -528,6 +666,24 @@ def _zatirax(width, vocab, layers, loop, scale=1.0, eps=1e-6) -> ModelConfig:
         "architecture": "Zatirax", "width": width, "vocab": vocab, "norm": {"eps": eps},
         "embedding": {"scale": scale}, "layers": out,
         "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop))})
+
+
+def _pererax(width, vocab, layers, eps=1e-6) -> ModelConfig:
+    """``layers``: (mixer, feed-forward) each, or the number of the layer whose weights are used.
+    The feed-forward is None or (ff, experts, identity experts, top, ff of the shared expert)."""
+    out = []
+    for l in layers:
+        if isinstance(l, int):
+            out.append({**out[l], "weights_of": l})
+            continue
+        m, f = l
+        kind = "parallel" if "left" in m else "channel_delta" if "conv" in m else "attention"
+        out.append({"type": kind, "mixer": m, "mlp": None if f is None else {
+            "kind": "moe", "expert": {"ff": f[0], "limit": 7.0},
+            "router": {"experts": f[1], "identity": f[2], "top": f[3], "scale": 1.5},
+            "shared": {"ff": f[4], "limit": 7.0} if f[4] else None}})
+    return ModelConfig.from_layer_list({"architecture": "Pererax", "width": width, "vocab": vocab,
+                                        "norm": {"eps": eps}, "layers": out})
 
 
 def _llama(layers, hidden, heads, kv, inter, **kw) -> ModelConfig:
@@ -606,6 +762,13 @@ PRESETS: dict[str, ModelConfig] = {
                                                            "original": 512}}}, 256),
         ({"heads": 4, "dim": 32, "vdim": 32, "kv_rank": 48, "rot_dim": 16, "scale": 0.2,
           "mask": {"size": 33}, "rot": {"base": 5000.0, "dims": 16}}, None)], loop=(1, 3, 2)),
+    "pererax-tiny": _pererax(160, 1024, [
+        ({"heads": 4, "kv_heads": 2, "dim": 40, "vdim": 56, "conv": 3}, (64, 6, 2, 3, 96)),
+        ({"left": {"heads": 4, "kv_heads": 2, "dim": 40, "vdim": 32, "scale": 0.16, "softcap": 20.0,
+                   "rot": {"base": 10000.0, "dims": 24}},
+          "right": {"heads": 3, "dim": 24, "vdim": 40, "gate_cap": 10.0}}, (48, 4, 1, 2, 0)),
+        ({"heads": 6, "kv_heads": 3, "dim": 32, "vdim": 32, "scale": 0.18, "mask": {"size": 50},
+          "rot": {"base": 10000.0, "dims": 32}}, None), 0, 1]),
 }
 
 
@@ -881,6 +1044,9 @@ class EngineConfig:
                                       "parallelism)" % m.architecture)
         if self.forest_cascade.enabled:
             raise NotImplementedError("forest cascade attention with %s" % m.architecture)
+        if m.has_state and self.speculative is not None:
+            raise NotImplementedError("speculative decoding with %s: the state of its recurrent "
+                                      "layers cannot take rejected tokens back" % m.architecture)
 
     @property
     def kv_replication(self) -> int:
@@ -1042,7 +1208,8 @@ class EngineArgs:
                             gpu_memory_utilization=self.gpu_memory_utilization,
                             num_gpu_blocks=self.num_gpu_blocks_override,
                             kv_cache_dtype=self.kv_cache_dtype,
-                            enable_prefix_caching=self.enable_prefix_caching)
+                            # (a cached block holds no state of the recurrent layers)
+                            enable_prefix_caching=self.enable_prefix_caching and not model.has_state)
         sched = SchedulerConfig(
             max_num_batched_tokens=self.max_num_batched_tokens or max(8192, 0),
             max_num_seqs=self.max_num_seqs, max_model_len=max_len,

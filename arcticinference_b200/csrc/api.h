@@ -112,7 +112,7 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
                         int max_blocks, const void* work, int num_work, const void* tok_splits,
                         int max_splits, long long T, int Hq, int Hkv, int Dk, int D, int mask_kind,
                         int mask_size, const void* sink, const void* gate, long long ldg,
-                        float scale, void* out, long long ldo, void* o_part, void* lse_part,
+                        float scale, float softcap, void* out, long long ldo, void* o_part, void* lse_part,
                         int tile_keys, int* status, cudaStream_t stream);
 int ab200_attention_merge(const void* o_part, const void* lse_part, const void* tok_splits,
                           long long T, int Hq, int D, void* out, long long ldo,
@@ -246,6 +246,10 @@ int ab200_stream_norm(const void* x, const void* rows, const void* y, long long 
 int ab200_stream_sandwich(void* x, const void* y, long long ldy, const void* w_out, const void* step,
                           const void* w_in, void* act, float eps, float offset, long long T, int W,
                           int dtype, cudaStream_t stream);
+int ab200_stream_add(void* x, void* act, const void* w, const void* y, long long ldy, const void* wy,
+                     const void* y2, long long ldy2, const void* wy2, const void* y_rows,
+                     const void* y_weights, int top, const void* shared, long long ld_shared,
+                     float eps, long long T, int W, int dtype, cudaStream_t stream);
 int ab200_latent_norm_cache(const void* ckv, long long ld, const void* weight, int R, int Rp,
                             float eps, const void* slots, void* cache, long long num_slots,
                             long long T, int dtype, int* status, cudaStream_t stream);
@@ -262,7 +266,7 @@ int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row
                           int max_blocks, const void* tok_seq, const void* positions,
                           const void* sink, const void* gate, long long ldg, void* out,
                           long long ldo, long long T, int H, int Hkv, int Dk, int Dv, int mask_kind,
-                          int mask_size, float scale, int dtype, int* status, cudaStream_t stream);
+                          int mask_size, float scale, float softcap, int dtype, int* status, cudaStream_t stream);
 
 // ---- rotary.cu
 int ab200_rotary_table(const void* positions, const void* freq, void* table, long long T, int half,
@@ -270,19 +274,35 @@ int ab200_rotary_table(const void* positions, const void* freq, void* table, lon
 int ab200_head_rope_cache(void* proj, long long ld, const void* table, int half,
                           const void* slots, const void* wq, const void* wk, void* k_cache,
                           void* v_cache, long long T, int Hq, int Hkv, int D, int dim, int Dv,
-                          int block_size, long long num_slots, float eps, int dtype, int* status,
-                          cudaStream_t stream);
+                          int block_size, long long num_slots, float eps, int whole, int shared_kv,
+                          int dtype, int* status, cudaStream_t stream);
 int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* table, int half,
                             const void* slots, const void* weight, void* cache, long long T, int H,
                             int dq, int dim, int R, int width, int rot_at, long long num_slots,
                             float eps, int dtype, int* status, cudaStream_t stream);
 
 // ---- moe.cu
-int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,
-                    void* ids, void* weights, void* state, void* cursor, void* tiles,
+int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E,
+                    int experts, int top, int all, float scale, void* ids, void* weights, void* state, void* cursor, void* tiles,
                     void* num_tiles, int dtype, cudaStream_t stream);
 int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, void* xp,
-                      long long T, int W, int top, int dtype, cudaStream_t stream);
+                      long long T, int W, int top, int experts, int dtype, cudaStream_t stream);
+
+// ---- recurrent.cu
+int ab200_scan_min_slices(int dim, int ncols);
+int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int b_at,
+                     const void* decay, long long ld_decay, const void* gate, long long ld_gate,
+                     const void* conv, int taps, const void* a_exp, const void* dt_bias,
+                     const void* norm, void* state, int state_cols, void* conv_state, int num_slots,
+                     const void* steps, int n_seq, int max_rows, long long T, int heads, int kv_heads,
+                     int dim, int vdim, int slices, float eps, void* raw, void* out, long long ldo,
+                     int dtype, int* status, cudaStream_t stream);
+int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int i_at, int f_at,
+                      const void* gate, long long ld_gate, const void* i_bias, const void* f_bias,
+                      float cap, const void* norm, void* state, int state_cols, void* max_state,
+                      int num_slots, const void* steps, int n_seq, int max_rows, long long T, int heads,
+                      int dim, int vdim, int slices, float eps, void* raw, void* out, long long ldo,
+                      int dtype, int* status, cudaStream_t stream);
 
 // ---- grouped_gemm.cu
 int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long long x_rows,

@@ -26,9 +26,10 @@
 //
 // Instances with EXT also take a mask with a lower bound (a window, or chunks of positions: the
 // planner starts a tile's keys at the first one its rows see, the softmax masks the rest), a
-// learned sink per head in the denominator (added once, at the end) and an output gate (the
+// sink per head in the denominator (added once, at the end) and an output gate (the
 // normalised rows times sigmoid of a projection, as they are stored). With split keys the merge
-// kernel adds the sink and applies the gate.
+// kernel adds the sink and applies the gate. CAP instances cap the scores softly before the
+// exponential.
 //
 // K/V come either from a paged cache [num_blocks, Hkv, block_size, D] through a
 // block table (one TMA box per block) or from a contiguous [T, Hkv*D]-strided
@@ -75,6 +76,7 @@ struct AttnArgs {
   int causal;
   float scale_log2;  // softmax scale * log2(e)
   float scale;
+  float cap_in, cap_log2;   // CAP instances: scale / cap and cap * log2(e)
   __nv_bfloat16* out;  // [T, Hq*D], row stride ldo
   long long ldo;
   float* o_part;    // [max_splits][T][Hq][D]
@@ -119,7 +121,15 @@ __device__ __forceinline__ uint4 gate8(const uint4& v, const uint4& g) {
   return make_uint4(r[0], r[1], r[2], r[3]);
 }
 
-template <int DK, int D, int TK, bool EXT>   // D: columns of values and outputs
+// cap * log2(e) * tanh(s * scale / cap): a capped score in units of the base-2 exponential. Through
+// 1 - 2 / (e^2x + 1), whose absolute error stays near 1e-7 of the cap.
+__device__ __forceinline__ float capped_score(float s, float in, float cap_log2) {
+  const float e = ex2_approx(s * in * 2.8853900817779268f);   // e^(2 x), inf for large x
+  return fmaf(-2.f * cap_log2, __fdividef(1.f, e + 1.f), cap_log2);
+}
+
+// D: columns of values and outputs; CAP (with EXT): softly capped scores
+template <int DK, int D, int TK, bool EXT, bool CAP>
 __global__ void __launch_bounds__(AttnShape<DK, TK>::kThreads, (AttnShape<DK, TK>::kPrefill ? 1 : 2))
 attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const AttnArgs p) {
@@ -407,7 +417,9 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     // Decode tiles hold a few valid rows: warps whose 32 rows are all padding only keep the
     // barrier protocol going (their rows of P are never read back by anyone).
     const bool warp_active = quad * 32 < n_q_tok * p.G;
-    const float sc = p.scale_log2;
+    // scores enter the exponential as rank(s) * sc; the cap is monotonic, so maxima are taken before it
+    const float sc = CAP ? 1.f : p.scale_log2;
+    auto rank = [&](float s) { return CAP ? capped_score(s, p.cap_in, p.cap_log2) : s; };
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int st = j & 1;
       const uint32_t ph = (uint32_t)(j >> 1) & 1u;
@@ -484,9 +496,9 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         m_tile = fmaxf(__bfloat162float(mine), __bfloat162float(__ushort_as_bfloat16(theirs)));
       }
       const float m_new = fmaxf(m, m_tile);
-      const float m_safe = (m_new == -INFINITY) ? 0.f : m_new;
+      const float m_safe = (m_new == -INFINITY) ? 0.f : rank(m_new);
       // rows that have seen no key yet (m = -inf) hold O = 0 and l = 0: nothing to rescale
-      const float alpha = (m == -INFINITY) ? 1.0f : ex2_approx((m - m_safe) * sc);
+      const float alpha = (m == -INFINITY) ? 1.0f : ex2_approx((rank(m) - m_safe) * sc);
       const float neg_ms = -m_safe * sc;
       // A rescale of O must not race with PV(j-1) accumulating into it, and P(j) overwrites the
       // buffer that PV(j - kPStages) reads from: wait for the later of the products concerned.
@@ -529,10 +541,10 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         uint32_t pk[16];
 #pragma unroll
         for (int t = 0; t < 32; t += 4) {
-          float e0 = ex2_approx(fmaf(__uint_as_float(cur[t + 0]), sc, neg_ms));
-          float e1 = ex2_approx(fmaf(__uint_as_float(cur[t + 1]), sc, neg_ms));
-          float e2 = ex2_approx(fmaf(__uint_as_float(cur[t + 2]), sc, neg_ms));
-          float e3 = ex2_approx(fmaf(__uint_as_float(cur[t + 3]), sc, neg_ms));
+          float e0 = ex2_approx(fmaf(rank(__uint_as_float(cur[t + 0])), sc, neg_ms));
+          float e1 = ex2_approx(fmaf(rank(__uint_as_float(cur[t + 1])), sc, neg_ms));
+          float e2 = ex2_approx(fmaf(rank(__uint_as_float(cur[t + 2])), sc, neg_ms));
+          float e3 = ex2_approx(fmaf(rank(__uint_as_float(cur[t + 3])), sc, neg_ms));
           if (need_mask) {
             const int k = key0 + c * 32 + t;
             e0 = sees(k + 0) ? e0 : 0.f;
@@ -605,11 +617,12 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     if (ok && warp_active) {  // warp-uniform: every lane takes part in the TMEM reads
       const long long tok = (long long)q_tok0 + tok_local;
       const int head = kvh * p.g_heads + g;
+      if (CAP) m = rank(m);
       // (split keys: the merge adds the sink, once)
       if (EXT && p.sink != nullptr && num_splits <= 1 && valid_row && l > 0.f)
         l += ex2_approx(p.sink[head] * 1.4426950408889634f - m * sc);
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      const float lse = l > 0.f ? m * p.scale + logf(l) : -INFINITY;
+      const float lse = l > 0.f ? m * (CAP ? 0.6931471805599453f : p.scale) + logf(l) : -INFINITY;
       __nv_bfloat16* dst16 = p.out + tok * p.ldo + (long long)head * D;
       if (p.peer_tokens > 0)
         dst16 = p.peer_out[tok / p.peer_tokens] + (tok % p.peer_tokens) * p.ldo + (long long)head * D;
@@ -785,9 +798,10 @@ struct AttnExt {
   const void* sink;
   const void* gate;
   long long ldg;
+  float softcap;
 };
 
-template <int DK, int D, int TK, bool EXT>
+template <int DK, int D, int TK, bool EXT, bool CAP = false>
 static int launch_attention(const void* q, long long ldq, const void* k, const void* v,
                             long long ld_kv, long long num_blocks, int block_size,
                             const int* block_tables, int max_blocks, const int* work, int num_work,
@@ -812,7 +826,7 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
       128 * DK * 2 + 2 * (size_t)TK * (DK + D) * 2 +
       (AttnShape<DK, TK>::kPrefill ? 2 : 1) * (size_t)128 * TK * 2 + 256;
   if (!attr_set[dev]) {
-    if (cudaFuncSetAttribute(attention_kernel<DK, D, TK, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attention_kernel<DK, D, TK, EXT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)smem) != cudaSuccess)
       return -3;
     attr_set[dev] = true;
@@ -871,6 +885,10 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
     a.sink = reinterpret_cast<const float*>(ext->sink);
     a.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);
     a.ldg = ext->ldg;
+    if (CAP) {
+      a.cap_in = scale / ext->softcap;
+      a.cap_log2 = ext->softcap * 1.4426950408889634f;
+    }
   }
   TailSignal sig;
   memset(&sig, 0, sizeof(sig));
@@ -885,8 +903,8 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
   }
   if (max_splits <= 1) a.sig = sig;
   dim3 grid((unsigned)num_work * (unsigned)Hkv);
-  (void)launch_pdl(attention_kernel<DK, D, TK, EXT>, grid, dim3(AttnShape<DK, TK>::kThreads), smem, stream, tq,
-                   tk, tv, a);
+  (void)launch_pdl(attention_kernel<DK, D, TK, EXT, CAP>, grid, dim3(AttnShape<DK, TK>::kThreads), smem,
+                   stream, tq, tk, tv, a);
   if (cudaGetLastError() != cudaSuccess) return -5;
   a.sig = sig;
   if (max_splits > 1) {
@@ -904,13 +922,13 @@ using namespace ab200;
 
 extern "C" {
 
-#define AB200_ATTN_DISPATCH(EXT, ...)                                                      \
+#define AB200_ATTN_DISPATCH(EXT, CAP, ...)                                                 \
   do {                                                                                     \
     const bool small = tile_keys == 64 && (block_size == 0 || block_size <= 64);           \
-    if (D == 128) return small ? launch_attention<128, 128, 64, EXT>(__VA_ARGS__)          \
-                               : launch_attention<128, 128, 128, EXT>(__VA_ARGS__);        \
-    if (D == 64) return small ? launch_attention<64, 64, 64, EXT>(__VA_ARGS__)             \
-                              : launch_attention<64, 64, 128, EXT>(__VA_ARGS__);           \
+    if (D == 128) return small ? launch_attention<128, 128, 64, EXT, CAP>(__VA_ARGS__)     \
+                               : launch_attention<128, 128, 128, EXT, CAP>(__VA_ARGS__);   \
+    if (D == 64) return small ? launch_attention<64, 64, 64, EXT, CAP>(__VA_ARGS__)        \
+                              : launch_attention<64, 64, 128, EXT, CAP>(__VA_ARGS__);      \
     return -2;                                                                             \
   } while (0)
 
@@ -929,7 +947,7 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
   if (num_work <= 0 || T <= 0) return 0;
   if ((ldq % 8) || (ldo % 8) || (ld_kv % 8)) return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
-  AB200_ATTN_DISPATCH(false, q, ldq, k, v, ld_kv, num_blocks, block_size,
+  AB200_ATTN_DISPATCH(false, false, q, ldq, k, v, ld_kv, num_blocks, block_size,
                       reinterpret_cast<const int*>(block_tables), max_blocks,
                       reinterpret_cast<const int*>(work), num_work,
                       reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, causal, scale,
@@ -937,7 +955,8 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
                       reinterpret_cast<float*>(lse_out), status, stream);
 }
 
-// The same with a mask (0 causal, 1 window, 2 chunk, see first_visible), an optional sink per query
+// The same with a mask (0 causal, 1 window, 2 chunk, see first_visible), softly capped scores
+// (softcap * tanh(score / softcap), 0: not), an optional sink per query
 // head (fp32 [Hq]) and an optional output gate (bf16 rows of stride ldg, columns like out's).
 // Always causal; the work list's kv_start must not lie above the first key a tile's rows see.
 // Queries and keys have Dk columns per head, values and outputs D; they may differ (192, 128) with
@@ -947,15 +966,16 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
                         int max_blocks, const void* work, int num_work, const void* tok_splits,
                         int max_splits, long long T, int Hq, int Hkv, int Dk, int D, int mask_kind,
                         int mask_size, const void* sink, const void* gate, long long ldg,
-                        float scale, void* out, long long ldo, void* o_part, void* lse_part,
-                        int tile_keys, int* status, cudaStream_t stream) {
+                        float scale, float softcap, void* out, long long ldo, void* o_part,
+                        void* lse_part, int tile_keys, int* status, cudaStream_t stream) {
   if (num_work <= 0 || T <= 0) return 0;
-  if ((ldq % 8) || (ldo % 8) || (ld_kv % 8)) return -2;
+  if ((ldq % 8) || (ldo % 8) || (ld_kv % 8) || softcap < 0.f) return -2;
   if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
     return -2;
   if (gate != nullptr && ((ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
-  const AttnExt ext = {mask_kind, mask_size, sink, gate, ldg};
+  const AttnExt ext = {mask_kind, mask_size, sink, gate, ldg, softcap};
+  if (softcap > 0.f && Dk != D) return -2;
   if (Dk == 192 && D == 128)
     return launch_attention<192, 128, 64, true>(
         q, ldq, k, v, ld_kv, num_blocks, block_size, reinterpret_cast<const int*>(block_tables),
@@ -964,7 +984,14 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
         reinterpret_cast<float*>(o_part), reinterpret_cast<float*>(lse_part), nullptr, status, stream,
         nullptr, 0, 0, nullptr, &ext);
   if (Dk != D) return -2;
-  AB200_ATTN_DISPATCH(true, q, ldq, k, v, ld_kv, num_blocks, block_size,
+  if (softcap > 0.f)
+    AB200_ATTN_DISPATCH(true, true, q, ldq, k, v, ld_kv, num_blocks, block_size,
+                        reinterpret_cast<const int*>(block_tables), max_blocks,
+                        reinterpret_cast<const int*>(work), num_work,
+                        reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, 1, scale,
+                        out, ldo, reinterpret_cast<float*>(o_part), reinterpret_cast<float*>(lse_part),
+                        nullptr, status, stream, nullptr, 0, 0, nullptr, &ext);
+  AB200_ATTN_DISPATCH(true, false, q, ldq, k, v, ld_kv, num_blocks, block_size,
                       reinterpret_cast<const int*>(block_tables), max_blocks,
                       reinterpret_cast<const int*>(work), num_work,
                       reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, 1, scale,
@@ -1020,7 +1047,7 @@ int ab200_attention_scatter_sync(const void* q, long long ldq, const void* k, co
   if (num_work <= 0 || T <= 0) return 0;
   if ((ldq % 8) || (ldo % 8) || peer_tokens <= 0) return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
-  AB200_ATTN_DISPATCH(false, q, ldq, k, v, 0, num_blocks, block_size,
+  AB200_ATTN_DISPATCH(false, false, q, ldq, k, v, 0, num_blocks, block_size,
                       reinterpret_cast<const int*>(block_tables), max_blocks,
                       reinterpret_cast<const int*>(work), num_work,
                       reinterpret_cast<const int*>(tok_splits), max_splits, T, Hq, Hkv, 1, scale,

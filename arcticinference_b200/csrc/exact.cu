@@ -114,7 +114,7 @@ struct ExactAttnArgs {
   long long ldo;
   int H, Hkv, Dk, Dv, num_blocks;
   int mask_kind, mask_size;
-  float scale;
+  float scale, softcap;     // softcap > 0: scores become softcap * tanh(score / softcap)
   int* status;
 };
 
@@ -156,6 +156,7 @@ __global__ void __launch_bounds__(kAttnKeys) attention_exact_kernel(const ExactA
         float d = 0.f;
         for (int i = 0; i < p.Dk; ++i) d = fmaf(q[i], to_f32<T>(kr[i]), d);
         s = d * p.scale;
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       } else {
         rowp[tid] = 0;
         report_error(p.status, kErrBounds, 42, (int)t);
@@ -224,7 +225,8 @@ int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row
                           int max_blocks, const void* tok_seq, const void* positions,
                           const void* sink, const void* gate, long long ldg, void* out,
                           long long ldo, long long T, int H, int Hkv, int Dk, int Dv, int mask_kind,
-                          int mask_size, float scale, int dtype, int* status, cudaStream_t stream) {
+                          int mask_size, float scale, float softcap, int dtype, int* status,
+                          cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H < 1 || Hkv < 1 || H % Hkv || Dk > k_row || Dv > v_row || block_size < 1) return -2;
   if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
@@ -246,6 +248,7 @@ int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row
   a.num_blocks = num_blocks;
   a.mask_kind = mask_kind; a.mask_size = mask_size;
   a.scale = scale;
+  a.softcap = softcap;
   a.status = status;
   const dim3 grid((unsigned)T, (unsigned)H);
   auto kern = dtype == 0 ? attention_exact_kernel<bf16> : attention_exact_kernel<float>;

@@ -6,7 +6,9 @@
 //                and the softmax over those; rows per expert are counted on the way, and the
 //                block that finishes last turns the counts into each expert's first row among
 //                the rows sorted by expert and into the list of 128-row tiles the grouped matrix
-//                products walk
+//                products walk. Or, scoring over all outputs: the softmax over all of them, the
+//                choice by score plus a correction, the chosen scores times a scale as weights;
+//                outputs beyond the experts are identity experts, which get no rows
 //   moe_permute  row of every (token, choice) and the copy of the token's activations there
 //
 // The weighted sum of the experts' outputs is taken by the norm kernel that follows (stream.cu).
@@ -44,9 +46,12 @@ struct Raw4<__nv_bfloat16> {
 struct RouteArgs {
   const float* x;
   const void* w;       // [E][W]
-  const float* b;
+  const float* b;      // [E] bias of the logits, or correction of the choice; may be null
   long long n;
-  int W, E, top;
+  int W, E, top;       // E: router outputs
+  int experts;         // of them the experts' (the others: identity)
+  int all;             // softmax over all outputs instead of the chosen ones
+  float scale;         // of the weights (all)
   int* ids;            // [n][top]
   float* weights;      // [n][top]
   int* state;          // [E] counts and [1] finished blocks; zero before and after every launch
@@ -57,7 +62,7 @@ struct RouteArgs {
 
 // Run by the last block: counts -> first rows and tiles; leaves the counts at zero.
 __device__ void moe_plan(const RouteArgs& p, int* sh) {
-  const int E = p.E;
+  const int E = p.experts;
   int* count = sh;            // [E]
   int* first = sh + E;        // [E]
   int* tile0 = sh + 2 * E;    // [E]
@@ -184,7 +189,8 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
 #pragma unroll
       for (int j = 0; j < EB; ++j) {
         const float s = warp_sum(acc[t][j]);
-        if (lane == 0 && e0 + j < E) z[t * E + e0 + j] = s + p.b[e0 + j];
+        if (lane == 0 && e0 + j < E)
+          z[t * E + e0 + j] = p.b != nullptr && !p.all ? s + p.b[e0 + j] : s;
       }
   }
   __syncthreads();
@@ -192,6 +198,22 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
   for (int t = warp; t < nt; t += kRouteThreads / 32) {
     float* zt = z + t * E;
     float first = 0.f, sum = 0.f;
+    if (p.all) {   // logits -> scores plus correction
+      float mx = -INFINITY;
+      for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zt[e]);
+      mx = warp_max(mx);
+      for (int e = lane; e < E; e += 32) {
+        const float ex = expf(zt[e] - mx);
+        sum += ex;
+        zt[e] = ex;
+      }
+      const float inv = 1.f / warp_sum(sum);
+      for (int e = lane; e < E; e += 32) {
+        zt[E * TB + e] = zt[e] * inv;
+        zt[e] = zt[e] * inv + (p.b != nullptr ? p.b[e] : 0.f);
+      }
+      __syncwarp();
+    }
     int* my_ids = p.ids + (t0 + t) * top;
     float* my_w = p.weights + (t0 + t) * top;
     for (int j = 0; j < top; ++j) {
@@ -215,16 +237,17 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
       }
       bi = min(bi, E - 1);   // (a row of NaNs must still name an expert)
       if (j == 0) first = best;
-      const float ex = expf(best - first);
+      const float ex = p.all ? zt[E * TB + bi] * p.scale : expf(best - first);
       sum += ex;
       if (lane == 0) {
         my_ids[j] = bi;
         my_w[j] = ex;
         zt[bi] = -INFINITY;
-        atomicAdd(p.state + bi, 1);
+        if (bi < p.experts) atomicAdd(p.state + bi, 1);
       }
       __syncwarp();
     }
+    if (p.all) continue;
     const float inv = 1.f / sum;
     for (int j = lane; j < top; j += 32) my_w[j] *= inv;
   }
@@ -232,8 +255,8 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
   __threadfence();
   __syncthreads();
   if (threadIdx.x == 0) {
-    last = atomicAdd(p.state + E, 1) == (int)gridDim.x - 1;
-    if (last) p.state[E] = 0;
+    last = atomicAdd(p.state + p.experts, 1) == (int)gridDim.x - 1;
+    if (last) p.state[p.experts] = 0;
   }
   __syncthreads();
   if (last) {
@@ -246,13 +269,14 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_permute_kernel(const T* __restrict__ x, const int* __restrict__ ids, int* __restrict__ cursor,
-                   int* __restrict__ rows, T* __restrict__ xp, int W, int top) {
+                   int* __restrict__ rows, T* __restrict__ xp, int W, int top, int experts) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ int row[];
   const long long t = blockIdx.x;
   for (int j = threadIdx.x; j < top; j += blockDim.x) {
-    row[j] = atomicAdd(&cursor[ids[t * top + j]], 1);
+    const int e = ids[t * top + j];
+    row[j] = e < experts ? atomicAdd(&cursor[e], 1) : -1;   // (an identity expert has no rows)
     rows[t * top + j] = row[j];
   }
   __syncthreads();
@@ -261,19 +285,21 @@ moe_permute_kernel(const T* __restrict__ x, const int* __restrict__ ids, int* __
   if (W % V == 0) {
     for (int c = threadIdx.x; c < W / V; c += blockDim.x) {
       const uint4 v = reinterpret_cast<const uint4*>(src)[c];
-      for (int j = 0; j < top; ++j) reinterpret_cast<uint4*>(xp + (long long)row[j] * W)[c] = v;
+      for (int j = 0; j < top; ++j)
+        if (row[j] >= 0) reinterpret_cast<uint4*>(xp + (long long)row[j] * W)[c] = v;
     }
   } else {
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
       const T v = src[c];
-      for (int j = 0; j < top; ++j) xp[(long long)row[j] * W + c] = v;
+      for (int j = 0; j < top; ++j)
+        if (row[j] >= 0) xp[(long long)row[j] * W + c] = v;
     }
   }
 }
 
 template <typename T, int TB>
 static int launch_route(const RouteArgs& a, cudaStream_t stream) {
-  size_t smem = ((size_t)TB * a.W + (size_t)TB * a.E) * sizeof(float);
+  size_t smem = ((size_t)TB * a.W + (size_t)TB * a.E * (a.all ? 2 : 1)) * sizeof(float);
   if (smem < (size_t)3 * a.E * sizeof(int)) smem = (size_t)3 * a.E * sizeof(int);
   if (smem > 220 * 1024) return -6;
   // few tokens: more warps per block, so that each has few experts to go through
@@ -295,14 +321,15 @@ typedef __nv_bfloat16 bf16;
 
 extern "C" {
 
-// x fp32 [T, W]; w [E, W] (dtype 0 = bf16, 1 = fp32); b fp32 [E]; ids int32 and weights fp32
-// [T, top]; state int32 [E + 1], zero; cursor int32 [E]; tiles int32 x 4 [T * top / 128 + E at
-// most]; num_tiles int32 [1]
-int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E, int top,
-                    void* ids, void* weights, void* state, void* cursor, void* tiles,
+// x fp32 [T, W]; w [E, W] (dtype 0 = bf16, 1 = fp32); b fp32 [E] or null; the first `experts` of the
+// E outputs are experts, the others the identity; all, scale: see RouteArgs. ids int32 and weights fp32
+// [T, top]; state int32 [experts + 1], zero; cursor int32 [experts]; tiles int32 x 4 [T * top / 128 +
+// experts at most]; num_tiles int32 [1]
+int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E,
+                    int experts, int top, int all, float scale, void* ids, void* weights, void* state, void* cursor, void* tiles,
                     void* num_tiles, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (top < 1 || top > E) return -2;
+  if (top < 1 || top > E || experts < 1 || experts > E) return -2;
   RouteArgs a;
   a.x = reinterpret_cast<const float*>(x);
   a.w = w;
@@ -311,6 +338,9 @@ int ab200_moe_route(const void* x, const void* w, const void* b, long long T, in
   a.W = W;
   a.E = E;
   a.top = top;
+  a.experts = experts;
+  a.all = all;
+  a.scale = scale;
   a.ids = reinterpret_cast<int*>(ids);
   a.weights = reinterpret_cast<float*>(weights);
   a.state = reinterpret_cast<int*>(state);
@@ -324,7 +354,7 @@ int ab200_moe_route(const void* x, const void* w, const void* b, long long T, in
 }
 
 int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, void* xp,
-                      long long T, int W, int top, int dtype, cudaStream_t stream) {
+                      long long T, int W, int top, int experts, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   const size_t smem = (size_t)top * sizeof(int);
   const cudaError_t e =
@@ -332,11 +362,11 @@ int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, 
           ? launch_pdl(moe_permute_kernel<bf16>, dim3((unsigned)T), dim3(256), smem, stream,
                        reinterpret_cast<const bf16*>(x), reinterpret_cast<const int*>(ids),
                        reinterpret_cast<int*>(cursor), reinterpret_cast<int*>(rows),
-                       reinterpret_cast<bf16*>(xp), W, top)
+                       reinterpret_cast<bf16*>(xp), W, top, experts)
           : launch_pdl(moe_permute_kernel<float>, dim3((unsigned)T), dim3(256), smem, stream,
                        reinterpret_cast<const float*>(x), reinterpret_cast<const int*>(ids),
                        reinterpret_cast<int*>(cursor), reinterpret_cast<int*>(rows),
-                       reinterpret_cast<float*>(xp), W, top);
+                       reinterpret_cast<float*>(xp), W, top, experts);
   return e == cudaSuccess ? 0 : -5;
 }
 

@@ -3,8 +3,10 @@
 //
 //   rotary_table       cosine and sine of every token's angles (angle = position * frequency in
 //                      fp32), once per step for all layers with the same frequencies
-//   head_rope_cache    per-head RMS norm of queries and keys (optional), rotation of their first
-//                      rot dimensions, queries in place, keys and values to the paged cache
+//   head_rope_cache    RMS norm of queries and keys (optional; per head, or over all query and all
+//                      key heads of a token at once), rotation of their first rot dimensions,
+//                      queries in place, keys and values to the paged cache; the values may be
+//                      the raw keys
 //   latent_rope_cache  RMS norm of a compressed K/V projection and rotation of the key part that
 //                      the heads share, both to the paged latent cache; rotation of every query
 //                      head's rotary part in place
@@ -47,15 +49,49 @@ struct HeadRopeArgs {
   long long ld;
   const float* table;       // [T][half][2]
   const long long* slots;
-  const float* wq;          // [D] or null: no norm
+  const float* wq;          // [D], with `whole` [Hq * D]; null: no norm
   const float* wk;
+  int whole;                // the norm's mean is over all heads' columns
+  int shared_kv;            // no value heads in proj: the unnormed, unrotated keys are the values
   void* k_cache;            // [num_blocks][Hkv][block_size][D]
   void* v_cache;            // [num_blocks][Hkv][block_size][Dv]
   long long num_slots;
   int Hq, Hkv, D, Dv, half, block_size;
-  float rdim, eps;          // 1 / (dimensions the norm's mean is over; columns beyond are zero)
+  float rdim, rdim_k, eps;  // 1 / (dimensions the norm's mean is over; columns beyond are zero)
   int* status;
 };
+
+// Sums of the squares of a token's query and key columns, for norms over the whole projection.
+template <typename T>
+__device__ __forceinline__ float2 projection_squares(const T* base, int nq, int nk, bool vec) {
+  __shared__ float red[2][32];
+  float q = 0.f, k = 0.f;
+  if (vec) {
+    for (int i = threadIdx.x * 4; i < nq + nk; i += kRopeThreads * 4) {
+      const float4 v = load4(base + i);
+      const float s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      if (i < nq) q += s;
+      else k += s;
+    }
+  } else {
+    for (int i = threadIdx.x; i < nq + nk; i += kRopeThreads) {
+      const float v = to_f32<T>(base[i]);
+      if (i < nq) q += v * v;
+      else k += v * v;
+    }
+  }
+  q = warp_sum(q);
+  k = warp_sum(k);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (lane == 0) {
+    red[0][warp] = q;
+    red[1][warp] = k;
+  }
+  __syncthreads();
+  q = lane < kRopeThreads / 32 ? red[0][lane] : 0.f;
+  k = lane < kRopeThreads / 32 ? red[1][lane] : 0.f;   // (all columns have been read)
+  return make_float2(warp_sum(q), warp_sum(k));
+}
 
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const HeadRopeArgs p) {
@@ -76,12 +112,18 @@ __global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const Hea
   const long long blk = slot >= 0 ? slot / p.block_size : 0;
   const long long off = slot >= 0 ? slot % p.block_size : 0;
   T* base = reinterpret_cast<T*>(p.proj) + t * p.ld;
+  float inv_q = 1.f, inv_k = 1.f;
+  if (p.whole) {
+    const float2 ss = projection_squares(base, p.Hq * p.D, p.Hkv * p.D, VEC);
+    inv_q = 1.f / sqrtf(ss.x * p.rdim + p.eps);
+    inv_k = 1.f / sqrtf(ss.y * p.rdim_k + p.eps);
+  }
   for (int j = warp; j < p.Hq + 2 * p.Hkv; j += kRopeThreads / 32) {
     const bool is_q = j < p.Hq, is_v = j >= p.Hq + p.Hkv;
     if (!is_q && slot < 0) continue;   // padding token: no key, no value
     if (is_v) {
       const int g = j - p.Hq - p.Hkv;
-      const T* src = base + (long long)(p.Hq + p.Hkv) * p.D + (long long)g * p.Dv;
+      const T* src = base + (long long)(p.shared_kv ? p.Hq : p.Hq + p.Hkv) * p.D + (long long)g * p.Dv;
       T* dst = reinterpret_cast<T*>(p.v_cache) + ((blk * p.Hkv + g) * p.block_size + off) * p.Dv;
       if (VEC) {
         for (int i = lane * 4; i < p.Dv; i += 128) store4(dst + i, load4(src + i));
@@ -93,7 +135,10 @@ __global__ void __launch_bounds__(kRopeThreads) head_rope_cache_kernel(const Hea
     T* src = base + (long long)j * p.D;
     const float* w = is_q ? p.wq : p.wk;
     float inv = 1.f;
-    if (w != nullptr) {
+    if (p.whole) {
+      w += (long long)(is_q ? j : j - p.Hq) * p.D;
+      inv = is_q ? inv_q : inv_k;
+    } else if (w != nullptr) {
       float ss = 0.f;
       if (VEC) {
         for (int i = lane * 4; i < p.D; i += 128) {
@@ -151,6 +196,7 @@ __global__ void __launch_bounds__(kRopeThreads, 4) head_rope_cache_wide_kernel(c
   const int i0 = (lane % kLanes) * 4;           // this lane's columns
   const int j0 = warp * kPer + lane / kLanes;   // its first head
   const int heads = p.Hq + 2 * p.Hkv;
+  const int v_back = p.shared_kv ? p.Hkv : 0;   // value heads read the key heads' columns
   __nv_bfloat16* base = reinterpret_cast<__nv_bfloat16*>(p.proj) + t * p.ld + i0;
   const int side = i0 < p.half ? 0 : i0 < 2 * p.half ? 1 : 2;   // first, second of a pair, neither
   const int other = side == 0 ? lane + p.half / 4 : side == 1 ? lane - p.half / 4 : lane;
@@ -159,9 +205,16 @@ __global__ void __launch_bounds__(kRopeThreads, 4) head_rope_cache_wide_kernel(c
 #pragma unroll
     for (int f = 0; f < kFlight; ++f) {
       const int j = first + f * kStep + j0;
-      v[f] = j < heads ? load4(base + (long long)j * D) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[f] = j < heads ? load4(base + (long long)(j < p.Hq + p.Hkv ? j : j - v_back) * D)
+                       : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   };
+  float inv_q = 1.f, inv_k = 1.f;
+  if (p.whole) {
+    const float2 ss = projection_squares(base - i0, p.Hq * D, p.Hkv * D, true);
+    inv_q = rsqrtf(ss.x * p.rdim + p.eps);
+    inv_k = rsqrtf(ss.y * p.rdim_k + p.eps);
+  }
   load(0);
   const long long slot = p.slots[t];
   float4 c = make_float4(1.f, 1.f, 1.f, 1.f), sn = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -173,7 +226,7 @@ __global__ void __launch_bounds__(kRopeThreads, 4) head_rope_cache_wide_kernel(c
     sn = make_float4(sg * a.y, sg * a.w, sg * b.y, sg * b.w);
   }
   float4 wq = make_float4(1.f, 1.f, 1.f, 1.f), wk = wq;
-  if (p.wq != nullptr) {
+  if (p.wq != nullptr && !p.whole) {
     wq = load4(p.wq + i0);
     wk = load4(p.wk + i0);
   }
@@ -194,7 +247,14 @@ __global__ void __launch_bounds__(kRopeThreads, 4) head_rope_cache_wide_kernel(c
       float4 x = v[f];
       if (first + f * kStep + warp * kPer < p.Hq + p.Hkv) {   // (else all of the warp's are values)
         float4 z = x;
-        if (p.wq != nullptr) {
+        if (p.whole) {
+          if (j < p.Hq + p.Hkv) {
+            const float4 w = j < p.Hq ? load4(p.wq + (long long)j * D + i0)
+                                      : load4(p.wk + (long long)(j - p.Hq) * D + i0);
+            const float inv = j < p.Hq ? inv_q : inv_k;
+            z = make_float4(x.x * inv * w.x, x.y * inv * w.y, x.z * inv * w.z, x.w * inv * w.w);
+          }
+        } else if (p.wq != nullptr) {
           float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
 #pragma unroll
           for (int o = kLanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -331,16 +391,19 @@ int ab200_rotary_table(const void* positions, const void* freq, void* table, lon
 }
 
 // proj [T, ld] holds Hq query and Hkv key heads of D columns, then Hkv value heads of Dv, of which
-// the first `dim` (query, key) columns are in use and the others zero; wq, wk fp32 [D] or null;
-// table fp32 [T, half, 2]: cosines and sines of the pairs (i, i + half).
+// the first `dim` (query, key) columns are in use and the others zero; wq, wk fp32 [D] or null, with
+// `whole` fp32 [Hq * D] and [Hkv * D] for a norm over all heads at once; table fp32 [T, half, 2]:
+// cosines and sines of the pairs (i, i + half). shared_kv: there are no value heads, the key heads as
+// they come are the values (Dv = D).
 int ab200_head_rope_cache(void* proj, long long ld, const void* table, int half,
                           const void* slots, const void* wq, const void* wk, void* k_cache,
                           void* v_cache, long long T, int Hq, int Hkv, int D, int dim, int Dv,
-                          int block_size, long long num_slots, float eps, int dtype, int* status,
-                          cudaStream_t stream) {
+                          int block_size, long long num_slots, float eps, int whole, int shared_kv,
+                          int dtype, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if ((whole && (wq == nullptr || wk == nullptr)) || (shared_kv && D != Dv)) return -2;
   if (dim < 1 || dim > D || 2 * half > D || half < 0 || block_size < 1 || Hq < 0 || Hkv < 0) return -2;
-  if (ld < (long long)(Hq + Hkv) * D + (long long)Hkv * Dv) return -2;
+  if (ld < (long long)(Hq + Hkv) * D + (shared_kv ? 0ll : (long long)Hkv * Dv)) return -2;
   HeadRopeArgs a;
   a.proj = proj; a.ld = ld;
   a.table = reinterpret_cast<const float*>(table);
@@ -351,7 +414,10 @@ int ab200_head_rope_cache(void* proj, long long ld, const void* table, int half,
   a.num_slots = num_slots;
   a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.Dv = Dv;
   a.half = half; a.block_size = block_size;
-  a.rdim = 1.f / (float)dim;
+  a.whole = whole;
+  a.shared_kv = shared_kv;
+  a.rdim = 1.f / (whole ? (float)Hq * (float)dim : (float)dim);
+  a.rdim_k = 1.f / (whole ? (float)Hkv * (float)dim : (float)dim);
   a.eps = eps;
   a.status = status;
   return dtype == 0 ? launch_head_rope<bf16>(a, T, stream) : launch_head_rope<float>(a, T, stream);

@@ -7,6 +7,9 @@
 //                      with a row list it also serves the final norm of the sampled rows
 //   stream_sandwich    x <- x + norm(y) * w_out (+ a vector), in place, and the next sublayer's
 //                      input act = norm(x) * w_in, in one pass over the row
+//   stream_add         x <- x + norm(y) * w, in place, and the 16-bit copy; y is a sublayer's output,
+//                      half the sum of two normed ones, or a mixture of experts' weighted sum with
+//                      identity experts and a shared expert, formed here in fp32
 //   latent_norm_cache  RMS norm of the compressed K/V projection and its write into the paged
 //                      latent cache
 //   gated_act          act(gate) * up on the interleaved gate / up layout
@@ -240,6 +243,167 @@ static int launch_stream_sandwich(const SandwichArgs& a, long long T_rows, cudaS
   return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), 0, stream, a) == cudaSuccess ? 0 : -5;
 }
 
+struct StreamAddArgs {
+  float* x;
+  void* act;               // optional copy in element type T
+  const float* w;          // norm weight
+  const void* y;           // a sublayer's output rows (a mixture: the experts' rows)
+  long long ldy;
+  const float* wy;         // with y2: weights of the two outputs' own norms
+  const void* y2;
+  long long ldy2;
+  const float* wy2;
+  const int* y_rows;       // mixture: [T][top] rows of y, -1: the token's own stream
+  const float* y_weights;
+  int top;
+  const void* shared;      // mixture: further rows to add, or null
+  long long ld_shared;
+  float eps;
+  int W;
+};
+
+// N4: four-element pieces a thread holds (0: any width, the sublayer's output through shared memory)
+template <typename T, int N4>
+__global__ void __launch_bounds__(256) stream_add_kernel(const StreamAddArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  extern __shared__ __align__(16) float row[];
+  const long long t = blockIdx.x;
+  float* xr = p.x + t * p.W;
+  const T* yb = reinterpret_cast<const T*>(p.y);
+  const T* y2 = p.y2 ? reinterpret_cast<const T*>(p.y2) + t * p.ldy2 : nullptr;
+  const T* sh = p.shared ? reinterpret_cast<const T*>(p.shared) + t * p.ld_shared : nullptr;
+  T* act = p.act ? reinterpret_cast<T*>(p.act) + t * p.W : nullptr;
+  const float rw = 1.f / (float)p.W;
+  if constexpr (N4 > 0) {
+    float4 x[N4], y[N4];
+    auto each = [&](auto f) {
+#pragma unroll
+      for (int j = 0; j < N4; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * 4;
+        if (i < p.W) f(i, x[j], y[j]);
+      }
+    };
+    auto square = [](const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+    float ss = 0.f;
+    if (p.y_rows != nullptr) {
+      each([&](int i, float4& xv, float4& yv) {
+        xv = load4(xr + i);
+        yv = sh != nullptr ? load4(sh + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < p.top; ++k) {
+          const float w = p.y_weights[t * p.top + k];
+          const int r = p.y_rows[t * p.top + k];
+          const float4 v = r >= 0 ? load4(yb + (long long)r * p.ldy + i) : xv;
+          yv.x += w * v.x; yv.y += w * v.y; yv.z += w * v.z; yv.w += w * v.w;
+        }
+        ss += square(yv);
+      });
+    } else if (y2 != nullptr) {
+      float s2 = 0.f;
+      float4 z[N4];
+      each([&](int i, float4& xv, float4& yv) {
+        xv = load4(xr + i);
+        yv = load4(yb + t * p.ldy + i);
+        ss += square(yv);
+      });
+#pragma unroll
+      for (int j = 0; j < N4; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * 4;
+        z[j] = i < p.W ? load4(y2 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s2 += square(z[j]);
+      }
+      const float a = 0.5f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+      const float b = 0.5f / sqrtf(block_sum_all(s2, red) * rw + p.eps);
+      ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < N4; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * 4;
+        if (i >= p.W) continue;
+        const float4 u = load4(p.wy + i), v = load4(p.wy2 + i);
+        y[j] = make_float4(y[j].x * a * u.x + z[j].x * b * v.x, y[j].y * a * u.y + z[j].y * b * v.y,
+                           y[j].z * a * u.z + z[j].z * b * v.z, y[j].w * a * u.w + z[j].w * b * v.w);
+        ss += square(y[j]);
+      }
+    } else {
+      each([&](int i, float4& xv, float4& yv) {
+        xv = load4(xr + i);
+        yv = load4(yb + t * p.ldy + i);
+        ss += square(yv);
+      });
+    }
+    const float inv = 1.f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+    each([&](int i, float4& xv, float4& yv) {
+      const float4 w = load4(p.w + i);
+      xv.x += yv.x * inv * w.x; xv.y += yv.y * inv * w.y;
+      xv.z += yv.z * inv * w.z; xv.w += yv.w * inv * w.w;
+      store4(xr + i, xv);
+      if (act != nullptr) store4(act + i, xv);
+    });
+  } else {
+    float ss = 0.f, s2 = 0.f, a = 0.f, b = 0.f;
+    if (y2 != nullptr) {
+      for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+        const float u = to_f32<T>(yb[t * p.ldy + i]), v = to_f32<T>(y2[i]);
+        ss += u * u;
+        s2 += v * v;
+      }
+      a = 0.5f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+      b = 0.5f / sqrtf(block_sum_all(s2, red) * rw + p.eps);
+      ss = 0.f;
+    }
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x) {   // a thread re-reads only its own columns
+      float v;
+      if (p.y_rows != nullptr) {
+        v = sh != nullptr ? to_f32<T>(sh[i]) : 0.f;
+        for (int k = 0; k < p.top; ++k) {
+          const int r = p.y_rows[t * p.top + k];
+          v += p.y_weights[t * p.top + k] * (r >= 0 ? to_f32<T>(yb[(long long)r * p.ldy + i]) : xr[i]);
+        }
+      } else {
+        v = to_f32<T>(yb[t * p.ldy + i]);
+        if (y2 != nullptr) v = v * a * p.wy[i] + to_f32<T>(y2[i]) * b * p.wy2[i];
+      }
+      row[i] = v;
+      ss += v * v;
+    }
+    const float inv = 1.f / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+      const float v = xr[i] + row[i] * inv * p.w[i];
+      xr[i] = v;
+      if (act != nullptr) act[i] = from_f32<T>(v);
+    }
+  }
+}
+
+template <typename T>
+static int launch_stream_add(const StreamAddArgs& a, long long T_rows, cudaStream_t stream) {
+  const bool vec = a.W % 4 == 0 && a.ldy % 4 == 0 && a.ldy2 % 4 == 0 && a.ld_shared % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.x) |
+                     reinterpret_cast<uintptr_t>(a.y2) | reinterpret_cast<uintptr_t>(a.shared) |
+                     reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.wy) |
+                     reinterpret_cast<uintptr_t>(a.wy2) | reinterpret_cast<uintptr_t>(a.act)) & 15) == 0;
+  const int n4 = (a.W + 3) / 4;
+  auto k = stream_add_kernel<T, 0>;
+  int threads = 256;
+  size_t smem = 0;
+  if (vec && n4 <= 256 * 8) {
+    while (threads > 64 && n4 <= threads) threads /= 2;
+    const int per = (n4 + threads - 1) / threads;
+    k = per <= 1   ? stream_add_kernel<T, 1>
+        : per <= 2 ? stream_add_kernel<T, 2>
+        : per <= 4 ? stream_add_kernel<T, 4>
+                   : stream_add_kernel<T, 8>;
+  } else {
+    smem = (size_t)a.W * sizeof(float);
+    if (smem > 200 * 1024) return -6;
+    if (smem > 48 * 1024 &&
+        cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return -3;
+  }
+  return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), smem, stream, a) == cudaSuccess ? 0 : -5;
+}
+
 // c = ckv / rms(ckv) * w over R columns -> cache row `slot` of Rp columns (the rest stays zero).
 // One warp per token.
 template <typename T>
@@ -398,6 +562,34 @@ int ab200_stream_sandwich(void* x, const void* y, long long ldy, const void* w_o
   a.W = W;
   return dtype == 0 ? launch_stream_sandwich<bf16>(a, T, stream)
                     : launch_stream_sandwich<float>(a, T, stream);
+}
+
+// In place on x [T, W]: x += norm(y) * w; act (may be null): the new x. y: rows of a sublayer's output;
+// with y2: half of norm(y) * wy + norm(y2) * wy2; with y_rows int32 and y_weights fp32 [T, top]: the
+// weighted sum of these rows (row -1: the token's own x, before the update) plus `shared`'s (may be null).
+int ab200_stream_add(void* x, void* act, const void* w, const void* y, long long ldy, const void* wy,
+                     const void* y2, long long ldy2, const void* wy2, const void* y_rows,
+                     const void* y_weights, int top, const void* shared, long long ld_shared,
+                     float eps, long long T, int W, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if ((y2 != nullptr && (wy == nullptr || wy2 == nullptr)) ||
+      (y_rows != nullptr && (y_weights == nullptr || y2 != nullptr)))
+    return -2;
+  StreamAddArgs a;
+  a.x = reinterpret_cast<float*>(x);
+  a.act = act;
+  a.w = reinterpret_cast<const float*>(w);
+  a.y = y; a.ldy = ldy;
+  a.wy = reinterpret_cast<const float*>(wy);
+  a.y2 = y2; a.ldy2 = ldy2;
+  a.wy2 = reinterpret_cast<const float*>(wy2);
+  a.y_rows = reinterpret_cast<const int*>(y_rows);
+  a.y_weights = reinterpret_cast<const float*>(y_weights);
+  a.top = top;
+  a.shared = shared; a.ld_shared = ld_shared;
+  a.eps = eps;
+  a.W = W;
+  return dtype == 0 ? launch_stream_add<bf16>(a, T, stream) : launch_stream_add<float>(a, T, stream);
 }
 
 int ab200_latent_norm_cache(const void* ckv, long long ld, const void* weight, int R, int Rp,

@@ -22,6 +22,7 @@ import torch
 
 from .. import ops
 from ..models.llama import ForwardBatch
+from ..ops.state_ops import StateDecodePlan
 
 
 def canonical_sizes(limit: int = 512) -> list[int]:
@@ -48,7 +49,10 @@ class DecodeGraph:
         max_q = 1 + (cfg.speculative.max_draft_tokens if cfg.speculative else 0)
         self.plans = m.decode_plans(bucket, max_q, runner.block_size)
         n64 = 4 * bucket      # ids | positions | slots | source rows of run-ahead tokens
+        self.state_plan = StateDecodePlan(bucket) if runner.num_state_slots else None
         n32 = bucket * self.max_blocks + sum(p.int32_words for p in self.plans)
+        if self.state_plan is not None:
+            n32 += self.state_plan.int32_words
         pin = dev.type == "cuda"
         self.h64 = torch.zeros(n64, dtype=torch.int64, pin_memory=pin)
         self.h32 = torch.zeros(n32, dtype=torch.int32, pin_memory=pin)
@@ -60,11 +64,15 @@ class DecodeGraph:
         for p in self.plans:
             p.bind(h32[off:off + p.int32_words], self.d32[off:off + p.int32_words], bt)
             off += p.int32_words
+        if self.state_plan is not None:
+            self.state_plan.bind(h32[off:], self.d32[off:])
         self.meta = m.decode_attention(self.plans, bt)
         self.logits_indices = torch.arange(bucket, dtype=torch.int64, device=dev)
         self.batch = ForwardBatch(input_ids=self.d64[:B], positions=self.d64[B:2 * B],
                                   slots=self.d64[2 * B:3 * B], attn_meta=self.meta,
                                   logits_indices=self.logits_indices, num_tokens=B, mode=mode)
+        if self.state_plan is not None:
+            self.batch.state = self.state_plan.step
         if cfg.model.is_swiftkv:
             self.batch.sel_positions = self.batch.positions
             self.batch.sel_attn_meta = self.meta
@@ -110,6 +118,8 @@ class DecodeGraph:
             kv_lens.append(B - N)
         for p in self.plans:
             p.fill(q_lens, kv_lens)
+        if self.state_plan is not None:
+            self.state_plan.fill(out.scheduled)
         return rows
 
     def upload(self) -> None:
@@ -135,7 +145,10 @@ class DecodeGraph:
         return ids, hidden
 
     def capture(self) -> None:
-        # warm-up run outside capture (lazy initialisation, autotuned scratch, tensor maps)
+        # warm-up run outside capture (lazy initialisation, autotuned scratch, tensor maps); it
+        # must leave the requests' states where they are
+        if self.state_plan is not None:
+            self.state_plan.detach()
         self.upload()
         torch.cuda.synchronize()
         self._body()

@@ -8,6 +8,10 @@ without moving KV (reference: arctic_inference/vllm/ulysses.py:60-70,402-416 and
 arctic_inference/vllm/model_runner.py:1758-1772). Every rank runs this manager
 with the same inputs, so block ids agree across ranks without communication.
 
+Models with recurrent layers also keep a state per request. It lies in a slot, one of a fixed number;
+a request takes one with its first blocks and gives it back with them. Slots need no clearing: the
+kernels start a sequence at position 0 from zeros.
+
 Prefix caching: full blocks are keyed by a hash chained over the tokens they
 hold; a finished request's blocks stay in an LRU pool and are revived when a
 later prompt hashes to the same chain.
@@ -16,6 +20,7 @@ later prompt hashes to the same chain.
 from __future__ import annotations
 
 import hashlib
+import math
 import struct
 from collections import OrderedDict
 from dataclasses import dataclass
@@ -106,12 +111,31 @@ class BlockPool:
         self.cached.clear()
 
 
-class KVCacheManager:
-    """Per-request block tables on top of a :class:`BlockPool`."""
+class StateSlots:
+    """Fixed pool of state slots; slot 0 is what padding rows name."""
 
-    def __init__(self, num_blocks: int, block_size: int, enable_prefix_caching: bool = True):
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self.free = list(range(num_slots - 1, 0, -1))
+
+    def take(self, request) -> None:
+        request.state_slot, request.state_phase = self.free.pop(), 0
+
+    def give_back(self, request) -> None:
+        if request.state_slot:
+            self.free.append(request.state_slot)
+            request.state_slot = 0
+
+
+class KVCacheManager:
+    """Per-request block tables on top of a :class:`BlockPool`, and state slots for models that keep
+    a state (``num_state_slots`` > 0)."""
+
+    def __init__(self, num_blocks: int, block_size: int, enable_prefix_caching: bool = True,
+                 num_state_slots: int = 0):
         self.block_size = block_size
         self.pool = BlockPool(num_blocks, enable_prefix_caching)
+        self.states = StateSlots(num_state_slots) if num_state_slots else None
         self._hashes: dict[str, list[bytes]] = {}
 
     # -- prefix cache -------------------------------------------------------------------
@@ -160,12 +184,18 @@ class KVCacheManager:
         return max(0, need - len(request.block_ids))
 
     def can_allocate(self, request, num_new_tokens: int) -> bool:
+        if self.states is not None and not request.state_slot and not self.states.free:
+            return False
         return self.blocks_needed(request, num_new_tokens) <= self.pool.num_free
 
     def allocate(self, request, num_new_tokens: int) -> None:
         n = self.blocks_needed(request, num_new_tokens)
         if n:
             request.block_ids.extend(self.pool.allocate(n))
+        if self.states is not None and not request.state_slot:
+            if not self.states.free:
+                raise RuntimeError("out of state slots")
+            self.states.take(request)
 
     def commit(self, request, num_computed: int) -> None:
         """Called after a step: tokens below ``num_computed`` now have valid KV."""
@@ -175,6 +205,8 @@ class KVCacheManager:
         self.pool.release(request.block_ids)
         request.block_ids = []
         request._block_array = None
+        if self.states is not None:
+            self.states.give_back(request)
         self._hashes.pop(request.request_id, None)
 
     def slot(self, request, position: int) -> int:
@@ -227,15 +259,18 @@ class KVCacheTensors:
 
 
 class RunCacheTensors:
-    """Device memory of a layer-list decoder's cache. Every run of a layer keeps one or two tensors
+    """Device memory of a layer-list decoder's cache. Every run of a layer keeps up to two tensors
     ``[num_blocks, heads, block_size, columns]``: keys and values, or latent rows. A run that takes
     an earlier one's latents has that run's tensors (the same objects), so it costs no memory.
-    The block tables, prefix cache and scheduler above it are those of any other model."""
+    The block tables, prefix cache and scheduler above it are those of any other model. Runs of
+    recurrent layers keep tensors ``[num_slots, ...]`` besides or instead."""
 
     def __init__(self, owners: list, rows: list, num_blocks: int, block_size: int,
-                 dtype: torch.dtype, device):
+                 dtype: torch.dtype, device, states: Optional[list] = None, num_slots: int = 0):
         """``owners[r]``: the run whose cache run r uses; ``rows[r]``: (heads, columns) of each of
-        its tensors."""
+        its tensors; ``states[r]``: (shape, element type) of what a state slot holds of it."""
+        self.states = [tuple(torch.zeros((num_slots, *shape), dtype=dt, device=device)
+                             for shape, dt in t) for t in states or [()] * len(owners)]
         self.runs = []
         for r, o in enumerate(owners):
             self.runs.append(self.runs[o] if o != r else tuple(
@@ -245,10 +280,17 @@ class RunCacheTensors:
     def of(self, run: int) -> tuple:
         return self.runs[run]
 
+    def state_of(self, run: int) -> tuple:
+        return self.states[run]
+
+    @staticmethod
+    def bytes_per_slot(states: list) -> int:
+        return sum(math.prod(shape) * dt.itemsize for t in states for shape, dt in t)
+
     @staticmethod
     def bytes_per_block(owners: list, rows: list, block_size: int, elem_bytes: int) -> int:
         return sum(h * c for r, (o, t) in enumerate(zip(owners, rows)) if o == r for h, c in t) * \
             block_size * elem_bytes
 
     def free(self) -> None:
-        self.runs = []
+        self.runs, self.states = [], []

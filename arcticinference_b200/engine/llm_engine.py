@@ -62,7 +62,8 @@ class LLMEngine:
             self.num_blocks = self.runner.pp.min_over_stages(self.num_blocks, self.device)
         self.runner.init_kv_cache(self.num_blocks)
         self.kv_manager = KVCacheManager(self.num_blocks, config.cache.block_size,
-                                         config.cache.enable_prefix_caching)
+                                         config.cache.enable_prefix_caching,
+                                         num_state_slots=self.runner.num_state_slots)
         self.scheduler = Scheduler(config.scheduler, self.kv_manager, config.speculative,
                                    token_multiple=config.parallel.sp)
         self.tokenizer = get_tokenizer(config.tokenizer or config.model.name_or_path,

@@ -25,6 +25,7 @@ import torch
 from .. import ops
 from ..config import EngineConfig
 from ..models.llama import ForwardBatch, ShardSpec
+from ..ops.state_ops import StateStep
 from ..plugin import model_class
 from ..utils.tracing import trace_range
 from .sampler import row_seed
@@ -125,6 +126,8 @@ class ModelRunner:
             self.model.set_pipeline(self.pp)
         self.kv = None                # the model's cache tensors (engine/kv_cache.py)
         self.num_blocks = 0
+        # state slots of models with recurrent layers: one per running request and the padding's
+        self.num_state_slots = config.scheduler.max_num_seqs + 1 if mcfg.has_state else 0
         self.block_size = config.cache.block_size
         self.sp = config.parallel.sp
         self.shift = config.parallel.enable_shift_parallel
@@ -179,8 +182,10 @@ class ModelRunner:
         # leave room for activations of the largest step and for split-K / split-KV scratch
         reserve = 6 << 30
         budget = int(total * cfg.cache.gpu_memory_utilization) - (total - free) - reserve
+        if self.num_state_slots:
+            budget -= self.num_state_slots * self.model.state_bytes_per_slot()
         need_max = (cfg.scheduler.max_model_len + self.block_size - 1) // self.block_size
-        n = max(budget // per_block, 0)
+        n = max(budget // max(per_block, 1), 0)
         if n < need_max + 1:
             raise RuntimeError("not enough GPU memory for one max_model_len sequence "
                                "(%d blocks available, %d needed)" % (n, need_max + 1))
@@ -189,7 +194,8 @@ class ModelRunner:
 
     def init_kv_cache(self, num_blocks: int) -> None:
         self.num_blocks = num_blocks
-        self.kv = self.model.new_kv_cache(num_blocks, self.block_size)
+        extra = {"num_slots": self.num_state_slots} if self.num_state_slots else {}
+        self.kv = self.model.new_kv_cache(num_blocks, self.block_size, **extra)
 
     # ------------------------------------------------------------- mode choice
     def choose_mode(self, total_tokens: int) -> str:
@@ -349,6 +355,10 @@ class ModelRunner:
                              attn_meta=meta, logits_indices=d[3 * Np:3 * Np + n_sel],
                              num_tokens=Np, mode=mode)
         batch.num_sampled = n_smp
+        if self.num_state_slots:
+            batch.state = StateStep.of(sched, q_lens, Np - N, dev)
+            self.h2d_bytes += batch.state.uploaded_bytes
+            self.h2d_total += batch.state.uploaded_bytes
         if prompt_rows:
             batch.prompt_rows = prompt_rows
             batch.prompt_targets = ops.upload(np.asarray(targets, dtype=np.int64), dev)
@@ -480,6 +490,13 @@ class ModelRunner:
             t += s.num_tokens
         return src if any_src else None
 
+    def _states_moved(self, out: SchedulerOutput) -> None:
+        """The step that has been queued moves its requests' states on: the next one reads what it
+        writes."""
+        if self.num_state_slots:
+            for s in out.scheduled:
+                s.request.state_phase ^= 1
+
     @torch.inference_mode()
     def launch(self, out: SchedulerOutput, prev: Optional["PendingStep"] = None) -> "PendingStep":
         """Queue one step on the device without waiting for its tokens. ``prev`` is the step
@@ -495,6 +512,7 @@ class ModelRunner:
             self.graph_replays += 1
             with trace_range("graph_replay"):
                 ids_dev, hidden = g.replay(prev.ids_dev if src_rows is not None else None)
+            self._states_moved(out)
             self.h2d_total += g.h64.numel() * 8 + g.h32.numel() * 4
             pend = PendingStep(out, rows, ids_dev, hidden, g.bucket, g.mode)
             input_sel = g.batch.input_ids       # every row of a decode graph is a sampled row
@@ -512,9 +530,11 @@ class ModelRunner:
             if batch.logits_indices.numel() == 0:
                 # pure prefill chunk: KV only
                 self.model.forward(batch, self.kv)
+                self._states_moved(out)
                 return PendingStep(out, rows, None, None, batch.num_tokens, batch.mode)
             with trace_range("forward", tokens=batch.num_tokens, mode=batch.mode):
                 hidden = self.model.forward(batch, self.kv)
+            self._states_moved(out)
             if self.pp is not None and hidden is None:
                 # an earlier pipeline stage: the last stage samples and sends the ids to all
                 if batch.prompt_rows:
@@ -566,6 +586,7 @@ class ModelRunner:
             batch, rows = self.prepare(out)
             self.mode_counts[batch.mode] += 1
             hidden = self.model.forward(batch, self.kv)
+        self._states_moved(out)
         of = {id(s): rr for s, rr in zip(out.scheduled, rows)}
         idx = [j for s in given for j in of[id(s)]]
         if not idx:

@@ -52,6 +52,10 @@ class Request:
     output_top_logprobs: Optional[list] = None
     prompt_logprobs: Optional[list] = None     # [None, log P(prompt[1] | prompt[:1]), ...]
     routing_key: Optional[str] = None
+    # models with recurrent layers: the request's state slot (0: none) and which of the slot's two
+    # places for small parts of the state its next step reads (it writes the other)
+    state_slot: int = 0
+    state_phase: int = 0
     _block_array: Optional[object] = field(default=None, repr=False)
     # run-ahead scheduling: the last output token is a placeholder for a token that has been
     # sampled on the device but not read yet / the request ends with that token whatever it is

@@ -1,5 +1,5 @@
 """Decoders whose config.json lists their layers one by one, each with its own mixer and
-feed-forward: Taralix and Zatirax. ``config.LAYER_LIST_DESIGNS`` says what each name stands for;
+feed-forward: Taralix, Zatirax and Pererax. ``config.LAYER_LIST_DESIGNS`` says what each name stands for;
 ``mixers.py`` has the mixers.
 
 Taralix: norms after the residual sum.
@@ -10,14 +10,20 @@ Zatirax: a norm before and after each sublayer, and layers that run several time
 
     x <- x + norm1b(mixer(norm1(x)));   x <- x + norm2b(feed_forward(norm2(x)))
 
+Pererax: a norm and a learned scale on each sublayer's output, which reads the stream itself; layers
+that use other layers' weights.
+
+    x <- x + norm1(mixer(x)) * ls1;   x <- x + norm2(feed_forward(x)) * ls2
+
 The residual stream ``x`` is fp32 from the embedding to the final norm; the projections read the
 model's element type, written by the same kernel that updates the stream. Per layer: one input
 projection, norms and rotation with the cache write, attention, output projection, stream update;
 then gate / up with the activation in the product's epilogue, down, stream update (for experts
 that kernel also takes the weighted sum of the chosen experts' rows). Routing stays on the device.
 
-A *run* is one execution of a layer: a layer inside the loop has one per pass, each with a cache of
-its own (``ModelConfig.layer_runs``).
+A *run* is one execution of a layer: a layer inside the loop has one per pass, and a layer whose
+weights others use one for each of them, each with a cache and state of its own
+(``ModelConfig.layer_runs``).
 
 Served in bfloat16 or, with every product and sum in IEEE fp32, in float32.
 """
@@ -35,7 +41,7 @@ from ..config import LatentAttentionSpec, ModelConfig
 from ..ops import latent_ops as lat
 from ..ops import stream_ops as st
 from .llama import ForwardBatch, ShardSpec
-from .mixers import Checkpoint, HeadMixer, LatentMixer, LayerWeights, mixer_class, padded, round_up
+from .mixers import Checkpoint, LatentMixer, LayerWeights, mixer_class, padded, round_up
 
 _NAME_RE = re.compile(r"^l(\d+)\.(.+)$")
 
@@ -48,12 +54,28 @@ def norm_names(cfg: ModelConfig, spec) -> list:
     return names + [n + "b" for n in names] if cfg.design.residual == "sandwich" else names
 
 
+def scale_names(cfg: ModelConfig, spec) -> list:
+    if cfg.design.residual != "output":
+        return []
+    return ["ls1"] + (["ls2"] if spec.mlp is not None else [])
+
+
+def router_vector(f) -> str:
+    """The vector beside the router's matrix: a bias, or a correction of the choice."""
+    return "mlp.correction" if f.scoring == "all" else "mlp.router.b"
+
+
 def required_tensors(cfg: ModelConfig, spec) -> list:
     """Checkpoint names (without the layer's prefix) of one layer."""
-    names = norm_names(cfg, spec) + mixer_class(spec.mixer).names(spec.mixer)
+    if spec.weights_of is not None:
+        return []
+    names = norm_names(cfg, spec) + scale_names(cfg, spec) + \
+        mixer_class(spec.mixer).names(spec.mixer)
     f = spec.mlp
+    if f is not None and f.shared is not None:
+        names += ["mlp.shared." + n for n in ("gate", "up", "down")]
     if f is not None and f.experts:
-        names += ["mlp.router", "mlp.router.b"]
+        names += ["mlp.router", router_vector(f)]
         names += ["mlp.e%d.%s" % (e, n) for e in range(f.experts) for n in ("gate", "up", "down")]
     elif f is not None:
         names += ["mlp.gate", "mlp.up", "mlp.down"]
@@ -75,25 +97,34 @@ def random_state(cfg: ModelConfig, seed: int, device, dtype) -> Iterable:
 
     W, one = cfg.hidden_size, 1.0 - cfg.design.norm_offset
     yield "embed", rnd(cfg.vocab_size, W, std=1.0)
-    yield "head", rnd(cfg.vocab_size, W)
+    if not cfg.tie_word_embeddings:
+        yield "head", rnd(cfg.vocab_size, W)
     yield "final.norm", one + rnd(W, std=0.1)
     if cfg.loop is not None:
         yield "loop.step", rnd(cfg.loop.times, W, std=0.1)
     for i, l in enumerate(cfg.layer_specs):
         f, p = l.mlp, "l%d." % i
+        if l.weights_of is not None:
+            continue
         for n in norm_names(cfg, l):
             yield p + n, one + rnd(W, std=0.1)
+        for n in scale_names(cfg, l):
+            yield p + n, 1.0 + rnd(W, std=0.1)
         for n, t in mixer_class(l.mixer).random(l.mixer, W, rnd):
             yield p + n, t
         if f is None:
             continue
         if f.experts:
-            yield p + "mlp.router", rnd(f.experts, W)
-            yield p + "mlp.router.b", rnd(f.experts, std=0.1)
-        for q in (["mlp.e%d." % e for e in range(f.experts)] if f.experts else ["mlp."]):
-            yield p + q + "gate", rnd(f.ff, W)
-            yield p + q + "up", rnd(f.ff, W)
-            yield p + q + "down", rnd(W, f.ff)
+            outputs = f.experts + f.identity
+            yield p + "mlp.router", rnd(outputs, W)
+            yield p + router_vector(f), rnd(outputs, std=0.1 if f.scoring == "chosen" else 0.1 / outputs)
+        ffs = {"mlp.e%d." % e: f.ff for e in range(f.experts)} if f.experts else {"mlp.": f.ff}
+        if f.shared is not None:
+            ffs["mlp.shared."] = f.shared.ff
+        for q, ff in ffs.items():
+            yield p + q + "gate", rnd(ff, W)
+            yield p + q + "up", rnd(ff, W)
+            yield p + q + "down", rnd(W, ff)
 
 
 class LayerListForCausalLM:
@@ -128,14 +159,18 @@ class LayerListForCausalLM:
                 sharing = max(k.mixer.heads for k, o in zip(specs, owner) if o == owner[i])
                 self.mixers.append(LatentMixer(l.mixer, sharing, self.dtype, self.device))
             else:
-                self.mixers.append(HeadMixer(l.mixer, self.dtype, self.device))
-        self.gates = [None if l.mlp is None else st.Gate(l.mlp.act, l.mlp.limit) for l in specs]
+                self.mixers.append(mixer_class(l.mixer)(l.mixer, self.dtype, self.device))
+        gate = lambda f: None if f is None else st.Gate(f.act, f.limit)
+        self.gates = [gate(l.mlp) for l in specs]
+        self.shared_gates = [gate(l.mlp and l.mlp.shared) for l in specs]
         self.runs = self.cfg.layer_runs
         # run whose cache a run reads (its own but for shared latents, which no loop contains)
-        run_of = {l: r for r, (l, _) in enumerate(self.runs)}
+        run_of = {l: r for r, (l, _) in enumerate(self.runs) if source[l] is None}
         self.owners = [r if source[l] is None else run_of[source[l]]
                        for r, (l, _) in enumerate(self.runs)]
         self._cache_rows = [self.mixers[l].cache_rows for l, _ in self.runs]
+        self._state_rows = [self.mixers[l].state_rows for l, _ in self.runs]
+        self.has_state = any(self._state_rows)
         # queries per sequence from which expanding its context costs fewer multiply-adds than
         # attending in latent space, for the layers together
         exp = [self.mixers[l] for l, _ in self.runs if self.mixers[l].expand]
@@ -161,7 +196,9 @@ class LayerListForCausalLM:
         V, W = cfg.vocab_size, cfg.hidden_size
         pending: dict = {}
         need = [set(required_tensors(cfg, l)) for l in cfg.layer_specs]
-        top = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+        top = {"embed": (V, W), "final.norm": (W,)}
+        if not cfg.tie_word_embeddings:
+            top["head"] = (V, W)
         if cfg.loop is not None:
             top["loop.step"] = (cfg.loop.times, W)
         missing = set(top)
@@ -169,14 +206,17 @@ class LayerListForCausalLM:
             if name in top:
                 t = Checkpoint({name: t}, self.dtype, self.device).take(name, *top[name])
                 missing.discard(name)
-                if name == "embed":
+                rows = round_up(V, 8) if self.dtype == torch.bfloat16 else V
+                if name == "embed" and cfg.tie_word_embeddings:
+                    self.embed = self.lm_head = padded(t, rows)
+                elif name == "embed":
                     self.embed = t
                 elif name == "final.norm":
                     self.norm = t.float()
                 elif name == "loop.step":
                     self.loop_step = t.float()
                 else:
-                    self.lm_head = padded(t, round_up(V, 8) if self.dtype == torch.bfloat16 else V)
+                    self.lm_head = padded(t, rows)
                 continue
             m = _NAME_RE.match(name)
             if m is None or int(m.group(1)) >= len(need) or m.group(2) not in need[int(m.group(1))]:
@@ -189,7 +229,7 @@ class LayerListForCausalLM:
                 self.layers[l] = self._pack(l, d)
                 del pending[l]
         missing = sorted(missing)
-        missing += ["l%d.%s" % (l, n) for l, lw in enumerate(self.layers) if lw is None
+        missing += ["l%d.%s" % (l, n) for l, lw in enumerate(self.layers) if lw is None and need[l]
                     for n in sorted(need[l] - set(pending.get(l, ())))]
         if missing:
             raise ValueError("checkpoint is incomplete: %s" % missing[:8])
@@ -199,13 +239,24 @@ class LayerListForCausalLM:
         f = spec.mlp
         c, lw = Checkpoint(t, self.dtype, self.device), LayerWeights()
         self.mixers[l].pack(c, lw, W)
+        scales = dict(zip(("norm1", "norm2"), scale_names(self.cfg, spec)))
         for n in norm_names(self.cfg, spec):
-            lw.put(**{n: c.vector(n, W)})
+            v = c.vector(n, W)
+            if n in scales:      # norm and layer scale are factors of the same vector
+                v = v * c.vector(scales[n], W)
+            lw.put(**{n: v})
         if f is None:
             return lw
+        if f.shared is not None:
+            ff = f.shared.ff
+            gate, up = (c.take("mlp.shared." + n, ff, W) for n in ("gate", "up"))
+            down = c.take("mlp.shared.down", W, ff)
+            lw.put(shared_gu=st.interleave_gate_up(gate, up),
+                   shared_down=padded(down, W, round_up(ff, st.GATE_BLOCK)).contiguous())
         if f.experts:
-            lw.put(router=c.take("mlp.router", f.experts, W),
-                   router_b=c.vector("mlp.router.b", f.experts))
+            outputs = f.experts + f.identity
+            lw.put(router=c.take("mlp.router", outputs, W),
+                   router_b=c.vector(router_vector(f), outputs))
             stack = lambda n, *s: torch.stack(
                 [c.take("mlp.e%d.%s" % (e, n), *s) for e in range(f.experts)])
             gate, up, down = stack("gate", f.ff, W), stack("up", f.ff, W), stack("down", W, f.ff)
@@ -239,10 +290,14 @@ class LayerListForCausalLM:
         return RunCacheTensors.bytes_per_block(self.owners, self._cache_rows, block_size,
                                                self.dtype.itemsize)
 
-    def new_kv_cache(self, num_blocks: int, block_size: int):
+    def state_bytes_per_slot(self) -> int:
+        from ..engine.kv_cache import RunCacheTensors
+        return RunCacheTensors.bytes_per_slot(self._state_rows)
+
+    def new_kv_cache(self, num_blocks: int, block_size: int, num_slots: int = 0):
         from ..engine.kv_cache import RunCacheTensors
         return RunCacheTensors(self.owners, self._cache_rows, num_blocks, block_size, self.dtype,
-                               self.device)
+                               self.device, self._state_rows, num_slots)
 
     def _expanded(self, q_lens, kv_lens) -> list:
         """Which sequences of a step go through expanded keys and values."""
@@ -297,10 +352,10 @@ class LayerListForCausalLM:
 
     def decode_plans(self, bucket: int, max_q: int, block_size: int) -> list:
         return [m.decode_plan(bucket, max_q, block_size)
-                for m in {m.shape: m for m in self.mixers}.values()]
+                for m in {m.shape: m for m in self.mixers if m.shape is not None}.values()]
 
     def decode_attention(self, plans: list, block_tables):
-        step = lat.AttentionStep(plans[0].bucket)
+        step = lat.AttentionStep(block_tables.shape[0])
         for p in plans:
             if isinstance(p, lat.LatentDecodePlan):
                 step.absorbed[(p.shape, True)] = p.meta
@@ -314,7 +369,8 @@ class LayerListForCausalLM:
         lw, f, gate = self.layers[l], self.cfg.layer_specs[l].mlp, self.gates[l]
         if not f.experts:
             return ops.linear(st.gated_linear(act, lw.w_gu, gate), lw.w_down), None
-        routing, rows = st.route(x, act, lw.router, lw.router_b, f.top)
+        routing, rows = st.route(x, act, lw.router, lw.router_b, f.top, f.identity,
+                                 f.router_scale if f.scoring == "all" else None)
         h = st.grouped_linear(rows, lw.w_gu, routing, act=gate)
         return st.grouped_linear(h, lw.w_down, routing), routing
 
@@ -323,9 +379,10 @@ class LayerListForCausalLM:
         residual stream after every run."""
         shared: dict = {}
         step, eps = batch.attn_meta, self.cfg.rms_norm_eps
-        mix = lambda r, l, act: self.mixers[l].run(act, self.layers[l], batch, kv.of(r), step,
-                                                   shared, eps)
-        body = self._post_norm_body if self.design.residual == "post" else self._sandwich_body
+        mix = lambda r, l, act: self.mixers[l].run(act, self.layers[l], batch, kv.of(r),
+                                                   kv.state_of(r), step, shared, eps)
+        body = {"post": self._post_norm_body, "sandwich": self._sandwich_body,
+                "output": self._output_norm_body}[self.design.residual]
         x = body(batch, mix, layers_out)
         return st.stream_final_norm(x, batch.logits_indices, self.norm, eps, self.dtype,
                                     self.design.norm_offset)
@@ -371,6 +428,25 @@ class LayerListForCausalLM:
                 layers_out.append(x.clone())
                 y = w_out = None
             enter(r + 1, y, w_out)
+        return x
+
+    def _output_norm_body(self, batch, mix, layers_out):
+        eps = self.cfg.rms_norm_eps
+        x, act = st.stream_embedding(batch.input_ids, self.embed, self.cfg.embedding_scale)
+        for r, (l, _) in enumerate(self.runs):
+            lw = self.layers[l]
+            y = mix(r, l, act)
+            y, pair = y if isinstance(y, tuple) else (y, None)
+            st.stream_add(x, act, lw.norm1, eps, y, pair=pair)
+            if self.cfg.layer_specs[l].mlp is not None:
+                y, routing = self._feed_forward(l, x, act)
+                shared = None
+                if self.shared_gates[l] is not None:
+                    shared = ops.linear(st.gated_linear(act, lw.shared_gu, self.shared_gates[l]),
+                                        lw.shared_down)
+                st.stream_add(x, act, lw.norm2, eps, y, experts=routing, shared=shared)
+            if layers_out is not None:
+                layers_out.append(x.clone())
         return x
 
     def compute_logits(self, hidden: torch.Tensor, fp32: bool = False) -> torch.Tensor:

@@ -292,6 +292,8 @@ class ForwardBatch:
     # SwiftKV: metadata / positions of the sampled rows only
     sel_attn_meta: object = None
     sel_positions: Optional[torch.Tensor] = None
+    # models with recurrent layers: the step's sequences and their state slots (ops.state_ops)
+    state: object = None
     # the first ``num_sampled`` selected rows are sampled; further rows are prompt positions
     # whose log-probabilities were asked for: (request, first position, count) per span and
     # the token that follows each such position

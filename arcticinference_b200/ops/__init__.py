@@ -1061,10 +1061,11 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
 
 def attention_masked(q, k, v, meta: AttentionMetadata, Hq: int, Hkv: int, D: int, scale: float, mask,
                      sink=None, gate=None, out=None, paged: bool = True,
-                     Dk: int | None = None) -> torch.Tensor:
+                     Dk: int | None = None, softcap: float = 0.0) -> torch.Tensor:
     """Causal attention with a lower bound on the keys (``mask``, a MaskSpec), an optional sink
-    (fp32 [Hq]: a further term of the softmax denominator) and an optional output gate (rows
-    [T, Hq * D]; the output is multiplied by their sigmoid). CUDA tensors only. Keys and values:
+    (fp32 [Hq]: a further term of the softmax denominator), an optional output gate (rows
+    [T, Hq * D]; the output is multiplied by their sigmoid) and, with ``softcap`` > 0, scores
+    softcap * tanh(score / softcap). CUDA tensors only. Keys and values:
     caches [num_blocks, Hkv, block_size, D], or with ``paged`` false rows [n, Hkv * D] (of queries
     and keys Hkv * Dk, where given: 192 with D = 128). ``meta`` must have been planned with the
     same mask."""
@@ -1083,8 +1084,8 @@ def attention_masked(q, k, v, meta: AttentionMetadata, Hq: int, Hkv: int, D: int
         k.shape[0], k.shape[2] if paged else 0, nat.ptr(bt), bt.shape[1] if paged else 0,
         meta.work.data_ptr(), meta.num_work, nat.ptr(meta.tok_splits) if meta.max_splits > 1 else None,
         meta.max_splits, T, Hq, Hkv, Dk or D, D, mask.code, mask.size, nat.ptr(sink), nat.ptr(gate),
-        gate.stride(0) if gate is not None else 0, float(scale), out.data_ptr(), out.stride(0),
-        nat.ptr(meta.o_part), nat.ptr(meta.lse_part), meta.tile_keys if paged else 128,
+        gate.stride(0) if gate is not None else 0, float(scale), float(softcap), out.data_ptr(),
+        out.stride(0), nat.ptr(meta.o_part), nat.ptr(meta.lse_part), meta.tile_keys if paged else 128,
         nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "attention_masked")
     launch_counter.add(2 if meta.max_splits > 1 else 1)

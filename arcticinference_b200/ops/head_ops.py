@@ -1,6 +1,6 @@
-"""Attention over cached keys and values with what a layer may ask beyond the plain form: per-head
-query / key norms, partial rotary positions, a mask with a lower bound (window or chunks), a learned
-sink per head and an output gate.
+"""Attention over cached keys and values with what a layer may ask beyond the plain form: query / key
+norms (per head or over the whole projection), partial rotary positions, keys that are the values too,
+a mask with a lower bound (window or chunks), softly capped scores, a sink per head and an output gate.
 
 CUDA tensors run ``csrc/rotary.cu`` and ``csrc/attention.cu`` or, for 32-bit models and heads wider
 than the tensor-core kernel's, ``csrc/exact.cu``. CPU tensors run the restatements below.
@@ -96,16 +96,24 @@ def rotate_ref(x, table):
 
 
 def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, table, eps: float, slots, k_cache,
-                    v_cache) -> None:
+                    v_cache, whole: bool = False, shared_kv: bool = False) -> None:
     """``proj`` [T, ...] holds the query heads, key heads (``D`` columns each, ``dim`` in use) and
     value heads (``Dv``). RMS norm of every query and key head over its ``dim`` columns with the
     weights ``wq`` / ``wk`` (fp32 [D], or None), rotation by ``table`` (rotary_table), queries in
-    place, keys and values to the rows ``slots`` of the caches; slot < 0: no write."""
+    place, keys and values to the rows ``slots`` of the caches; slot < 0: no write. ``whole``: the
+    norm is over all query (key) heads of a token at once, weights fp32 [heads * D]. ``shared_kv``:
+    there are no value heads; the keys before norm and rotation are the values."""
     H, G, D, Dv = shape.heads, shape.kv_heads, shape.D, shape.Dv
     T, bs = proj.shape[0], k_cache.shape[2]
     if not proj.is_cuda:
         x = proj[:, :(H + G) * D].reshape(T, H + G, D).float()
-        if wq is not None:
+        raw = proj[:, H * D:(H + G) * D].clone()
+        if whole:
+            for a, n, w in ((0, H, wq), (H, G, wk)):
+                y = x[:, a:a + n]
+                ss = y.pow(2).sum((1, 2), keepdim=True) / (n * dim)
+                x[:, a:a + n] = y / torch.sqrt(ss + eps) * w.view(n, D)
+        elif wq is not None:
             w = torch.cat([wq.expand(H, D), wk.expand(G, D)])
             x = x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) / dim + eps) * w
         x = rotate_ref(x, table).to(proj.dtype)
@@ -113,7 +121,8 @@ def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, table, eps: float,
         ok = slots >= 0
         blk, off = slots[ok] // bs, slots[ok] % bs
         k_cache[blk, :, off] = x[ok, H:]
-        v_cache[blk, :, off] = proj[ok, (H + G) * D:(H + G) * D + G * Dv].reshape(-1, G, Dv)
+        v = raw if shared_kv else proj[:, (H + G) * D:(H + G) * D + G * Dv]
+        v_cache[blk, :, off] = v[ok].reshape(-1, G, Dv)
         return
     nat = _nat()
     assert proj.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
@@ -121,14 +130,15 @@ def head_rope_cache(proj, shape: HeadShape, dim: int, wq, wk, table, eps: float,
     rc = nat.lib().ab200_head_rope_cache(
         proj.data_ptr(), proj.stride(0), table.data_ptr(), table.shape[1], slots.data_ptr(),
         nat.ptr(wq), nat.ptr(wk), k_cache.data_ptr(), v_cache.data_ptr(), T, H, G, D, dim, Dv, bs,
-        k_cache.shape[0] * bs, float(eps), dtype_code(proj.dtype),
+        k_cache.shape[0] * bs, float(eps), int(whole), int(shared_kv), dtype_code(proj.dtype),
         nat.status_buffer(proj.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "head_rope_cache")
     launch_counter.add(1)
 
 
 def attention_exact(q, k_cache, v_cache, block_tables, tok_seq, positions, H: int, Hkv: int, Dk: int,
-                    Dv: int, scale: float, mask: MaskSpec, sink=None, gate=None) -> torch.Tensor:
+                    Dv: int, scale: float, mask: MaskSpec, sink=None, gate=None,
+                    softcap: float = 0.0) -> torch.Tensor:
     """fp32-accumulating attention without tensor cores; q [T, H * Dk], caches [num_blocks, Hkv,
     block_size, >= Dk / Dv] (they may be one tensor). Returns [T, H * Dv]."""
     nat = _nat()
@@ -140,14 +150,14 @@ def attention_exact(q, k_cache, v_cache, block_tables, tok_seq, positions, H: in
         v_cache.shape[3], k_cache.shape[0], k_cache.shape[2], block_tables.data_ptr(),
         block_tables.shape[1], tok_seq.data_ptr(), positions.data_ptr(), nat.ptr(sink),
         nat.ptr(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), T, H,
-        Hkv, Dk, Dv, mask.code, mask.size, float(scale), dtype_code(q.dtype),
+        Hkv, Dk, Dv, mask.code, mask.size, float(scale), float(softcap), dtype_code(q.dtype),
         nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "attention_exact")
     launch_counter.add(1)
     return out
 
 
-def head_attention_ref(q, k_cache, v_cache, meta, shape: HeadShape, scale, sink, gate):
+def head_attention_ref(q, k_cache, v_cache, meta, shape: HeadShape, scale, sink, gate, softcap=0.0):
     H, G, D, Dv = shape.heads, shape.kv_heads, shape.D, shape.Dv
     bs = k_cache.shape[2]
     out = torch.empty(q.shape[0], H * Dv, dtype=q.dtype)
@@ -161,6 +171,8 @@ def head_attention_ref(q, k_cache, v_cache, meta, shape: HeadShape, scale, sink,
         k, v = (c[blk, :, pos % bs].float().repeat_interleave(H // G, 1)
                 for c in (k_cache, v_cache))
         s = torch.einsum("thd,khd->htk", q[t:t + n].reshape(n, H, D).float(), k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         at = torch.arange(kl - n, kl).view(n, 1)
         s = s.masked_fill((pos > at) | (pos < shape.mask.first_key(at)), float("-inf"))
         if sink is not None:
@@ -174,15 +186,16 @@ def head_attention_ref(q, k_cache, v_cache, meta, shape: HeadShape, scale, sink,
 
 
 def head_attention(q, k_cache, v_cache, meta: AttentionMetadata, shape: HeadShape, scale: float,
-                   sink=None, gate=None, tok_seq=None, positions=None) -> torch.Tensor:
+                   sink=None, gate=None, tok_seq=None, positions=None,
+                   softcap: float = 0.0) -> torch.Tensor:
     """q [T, heads * D] (row stride free); caches [num_blocks, kv_heads, block_size, D / Dv]; ``sink``
-    fp32 [heads] and ``gate`` [T, heads * Dv] (row stride free) may be None. Returns
-    [T, heads * Dv]. ``tok_seq`` and ``positions`` (per token) are read by the "exact" kernel only."""
+    fp32 [heads] and ``gate`` [T, heads * Dv] (row stride free) may be None; ``softcap`` > 0 caps the
+    scores. Returns [T, heads * Dv]. ``tok_seq`` and ``positions`` (per token) are read by the "exact" kernel only."""
     if not q.is_cuda:
-        return head_attention_ref(q, k_cache, v_cache, meta, shape, scale, sink, gate)
+        return head_attention_ref(q, k_cache, v_cache, meta, shape, scale, sink, gate, softcap)
     if shape.kernel == "exact":
         return attention_exact(q, k_cache, v_cache, meta.block_tables, tok_seq, positions,
                                shape.heads, shape.kv_heads, shape.D, shape.Dv, scale, shape.mask,
-                               sink, gate)
+                               sink, gate, softcap)
     return attention_masked(q, k_cache, v_cache, meta, shape.heads, shape.kv_heads, shape.D, scale,
-                            shape.mask, sink, gate)
+                            shape.mask, sink, gate, softcap=softcap)

@@ -140,6 +140,45 @@ def stream_sandwich(x, y=None, w_out=None, step=None, w_in=None, act=None, eps: 
     launch_counter.add(1)
 
 
+def stream_add(x, act, w, eps: float, y=None, pair=None, experts: "Routing" = None,
+               shared=None) -> None:
+    """In place: ``x += norm(f) * w``, ``act`` (where it is not x itself) its rounding. f is a
+    sublayer's output ``y``; with ``pair`` = (y2, wy, wy2) half the sum of norm(y) * wy and
+    norm(y2) * wy2; with ``experts`` (``y``: the experts' rows) each token's weighted sum, in which an
+    identity expert contributes the token's x, plus the rows of ``shared``."""
+    T, W = x.shape
+    if not x.is_cuda:
+        f = y.float()
+        if pair is not None:
+            f = 0.5 * (_scaled_norm_ref(f, pair[1], eps, 0.0) +
+                       _scaled_norm_ref(pair[0].float(), pair[2], eps, 0.0))
+        elif experts is not None:
+            own = experts.rows < 0
+            rows = torch.cat([f, torch.zeros(1, W)])[experts.rows.long()]     # (-1: the zero row)
+            rows = torch.where(own.unsqueeze(-1), x.unsqueeze(1), rows)
+            f = (rows * experts.weights.unsqueeze(-1)).sum(1)
+            if shared is not None:
+                f = f + shared.float()
+        x += _scaled_norm_ref(f, w, eps, 0.0)
+        if act is not x:
+            act.copy_(x)
+        return
+    nat = _nat()
+    y2, wy, wy2 = pair or (None, None, None)
+    assert x.is_contiguous() and act.is_contiguous()
+    assert all(t is None or (t.stride(1) == 1 and t.dtype == act.dtype) for t in (y, y2, shared))
+    rc = nat.lib().ab200_stream_add(
+        x.data_ptr(), None if act is x else act.data_ptr(), w.data_ptr(), y.data_ptr(), y.stride(0),
+        nat.ptr(wy), nat.ptr(y2), y2.stride(0) if y2 is not None else 0, nat.ptr(wy2),
+        experts.rows.data_ptr() if experts is not None else None,
+        experts.weights.data_ptr() if experts is not None else None,
+        experts.top if experts is not None else 0, nat.ptr(shared),
+        shared.stride(0) if shared is not None else 0, float(eps), T, W, dtype_code(act.dtype),
+        nat.stream_ptr())
+    nat.check(rc, "stream_add")
+    launch_counter.add(1)
+
+
 def stream_final_norm(x, rows, weight, eps: float, dtype: torch.dtype,
                       offset: float = 1.0) -> torch.Tensor:
     """norm(x[rows]) * (offset + weight), rounded to ``dtype``: the state the LM head reads."""
@@ -197,9 +236,9 @@ def gated_act(gu: torch.Tensor, act) -> torch.Tensor:
 @dataclass
 class Routing:
     """Which experts each token uses and where its rows lie among the rows sorted by expert."""
-    ids: torch.Tensor         # int32 [T, top]
+    ids: torch.Tensor         # int32 [T, top]; from num_experts on: identity experts
     weights: torch.Tensor     # fp32 [T, top]
-    rows: torch.Tensor        # int32 [T, top]
+    rows: torch.Tensor        # int32 [T, top]; -1 for an identity expert
     top: int
     num_experts: int
     tiles: torch.Tensor = None        # int32 [max_tiles, 4]: expert, first row, rows
@@ -207,8 +246,13 @@ class Routing:
     counts: list = None               # CPU path: rows per expert
 
 
-def route_ref(x, w, b, top: int):
-    z = x.float() @ w.float().t() + b
+def route_ref(x, w, b, top: int, scale=None):
+    z = x.float() @ w.float().t()
+    if scale is not None:      # softmax over all outputs, b: correction of the choice
+        s = torch.softmax(z, -1)
+        order = torch.argsort(s if b is None else s + b, dim=-1, descending=True, stable=True)[:, :top]
+        return order, s.gather(1, order) * scale
+    z = z + b
     order = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :top]
     return order, torch.softmax(z.gather(1, order), -1)
 
@@ -226,19 +270,24 @@ def _route_state(E: int, device) -> torch.Tensor:
     return t
 
 
-def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, top: int):
+def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, top: int,
+          identity: int = 0, scale: float = None):
     """Router of a mixture of experts. ``x`` fp32 [T, W] stream, ``act`` its rounding (what the
-    experts read), ``w`` [E, W], ``b`` fp32 [E]. Returns (Routing, act rows sorted by expert)."""
+    experts read), ``w`` [outputs, W], ``b`` fp32 [outputs] or None. The weights are the softmax over
+    the chosen logits (with the bias ``b``) or, with a ``scale``, the chosen ones of the softmax over
+    all outputs times it (``b`` then corrects the choice only). The last ``identity`` outputs are
+    identity experts. Returns (Routing, act rows sorted by expert)."""
     T, W = x.shape
-    E = w.shape[0]
+    E = w.shape[0] - identity
     if not x.is_cuda:
-        ids, weights = route_ref(x, w, b, top)
+        ids, weights = route_ref(x, w, b, top, scale)
         order = torch.argsort(ids.reshape(-1), stable=True)
         rows = torch.empty_like(order)
         rows[order] = torch.arange(order.numel())
-        counts = torch.bincount(ids.reshape(-1), minlength=E).tolist()
-        r = Routing(ids.int(), weights, rows.reshape(T, top).int(), top, E, counts=counts)
-        return r, act[order // top]
+        counts = torch.bincount(ids.reshape(-1), minlength=E)[:E].tolist()
+        rows = torch.where(ids < E, rows.reshape(T, top), -1).int()
+        r = Routing(ids.int(), weights, rows, top, E, counts=counts)
+        return r, act[order[:sum(counts)] // top]
     nat = _nat()
     L, dev, dc = nat.lib(), x.device, dtype_code(act.dtype)
     assert x.is_contiguous() and act.is_contiguous() and w.is_contiguous() and w.dtype == act.dtype
@@ -251,9 +300,10 @@ def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, 
     num_tiles = plan[4 * max_tiles:4 * max_tiles + 1]
     cursor = plan[4 * max_tiles + 4:4 * max_tiles + 4 + E]
     rows = plan[4 * max_tiles + 4 + E:].view(T, top)
-    rc = L.ab200_moe_route(x.data_ptr(), w.data_ptr(), b.data_ptr(), T, W, E, top, ids.data_ptr(),
-                           weights.data_ptr(), _route_state(E, dev).data_ptr(), cursor.data_ptr(),
-                           tiles.data_ptr(), num_tiles.data_ptr(), dc, nat.stream_ptr())
+    rc = L.ab200_moe_route(x.data_ptr(), w.data_ptr(), nat.ptr(b), T, W, E + identity, E, top,
+                           int(scale is not None), scale or 0.0, ids.data_ptr(), weights.data_ptr(),
+                           _route_state(E, dev).data_ptr(), cursor.data_ptr(), tiles.data_ptr(),
+                           num_tiles.data_ptr(), dc, nat.stream_ptr())
     nat.check(rc, "moe_route")
     launch_counter.add(1)
     r = Routing(ids, weights, rows, top, E, tiles, num_tiles)
@@ -265,7 +315,7 @@ def _permute(act, r: Routing, cursor) -> torch.Tensor:
     T, W = act.shape
     xp = torch.empty(T * r.top, W, dtype=act.dtype, device=act.device)
     rc = nat.lib().ab200_moe_permute(act.data_ptr(), r.ids.data_ptr(), cursor.data_ptr(),
-                                     r.rows.data_ptr(), xp.data_ptr(), T, W, r.top,
+                                     r.rows.data_ptr(), xp.data_ptr(), T, W, r.top, r.num_experts,
                                      dtype_code(act.dtype), nat.stream_ptr())
     nat.check(rc, "moe_permute")
     launch_counter.add(1)

@@ -79,6 +79,10 @@ def _ensure_registered() -> None:
     register_config("zatirax", "layer list: windowed latent attention with rotary keys, chunked "
                                "attention with sinks and output gates, a loop over layers")
     register_model("Zatirax", _layer_list)
+    register_config("pererax", "layer list: gated delta rule, attention beside a matrix memory, "
+                               "windowed attention; experts with identity and shared ones; layers "
+                               "that use others' weights")
+    register_model("Pererax", _layer_list)
     for arch in ("ArcticMLPSpeculatorPreTrainedModel", "ArcticLSTMSpeculatorPreTrainedModel",
                  "MLPVariantSpeculatorPreTrainedModel", "MLPSpeculatorPreTrainedModel"):
         register_model(arch, _speculator)
