@@ -289,20 +289,23 @@ int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, 
                       long long T, int W, int top, int experts, int dtype, cudaStream_t stream);
 
 // ---- recurrent.cu
-int ab200_scan_min_slices(int dim, int ncols);
+int ab200_scan_min_slices(int dim, int ncols, int delta);
+long long ab200_scan_record(int dim, int ncols, int slices, int delta);
 int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int b_at,
                      const void* decay, long long ld_decay, const void* gate, long long ld_gate,
                      const void* conv, int taps, const void* a_exp, const void* dt_bias,
                      const void* norm, void* state, int state_cols, void* conv_state, int num_slots,
-                     const void* steps, int n_seq, int max_rows, long long T, int heads, int kv_heads,
-                     int dim, int vdim, int slices, float eps, void* raw, void* out, long long ldo,
-                     int dtype, int* status, cudaStream_t stream);
+                     const void* steps, int n_seq, int max_rows, const void* tiles,
+                     const void* first_tile, int n_tiles, void* records, long long T, int heads,
+                     int kv_heads, int dim, int vdim, int slices, float eps, void* raw, void* out,
+                     long long ldo, int dtype, int* status, cudaStream_t stream);
 int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int i_at, int f_at,
                       const void* gate, long long ld_gate, const void* i_bias, const void* f_bias,
                       float cap, const void* norm, void* state, int state_cols, void* max_state,
-                      int num_slots, const void* steps, int n_seq, int max_rows, long long T, int heads,
-                      int dim, int vdim, int slices, float eps, void* raw, void* out, long long ldo,
-                      int dtype, int* status, cudaStream_t stream);
+                      int num_slots, const void* steps, int n_seq, int max_rows, const void* tiles,
+                      const void* first_tile, int n_tiles, void* records, void* gates, long long T,
+                      int heads, int dim, int vdim, int slices, float eps, void* raw, void* out,
+                      long long ldo, int dtype, int* status, cudaStream_t stream);
 
 // ---- grouped_gemm.cu
 int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long long x_rows,

@@ -11,19 +11,20 @@
 // Both are followed by the RMS norm of each head's o, a weight and an output gate. Everything that
 // enters the recurrence is fp32, and so is its arithmetic (FMAs on pairs of rows).
 //
-// A block owns a sequence's head, or some of the head's columns, which do not depend on one another,
-// and keeps its part of S in registers for all of the sequence's tokens in this step: a lane holds
-// DP / 8 rows by kCols columns. Tokens come in tiles. Per tile the block first prepares the vectors
-// the recurrence needs in shared memory (convolution, norms, gates, decays), then runs the
-// recurrence B tokens at a time, then writes the tile's normed and gated outputs.
+// Steps of one token per sequence run in one kernel (step_kernel): a block owns a sequence's head, or
+// some of the head's columns, which do not depend on one another.
 //
+// Longer portions take two. tile_kernel prepares, for tiles of 16 tokens and all of them at once, the
+// vectors that the recurrence needs (convolution, norms, gates, decays) as records in memory;
+// scan_kernel then walks a sequence's records with a head's part of S in registers (a lane holds DP / 8
+// rows by kCols columns), four tokens at a time, the next records on their way to shared memory.
 // Within a tile S is held undecayed: S = G * Z with G the product of the tile's decays so far (per
 // row), so that a token costs three multiply-adds per element and not four,
 //     Z^T (G k), Z^T (G q) and Z <- Z + (k / G) u^T,
-// and B tokens need no exchange but their scalar products: with a = G k, b = k / G, c = G q
+// and a group of tokens needs no exchange but its scalar products: with a = G k, b = k / G, c = G q
 //     u_i = beta_i (v_i - Z^T a_i - sum_{j<i} (a_i . b_j) u_j),  o_i = Z^T c_i + sum_{j<=i} (c_i . b_j) u_j
-// where Z is the one before the first of them. G goes back to 1 at a tile's end, and after every B
-// tokens when a channel decays so much within the tile that 1 / G would leave fp32's range.
+// where Z is the one before the group. G goes back to 1 at a tile's end, and after every group when a
+// channel decays so much within the tile that 1 / G would leave fp32's range.
 //
 // What a sequence carries over lies in its slot: S in fp32; the convolution's last inputs and m twice,
 // for even and odd steps of the sequence (`phase`), so that blocks which read them never race with the
@@ -35,7 +36,11 @@
 
 namespace ab200 {
 
-constexpr int kScanMaxWarps = 10;
+// warps of a block: 128 columns of wide states, and the normaliser's beside them
+__host__ __device__ constexpr int max_warps(bool delta) { return delta ? 8 : 9; }
+
+constexpr int kTT = 16, kB = 4;           // tokens per tile and per group
+constexpr int kTaps = 4;                  // convolutions of up to this many taps stay in registers
 constexpr float kMinLogDecay = -20.f;     // per token: a factor below 2e-9 is as good as that
 constexpr float kTileLogDecay = -60.f;    // a tile whose decays multiply to less is cut
 constexpr int kStepInts = 5;              // first row, rows, slot, start position, phase
@@ -62,6 +67,11 @@ struct ScanArgs {
   void* conv_state;          // delta: [slots][2][taps - 1][channels] (element type T)
   float* max_state;          // memory: [slots][2][heads]
   const int* steps;          // [n][kStepInts]
+  const int* tiles;          // [n_tiles][2]: sequence, its first token of the tile; in order
+  const int* first_tile;     // [n]
+  float* gates;              // memory: [T][heads][3]: log decay, log input factor, m
+  float* records;            // [n_tiles][heads][record]
+  long long record;          // floats
   void* out;                 // [T][ldo], head h at column h * vdim (one block per head) ...
   long long ldo;
   float* raw;                // ... or [T][heads][raw_cols] unnormed, for scan_output
@@ -69,10 +79,12 @@ struct ScanArgs {
   int num_slots, heads, group, dim, vdim, ncols, taps, channels;
   int slices, nc;            // blocks per head, columns of each
   int vec;                   // four channels at a time are aligned
+  int vec_out;               // eight output columns at a time are aligned, a power of two of them
   float q_scale, cap, eps;
   int* status;
 };
 
+// Packed fp32 pairs
 __device__ __forceinline__ void fma2(float2& d, const float2& a, const float2& b) {
   asm("fma.rn.f32x2 %0, %1, %2, %0;"
       : "+l"(reinterpret_cast<unsigned long long&>(d))
@@ -84,14 +96,42 @@ __device__ __forceinline__ void mul2(float2& d, const float2& a) {
       : "+l"(reinterpret_cast<unsigned long long&>(d))
       : "l"(reinterpret_cast<const unsigned long long&>(a)));
 }
-
-__device__ __forceinline__ float softplus_f(float z) {
-  return fmaxf(z, 0.f) + log1pf(__expf(-fabsf(z)));
+__device__ __forceinline__ void copy16_async(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
-__device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.f + __expf(-z)); }
-__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void copies_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
 
-// DP: rows (dim, zero-padded); B tokens at a time, TT per tile
+// log(1 + e^z); log1p's first terms where the fast logarithm would lose them
+__device__ __forceinline__ float softplus_f(float z) {
+  const float e = __expf(-fabsf(z));
+  const float l = e < 0.03f ? e * (1.f + e * (-0.5f + e * (0.33333333f - 0.25f * e))) : __logf(1.f + e);
+  return fmaxf(z, 0.f) + l;
+}
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
+__device__ __forceinline__ float4 silu4(const float4& y) {
+  return make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w));
+}
+__device__ __forceinline__ void axpy4(float4& y, const float4& w, const float4& v) {
+  y.x = fmaf(w.x, v.x, y.x);
+  y.y = fmaf(w.y, v.y, y.y);
+  y.z = fmaf(w.z, v.z, y.z);
+  y.w = fmaf(w.w, v.w, y.w);
+}
+__device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
+  return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
+}
+// log gates of the matrix memory
+__device__ __forceinline__ float2 memory_log_gates(float zi, float zf, float cap) {
+  const float z = cap * tanhf(zf / cap);
+  return make_float2(cap * tanhf(zi / cap), fminf(z, 0.f) - log1pf(expf(-fabsf(z))));
+}
+
+// DP: rows (dim, zero-padded)
 template <int DP>
 struct ScanShape {
   static constexpr int kRows = DP / 8;                  // per lane, in chunks of four
@@ -99,77 +139,96 @@ struct ScanShape {
   static constexpr int kWarpCols = 4 * kCols;
 };
 
-template <int DP, int TT, int B, bool DELTA>
-struct ScanSmem {   // offsets in floats
-  static constexpr int kB = 0, kC = kB + TT * DP, kA = kC + TT * DP, kG = kA + (DELTA ? TT * DP : 0);
-  static constexpr int kDotB = kG + TT / B * DP, kDotC = kDotB + TT * B, kBeta = kDotC + TT * B;
-  static constexpr int kInvQ = kBeta + TT, kInvK = kInvQ + TT, kMax = kInvK + TT, kV = (kMax + TT + 2 + 3) / 4 * 4;
-  static constexpr int total(int nc) { return kV + TT * nc; }
+// A record: offsets in floats. Its values [kTT][value columns] follow.
+template <int DP, bool DELTA>
+struct Record {
+  static constexpr int kKeys = 0, kQ = kTT * DP, kA = 2 * kTT * DP, kG = (DELTA ? 3 : 2) * kTT * DP;
+  static constexpr int kDotB = kG + kTT / kB * DP, kDotC = kDotB + kTT * kB;
+  static constexpr int kBeta = kDotC + kTT * kB;    // memory: exp(-m)
+  static constexpr int kStrong = kBeta + kTT, kV = kStrong + 4;
 };
 
-template <typename T, int DP, int TT, int B, bool DELTA>
-__global__ void __launch_bounds__(kScanMaxWarps * 32, 1) scan_kernel(const ScanArgs p) {
-  using Sh = ScanShape<DP>;
-  using Sm = ScanSmem<DP, TT, B, DELTA>;
-  constexpr int kRows = Sh::kRows, kCols = Sh::kCols, kChunks = kRows / 4;
-  extern __shared__ __align__(16) float sm[];
-  float* sB = sm + Sm::kB;       // keys, then k / G
-  float* sC = sm + Sm::kC;       // queries, then G q
-  float* sA = sm + Sm::kA;       // G k
-  float* sG = sm + Sm::kG;
-  float* dotB = sm + Sm::kDotB;  // [token][earlier token of its group]: a . b
-  float* dotC = sm + Sm::kDotC;  // c . b
-  float* sBeta = sm + Sm::kBeta; // delta: step size; memory: log of the input factor
-  float* invQ = sm + Sm::kInvQ;  // memory: cumulative log decay
-  float* invK = sm + Sm::kInvK;
-  float* sMax = sm + Sm::kMax;   // memory: m per token; [TT]: m carried over, [TT + 1]: flag
-  float* sV = sm + Sm::kV;       // values, then outputs [TT][nc]
-  pdl_wait();
-  pdl_trigger();
+// A sequence of a step and a head of it
+struct Seq {
+  long long first;
+  int n, slot, start, phase;
+  __device__ __forceinline__ explicit Seq(const int* s)
+      : first(s[0]), n(s[1]), slot(s[2]), start(s[3]), phase(s[4] & 1) {}
+};
 
-  const int slice = blockIdx.x % p.slices;
-  const int h = blockIdx.x / p.slices % p.heads;
-  const int* step = p.steps + (long long)(blockIdx.x / p.slices / p.heads) * kStepInts;
-  const long long first = step[0];
-  const int n = step[1], slot = step[2], start = step[3], phase = step[4] & 1;
-  if (n <= 0) return;
-  const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31;
-  const int warps = threads >> 5;
-  const int nc = p.nc, c_first = slice * nc;
-  const int hv = h;                                // value head
-  const int hk = DELTA ? h / p.group : h;          // query / key head
-  const T* proj = reinterpret_cast<const T*>(p.proj);
-  if (slot <= 0 || slot >= p.num_slots) {          // padding rows: finite outputs, no state
-    if (slot >= p.num_slots && tid == 0) report_error(p.status, kErrBounds, 50, slot);
-    for (int t = 0; t < n; ++t) {
-      if (p.raw != nullptr) {
-        float* dst = p.raw + ((first + t) * p.heads + h) * p.raw_cols;
-        for (int c = c_first + tid; c < min(c_first + nc, p.raw_cols); c += threads) dst[c] = 0.f;
-        if (!DELTA && slice == 0 && tid == 0) dst[p.ncols] = 1.f;
-      } else {
-        T* dst = reinterpret_cast<T*>(p.out) + (first + t) * p.ldo + (long long)h * p.vdim;
-        for (int c = tid; c < p.vdim; c += threads) dst[c] = from_f32<T>(0.f);
-      }
-    }
-    return;
+// What a block reads of the projections: columns and convolution channels of its head's query, key and
+// value, and the inputs of tokens before the step's.
+template <typename T>
+struct Inputs {
+  const T* proj;
+  const T* old;
+  long long ld;
+  int back, start, channels;
+  int q_col, k_col, v_col, q_ch, k_ch, v_ch;
+  __device__ __forceinline__ Inputs(const ScanArgs& p, const Seq& s, int h, bool delta) {
+    const int hk = delta ? h / p.group : h, G = p.heads / p.group;
+    proj = reinterpret_cast<const T*>(p.proj) + s.first * p.ld;
+    ld = p.ld;
+    back = delta ? p.taps - 1 : 0;
+    start = s.start;
+    channels = p.channels;
+    old = reinterpret_cast<const T*>(p.conv_state) + ((long long)s.slot * 2 + s.phase) * back * channels;
+    q_col = p.q_at + hk * p.dim;
+    k_col = p.k_at + hk * p.dim;
+    v_col = p.v_at + h * p.vdim;
+    q_ch = hk * p.dim;
+    k_ch = (G + hk) * p.dim;
+    v_ch = 2 * G * p.dim + h * p.vdim;
   }
+  __device__ __forceinline__ int col(int part) const { return part == 0 ? q_col : part == 1 ? k_col : v_col; }
+  __device__ __forceinline__ int ch(int part) const { return part == 0 ? q_ch : part == 1 ? k_ch : v_ch; }
+  // part 0 query, 1 key, 2 value; token t of the step (t < 0: an earlier one)
+  __device__ __forceinline__ float one(int part, int d, int t) const {
+    if (t >= 0) return to_f32<T>(proj[t * ld + col(part) + d]);
+    return start + t >= 0 ? to_f32<T>(old[(long long)(back + t) * channels + ch(part) + d]) : 0.f;
+  }
+  __device__ __forceinline__ float4 four(int part, int d, int t) const {
+    if (t >= 0) return load4(proj + t * ld + col(part) + d);
+    return start + t >= 0 ? load4(old + (long long)(back + t) * channels + ch(part) + d)
+                          : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+};
 
-  // ---- this lane's part of the state
-  const int rl = lane & 7;
-  const int c_local = warp * Sh::kWarpCols + (lane >> 3) * kCols;   // of the block's columns
-  const int c0 = c_first + c_local;
-  float* state = p.state + ((long long)slot * p.heads + h) * p.dim * p.state_cols;
-  float2 S[kRows / 2][kCols];   // row pairs
-  const bool mine = c0 < p.state_cols;
+// The convolution's inputs that the sequence's next step reads, written by the blocks `qk` (queries and
+// keys) and those of the value columns [v0, v0 + nv).
+template <typename T>
+__device__ __forceinline__ void save_inputs(const ScanArgs& p, const Seq& s, const Inputs<T>& in, bool qk,
+                                            int v0, int nv) {
+  T* next = reinterpret_cast<T*>(p.conv_state) +
+            ((long long)s.slot * 2 + (s.phase ^ 1)) * in.back * p.channels;
+  const int per = (qk ? 2 * p.dim : 0) + nv;
+  for (int it = threadIdx.x; it < in.back * per; it += blockDim.x) {
+    const int j = it / per;
+    int x = it - j * per, part = 2;
+    if (qk) {
+      part = x < p.dim ? 0 : x < 2 * p.dim ? 1 : 2;
+      x -= part * p.dim;
+    }
+    if (part == 2) x += v0;
+    next[(long long)j * p.channels + in.ch(part) + x] = from_f32<T>(in.one(part, x, s.n - in.back + j));
+  }
+}
+
+// Lane's part of the state: rows j * 32 + rl * 4 + {0 .. 3}, kCols columns from c0, in row pairs
+template <int DP>
+__device__ __forceinline__ void load_state(float2 (&S)[ScanShape<DP>::kRows / 2][ScanShape<DP>::kCols],
+                                           const float* state, const ScanArgs& p, int rl, int c0,
+                                           bool any) {
+  constexpr int kCols = ScanShape<DP>::kCols;
 #pragma unroll
-  for (int j = 0; j < kChunks; ++j) {
+  for (int j = 0; j < ScanShape<DP>::kRows / 4; ++j) {
     const int r = j * 32 + rl * 4;
     float f[4][kCols];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
 #pragma unroll
       for (int c = 0; c < kCols; ++c) f[i][c] = 0.f;
-      if (start > 0 && mine && r + i < p.dim) {
+      if (any && c0 < p.state_cols && r + i < p.dim) {
         const float* src = state + (long long)(r + i) * p.state_cols + c0;
         if constexpr (kCols == 4) {
           const float4 v = load4(src);
@@ -186,409 +245,17 @@ __global__ void __launch_bounds__(kScanMaxWarps * 32, 1) scan_kernel(const ScanA
       S[2 * j + 1][c] = make_float2(f[2][c], f[3][c]);
     }
   }
-  if (!DELTA && tid == 0)
-    sMax[TT] = start > 0 ? p.max_state[((long long)slot * 2 + phase) * p.heads + h] : 0.f;
-
-  // ---- inputs: the projection's value of a channel at token t of this step (t < 0: earlier)
-  const int back = DELTA ? p.taps - 1 : 0;
-  const T* old_inputs = DELTA ? reinterpret_cast<const T*>(p.conv_state) +
-                                    ((long long)slot * 2 + phase) * back * p.channels
-                              : nullptr;
-  auto raw1 = [&](int t, int col, int ch) -> float {
-    if (t >= 0) return to_f32<T>(proj[(first + t) * p.ld + col]);
-    return start + t >= 0 ? to_f32<T>(old_inputs[(long long)(back + t) * p.channels + ch]) : 0.f;
-  };
-  auto raw4 = [&](int t, int col, int ch) -> float4 {
-    if (t >= 0) return load4(proj + (first + t) * p.ld + col);
-    return start + t >= 0 ? load4(old_inputs + (long long)(back + t) * p.channels + ch)
-                          : make_float4(0.f, 0.f, 0.f, 0.f);
-  };
-  const int q_col = p.q_at + hk * p.dim, k_col = p.k_at + hk * p.dim, v_col = p.v_at + hv * p.vdim;
-  const int q_ch = hk * p.dim, k_ch = (p.heads / p.group + hk) * p.dim;
-  const int v_ch = 2 * (p.heads / p.group) * p.dim + hv * p.vdim;
-  const int nv = min(nc, p.vdim - c_first);   // value columns of this block (the rest: zeros or 1)
-
-  for (int t0 = 0; t0 < n; t0 += TT) {
-    const int nt = min(TT, n - t0);
-    __syncthreads();   // the last tile's outputs have been read
-    // ---- 1. queries, keys and values (convolved)
-    {
-      const int step4 = p.vec ? 4 : 1;
-      const int per = (2 * DP + nc) / step4;
-      for (int it = tid; it < TT * per; it += threads) {
-        const int t = it / per, x = (it - t * per) * step4;
-        const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
-        const int d = part == 0 ? x : part == 1 ? x - DP : x - 2 * DP;
-        const int limit = part == 2 ? nv : p.dim;
-        const int col = (part == 0 ? q_col : part == 1 ? k_col : v_col + c_first) + d;
-        const int ch = (part == 0 ? q_ch : part == 1 ? k_ch : v_ch + c_first) + d;
-        float* dst = (part == 0 ? sC + t * DP : part == 1 ? sB + t * DP : sV + t * nc) + d;
-        if (p.vec) {
-          float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (t < nt && d < limit) {
-            if (DELTA) {
-              for (int j = 0; j < p.taps; ++j) {
-                const float4 w = load4(p.conv + (long long)j * p.channels + ch);
-                const float4 v = raw4(t0 + t - back + j, col, ch);
-                y.x = fmaf(w.x, v.x, y.x); y.y = fmaf(w.y, v.y, y.y);
-                y.z = fmaf(w.z, v.z, y.z); y.w = fmaf(w.w, v.w, y.w);
-              }
-              y = make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w));
-            } else {
-              y = raw4(t0 + t, col, 0);
-            }
-          }
-          if (!DELTA && part == 2) {   // the normaliser's column
-            const int one = p.vdim - c_first - d;
-            if (one == 0) y.x = 1.f;
-            if (one == 1) y.y = 1.f;
-            if (one == 2) y.z = 1.f;
-            if (one == 3) y.w = 1.f;
-          }
-          store4(dst, y);
-        } else {
-          float y = 0.f;
-          if (t < nt && d < limit) {
-            if (DELTA) {
-              for (int j = 0; j < p.taps; ++j)
-                y = fmaf(p.conv[(long long)j * p.channels + ch], raw1(t0 + t - back + j, col, ch), y);
-              y = silu_f(y);
-            } else {
-              y = raw1(t0 + t, col, 0);
-            }
-          }
-          if (!DELTA && part == 2 && d == p.vdim - c_first) y = 1.f;
-          *dst = y;
-        }
-      }
-    }
-    if (!DELTA && tid < 32) {
-      // m' = max(f + m, i) of the tile's tokens one after the other; lane t holds token t's logs
-      float gi = 0.f, gf = 0.f;
-      if (lane < nt) {
-        const T* r = proj + (first + t0 + lane) * p.ld;
-        gi = p.cap * tanhf((to_f32<T>(r[p.i_at + h]) + p.i_bias[h]) / p.cap);
-        const float z = p.cap * tanhf((to_f32<T>(r[p.f_at + h]) + p.f_bias[h]) / p.cap);
-        gf = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-      }
-      float m = sMax[TT], cum = 0.f;
-      for (int t = 0; t < nt; ++t) {
-        const float i = __shfl_sync(0xffffffffu, gi, t), f = __shfl_sync(0xffffffffu, gf, t);
-        const float m_new = fmaxf(f + m, i);
-        cum += fmaxf(f + m - m_new, kMinLogDecay);
-        if (lane == 0) {
-          sBeta[t] = i - m_new;
-          invQ[t] = cum;
-          sMax[t] = m_new;
-        }
-        m = m_new;
-      }
-      if (lane == 0) {
-        for (int t = nt; t < TT; ++t) {
-          sBeta[t] = 0.f;
-          invQ[t] = cum;
-        }
-        sMax[TT] = m;
-      }
-    }
-    __syncthreads();
-    // ---- 2. unit length, step sizes
-    if (DELTA) {
-      for (int t = warp; t < TT; t += warps) {
-        float a = 0.f, b = 0.f;
-        for (int d = lane; d < DP; d += 32) {
-          const float q = sC[t * DP + d], k = sB[t * DP + d];
-          a = fmaf(q, q, a);
-          b = fmaf(k, k, b);
-        }
-        a = warp_sum(a);
-        b = warp_sum(b);
-        if (lane == 0) {
-          invQ[t] = p.q_scale / sqrtf(a + 1e-6f);
-          invK[t] = 1.f / sqrtf(b + 1e-6f);
-          sBeta[t] = t < nt ? 1.f / (1.f + expf(-to_f32<T>(proj[(first + t0 + t) * p.ld + p.b_at + h])))
-                            : 0.f;
-        }
-      }
-      __syncthreads();
-    }
-    // ---- 3. decays; a, b, c
-    bool strong = false;
-    if (DELTA) {
-      // a thread owns a channel (blocks of fewer threads than channels: several, one after the
-      // other); its cumulative logs of the tile go through sA
-      bool deep = false;
-      for (int d = tid; d < DP; d += threads) {
-        float cum = 0.f;
-        if (d < p.dim) {
-          const T* z = reinterpret_cast<const T*>(p.decay) + (first + t0) * p.ld_decay + h * p.dim + d;
-          const float ae = p.a_exp[h], bias = p.dt_bias[h * p.dim + d];
-          float raw[TT];
+}
+template <int DP>
+__device__ __forceinline__ void store_state(const float2 (&S)[ScanShape<DP>::kRows / 2][ScanShape<DP>::kCols],
+                                            float* state, const ScanArgs& p, int rl, int c0) {
+  constexpr int kCols = ScanShape<DP>::kCols;
 #pragma unroll
-          for (int t = 0; t < TT; ++t) raw[t] = t < nt ? to_f32<T>(z[(long long)t * p.ld_decay]) : 0.f;
-#pragma unroll
-          for (int t = 0; t < TT; ++t) {
-            if (t < nt) cum += fmaxf(-ae * softplus_f(raw[t] + bias), kMinLogDecay);
-            sA[t * DP + d] = cum;
-          }
-        } else {
-          for (int t = 0; t < TT; ++t) sA[t * DP + d] = 0.f;
-        }
-        deep |= cum < kTileLogDecay;
-      }
-      strong = TT > B && __syncthreads_or(deep);
-      for (int d = tid; d < DP; d += threads) {
-        float base = 0.f;
-        for (int t = 0; t < TT; ++t) {
-          const float cum = sA[t * DP + d] - base;
-          const float g = __expf(cum), k = sB[t * DP + d] * invK[t];
-          sA[t * DP + d] = k * g;
-          sB[t * DP + d] = k * __expf(-cum);
-          sC[t * DP + d] *= invQ[t] * g;
-          if (t % B == B - 1) {
-            sG[t / B * DP + d] = g;
-            if (strong) base += cum;
-          }
-        }
-      }
-    } else {
-      strong = TT > B && invQ[TT - 1] < kTileLogDecay;
-      for (int it = tid; it < TT * DP; it += threads) {
-        const int t = it / DP;
-        const float base = strong && t >= B ? invQ[t / B * B - 1] : 0.f;
-        const float cum = invQ[t] - base;
-        sB[it] *= __expf(sBeta[t] - cum);
-        sC[it] *= p.q_scale * __expf(cum);
-        if (t % B == B - 1) sG[t / B * DP + it - t * DP] = __expf(cum);
-      }
-    }
-    __syncthreads();
-    // ---- 4. scalar products within groups of B tokens
-    for (int i = warp; i < TT; i += warps) {
-      const int g0 = i / B * B;
-      float a[B], c[B];
-#pragma unroll
-      for (int j = 0; j < B; ++j) a[j] = c[j] = 0.f;
-      for (int d = lane; d < DP; d += 32) {
-        const float ai = DELTA ? sA[i * DP + d] : 0.f, ci = sC[i * DP + d];
-#pragma unroll
-        for (int j = 0; j < B; ++j) {
-          const float b = sB[(g0 + j) * DP + d];
-          if (DELTA) a[j] = fmaf(ai, b, a[j]);
-          c[j] = fmaf(ci, b, c[j]);
-        }
-      }
-#pragma unroll
-      for (int j = 0; j < B; ++j) {
-        const float x = DELTA ? warp_sum(a[j]) : 0.f, y = warp_sum(c[j]);
-        if (lane == 0) {
-          dotB[i * B + j] = x;
-          dotC[i * B + j] = y;
-        }
-      }
-    }
-    __syncthreads();
-    // ---- 5. the recurrence
-    if (c_local < nc) {
-      for (int g0 = 0; g0 < nt; g0 += B) {
-        constexpr int kKinds = DELTA ? 2 : 1;
-        float2 acc[kKinds][kCols][B];
-#pragma unroll
-        for (int e = 0; e < kKinds; ++e)
-#pragma unroll
-          for (int c = 0; c < kCols; ++c)
-#pragma unroll
-            for (int i = 0; i < B; ++i) acc[e][c][i] = make_float2(0.f, 0.f);
-#pragma unroll
-        for (int j = 0; j < kChunks; ++j) {
-          const int r = j * 32 + rl * 4;
-#pragma unroll
-          for (int i = 0; i < B; ++i) {
-            const float4 vc = load4(sC + (g0 + i) * DP + r);
-            if constexpr (DELTA) {
-              const float4 va = load4(sA + (g0 + i) * DP + r);
-#pragma unroll
-              for (int c = 0; c < kCols; ++c) {
-                fma2(acc[0][c][i], S[2 * j][c], make_float2(va.x, va.y));
-                fma2(acc[0][c][i], S[2 * j + 1][c], make_float2(va.z, va.w));
-              }
-            }
-#pragma unroll
-            for (int c = 0; c < kCols; ++c) {
-              fma2(acc[kKinds - 1][c][i], S[2 * j][c], make_float2(vc.x, vc.y));
-              fma2(acc[kKinds - 1][c][i], S[2 * j + 1][c], make_float2(vc.z, vc.w));
-            }
-          }
-        }
-        // Sums over the eight lanes of a column: each exchange halves what a lane still carries, so
-        // that in the end it has one kind (delta: lanes 0 - 3 Z^T a, 4 - 7 Z^T c) of one column.
-        float my[B];
-        int my_c;
-        if constexpr (DELTA) {
-          float v[kCols][B];
-          const bool hi = lane & 4;
-#pragma unroll
-          for (int c = 0; c < kCols; ++c)
-#pragma unroll
-            for (int i = 0; i < B; ++i) {
-              const float x = acc[0][c][i].x + acc[0][c][i].y, y = acc[1][c][i].x + acc[1][c][i].y;
-              const float got = __shfl_xor_sync(0xffffffffu, hi ? x : y, 4);
-              v[c][i] = (hi ? y : x) + got;
-            }
-          if constexpr (kCols == 4) {
-            const bool c2 = lane & 2, c1 = lane & 1;
-            float w[2][B];
-#pragma unroll
-            for (int c = 0; c < 2; ++c)
-#pragma unroll
-              for (int i = 0; i < B; ++i) {
-                const float got = __shfl_xor_sync(0xffffffffu, c2 ? v[c][i] : v[c + 2][i], 2);
-                w[c][i] = (c2 ? v[c + 2][i] : v[c][i]) + got;
-              }
-#pragma unroll
-            for (int i = 0; i < B; ++i) {
-              const float got = __shfl_xor_sync(0xffffffffu, c1 ? w[0][i] : w[1][i], 1);
-              my[i] = (c1 ? w[1][i] : w[0][i]) + got;
-            }
-            my_c = lane & 3;
-          } else {
-            const bool c1 = lane & 1;
-#pragma unroll
-            for (int i = 0; i < B; ++i) {
-              const float got = __shfl_xor_sync(0xffffffffu, c1 ? v[0][i] : v[1][i], 1);
-              const float x = (c1 ? v[1][i] : v[0][i]) + got;
-              my[i] = x + __shfl_xor_sync(0xffffffffu, x, 2);
-            }
-            my_c = lane & 1;
-          }
-        } else {
-          if constexpr (kCols == 4) {
-            const bool c2 = lane & 2, c1 = lane & 1;
-            float w[2][B];
-#pragma unroll
-            for (int c = 0; c < 2; ++c)
-#pragma unroll
-              for (int i = 0; i < B; ++i) {
-                const float x = acc[0][c][i].x + acc[0][c][i].y, y = acc[0][c + 2][i].x + acc[0][c + 2][i].y;
-                const float got = __shfl_xor_sync(0xffffffffu, c2 ? x : y, 2);
-                w[c][i] = (c2 ? y : x) + got;
-              }
-#pragma unroll
-            for (int i = 0; i < B; ++i) {
-              const float got = __shfl_xor_sync(0xffffffffu, c1 ? w[0][i] : w[1][i], 1);
-              const float x = (c1 ? w[1][i] : w[0][i]) + got;
-              my[i] = x + __shfl_xor_sync(0xffffffffu, x, 4);
-            }
-            my_c = lane & 3;
-          } else {
-            const bool c1 = lane & 1;
-#pragma unroll
-            for (int i = 0; i < B; ++i) {
-              const float a = acc[0][0][i].x + acc[0][0][i].y, b = acc[0][1][i].x + acc[0][1][i].y;
-              const float got = __shfl_xor_sync(0xffffffffu, c1 ? a : b, 1);
-              float x = (c1 ? b : a) + got;
-              x += __shfl_xor_sync(0xffffffffu, x, 2);
-              my[i] = x + __shfl_xor_sync(0xffffffffu, x, 4);
-            }
-            my_c = lane & 1;
-          }
-        }
-        // u of every token and column; o
-        float u[B];
-#pragma unroll
-        for (int i = 0; i < B; ++i) {
-          const float v = sV[(g0 + i) * nc + c_local + my_c];
-          u[i] = v;
-          if constexpr (DELTA) {
-            float x = v - my[i];
-#pragma unroll
-            for (int j = 0; j < B; ++j)
-              if (j < i) x = fmaf(-dotB[(g0 + i) * B + j], u[j], x);
-            u[i] = sBeta[g0 + i] * x;   // (of use in lanes 0 - 3)
-          }
-        }
-        float U[B][kCols];
-        if constexpr (DELTA) {
-#pragma unroll
-          for (int i = 0; i < B; ++i) {
-#pragma unroll
-            for (int c = 0; c < kCols; ++c) U[i][c] = __shfl_sync(0xffffffffu, u[i], (lane & 24) | c);
-            u[i] = __shfl_sync(0xffffffffu, u[i], (lane & 24) | my_c);
-          }
-        } else {
-#pragma unroll
-          for (int i = 0; i < B; ++i)
-#pragma unroll
-            for (int c = 0; c < kCols; ++c) U[i][c] = sV[(g0 + i) * nc + c_local + c];
-        }
-        __syncwarp();   // the values of these tokens have been read: the outputs take their place
-#pragma unroll
-        for (int i = 0; i < B; ++i) {
-          float o = my[i];
-#pragma unroll
-          for (int j = 0; j < B; ++j)
-            if (j <= i) o = fmaf(dotC[(g0 + i) * B + j], u[j], o);
-          if (rl >= 4 && rl < 4 + kCols) sV[(g0 + i) * nc + c_local + my_c] = o;
-        }
-        const bool renorm = strong || g0 + B >= nt;
-        const float* ge = sG + (strong ? g0 / B : TT / B - 1) * DP;
-#pragma unroll
-        for (int j = 0; j < kChunks; ++j) {
-          const int r = j * 32 + rl * 4;
-#pragma unroll
-          for (int i = 0; i < B; ++i) {
-            const float4 b = load4(sB + (g0 + i) * DP + r);
-#pragma unroll
-            for (int c = 0; c < kCols; ++c) {
-              const float2 uu = make_float2(U[i][c], U[i][c]);
-              fma2(S[2 * j][c], make_float2(b.x, b.y), uu);
-              fma2(S[2 * j + 1][c], make_float2(b.z, b.w), uu);
-            }
-          }
-          if (renorm) {
-            const float4 g = load4(ge + r);
-#pragma unroll
-            for (int c = 0; c < kCols; ++c) {
-              mul2(S[2 * j][c], make_float2(g.x, g.y));
-              mul2(S[2 * j + 1][c], make_float2(g.z, g.w));
-            }
-          }
-        }
-      }
-    }
-    __syncthreads();
-    // ---- 6. outputs
-    for (int t = warp; t < nt; t += warps) {
-      const float* o = sV + t * nc;
-      const long long row = first + t0 + t;
-      if (p.raw != nullptr) {
-        float* dst = p.raw + (row * p.heads + h) * p.raw_cols + c_first;
-        for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = o[c];
-        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = expf(-sMax[t]);
-        continue;
-      }
-      float scale = 1.f, ss = 0.f;
-      if (!DELTA) scale = 1.f / (fmaxf(fabsf(o[p.vdim]), expf(-sMax[t])) + 1e-6f);
-      for (int c = lane; c < p.vdim; c += 32) {
-        const float x = o[c] * scale;
-        ss = fmaf(x, x, ss);
-      }
-      scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
-      const T* g = reinterpret_cast<const T*>(p.gate) + row * p.ld_gate + (long long)h * p.vdim;
-      const float* w = p.norm + (long long)h * p.norm_step;
-      T* dst = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
-      for (int c = lane; c < p.vdim; c += 32)
-        dst[c] = from_f32<T>(o[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
-    }
-  }
-
-  // ---- what the sequence's next step starts from
-#pragma unroll
-  for (int j = 0; j < kChunks; ++j) {
+  for (int j = 0; j < ScanShape<DP>::kRows / 4; ++j) {
     const int r = j * 32 + rl * 4;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      if (!mine || c_local >= nc || r + i >= p.dim) continue;
+      if (c0 >= p.state_cols || r + i >= p.dim) continue;
       float* dst = state + (long long)(r + i) * p.state_cols + c0;
       auto at = [&](int c) { return (i & 1) ? S[2 * j + i / 2][c].y : S[2 * j + i / 2][c].x; };
       if constexpr (kCols == 4)
@@ -597,19 +264,715 @@ __global__ void __launch_bounds__(kScanMaxWarps * 32, 1) scan_kernel(const ScanA
         *reinterpret_cast<float2*>(dst) = make_float2(at(0), at(1));
     }
   }
-  if (DELTA) {
-    T* next = reinterpret_cast<T*>(p.conv_state) + ((long long)slot * 2 + (phase ^ 1)) * back * p.channels;
-    const bool qk = slice == 0 && h % p.group == 0;
-    for (int it = tid; it < back * (2 * p.dim + nv); it += threads) {
-      const int j = it / (2 * p.dim + nv), x = it - j * (2 * p.dim + nv);
-      if (x < 2 * p.dim && !qk) continue;
-      const int col = x < p.dim ? q_col + x : x < 2 * p.dim ? k_col + x - p.dim : v_col + c_first + x - 2 * p.dim;
-      const int ch = x < p.dim ? q_ch + x : x < 2 * p.dim ? k_ch + x - p.dim : v_ch + c_first + x - 2 * p.dim;
-      next[(long long)j * p.channels + ch] = from_f32<T>(raw1(n - back + j, col, ch));
+}
+
+// Sums of acc over the eight lanes of a column group. Each exchange halves what a lane still carries,
+// so that in the end it has one kind (two kinds: lanes 0 - 3 the first, 4 - 7 the second) of one
+// column, which is returned.
+template <int KINDS, int COLS, int N>
+__device__ __forceinline__ int reduce_columns(const float2 (&acc)[KINDS][COLS][N], float (&my)[N]) {
+  const int lane = threadIdx.x & 31;
+  const bool hi = lane & 4, c2 = lane & 2, c1 = lane & 1;
+  float v[COLS][N];
+#pragma unroll
+  for (int c = 0; c < COLS; ++c)
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      v[c][i] = acc[0][c][i].x + acc[0][c][i].y;
+      if constexpr (KINDS == 2) {
+        const float y = acc[1][c][i].x + acc[1][c][i].y;
+        const float got = __shfl_xor_sync(0xffffffffu, hi ? v[c][i] : y, 4);
+        v[c][i] = (hi ? y : v[c][i]) + got;
+      }
     }
-  } else if (slice == 0 && tid == 0) {
-    p.max_state[((long long)slot * 2 + (phase ^ 1)) * p.heads + h] = sMax[TT];
+  float w[2][N];
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      if constexpr (COLS == 4) {
+        const float got = __shfl_xor_sync(0xffffffffu, c2 ? v[c][i] : v[c + 2][i], 2);
+        w[c][i] = (c2 ? v[c + 2][i] : v[c][i]) + got;
+      } else {
+        w[c][i] = v[c][i];
+      }
+    }
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const float got = __shfl_xor_sync(0xffffffffu, c1 ? w[0][i] : w[1][i], 1);
+    my[i] = (c1 ? w[1][i] : w[0][i]) + got;
+    if constexpr (COLS == 2) my[i] += __shfl_xor_sync(0xffffffffu, my[i], 2);
+    if constexpr (KINDS == 1) my[i] += __shfl_xor_sync(0xffffffffu, my[i], 4);
   }
+  return lane & (COLS - 1);
+}
+
+// Outputs of padding rows: finite, no state involved
+template <typename T, bool DELTA>
+__device__ __forceinline__ void put_zeros(const ScanArgs& p, const Seq& s, int h, int slice) {
+  if (s.slot >= p.num_slots && threadIdx.x == 0) report_error(p.status, kErrBounds, 50, s.slot);
+  for (int t = 0; t < s.n; ++t) {
+    if (p.raw != nullptr) {
+      float* dst = p.raw + ((s.first + t) * p.heads + h) * p.raw_cols;
+      const int c1 = min((slice + 1) * p.nc, p.ncols);
+      for (int c = slice * p.nc + threadIdx.x; c < c1; c += blockDim.x) dst[c] = 0.f;
+      if (!DELTA && slice == 0 && threadIdx.x == 0) dst[p.ncols] = 1.f;
+    } else {
+      T* dst = reinterpret_cast<T*>(p.out) + (s.first + t) * p.ldo + (long long)h * p.vdim;
+      for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) dst[c] = from_f32<T>(0.f);
+    }
+  }
+}
+
+// A warp's token: norm, weight and gate of a head's outputs o (memory: with the normaliser's product
+// in column vdim and `floor` = exp(-m)).
+template <typename T, bool DELTA>
+__device__ __forceinline__ void head_output(const ScanArgs& p, const float* o, long long row, int h,
+                                            float floor) {
+  const int lane = threadIdx.x & 31;
+  const T* g = reinterpret_cast<const T*>(p.gate) + row * p.ld_gate + (long long)h * p.vdim;
+  const float* w = p.norm + (long long)h * p.norm_step;
+  T* dst = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
+  float scale = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floor) + 1e-6f);
+  float ss = 0.f;
+  for (int c = lane; c < p.vdim; c += 32) {
+    const float x = o[c] * scale;
+    ss = fmaf(x, x, ss);
+  }
+  scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+  for (int c = lane; c < p.vdim; c += 32)
+    dst[c] = from_f32<T>(o[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
+}
+
+// ------------------------------------------------------------------ one token per sequence
+template <typename T, int DP, bool DELTA>
+__global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_kernel(const ScanArgs p) {
+  using Sh = ScanShape<DP>;
+  constexpr int kCols = Sh::kCols, kChunks = Sh::kRows / 4;
+  extern __shared__ __align__(16) float sm[];
+  float* sQ = sm;              // query, key (before their norms), decay, values / outputs
+  float* sK = sm + DP;
+  float* sG = sm + 2 * DP;
+  float* sV = sm + 3 * DP;
+  pdl_wait();
+  pdl_trigger();
+  const int slice = blockIdx.x % p.slices, h = blockIdx.x / p.slices % p.heads;
+  const Seq s(p.steps + (long long)(blockIdx.x / p.slices / p.heads) * kStepInts);
+  if (s.n <= 0) return;
+  if (s.slot <= 0 || s.slot >= p.num_slots) {
+    put_zeros<T, DELTA>(p, s, h, slice);
+    return;
+  }
+  const int tid = threadIdx.x, threads = blockDim.x, lane = tid & 31, rl = lane & 7;
+  const int c_first = slice * p.nc, c_local = (tid >> 5) * Sh::kWarpCols + (lane >> 3) * kCols;
+  float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols;
+  float2 S[Sh::kRows / 2][kCols];
+  load_state<DP>(S, state, p, rl, c_first + c_local, s.start > 0);
+
+  const Inputs<T> in(p, s, h, DELTA);
+  const int nv = min(p.nc, p.vdim - c_first);
+  float keep = 0.f, put = 0.f, m_new = 0.f, beta = 0.f;
+  if (DELTA) {
+    beta = sigmoid_f(to_f32<T>(in.proj[p.b_at + h]));
+  } else {
+    const float2 g = memory_log_gates(to_f32<T>(in.proj[p.i_at + h]) + p.i_bias[h],
+                                      to_f32<T>(in.proj[p.f_at + h]) + p.f_bias[h], p.cap);
+    const float m = s.start > 0 ? p.max_state[((long long)s.slot * 2 + s.phase) * p.heads + h] : 0.f;
+    m_new = fmaxf(g.y + m, g.x);
+    keep = expf(g.y + m - m_new);
+    put = expf(g.x - m_new);
+  }
+  for (int x = tid; x < 2 * DP + p.nc; x += threads) {
+    const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
+    const int d = x - part * DP + (part == 2 ? c_first : 0);
+    const bool ok = part == 2 ? d < c_first + nv : d < p.dim;
+    float y = 0.f;
+    if (DELTA && ok) {
+      const float* w = p.conv + in.ch(part) + d;
+      float xv[kTaps], wv[kTaps];
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) {   // all loads at once
+        const bool use = j < p.taps;
+        xv[j] = use ? in.one(part, d, j - in.back) : 0.f;
+        wv[j] = use ? w[(long long)j * p.channels] : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) y = fmaf(wv[j], xv[j], y);
+      for (int j = kTaps; j < p.taps; ++j)
+        y = fmaf(w[(long long)j * p.channels], in.one(part, d, j - in.back), y);
+      y = silu_f(y);
+      if (part == 0)
+        sG[d] = expf(-p.a_exp[h] *
+                     softplus_f(to_f32<T>(reinterpret_cast<const T*>(p.decay)[s.first * p.ld_decay +
+                                                                              h * p.dim + d]) +
+                                p.dt_bias[h * p.dim + d]));
+    } else if (!DELTA) {
+      if (ok) y = in.one(part, d, 0);
+      if (part == 2 && d == p.vdim) y = 1.f;
+    }
+    if (DELTA && part == 0 && !ok) sG[d] = 1.f;
+    (part == 0 ? sQ : part == 1 ? sK : sV)[part == 2 ? d - c_first : d] = y;
+  }
+  __syncthreads();
+  // every warp: norms and the product of query and key
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  for (int d = lane; d < DP; d += 32) {
+    const float q = sQ[d], k = sK[d];
+    qq = fmaf(q, q, qq);
+    kk = fmaf(k, k, kk);
+    qk = fmaf(q, k, qk);
+  }
+  qk = warp_sum(qk);
+  float fq = p.q_scale, fk = 1.f;
+  if (DELTA) {
+    fq /= sqrtf(warp_sum(qq) + 1e-6f);
+    fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+  }
+  qk *= fq * fk * (DELTA ? 1.f : put);
+  constexpr int kKinds = DELTA ? 2 : 1;
+  float2 acc[kKinds][kCols][1];
+#pragma unroll
+  for (int e = 0; e < kKinds; ++e)
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) acc[e][c][0] = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < kChunks; ++j) {
+    const int r = j * 32 + rl * 4;
+    const float4 q = load4(sQ + r);
+    if constexpr (DELTA) {
+      const float4 k = load4(sK + r), g = load4(sG + r);
+#pragma unroll
+      for (int c = 0; c < kCols; ++c) {   // S <- g * S; S^T k
+        mul2(S[2 * j][c], make_float2(g.x, g.y));
+        mul2(S[2 * j + 1][c], make_float2(g.z, g.w));
+        fma2(acc[0][c][0], S[2 * j][c], make_float2(k.x, k.y));
+        fma2(acc[0][c][0], S[2 * j + 1][c], make_float2(k.z, k.w));
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) {
+      fma2(acc[kKinds - 1][c][0], S[2 * j][c], make_float2(q.x, q.y));
+      fma2(acc[kKinds - 1][c][0], S[2 * j + 1][c], make_float2(q.z, q.w));
+    }
+  }
+  float my[1];
+  const int my_c = reduce_columns<kKinds, kCols, 1>(acc, my);
+  float U[kCols], u = sV[c_local + my_c], o;
+  if constexpr (DELTA) {
+    u = beta * (u - fk * my[0]);          // (of use in lanes 0 - 3)
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) U[c] = fk * __shfl_sync(0xffffffffu, u, (lane & 24) | c);
+    u = __shfl_sync(0xffffffffu, u, (lane & 24) | my_c);
+    o = fmaf(qk, u, fq * my[0]);
+  } else {
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) U[c] = put * sV[c_local + c];
+    o = fmaf(qk, u, keep * fq * my[0]);
+  }
+  __syncwarp();   // the values have been read: the outputs take their place
+  if (rl >= 4 && rl < 4 + kCols) sV[c_local + my_c] = o;
+#pragma unroll
+  for (int j = 0; j < kChunks; ++j) {
+    const float4 k = load4(sK + j * 32 + rl * 4);
+#pragma unroll
+    for (int c = 0; c < kCols; ++c) {
+      if constexpr (!DELTA) {
+        mul2(S[2 * j][c], make_float2(keep, keep));
+        mul2(S[2 * j + 1][c], make_float2(keep, keep));
+      }
+      const float2 uu = make_float2(U[c], U[c]);
+      fma2(S[2 * j][c], make_float2(k.x, k.y), uu);
+      fma2(S[2 * j + 1][c], make_float2(k.z, k.w), uu);
+    }
+  }
+  store_state<DP>(S, state, p, rl, c_first + c_local);
+  __syncthreads();
+  if (p.raw != nullptr) {
+    float* dst = p.raw + (s.first * p.heads + h) * p.raw_cols + c_first;
+    for (int c = tid; c < min(p.nc, p.ncols - c_first); c += threads) dst[c] = sV[c];
+    if (!DELTA && slice == 0 && tid == 0) dst[p.ncols] = expf(-m_new);
+  } else {   // every warp the norm, then its own columns
+    float scale = DELTA ? 1.f : 1.f / (fmaxf(fabsf(sV[p.vdim]), expf(-m_new)) + 1e-6f), ss = 0.f;
+    for (int c = lane; c < p.vdim; c += 32) {
+      const float x = sV[c] * scale;
+      ss = fmaf(x, x, ss);
+    }
+    scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+    const T* g = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
+    const float* w = p.norm + (long long)h * p.norm_step;
+    T* dst = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
+    for (int c = tid; c < p.vdim; c += threads)
+      dst[c] = from_f32<T>(sV[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
+  }
+  if (DELTA)
+    save_inputs<T>(p, s, in, slice == 0 && h % p.group == 0, c_first, max(0, nv));
+  else if (slice == 0 && tid == 0)
+    p.max_state[((long long)s.slot * 2 + (s.phase ^ 1)) * p.heads + h] = m_new;
+}
+
+// ------------------------------------------------------------------ portions of several tokens
+// Gates of the matrix memory: m' = max(f + m, i) composes as (F, I) -> max(F + m, I), so a block scans
+// a head's tokens 1024 at a time.
+template <typename T>
+__global__ void __launch_bounds__(1024) memory_gates_kernel(const ScanArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float2 part[32];
+  __shared__ float carry;
+  const int h = blockIdx.x % p.heads;
+  const Seq s(p.steps + (long long)(blockIdx.x / p.heads) * kStepInts);
+  if (s.n <= 0 || s.slot <= 0 || s.slot >= p.num_slots) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float m0 = s.start > 0 ? p.max_state[((long long)s.slot * 2 + s.phase) * p.heads + h] : 0.f;
+  const T* proj = reinterpret_cast<const T*>(p.proj) + s.first * p.ld;
+  for (int t0 = 0; t0 < s.n; t0 += blockDim.x) {
+    const int t = t0 + tid;
+    float2 g = make_float2(-INFINITY, 0.f);   // i, f: neither puts nor forgets
+    if (t < s.n)
+      g = memory_log_gates(to_f32<T>(proj[t * p.ld + p.i_at + h]) + p.i_bias[h],
+                           to_f32<T>(proj[t * p.ld + p.f_at + h]) + p.f_bias[h], p.cap);
+    float I = g.x, F = g.y;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float i1 = __shfl_up_sync(0xffffffffu, I, o), f1 = __shfl_up_sync(0xffffffffu, F, o);
+      if (lane >= o) {
+        I = fmaxf(i1 + F, I);
+        F += f1;
+      }
+    }
+    if (lane == 31) part[warp] = make_float2(I, F);
+    __syncthreads();
+    float m = m0;                              // the maximum before this warp's tokens
+    for (int w = 0; w < warp; ++w) m = fmaxf(m + part[w].y, part[w].x);
+    const float m_new = fmaxf(F + m, I);
+    float m_old = __shfl_up_sync(0xffffffffu, m_new, 1);
+    if (lane == 0) m_old = m;
+    if (t < s.n) {
+      float* dst = p.gates + ((s.first + t) * p.heads + h) * 3;
+      dst[0] = fmaxf(g.y + m_old - m_new, kMinLogDecay);
+      dst[1] = g.x - m_new;
+      dst[2] = m_new;
+    }
+    if (tid == blockDim.x - 1) carry = m_new;
+    __syncthreads();
+    m0 = carry;
+    __syncthreads();
+  }
+  if (tid == 0) p.max_state[((long long)s.slot * 2 + (s.phase ^ 1)) * p.heads + h] = m0;
+}
+
+// A tile's records of a head: queries, keys, values (convolved), unit lengths, decays, products.
+template <typename T, int DP, bool DELTA>
+__global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanArgs p) {
+  using R = Record<DP, DELTA>;
+  constexpr int kThreads = DP <= 128 ? 128 : 256, kWarps = kThreads / 32;
+  constexpr int kOwn = (DP + kThreads - 1) / kThreads;
+  static_assert(kOwn == 1, "a thread owns a channel");
+  extern __shared__ __align__(16) float sm[];
+  float* sB = sm;                                // keys, then k / G
+  float* sC = sm + kTT * DP;                     // queries, then G q
+  float* sA = sm + 2 * kTT * DP;                 // delta: G k
+  __shared__ float invQ[kTT], invK[kTT];         // memory: log decay (cumulative), log input factor
+  pdl_wait();
+  pdl_trigger();
+  const int h = blockIdx.x % p.heads;
+  const long long tile = blockIdx.x / p.heads;
+  const int* tl = p.tiles + tile * 2;
+  const Seq s(p.steps + (long long)tl[0] * kStepInts);
+  if (s.slot <= 0 || s.slot >= p.num_slots) return;
+  const int t0 = tl[1], nt = min(kTT, s.n - t0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* rec = p.records + (tile * p.heads + h) * p.record;
+  const Inputs<T> in(p, s, h, DELTA);
+  const int vcols = p.slices * p.nc;
+
+  // this thread's channel of the decays, on its way
+  float z[kTT];
+  if (DELTA) {
+    const T* src = reinterpret_cast<const T*>(p.decay) + (s.first + t0) * p.ld_decay + h * p.dim + tid;
+#pragma unroll
+    for (int t = 0; t < kTT; ++t)
+      z[t] = tid < p.dim && t < nt ? to_f32<T>(src[(long long)t * p.ld_decay]) : 0.f;
+  } else if (tid < kTT) {
+    const float* g = p.gates + ((s.first + t0 + tid) * p.heads + h) * 3;
+    const bool ok = tid < nt;
+    invQ[tid] = ok ? g[0] : 0.f;
+    invK[tid] = ok ? g[1] : 0.f;
+    rec[R::kBeta + tid] = ok ? expf(-g[2]) : 1.f;
+  }
+  if (DELTA && tid < kTT)
+    rec[R::kBeta + tid] =
+        tid < nt ? sigmoid_f(to_f32<T>(in.proj[(long long)(t0 + tid) * p.ld + p.b_at + h])) : 0.f;
+
+  // ---- 1. four channels and all of the tile's tokens a thread
+  auto put = [&](int part, int d, int t, const float4& y) {
+    if (part == 2) store4(rec + R::kV + t * vcols + d, y);
+    else store4((part == 0 ? sC : sB) + t * DP + d, y);
+  };
+  for (int x = tid * 4; x < 2 * DP + vcols; x += kThreads * 4) {
+    const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
+    const int d = x - part * DP, limit = part == 2 ? p.vdim : p.dim;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (p.vec && (!DELTA || p.taps <= kTaps)) {
+      const bool ok = d < limit;
+      if constexpr (DELTA) {
+        float4 w[kTaps], v[kTaps + 3];
+#pragma unroll
+        for (int j = 0; j < kTaps; ++j) {   // the last tap is the current token's
+          const int k = j - (kTaps - p.taps);
+          w[j] = ok && k >= 0 ? load4(p.conv + (long long)k * p.channels + in.ch(part) + d) : zero;
+        }
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j)
+          v[j] = ok && j >= kTaps - p.taps ? in.four(part, d, t0 + j - (kTaps - 1)) : zero;
+#pragma unroll
+        for (int tb = 0; tb < kTT; tb += 4) {
+#pragma unroll
+          for (int t = 0; t < 4; ++t)
+            v[kTaps - 1 + t] = ok && tb + t < nt ? in.four(part, d, t0 + tb + t) : zero;
+#pragma unroll
+          for (int t = 0; t < 4; ++t) {
+            float4 y = zero;
+#pragma unroll
+            for (int j = 0; j < kTaps; ++j) axpy4(y, w[j], v[t + j]);
+            put(part, d, tb + t, tb + t < nt ? silu4(y) : zero);
+          }
+#pragma unroll
+          for (int j = 0; j < kTaps - 1; ++j) v[j] = v[4 + j];
+        }
+      } else {
+        const int one = part == 2 ? p.vdim - d : -1;   // the normaliser's column
+#pragma unroll
+        for (int t = 0; t < kTT; ++t) {
+          float4 y = ok && t < nt ? in.four(part, d, t0 + t) : zero;
+          if (one == 0) y.x = 1.f;
+          if (one == 1) y.y = 1.f;
+          if (one == 2) y.z = 1.f;
+          if (one == 3) y.w = 1.f;
+          put(part, d, t, y);
+        }
+      }
+      continue;
+    }
+    for (int t = 0; t < kTT; ++t) {
+      float y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        y[e] = 0.f;
+        if (t < nt && d + e < limit) {
+          if (DELTA) {
+            const float* w = p.conv + in.ch(part) + d + e;
+            for (int j = 0; j < p.taps; ++j)
+              y[e] = fmaf(w[(long long)j * p.channels], in.one(part, d + e, t0 + t - in.back + j), y[e]);
+            y[e] = silu_f(y[e]);
+          } else {
+            y[e] = in.one(part, d + e, t0 + t);
+          }
+        }
+        if (!DELTA && part == 2 && d + e == p.vdim) y[e] = 1.f;
+      }
+      put(part, d, t, make_float4(y[0], y[1], y[2], y[3]));
+    }
+  }
+  __syncthreads();
+
+  // ---- 2. unit length
+  if (DELTA) {
+    for (int t = warp; t < kTT; t += kWarps) {
+      float a = 0.f, b = 0.f;
+      for (int d = lane * 4; d < DP; d += 128) {
+        const float4 q = load4(sC + t * DP + d), k = load4(sB + t * DP + d);
+        a = dot4(q, q, a);
+        b = dot4(k, k, b);
+      }
+      a = warp_sum(a);
+      b = warp_sum(b);
+      if (lane == 0) {
+        invQ[t] = p.q_scale / sqrtf(a + 1e-6f);
+        invK[t] = 1.f / sqrtf(b + 1e-6f);
+      }
+    }
+  }
+  // ---- 3. decays; a, b, c
+  float cum = 0.f;
+  if (DELTA) {
+    const float ae = tid < p.dim ? p.a_exp[h] : 0.f;
+    const float bias = tid < p.dim ? p.dt_bias[h * p.dim + tid] : 0.f;
+#pragma unroll
+    for (int t = 0; t < kTT; ++t) {
+      if (t < nt) cum += fmaxf(-ae * softplus_f(z[t] + bias), kMinLogDecay);
+      z[t] = cum;
+    }
+  } else {
+#pragma unroll
+    for (int t = 0; t < kTT; ++t) {
+      cum += invQ[t];
+      z[t] = cum;
+    }
+  }
+  const bool strong = __syncthreads_or(cum < kTileLogDecay);
+  if (tid == 0) rec[R::kStrong] = strong ? 1.f : 0.f;
+  if (tid < DP) {
+    float base = 0.f;
+#pragma unroll
+    for (int t = 0; t < kTT; ++t) {
+      const float l = z[t] - base, g = __expf(l);
+      const float k = sB[t * DP + tid], q = sC[t * DP + tid];
+      const float kn = DELTA ? k * invK[t] : k;
+      const float b = kn * __expf((DELTA ? 0.f : invK[t]) - l);
+      const float c = q * g * (DELTA ? invQ[t] : p.q_scale);
+      sB[t * DP + tid] = b;
+      sC[t * DP + tid] = c;
+      rec[R::kKeys + t * DP + tid] = b;
+      rec[R::kQ + t * DP + tid] = c;
+      if (DELTA) {
+        sA[t * DP + tid] = kn * g;
+        rec[R::kA + t * DP + tid] = kn * g;
+      }
+      if (t % kB == kB - 1) {
+        rec[R::kG + t / kB * DP + tid] = g;
+        if (strong) base += l;
+      }
+    }
+  }
+  __syncthreads();
+  // ---- 4. scalar products within groups
+  for (int g = warp; g < kTT / kB; g += kWarps) {
+    float a[kB][kB], c[kB][kB];   // [token][earlier token]
+#pragma unroll
+    for (int i = 0; i < kB; ++i)
+#pragma unroll
+      for (int j = 0; j < kB; ++j) a[i][j] = c[i][j] = 0.f;
+    for (int d = lane * 4; d < DP; d += 128) {
+      float4 b[kB];
+#pragma unroll
+      for (int j = 0; j < kB; ++j) b[j] = load4(sB + (g * kB + j) * DP + d);
+#pragma unroll
+      for (int i = 0; i < kB; ++i) {
+        const float4 ci = load4(sC + (g * kB + i) * DP + d);
+        float4 ai = ci;
+        if (DELTA) ai = load4(sA + (g * kB + i) * DP + d);
+#pragma unroll
+        for (int j = 0; j <= i; ++j) {
+          c[i][j] = dot4(ci, b[j], c[i][j]);
+          if (DELTA && j < i) a[i][j] = dot4(ai, b[j], a[i][j]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kB; ++i)
+#pragma unroll
+      for (int j = 0; j <= i; ++j) {
+        const float y = warp_sum(c[i][j]);
+        const float x = DELTA && j < i ? warp_sum(a[i][j]) : 0.f;
+        if (lane == 0) {
+          rec[R::kDotC + (g * kB + i) * kB + j] = y;
+          if (j < i) rec[R::kDotB + (g * kB + i) * kB + j] = x;
+        }
+      }
+  }
+  if (DELTA && t0 + nt == s.n) save_inputs<T>(p, s, in, h % p.group == 0, 0, p.vdim);
+}
+
+// Floats of a stage of scan_kernel's shared memory
+template <int DP, bool DELTA>
+__host__ __device__ constexpr int stage_floats(int nc) {
+  return Record<DP, DELTA>::kV + kTT * nc;
+}
+
+template <typename T, int DP, bool DELTA, int STAGES>
+__global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const ScanArgs p) {
+  using Sh = ScanShape<DP>;
+  using R = Record<DP, DELTA>;
+  constexpr int kCols = Sh::kCols, kChunks = Sh::kRows / 4, kKinds = DELTA ? 2 : 1;
+  extern __shared__ __align__(16) float sm[];
+  pdl_wait();
+  pdl_trigger();
+  const int slice = blockIdx.x % p.slices, h = blockIdx.x / p.slices % p.heads;
+  const int seq = blockIdx.x / p.slices / p.heads;
+  const Seq s(p.steps + (long long)seq * kStepInts);
+  if (s.n <= 0) return;
+  if (s.slot <= 0 || s.slot >= p.num_slots) {
+    put_zeros<T, DELTA>(p, s, h, slice);
+    return;
+  }
+  const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31, rl = lane & 7;
+  const int nc = p.nc, c_first = slice * nc, vcols = p.slices * nc;
+  const int c_local = warp * Sh::kWarpCols + (lane >> 3) * kCols;
+  const int stage_size = stage_floats<DP, DELTA>(nc);
+  const int tiles = (s.n + kTT - 1) / kTT;
+  const float* rec0 = p.records + ((long long)p.first_tile[seq] * p.heads + h) * p.record;
+  auto fetch = [&](int i) {   // (one group of copies per tile, also when there is none)
+    if (i < tiles) {
+      const float* src = rec0 + (long long)i * p.heads * p.record;
+      float* dst = sm + i % STAGES * stage_size;
+      for (int x = tid * 4; x < R::kV; x += threads * 4) copy16_async(dst + x, src + x);
+      const int per = nc / 4;
+      for (int x = tid; x < kTT * per; x += threads) {
+        const int t = x / per, c = (x - t * per) * 4;
+        copy16_async(dst + R::kV + t * nc + c, src + R::kV + t * vcols + c_first + c);
+      }
+    }
+    copies_commit();
+  };
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) fetch(i);
+  float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols;
+  float2 S[Sh::kRows / 2][kCols];
+  load_state<DP>(S, state, p, rl, c_first + c_local, s.start > 0);
+  // outputs: eight columns of a token a thread, where they are a power of two
+  const int lanes = p.vdim / 8;
+  const T* gate = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
+  T* out = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
+  const float* w = p.norm + (long long)h * p.norm_step;
+
+  for (int it = 0; it < tiles; ++it) {
+    const int t0 = it * kTT, nt = min(kTT, s.n - t0);
+    copies_wait<STAGES - 2>();
+    __syncthreads();       // the tile's record is there; the stage of the tile before is free
+    fetch(it + STAGES - 1);
+    float* st = sm + it % STAGES * stage_size;
+    const float* sB = st + R::kKeys;
+    const float* sC = st + R::kQ;
+    const float* sA = st + R::kA;
+    const float* dotB = st + R::kDotB;
+    const float* dotC = st + R::kDotC;
+    float* sV = st + R::kV;
+    const bool strong = st[R::kStrong] != 0.f;
+    float4 g0 = make_float4(0.f, 0.f, 0.f, 0.f), g1 = g0;
+    const int o_t = p.vec_out ? tid / lanes : 0, o_c = p.vec_out ? (tid - o_t * lanes) * 8 : 0;
+    if (p.vec_out && o_t < nt) {   // the first outputs' gates, ahead
+      g0 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
+      g1 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c + 4);
+    }
+    for (int q0 = 0; q0 < nt; q0 += kB) {
+      float2 acc[kKinds][kCols][kB];
+#pragma unroll
+      for (int e = 0; e < kKinds; ++e)
+#pragma unroll
+        for (int c = 0; c < kCols; ++c)
+#pragma unroll
+          for (int i = 0; i < kB; ++i) acc[e][c][i] = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < kChunks; ++j) {
+        const int r = j * 32 + rl * 4;
+#pragma unroll
+        for (int i = 0; i < kB; ++i) {
+          const float4 vc = load4(sC + (q0 + i) * DP + r);
+          if constexpr (DELTA) {
+            const float4 va = load4(sA + (q0 + i) * DP + r);
+#pragma unroll
+            for (int c = 0; c < kCols; ++c) {
+              fma2(acc[0][c][i], S[2 * j][c], make_float2(va.x, va.y));
+              fma2(acc[0][c][i], S[2 * j + 1][c], make_float2(va.z, va.w));
+            }
+          }
+#pragma unroll
+          for (int c = 0; c < kCols; ++c) {
+            fma2(acc[kKinds - 1][c][i], S[2 * j][c], make_float2(vc.x, vc.y));
+            fma2(acc[kKinds - 1][c][i], S[2 * j + 1][c], make_float2(vc.z, vc.w));
+          }
+        }
+      }
+      float my[kB];
+      const int my_c = reduce_columns<kKinds, kCols, kB>(acc, my);
+      // u of every token and column; o
+      float u[kB], U[kB][kCols];
+#pragma unroll
+      for (int i = 0; i < kB; ++i) {
+        u[i] = sV[(q0 + i) * nc + c_local + my_c];
+        if constexpr (DELTA) {
+          float x = u[i] - my[i];
+#pragma unroll
+          for (int j = 0; j < kB; ++j)
+            if (j < i) x = fmaf(-dotB[(q0 + i) * kB + j], u[j], x);
+          u[i] = st[R::kBeta + q0 + i] * x;   // (of use in lanes 0 - 3)
+        }
+      }
+      if constexpr (DELTA) {
+#pragma unroll
+        for (int i = 0; i < kB; ++i) {
+#pragma unroll
+          for (int c = 0; c < kCols; ++c) U[i][c] = __shfl_sync(0xffffffffu, u[i], (lane & 24) | c);
+          u[i] = __shfl_sync(0xffffffffu, u[i], (lane & 24) | my_c);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < kB; ++i)
+#pragma unroll
+          for (int c = 0; c < kCols; ++c) U[i][c] = sV[(q0 + i) * nc + c_local + c];
+      }
+      __syncwarp();   // the values of these tokens have been read: the outputs take their place
+#pragma unroll
+      for (int i = 0; i < kB; ++i) {
+        float o = my[i];
+#pragma unroll
+        for (int j = 0; j < kB; ++j)
+          if (j <= i) o = fmaf(dotC[(q0 + i) * kB + j], u[j], o);
+        if (rl >= 4 && rl < 4 + kCols) sV[(q0 + i) * nc + c_local + my_c] = o;
+      }
+      const bool renorm = strong || q0 + kB >= nt;
+      const float* ge = st + R::kG + (strong ? q0 / kB : kTT / kB - 1) * DP;
+#pragma unroll
+      for (int j = 0; j < kChunks; ++j) {
+        const int r = j * 32 + rl * 4;
+#pragma unroll
+        for (int i = 0; i < kB; ++i) {
+          const float4 b = load4(sB + (q0 + i) * DP + r);
+#pragma unroll
+          for (int c = 0; c < kCols; ++c) {
+            const float2 uu = make_float2(U[i][c], U[i][c]);
+            fma2(S[2 * j][c], make_float2(b.x, b.y), uu);
+            fma2(S[2 * j + 1][c], make_float2(b.z, b.w), uu);
+          }
+        }
+        if (renorm) {
+          const float4 g = load4(ge + r);
+#pragma unroll
+          for (int c = 0; c < kCols; ++c) {
+            mul2(S[2 * j][c], make_float2(g.x, g.y));
+            mul2(S[2 * j + 1][c], make_float2(g.z, g.w));
+          }
+        }
+      }
+    }
+    __syncthreads();   // the tile's outputs are there
+    if (p.raw != nullptr) {
+      for (int t = warp; t < nt; t += threads / 32) {
+        float* dst = p.raw + ((s.first + t0 + t) * p.heads + h) * p.raw_cols + c_first;
+        for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = sV[t * nc + c];
+        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = st[R::kBeta + t];
+      }
+    } else if (p.vec_out) {
+      // (whole warps: the lanes of a token lie in one)
+      for (int x = tid; x < (kTT * lanes + 31) / 32 * 32; x += threads) {
+        const int t = x / lanes, c = (x - t * lanes) * 8;
+        const bool ok = t < nt;
+        const float* o = sV + (ok ? t : 0) * nc;
+        if (x != tid && ok) {
+          g0 = load4(gate + (long long)(t0 + t) * p.ld_gate + c);
+          g1 = load4(gate + (long long)(t0 + t) * p.ld_gate + c + 4);
+        }
+        const float4 a = load4(o + c), b = load4(o + c + 4);
+        float f = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), st[R::kBeta + (ok ? t : 0)]) + 1e-6f);
+        float ss = dot4(a, a, dot4(b, b, 0.f)) * f * f;
+        for (int k = lanes / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+        f *= 1.f / sqrtf(ss / (float)p.vdim + p.eps);
+        if (!ok) continue;
+        const float4 wa = load4(w + c), wb = load4(w + c + 4);
+        T* dst = out + (long long)(t0 + t) * p.ldo + c;
+        store4(dst, make_float4(a.x * f * wa.x * sigmoid_f(g0.x), a.y * f * wa.y * sigmoid_f(g0.y),
+                                a.z * f * wa.z * sigmoid_f(g0.z), a.w * f * wa.w * sigmoid_f(g0.w)));
+        store4(dst + 4, make_float4(b.x * f * wb.x * sigmoid_f(g1.x), b.y * f * wb.y * sigmoid_f(g1.y),
+                                    b.z * f * wb.z * sigmoid_f(g1.z), b.w * f * wb.w * sigmoid_f(g1.w)));
+      }
+    } else {
+      for (int t = warp; t < nt; t += threads / 32)
+        head_output<T, DELTA>(p, sV + t * nc, s.first + t0 + t, h, st[R::kBeta + t]);
+    }
+  }
+  copies_wait<0>();
+  store_state<DP>(S, state, p, rl, c_first + c_local);
 }
 
 // Heads whose columns several blocks share: norm, weight and gate of the raw outputs. A warp per
@@ -619,53 +982,62 @@ __global__ void __launch_bounds__(256) scan_output_kernel(const ScanArgs p, long
   pdl_wait();
   pdl_trigger();
   const long long k = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
   if (k >= n) return;
-  const long long row = k / p.heads;
-  const int h = (int)(k - row * p.heads);
   const float* o = p.raw + k * p.raw_cols;
-  float scale = 1.f, ss = 0.f;
-  if (!DELTA) scale = 1.f / (fmaxf(fabsf(o[p.vdim]), o[p.vdim + 1]) + 1e-6f);
-  for (int c = lane; c < p.vdim; c += 32) {
-    const float x = o[c] * scale;
-    ss = fmaf(x, x, ss);
-  }
-  scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
-  const T* g = reinterpret_cast<const T*>(p.gate) + row * p.ld_gate + (long long)h * p.vdim;
-  const float* w = p.norm + (long long)h * p.norm_step;
-  T* dst = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
-  for (int c = lane; c < p.vdim; c += 32)
-    dst[c] = from_f32<T>(o[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
+  head_output<T, DELTA>(p, o, k / p.heads, (int)(k % p.heads), DELTA ? 0.f : o[p.vdim + 1]);
 }
 
-template <typename T, int DP, int TT, int B, bool DELTA>
-static int launch_scan(ScanArgs a, int n_seq, cudaStream_t stream) {
+template <typename K>
+static bool set_smem(K k, size_t bytes) {
+  return bytes <= 40 * 1024 ||
+         cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess;
+}
+
+template <typename T, int DP, bool DELTA>
+static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, cudaStream_t stream) {
   constexpr int wc = ScanShape<DP>::kWarpCols;
-  a.nc = (a.ncols + a.slices - 1) / a.slices;
-  a.nc = (a.nc + wc - 1) / wc * wc;
-  if (a.nc / wc > kScanMaxWarps || (long long)a.nc * (a.slices - 1) >= a.ncols) return -2;
-  const size_t smem = (size_t)ScanSmem<DP, TT, B, DELTA>::total(a.nc) * sizeof(float);
-  if (smem > 220 * 1024) return -6;
-  auto k = scan_kernel<T, DP, TT, B, DELTA>;
-  if (smem > 48 * 1024 &&
-      cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
-    return -3;
+  if (a.nc % wc || a.nc / wc > max_warps(DELTA) || (long long)a.nc * (a.slices - 1) >= a.ncols ||
+      (long long)a.nc * a.slices < a.ncols)
+    return -2;
   const long long blocks = (long long)n_seq * a.heads * a.slices;
-  if (blocks > 0x7fffffffll) return -6;
-  return launch_pdl(k, dim3((unsigned)blocks), dim3(a.nc / wc * 32), smem, stream, a) == cudaSuccess ? 0 : -5;
+  const dim3 threads(a.nc / wc * 32);
+  if (blocks > 0x7fffffffll || (long long)n_tiles * a.heads > 0x7fffffffll) return -6;
+  if (max_rows == 1) {
+    const size_t smem = (size_t)(3 * DP + a.nc) * sizeof(float);
+    return launch_pdl(step_kernel<T, DP, DELTA>, dim3((unsigned)blocks), threads, smem, stream, a) ==
+                   cudaSuccess
+               ? 0
+               : -5;
+  }
+  if (n_tiles < 1 || a.records == nullptr || a.tiles == nullptr || a.first_tile == nullptr ||
+      a.record < stage_floats<DP, DELTA>(a.nc * a.slices))
+    return -2;
+  if (!DELTA && launch_pdl(memory_gates_kernel<T>, dim3((unsigned)(n_seq * a.heads)),
+                           dim3(max_rows <= 128 ? 128 : max_rows <= 512 ? 512 : 1024), 0, stream,
+                           a) != cudaSuccess)
+    return -5;
+  const size_t tile_smem = (size_t)(DELTA ? 3 : 2) * kTT * DP * sizeof(float);
+  if (!set_smem(tile_kernel<T, DP, DELTA>, tile_smem)) return -3;
+  if (launch_pdl(tile_kernel<T, DP, DELTA>, dim3((unsigned)(n_tiles * a.heads)),
+                 dim3(DP <= 128 ? 128 : 256), tile_smem, stream, a) != cudaSuccess)
+    return -5;
+  const size_t stage = (size_t)stage_floats<DP, DELTA>(a.nc) * sizeof(float);
+  const bool three = 3 * stage <= 220 * 1024;
+  auto k = three ? scan_kernel<T, DP, DELTA, 3> : scan_kernel<T, DP, DELTA, 2>;
+  const size_t smem = (three ? 3 : 2) * stage;
+  if (smem > 220 * 1024) return -6;
+  if (!set_smem(k, smem)) return -3;
+  return launch_pdl(k, dim3((unsigned)blocks), threads, smem, stream, a) == cudaSuccess ? 0 : -5;
 }
 
 template <typename T, bool DELTA>
-static int run_scan(ScanArgs a, int n_seq, int max_rows, long long rows, cudaStream_t stream) {
-  int rc = -6;
-#define AB200_SCAN(DP)                                                             \
-  rc = max_rows == 1 ? launch_scan<T, DP, 1, 1, DELTA>(a, n_seq, stream)           \
-                     : launch_scan<T, DP, 16, 4, DELTA>(a, n_seq, stream)
-  if (a.dim <= 32) AB200_SCAN(32);
-  else if (a.dim <= 64) AB200_SCAN(64);
-  else if (a.dim <= 128) AB200_SCAN(128);
-  else if (a.dim <= 256) AB200_SCAN(256);
-#undef AB200_SCAN
+static int run_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, long long rows,
+                    cudaStream_t stream) {
+  const int rc = a.dim <= 32    ? launch_scan<T, 32, DELTA>(a, n_seq, n_tiles, max_rows, stream)
+                 : a.dim <= 64  ? launch_scan<T, 64, DELTA>(a, n_seq, n_tiles, max_rows, stream)
+                 : a.dim <= 128 ? launch_scan<T, 128, DELTA>(a, n_seq, n_tiles, max_rows, stream)
+                 : a.dim <= 256 ? launch_scan<T, 256, DELTA>(a, n_seq, n_tiles, max_rows, stream)
+                                : -6;
   if (rc != 0 || a.raw == nullptr) return rc;
   const long long n = rows * a.heads;
   return launch_pdl(scan_output_kernel<T, DELTA>, dim3((unsigned)((n + 7) / 8)), dim3(256), 0, stream, a,
@@ -678,6 +1050,25 @@ static int aligned4(const void* p, long long ld, int dtype) {
   return ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p) & (dtype == 0 ? 7 : 15)) == 0;
 }
 
+static int warp_cols(int dim) { return dim <= 128 ? 16 : 8; }
+
+// The common part of both entry points
+static void finish_args(ScanArgs& a, int slices, int ncols, int raw_cols, void* raw, int dtype) {
+  a.slices = slices;
+  a.ncols = ncols;
+  a.nc = (ncols + slices - 1) / slices;
+  a.nc = (a.nc + warp_cols(a.dim) - 1) / warp_cols(a.dim) * warp_cols(a.dim);
+  a.raw = slices > 1 ? reinterpret_cast<float*>(raw) : nullptr;
+  a.raw_cols = raw_cols;
+  a.q_scale = 1.f / sqrtf((float)a.dim);
+  const int lanes = a.vdim / 8;
+  a.vec_out = slices == 1 && a.vdim % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 &&
+              aligned4(a.gate, a.ld_gate, dtype) && aligned4(a.out, a.ldo, dtype) &&
+              aligned4(a.norm, a.norm_step, 1);
+  a.vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.q_at % 4 == 0 && a.k_at % 4 == 0 && a.v_at % 4 == 0 &&
+          aligned4(a.proj, a.ld, dtype) && aligned4(a.conv_state, 0, dtype) && aligned4(a.conv, 0, 1);
+}
+
 }  // namespace ab200
 
 using namespace ab200;
@@ -686,22 +1077,33 @@ typedef __nv_bfloat16 bf16;
 extern "C" {
 
 // Blocks per head so that each block's columns fit: 0 if dim is beyond the kernel's.
-int ab200_scan_min_slices(int dim, int ncols) {
+int ab200_scan_min_slices(int dim, int ncols, int delta) {
   if (dim < 1 || dim > 256) return 0;
-  const int most = kScanMaxWarps * (dim <= 128 ? 16 : 8);
+  const int most = max_warps(delta != 0) * warp_cols(dim);
   return (ncols + most - 1) / most;
+}
+
+// Floats of a tile's record of a head (portions of more than one token).
+long long ab200_scan_record(int dim, int ncols, int slices, int delta) {
+  const int wc = warp_cols(dim), nc = ((ncols + slices - 1) / slices + wc - 1) / wc * wc;
+  const int dp = dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256;
+  const int vectors = delta ? 3 * kTT + kTT / kB : 2 * kTT + kTT / kB;
+  return (long long)vectors * dp + 2 * kTT * kB + kTT + 4 + (long long)kTT * nc * slices;
 }
 
 // Gated delta rule over n_seq sequences. proj [T, ld]: query and key heads of dim at q_at, k_at, value
 // heads of vdim at v_at, step sizes at b_at. steps int32 [n_seq, 5]: first row, rows, slot (0: padding),
-// start position, phase. raw fp32 [T, heads, vdim] when slices > 1. See ScanArgs.
+// start position, phase. When max_rows > 1: tiles int32 [n_tiles, 2] and first_tile int32 [n_seq] cut the
+// sequences into tiles of 16 tokens, records fp32 [n_tiles, heads, ab200_scan_record]. raw fp32
+// [T, heads, vdim] when slices > 1. See ScanArgs.
 int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int b_at,
                      const void* decay, long long ld_decay, const void* gate, long long ld_gate,
                      const void* conv, int taps, const void* a_exp, const void* dt_bias,
                      const void* norm, void* state, int state_cols, void* conv_state, int num_slots,
-                     const void* steps, int n_seq, int max_rows, long long T, int heads, int kv_heads,
-                     int dim, int vdim, int slices, float eps, void* raw, void* out, long long ldo,
-                     int dtype, int* status, cudaStream_t stream) {
+                     const void* steps, int n_seq, int max_rows, const void* tiles,
+                     const void* first_tile, int n_tiles, void* records, long long T, int heads,
+                     int kv_heads, int dim, int vdim, int slices, float eps, void* raw, void* out,
+                     long long ldo, int dtype, int* status, cudaStream_t stream) {
   if (T <= 0 || n_seq <= 0) return 0;
   if (heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || taps < 1 || slices < 1 ||
       state_cols < vdim || state_cols % 4 || (slices > 1 && raw == nullptr))
@@ -720,34 +1122,34 @@ int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_a
   a.conv_state = conv_state;
   a.num_slots = num_slots;
   a.steps = reinterpret_cast<const int*>(steps);
-  a.heads = heads; a.group = heads / kv_heads; a.dim = dim; a.vdim = vdim; a.ncols = vdim;
+  a.tiles = reinterpret_cast<const int*>(tiles);
+  a.first_tile = reinterpret_cast<const int*>(first_tile);
+  a.records = reinterpret_cast<float*>(records);
+  a.record = ab200_scan_record(dim, vdim, slices, 1);
+  a.heads = heads; a.group = heads / kv_heads; a.dim = dim; a.vdim = vdim;
   a.taps = taps;
   a.channels = 2 * kv_heads * dim + heads * vdim;
-  a.slices = slices;
-  a.q_scale = 1.f / sqrtf((float)dim);
   a.eps = eps;
-  a.raw = slices > 1 ? reinterpret_cast<float*>(raw) : nullptr;
-  a.raw_cols = vdim;
   a.out = out; a.ldo = ldo;
   a.status = status;
-  a.vec = dim % 4 == 0 && vdim % 4 == 0 && q_at % 4 == 0 && k_at % 4 == 0 && v_at % 4 == 0 &&
-          aligned4(proj, ld, dtype) && aligned4(conv_state, 0, dtype) && aligned4(conv, 0, 1);
-  return dtype == 0 ? run_scan<bf16, true>(a, n_seq, max_rows, T, stream)
-                    : run_scan<float, true>(a, n_seq, max_rows, T, stream);
+  finish_args(a, slices, vdim, vdim, raw, dtype);
+  return dtype == 0 ? run_scan<bf16, true>(a, n_seq, n_tiles, max_rows, T, stream)
+                    : run_scan<float, true>(a, n_seq, n_tiles, max_rows, T, stream);
 }
 
 // Matrix memory: query and key heads of dim, value heads of vdim, gates at i_at and f_at; state
 // [slots, heads, dim, state_cols] with the normaliser in column vdim; max_state fp32 [slots, 2, heads];
-// raw fp32 [T, heads, vdim + 2] when slices > 1.
+// gates fp32 [T, heads, 3] when max_rows > 1; raw fp32 [T, heads, vdim + 2] when slices > 1.
 int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int i_at, int f_at,
                       const void* gate, long long ld_gate, const void* i_bias, const void* f_bias,
                       float cap, const void* norm, void* state, int state_cols, void* max_state,
-                      int num_slots, const void* steps, int n_seq, int max_rows, long long T, int heads,
-                      int dim, int vdim, int slices, float eps, void* raw, void* out, long long ldo,
-                      int dtype, int* status, cudaStream_t stream) {
+                      int num_slots, const void* steps, int n_seq, int max_rows, const void* tiles,
+                      const void* first_tile, int n_tiles, void* records, void* gates, long long T,
+                      int heads, int dim, int vdim, int slices, float eps, void* raw, void* out,
+                      long long ldo, int dtype, int* status, cudaStream_t stream) {
   if (T <= 0 || n_seq <= 0) return 0;
   if (heads < 1 || dim < 1 || vdim < 1 || slices < 1 || state_cols < vdim + 1 || state_cols % 4 ||
-      !(cap > 0.f) || (slices > 1 && raw == nullptr))
+      !(cap > 0.f) || (slices > 1 && raw == nullptr) || (max_rows > 1 && gates == nullptr))
     return -2;
   ScanArgs a = {};
   a.proj = proj; a.ld = ld;
@@ -763,19 +1165,19 @@ int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_
   a.max_state = reinterpret_cast<float*>(max_state);
   a.num_slots = num_slots;
   a.steps = reinterpret_cast<const int*>(steps);
-  a.heads = heads; a.group = 1; a.dim = dim; a.vdim = vdim; a.ncols = vdim + 1;
+  a.tiles = reinterpret_cast<const int*>(tiles);
+  a.first_tile = reinterpret_cast<const int*>(first_tile);
+  a.records = reinterpret_cast<float*>(records);
+  a.record = ab200_scan_record(dim, vdim + 1, slices, 0);
+  a.gates = reinterpret_cast<float*>(gates);
+  a.heads = heads; a.group = 1; a.dim = dim; a.vdim = vdim;
   a.taps = 1;
-  a.slices = slices;
-  a.q_scale = 1.f / sqrtf((float)dim);
   a.eps = eps;
-  a.raw = slices > 1 ? reinterpret_cast<float*>(raw) : nullptr;
-  a.raw_cols = vdim + 2;
   a.out = out; a.ldo = ldo;
   a.status = status;
-  a.vec = dim % 4 == 0 && vdim % 4 == 0 && q_at % 4 == 0 && k_at % 4 == 0 && v_at % 4 == 0 &&
-          aligned4(proj, ld, dtype);
-  return dtype == 0 ? run_scan<bf16, false>(a, n_seq, max_rows, T, stream)
-                    : run_scan<float, false>(a, n_seq, max_rows, T, stream);
+  finish_args(a, slices, vdim + 1, vdim + 2, raw, dtype);
+  return dtype == 0 ? run_scan<bf16, false>(a, n_seq, n_tiles, max_rows, T, stream)
+                    : run_scan<float, false>(a, n_seq, n_tiles, max_rows, T, stream);
 }
 
 }  // extern "C"

@@ -127,11 +127,12 @@ def _declare(L: ctypes.CDLL) -> None:
         "ab200_stream_norm": (I, [P, P, P, LL, P, P, I, P, F, F, F, P, P, LL, I, I, P]),
         "ab200_stream_sandwich": (I, [P, P, LL, P, P, P, P, F, F, LL, I, I, P]),
         "ab200_stream_add": (I, [P, P, P, P, LL, P, P, LL, P, P, P, I, P, LL, F, LL, I, I, P]),
-        "ab200_scan_min_slices": (I, [I, I]),
-        "ab200_delta_scan": (I, [P, LL, I, I, I, I, P, LL, P, LL, P, I, P, P, P, P, I, P, I, P, I, I, LL,
-                                 I, I, I, I, I, F, P, P, LL, I, P, P]),
-        "ab200_memory_scan": (I, [P, LL, I, I, I, I, I, P, LL, P, P, F, P, P, I, P, I, P, I, I, LL, I, I,
-                                  I, I, F, P, P, LL, I, P, P]),
+        "ab200_scan_min_slices": (I, [I, I, I]),
+        "ab200_scan_record": (LL, [I, I, I, I]),
+        "ab200_delta_scan": (I, [P, LL, I, I, I, I, P, LL, P, LL, P, I, P, P, P, P, I, P, I, P, I, I, P, P,
+                                 I, P, LL, I, I, I, I, I, F, P, P, LL, I, P, P]),
+        "ab200_memory_scan": (I, [P, LL, I, I, I, I, I, P, LL, P, P, F, P, P, I, P, I, P, I, I, P, P, I, P,
+                                  P, LL, I, I, I, I, F, P, P, LL, I, P, P]),
         "ab200_latent_norm_cache": (I, [P, LL, P, I, I, F, P, P, LL, LL, I, P, P]),
         "ab200_gated_act": (I, [P, P, LL, I, I, F, F, I, P]),
         "ab200_linear_exact": (I, [P, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P]),

@@ -17,6 +17,7 @@ from . import launch_counter, upload
 from .stream_ops import dtype_code
 
 STEP_INTS = 5       # first row, rows, slot, start position, phase (csrc/recurrent.cu)
+TILE_ROWS = 16      # tokens that portions are prepared by
 
 
 def _nat():
@@ -39,6 +40,23 @@ class StateStep:
     state, write none, and put out zeros."""
     table: torch.Tensor       # int32 [n, STEP_INTS]
     max_rows: int             # most rows of a sequence
+    # steps with longer portions: the sequences cut into tiles of TILE_ROWS tokens
+    tiles: torch.Tensor = None        # int32 [tiles, 2]: sequence, first of its tokens
+    first_tile: torch.Tensor = None   # int32 [n]
+
+    @staticmethod
+    def build(table: np.ndarray, device) -> "StateStep":
+        n, rows = table.shape[0], table[:, 1].astype(np.int64)
+        if rows.max() == 1:
+            return StateStep(upload(table, device), 1)
+        count = -(-rows // TILE_ROWS)
+        first = np.cumsum(count) - count
+        seq = np.repeat(np.arange(n), count)
+        tiles = np.stack([seq, (np.arange(seq.size) - first[seq]) * TILE_ROWS], 1)
+        packed = upload(np.concatenate([table.ravel(), tiles.ravel(), first]).astype(np.int32), device)
+        a, b = table.size, table.size + tiles.size
+        return StateStep(packed[:a].view(n, STEP_INTS), int(rows.max()), packed[a:b].view(-1, 2),
+                         packed[b:])
 
     @staticmethod
     def of(scheduled, q_lens, pad_rows: int, device) -> "StateStep":
@@ -47,11 +65,11 @@ class StateStep:
         pack_steps(scheduled, q_lens, t)
         if pad_rows:
             t[n] = (sum(q_lens), pad_rows, 0, 0, 0)
-        return StateStep(upload(t, device), max(max(q_lens), pad_rows))
+        return StateStep.build(t, device)
 
     @property
     def uploaded_bytes(self) -> int:
-        return self.table.numel() * 4
+        return 4 * sum(t.numel() for t in (self.table, self.tiles, self.first_tile) if t is not None)
 
 
 class StateDecodePlan:
@@ -80,19 +98,31 @@ class StateDecodePlan:
         self._host[:, 2] = 0
 
 
-def slices_for(dim: int, ncols: int, blocks: int, long: bool) -> int:
+def slices_for(dim: int, ncols: int, delta: bool, blocks: int, long: bool) -> int:
     """Blocks that share a head's columns: as few as hold them, more where a prompt's few heads
     would leave most of the GPU idle."""
-    least = _nat().lib().ab200_scan_min_slices(dim, ncols)
+    least = _nat().lib().ab200_scan_min_slices(dim, ncols, int(delta))
     if least == 0:
         raise NotImplementedError("recurrent layers with keys of more than 256 dimensions")
     width = 16 if dim <= 128 else 8
     most = -(-ncols // width)
-    want = -(-148 // max(1, blocks)) if long else 1
+    want = 148 // max(1, blocks) if long else 1
     n = max(least, min(most, want))
     # blocks of whole warps: as many as the columns then take
     cols = -(-(-(-ncols // n)) // width) * width
     return -(-ncols // cols)
+
+
+def _scratch(s, ncols: int, delta: bool, steps: StateStep, T: int, device):
+    """(slices, raw outputs or None, tile records or None) of a scan."""
+    slices = slices_for(s.dim, ncols, delta, steps.table.shape[0] * s.heads, steps.max_rows > 1)
+    f32 = dict(dtype=torch.float32, device=device)
+    raw = torch.empty(T, s.heads, ncols + (not delta), **f32) if slices > 1 else None
+    records = None
+    if steps.max_rows > 1:
+        size = _nat().lib().ab200_scan_record(s.dim, ncols, slices, int(delta))
+        records = torch.empty(steps.tiles.shape[0], s.heads, size, **f32)
+    return slices, raw, records
 
 
 # ------------------------------------------------------------------------------ delta rule
@@ -174,21 +204,20 @@ def delta_scan(proj, decay, gate, conv, a_exp, dt_bias, norm, s: DeltaShape, sta
     nat = _nat()
     T, n = proj.shape[0], steps.table.shape[0]
     out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
-    slices = slices_for(s.dim, s.vdim, n * s.heads, steps.max_rows > 1)
-    raw = torch.empty(T, s.heads, s.vdim, dtype=torch.float32, device=proj.device) \
-        if slices > 1 else None
+    slices, raw, records = _scratch(s, s.vdim, True, steps, T, proj.device)
     assert proj.stride(1) == decay.stride(1) == gate.stride(1) == 1
     assert state.is_contiguous() and conv_state.is_contiguous() and steps.table.is_contiguous()
     rc = nat.lib().ab200_delta_scan(
         proj.data_ptr(), proj.stride(0), s.q_at, s.k_at, s.v_at, s.b_at, decay.data_ptr(),
         decay.stride(0), gate.data_ptr(), gate.stride(0), conv.data_ptr(), s.taps, a_exp.data_ptr(),
         dt_bias.data_ptr(), norm.data_ptr(), state.data_ptr(), state.shape[3],
-        conv_state.data_ptr(), state.shape[0], steps.table.data_ptr(), n, steps.max_rows, T,
-        s.heads, s.kv_heads, s.dim, s.vdim, slices, float(eps), nat.ptr(raw), out.data_ptr(),
+        conv_state.data_ptr(), state.shape[0], steps.table.data_ptr(), n, steps.max_rows,
+        nat.ptr(steps.tiles), nat.ptr(steps.first_tile),
+        steps.tiles.shape[0] if records is not None else 0, nat.ptr(records), T, s.heads, s.kv_heads, s.dim, s.vdim, slices, float(eps), nat.ptr(raw), out.data_ptr(),
         out.stride(0), dtype_code(proj.dtype), nat.status_buffer(proj.device).data_ptr(),
         nat.stream_ptr())
     nat.check(rc, "delta_scan")
-    launch_counter.add(2 if slices > 1 else 1)
+    launch_counter.add(1 + (slices > 1) + (records is not None))
     return out
 
 
@@ -254,18 +283,20 @@ def memory_scan(proj, gate, i_bias, f_bias, norm, s: MemoryShape, state, max_sta
     nat = _nat()
     T, n = proj.shape[0], steps.table.shape[0]
     out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
-    slices = slices_for(s.dim, s.vdim + 1, n * s.heads, steps.max_rows > 1)
-    raw = torch.empty(T, s.heads, s.vdim + 2, dtype=torch.float32, device=proj.device) \
-        if slices > 1 else None
+    slices, raw, records = _scratch(s, s.vdim + 1, False, steps, T, proj.device)
+    gates = torch.empty(T, s.heads, 3, dtype=torch.float32, device=proj.device) \
+        if records is not None else None
     assert proj.stride(1) == gate.stride(1) == 1
     assert state.is_contiguous() and max_state.is_contiguous() and steps.table.is_contiguous()
     rc = nat.lib().ab200_memory_scan(
         proj.data_ptr(), proj.stride(0), s.q_at, s.k_at, s.v_at, s.i_at, s.f_at, gate.data_ptr(),
         gate.stride(0), i_bias.data_ptr(), f_bias.data_ptr(), float(s.cap), norm.data_ptr(),
         state.data_ptr(), state.shape[3], max_state.data_ptr(), state.shape[0],
-        steps.table.data_ptr(), n, steps.max_rows, T, s.heads, s.dim, s.vdim, slices, float(eps),
+        steps.table.data_ptr(), n, steps.max_rows, nat.ptr(steps.tiles), nat.ptr(steps.first_tile),
+        steps.tiles.shape[0] if records is not None else 0, nat.ptr(records), nat.ptr(gates), T,
+        s.heads, s.dim, s.vdim, slices, float(eps),
         nat.ptr(raw), out.data_ptr(), out.stride(0), dtype_code(proj.dtype),
         nat.status_buffer(proj.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "memory_scan")
-    launch_counter.add(2 if slices > 1 else 1)
+    launch_counter.add(1 + (slices > 1) + 2 * (records is not None))
     return out

@@ -136,7 +136,7 @@ def test_every_run_has_its_own_cache_and_state(tmp_path):
 
 # ---------------------------------------------------------------- mechanisms by themselves
 def step_of(table):
-    return states.StateStep(torch.tensor(table, dtype=torch.int32), max(r[1] for r in table))
+    return states.StateStep.build(np.asarray(table, dtype=np.int32), "cpu")
 
 
 def delta_case(H, G, d, dv, taps, lens, seed=0):

@@ -1,6 +1,7 @@
 """Pererax on a GPU: each kernel against the fp64 restatement, then the model through the engine's
 step function, captured decode steps and scheduler."""
 
+import numpy as np
 import pytest
 import torch
 
@@ -41,8 +42,7 @@ def steps_of(lens, cuts, slots):
                 table.append((len(rows), n, slots[i], at[i], phase[i]))
                 rows += range(base[i] + at[i], base[i] + at[i] + n)
                 at[i], phase[i] = at[i] + n, phase[i] ^ 1
-        yield rows, states.StateStep(torch.tensor(table, dtype=torch.int32, device=DEV),
-                                     max(r[1] for r in table))
+        yield rows, states.StateStep.build(np.asarray(table, dtype=np.int32), DEV)
     assert at == list(lens)
 
 
@@ -129,8 +129,8 @@ def test_padding_rows_put_out_zeros(rows):
     dev = lambda t: t.to(DEV)
     state = torch.ones(2, H, d, s.state_cols, device=DEV)
     conv = torch.ones(2, 2, taps - 1, s.channels, device=DEV)
-    step = states.StateStep(torch.tensor([(0, rows, 1, 0, 0), (rows, rows, 0, 0, 0)], device=DEV,
-                                         dtype=torch.int32), rows)
+    step = states.StateStep.build(np.asarray([(0, rows, 1, 0, 0), (rows, rows, 0, 0, 0)],
+                                             dtype=np.int32), DEV)
     out = states.delta_scan(dev(proj), dev(decay), dev(gate), *map(dev, w.values()), s, state, conv,
                             step, 0.01)
     assert float(out[rows:].abs().max()) == 0 < float(out[:rows].abs().max())
@@ -145,7 +145,7 @@ def test_the_split_of_a_head_does_not_matter():
     for blocks in (1, 1000):      # as one block per head, or as many as its columns allow
         state = torch.zeros(2, H, d, s.state_cols, device=DEV)
         conv = torch.zeros(2, 2, taps - 1, s.channels, device=DEV)
-        step = states.StateStep(torch.tensor([(0, 70, 1, 0, 0)], device=DEV, dtype=torch.int32), 70)
+        step = states.StateStep.build(np.asarray([(0, 70, 1, 0, 0)], dtype=np.int32), DEV)
         saved, states.slices_for = states.slices_for, lambda *a: 1 if blocks == 1 else 8
         try:
             outs.append((states.delta_scan(*(t.to(DEV) for t in (proj, decay, gate, *w.values())), s,
