@@ -289,8 +289,8 @@ int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, 
                       long long T, int W, int top, int experts, int dtype, cudaStream_t stream);
 
 // ---- recurrent.cu
-int ab200_scan_min_slices(int dim, int ncols, int delta);
-long long ab200_scan_record(int dim, int ncols, int slices, int delta);
+int ab200_scan_min_slices(int dim, int ncols, int delta, int dtype, int several);
+long long ab200_scan_record(int dim, int ncols, int slices, int delta, int dtype);
 int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int b_at,
                      const void* decay, long long ld_decay, const void* gate, long long ld_gate,
                      const void* conv, int taps, const void* a_exp, const void* dt_bias,

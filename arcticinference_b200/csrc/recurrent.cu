@@ -26,6 +26,13 @@
 // where Z is the one before the group. G goes back to 1 at a tile's end, and after every group when a
 // channel decays so much within the tile that 1 / G would leave fp32's range.
 //
+// For 16-bit models the products of a tile run on the tensor cores (mma.sync: Z lives in the registers
+// of the warps that own its columns, as the accumulator of the update and, converted in place, as the
+// left operand of the read-outs; nothing but the small token-side operands passes through shared
+// memory). Every operand is the sum of two bf16 numbers, so that products carry 16 significant bits,
+// and sums and Z are fp32. The 16 tokens are then one group, solved with the inverse of the unit
+// triangular matrix that the tile's a, b and beta form. 32-bit models use fp32 multiply-adds.
+//
 // What a sequence carries over lies in its slot: S in fp32; the convolution's last inputs and m twice,
 // for even and odd steps of the sequence (`phase`), so that blocks which read them never race with the
 // block that writes them. A sequence that starts at position 0 reads nothing from its slot.
@@ -78,6 +85,7 @@ struct ScanArgs {
   int raw_cols;
   int num_slots, heads, group, dim, vdim, ncols, taps, channels;
   int slices, nc;            // blocks per head, columns of each
+  int warp_cols;             // columns of a warp
   int vec;                   // four channels at a time are aligned
   int vec_out;               // eight output columns at a time are aligned, a power of two of them
   float q_scale, cap, eps;
@@ -124,6 +132,47 @@ __device__ __forceinline__ void axpy4(float4& y, const float4& w, const float4& 
 }
 __device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
   return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
+}
+// D[16 x 8] += A[16 x 16] B[16 x 8], bf16 operands: lane (g = lane / 4, t = lane % 4) holds D's rows g
+// and g + 8, columns 2 t and 2 t + 1; A's a0 (g, 2 t ..), a1 (g + 8, 2 t ..), a2, a3 eight columns
+// further; B's b0 (rows 2 t .., column g), b1 eight rows further
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void load_matrices(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void load_matrices_trans(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+// x and y as sums of two bf16 numbers each
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x, y);
+  lo = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+}
+// An accumulator pair [16 x 16] as a left operand
+__device__ __forceinline__ void split_left(const float (&d0)[4], const float (&d1)[4], uint32_t (&hi)[4],
+                                           uint32_t (&lo)[4]) {
+  split2(d0[0], d0[1], hi[0], lo[0]);
+  split2(d0[2], d0[3], hi[1], lo[1]);
+  split2(d1[0], d1[1], hi[2], lo[2]);
+  split2(d1[2], d1[3], hi[3], lo[3]);
+}
+// d[n] += (hi + lo) (bh + bl), n = 0, 1: right operands' registers 2 n, 2 n + 1
+__device__ __forceinline__ void mma_split(float (&d)[2][4], const uint32_t (&hi)[4], const uint32_t (&lo)[4],
+                                          const uint32_t (&bh)[4], const uint32_t (&bl)[4]) {
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    mma_bf16(d[n], hi, bl[2 * n], bl[2 * n + 1]);
+    mma_bf16(d[n], lo, bh[2 * n], bh[2 * n + 1]);
+    mma_bf16(d[n], hi, bh[2 * n], bh[2 * n + 1]);
+  }
 }
 // log gates of the matrix memory
 __device__ __forceinline__ float2 memory_log_gates(float zi, float zf, float cap) {
@@ -342,6 +391,36 @@ __device__ __forceinline__ void head_output(const ScanArgs& p, const float* o, l
   scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
   for (int c = lane; c < p.vdim; c += 32)
     dst[c] = from_f32<T>(o[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
+}
+
+// A block's tile: the same eight columns a thread, the `lanes` lanes of a token side by side. g0, g1: the
+// gate of the thread's first columns.
+template <typename T, bool DELTA>
+__device__ __forceinline__ void vector_outputs(const ScanArgs& p, const float* o_tile, int ld, const float* floors,
+                                               int nt, int lanes, const T* gate, T* out, const float* w,
+                                               float4 g0, float4 g1) {
+  // (whole warps: the lanes of a token lie in one)
+  for (int x = threadIdx.x; x < (kTT * lanes + 31) / 32 * 32; x += blockDim.x) {
+    const int t = x / lanes, c = (x - t * lanes) * 8;
+    const bool ok = t < nt;
+    const float* o = o_tile + (ok ? t : 0) * ld;
+    if (x != threadIdx.x && ok) {
+      g0 = load4(gate + t * p.ld_gate + c);
+      g1 = load4(gate + t * p.ld_gate + c + 4);
+    }
+    const float4 a = load4(o + c), b = load4(o + c + 4);
+    float f = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floors[ok ? t : 0]) + 1e-6f);
+    float ss = dot4(a, a, dot4(b, b, 0.f)) * f * f;
+    for (int k = lanes / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    f *= 1.f / sqrtf(ss / (float)p.vdim + p.eps);
+    if (!ok) continue;
+    const float4 wa = load4(w + c), wb = load4(w + c + 4);
+    T* dst = out + t * p.ldo + c;
+    store4(dst, make_float4(a.x * f * wa.x * sigmoid_f(g0.x), a.y * f * wa.y * sigmoid_f(g0.y),
+                            a.z * f * wa.z * sigmoid_f(g0.z), a.w * f * wa.w * sigmoid_f(g0.w)));
+    store4(dst + 4, make_float4(b.x * f * wb.x * sigmoid_f(g1.x), b.y * f * wb.y * sigmoid_f(g1.y),
+                                b.z * f * wb.z * sigmoid_f(g1.z), b.w * f * wb.w * sigmoid_f(g1.w)));
+  }
 }
 
 // ------------------------------------------------------------------ one token per sequence
@@ -944,28 +1023,8 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
         if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = st[R::kBeta + t];
       }
     } else if (p.vec_out) {
-      // (whole warps: the lanes of a token lie in one)
-      for (int x = tid; x < (kTT * lanes + 31) / 32 * 32; x += threads) {
-        const int t = x / lanes, c = (x - t * lanes) * 8;
-        const bool ok = t < nt;
-        const float* o = sV + (ok ? t : 0) * nc;
-        if (x != tid && ok) {
-          g0 = load4(gate + (long long)(t0 + t) * p.ld_gate + c);
-          g1 = load4(gate + (long long)(t0 + t) * p.ld_gate + c + 4);
-        }
-        const float4 a = load4(o + c), b = load4(o + c + 4);
-        float f = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), st[R::kBeta + (ok ? t : 0)]) + 1e-6f);
-        float ss = dot4(a, a, dot4(b, b, 0.f)) * f * f;
-        for (int k = lanes / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
-        f *= 1.f / sqrtf(ss / (float)p.vdim + p.eps);
-        if (!ok) continue;
-        const float4 wa = load4(w + c), wb = load4(w + c + 4);
-        T* dst = out + (long long)(t0 + t) * p.ldo + c;
-        store4(dst, make_float4(a.x * f * wa.x * sigmoid_f(g0.x), a.y * f * wa.y * sigmoid_f(g0.y),
-                                a.z * f * wa.z * sigmoid_f(g0.z), a.w * f * wa.w * sigmoid_f(g0.w)));
-        store4(dst + 4, make_float4(b.x * f * wb.x * sigmoid_f(g1.x), b.y * f * wb.y * sigmoid_f(g1.y),
-                                    b.z * f * wb.z * sigmoid_f(g1.z), b.w * f * wb.w * sigmoid_f(g1.w)));
-      }
+      vector_outputs<T, DELTA>(p, sV, nc, st + R::kBeta, nt, lanes, gate + (long long)t0 * p.ld_gate,
+                               out + (long long)t0 * p.ldo, w, g0, g1);
     } else {
       for (int t = warp; t < nt; t += threads / 32)
         head_output<T, DELTA>(p, sV + t * nc, s.first + t0 + t, h, st[R::kBeta + t]);
@@ -973,6 +1032,464 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
   }
   copies_wait<0>();
   store_state<DP>(S, state, p, rl, c_first + c_local);
+}
+
+// ------------------------------------------------------------------ the same on tensor cores
+// A record, in bytes: a (delta), b and c as pairs of bf16 matrices [kTT][kLd], the solving matrix
+// (delta) and c . b as pairs [kTT][kLdT], decays, step sizes (memory: exp(-m)), values fp32 [kTT][vld].
+template <int DP, bool DELTA>
+struct MmaRecord {
+  static constexpr int kLd = DP + 8, kLdT = kTT + 8;    // rows shifted over the banks
+  static constexpr int kMat = kTT * kLd * 2, kSmall = kTT * kLdT * 2;
+  static constexpr int kB = 0, kC = 2 * kMat, kA = 4 * kMat, kQ = (DELTA ? 6 : 4) * kMat;
+  static constexpr int kT = kQ + 2 * kSmall, kG = kT + (DELTA ? 2 * kSmall : 0);
+  static constexpr int kBeta = kG + 4 * DP * 4, kStrong = kBeta + kTT * 4, kV = kStrong + 16;
+  __host__ __device__ static constexpr int vld(int cols) { return cols + 4; }
+  __host__ __device__ static constexpr int bytes(int cols) { return kV + kTT * vld(cols) * 4; }
+};
+
+template <int DP, bool DELTA>
+__global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const ScanArgs p) {
+  typedef __nv_bfloat16 T;
+  using R = MmaRecord<DP, DELTA>;
+  constexpr int kThreads = DP <= 128 ? 128 : 256, kWarps = kThreads / 32, kLd = R::kLd;
+  extern __shared__ __align__(16) float sm[];
+  float* sB = sm;                                // keys
+  float* sC = sm + kTT * DP;                     // queries
+  uint8_t* mats = reinterpret_cast<uint8_t*>(sm + 2 * kTT * DP);   // the record up to its values
+  float* tri = reinterpret_cast<float*>(mats + R::kV);             // [kTT][kTT + 1]
+  __shared__ float invQ[kTT], invK[kTT], beta[kTT];   // memory: log decay, log input factor, exp(-m)
+  pdl_wait();
+  pdl_trigger();
+  const int h = blockIdx.x % p.heads;
+  const long long tile = blockIdx.x / p.heads;
+  const int* tl = p.tiles + tile * 2;
+  const Seq s(p.steps + (long long)tl[0] * kStepInts);
+  if (s.slot <= 0 || s.slot >= p.num_slots) return;
+  const int t0 = tl[1], nt = min(kTT, s.n - t0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  uint8_t* rec = reinterpret_cast<uint8_t*>(p.records) + (tile * p.heads + h) * p.record * 4;
+  const Inputs<T> in(p, s, h, DELTA);
+  const int vcols = p.slices * p.nc, vld = R::vld(vcols);
+  float* rec_v = reinterpret_cast<float*>(rec + R::kV);
+
+  // Decays: a thread has two channels and eight of the tokens; lane ^ 16 has the others.
+  const int d0 = 2 * ((tid & 15) + (tid >> 5) * 16), half = (tid >> 4) & 1;
+  float2 z[8];
+  float2 bias = make_float2(0.f, 0.f);
+  float ae = 0.f;
+  if (DELTA) {
+#pragma unroll
+    for (int t = 0; t < 8; ++t) z[t] = make_float2(0.f, 0.f);
+    if (d0 < p.dim) {
+      const T* src = reinterpret_cast<const T*>(p.decay) + (s.first + t0 + half * 8) * p.ld_decay + h * p.dim + d0;
+      const bool two = d0 + 1 < p.dim;
+      ae = p.a_exp[h];
+      bias.x = p.dt_bias[h * p.dim + d0];
+      if (two) bias.y = p.dt_bias[h * p.dim + d0 + 1];
+      const int mine = nt - half * 8;
+      if (p.vec) {
+#pragma unroll
+        for (int t = 0; t < 8; ++t)
+          if (t < mine) z[t] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + t * p.ld_decay));
+      } else {
+        for (int t = 0; t < 8; ++t)
+          if (t < mine)
+            z[t] = make_float2(to_f32<T>(src[t * p.ld_decay]), two ? to_f32<T>(src[t * p.ld_decay + 1]) : 0.f);
+      }
+    }
+    if (tid < kTT)
+      beta[tid] = tid < nt ? sigmoid_f(to_f32<T>(in.proj[(long long)(t0 + tid) * p.ld + p.b_at + h])) : 0.f;
+  } else if (tid < kTT) {
+    const float* g = p.gates + ((s.first + t0 + tid) * p.heads + h) * 3;
+    const bool ok = tid < nt;
+    invQ[tid] = ok ? g[0] : 0.f;
+    invK[tid] = ok ? g[1] : 0.f;
+    beta[tid] = ok ? expf(-g[2]) : 1.f;
+  }
+
+  // ---- 1. queries, keys, values: four channels and all of the tile's tokens a thread
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int x = tid * 4; x < 2 * DP + vcols; x += kThreads * 4) {
+    const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
+    const int d = x - part * DP, limit = part == 2 ? p.vdim : p.dim;
+    float* dst = part == 2 ? rec_v + d : (part == 0 ? sC : sB) + d;
+    const int dst_ld = part == 2 ? vld : DP;
+    if (p.vec && (!DELTA || p.taps <= kTaps)) {
+      const bool ok = d < limit;
+      const T* src = in.proj + (long long)t0 * p.ld + in.col(part) + (ok ? d : 0);
+      if constexpr (DELTA) {
+        float4 w[kTaps], v[kTaps + 3];
+        const float* cw = p.conv + in.ch(part) + (ok ? d : 0);
+#pragma unroll
+        for (int j = 0; j < kTaps; ++j) {   // the last tap is the current token's
+          const int k = j - (kTaps - p.taps);
+          w[j] = k >= 0 ? load4(cw + (long long)k * p.channels) : zero;
+        }
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j)
+          v[j] = ok && j >= kTaps - p.taps ? in.four(part, d, t0 + j - (kTaps - 1)) : zero;
+#pragma unroll
+        for (int tb = 0; tb < kTT; tb += 4) {
+#pragma unroll
+          for (int t = 0; t < 4; ++t)
+            v[kTaps - 1 + t] = tb + t < nt ? load4(src + (tb + t) * p.ld) : zero;
+#pragma unroll
+          for (int t = 0; t < 4; ++t) {
+            float4 y = zero;
+#pragma unroll
+            for (int j = 0; j < kTaps; ++j) axpy4(y, w[j], v[t + j]);
+            store4(dst + (tb + t) * dst_ld, ok && tb + t < nt ? silu4(y) : zero);
+          }
+#pragma unroll
+          for (int j = 0; j < kTaps - 1; ++j) v[j] = v[4 + j];
+        }
+      } else {
+        const int one = part == 2 ? p.vdim - d : -1;   // the normaliser's column
+#pragma unroll
+        for (int t = 0; t < kTT; ++t) {
+          float4 y = ok && t < nt ? load4(src + t * p.ld) : zero;
+          if (one == 0) y.x = 1.f;
+          if (one == 1) y.y = 1.f;
+          if (one == 2) y.z = 1.f;
+          if (one == 3) y.w = 1.f;
+          store4(dst + t * dst_ld, y);
+        }
+      }
+      continue;
+    }
+    for (int t = 0; t < kTT; ++t) {
+      float y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        y[e] = 0.f;
+        if (t < nt && d + e < limit) {
+          if (DELTA) {
+            const float* w = p.conv + in.ch(part) + d + e;
+            for (int j = 0; j < p.taps; ++j)
+              y[e] = fmaf(w[(long long)j * p.channels], in.one(part, d + e, t0 + t - in.back + j), y[e]);
+            y[e] = silu_f(y[e]);
+          } else {
+            y[e] = in.one(part, d + e, t0 + t);
+          }
+        }
+        if (!DELTA && part == 2 && d + e == p.vdim) y[e] = 1.f;
+      }
+      store4(dst + t * dst_ld, make_float4(y[0], y[1], y[2], y[3]));
+    }
+  }
+  // cumulative log decays
+  float2 cum = make_float2(0.f, 0.f);
+  if (DELTA) {
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      if (half * 8 + t < nt) {
+        cum.x += fmaxf(-ae * softplus_f(z[t].x + bias.x), kMinLogDecay);
+        cum.y += fmaxf(-ae * softplus_f(z[t].y + bias.y), kMinLogDecay);
+      }
+      z[t] = cum;
+    }
+    const float bx = __shfl_xor_sync(0xffffffffu, cum.x, 16), by = __shfl_xor_sync(0xffffffffu, cum.y, 16);
+    if (half) {
+#pragma unroll
+      for (int t = 0; t < 8; ++t) z[t] = make_float2(z[t].x + bx, z[t].y + by);
+      cum = z[7];
+    }
+  }
+  __syncthreads();
+  // ---- 2. unit length
+  if (DELTA) {
+    for (int t = warp; t < kTT; t += kWarps) {
+      float a = 0.f, b = 0.f;
+      for (int d = lane * 4; d < DP; d += 128) {
+        const float4 q = load4(sC + t * DP + d), k = load4(sB + t * DP + d);
+        a = dot4(q, q, a);
+        b = dot4(k, k, b);
+      }
+      a = warp_sum(a);
+      b = warp_sum(b);
+      if (lane == 0) {
+        invQ[t] = p.q_scale / sqrtf(a + 1e-6f);
+        invK[t] = 1.f / sqrtf(b + 1e-6f);
+      }
+    }
+  } else {
+    float c = 0.f;
+    for (int t = 0; t < half * 8; ++t) c += invQ[t];
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      c += invQ[half * 8 + t];
+      z[t] = make_float2(c, c);
+    }
+    cum = make_float2(c, c);
+  }
+  const bool strong = __syncthreads_or(fminf(cum.x, cum.y) < kTileLogDecay);
+  // ---- 3. a, b, c and the groups' decays
+  if (tid < DP) {
+    float2 base = make_float2(0.f, 0.f);
+    if (strong) {   // logs from the group's start: the second half's begins where the first ends
+      base.x = __shfl_xor_sync(0xffffffffu, z[7].x, 16);
+      base.y = __shfl_xor_sync(0xffffffffu, z[7].y, 16);
+      if (!half) base = make_float2(0.f, 0.f);
+    }
+    float* G = reinterpret_cast<float*>(mats + R::kG);
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      const int tok = half * 8 + t;
+      const float lx = z[t].x - base.x, ly = z[t].y - base.y;
+      const float gx = __expf(lx), gy = __expf(ly);
+      const float2 k = *reinterpret_cast<const float2*>(sB + tok * DP + d0);
+      const float2 q = *reinterpret_cast<const float2*>(sC + tok * DP + d0);
+      const float fk = DELTA ? invK[tok] : 1.f, fq = DELTA ? invQ[tok] : p.q_scale;
+      const float put = DELTA ? 0.f : invK[tok];
+      const float kx = k.x * fk, ky = k.y * fk;
+      auto split_to = [&](int at, float x, float y) {
+        uint32_t hi, lo;
+        split2(x, y, hi, lo);
+        *reinterpret_cast<uint32_t*>(mats + at + (tok * kLd + d0) * 2) = hi;
+        *reinterpret_cast<uint32_t*>(mats + at + R::kMat + (tok * kLd + d0) * 2) = lo;
+      };
+      split_to(R::kB, kx * __expf(put - lx), ky * __expf(put - ly));
+      split_to(R::kC, q.x * fq * gx, q.y * fq * gy);
+      if (DELTA) split_to(R::kA, kx * gx, ky * gy);
+      if (tok % kB == kB - 1) {
+        *reinterpret_cast<float2*>(G + tok / kB * DP + d0) = make_float2(gx, gy);
+        if (strong) base = z[t];
+      }
+    }
+  }
+  if (tid < kTT) reinterpret_cast<float*>(mats + R::kBeta)[tid] = beta[tid];
+  if (tid == 0) *reinterpret_cast<float4*>(mats + R::kStrong) = make_float4(strong ? 1.f : 0.f, 0.f, 0.f, 0.f);
+  __syncthreads();
+  // ---- 4. products of the tokens: warp 0 c . b, warp 1 a . b
+  const uint32_t mb = smem_u32(mats);
+  if (warp < (DELTA ? 2 : 1)) {
+    const int m = lane >> 3, rr = lane & 7;
+    const uint32_t la = mb + (warp == 0 ? R::kC : R::kA) + (((m & 1) * 8 + rr) * kLd + (m >> 1) * 8) * 2;
+    const uint32_t lb = mb + R::kB + (((m >> 1) * 8 + rr) * kLd + (m & 1) * 8) * 2;
+    float acc[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < DP / 16; ++k) {
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      load_matrices(ah, la + k * 32);
+      load_matrices(al, la + R::kMat + k * 32);
+      load_matrices(bh, lb + k * 32);
+      load_matrices(bl, lb + R::kMat + k * 32);
+      mma_split(acc, ah, al, bh, bl);
+    }
+    const int g = lane >> 2, t2 = (lane & 3) * 2;
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const int i = g + (e >> 1) * 8, j = nb * 8 + t2;
+        const bool same = !strong || i / kB == j / kB;   // (j and j + 1 are of one group)
+        if (warp == 0) {
+          uint32_t hi, lo;
+          split2(same && j <= i ? acc[nb][e] : 0.f, same && j + 1 <= i ? acc[nb][e + 1] : 0.f, hi, lo);
+          *reinterpret_cast<uint32_t*>(mats + R::kQ + (i * R::kLdT + j) * 2) = hi;
+          *reinterpret_cast<uint32_t*>(mats + R::kQ + R::kSmall + (i * R::kLdT + j) * 2) = lo;
+        } else {
+          tri[i * (kTT + 1) + j] = same && j < i ? beta[i] * acc[nb][e] : 0.f;
+          tri[i * (kTT + 1) + j + 1] = same && j + 1 < i ? beta[i] * acc[nb][e + 1] : 0.f;
+        }
+      }
+    if (DELTA && warp == 1) {   // (I + diag(beta) a b^T)^-1, a column a lane
+      __syncwarp();
+      const int c = lane & 15;
+      float x[kTT];
+#pragma unroll
+      for (int i = 0; i < kTT; ++i) {
+        float v = i == c ? 1.f : 0.f;
+#pragma unroll
+        for (int j = 0; j < kTT; ++j)
+          if (j < i) v = fmaf(-tri[i * (kTT + 1) + j], x[j], v);
+        x[i] = v;
+      }
+#pragma unroll
+      for (int i = 0; i < kTT; ++i) {
+        const __nv_bfloat16 hi = __float2bfloat16(x[i]);
+        const __nv_bfloat16 lo = __float2bfloat16(x[i] - __bfloat162float(hi));
+        // lanes 0 - 15 the first part, 16 - 31 the second
+        reinterpret_cast<__nv_bfloat16*>(mats + R::kT + (lane >> 4) * R::kSmall)[i * R::kLdT + c] =
+            lane < 16 ? hi : lo;
+      }
+    }
+  }
+  if (DELTA && t0 + nt == s.n) save_inputs<T>(p, s, in, h % p.group == 0, 0, p.vdim);
+  __syncthreads();
+  for (int x = tid; x < R::kV / 16; x += kThreads)
+    reinterpret_cast<uint4*>(rec)[x] = reinterpret_cast<const uint4*>(mats)[x];
+}
+
+// A warp owns 16 columns: Z transposed, as accumulators of 16 columns by 8 rows.
+template <int DP, bool DELTA, int STAGES>
+__global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(const ScanArgs p) {
+  typedef __nv_bfloat16 T;
+  using R = MmaRecord<DP, DELTA>;
+  constexpr int kN = DP / 8, kLd = R::kLd;
+  extern __shared__ __align__(16) uint8_t smem[];
+  pdl_wait();
+  pdl_trigger();
+  const int slice = blockIdx.x % p.slices, h = blockIdx.x / p.slices % p.heads;
+  const int seq = blockIdx.x / p.slices / p.heads;
+  const Seq s(p.steps + (long long)seq * kStepInts);
+  if (s.n <= 0) return;
+  if (s.slot <= 0 || s.slot >= p.num_slots) {
+    put_zeros<T, DELTA>(p, s, h, slice);
+    return;
+  }
+  const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, t2 = (lane & 3) * 2;
+  const int nc = p.nc, c_first = slice * nc, vld = R::vld(nc), rec_vld = R::vld(p.slices * nc);
+  const int stage_size = R::bytes(nc);
+  const int tiles = (s.n + kTT - 1) / kTT;
+  const uint8_t* rec0 = reinterpret_cast<const uint8_t*>(p.records) +
+                        ((long long)p.first_tile[seq] * p.heads + h) * p.record * 4;
+  auto copy16 = [](uint8_t* dst, const uint8_t* src) {
+    copy16_async(reinterpret_cast<float*>(dst), reinterpret_cast<const float*>(src));
+  };
+  auto fetch = [&](int i) {   // (one group of copies per tile, also when there is none)
+    if (i < tiles) {
+      const uint8_t* src = rec0 + (long long)i * p.heads * p.record * 4;
+      uint8_t* dst = smem + i % STAGES * stage_size;
+      for (int x = tid * 16; x < R::kV; x += threads * 16) copy16(dst + x, src + x);
+      const int per = nc / 4;
+      for (int x = tid; x < kTT * per; x += threads) {
+        const int t = x / per, c = (x - t * per) * 4;
+        copy16(dst + R::kV + (t * vld + c) * 4, src + R::kV + (t * rec_vld + c_first + c) * 4);
+      }
+    }
+    copies_commit();
+  };
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) fetch(i);
+  // state: Z[n]: columns c and c + 8, rows 8 n + t2 and the next
+  float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols;
+  const int c0 = c_first + warp * 16 + g;
+  float Z[kN][4];
+#pragma unroll
+  for (int n = 0; n < kN; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = 8 * n + t2 + (e & 1), c = c0 + (e >> 1) * 8;
+      Z[n][e] = s.start > 0 && r < p.dim && c < p.state_cols ? state[(long long)r * p.state_cols + c] : 0.f;
+    }
+  const int lanes = p.vdim / 8;
+  const T* gate = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
+  T* out = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
+  const float* w = p.norm + (long long)h * p.norm_step;
+  // ldmatrix addresses within a stage: right operands with tokens as columns, and as rows
+  const int m = lane >> 3, rr = lane & 7;
+  const uint32_t tok_cols = (((m >> 1) * 8 + rr) * kLd + (m & 1) * 8) * 2;
+  const uint32_t tok_cols_t = (((m >> 1) * 8 + rr) * R::kLdT + (m & 1) * 8) * 2;
+  const uint32_t tok_rows = (((m & 1) * 8 + rr) * kLd + (m >> 1) * 8) * 2;
+
+  for (int it = 0; it < tiles; ++it) {
+    const int t0 = it * kTT, nt = min(kTT, s.n - t0);
+    copies_wait<STAGES - 2>();
+    __syncthreads();       // the tile's record is there; the stage of the tile before is free
+    fetch(it + STAGES - 1);
+    uint8_t* st = smem + it % STAGES * stage_size;
+    const uint32_t sb = smem_u32(st);
+    const float* beta = reinterpret_cast<const float*>(st + R::kBeta);
+    float* sV = reinterpret_cast<float*>(st + R::kV);
+    const bool strong = *reinterpret_cast<const float*>(st + R::kStrong) != 0.f;
+    float4 g0 = make_float4(0.f, 0.f, 0.f, 0.f), g1 = g0;
+    const int o_t = p.vec_out ? tid / lanes : 0, o_c = p.vec_out ? (tid - o_t * lanes) * 8 : 0;
+    if (p.vec_out && o_t < nt) {   // the first outputs' gates, ahead
+      g0 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
+      g1 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c + 4);
+    }
+    const int groups = strong ? kTT / kB : 1;
+    for (int grp = 0; grp < groups; ++grp) {
+      // read-outs: [16 columns x 16 tokens]
+      float P[2][4] = {}, O[2][4] = {};
+#pragma unroll
+      for (int k = 0; k < DP / 16; ++k) {
+        uint32_t zh[4], zl[4], bh[4], bl[4];
+        split_left(Z[2 * k], Z[2 * k + 1], zh, zl);
+        if constexpr (DELTA) {
+          load_matrices(bh, sb + R::kA + tok_cols + k * 32);
+          load_matrices(bl, sb + R::kA + R::kMat + tok_cols + k * 32);
+          mma_split(P, zh, zl, bh, bl);
+        }
+        load_matrices(bh, sb + R::kC + tok_cols + k * 32);
+        load_matrices(bl, sb + R::kC + R::kMat + tok_cols + k * 32);
+        mma_split(O, zh, zl, bh, bl);
+      }
+      // what is put: beta (v - P), solved; a strong tile's other groups wait
+      float U[2][4];
+      auto mine = [&](int tok) { return !strong || tok / kB == grp; };
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int tok = n * 8 + t2 + (e & 1);
+          const float v = sV[tok * vld + warp * 16 + g + (e >> 1) * 8];
+          U[n][e] = !mine(tok) ? 0.f : DELTA ? beta[tok] * (v - P[n][e]) : v;
+        }
+      uint32_t uh[4], ul[4], bh[4], bl[4];
+      split_left(U[0], U[1], uh, ul);
+      if constexpr (DELTA) {
+        load_matrices(bh, sb + R::kT + tok_cols_t);
+        load_matrices(bl, sb + R::kT + R::kSmall + tok_cols_t);
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) U[n][e] = 0.f;
+        mma_split(U, uh, ul, bh, bl);
+        split_left(U[0], U[1], uh, ul);
+      }
+      load_matrices(bh, sb + R::kQ + tok_cols_t);
+      load_matrices(bl, sb + R::kQ + R::kSmall + tok_cols_t);
+      mma_split(O, uh, ul, bh, bl);
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {   // (a lane alone reads and writes these values)
+          const int tok = n * 8 + t2 + (e & 1);
+          if (mine(tok)) sV[tok * vld + warp * 16 + g + (e >> 1) * 8] = O[n][e];
+        }
+      const float* G = reinterpret_cast<const float*>(st + R::kG) + (strong ? grp : kTT / kB - 1) * DP + t2;
+#pragma unroll
+      for (int n = 0; n < kN; n += 2) {
+        load_matrices_trans(bh, sb + R::kB + tok_rows + n * 16);
+        load_matrices_trans(bl, sb + R::kB + R::kMat + tok_rows + n * 16);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          mma_bf16(Z[n + e], uh, bl[2 * e], bl[2 * e + 1]);
+          mma_bf16(Z[n + e], ul, bh[2 * e], bh[2 * e + 1]);
+          mma_bf16(Z[n + e], uh, bh[2 * e], bh[2 * e + 1]);
+          const float2 f = *reinterpret_cast<const float2*>(G + 8 * (n + e));
+          Z[n + e][0] *= f.x; Z[n + e][1] *= f.y;
+          Z[n + e][2] *= f.x; Z[n + e][3] *= f.y;
+        }
+      }
+    }
+    __syncthreads();   // the tile's outputs are there
+    if (p.raw != nullptr) {
+      for (int t = warp; t < nt; t += threads / 32) {
+        float* dst = p.raw + ((s.first + t0 + t) * p.heads + h) * p.raw_cols + c_first;
+        for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = sV[t * vld + c];
+        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = beta[t];
+      }
+    } else if (p.vec_out) {
+      vector_outputs<T, DELTA>(p, sV, vld, beta, nt, lanes, gate + (long long)t0 * p.ld_gate,
+                               out + (long long)t0 * p.ldo, w, g0, g1);
+    } else {
+      for (int t = warp; t < nt; t += threads / 32)
+        head_output<T, DELTA>(p, sV + t * vld, s.first + t0 + t, h, beta[t]);
+    }
+  }
+  copies_wait<0>();
+#pragma unroll
+  for (int n = 0; n < kN; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = 8 * n + t2 + (e & 1), c = c0 + (e >> 1) * 8;
+      if (r < p.dim && c < p.state_cols) state[(long long)r * p.state_cols + c] = Z[n][e];
+    }
 }
 
 // Heads whose columns several blocks share: norm, weight and gate of the raw outputs. A warp per
@@ -995,7 +1512,8 @@ static bool set_smem(K k, size_t bytes) {
 
 template <typename T, int DP, bool DELTA>
 static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, cudaStream_t stream) {
-  constexpr int wc = ScanShape<DP>::kWarpCols;
+  // (one-token steps and 32-bit models; on tensor cores a warp has 16 columns)
+  const int wc = a.warp_cols;
   if (a.nc % wc || a.nc / wc > max_warps(DELTA) || (long long)a.nc * (a.slices - 1) >= a.ncols ||
       (long long)a.nc * a.slices < a.ncols)
     return -2;
@@ -1010,24 +1528,40 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
                : -5;
   }
   if (n_tiles < 1 || a.records == nullptr || a.tiles == nullptr || a.first_tile == nullptr ||
-      a.record < stage_floats<DP, DELTA>(a.nc * a.slices))
+      a.record < (sizeof(T) == 2 ? MmaRecord<DP, DELTA>::bytes(a.nc * a.slices) / 4
+                                 : stage_floats<DP, DELTA>(a.nc * a.slices)))
     return -2;
   if (!DELTA && launch_pdl(memory_gates_kernel<T>, dim3((unsigned)(n_seq * a.heads)),
                            dim3(max_rows <= 128 ? 128 : max_rows <= 512 ? 512 : 1024), 0, stream,
                            a) != cudaSuccess)
     return -5;
-  const size_t tile_smem = (size_t)(DELTA ? 3 : 2) * kTT * DP * sizeof(float);
-  if (!set_smem(tile_kernel<T, DP, DELTA>, tile_smem)) return -3;
-  if (launch_pdl(tile_kernel<T, DP, DELTA>, dim3((unsigned)(n_tiles * a.heads)),
-                 dim3(DP <= 128 ? 128 : 256), tile_smem, stream, a) != cudaSuccess)
-    return -5;
-  const size_t stage = (size_t)stage_floats<DP, DELTA>(a.nc) * sizeof(float);
-  const bool three = 3 * stage <= 220 * 1024;
-  auto k = three ? scan_kernel<T, DP, DELTA, 3> : scan_kernel<T, DP, DELTA, 2>;
-  const size_t smem = (three ? 3 : 2) * stage;
-  if (smem > 220 * 1024) return -6;
-  if (!set_smem(k, smem)) return -3;
-  return launch_pdl(k, dim3((unsigned)blocks), threads, smem, stream, a) == cudaSuccess ? 0 : -5;
+  const dim3 tile_grid((unsigned)(n_tiles * a.heads)), tile_threads(DP <= 128 ? 128 : 256);
+  if constexpr (sizeof(T) == 2) {
+    using R = MmaRecord<DP, DELTA>;
+    const size_t tile_smem = (size_t)2 * kTT * DP * 4 + R::kV + kTT * (kTT + 1) * 4;
+    if (!set_smem(tile_mma_kernel<DP, DELTA>, tile_smem)) return -3;
+    if (launch_pdl(tile_mma_kernel<DP, DELTA>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
+      return -5;
+    const size_t stage = R::bytes(a.nc);
+    const bool three = 3 * stage <= 220 * 1024;
+    auto k = three ? scan_mma_kernel<DP, DELTA, 3> : scan_mma_kernel<DP, DELTA, 2>;
+    const size_t smem = (three ? 3 : 2) * stage;
+    if (smem > 220 * 1024) return -6;
+    if (!set_smem(k, smem)) return -3;
+    return launch_pdl(k, dim3((unsigned)blocks), dim3(a.nc / 16 * 32), smem, stream, a) == cudaSuccess ? 0 : -5;
+  } else {
+    const size_t tile_smem = (size_t)(DELTA ? 3 : 2) * kTT * DP * sizeof(float);
+    if (!set_smem(tile_kernel<T, DP, DELTA>, tile_smem)) return -3;
+    if (launch_pdl(tile_kernel<T, DP, DELTA>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
+      return -5;
+    const size_t stage = (size_t)stage_floats<DP, DELTA>(a.nc) * sizeof(float);
+    const bool three = 3 * stage <= 220 * 1024;
+    auto k = three ? scan_kernel<T, DP, DELTA, 3> : scan_kernel<T, DP, DELTA, 2>;
+    const size_t smem = (three ? 3 : 2) * stage;
+    if (smem > 220 * 1024) return -6;
+    if (!set_smem(k, smem)) return -3;
+    return launch_pdl(k, dim3((unsigned)blocks), threads, smem, stream, a) == cudaSuccess ? 0 : -5;
+  }
 }
 
 template <typename T, bool DELTA>
@@ -1050,14 +1584,19 @@ static int aligned4(const void* p, long long ld, int dtype) {
   return ld % 4 == 0 && (reinterpret_cast<uintptr_t>(p) & (dtype == 0 ? 7 : 15)) == 0;
 }
 
-static int warp_cols(int dim) { return dim <= 128 ? 16 : 8; }
+// Columns of a warp: on tensor cores (16-bit models, portions of several tokens) always 16
+static int warp_cols(int dim, int dtype, bool several) {
+  return dim <= 128 || (several && dtype == 0) ? 16 : 8;
+}
 
 // The common part of both entry points
-static void finish_args(ScanArgs& a, int slices, int ncols, int raw_cols, void* raw, int dtype) {
+static void finish_args(ScanArgs& a, int slices, int ncols, int raw_cols, void* raw, int dtype,
+                        bool several) {
   a.slices = slices;
   a.ncols = ncols;
+  a.warp_cols = warp_cols(a.dim, dtype, several);
   a.nc = (ncols + slices - 1) / slices;
-  a.nc = (a.nc + warp_cols(a.dim) - 1) / warp_cols(a.dim) * warp_cols(a.dim);
+  a.nc = (a.nc + a.warp_cols - 1) / a.warp_cols * a.warp_cols;
   a.raw = slices > 1 ? reinterpret_cast<float*>(raw) : nullptr;
   a.raw_cols = raw_cols;
   a.q_scale = 1.f / sqrtf((float)a.dim);
@@ -1066,7 +1605,8 @@ static void finish_args(ScanArgs& a, int slices, int ncols, int raw_cols, void* 
               aligned4(a.gate, a.ld_gate, dtype) && aligned4(a.out, a.ldo, dtype) &&
               aligned4(a.norm, a.norm_step, 1);
   a.vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.q_at % 4 == 0 && a.k_at % 4 == 0 && a.v_at % 4 == 0 &&
-          aligned4(a.proj, a.ld, dtype) && aligned4(a.conv_state, 0, dtype) && aligned4(a.conv, 0, 1);
+          aligned4(a.proj, a.ld, dtype) && aligned4(a.conv_state, 0, dtype) && aligned4(a.conv, 0, 1) &&
+          aligned4(a.decay, a.ld_decay, dtype);
 }
 
 }  // namespace ab200
@@ -1077,16 +1617,27 @@ typedef __nv_bfloat16 bf16;
 extern "C" {
 
 // Blocks per head so that each block's columns fit: 0 if dim is beyond the kernel's.
-int ab200_scan_min_slices(int dim, int ncols, int delta) {
+int ab200_scan_min_slices(int dim, int ncols, int delta, int dtype, int several) {
   if (dim < 1 || dim > 256) return 0;
-  const int most = max_warps(delta != 0) * warp_cols(dim);
+  const int most = max_warps(delta != 0) * warp_cols(dim, dtype, several != 0);
   return (ncols + most - 1) / most;
 }
 
 // Floats of a tile's record of a head (portions of more than one token).
-long long ab200_scan_record(int dim, int ncols, int slices, int delta) {
-  const int wc = warp_cols(dim), nc = ((ncols + slices - 1) / slices + wc - 1) / wc * wc;
+long long ab200_scan_record(int dim, int ncols, int slices, int delta, int dtype) {
+  const int wc = warp_cols(dim, dtype, true), nc = ((ncols + slices - 1) / slices + wc - 1) / wc * wc;
   const int dp = dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256;
+  if (dtype == 0) {
+    const int cols = nc * slices;
+    return (delta ? (dp == 32    ? MmaRecord<32, true>::bytes(cols)
+                     : dp == 64  ? MmaRecord<64, true>::bytes(cols)
+                     : dp == 128 ? MmaRecord<128, true>::bytes(cols)
+                                 : MmaRecord<256, true>::bytes(cols))
+                  : (dp == 32    ? MmaRecord<32, false>::bytes(cols)
+                     : dp == 64  ? MmaRecord<64, false>::bytes(cols)
+                     : dp == 128 ? MmaRecord<128, false>::bytes(cols)
+                                 : MmaRecord<256, false>::bytes(cols))) / 4;
+  }
   const int vectors = delta ? 3 * kTT + kTT / kB : 2 * kTT + kTT / kB;
   return (long long)vectors * dp + 2 * kTT * kB + kTT + 4 + (long long)kTT * nc * slices;
 }
@@ -1125,14 +1676,14 @@ int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_a
   a.tiles = reinterpret_cast<const int*>(tiles);
   a.first_tile = reinterpret_cast<const int*>(first_tile);
   a.records = reinterpret_cast<float*>(records);
-  a.record = ab200_scan_record(dim, vdim, slices, 1);
+  a.record = ab200_scan_record(dim, vdim, slices, 1, dtype);
   a.heads = heads; a.group = heads / kv_heads; a.dim = dim; a.vdim = vdim;
   a.taps = taps;
   a.channels = 2 * kv_heads * dim + heads * vdim;
   a.eps = eps;
   a.out = out; a.ldo = ldo;
   a.status = status;
-  finish_args(a, slices, vdim, vdim, raw, dtype);
+  finish_args(a, slices, vdim, vdim, raw, dtype, max_rows > 1);
   return dtype == 0 ? run_scan<bf16, true>(a, n_seq, n_tiles, max_rows, T, stream)
                     : run_scan<float, true>(a, n_seq, n_tiles, max_rows, T, stream);
 }
@@ -1168,14 +1719,14 @@ int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_
   a.tiles = reinterpret_cast<const int*>(tiles);
   a.first_tile = reinterpret_cast<const int*>(first_tile);
   a.records = reinterpret_cast<float*>(records);
-  a.record = ab200_scan_record(dim, vdim + 1, slices, 0);
+  a.record = ab200_scan_record(dim, vdim + 1, slices, 0, dtype);
   a.gates = reinterpret_cast<float*>(gates);
   a.heads = heads; a.group = 1; a.dim = dim; a.vdim = vdim;
   a.taps = 1;
   a.eps = eps;
   a.out = out; a.ldo = ldo;
   a.status = status;
-  finish_args(a, slices, vdim + 1, vdim + 2, raw, dtype);
+  finish_args(a, slices, vdim + 1, vdim + 2, raw, dtype, max_rows > 1);
   return dtype == 0 ? run_scan<bf16, false>(a, n_seq, n_tiles, max_rows, T, stream)
                     : run_scan<float, false>(a, n_seq, n_tiles, max_rows, T, stream);
 }

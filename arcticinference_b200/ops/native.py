@@ -127,8 +127,8 @@ def _declare(L: ctypes.CDLL) -> None:
         "ab200_stream_norm": (I, [P, P, P, LL, P, P, I, P, F, F, F, P, P, LL, I, I, P]),
         "ab200_stream_sandwich": (I, [P, P, LL, P, P, P, P, F, F, LL, I, I, P]),
         "ab200_stream_add": (I, [P, P, P, P, LL, P, P, LL, P, P, P, I, P, LL, F, LL, I, I, P]),
-        "ab200_scan_min_slices": (I, [I, I, I]),
-        "ab200_scan_record": (LL, [I, I, I, I]),
+        "ab200_scan_min_slices": (I, [I, I, I, I, I]),
+        "ab200_scan_record": (LL, [I, I, I, I, I]),
         "ab200_delta_scan": (I, [P, LL, I, I, I, I, P, LL, P, LL, P, I, P, P, P, P, I, P, I, P, I, I, P, P,
                                  I, P, LL, I, I, I, I, I, F, P, P, LL, I, P, P]),
         "ab200_memory_scan": (I, [P, LL, I, I, I, I, I, P, LL, P, P, F, P, P, I, P, I, P, I, I, P, P, I, P,

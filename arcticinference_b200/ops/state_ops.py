@@ -98,13 +98,13 @@ class StateDecodePlan:
         self._host[:, 2] = 0
 
 
-def slices_for(dim: int, ncols: int, delta: bool, blocks: int, long: bool) -> int:
+def slices_for(dim: int, ncols: int, delta: bool, dtype: torch.dtype, blocks: int, long: bool) -> int:
     """Blocks that share a head's columns: as few as hold them, more where a prompt's few heads
     would leave most of the GPU idle."""
-    least = _nat().lib().ab200_scan_min_slices(dim, ncols, int(delta))
+    least = _nat().lib().ab200_scan_min_slices(dim, ncols, int(delta), dtype_code(dtype), int(long))
     if least == 0:
         raise NotImplementedError("recurrent layers with keys of more than 256 dimensions")
-    width = 16 if dim <= 128 else 8
+    width = 16 if dim <= 128 or (long and dtype == torch.bfloat16) else 8     # of a warp
     most = -(-ncols // width)
     want = 148 // max(1, blocks) if long else 1
     n = max(least, min(most, want))
@@ -113,14 +113,15 @@ def slices_for(dim: int, ncols: int, delta: bool, blocks: int, long: bool) -> in
     return -(-ncols // cols)
 
 
-def _scratch(s, ncols: int, delta: bool, steps: StateStep, T: int, device):
+def _scratch(s, ncols: int, delta: bool, steps: StateStep, proj: torch.Tensor):
     """(slices, raw outputs or None, tile records or None) of a scan."""
-    slices = slices_for(s.dim, ncols, delta, steps.table.shape[0] * s.heads, steps.max_rows > 1)
-    f32 = dict(dtype=torch.float32, device=device)
-    raw = torch.empty(T, s.heads, ncols + (not delta), **f32) if slices > 1 else None
+    slices = slices_for(s.dim, ncols, delta, proj.dtype, steps.table.shape[0] * s.heads,
+                        steps.max_rows > 1)
+    f32 = dict(dtype=torch.float32, device=proj.device)
+    raw = torch.empty(proj.shape[0], s.heads, ncols + (not delta), **f32) if slices > 1 else None
     records = None
     if steps.max_rows > 1:
-        size = _nat().lib().ab200_scan_record(s.dim, ncols, slices, int(delta))
+        size = _nat().lib().ab200_scan_record(s.dim, ncols, slices, int(delta), dtype_code(proj.dtype))
         records = torch.empty(steps.tiles.shape[0], s.heads, size, **f32)
     return slices, raw, records
 
@@ -204,7 +205,7 @@ def delta_scan(proj, decay, gate, conv, a_exp, dt_bias, norm, s: DeltaShape, sta
     nat = _nat()
     T, n = proj.shape[0], steps.table.shape[0]
     out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
-    slices, raw, records = _scratch(s, s.vdim, True, steps, T, proj.device)
+    slices, raw, records = _scratch(s, s.vdim, True, steps, proj)
     assert proj.stride(1) == decay.stride(1) == gate.stride(1) == 1
     assert state.is_contiguous() and conv_state.is_contiguous() and steps.table.is_contiguous()
     rc = nat.lib().ab200_delta_scan(
@@ -283,7 +284,7 @@ def memory_scan(proj, gate, i_bias, f_bias, norm, s: MemoryShape, state, max_sta
     nat = _nat()
     T, n = proj.shape[0], steps.table.shape[0]
     out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
-    slices, raw, records = _scratch(s, s.vdim + 1, False, steps, T, proj.device)
+    slices, raw, records = _scratch(s, s.vdim + 1, False, steps, proj)
     gates = torch.empty(T, s.heads, 3, dtype=torch.float32, device=proj.device) \
         if records is not None else None
     assert proj.stride(1) == gate.stride(1) == 1
