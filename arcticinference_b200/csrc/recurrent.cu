@@ -113,13 +113,29 @@ __device__ __forceinline__ void copies_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float exp2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float log2_fast(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // log(1 + e^z); log1p's first terms where the fast logarithm would lose them
 __device__ __forceinline__ float softplus_f(float z) {
-  const float e = __expf(-fabsf(z));
-  const float l = e < 0.03f ? e * (1.f + e * (-0.5f + e * (0.33333333f - 0.25f * e))) : __logf(1.f + e);
-  return fmaxf(z, 0.f) + l;
+  const float e = exp2_fast(-kLog2e * fabsf(z));
+  const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333333f), -0.5f), 1.f);
+  return fmaxf(z, 0.f) + (e < 0.03f ? series : log2_fast(1.f + e) * (1.f / kLog2e));
 }
-__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return rcp_fast(1.f + exp2_fast(-kLog2e * z)); }
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
 __device__ __forceinline__ float4 silu4(const float4& y) {
   return make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w));
@@ -137,8 +153,7 @@ __device__ __forceinline__ float dot4(const float4& a, const float4& b, float ac
 // and g + 8, columns 2 t and 2 t + 1; A's a0 (g, 2 t ..), a1 (g + 8, 2 t ..), a2, a3 eight columns
 // further; B's b0 (rows 2 t .., column g), b1 eight rows further
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
       "{%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -174,6 +189,30 @@ __device__ __forceinline__ void mma_split(float (&d)[2][4], const uint32_t (&hi)
     mma_bf16(d[n], hi, bh[2 * n], bh[2 * n + 1]);
   }
 }
+// Elements as they lie in memory, widened when they are used (so that nothing waits for a load early)
+template <typename T>
+struct Raw8;
+template <>
+struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = load4(p); b = load4(p + 4); }
+  __device__ __forceinline__ float4 lo() const { return a; }
+  __device__ __forceinline__ float4 hi() const { return b; }
+};
+__device__ __forceinline__ float4 widen(uint32_t x, uint32_t y) {
+  return make_float4(__uint_as_float(x << 16), __uint_as_float(x & 0xffff0000u), __uint_as_float(y << 16),
+                     __uint_as_float(y & 0xffff0000u));
+}
+template <>
+struct Raw8<__nv_bfloat16> {   // (8-byte aligned)
+  uint2 a, b;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) {
+    a = *reinterpret_cast<const uint2*>(p);
+    b = *reinterpret_cast<const uint2*>(p + 4);
+  }
+  __device__ __forceinline__ float4 lo() const { return widen(a.x, a.y); }
+  __device__ __forceinline__ float4 hi() const { return widen(b.x, b.y); }
+};
 // log gates of the matrix memory
 __device__ __forceinline__ float2 memory_log_gates(float zi, float zf, float cap) {
   const float z = cap * tanhf(zf / cap);
@@ -393,20 +432,21 @@ __device__ __forceinline__ void head_output(const ScanArgs& p, const float* o, l
     dst[c] = from_f32<T>(o[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
 }
 
-// A block's tile: the same eight columns a thread, the `lanes` lanes of a token side by side. g0, g1: the
-// gate of the thread's first columns.
+// A block's tile: eight columns a thread, the `lanes` lanes of a token side by side. g, wa, wb: gate
+// and norm weights of the thread's first columns.
 template <typename T, bool DELTA>
 __device__ __forceinline__ void vector_outputs(const ScanArgs& p, const float* o_tile, int ld, const float* floors,
                                                int nt, int lanes, const T* gate, T* out, const float* w,
-                                               float4 g0, float4 g1) {
+                                               Raw8<T> g, float4 wa, float4 wb) {
   // (whole warps: the lanes of a token lie in one)
   for (int x = threadIdx.x; x < (kTT * lanes + 31) / 32 * 32; x += blockDim.x) {
     const int t = x / lanes, c = (x - t * lanes) * 8;
     const bool ok = t < nt;
     const float* o = o_tile + (ok ? t : 0) * ld;
     if (x != threadIdx.x && ok) {
-      g0 = load4(gate + t * p.ld_gate + c);
-      g1 = load4(gate + t * p.ld_gate + c + 4);
+      g.load(gate + t * p.ld_gate + c);
+      wa = load4(w + c);
+      wb = load4(w + c + 4);
     }
     const float4 a = load4(o + c), b = load4(o + c + 4);
     float f = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floors[ok ? t : 0]) + 1e-6f);
@@ -414,7 +454,7 @@ __device__ __forceinline__ void vector_outputs(const ScanArgs& p, const float* o
     for (int k = lanes / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
     f *= 1.f / sqrtf(ss / (float)p.vdim + p.eps);
     if (!ok) continue;
-    const float4 wa = load4(w + c), wb = load4(w + c + 4);
+    const float4 g0 = g.lo(), g1 = g.hi();
     T* dst = out + t * p.ldo + c;
     store4(dst, make_float4(a.x * f * wa.x * sigmoid_f(g0.x), a.y * f * wa.y * sigmoid_f(g0.y),
                             a.z * f * wa.z * sigmoid_f(g0.z), a.w * f * wa.w * sigmoid_f(g0.w)));
@@ -904,6 +944,12 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
   const T* gate = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
   T* out = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
   const float* w = p.norm + (long long)h * p.norm_step;
+  const int o_t = p.vec_out ? tid / lanes : 0, o_c = p.vec_out ? (tid - o_t * lanes) * 8 : 0;
+  float4 wa = make_float4(0.f, 0.f, 0.f, 0.f), wb = wa;
+  if (p.vec_out) {
+    wa = load4(w + o_c);
+    wb = load4(w + o_c + 4);
+  }
 
   for (int it = 0; it < tiles; ++it) {
     const int t0 = it * kTT, nt = min(kTT, s.n - t0);
@@ -918,12 +964,9 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
     const float* dotC = st + R::kDotC;
     float* sV = st + R::kV;
     const bool strong = st[R::kStrong] != 0.f;
-    float4 g0 = make_float4(0.f, 0.f, 0.f, 0.f), g1 = g0;
-    const int o_t = p.vec_out ? tid / lanes : 0, o_c = p.vec_out ? (tid - o_t * lanes) * 8 : 0;
-    if (p.vec_out && o_t < nt) {   // the first outputs' gates, ahead
-      g0 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
-      g1 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c + 4);
-    }
+    Raw8<T> gates = {};
+    if (p.vec_out && o_t < nt)   // the first outputs' gates, ahead
+      gates.load(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
     for (int q0 = 0; q0 < nt; q0 += kB) {
       float2 acc[kKinds][kCols][kB];
 #pragma unroll
@@ -1024,7 +1067,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
       }
     } else if (p.vec_out) {
       vector_outputs<T, DELTA>(p, sV, nc, st + R::kBeta, nt, lanes, gate + (long long)t0 * p.ld_gate,
-                               out + (long long)t0 * p.ldo, w, g0, g1);
+                               out + (long long)t0 * p.ldo, w, gates, wa, wb);
     } else {
       for (int t = warp; t < nt; t += threads / 32)
         head_output<T, DELTA>(p, sV + t * nc, s.first + t0 + t, h, st[R::kBeta + t]);
@@ -1049,7 +1092,7 @@ struct MmaRecord {
 };
 
 template <int DP, bool DELTA>
-__global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const ScanArgs p) {
+__global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile_mma_kernel(const ScanArgs p) {
   typedef __nv_bfloat16 T;
   using R = MmaRecord<DP, DELTA>;
   constexpr int kThreads = DP <= 128 ? 128 : 256, kWarps = kThreads / 32, kLd = R::kLd;
@@ -1057,7 +1100,8 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
   float* sB = sm;                                // keys
   float* sC = sm + kTT * DP;                     // queries
   uint8_t* mats = reinterpret_cast<uint8_t*>(sm + 2 * kTT * DP);   // the record up to its values
-  float* tri = reinterpret_cast<float*>(mats + R::kV);             // [kTT][kTT + 1]
+  constexpr int kTriLd = kTT + 4;
+  float* tri = reinterpret_cast<float*>(mats + R::kV);             // [kTT][kTriLd]
   __shared__ float invQ[kTT], invK[kTT], beta[kTT];   // memory: log decay, log input factor, exp(-m)
   pdl_wait();
   pdl_trigger();
@@ -1075,27 +1119,27 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
 
   // Decays: a thread has two channels and eight of the tokens; lane ^ 16 has the others.
   const int d0 = 2 * ((tid & 15) + (tid >> 5) * 16), half = (tid >> 4) & 1;
+  uint32_t zr[8] = {};
   float2 z[8];
   float2 bias = make_float2(0.f, 0.f);
   float ae = 0.f;
   if (DELTA) {
-#pragma unroll
-    for (int t = 0; t < 8; ++t) z[t] = make_float2(0.f, 0.f);
     if (d0 < p.dim) {
       const T* src = reinterpret_cast<const T*>(p.decay) + (s.first + t0 + half * 8) * p.ld_decay + h * p.dim + d0;
       const bool two = d0 + 1 < p.dim;
-      ae = p.a_exp[h];
+      ae = -kLog2e * p.a_exp[h];     // (logs are to base 2 from here on)
       bias.x = p.dt_bias[h * p.dim + d0];
       if (two) bias.y = p.dt_bias[h * p.dim + d0 + 1];
       const int mine = nt - half * 8;
       if (p.vec) {
 #pragma unroll
         for (int t = 0; t < 8; ++t)
-          if (t < mine) z[t] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + t * p.ld_decay));
+          if (t < mine) zr[t] = *reinterpret_cast<const uint32_t*>(src + t * p.ld_decay);
       } else {
+#pragma unroll
         for (int t = 0; t < 8; ++t)
           if (t < mine)
-            z[t] = make_float2(to_f32<T>(src[t * p.ld_decay]), two ? to_f32<T>(src[t * p.ld_decay + 1]) : 0.f);
+            zr[t] = pack_bf16x2(to_f32<T>(src[t * p.ld_decay]), two ? to_f32<T>(src[t * p.ld_decay + 1]) : 0.f);
       }
     }
     if (tid < kTT)
@@ -1103,8 +1147,8 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
   } else if (tid < kTT) {
     const float* g = p.gates + ((s.first + t0 + tid) * p.heads + h) * 3;
     const bool ok = tid < nt;
-    invQ[tid] = ok ? g[0] : 0.f;
-    invK[tid] = ok ? g[1] : 0.f;
+    invQ[tid] = ok ? g[0] * kLog2e : 0.f;
+    invK[tid] = ok ? g[1] * kLog2e : 0.f;
     beta[tid] = ok ? expf(-g[2]) : 1.f;
   }
 
@@ -1119,27 +1163,35 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
       const bool ok = d < limit;
       const T* src = in.proj + (long long)t0 * p.ld + in.col(part) + (ok ? d : 0);
       if constexpr (DELTA) {
+        // all loads at once: the tile's tokens, the ones before it, the taps (the last one is the
+        // current token's)
+        uint2 raw[kTT];
+#pragma unroll
+        for (int t = 0; t < kTT; ++t, src += p.ld) {
+          raw[t] = make_uint2(0u, 0u);
+          if (t < nt) raw[t] = *reinterpret_cast<const uint2*>(src);
+        }
         float4 w[kTaps], v[kTaps + 3];
         const float* cw = p.conv + in.ch(part) + (ok ? d : 0);
-#pragma unroll
-        for (int j = 0; j < kTaps; ++j) {   // the last tap is the current token's
-          const int k = j - (kTaps - p.taps);
-          w[j] = k >= 0 ? load4(cw + (long long)k * p.channels) : zero;
-        }
 #pragma unroll
         for (int j = 0; j < kTaps - 1; ++j)
           v[j] = ok && j >= kTaps - p.taps ? in.four(part, d, t0 + j - (kTaps - 1)) : zero;
 #pragma unroll
+        for (int j = 0; j < kTaps; ++j) {
+          const int k = j - (kTaps - p.taps);
+          w[j] = k >= 0 ? load4(cw + (long long)k * p.channels) : zero;
+        }
+#pragma unroll
         for (int tb = 0; tb < kTT; tb += 4) {
 #pragma unroll
-          for (int t = 0; t < 4; ++t)
-            v[kTaps - 1 + t] = tb + t < nt ? load4(src + (tb + t) * p.ld) : zero;
+          for (int t = 0; t < 4; ++t) v[kTaps - 1 + t] = widen(raw[tb + t].x, raw[tb + t].y);
 #pragma unroll
           for (int t = 0; t < 4; ++t) {
             float4 y = zero;
 #pragma unroll
             for (int j = 0; j < kTaps; ++j) axpy4(y, w[j], v[t + j]);
-            store4(dst + (tb + t) * dst_ld, ok && tb + t < nt ? silu4(y) : zero);
+            store4(dst, ok && tb + t < nt ? silu4(y) : zero);
+            dst += dst_ld;
           }
 #pragma unroll
           for (int j = 0; j < kTaps - 1; ++j) v[j] = v[4 + j];
@@ -1147,13 +1199,13 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
       } else {
         const int one = part == 2 ? p.vdim - d : -1;   // the normaliser's column
 #pragma unroll
-        for (int t = 0; t < kTT; ++t) {
-          float4 y = ok && t < nt ? load4(src + t * p.ld) : zero;
+        for (int t = 0; t < kTT; ++t, src += p.ld, dst += dst_ld) {
+          float4 y = ok && t < nt ? load4(src) : zero;
           if (one == 0) y.x = 1.f;
           if (one == 1) y.y = 1.f;
           if (one == 2) y.z = 1.f;
           if (one == 3) y.w = 1.f;
-          store4(dst + t * dst_ld, y);
+          store4(dst, y);
         }
       }
       continue;
@@ -1184,8 +1236,9 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
 #pragma unroll
     for (int t = 0; t < 8; ++t) {
       if (half * 8 + t < nt) {
-        cum.x += fmaxf(-ae * softplus_f(z[t].x + bias.x), kMinLogDecay);
-        cum.y += fmaxf(-ae * softplus_f(z[t].y + bias.y), kMinLogDecay);
+        const float zx = __uint_as_float(zr[t] << 16), zy = __uint_as_float(zr[t] & 0xffff0000u);
+        cum.x += fmaxf(ae * softplus_f(zx + bias.x), kMinLogDecay * kLog2e);
+        cum.y += fmaxf(ae * softplus_f(zy + bias.y), kMinLogDecay * kLog2e);
       }
       z[t] = cum;
     }
@@ -1223,7 +1276,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
     }
     cum = make_float2(c, c);
   }
-  const bool strong = __syncthreads_or(fminf(cum.x, cum.y) < kTileLogDecay);
+  const bool strong = __syncthreads_or(fminf(cum.x, cum.y) < kTileLogDecay * kLog2e);
   // ---- 3. a, b, c and the groups' decays
   if (tid < DP) {
     float2 base = make_float2(0.f, 0.f);
@@ -1237,7 +1290,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
     for (int t = 0; t < 8; ++t) {
       const int tok = half * 8 + t;
       const float lx = z[t].x - base.x, ly = z[t].y - base.y;
-      const float gx = __expf(lx), gy = __expf(ly);
+      const float gx = exp2_fast(lx), gy = exp2_fast(ly);
       const float2 k = *reinterpret_cast<const float2*>(sB + tok * DP + d0);
       const float2 q = *reinterpret_cast<const float2*>(sC + tok * DP + d0);
       const float fk = DELTA ? invK[tok] : 1.f, fq = DELTA ? invQ[tok] : p.q_scale;
@@ -1249,7 +1302,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
         *reinterpret_cast<uint32_t*>(mats + at + (tok * kLd + d0) * 2) = hi;
         *reinterpret_cast<uint32_t*>(mats + at + R::kMat + (tok * kLd + d0) * 2) = lo;
       };
-      split_to(R::kB, kx * __expf(put - lx), ky * __expf(put - ly));
+      split_to(R::kB, kx * exp2_fast(put - lx), ky * exp2_fast(put - ly));
       split_to(R::kC, q.x * fq * gx, q.y * fq * gy);
       if (DELTA) split_to(R::kA, kx * gx, ky * gy);
       if (tok % kB == kB - 1) {
@@ -1261,9 +1314,16 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
   if (tid < kTT) reinterpret_cast<float*>(mats + R::kBeta)[tid] = beta[tid];
   if (tid == 0) *reinterpret_cast<float4*>(mats + R::kStrong) = make_float4(strong ? 1.f : 0.f, 0.f, 0.f, 0.f);
   __syncthreads();
-  // ---- 4. products of the tokens: warp 0 c . b, warp 1 a . b
-  const uint32_t mb = smem_u32(mats);
-  if (warp < (DELTA ? 2 : 1)) {
+  // ---- 4. products of the tokens: the first warp c . b, the second a . b; the others write the rest out
+  constexpr int kGram = DELTA ? 2 : 1;
+  if (warp >= kGram) {
+    constexpr int kSkip = (R::kG - R::kQ) / 16, kAll = R::kV / 16 - kSkip;
+    for (int x = tid - kGram * 32; x < kAll; x += kThreads - kGram * 32) {
+      const int y = x < R::kQ / 16 ? x : x + kSkip;
+      reinterpret_cast<uint4*>(rec)[y] = reinterpret_cast<const uint4*>(mats)[y];
+    }
+  } else {
+    const uint32_t mb = smem_u32(mats);
     const int m = lane >> 3, rr = lane & 7;
     const uint32_t la = mb + (warp == 0 ? R::kC : R::kA) + (((m & 1) * 8 + rr) * kLd + (m >> 1) * 8) * 2;
     const uint32_t lb = mb + R::kB + (((m >> 1) * 8 + rr) * kLd + (m & 1) * 8) * 2;
@@ -1287,11 +1347,12 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
         if (warp == 0) {
           uint32_t hi, lo;
           split2(same && j <= i ? acc[nb][e] : 0.f, same && j + 1 <= i ? acc[nb][e + 1] : 0.f, hi, lo);
-          *reinterpret_cast<uint32_t*>(mats + R::kQ + (i * R::kLdT + j) * 2) = hi;
-          *reinterpret_cast<uint32_t*>(mats + R::kQ + R::kSmall + (i * R::kLdT + j) * 2) = lo;
+          *reinterpret_cast<uint32_t*>(rec + R::kQ + (i * R::kLdT + j) * 2) = hi;
+          *reinterpret_cast<uint32_t*>(rec + R::kQ + R::kSmall + (i * R::kLdT + j) * 2) = lo;
         } else {
-          tri[i * (kTT + 1) + j] = same && j < i ? beta[i] * acc[nb][e] : 0.f;
-          tri[i * (kTT + 1) + j + 1] = same && j + 1 < i ? beta[i] * acc[nb][e + 1] : 0.f;
+          *reinterpret_cast<float2*>(tri + i * kTriLd + j) =
+              make_float2(same && j < i ? beta[i] * acc[nb][e] : 0.f,
+                          same && j + 1 < i ? beta[i] * acc[nb][e + 1] : 0.f);
         }
       }
     if (DELTA && warp == 1) {   // (I + diag(beta) a b^T)^-1, a column a lane
@@ -1300,26 +1361,27 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_mma_kernel(const S
       float x[kTT];
 #pragma unroll
       for (int i = 0; i < kTT; ++i) {
-        float v = i == c ? 1.f : 0.f;
+        float v0 = i == c ? 1.f : 0.f, v1 = 0.f;
 #pragma unroll
-        for (int j = 0; j < kTT; ++j)
-          if (j < i) v = fmaf(-tri[i * (kTT + 1) + j], x[j], v);
-        x[i] = v;
+        for (int j = 0; j < i; j += 4) {
+          const float4 t = load4(tri + i * kTriLd + j);
+          v0 = fmaf(-t.x, x[j], v0);
+          if (j + 1 < i) v1 = fmaf(-t.y, x[j + 1], v1);
+          if (j + 2 < i) v0 = fmaf(-t.z, x[j + 2], v0);
+          if (j + 3 < i) v1 = fmaf(-t.w, x[j + 3], v1);
+        }
+        x[i] = v0 + v1;
       }
+      // lanes 0 - 15 write the first part of the split, 16 - 31 the second
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(rec + R::kT + (lane >> 4) * R::kSmall) + c;
 #pragma unroll
       for (int i = 0; i < kTT; ++i) {
         const __nv_bfloat16 hi = __float2bfloat16(x[i]);
-        const __nv_bfloat16 lo = __float2bfloat16(x[i] - __bfloat162float(hi));
-        // lanes 0 - 15 the first part, 16 - 31 the second
-        reinterpret_cast<__nv_bfloat16*>(mats + R::kT + (lane >> 4) * R::kSmall)[i * R::kLdT + c] =
-            lane < 16 ? hi : lo;
+        dst[i * R::kLdT] = lane < 16 ? hi : __float2bfloat16(x[i] - __bfloat162float(hi));
       }
     }
   }
   if (DELTA && t0 + nt == s.n) save_inputs<T>(p, s, in, h % p.group == 0, 0, p.vdim);
-  __syncthreads();
-  for (int x = tid; x < R::kV / 16; x += kThreads)
-    reinterpret_cast<uint4*>(rec)[x] = reinterpret_cast<const uint4*>(mats)[x];
 }
 
 // A warp owns 16 columns: Z transposed, as accumulators of 16 columns by 8 rows.
@@ -1362,8 +1424,9 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
     }
     copies_commit();
   };
+  // (a tile's outputs are written out while the next one's are computed: two stages are in use)
 #pragma unroll
-  for (int i = 0; i < STAGES - 1; ++i) fetch(i);
+  for (int i = 0; i < STAGES - 2; ++i) fetch(i);
   // state: Z[n]: columns c and c + 8, rows 8 n + t2 and the next
   float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols;
   const int c0 = c_first + warp * 16 + g;
@@ -1379,57 +1442,85 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
   const T* gate = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
   T* out = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
   const float* w = p.norm + (long long)h * p.norm_step;
+  const int o_t = p.vec_out ? tid / lanes : 0, o_c = p.vec_out ? (tid - o_t * lanes) * 8 : 0;
+  float4 wa = make_float4(0.f, 0.f, 0.f, 0.f), wb = wa;
+  if (p.vec_out) {
+    wa = load4(w + o_c);
+    wb = load4(w + o_c + 4);
+  }
   // ldmatrix addresses within a stage: right operands with tokens as columns, and as rows
   const int m = lane >> 3, rr = lane & 7;
   const uint32_t tok_cols = (((m >> 1) * 8 + rr) * kLd + (m & 1) * 8) * 2;
   const uint32_t tok_cols_t = (((m >> 1) * 8 + rr) * R::kLdT + (m & 1) * 8) * 2;
   const uint32_t tok_rows = (((m & 1) * 8 + rr) * kLd + (m >> 1) * 8) * 2;
 
+  // norm, weight and gate of a tile's outputs
+  Raw8<T> gates = {};
+  auto put_out = [&](int it) {
+    const int t0 = it * kTT, nt = min(kTT, s.n - t0);
+    uint8_t* st = smem + it % STAGES * stage_size;
+    const float* beta = reinterpret_cast<const float*>(st + R::kBeta);
+    float* sV = reinterpret_cast<float*>(st + R::kV);
+    if (p.raw != nullptr) {
+      for (int t = warp; t < nt; t += threads / 32) {
+        float* dst = p.raw + ((s.first + t0 + t) * p.heads + h) * p.raw_cols + c_first;
+        for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = sV[t * vld + c];
+        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = beta[t];
+      }
+    } else if (p.vec_out) {
+      vector_outputs<T, DELTA>(p, sV, vld, beta, nt, lanes, gate + (long long)t0 * p.ld_gate,
+                               out + (long long)t0 * p.ldo, w, gates, wa, wb);
+    } else {
+      for (int t = warp; t < nt; t += threads / 32)
+        head_output<T, DELTA>(p, sV + t * vld, s.first + t0 + t, h, beta[t]);
+    }
+  };
+
   for (int it = 0; it < tiles; ++it) {
     const int t0 = it * kTT, nt = min(kTT, s.n - t0);
-    copies_wait<STAGES - 2>();
-    __syncthreads();       // the tile's record is there; the stage of the tile before is free
-    fetch(it + STAGES - 1);
+    copies_wait<STAGES - 3>();
+    __syncthreads();       // the tile's record and the outputs of the tile before are there
+    fetch(it + STAGES - 2);   // (into the stage of two tiles before, whose outputs are written)
     uint8_t* st = smem + it % STAGES * stage_size;
     const uint32_t sb = smem_u32(st);
     const float* beta = reinterpret_cast<const float*>(st + R::kBeta);
     float* sV = reinterpret_cast<float*>(st + R::kV);
     const bool strong = *reinterpret_cast<const float*>(st + R::kStrong) != 0.f;
-    float4 g0 = make_float4(0.f, 0.f, 0.f, 0.f), g1 = g0;
-    const int o_t = p.vec_out ? tid / lanes : 0, o_c = p.vec_out ? (tid - o_t * lanes) * 8 : 0;
-    if (p.vec_out && o_t < nt) {   // the first outputs' gates, ahead
-      g0 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
-      g1 = load4(gate + (long long)(t0 + o_t) * p.ld_gate + o_c + 4);
-    }
+    if (it > 0) put_out(it - 1);
+    if (p.vec_out && o_t < nt)   // the first outputs' gates, ahead
+      gates.load(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
     const int groups = strong ? kTT / kB : 1;
     for (int grp = 0; grp < groups; ++grp) {
-      // read-outs: [16 columns x 16 tokens]
-      float P[2][4] = {}, O[2][4] = {};
+      // read-outs [16 columns x 16 tokens]: P, what is put (beta (v - P), solved), O. The products of O do
+      // not wait for the solving.
+      float P[2][4] = {}, O[2][4] = {}, U[2][4];
+      uint32_t uh[4], ul[4], bh[4], bl[4];
+      auto mine = [&](int tok) { return !strong || tok / kB == grp; };   // (other groups wait)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          U[n][e] = sV[(n * 8 + t2 + (e & 1)) * vld + warp * 16 + g + (e >> 1) * 8];
+      constexpr int kHeld = DP <= 128 ? DP / 16 : 1;   // Z's split operands stay in registers
+      uint32_t zh[kHeld][4], zl[kHeld][4];
+      auto split_z = [&](int k) { split_left(Z[2 * k], Z[2 * k + 1], zh[k % kHeld], zl[k % kHeld]); };
 #pragma unroll
       for (int k = 0; k < DP / 16; ++k) {
-        uint32_t zh[4], zl[4], bh[4], bl[4];
-        split_left(Z[2 * k], Z[2 * k + 1], zh, zl);
+        split_z(k);
         if constexpr (DELTA) {
           load_matrices(bh, sb + R::kA + tok_cols + k * 32);
           load_matrices(bl, sb + R::kA + R::kMat + tok_cols + k * 32);
-          mma_split(P, zh, zl, bh, bl);
+          mma_split(P, zh[k % kHeld], zl[k % kHeld], bh, bl);
         }
-        load_matrices(bh, sb + R::kC + tok_cols + k * 32);
-        load_matrices(bl, sb + R::kC + R::kMat + tok_cols + k * 32);
-        mma_split(O, zh, zl, bh, bl);
       }
-      // what is put: beta (v - P), solved; a strong tile's other groups wait
-      float U[2][4];
-      auto mine = [&](int tok) { return !strong || tok / kB == grp; };
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int tok = n * 8 + t2 + (e & 1);
-          const float v = sV[tok * vld + warp * 16 + g + (e >> 1) * 8];
-          U[n][e] = !mine(tok) ? 0.f : DELTA ? beta[tok] * (v - P[n][e]) : v;
+          if (DELTA) U[n][e] = beta[tok] * (U[n][e] - P[n][e]);
+          if (!mine(tok)) U[n][e] = 0.f;
         }
-      uint32_t uh[4], ul[4], bh[4], bl[4];
       split_left(U[0], U[1], uh, ul);
       if constexpr (DELTA) {
         load_matrices(bh, sb + R::kT + tok_cols_t);
@@ -1439,8 +1530,15 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
 #pragma unroll
           for (int e = 0; e < 4; ++e) U[n][e] = 0.f;
         mma_split(U, uh, ul, bh, bl);
-        split_left(U[0], U[1], uh, ul);
       }
+#pragma unroll
+      for (int k = 0; k < DP / 16; ++k) {
+        if (kHeld == 1) split_z(k);
+        load_matrices(bh, sb + R::kC + tok_cols + k * 32);
+        load_matrices(bl, sb + R::kC + R::kMat + tok_cols + k * 32);
+        mma_split(O, zh[k % kHeld], zl[k % kHeld], bh, bl);
+      }
+      if constexpr (DELTA) split_left(U[0], U[1], uh, ul);
       load_matrices(bh, sb + R::kQ + tok_cols_t);
       load_matrices(bl, sb + R::kQ + R::kSmall + tok_cols_t);
       mma_split(O, uh, ul, bh, bl);
@@ -1467,22 +1565,10 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
         }
       }
     }
-    __syncthreads();   // the tile's outputs are there
-    if (p.raw != nullptr) {
-      for (int t = warp; t < nt; t += threads / 32) {
-        float* dst = p.raw + ((s.first + t0 + t) * p.heads + h) * p.raw_cols + c_first;
-        for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = sV[t * vld + c];
-        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = beta[t];
-      }
-    } else if (p.vec_out) {
-      vector_outputs<T, DELTA>(p, sV, vld, beta, nt, lanes, gate + (long long)t0 * p.ld_gate,
-                               out + (long long)t0 * p.ldo, w, g0, g1);
-    } else {
-      for (int t = warp; t < nt; t += threads / 32)
-        head_output<T, DELTA>(p, sV + t * vld, s.first + t0 + t, h, beta[t]);
-    }
   }
   copies_wait<0>();
+  __syncthreads();
+  put_out(tiles - 1);
 #pragma unroll
   for (int n = 0; n < kN; ++n)
 #pragma unroll
@@ -1538,14 +1624,14 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
   const dim3 tile_grid((unsigned)(n_tiles * a.heads)), tile_threads(DP <= 128 ? 128 : 256);
   if constexpr (sizeof(T) == 2) {
     using R = MmaRecord<DP, DELTA>;
-    const size_t tile_smem = (size_t)2 * kTT * DP * 4 + R::kV + kTT * (kTT + 1) * 4;
+    const size_t tile_smem = (size_t)2 * kTT * DP * 4 + R::kV + kTT * (kTT + 4) * 4;
     if (!set_smem(tile_mma_kernel<DP, DELTA>, tile_smem)) return -3;
     if (launch_pdl(tile_mma_kernel<DP, DELTA>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
       return -5;
     const size_t stage = R::bytes(a.nc);
-    const bool three = 3 * stage <= 220 * 1024;
-    auto k = three ? scan_mma_kernel<DP, DELTA, 3> : scan_mma_kernel<DP, DELTA, 2>;
-    const size_t smem = (three ? 3 : 2) * stage;
+    const bool four = 4 * stage <= 220 * 1024;
+    auto k = four ? scan_mma_kernel<DP, DELTA, 4> : scan_mma_kernel<DP, DELTA, 3>;
+    const size_t smem = (four ? 4 : 3) * stage;
     if (smem > 220 * 1024) return -6;
     if (!set_smem(k, smem)) return -3;
     return launch_pdl(k, dim3((unsigned)blocks), dim3(a.nc / 16 * 32), smem, stream, a) == cudaSuccess ? 0 : -5;
