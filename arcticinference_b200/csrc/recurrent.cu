@@ -1384,12 +1384,20 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile
   if (DELTA && t0 + nt == s.n) save_inputs<T>(p, s, in, h % p.group == 0, 0, p.vdim);
 }
 
-// A warp owns 16 columns: Z transposed, as accumulators of 16 columns by 8 rows.
+// Two warps own 16 columns, half of the rows each: Z transposed, as accumulators of 16 columns by 8 rows.
+// They add up their read-outs through shared memory; the first one writes the outputs.
+__device__ __forceinline__ void pair_sync(int pair) {
+  asm volatile("bar.sync %0, 64;" ::"r"(1 + pair) : "memory");
+}
+// floats a lane of a pair swaps: both halves of P, one of O
+__host__ __device__ constexpr int swap_floats(bool delta) { return delta ? 24 : 8; }
+
 template <int DP, bool DELTA, int STAGES>
-__global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(const ScanArgs p) {
+__global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(const ScanArgs p) {
   typedef __nv_bfloat16 T;
   using R = MmaRecord<DP, DELTA>;
-  constexpr int kN = DP / 8, kLd = R::kLd;
+  constexpr int kSwap = swap_floats(DELTA);
+  constexpr int kN = DP / 16, kSteps = DP / 32, kLd = R::kLd;   // of a warp's half of the rows
   extern __shared__ __align__(16) uint8_t smem[];
   pdl_wait();
   pdl_trigger();
@@ -1403,8 +1411,10 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
   }
   const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t2 = (lane & 3) * 2;
+  const int pairs = p.nc / 16, second = warp >= pairs, pair = warp - second * pairs;
   const int nc = p.nc, c_first = slice * nc, vld = R::vld(nc), rec_vld = R::vld(p.slices * nc);
   const int stage_size = R::bytes(nc);
+  float* swap = reinterpret_cast<float*>(smem + STAGES * stage_size) + pair * kSwap * 32 + lane;
   const int tiles = (s.n + kTT - 1) / kTT;
   const uint8_t* rec0 = reinterpret_cast<const uint8_t*>(p.records) +
                         ((long long)p.first_tile[seq] * p.heads + h) * p.record * 4;
@@ -1427,15 +1437,15 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
   // (a tile's outputs are written out while the next one's are computed: two stages are in use)
 #pragma unroll
   for (int i = 0; i < STAGES - 2; ++i) fetch(i);
-  // state: Z[n]: columns c and c + 8, rows 8 n + t2 and the next
+  // state: Z[n]: columns c and c + 8, rows r0 + 8 n + t2 and the next
   float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols;
-  const int c0 = c_first + warp * 16 + g;
+  const int c0 = c_first + pair * 16 + g, r0 = second * (DP / 2);
   float Z[kN][4];
 #pragma unroll
   for (int n = 0; n < kN; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int r = 8 * n + t2 + (e & 1), c = c0 + (e >> 1) * 8;
+      const int r = r0 + 8 * n + t2 + (e & 1), c = c0 + (e >> 1) * 8;
       Z[n][e] = s.start > 0 && r < p.dim && c < p.state_cols ? state[(long long)r * p.state_cols + c] : 0.f;
     }
   const int lanes = p.vdim / 8;
@@ -1450,9 +1460,9 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
   }
   // ldmatrix addresses within a stage: right operands with tokens as columns, and as rows
   const int m = lane >> 3, rr = lane & 7;
-  const uint32_t tok_cols = (((m >> 1) * 8 + rr) * kLd + (m & 1) * 8) * 2;
+  const uint32_t tok_cols = (((m >> 1) * 8 + rr) * kLd + (m & 1) * 8 + r0) * 2;
   const uint32_t tok_cols_t = (((m >> 1) * 8 + rr) * R::kLdT + (m & 1) * 8) * 2;
-  const uint32_t tok_rows = (((m & 1) * 8 + rr) * kLd + (m >> 1) * 8) * 2;
+  const uint32_t tok_rows = (((m & 1) * 8 + rr) * kLd + (m >> 1) * 8 + r0) * 2;
 
   // norm, weight and gate of a tile's outputs
   Raw8<T> gates = {};
@@ -1491,8 +1501,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
       gates.load(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
     const int groups = strong ? kTT / kB : 1;
     for (int grp = 0; grp < groups; ++grp) {
-      // read-outs [16 columns x 16 tokens]: P, what is put (beta (v - P), solved), O. The products of O do
-      // not wait for the solving.
+      // read-outs [16 columns x 16 tokens]: P, what is put (U = beta (v - P), solved), O
       float P[2][4] = {}, O[2][4] = {}, U[2][4];
       uint32_t uh[4], ul[4], bh[4], bl[4];
       auto mine = [&](int tok) { return !strong || tok / kB == grp; };   // (other groups wait)
@@ -1500,19 +1509,36 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e)
-          U[n][e] = sV[(n * 8 + t2 + (e & 1)) * vld + warp * 16 + g + (e >> 1) * 8];
-      constexpr int kHeld = DP <= 128 ? DP / 16 : 1;   // Z's split operands stay in registers
-      uint32_t zh[kHeld][4], zl[kHeld][4];
-      auto split_z = [&](int k) { split_left(Z[2 * k], Z[2 * k + 1], zh[k % kHeld], zl[k % kHeld]); };
+          U[n][e] = sV[(n * 8 + t2 + (e & 1)) * vld + pair * 16 + g + (e >> 1) * 8];
 #pragma unroll
-      for (int k = 0; k < DP / 16; ++k) {
-        split_z(k);
+      for (int k = 0; k < kSteps; ++k) {
+        uint32_t zh[4], zl[4];
+        split_left(Z[2 * k], Z[2 * k + 1], zh, zl);
         if constexpr (DELTA) {
           load_matrices(bh, sb + R::kA + tok_cols + k * 32);
           load_matrices(bl, sb + R::kA + R::kMat + tok_cols + k * 32);
-          mma_split(P, zh[k % kHeld], zl[k % kHeld], bh, bl);
+          mma_split(P, zh, zl, bh, bl);
         }
+        load_matrices(bh, sb + R::kC + tok_cols + k * 32);
+        load_matrices(bl, sb + R::kC + R::kMat + tok_cols + k * 32);
+        mma_split(O, zh, zl, bh, bl);
       }
+      // the other half's sums: both warps need P, the first one O
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (DELTA) swap[(second * 8 + n * 4 + e) * 32] = P[n][e];
+          if (second) swap[((DELTA ? 16 : 0) + n * 4 + e) * 32] = O[n][e];
+        }
+      pair_sync(pair);
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (DELTA) P[n][e] += swap[((second ^ 1) * 8 + n * 4 + e) * 32];
+          if (!second) O[n][e] += swap[((DELTA ? 16 : 0) + n * 4 + e) * 32];
+        }
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -1531,25 +1557,20 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
           for (int e = 0; e < 4; ++e) U[n][e] = 0.f;
         mma_split(U, uh, ul, bh, bl);
       }
-#pragma unroll
-      for (int k = 0; k < DP / 16; ++k) {
-        if (kHeld == 1) split_z(k);
-        load_matrices(bh, sb + R::kC + tok_cols + k * 32);
-        load_matrices(bl, sb + R::kC + R::kMat + tok_cols + k * 32);
-        mma_split(O, zh[k % kHeld], zl[k % kHeld], bh, bl);
-      }
       if constexpr (DELTA) split_left(U[0], U[1], uh, ul);
-      load_matrices(bh, sb + R::kQ + tok_cols_t);
-      load_matrices(bl, sb + R::kQ + R::kSmall + tok_cols_t);
-      mma_split(O, uh, ul, bh, bl);
+      if (!second) {
+        load_matrices(bh, sb + R::kQ + tok_cols_t);
+        load_matrices(bl, sb + R::kQ + R::kSmall + tok_cols_t);
+        mma_split(O, uh, ul, bh, bl);
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {   // (a lane alone reads and writes these values)
-          const int tok = n * 8 + t2 + (e & 1);
-          if (mine(tok)) sV[tok * vld + warp * 16 + g + (e >> 1) * 8] = O[n][e];
-        }
-      const float* G = reinterpret_cast<const float*>(st + R::kG) + (strong ? grp : kTT / kB - 1) * DP + t2;
+          for (int e = 0; e < 4; ++e) {   // (where the value was, which both warps have read)
+            const int tok = n * 8 + t2 + (e & 1);
+            if (mine(tok)) sV[tok * vld + pair * 16 + g + (e >> 1) * 8] = O[n][e];
+          }
+      }
+      const float* G = reinterpret_cast<const float*>(st + R::kG) + (strong ? grp : kTT / kB - 1) * DP + r0 + t2;
 #pragma unroll
       for (int n = 0; n < kN; n += 2) {
         load_matrices_trans(bh, sb + R::kB + tok_rows + n * 16);
@@ -1564,6 +1585,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
           Z[n + e][2] *= f.x; Z[n + e][3] *= f.y;
         }
       }
+      if (strong) pair_sync(pair);   // (the sums are swapped once more)
     }
   }
   copies_wait<0>();
@@ -1573,7 +1595,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_mma_kernel(cons
   for (int n = 0; n < kN; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int r = 8 * n + t2 + (e & 1), c = c0 + (e >> 1) * 8;
+      const int r = r0 + 8 * n + t2 + (e & 1), c = c0 + (e >> 1) * 8;
       if (r < p.dim && c < p.state_cols) state[(long long)r * p.state_cols + c] = Z[n][e];
     }
 }
@@ -1629,12 +1651,13 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
     if (launch_pdl(tile_mma_kernel<DP, DELTA>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
       return -5;
     const size_t stage = R::bytes(a.nc);
-    const bool four = 4 * stage <= 220 * 1024;
+    const size_t swap = (size_t)a.nc / 16 * swap_floats(DELTA) * 32 * 4;
+    const bool four = 4 * stage + swap <= 220 * 1024;
     auto k = four ? scan_mma_kernel<DP, DELTA, 4> : scan_mma_kernel<DP, DELTA, 3>;
-    const size_t smem = (four ? 4 : 3) * stage;
+    const size_t smem = (four ? 4 : 3) * stage + swap;
     if (smem > 220 * 1024) return -6;
     if (!set_smem(k, smem)) return -3;
-    return launch_pdl(k, dim3((unsigned)blocks), dim3(a.nc / 16 * 32), smem, stream, a) == cudaSuccess ? 0 : -5;
+    return launch_pdl(k, dim3((unsigned)blocks), dim3(a.nc / 16 * 64), smem, stream, a) == cudaSuccess ? 0 : -5;
   } else {
     const size_t tile_smem = (size_t)(DELTA ? 3 : 2) * kTT * DP * sizeof(float);
     if (!set_smem(tile_kernel<T, DP, DELTA>, tile_smem)) return -3;
