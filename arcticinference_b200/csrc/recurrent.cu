@@ -490,8 +490,9 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_
 
   const Inputs<T> in(p, s, h, DELTA);
   const int nv = min(p.nc, p.vdim - c_first);
-  float keep = 0.f, put = 0.f, m_new = 0.f, beta = 0.f;
+  float keep = 0.f, put = 0.f, m_new = 0.f, beta = 0.f, a_exp = 0.f;
   if (DELTA) {
+    a_exp = p.a_exp[h];
     beta = sigmoid_f(to_f32<T>(in.proj[p.b_at + h]));
   } else {
     const float2 g = memory_log_gates(to_f32<T>(in.proj[p.i_at + h]) + p.i_bias[h],
@@ -501,36 +502,75 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_
     keep = expf(g.y + m - m_new);
     put = expf(g.x - m_new);
   }
-  for (int x = tid; x < 2 * DP + p.nc; x += threads) {
-    const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
-    const int d = x - part * DP + (part == 2 ? c_first : 0);
-    const bool ok = part == 2 ? d < c_first + nv : d < p.dim;
+  // a thread's output columns: gate and norm weight, ahead
+  const T* gate = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
+  const float* norm = p.norm + (long long)h * p.norm_step;
+  T gate0 = from_f32<T>(0.f);
+  float norm0 = 0.f;
+  if (p.raw == nullptr && tid < p.vdim) {
+    gate0 = gate[tid];
+    norm0 = norm[tid];
+  }
+  // a channel a thread and turn, two turns' loads at once
+  const bool qk_block = slice == 0 && h % p.group == 0;   // saves the queries' and keys' inputs
+  T* next = reinterpret_cast<T*>(p.conv_state) + ((long long)s.slot * 2 + (s.phase ^ 1)) * in.back * p.channels;
+  struct Channel {
+    float x[kTaps], w[kTaps], z, bias;
+  };
+  const int channels = 2 * DP + p.nc;
+  auto place = [&](int x, int& part, int& d) {
+    part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
+    d = x - part * DP + (part == 2 ? c_first : 0);
+    return x < channels && (part == 2 ? d < c_first + nv : d < p.dim);
+  };
+  auto fetch = [&](int x, Channel& c) {
+    int part, d;
+    if (!place(x, part, d)) return;
+    if (DELTA) {
+      const float* w = p.conv + in.ch(part) + d;
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) {
+        const bool use = j < p.taps;
+        c.x[j] = use ? in.one(part, d, j - in.back) : 0.f;
+        c.w[j] = use ? w[(long long)j * p.channels] : 0.f;
+      }
+      if (part == 0) {
+        c.z = to_f32<T>(reinterpret_cast<const T*>(p.decay)[s.first * p.ld_decay + h * p.dim + d]);
+        c.bias = p.dt_bias[h * p.dim + d];
+      }
+    } else {
+      c.x[0] = in.one(part, d, 0);
+    }
+  };
+  auto finish = [&](int x, const Channel& c) {
+    int part, d;
+    const bool ok = place(x, part, d);
+    if (x >= channels) return;
     float y = 0.f;
     if (DELTA && ok) {
+#pragma unroll
+      for (int j = 0; j < kTaps; ++j) y = fmaf(c.w[j], c.x[j], y);
       const float* w = p.conv + in.ch(part) + d;
-      float xv[kTaps], wv[kTaps];
-#pragma unroll
-      for (int j = 0; j < kTaps; ++j) {   // all loads at once
-        const bool use = j < p.taps;
-        xv[j] = use ? in.one(part, d, j - in.back) : 0.f;
-        wv[j] = use ? w[(long long)j * p.channels] : 0.f;
-      }
-#pragma unroll
-      for (int j = 0; j < kTaps; ++j) y = fmaf(wv[j], xv[j], y);
       for (int j = kTaps; j < p.taps; ++j)
         y = fmaf(w[(long long)j * p.channels], in.one(part, d, j - in.back), y);
       y = silu_f(y);
-      if (part == 0)
-        sG[d] = expf(-p.a_exp[h] *
-                     softplus_f(to_f32<T>(reinterpret_cast<const T*>(p.decay)[s.first * p.ld_decay +
-                                                                              h * p.dim + d]) +
-                                p.dt_bias[h * p.dim + d]));
+      if (part == 2 || qk_block) {
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j)
+          if (j < in.back && p.taps <= kTaps) next[(long long)j * p.channels + in.ch(part) + d] = from_f32<T>(c.x[j + 1]);
+      }
     } else if (!DELTA) {
-      if (ok) y = in.one(part, d, 0);
-      if (part == 2 && d == p.vdim) y = 1.f;
+      y = ok ? c.x[0] : part == 2 && d == p.vdim ? 1.f : 0.f;
     }
-    if (DELTA && part == 0 && !ok) sG[d] = 1.f;
+    if (DELTA && part == 0) sG[d] = ok ? exp2_fast(-kLog2e * a_exp * softplus_f(c.z + c.bias)) : 1.f;
     (part == 0 ? sQ : part == 1 ? sK : sV)[part == 2 ? d - c_first : d] = y;
+  };
+  for (int x = tid; x < channels; x += 2 * threads) {
+    Channel a, b;
+    fetch(x, a);
+    fetch(x + threads, b);
+    finish(x, a);
+    finish(x + threads, b);
   }
   __syncthreads();
   // every warp: norms and the product of query and key
@@ -617,15 +657,14 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_
       ss = fmaf(x, x, ss);
     }
     scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
-    const T* g = reinterpret_cast<const T*>(p.gate) + s.first * p.ld_gate + (long long)h * p.vdim;
-    const float* w = p.norm + (long long)h * p.norm_step;
     T* dst = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
     for (int c = tid; c < p.vdim; c += threads)
-      dst[c] = from_f32<T>(sV[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
+      dst[c] = from_f32<T>(sV[c] * scale * (c == tid ? norm0 : norm[c]) *
+                           sigmoid_f(to_f32<T>(c == tid ? gate0 : gate[c])));
   }
-  if (DELTA)
-    save_inputs<T>(p, s, in, slice == 0 && h % p.group == 0, c_first, max(0, nv));
-  else if (slice == 0 && tid == 0)
+  if (DELTA) {
+    if (p.taps > kTaps) save_inputs<T>(p, s, in, qk_block, c_first, max(0, nv));
+  } else if (slice == 0 && tid == 0)
     p.max_state[((long long)s.slot * 2 + (s.phase ^ 1)) * p.heads + h] = m_new;
 }
 
