@@ -464,15 +464,27 @@ __device__ __forceinline__ void vector_outputs(const ScanArgs& p, const float* o
 }
 
 // ------------------------------------------------------------------ one token per sequence
+// A thread holds four neighbouring columns of kRows consecutive rows, so that a warp reads and writes
+// whole rows of the state; nc / 4 threads side by side, kGroups groups of rows.
+template <int DP>
+struct StepShape {
+  static constexpr int kGroups = DP <= 128 ? 8 : 16, kRows = DP / kGroups;
+  static constexpr int max_threads(bool delta) { return kGroups * max_warps(delta) * 4; }
+  static constexpr int smem_floats(int nc) { return 3 * DP + nc + 2 * kGroups * nc; }
+};
+
 template <typename T, int DP, bool DELTA>
-__global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_kernel(const ScanArgs p) {
-  using Sh = ScanShape<DP>;
-  constexpr int kCols = Sh::kCols, kChunks = Sh::kRows / 4;
+__global__ void __launch_bounds__(StepShape<DP>::max_threads(DELTA), DP <= 128 ? 2 : 1)
+step_kernel(const ScanArgs p) {
+  using Sh = StepShape<DP>;
+  constexpr int kRows = Sh::kRows;
   extern __shared__ __align__(16) float sm[];
   float* sQ = sm;              // query, key (before their norms), decay, values / outputs
   float* sK = sm + DP;
   float* sG = sm + 2 * DP;
   float* sV = sm + 3 * DP;
+  float* sP = sV + p.nc;       // [kGroups][nc]: S^T k of a group's rows; then what is put
+  float* sR = sP + Sh::kGroups * p.nc;   // S^T q
   pdl_wait();
   pdl_trigger();
   const int slice = blockIdx.x % p.slices, h = blockIdx.x / p.slices % p.heads;
@@ -482,11 +494,17 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_
     put_zeros<T, DELTA>(p, s, h, slice);
     return;
   }
-  const int tid = threadIdx.x, threads = blockDim.x, lane = tid & 31, rl = lane & 7;
-  const int c_first = slice * p.nc, c_local = (tid >> 5) * Sh::kWarpCols + (lane >> 3) * kCols;
-  float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols;
-  float2 S[Sh::kRows / 2][kCols];
-  load_state<DP>(S, state, p, rl, c_first + c_local, s.start > 0);
+  const int tid = threadIdx.x, threads = blockDim.x, lane = tid & 31;
+  const int quads = p.nc / 4, group = tid / quads, c_local = (tid - group * quads) * 4;
+  const int c_first = slice * p.nc, r0 = group * kRows;
+  float* state = p.state + ((long long)s.slot * p.heads + h) * p.dim * p.state_cols +
+                 (long long)r0 * p.state_cols + c_first + c_local;
+  const bool mine = c_first + c_local < p.state_cols;
+  float4 S[kRows];
+#pragma unroll
+  for (int i = 0; i < kRows; ++i)
+    S[i] = mine && s.start > 0 && r0 + i < p.dim ? load4(state + (long long)i * p.state_cols)
+                                                 : make_float4(0.f, 0.f, 0.f, 0.f);
 
   const Inputs<T> in(p, s, h, DELTA);
   const int nv = min(p.nc, p.vdim - c_first);
@@ -588,64 +606,46 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, DP <= 64 ? 3 : 2) step_
     fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
   }
   qk *= fq * fk * (DELTA ? 1.f : put);
-  constexpr int kKinds = DELTA ? 2 : 1;
-  float2 acc[kKinds][kCols][1];
+  float4 P = make_float4(0.f, 0.f, 0.f, 0.f), Q = P;
 #pragma unroll
-  for (int e = 0; e < kKinds; ++e)
+  for (int i = 0; i < kRows; i += 4) {
+    const float4 q = load4(sQ + r0 + i), k = load4(sK + r0 + i), g = load4(sG + r0 + i);
+    const float qs[4] = {q.x, q.y, q.z, q.w}, ks[4] = {k.x, k.y, k.z, k.w}, gs[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
-    for (int c = 0; c < kCols; ++c) acc[e][c][0] = make_float2(0.f, 0.f);
-#pragma unroll
-  for (int j = 0; j < kChunks; ++j) {
-    const int r = j * 32 + rl * 4;
-    const float4 q = load4(sQ + r);
-    if constexpr (DELTA) {
-      const float4 k = load4(sK + r), g = load4(sG + r);
-#pragma unroll
-      for (int c = 0; c < kCols; ++c) {   // S <- g * S; S^T k
-        mul2(S[2 * j][c], make_float2(g.x, g.y));
-        mul2(S[2 * j + 1][c], make_float2(g.z, g.w));
-        fma2(acc[0][c][0], S[2 * j][c], make_float2(k.x, k.y));
-        fma2(acc[0][c][0], S[2 * j + 1][c], make_float2(k.z, k.w));
-      }
-    }
-#pragma unroll
-    for (int c = 0; c < kCols; ++c) {
-      fma2(acc[kKinds - 1][c][0], S[2 * j][c], make_float2(q.x, q.y));
-      fma2(acc[kKinds - 1][c][0], S[2 * j + 1][c], make_float2(q.z, q.w));
+    for (int e = 0; e < 4; ++e) {   // S <- g * S; S^T k, S^T q
+      float4& x = S[i + e];
+      const float f = DELTA ? gs[e] : keep;
+      x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
+      if (DELTA) axpy4(P, make_float4(ks[e], ks[e], ks[e], ks[e]), x);
+      axpy4(Q, make_float4(qs[e], qs[e], qs[e], qs[e]), x);
     }
   }
-  float my[1];
-  const int my_c = reduce_columns<kKinds, kCols, 1>(acc, my);
-  float U[kCols], u = sV[c_local + my_c], o;
-  if constexpr (DELTA) {
-    u = beta * (u - fk * my[0]);          // (of use in lanes 0 - 3)
-#pragma unroll
-    for (int c = 0; c < kCols; ++c) U[c] = fk * __shfl_sync(0xffffffffu, u, (lane & 24) | c);
-    u = __shfl_sync(0xffffffffu, u, (lane & 24) | my_c);
-    o = fmaf(qk, u, fq * my[0]);
-  } else {
-#pragma unroll
-    for (int c = 0; c < kCols; ++c) U[c] = put * sV[c_local + c];
-    o = fmaf(qk, u, keep * fq * my[0]);
-  }
-  __syncwarp();   // the values have been read: the outputs take their place
-  if (rl >= 4 && rl < 4 + kCols) sV[c_local + my_c] = o;
-#pragma unroll
-  for (int j = 0; j < kChunks; ++j) {
-    const float4 k = load4(sK + j * 32 + rl * 4);
-#pragma unroll
-    for (int c = 0; c < kCols; ++c) {
-      if constexpr (!DELTA) {
-        mul2(S[2 * j][c], make_float2(keep, keep));
-        mul2(S[2 * j + 1][c], make_float2(keep, keep));
-      }
-      const float2 uu = make_float2(U[c], U[c]);
-      fma2(S[2 * j][c], make_float2(k.x, k.y), uu);
-      fma2(S[2 * j + 1][c], make_float2(k.z, k.w), uu);
-    }
-  }
-  store_state<DP>(S, state, p, rl, c_first + c_local);
+  if (DELTA) store4(sP + group * p.nc + c_local, P);
+  store4(sR + group * p.nc + c_local, Q);
   __syncthreads();
+  for (int c = tid; c < p.nc; c += threads) {
+    float pk = 0.f, o = 0.f, u = sV[c];
+#pragma unroll
+    for (int g = 0; g < Sh::kGroups; ++g) {
+      if (DELTA) pk += sP[g * p.nc + c];
+      o += sR[g * p.nc + c];
+    }
+    if (DELTA) u = beta * (u - fk * pk);
+    sV[c] = fmaf(qk, u, fq * o);
+    sP[c] = u * (DELTA ? fk : put);   // what the rows' keys are multiplied by
+  }
+  __syncthreads();
+  const float4 u = load4(sP + c_local);
+#pragma unroll
+  for (int i = 0; i < kRows; i += 4) {
+    const float4 k = load4(sK + r0 + i);
+    const float ks[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      axpy4(S[i + e], make_float4(ks[e], ks[e], ks[e], ks[e]), u);
+      if (mine && r0 + i + e < p.dim) store4(state + (long long)(i + e) * p.state_cols, S[i + e]);
+    }
+  }
   if (p.raw != nullptr) {
     float* dst = p.raw + (s.first * p.heads + h) * p.raw_cols + c_first;
     for (int c = tid; c < min(p.nc, p.ncols - c_first); c += threads) dst[c] = sV[c];
@@ -1668,8 +1668,12 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
   const dim3 threads(a.nc / wc * 32);
   if (blocks > 0x7fffffffll || (long long)n_tiles * a.heads > 0x7fffffffll) return -6;
   if (max_rows == 1) {
-    const size_t smem = (size_t)(3 * DP + a.nc) * sizeof(float);
-    return launch_pdl(step_kernel<T, DP, DELTA>, dim3((unsigned)blocks), threads, smem, stream, a) ==
+    using Sh = StepShape<DP>;
+    const size_t smem = (size_t)Sh::smem_floats(a.nc) * sizeof(float);
+    const dim3 step_threads(a.nc / 4 * Sh::kGroups);
+    if (step_threads.x > Sh::max_threads(DELTA)) return -2;
+    if (!set_smem(step_kernel<T, DP, DELTA>, smem)) return -3;
+    return launch_pdl(step_kernel<T, DP, DELTA>, dim3((unsigned)blocks), step_threads, smem, stream, a) ==
                    cudaSuccess
                ? 0
                : -5;
