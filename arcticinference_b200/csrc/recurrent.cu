@@ -501,10 +501,11 @@ step_kernel(const ScanArgs p) {
                  (long long)r0 * p.state_cols + c_first + c_local;
   const bool mine = c_first + c_local < p.state_cols;
   float4 S[kRows];
+  const int rows = mine ? p.dim - r0 : 0, rows_in = s.start > 0 ? rows : 0;   // of the thread's, in use
+  float* row = state;
 #pragma unroll
-  for (int i = 0; i < kRows; ++i)
-    S[i] = mine && s.start > 0 && r0 + i < p.dim ? load4(state + (long long)i * p.state_cols)
-                                                 : make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int i = 0; i < kRows; ++i, row += p.state_cols)
+    S[i] = i < rows_in ? load4(row) : make_float4(0.f, 0.f, 0.f, 0.f);
 
   const Inputs<T> in(p, s, h, DELTA);
   const int nv = min(p.nc, p.vdim - c_first);
@@ -532,9 +533,12 @@ step_kernel(const ScanArgs p) {
   // a channel a thread and turn, two turns' loads at once
   const bool qk_block = slice == 0 && h % p.group == 0;   // saves the queries' and keys' inputs
   T* next = reinterpret_cast<T*>(p.conv_state) + ((long long)s.slot * 2 + (s.phase ^ 1)) * in.back * p.channels;
-  struct Channel {
-    float x[kTaps], w[kTaps], z, bias;
+  struct Channel {   // the inputs as they lie in memory: earlier ones, the token's own
+    T old[kTaps - 1], x, z;
+    float w[kTaps], bias;
   };
+  const T* decay = reinterpret_cast<const T*>(p.decay) + s.first * p.ld_decay + h * p.dim;
+  const long long last_tap = (long long)in.back * p.channels;
   const int channels = 2 * DP + p.nc;
   auto place = [&](int x, int& part, int& d) {
     part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
@@ -546,18 +550,20 @@ step_kernel(const ScanArgs p) {
     if (!place(x, part, d)) return;
     if (DELTA) {
       const float* w = p.conv + in.ch(part) + d;
+      const T* o = in.old + in.ch(part) + d;
+      c.x = in.proj[in.col(part) + d];
+      c.w[kTaps - 1] = w[last_tap];
 #pragma unroll
-      for (int j = 0; j < kTaps; ++j) {
-        const bool use = j < p.taps;
-        c.x[j] = use ? in.one(part, d, j - in.back) : 0.f;
-        c.w[j] = use ? w[(long long)j * p.channels] : 0.f;
+      for (int j = 0; j < kTaps - 1; ++j, w += p.channels, o += p.channels) {
+        c.w[j] = j < in.back ? *w : 0.f;
+        c.old[j] = j < in.back && s.start + j >= in.back ? *o : from_f32<T>(0.f);
       }
       if (part == 0) {
-        c.z = to_f32<T>(reinterpret_cast<const T*>(p.decay)[s.first * p.ld_decay + h * p.dim + d]);
+        c.z = decay[d];
         c.bias = p.dt_bias[h * p.dim + d];
       }
     } else {
-      c.x[0] = in.one(part, d, 0);
+      c.x = in.proj[in.col(part) + d];
     }
   };
   auto finish = [&](int x, const Channel& c) {
@@ -566,21 +572,24 @@ step_kernel(const ScanArgs p) {
     if (x >= channels) return;
     float y = 0.f;
     if (DELTA && ok) {
+      y = c.w[kTaps - 1] * to_f32<T>(c.x);
 #pragma unroll
-      for (int j = 0; j < kTaps; ++j) y = fmaf(c.w[j], c.x[j], y);
-      const float* w = p.conv + in.ch(part) + d;
-      for (int j = kTaps; j < p.taps; ++j)
-        y = fmaf(w[(long long)j * p.channels], in.one(part, d, j - in.back), y);
-      y = silu_f(y);
-      if (part == 2 || qk_block) {
+      for (int j = 0; j < kTaps - 1; ++j) y = fmaf(c.w[j], to_f32<T>(c.old[j]), y);
+      if (p.taps > kTaps) {   // (the first ones are there)
+        const float* w = p.conv + in.ch(part) + d;
+        for (int j = kTaps - 1; j < in.back; ++j)
+          y = fmaf(w[(long long)j * p.channels], in.one(part, d, j - in.back), y);
+      } else if (part == 2 || qk_block) {
+        T* o = next + in.ch(part) + d;
 #pragma unroll
-        for (int j = 0; j < kTaps - 1; ++j)
-          if (j < in.back && p.taps <= kTaps) next[(long long)j * p.channels + in.ch(part) + d] = from_f32<T>(c.x[j + 1]);
+        for (int j = 0; j < kTaps - 1; ++j, o += p.channels)
+          if (j < in.back) *o = j == in.back - 1 ? c.x : c.old[j + 1 < kTaps - 1 ? j + 1 : j];
       }
+      y = silu_f(y);
     } else if (!DELTA) {
-      y = ok ? c.x[0] : part == 2 && d == p.vdim ? 1.f : 0.f;
+      y = ok ? to_f32<T>(c.x) : part == 2 && d == p.vdim ? 1.f : 0.f;
     }
-    if (DELTA && part == 0) sG[d] = ok ? exp2_fast(-kLog2e * a_exp * softplus_f(c.z + c.bias)) : 1.f;
+    if (DELTA && part == 0) sG[d] = ok ? exp2_fast(-kLog2e * a_exp * softplus_f(to_f32<T>(c.z) + c.bias)) : 1.f;
     (part == 0 ? sQ : part == 1 ? sK : sV)[part == 2 ? d - c_first : d] = y;
   };
   for (int x = tid; x < channels; x += 2 * threads) {
@@ -636,6 +645,7 @@ step_kernel(const ScanArgs p) {
   }
   __syncthreads();
   const float4 u = load4(sP + c_local);
+  row = state;
 #pragma unroll
   for (int i = 0; i < kRows; i += 4) {
     const float4 k = load4(sK + r0 + i);
@@ -643,7 +653,8 @@ step_kernel(const ScanArgs p) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       axpy4(S[i + e], make_float4(ks[e], ks[e], ks[e], ks[e]), u);
-      if (mine && r0 + i + e < p.dim) store4(state + (long long)(i + e) * p.state_cols, S[i + e]);
+      if (i + e < rows) store4(row, S[i + e]);
+      row += p.state_cols;
     }
   }
   if (p.raw != nullptr) {
