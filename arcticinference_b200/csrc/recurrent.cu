@@ -1136,13 +1136,13 @@ struct MmaRecord {
   static constexpr int kMat = kTT * kLd * 2, kSmall = kTT * kLdT * 2;
   static constexpr int kB = 0, kC = 2 * kMat, kA = 4 * kMat, kQ = (DELTA ? 6 : 4) * kMat;
   static constexpr int kT = kQ + 2 * kSmall, kG = kT + (DELTA ? 2 * kSmall : 0);
-  static constexpr int kBeta = kG + 4 * DP * 4, kStrong = kBeta + kTT * 4, kV = kStrong + 16;
+  static constexpr int kBeta = kG + 4 * DP * 4, kGroups = kBeta + kTT * 4, kV = kGroups + 16;
   __host__ __device__ static constexpr int vld(int cols) { return cols + 4; }
   __host__ __device__ static constexpr int bytes(int cols) { return kV + kTT * vld(cols) * 4; }
 };
 
 template <int DP, bool DELTA>
-__global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile_mma_kernel(const ScanArgs p) {
+__global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 4 : 6) tile_mma_kernel(const ScanArgs p) {
   typedef __nv_bfloat16 T;
   using R = MmaRecord<DP, DELTA>;
   constexpr int kThreads = DP <= 128 ? 128 : 256, kWarps = kThreads / 32, kLd = R::kLd;
@@ -1296,7 +1296,6 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile
     if (half) {
 #pragma unroll
       for (int t = 0; t < 8; ++t) z[t] = make_float2(z[t].x + bx, z[t].y + by);
-      cum = z[7];
     }
   }
   __syncthreads();
@@ -1324,17 +1323,19 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile
       c += invQ[half * 8 + t];
       z[t] = make_float2(c, c);
     }
-    cum = make_float2(c, c);
   }
-  const bool strong = __syncthreads_or(fminf(cum.x, cum.y) < kTileLogDecay * kLog2e);
+  // one group of tokens, or two or four where 1 / G would leave its range
+  const float2 other = make_float2(__shfl_xor_sync(0xffffffffu, z[7].x, 16),
+                                   __shfl_xor_sync(0xffffffffu, z[7].y, 16));
+  const float2 first = half ? other : z[7], whole = half ? z[7] : other;   // logs of the half, the tile
+  const float low = kTileLogDecay * kLog2e;
+  const bool deep = __syncthreads_or(fminf(whole.x, whole.y) < low);
+  const bool deeper = __syncthreads_or(fminf(fminf(first.x, first.y),
+                                             fminf(whole.x - first.x, whole.y - first.y)) < low);
+  const int groups = !deep ? 1 : !deeper ? 2 : kTT / kB;
   // ---- 3. a, b, c and the groups' decays
   if (tid < DP) {
-    float2 base = make_float2(0.f, 0.f);
-    if (strong) {   // logs from the group's start: the second half's begins where the first ends
-      base.x = __shfl_xor_sync(0xffffffffu, z[7].x, 16);
-      base.y = __shfl_xor_sync(0xffffffffu, z[7].y, 16);
-      if (!half) base = make_float2(0.f, 0.f);
-    }
+    float2 base = half && groups > 1 ? first : make_float2(0.f, 0.f);   // logs at the group's start
     float* G = reinterpret_cast<float*>(mats + R::kG);
 #pragma unroll
     for (int t = 0; t < 8; ++t) {
@@ -1357,12 +1358,12 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile
       if (DELTA) split_to(R::kA, kx * gx, ky * gy);
       if (tok % kB == kB - 1) {
         *reinterpret_cast<float2*>(G + tok / kB * DP + d0) = make_float2(gx, gy);
-        if (strong) base = z[t];
+        if (groups == kTT / kB) base = z[t];
       }
     }
   }
   if (tid < kTT) reinterpret_cast<float*>(mats + R::kBeta)[tid] = beta[tid];
-  if (tid == 0) *reinterpret_cast<float4*>(mats + R::kStrong) = make_float4(strong ? 1.f : 0.f, 0.f, 0.f, 0.f);
+  if (tid == 0) *reinterpret_cast<float4*>(mats + R::kGroups) = make_float4((float)groups, 0.f, 0.f, 0.f);
   __syncthreads();
   // ---- 4. products of the tokens: the first warp c . b, the second a . b; the others write the rest out
   constexpr int kGram = DELTA ? 2 : 1;
@@ -1393,7 +1394,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP <= 128 ? 4 : 2) tile
 #pragma unroll
       for (int e = 0; e < 4; e += 2) {
         const int i = g + (e >> 1) * 8, j = nb * 8 + t2;
-        const bool same = !strong || i / kB == j / kB;   // (j and j + 1 are of one group)
+        const bool same = i * groups / kTT == j * groups / kTT;   // (j and j + 1 are of one group)
         if (warp == 0) {
           uint32_t hi, lo;
           split2(same && j <= i ? acc[nb][e] : 0.f, same && j + 1 <= i ? acc[nb][e + 1] : 0.f, hi, lo);
@@ -1545,16 +1546,15 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
     const uint32_t sb = smem_u32(st);
     const float* beta = reinterpret_cast<const float*>(st + R::kBeta);
     float* sV = reinterpret_cast<float*>(st + R::kV);
-    const bool strong = *reinterpret_cast<const float*>(st + R::kStrong) != 0.f;
+    const int groups = (int)*reinterpret_cast<const float*>(st + R::kGroups);
     if (it > 0) put_out(it - 1);
     if (p.vec_out && o_t < nt)   // the first outputs' gates, ahead
       gates.load(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
-    const int groups = strong ? kTT / kB : 1;
     for (int grp = 0; grp < groups; ++grp) {
       // read-outs [16 columns x 16 tokens]: P, what is put (U = beta (v - P), solved), O
       float P[2][4] = {}, O[2][4] = {}, U[2][4];
       uint32_t uh[4], ul[4], bh[4], bl[4];
-      auto mine = [&](int tok) { return !strong || tok / kB == grp; };   // (other groups wait)
+      auto mine = [&](int tok) { return tok * groups / kTT == grp; };   // (other groups wait)
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -1620,7 +1620,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
             if (mine(tok)) sV[tok * vld + pair * 16 + g + (e >> 1) * 8] = O[n][e];
           }
       }
-      const float* G = reinterpret_cast<const float*>(st + R::kG) + (strong ? grp : kTT / kB - 1) * DP + r0 + t2;
+      const float* G = reinterpret_cast<const float*>(st + R::kG) + ((grp + 1) * (kTT / kB) / groups - 1) * DP + r0 + t2;
 #pragma unroll
       for (int n = 0; n < kN; n += 2) {
         load_matrices_trans(bh, sb + R::kB + tok_rows + n * 16);
@@ -1635,7 +1635,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
           Z[n + e][2] *= f.x; Z[n + e][3] *= f.y;
         }
       }
-      if (strong) pair_sync(pair);   // (the sums are swapped once more)
+      if (groups > 1) pair_sync(pair);   // (the sums are swapped once more)
     }
   }
   copies_wait<0>();

@@ -386,8 +386,8 @@ class DeltaMixer(StatefulMixer):
         yield "mix.A_log", rnd(m.heads, std=0.5)
         yield "mix.norm", 1.0 + rnd(m.vdim, std=0.1)
         yield "mix.a1", rnd(rank, W)
-        yield "mix.a2", rnd(m.heads * m.dim, rank)
-        yield "mix.dt_bias", rnd(m.heads * m.dim, std=0.5) - 4.0     # slow decays
+        yield "mix.a2", rnd(m.heads * m.dim, rank, std=0.25 * rank ** -0.5)     # slow decays
+        yield "mix.dt_bias", rnd(m.heads * m.dim, std=0.5) - 4.0
         yield "mix.g1", rnd(rank, W)
         yield "mix.g2", rnd(nv, rank)
         yield "mix.o", rnd(W, nv)
