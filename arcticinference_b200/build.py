@@ -81,7 +81,7 @@ KERNEL_SETS = {
     "Zatirax": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm",
                 "latent_attention", "rotary", "sampling", "stream"),
     "Pererax": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm", "moe", "recurrent",
-                "rotary", "sampling", "stream"),
+                "recurrent_mma", "rotary", "sampling", "stream"),
 }
 _kernel_set: str | None = None
 
