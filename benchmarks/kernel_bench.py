@@ -152,6 +152,13 @@ CASES = {
     "silu_mul": ("silu", (8192, 14336)),
     "silu_mul_quant": ("silu_q", (8192, 14336)),
     "quant_fp8_row": ("quant_row", (8192, 4096)),
+    # recurrent layers (keys and values of 128; the matrix memory's keys of 64): heads, sequences, tokens
+    "delta_prefill_4x2048": ("delta", (32, 4, 2048)),
+    "delta_prefill_4x256": ("delta", (32, 4, 256)),
+    "delta_decode_128": ("delta", (32, 128, 1)),
+    "delta_decode_64": ("delta", (32, 64, 1)),
+    "memory_prefill_4x2048": ("memory", (16, 4, 2048)),
+    "memory_decode_128": ("memory", (16, 128, 1)),
 }
 
 
@@ -298,6 +305,33 @@ def run_case(a, case):
         fn = lambda i=0: lat.latent_rope_cache(sets[i][0], sets[i][0][:, nq:], H, dim + rot, dim, w,
                                                rank, table, 1e-6, at, sets[i][1], rank)
         flops = 0.0
+    elif kind in ("delta", "memory"):
+        import numpy as np
+        from arcticinference_b200.ops import state_ops as states
+        H, nseq, n = prm
+        T, dv, d = nseq * n, 128, 128 if kind == "delta" else 64
+        nk, nv, bf16 = H * d, H * dv, torch.bfloat16
+        rnd = lambda *s: torch.randn(*s, device=DEV)
+        step = states.StateStep.build(np.asarray([(i * n, n, i + 1, 0 if n > 1 else 5, 0)
+                                                  for i in range(nseq)], dtype=np.int32), DEV)
+        cols = dv if kind == "delta" else dv + 4
+        byts = 2.0 * T * (2 * nk + 3 * nv + (nk if kind == "delta" else 0)) + \
+            4.0 * nseq * H * d * cols * (1 if n > 1 else 2)
+        flops = (6.0 if kind == "delta" else 4.0) * T * H * d * dv
+        nc = copies_for(byts)
+        if kind == "delta":
+            sh = states.DeltaShape(H, H, d, dv, 4, 0, nk, 2 * nk, 2 * nk + nv)
+            w = (rnd(4, sh.channels), torch.rand(H, device=DEV) + 0.5, rnd(nk) * 0.5 - 4, rnd(dv))
+            sets = [(R(T, 2 * nk + nv + H), R(T, nk + nv), rnd(nseq + 1, H, d, cols),
+                     rnd(nseq + 1, 2, 3, sh.channels).to(bf16)) for _ in range(nc)]
+            fn = lambda i=0: states.delta_scan(sets[i][0], sets[i][1], sets[i][1][:, nk:], *w, sh,
+                                               *sets[i][2:], step, 1e-6)
+        else:
+            sh = states.MemoryShape(H, d, dv, 15.0, 0, nk, 2 * nk, 2 * nk + nv, 2 * nk + nv + H)
+            w = (rnd(H), rnd(H) + 4, rnd(nv))
+            sets = [(R(T, 2 * nk + nv + 2 * H), R(T, nv), rnd(nseq + 1, H, d, cols), rnd(nseq + 1, 2, H))
+                    for _ in range(nc)]
+            fn = lambda i=0: states.memory_scan(*sets[i][:2], *w, sh, *sets[i][2:], step, 1e-6)
     elif kind == "sandwich":
         from arcticinference_b200.ops import stream_ops as st
         T, W = prm

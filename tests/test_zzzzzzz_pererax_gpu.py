@@ -431,3 +431,29 @@ def test_preemption_sampling_and_sleep(tmp_path):
     a = plain.generate(prompts, [hot, sp, hot])
     assert a[1].outputs[0].token_ids == want[1] and len(a[0].outputs[0].token_ids) == 8
     ops.check_status()
+
+
+def test_states_after_portions_and_after_single_tokens_agree():
+    """The state of a 16-bit model's recurrences is fp32: portions (tensor cores, operands of 16 bits)
+    leave what one-token steps (fp32 multiply-adds) leave."""
+    n = 70
+    s, proj, decay, gate, w = delta_case(2, 1, 64, 96, 4, [n], seed=5)
+    args = [t.to(DEV) for t in (proj.to(BF16), decay.to(BF16), gate.to(BF16), *w.values())]
+    nk, nv = 2 * 64, 2 * 96
+    ms = states.MemoryShape(2, 64, 96, 8.0, 0, nk, 2 * nk, 2 * nk + nv, 2 * nk + nv + 2)
+    mem = [rnd(n, 2 * nk + nv + 4), rnd(n, nv), rnd(2, dtype=F32), rnd(2, dtype=F32) + 4, rnd(nv, dtype=F32)]
+    left = []
+    for cuts in ([n], [1] * n):
+        S, conv = torch.zeros(2, 2, 64, 96, device=DEV), torch.zeros(2, 2, 3, s.channels, dtype=BF16, device=DEV)
+        Z, top = torch.zeros(2, 2, 64, ms.state_cols, device=DEV), torch.zeros(2, 2, 2, device=DEV)
+        at = phase = 0
+        for k in cuts:
+            step = states.StateStep.build(np.asarray([(0, k, 1, at, phase)], dtype=np.int32), DEV)
+            r = slice(at, at + k)
+            states.delta_scan(*(t[r] for t in args[:3]), *args[3:], s, S, conv, step, 1e-6)
+            states.memory_scan(*(t[r] for t in mem[:2]), *mem[2:], ms, Z, top, step, 1e-6)
+            at, phase = at + k, phase ^ 1
+        left.append((S[1], conv[1, phase].float(), Z[1], top[1, phase]))
+    ops.check_status()
+    for a, b in zip(*left):
+        assert float((a - b).abs().max()) < 1e-4 * float(b.abs().max())
