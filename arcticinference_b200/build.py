@@ -82,6 +82,8 @@ KERNEL_SETS = {
                 "latent_attention", "rotary", "sampling", "stream"),
     "Pererax": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm", "moe", "recurrent",
                 "recurrent_mma", "rotary", "sampling", "stream"),
+    "Pefivik": ("attention", "elementwise", "exact", "gemm_bf16", "grouped_gemm", "latent_attention",
+                "moe", "recurrent", "recurrent_mma", "sampling", "stream"),
 }
 _kernel_set: str | None = None
 

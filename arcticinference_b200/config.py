@@ -99,6 +99,9 @@ class LatentAttentionSpec:
     rot_dim: int = 0
     rotary: Optional[RotarySpec] = None
     mask: MaskSpec = MaskSpec()
+    # a further term of the softmax denominator: exp of a "learned" number per head, or None
+    sink: Optional[str] = None
+    head_gate: bool = False     # heads' outputs times sigmoid of one projected number per head
 
 
 @dataclass(frozen=True)
@@ -146,6 +149,16 @@ class MatrixMemorySpec:
 
 
 @dataclass(frozen=True)
+class ForgetScanSpec:
+    """Linear attention whose forget gate also decides what is written (HGRN2): a [dim, vdim] state
+    per head, f = lower + (1 - lower) * sigmoid(projection + bias) per channel, and 1 - f in the
+    place of a key."""
+    heads: int
+    dim: int
+    vdim: int
+
+
+@dataclass(frozen=True)
 class ParallelSpec:
     """Two mixers that read the same input; the result is half the sum of their normed outputs."""
     left: AttentionSpec
@@ -159,21 +172,28 @@ def mixer_parts(m) -> tuple:
 
 def has_state(m) -> bool:
     """Whether a mixer carries a state from token to token, which cannot be taken back."""
-    return any(isinstance(x, (DeltaRuleSpec, MatrixMemorySpec)) for x in mixer_parts(m))
+    return any(isinstance(x, (DeltaRuleSpec, MatrixMemorySpec, ForgetScanSpec))
+               for x in mixer_parts(m))
 
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
-    """A gated feed-forward layer, or ``experts`` of them of which every token uses ``top``."""
+    """A gated feed-forward layer, or ``experts`` of them of which every token uses ``top``; with the
+    activation ``poly_norm`` one without a gate and with biases."""
     ff: int
-    act: str = "silu"     # silu | gelu_tanh | clamped_swish (see ops.stream_ops.GATES)
+    act: str = "silu"     # silu | gelu_tanh | clamped_swish (ops.stream_ops.Gate) | poly_norm
     experts: int = 0      # 0: dense
     top: int = 0
     limit: float = 0.0    # clamped_swish: bound of gate (above) and up (both sides)
     # router: "chosen" (largest logits plus bias, softmax over the chosen ones) or "all" (softmax
-    # over all; a correction enters the choice, not the weights; weights times ``router_scale``)
+    # over all; a correction enters the choice, not the weights; weights times ``router_scale``) or
+    # "sigmoid" (of each logit; chosen among the ``keep_groups`` best of ``groups`` groups of
+    # neighbours, a group's score being the sum of its two best; the chosen scores are normalised to
+    # the sum ``router_scale``)
     scoring: str = "chosen"
     router_scale: float = 1.0
+    groups: int = 1
+    keep_groups: int = 1
     identity: int = 0     # further router outputs behind the experts' whose expert is the identity
     shared: Optional["FeedForwardSpec"] = None   # runs for every token beside the chosen ones
 
@@ -181,7 +201,7 @@ class FeedForwardSpec:
 @dataclass(frozen=True)
 class LayerSpec:
     """One decoder layer of a model that lists its layers one by one."""
-    mixer: Any            # AttentionSpec | LatentAttentionSpec | DeltaRuleSpec | ParallelSpec
+    mixer: Any            # AttentionSpec | LatentAttentionSpec | DeltaRuleSpec | ForgetScanSpec | ...
     mlp: Optional[FeedForwardSpec] = None
     weights_of: Optional[int] = None    # layer whose tensors this one uses (cache and state are its own)
 
@@ -190,10 +210,20 @@ class LayerSpec:
 class LoopSpec:
     """The slice ``[start, stop)`` of the layer list is executed ``times`` times before the layers
     behind it. Passes share weights, not caches; a learned vector per pass is added to the stream as
-    the pass begins."""
+    the pass begins, and with ``reenter`` the embedding before it, from the second pass on."""
     start: int
     stop: int
     times: int
+    reenter: bool = False
+
+
+@dataclass(frozen=True)
+class BigramSpec:
+    """A second embedding, looked up by (previous token * mul_prev + token * mul_cur) mod buckets; a
+    sequence's first token has the row behind the others."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass(frozen=True)
@@ -201,10 +231,12 @@ class LayerListDesign:
     """What the name of a layer-list architecture stands for, beyond the numbers of config.json.
 
     ``residual``: where the norms are. "post": x <- norm(alpha * x + f(x)); "sandwich":
-    x <- x + norm_b(f(norm_a(x))); "output": x <- x + norm(f(x)) * scale. ``norm_offset``: added to
-    the stored weights of the stream's norms. ``masks``: kind of each mixer type's mask.
-    ``attention``: options of :class:`AttentionSpec` by mixer type ("left": the attention side of
-    a parallel mixer). ``scoring``: the router's. ``tied``: the embedding is the output matrix."""
+    x <- x + norm_b(f(norm_a(x))); "output": x <- x + norm(f(x)) * scale; "pre": x <- x +
+    residual_mult * f(norm(x)). ``norm_offset``: added to the stored weights of the stream's norms.
+    ``scalar_norms``: those weights are one number for all coordinates. ``masks``: kind of each mixer
+    type's mask. ``attention``: options of :class:`AttentionSpec` or :class:`LatentAttentionSpec` by
+    mixer type ("left": the attention side of a parallel mixer). ``scoring``: the router's.
+    ``loop_reenters``: see :class:`LoopSpec`. ``tied``: the embedding is the output matrix."""
     residual: str
     norm_offset: float
     dense_act: str
@@ -215,6 +247,8 @@ class LayerListDesign:
     expert_act: str = "silu"
     scoring: str = "chosen"
     tied: bool = False
+    scalar_norms: bool = False
+    loop_reenters: bool = False
 
 
 LAYER_LIST_DESIGNS = {
@@ -232,6 +266,10 @@ LAYER_LIST_DESIGNS = {
                                                             values_are_keys=True),
                                           "left": dict(qk_norm="projection", sink="zero")},
                                expert_act="clamped_swish", scoring="all", tied=True),
+    "Pefivik": LayerListDesign(residual="pre", norm_offset=0.0, dense_act="poly_norm",
+                               mixers=("latent_attention", "hgrn2"), feed_forwards=("dense", "moe"),
+                               attention={"latent_attention": dict(sink="learned", head_gate=True)},
+                               scoring="sigmoid", scalar_norms=True, loop_reenters=True),
 }
 
 
@@ -253,6 +291,8 @@ def _read_mixer(kind: str, m: dict, design: LayerListDesign):
     if kind == "channel_delta":
         return DeltaRuleSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
                              vdim=int(m["vdim"]), conv=int(m["conv"]))
+    if kind == "hgrn2":
+        return ForgetScanSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
     rotary, mask = _read_rotary(m.get("rot")), MaskSpec()
     if m.get("mask") is not None:
         mask = MaskSpec(design.masks[kind], int(m["mask"]["size"]))
@@ -265,15 +305,17 @@ def _read_mixer(kind: str, m: dict, design: LayerListDesign):
                              **options, **shape)
     src = m.get("kv_from")
     return LatentAttentionSpec(kv_rank=int(m["kv_rank"]), rot_dim=int(m.get("rot_dim") or 0),
-                               kv_from=None if src is None else int(src), **shape)
+                               kv_from=None if src is None else int(src), **options, **shape)
 
 
 def _read_experts(f: dict, design: LayerListDesign) -> FeedForwardSpec:
     gated = lambda d: dict(ff=int(d["ff"]), act=design.expert_act, limit=float(d.get("limit", 0.0)))
     r, shared = f["router"], f.get("shared")
+    groups = r.get("groups") or {"count": 1, "keep": 1}
     return FeedForwardSpec(experts=int(r["experts"]), top=int(r["top"]), scoring=design.scoring,
                            router_scale=float(r.get("scale", 1.0)),
                            identity=int(r.get("identity") or 0),
+                           groups=int(groups["count"]), keep_groups=int(groups["keep"]),
                            shared=FeedForwardSpec(**gated(shared)) if shared else None,
                            **gated(f["expert"]))
 
@@ -316,6 +358,8 @@ def _validate_mixer(i: int, m, specs: tuple) -> None:
         if m.conv < 1:
             raise ValueError("layer %d: a convolution of %d taps" % (i, m.conv))
         return
+    if isinstance(m, ForgetScanSpec):
+        return
     if m.mask.kind != "causal" and m.mask.size < 1:
         raise ValueError("layer %d: a %s of %d positions" % (i, m.mask.kind, m.mask.size))
     if m.rotary is not None and (m.rotary.dims % 2 or m.rotary.dims < 0):
@@ -344,6 +388,12 @@ def _validate_mixer(i: int, m, specs: tuple) -> None:
 def _validate_feed_forward(i: int, f: FeedForwardSpec) -> None:
     if f.experts and not 1 <= f.top <= f.experts + f.identity:
         raise ValueError("layer %d: top must lie between 1 and the number of experts" % i)
+    if f.ff < 1:
+        raise ValueError("layer %d: ff must be positive" % i)
+    if f.experts and (f.groups < 1 or f.experts % f.groups or not 1 <= f.keep_groups <= f.groups):
+        raise ValueError("layer %d: router.groups must divide the experts, and keep some of them" % i)
+    if f.experts and f.groups > 1 and f.top > f.keep_groups * (f.experts // f.groups):
+        raise ValueError("layer %d: top exceeds the experts of the kept groups" % i)
     if f.identity < 0:
         raise ValueError("layer %d: router.identity must not be negative" % i)
     if f.act == "clamped_swish" and not f.limit > 0:
@@ -393,7 +443,7 @@ def weights_index(specs: tuple, i: int) -> int:
 @dataclass
 class ModelConfig:
     """Architecture of a decoder (Llama, Mistral, Qwen2 and Qwen3 dense models, optionally
-    SwiftKV for Llama; Taralix, Zatirax and Pererax, which list their layers one by one) or
+    SwiftKV for Llama; Taralix, Zatirax, Pererax and Pefivik, which list their layers one by one) or
     encoder (BERT)."""
 
     architecture: str = "LlamaForCausalLM"
@@ -427,6 +477,10 @@ class ModelConfig:
     # factor of the residual stream in "norm after the sum" layers: x <- norm(alpha * x + f(x))
     postln_alpha: float = 1.0
     embedding_scale: float = 1.0
+    bigram: Optional[BigramSpec] = None
+    # factor of every sublayer's output in "pre" layers: x <- x + residual_mult * f(norm(x))
+    residual_mult: float = 1.0
+    logit_softcap: float = 0.0  # logits become softcap * tanh(logits / softcap); 0: they do not
     loop: Optional[LoopSpec] = None
     # encoder-only fields
     type_vocab_size: int = 2
@@ -491,6 +545,10 @@ class ModelConfig:
     def validate(self) -> None:
         if self.layer_specs is not None:
             validate_layer_specs(self.layer_specs, self.loop)
+            if self.bigram is not None and self.bigram.buckets < 1:
+                raise ValueError("embedding.bigram.buckets must be positive")
+            if self.logit_softcap < 0:
+                raise ValueError("logit_softcap must not be negative")
             if self.quantization is not None:
                 raise NotImplementedError("quantization=%r for %s" % (self.quantization,
                                                                       self.architecture))
@@ -562,7 +620,8 @@ class ModelConfig:
     @classmethod
     def from_layer_list(cls, d: dict, name_or_path: str = "") -> "ModelConfig":
         """config.json of a layer-list model (``architecture``, ``width``, ``vocab``, ``norm`` and
-        ``layers``; by design ``postln_alpha``, ``embedding.scale``, ``loop``). The head fields
+        ``layers``; by design ``postln_alpha``, ``residual_mult``, ``embedding.scale``,
+        ``embedding.bigram``, ``logit_softcap``, ``loop``). The head fields
         describe the cache as the engine sees it: one "head" of as many numbers as the widest
         layer keeps per token."""
         design = LAYER_LIST_DESIGNS[d["architecture"]]
@@ -575,7 +634,8 @@ class ModelConfig:
             if isinstance(m, AttentionSpec):
                 return m.kv_heads * (m.dim + m.vdim)
             return m.kv_rank + m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim
-        eos, loop = d.get("eos_token_id"), d.get("loop")
+        eos, loop, emb = d.get("eos_token_id"), d.get("loop"), d.get("embedding") or {}
+        bigram = emb.get("bigram")
         return cls(
             architecture=d["architecture"], model_type=d["architecture"].lower(),
             hidden_size=int(d["width"]), num_hidden_layers=len(specs),
@@ -584,9 +644,13 @@ class ModelConfig:
             intermediate_size=max((l.mlp.ff for l in specs if l.mlp is not None), default=0),
             vocab_size=int(d["vocab"]), rms_norm_eps=float(d["norm"]["eps"]),
             postln_alpha=float(d["postln_alpha"]) if design.residual == "post" else 1.0,
-            embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+            embedding_scale=float(emb.get("scale", 1.0)),
+            bigram=None if not bigram else BigramSpec(*(int(bigram[k]) for k in (
+                "buckets", "mul_prev", "mul_cur"))),
+            residual_mult=float(d["residual_mult"]) if design.residual == "pre" else 1.0,
+            logit_softcap=float(d.get("logit_softcap") or 0.0),
             loop=None if not loop else LoopSpec(int(loop["start"]), int(loop["stop"]),
-                                                int(loop["times"])),
+                                                int(loop["times"]), design.loop_reenters),
             layer_specs=specs, tie_word_embeddings=design.tied,
             # no table is indexed by position, so nothing bounds it
             max_position_embeddings=1 << 20, hidden_act="",
@@ -686,6 +750,27 @@ def _pererax(width, vocab, layers, eps=1e-6) -> ModelConfig:
                                         "norm": {"eps": eps}, "layers": out})
 
 
+def _pefivik(width, vocab, layers, loop, bigram, mult=0.5, cap=30.0, eps=1e-6) -> ModelConfig:
+    """``layers``: (mixer, feed-forward) each; the feed-forward is None, ff (dense) or (ff, experts,
+    top, (groups, kept), ff of the shared expert)."""
+    out = []
+    for m, f in layers:
+        mlp = None
+        if isinstance(f, int):
+            mlp = {"kind": "dense", "ff": f}
+        elif f is not None:
+            mlp = {"kind": "moe", "expert": {"ff": f[0]}, "shared": {"ff": f[4]} if f[4] else None,
+                   "router": {"experts": f[1], "top": f[2], "scale": 1.5,
+                              "groups": dict(zip(("count", "keep"), f[3]))}}
+        out.append({"type": "latent_attention" if "kv_rank" in m else "hgrn2", "mixer": m,
+                    "mlp": mlp})
+    return ModelConfig.from_layer_list({
+        "architecture": "Pefivik", "width": width, "vocab": vocab, "norm": {"eps": eps},
+        "embedding": {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))},
+        "residual_mult": mult, "logit_softcap": cap, "layers": out,
+        "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop))})
+
+
 def _llama(layers, hidden, heads, kv, inter, **kw) -> ModelConfig:
     return ModelConfig(hidden_size=hidden, num_hidden_layers=layers, num_attention_heads=heads,
                        num_key_value_heads=kv, head_dim=128, intermediate_size=inter, **kw)
@@ -769,6 +854,11 @@ PRESETS: dict[str, ModelConfig] = {
           "right": {"heads": 3, "dim": 24, "vdim": 40, "gate_cap": 10.0}}, (48, 4, 1, 2, 0)),
         ({"heads": 6, "kv_heads": 3, "dim": 32, "vdim": 32, "scale": 0.18, "mask": {"size": 50},
           "rot": {"base": 10000.0, "dims": 32}}, None), 0, 1]),
+    "pefivik-tiny": _pefivik(160, 1024, [
+        ({"heads": 5, "dim": 40, "vdim": 24, "kv_rank": 56, "scale": 0.16}, 288),
+        ({"heads": 3, "dim": 56, "vdim": 40}, (48, 10, 3, (5, 2), 72)),
+        ({"heads": 4, "dim": 32, "vdim": 48, "kv_rank": 72, "scale": 0.18}, None)], loop=(1, 3, 2),
+        bigram=(301, 13, 7)),
 }
 
 

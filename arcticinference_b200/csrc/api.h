@@ -112,11 +112,12 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
                         int max_blocks, const void* work, int num_work, const void* tok_splits,
                         int max_splits, long long T, int Hq, int Hkv, int Dk, int D, int mask_kind,
                         int mask_size, const void* sink, const void* gate, long long ldg,
-                        float scale, float softcap, void* out, long long ldo, void* o_part, void* lse_part,
-                        int tile_keys, int* status, cudaStream_t stream);
+                        int gate_head, float scale, float softcap, void* out, long long ldo,
+                        void* o_part, void* lse_part, int tile_keys, int* status,
+                        cudaStream_t stream);
 int ab200_attention_merge(const void* o_part, const void* lse_part, const void* tok_splits,
-                          long long T, int Hq, int D, void* out, long long ldo,
-                          cudaStream_t stream);
+                          long long T, int Hq, int D, const void* sink, const void* gate,
+                          long long ldg, void* out, long long ldo, cudaStream_t stream);
 int ab200_attention_scatter(const void* q, long long ldq, const void* k, const void* v,
                             long long num_blocks, int block_size, const void* block_tables,
                             int max_blocks, const void* work, int num_work,
@@ -237,8 +238,18 @@ int ab200_argmax_exchange(const void* ids, const void* vals, int B, int max_rows
                           cudaStream_t stream);
 
 // ---- stream.cu (dtype: 0 = bf16, 1 = fp32 elements; the residual stream is always fp32)
-int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, float scale,
-                           long long T, int W, long long vocab, int dtype, int* status, cudaStream_t stream);
+int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, void* keep, float scale,
+                           long long T, int W, long long vocab, const void* prev, const void* second,
+                           long long buckets, long long mul_prev, long long mul_cur, int dtype,
+                           int* status, cudaStream_t stream);
+int ab200_stream_pre(void* x, const void* y, long long ldy, const void* bias, const void* y_rows,
+                     const void* y_weights, int top, const void* shared, long long ld_shared,
+                     float mult, const void* base, const void* step, const void* w_in, int w_scalar,
+                     void* act, float eps, long long T, int W, int dtype, cudaStream_t stream);
+int ab200_poly_norm(const void* z, const void* bias, const void* coef, void* out, long long T, int n,
+                    int ff, float eps, int dtype, cudaStream_t stream);
+int ab200_soft_cap(const void* z, long long ld, void* out, long long T, int V, float cap, int dtype,
+                   cudaStream_t stream);
 int ab200_stream_norm(const void* x, const void* rows, const void* y, long long ldy,
                       const void* y_rows, const void* y_weights, int top, const void* weight,
                       float alpha, float eps, float offset, void* x_out, void* act_out,
@@ -264,9 +275,10 @@ int ab200_linear_exact(const void* x, long long ldx, long long x_gstride, const 
 int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row, const void* v,
                           int v_row, int num_blocks, int block_size, const void* block_tables,
                           int max_blocks, const void* tok_seq, const void* positions,
-                          const void* sink, const void* gate, long long ldg, void* out,
-                          long long ldo, long long T, int H, int Hkv, int Dk, int Dv, int mask_kind,
-                          int mask_size, float scale, float softcap, int dtype, int* status, cudaStream_t stream);
+                          const void* sink, const void* gate, long long ldg, int gate_head,
+                          void* out, long long ldo, long long T, int H, int Hkv, int Dk, int Dv,
+                          int mask_kind, int mask_size, float scale, float softcap, int dtype,
+                          int* status, cudaStream_t stream);
 
 // ---- rotary.cu
 int ab200_rotary_table(const void* positions, const void* freq, void* table, long long T, int half,
@@ -282,15 +294,16 @@ int ab200_latent_rope_cache(void* q, const void* ckv, long long ld, const void* 
                             float eps, int dtype, int* status, cudaStream_t stream);
 
 // ---- moe.cu
-int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E,
-                    int experts, int top, int all, float scale, void* ids, void* weights, void* state, void* cursor, void* tiles,
-                    void* num_tiles, int dtype, cudaStream_t stream);
+int ab200_moe_route(const void* x, int x_dtype, const void* w, const void* b, long long T, int W, int E,
+                    int experts, int top, int mode, float scale, int groups, int keep, void* ids,
+                    void* weights, void* state, void* cursor, void* tiles, void* num_tiles, int dtype,
+                    cudaStream_t stream);
 int ab200_moe_permute(const void* x, const void* ids, void* cursor, void* rows, void* xp,
                       long long T, int W, int top, int experts, int dtype, cudaStream_t stream);
 
 // ---- recurrent.cu
-int ab200_scan_min_slices(int dim, int ncols, int delta, int dtype, int several);
-long long ab200_scan_record(int dim, int ncols, int slices, int delta, int dtype);
+int ab200_scan_min_slices(int dim, int ncols, int rule, int dtype, int several);
+long long ab200_scan_record(int dim, int ncols, int slices, int rule, int dtype);
 int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_at, int b_at,
                      const void* decay, long long ld_decay, const void* gate, long long ld_gate,
                      const void* conv, int taps, const void* a_exp, const void* dt_bias,
@@ -306,6 +319,12 @@ int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_
                       const void* first_tile, int n_tiles, void* records, void* gates, long long T,
                       int heads, int dim, int vdim, int slices, float eps, void* raw, void* out,
                       long long ldo, int dtype, int* status, cudaStream_t stream);
+int ab200_forget_scan(const void* proj, long long ld, int q_at, int f_at, int v_at, const void* f_bias,
+                      const void* lower, const void* norm, void* state, int state_cols, int num_slots,
+                      const void* steps, int n_seq, int max_rows, const void* tiles,
+                      const void* first_tile, int n_tiles, void* records, long long T, int heads, int dim,
+                      int vdim, int slices, float eps, void* raw, void* out, long long ldo, int dtype,
+                      int* status, cudaStream_t stream);
 
 // ---- grouped_gemm.cu
 int ab200_grouped_gemm(const void* x, long long ldx, long long x_gstride, long long x_rows,
@@ -319,8 +338,9 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
                            int block_size, const void* block_tables, int max_blocks,
                            const void* work, int num_work, const void* tok_splits, int max_splits,
                            long long T, int H, int R, int key_extra, int mask_kind, int mask_size,
-                           int tile_rows, float scale, void* out, void* o_part, void* lse_part,
-                           int* status, cudaStream_t stream);
+                           int tile_rows, float scale, const void* sink, const void* gate,
+                           long long ldg, void* out, void* o_part, void* lse_part, int* status,
+                           cudaStream_t stream);
 
 #ifdef __cplusplus
 }

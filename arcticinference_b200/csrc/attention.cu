@@ -27,7 +27,8 @@
 // Instances with EXT also take a mask with a lower bound (a window, or chunks of positions: the
 // planner starts a tile's keys at the first one its rows see, the softmax masks the rest), a
 // sink per head in the denominator (added once, at the end) and an output gate (the
-// normalised rows times sigmoid of a projection, as they are stored). With split keys the merge
+// normalised rows times sigmoid of a projection, as they are stored; a number per column or one per
+// head). With split keys the merge
 // kernel adds the sink and applies the gate. CAP instances cap the scores softly before the
 // exponential.
 //
@@ -90,11 +91,12 @@ struct AttnArgs {
   int peer_tokens;
   __nv_bfloat16* peer_out[16];
   // EXT instances: mask (first_visible), sink per query head [Hq] and output gate [T][ldg], the
-  // columns laid out like out's
+  // columns laid out like out's or (gate_head) one per query head
   int mask_kind, mask_size;
   const float* sink;
   const __nv_bfloat16* gate;
   long long ldg;
+  int gate_head;
   // completion signal to every rank once the last block has stored its rows (common/peer.cuh);
   // with split-KV the merge kernel sends it instead
   TailSignal sig;
@@ -119,6 +121,14 @@ __device__ __forceinline__ uint4 gate8(const uint4& v, const uint4& g) {
     r[i] = pack_bf16x2(x.x * sigmoid_fast(y.x), x.y * sigmoid_fast(y.y));
   }
   return make_uint4(r[0], r[1], r[2], r[3]);
+}
+
+// Eight columns from d on of a (token, head) row's output gate
+__device__ __forceinline__ uint4 load_gate8(const AttnArgs& p, long long tok, int head, int D, int d) {
+  const __nv_bfloat16* g = p.gate + tok * p.ldg;
+  if (!p.gate_head) return *reinterpret_cast<const uint4*>(g + (long long)head * D + d);
+  const uint32_t x = reinterpret_cast<const unsigned short*>(g)[head], xx = x | (x << 16);
+  return make_uint4(xx, xx, xx, xx);
 }
 
 // cap * log2(e) * tanh(s * scale / cap): a capped score in units of the base-2 exponential. Through
@@ -588,9 +598,7 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         const int rr = quad * 32 + (i * kHalves2 + half) * (32 / kCh) + lane / kCh;
         gates[i] = make_uint4(0, 0, 0, 0);
         if (rr / p.G < n_q_tok && rr % p.G < p.g_heads)
-          gates[i] = *reinterpret_cast<const uint4*>(
-              p.gate + (long long)(q_tok0 + rr / p.G) * p.ldg +
-              (long long)(kvh * p.g_heads + rr % p.G) * D + 8 * (lane % kCh));
+          gates[i] = load_gate8(p, q_tok0 + rr / p.G, kvh * p.g_heads + rr % p.G, D, 8 * (lane % kCh));
       }
     }
     if (ok && n_tiles > 0 && warp_active) {
@@ -672,9 +680,7 @@ attention_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
               if (kPrefill)
                 q = gate8(q, gates[it / kHalves2 % kHeld]);
               else
-                q = gate8(q, *reinterpret_cast<const uint4*>(
-                                 p.gate + (long long)(q_tok0 + rr / p.G) * p.ldg +
-                                 (long long)(kvh * p.g_heads + rr % p.G) * D + 8 * j));
+                q = gate8(q, load_gate8(p, q_tok0 + rr / p.G, kvh * p.g_heads + rr % p.G, D, 8 * j));
             }
             *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(d) + 8 * j) = q;
           }
@@ -778,7 +784,13 @@ __global__ void attention_merge_kernel(const float* __restrict__ o_part,
     }
     const float inv = wsum > 0.f ? 1.f / wsum : 0.f;
     if (EXT && pa.gate != nullptr) {
-      const float4 g = load4(pa.gate + tok * pa.ldg + (long long)head * D + d4);
+      float4 g;
+      if (pa.gate_head) {
+        const float x = __bfloat162float(pa.gate[tok * pa.ldg + head]);
+        g = make_float4(x, x, x, x);
+      } else {
+        g = load4(pa.gate + tok * pa.ldg + (long long)head * D + d4);
+      }
       acc.x *= sigmoid_fast(g.x);
       acc.y *= sigmoid_fast(g.y);
       acc.z *= sigmoid_fast(g.z);
@@ -798,6 +810,7 @@ struct AttnExt {
   const void* sink;
   const void* gate;
   long long ldg;
+  int gate_head;
   float softcap;
 };
 
@@ -885,6 +898,7 @@ static int launch_attention(const void* q, long long ldq, const void* k, const v
     a.sink = reinterpret_cast<const float*>(ext->sink);
     a.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);
     a.ldg = ext->ldg;
+    a.gate_head = ext->gate_head;
     if (CAP) {
       a.cap_in = scale / ext->softcap;
       a.cap_log2 = ext->softcap * 1.4426950408889634f;
@@ -957,7 +971,8 @@ int ab200_attention(const void* q, long long ldq, const void* k, const void* v, 
 
 // The same with a mask (0 causal, 1 window, 2 chunk, see first_visible), softly capped scores
 // (softcap * tanh(score / softcap), 0: not), an optional sink per query
-// head (fp32 [Hq]) and an optional output gate (bf16 rows of stride ldg, columns like out's).
+// head (fp32 [Hq]) and an optional output gate (bf16 rows of stride ldg, columns like out's or, with
+// gate_head, one per query head).
 // Always causal; the work list's kv_start must not lie above the first key a tile's rows see.
 // Queries and keys have Dk columns per head, values and outputs D; they may differ (192, 128) with
 // contiguous keys and values.
@@ -966,15 +981,17 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
                         int max_blocks, const void* work, int num_work, const void* tok_splits,
                         int max_splits, long long T, int Hq, int Hkv, int Dk, int D, int mask_kind,
                         int mask_size, const void* sink, const void* gate, long long ldg,
-                        float scale, float softcap, void* out, long long ldo, void* o_part,
-                        void* lse_part, int tile_keys, int* status, cudaStream_t stream) {
+                        int gate_head, float scale, float softcap, void* out, long long ldo,
+                        void* o_part, void* lse_part, int tile_keys, int* status,
+                        cudaStream_t stream) {
   if (num_work <= 0 || T <= 0) return 0;
   if ((ldq % 8) || (ldo % 8) || (ld_kv % 8) || softcap < 0.f) return -2;
   if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
     return -2;
-  if (gate != nullptr && ((ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -2;
+  if (gate != nullptr && !gate_head && ((ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15)))
+    return -2;
   if (max_splits > 1 && (o_part == nullptr || lse_part == nullptr || tok_splits == nullptr)) return -2;
-  const AttnExt ext = {mask_kind, mask_size, sink, gate, ldg, softcap};
+  const AttnExt ext = {mask_kind, mask_size, sink, gate, ldg, gate_head, softcap};
   if (softcap > 0.f && Dk != D) return -2;
   if (Dk == 192 && D == 128)
     return launch_attention<192, 128, 64, true>(
@@ -1000,16 +1017,22 @@ int ab200_attention_ext(const void* q, long long ldq, const void* k, const void*
 }
 
 // Folds split-KV partials of another attention kernel (same layouts as above): o_part fp32
-// [splits, T, Hq, D], D a multiple of 128 up to 512, out bf16.
+// [splits, T, Hq, D], D a multiple of 128 up to 512, out bf16; sink fp32 [Hq] and gate bf16 [T, ldg], one
+// per head, may be null.
 int ab200_attention_merge(const void* o_part, const void* lse_part, const void* tok_splits,
-                          long long T, int Hq, int D, void* out, long long ldo,
-                          cudaStream_t stream) {
+                          long long T, int Hq, int D, const void* sink, const void* gate,
+                          long long ldg, void* out, long long ldo, cudaStream_t stream) {
   AttnArgs a;
   memset(&a, 0, sizeof(a));
-  auto k = D == 128   ? attention_merge_kernel<128, false>
-           : D == 256 ? attention_merge_kernel<256, false>
-           : D == 384 ? attention_merge_kernel<384, false>
-                      : attention_merge_kernel<512, false>;
+  a.sink = reinterpret_cast<const float*>(sink);
+  a.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  a.ldg = ldg;
+  a.gate_head = 1;
+  const bool ext = sink != nullptr || gate != nullptr;
+  auto k = D == 128   ? (ext ? attention_merge_kernel<128, true> : attention_merge_kernel<128, false>)
+           : D == 256 ? (ext ? attention_merge_kernel<256, true> : attention_merge_kernel<256, false>)
+           : D == 384 ? (ext ? attention_merge_kernel<384, true> : attention_merge_kernel<384, false>)
+                      : (ext ? attention_merge_kernel<512, true> : attention_merge_kernel<512, false>);
   if (D != 128 && D != 256 && D != 384 && D != 512) return -2;
   return launch_pdl(k, dim3((unsigned)T), dim3(D >= 256 ? 256 : 128), 0, stream,
                     reinterpret_cast<const float*>(o_part), reinterpret_cast<const float*>(lse_part),

@@ -7,8 +7,11 @@
 
 namespace ab200 {
 
+// The recurrences (recurrent.cu)
+enum Rule : int { kMemory = 0, kDelta = 1, kForget = 2 };
+
 // warps of a block: 128 columns of wide states, and the normaliser's beside them
-__host__ __device__ constexpr int max_warps(bool delta) { return delta ? 8 : 9; }
+__host__ __device__ constexpr int max_warps(int rule) { return rule == kMemory ? 9 : 8; }
 
 constexpr int kTT = 16, kB = 4;           // tokens per tile and per group
 constexpr int kTaps = 4;                  // convolutions of up to this many taps stay in registers
@@ -22,13 +25,14 @@ struct ScanArgs {
   int q_at, k_at, v_at;      // columns of head 0's query, key and value
   int b_at;                  // delta: step sizes [heads]
   int i_at, f_at;            // memory: gates [heads]
-  const void* decay;         // delta: [T][ld_decay], head h's channels at column h * dim
-  long long ld_decay;
-  const void* gate;          // output gate [T][ld_gate], head h at column h * vdim
+  const void* decay;         // delta: [T][ld_decay], head h's channels at column h * dim; forget: the
+  long long ld_decay;        // gates' projection, likewise
+  const void* gate;          // output gate [T][ld_gate], head h at column h * vdim (forget: none)
   long long ld_gate;
   const float* conv;         // delta: [taps][channels]: queries', keys', values' weights
   const float* a_exp;        // delta: [heads] exp(A_log)
-  const float* dt_bias;      // delta: [heads][dim]
+  const float* dt_bias;      // delta, forget: [heads][dim]
+  const float* lower;        // forget: [heads][dim], lower bound of the gates
   const float* i_bias;       // memory: [heads]
   const float* f_bias;
   const float* norm;         // head h's weights at h * norm_step
@@ -125,6 +129,16 @@ struct Raw8<__nv_bfloat16> {   // (8-byte aligned)
   __device__ __forceinline__ float4 lo() const { return widen(a.x, a.y); }
   __device__ __forceinline__ float4 hi() const { return widen(b.x, b.y); }
 };
+// Forget gate f = lower + (1 - lower) sigmoid(z): 1 - f, which keeps its digits where f is near 1
+__device__ __forceinline__ float forget_put(float z, float lower) { return (1.f - lower) * sigmoid_f(-z); }
+__device__ __forceinline__ float forget_keep(float z, float lower) {
+  return fmaf(1.f - lower, sigmoid_f(z), lower);
+}
+// log2 of f; log(1 - x)'s first terms in x = 1 - f where the fast logarithm would lose them
+__device__ __forceinline__ float forget_log2(float keep, float put) {
+  const float series = -put * fmaf(put, fmaf(put, fmaf(put, 0.25f, 0.33333333f), 0.5f), 1.f);
+  return put < 0.03f ? series * kLog2e : log2_fast(keep);
+}
 // log gates of the matrix memory
 __device__ __forceinline__ float2 memory_log_gates(float zi, float zf, float cap) {
   const float z = cap * tanhf(zf / cap);
@@ -198,7 +212,7 @@ __device__ __forceinline__ void save_inputs(const ScanArgs& p, const Seq& s, con
 }
 
 // Outputs of padding rows: finite, no state involved
-template <typename T, bool DELTA>
+template <typename T, int RULE>
 __device__ __forceinline__ void put_zeros(const ScanArgs& p, const Seq& s, int h, int slice) {
   if (s.slot >= p.num_slots && threadIdx.x == 0) report_error(p.status, kErrBounds, 50, s.slot);
   for (int t = 0; t < s.n; ++t) {
@@ -206,7 +220,7 @@ __device__ __forceinline__ void put_zeros(const ScanArgs& p, const Seq& s, int h
       float* dst = p.raw + ((s.first + t) * p.heads + h) * p.raw_cols;
       const int c1 = min((slice + 1) * p.nc, p.ncols);
       for (int c = slice * p.nc + threadIdx.x; c < c1; c += blockDim.x) dst[c] = 0.f;
-      if (!DELTA && slice == 0 && threadIdx.x == 0) dst[p.ncols] = 1.f;
+      if (RULE == kMemory && slice == 0 && threadIdx.x == 0) dst[p.ncols] = 1.f;
     } else {
       T* dst = reinterpret_cast<T*>(p.out) + (s.first + t) * p.ldo + (long long)h * p.vdim;
       for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) dst[c] = from_f32<T>(0.f);
@@ -214,16 +228,16 @@ __device__ __forceinline__ void put_zeros(const ScanArgs& p, const Seq& s, int h
   }
 }
 
-// A warp's token: norm, weight and gate of a head's outputs o (memory: with the normaliser's product
-// in column vdim and `floor` = exp(-m)).
-template <typename T, bool DELTA>
+// A warp's token: norm, weight and gate (none: forget) of a head's outputs o (memory: with the
+// normaliser's product in column vdim and `floor` = exp(-m)).
+template <typename T, int RULE>
 __device__ __forceinline__ void head_output(const ScanArgs& p, const float* o, long long row, int h,
                                             float floor) {
   const int lane = threadIdx.x & 31;
   const T* g = reinterpret_cast<const T*>(p.gate) + row * p.ld_gate + (long long)h * p.vdim;
   const float* w = p.norm + (long long)h * p.norm_step;
   T* dst = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
-  float scale = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floor) + 1e-6f);
+  float scale = RULE != kMemory ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floor) + 1e-6f);
   float ss = 0.f;
   for (int c = lane; c < p.vdim; c += 32) {
     const float x = o[c] * scale;
@@ -231,12 +245,12 @@ __device__ __forceinline__ void head_output(const ScanArgs& p, const float* o, l
   }
   scale *= 1.f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
   for (int c = lane; c < p.vdim; c += 32)
-    dst[c] = from_f32<T>(o[c] * scale * w[c] * sigmoid_f(to_f32<T>(g[c])));
+    dst[c] = from_f32<T>(o[c] * scale * w[c] * (RULE == kForget ? 1.f : sigmoid_f(to_f32<T>(g[c]))));
 }
 
 // A block's tile: eight columns a thread, the `lanes` lanes of a token side by side. g, wa, wb: gate
 // and norm weights of the thread's first columns.
-template <typename T, bool DELTA>
+template <typename T, int RULE>
 __device__ __forceinline__ void vector_outputs(const ScanArgs& p, const float* o_tile, int ld, const float* floors,
                                                int nt, int lanes, const T* gate, T* out, const float* w,
                                                Raw8<T> g, float4 wa, float4 wb) {
@@ -246,18 +260,23 @@ __device__ __forceinline__ void vector_outputs(const ScanArgs& p, const float* o
     const bool ok = t < nt;
     const float* o = o_tile + (ok ? t : 0) * ld;
     if (x != threadIdx.x && ok) {
-      g.load(gate + t * p.ld_gate + c);
+      if (RULE != kForget) g.load(gate + t * p.ld_gate + c);
       wa = load4(w + c);
       wb = load4(w + c + 4);
     }
     const float4 a = load4(o + c), b = load4(o + c + 4);
-    float f = DELTA ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floors[ok ? t : 0]) + 1e-6f);
+    float f = RULE != kMemory ? 1.f : 1.f / (fmaxf(fabsf(o[p.vdim]), floors[ok ? t : 0]) + 1e-6f);
     float ss = dot4(a, a, dot4(b, b, 0.f)) * f * f;
     for (int k = lanes / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
     f *= 1.f / sqrtf(ss / (float)p.vdim + p.eps);
     if (!ok) continue;
-    const float4 g0 = g.lo(), g1 = g.hi();
     T* dst = out + t * p.ldo + c;
+    if (RULE == kForget) {
+      store4(dst, make_float4(a.x * f * wa.x, a.y * f * wa.y, a.z * f * wa.z, a.w * f * wa.w));
+      store4(dst + 4, make_float4(b.x * f * wb.x, b.y * f * wb.y, b.z * f * wb.z, b.w * f * wb.w));
+      continue;
+    }
+    const float4 g0 = g.lo(), g1 = g.hi();
     store4(dst, make_float4(a.x * f * wa.x * sigmoid_f(g0.x), a.y * f * wa.y * sigmoid_f(g0.y),
                             a.z * f * wa.z * sigmoid_f(g0.z), a.w * f * wa.w * sigmoid_f(g0.w)));
     store4(dst + 4, make_float4(b.x * f * wb.x * sigmoid_f(g1.x), b.y * f * wb.y * sigmoid_f(g1.y),
@@ -285,6 +304,6 @@ inline bool set_smem(K k, size_t bytes) {
 }
 
 // Portions of several tokens of 16-bit models (recurrent_mma.cu).
-int launch_tiles_mma(const ScanArgs& a, bool delta, int n_seq, int n_tiles, cudaStream_t stream);
+int launch_tiles_mma(const ScanArgs& a, int rule, int n_seq, int n_tiles, cudaStream_t stream);
 
 }  // namespace ab200

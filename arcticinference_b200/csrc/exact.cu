@@ -108,8 +108,9 @@ struct ExactAttnArgs {
   const int* tok_seq;       // [T] sequence (row of block_tables) of each token
   const long long* positions;
   const float* sink;        // [H] or null
-  const void* gate;         // [T][ldg], head h at column h * Dv, or null
+  const void* gate;         // [T][ldg], head h at column h * Dv (gate_head: at column h, one), or null
   long long ldg;
+  int gate_head;
   void* out;                // [T][ldo], head h at column h * Dv
   long long ldo;
   int H, Hkv, Dk, Dv, num_blocks;
@@ -178,11 +179,12 @@ __global__ void __launch_bounds__(kAttnKeys) attention_exact_kernel(const ExactA
   }
   if (p.sink != nullptr && m != -INFINITY) l += expf(p.sink[h] - m);
   T* o = reinterpret_cast<T*>(p.out) + t * p.ldo + (long long)h * p.Dv;
-  const T* gate = p.gate ? reinterpret_cast<const T*>(p.gate) + t * p.ldg + (long long)h * p.Dv : nullptr;
+  const T* gate = p.gate ? reinterpret_cast<const T*>(p.gate) + t * p.ldg +
+                               (long long)h * (p.gate_head ? 1 : p.Dv) : nullptr;
   const float inv = l > 0.f ? 1.f / l : 0.f;
   for (int i = tid; i < p.Dv; i += kAttnKeys) {   // own columns
     float v = acc[i] * inv;
-    if (gate != nullptr) v /= 1.f + expf(-to_f32<T>(gate[i]));
+    if (gate != nullptr) v /= 1.f + expf(-to_f32<T>(gate[p.gate_head ? 0 : i]));
     o[i] = from_f32<T>(v);
   }
 }
@@ -219,14 +221,15 @@ int ab200_linear_exact(const void* x, long long ldx, long long x_gstride, const 
 }
 
 // k: [num_blocks, Hkv, block_size, k_row] of which the first Dk columns count, v likewise (it may
-// be the same tensor); sink fp32 [H] and gate [T, ldg] may be null.
+// be the same tensor); sink fp32 [H] and gate [T, ldg] (a number per column, or with gate_head one per
+// head) may be null.
 int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row, const void* v,
                           int v_row, int num_blocks, int block_size, const void* block_tables,
                           int max_blocks, const void* tok_seq, const void* positions,
-                          const void* sink, const void* gate, long long ldg, void* out,
-                          long long ldo, long long T, int H, int Hkv, int Dk, int Dv, int mask_kind,
-                          int mask_size, float scale, float softcap, int dtype, int* status,
-                          cudaStream_t stream) {
+                          const void* sink, const void* gate, long long ldg, int gate_head,
+                          void* out, long long ldo, long long T, int H, int Hkv, int Dk, int Dv,
+                          int mask_kind, int mask_size, float scale, float softcap, int dtype,
+                          int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H < 1 || Hkv < 1 || H % Hkv || Dk > k_row || Dv > v_row || block_size < 1) return -2;
   if (mask_kind < kMaskCausal || mask_kind > kMaskChunk || (mask_kind != kMaskCausal && mask_size < 1))
@@ -242,7 +245,7 @@ int ab200_attention_exact(const void* q, long long ldq, const void* k, int k_row
   a.tok_seq = reinterpret_cast<const int*>(tok_seq);
   a.positions = reinterpret_cast<const long long*>(positions);
   a.sink = reinterpret_cast<const float*>(sink);
-  a.gate = gate; a.ldg = ldg;
+  a.gate = gate; a.ldg = ldg; a.gate_head = gate_head;
   a.out = out; a.ldo = ldo;
   a.H = H; a.Hkv = Hkv; a.Dk = Dk; a.Dv = Dv;
   a.num_blocks = num_blocks;

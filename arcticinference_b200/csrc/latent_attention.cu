@@ -23,8 +23,11 @@
 // the warp's lanes (16 columns in 16 shuffles) and four words of shared memory; sums stay
 // per-thread until the end. O is rescaled only in tiles where a maximum moved.
 //
+// A sink per head is one more term of a row's sum, added at the end; an output gate per head scales
+// the row as it is written.
+//
 // With several pieces of the keys per sequence a CTA writes normalised fp32 partials and their
-// log-sum-exp, folded by the merge kernel of attention.cu.
+// log-sum-exp, folded by the merge kernel of attention.cu (which then adds the sink and applies the gate).
 
 #include <math.h>
 #include <string.h>
@@ -52,6 +55,9 @@ struct LatentArgs {
   int x_bufs;              // buffers of the key-only piece (0: none)
   int mask_kind, mask_size;
   float scale, scale_log2;
+  const float* sink;           // [H] or null
+  const __nv_bfloat16* gate;   // [T][ldg], one per head, or null
+  long long ldg;
   uint32_t tmem_cols;
   __nv_bfloat16* out;      // [T * H][R]
   float* o_part;           // [pieces of keys][T * H][R]
@@ -502,11 +508,18 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
     bar_softmax();
     if (tid < NR) {
       const float4 q = *reinterpret_cast<const float4*>(&wred[tid * 4]);
-      const float sum = (q.x + q.y) + (q.z + q.w);
-      inv_s[tid] = sum > 0.f ? 1.f / sum : 0.f;
+      float sum = (q.x + q.y) + (q.z + q.w);
       if (n_pieces > 1 && tid < n_rows)
         p.lse_part[(long long)piece * p.rows_total + row0 + tid] =
             sum > 0.f ? m_s[tid] * p.scale + logf(sum) : -INFINITY;
+      const bool last = n_pieces <= 1 && tid < n_rows && sum > 0.f;   // (else the merge does it)
+      const int tok = (row0 + tid) / p.H, head = row0 + tid - tok * p.H;
+      if (last && p.sink != nullptr)
+        sum += ex2_approx(fmaf(p.sink[head], 1.4426950408889634f, neg_s[tid]));
+      float inv = sum > 0.f ? 1.f / sum : 0.f;
+      if (last && p.gate != nullptr)
+        inv *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[tok * p.ldg + head])));
+      inv_s[tid] = inv;
     }
     bar_softmax();
     if (n_tiles > 0) {
@@ -608,13 +621,15 @@ extern "C" {
 
 // q bf16 [T * H, R + key_extra], out [T * H, R], both contiguous; cache [num_blocks, block_size,
 // R + key_extra]; R a multiple of 128 up to 512, key_extra 0 or 64 (columns of the key only);
-// tile_rows 16, 32, 48 or 64, the rows per work item (at most 48 with R = 512 and key_extra).
+// tile_rows 16, 32, 48 or 64, the rows per work item (at most 48 with R = 512 and key_extra). sink
+// fp32 [H] and gate bf16 [T, ldg] (column h: head h's, of which the sigmoid is taken) may be null.
 int ab200_latent_attention(const void* q, long long q_rows, const void* cache, int num_blocks,
                            int block_size, const void* block_tables, int max_blocks,
                            const void* work, int num_work, const void* tok_splits, int max_splits,
                            long long T, int H, int R, int key_extra, int mask_kind, int mask_size,
-                           int tile_rows, float scale, void* out, void* o_part, void* lse_part,
-                           int* status, cudaStream_t stream) {
+                           int tile_rows, float scale, const void* sink, const void* gate,
+                           long long ldg, void* out, void* o_part, void* lse_part, int* status,
+                           cudaStream_t stream) {
   if (num_work <= 0 || T <= 0) return 0;
   if (R % 128 || R < 128 || R > 512 || H <= 0 || q_rows != T * H) return -2;
   if (key_extra != 0 && key_extra != 64) return -2;
@@ -642,6 +657,9 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
   a.x_bufs = key_extra / 64;
   a.mask_kind = mask_kind;
   a.mask_size = mask_size;
+  a.sink = reinterpret_cast<const float*>(sink);
+  a.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  a.ldg = ldg;
   a.scale = scale;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
@@ -658,7 +676,8 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
     default: return -2;
   }
   if (rc != 0 || max_splits <= 1) return rc;
-  return ab200_attention_merge(o_part, lse_part, tok_splits, T, H, R, out, (long long)H * R, stream);
+  return ab200_attention_merge(o_part, lse_part, tok_splits, T, H, R, sink, gate, ldg, out,
+                               (long long)H * R, stream);
 }
 
 }  // extern "C"

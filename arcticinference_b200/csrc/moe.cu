@@ -8,12 +8,16 @@
 //                the rows sorted by expert and into the list of 128-row tiles the grouped matrix
 //                products walk. Or, scoring over all outputs: the softmax over all of them, the
 //                choice by score plus a correction, the chosen scores times a scale as weights;
-//                outputs beyond the experts are identity experts, which get no rows
+//                outputs beyond the experts are identity experts, which get no rows. Or sigmoid
+//                scores: the choice among the experts of the best groups of neighbours (by the sum
+//                of a group's two best), the chosen scores normalised to the sum `scale`
 //   moe_permute  row of every (token, choice) and the copy of the token's activations there
 //
 // The weighted sum of the experts' outputs is taken by the norm kernel that follows (stream.cu).
 
 #include <float.h>
+
+#include <type_traits>
 
 #include "api.h"
 #include "common/elem.cuh"
@@ -43,15 +47,19 @@ struct Raw4<__nv_bfloat16> {
   }
 };
 
+enum RouteMode : int { kRouteChosen = 0, kRouteAll = 1, kRouteSigmoid = 2 };
+
 struct RouteArgs {
-  const float* x;
+  const void* x;       // [n][W]: fp32, or (x_act) in the router weights' element type
+  int x_act;
   const void* w;       // [E][W]
   const float* b;      // [E] bias of the logits, or correction of the choice; may be null
   long long n;
   int W, E, top;       // E: router outputs
   int experts;         // of them the experts' (the others: identity)
-  int all;             // softmax over all outputs instead of the chosen ones
-  float scale;         // of the weights (all)
+  int mode;            // RouteMode: softmax over the chosen logits or over all, or sigmoids
+  float scale;         // of the weights (all), their sum (sigmoids)
+  int groups, keep;    // sigmoids: equal groups of experts, how many of them can be chosen from
   int* ids;            // [n][top]
   float* weights;      // [n][top]
   int* state;          // [E] counts and [1] finished blocks; zero before and after every launch
@@ -104,6 +112,28 @@ __device__ void moe_plan(const RouteArgs& p, int* sh) {
   }
 }
 
+// The largest of n values (ties, NaNs: the lower index), by a warp; `best` its value
+__device__ __forceinline__ int warp_argmax(const float* v, int n, float& best) {
+  const int lane = threadIdx.x & 31;
+  best = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int e = lane; e < n; e += 32)
+    if (v[e] > best || bi == 0x7fffffff) {
+      best = v[e];
+      bi = e;
+    }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ov > best || (ov == best && oi < bi)) {
+      best = ov;
+      bi = oi;
+    }
+  }
+  return min(bi, n - 1);   // (a row of NaNs must still name one)
+}
+
 // Router weights of type T; TB tokens per block. Shared memory: x rows [TB][W], logits [TB][E],
 // at least 3 * E words for the plan.
 template <typename T, int TB, int kRouteThreads>
@@ -119,13 +149,18 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
   const long long t0 = (long long)blockIdx.x * TB;
   const int nt = (int)min((long long)TB, p.n - t0);
   const bool vec = W % 4 == 0;
-  if (vec) {
-    for (int i = threadIdx.x * 4; i < TB * W; i += kRouteThreads * 4)
-      store4(xs + i, i / W < nt ? load4(p.x + t0 * W + i) : make_float4(0.f, 0.f, 0.f, 0.f));
-  } else {
-    for (int i = threadIdx.x; i < TB * W; i += kRouteThreads)
-      xs[i] = i / W < nt ? p.x[t0 * W + i] : 0.f;
-  }
+  auto fill = [&](const auto* x) {
+    typedef typename std::remove_const<typename std::remove_pointer<decltype(x)>::type>::type X;
+    if (vec) {
+      for (int i = threadIdx.x * 4; i < TB * W; i += kRouteThreads * 4)
+        store4(xs + i, i / W < nt ? load4(x + t0 * W + i) : make_float4(0.f, 0.f, 0.f, 0.f));
+    } else {
+      for (int i = threadIdx.x; i < TB * W; i += kRouteThreads)
+        xs[i] = i / W < nt ? to_f32<X>(x[t0 * W + i]) : 0.f;
+    }
+  };
+  if (p.x_act) fill(reinterpret_cast<const T*>(p.x));
+  else fill(reinterpret_cast<const float*>(p.x));
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr int EB = 4;   // experts a warp takes at a time
@@ -190,7 +225,7 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
       for (int j = 0; j < EB; ++j) {
         const float s = warp_sum(acc[t][j]);
         if (lane == 0 && e0 + j < E)
-          z[t * E + e0 + j] = p.b != nullptr && !p.all ? s + p.b[e0 + j] : s;
+          z[t * E + e0 + j] = p.b != nullptr && p.mode == kRouteChosen ? s + p.b[e0 + j] : s;
       }
   }
   __syncthreads();
@@ -198,7 +233,34 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
   for (int t = warp; t < nt; t += kRouteThreads / 32) {
     float* zt = z + t * E;
     float first = 0.f, sum = 0.f;
-    if (p.all) {   // logits -> scores plus correction
+    if (p.mode == kRouteSigmoid) {
+      for (int e = lane; e < E; e += 32) zt[e] = 1.f / (1.f + expf(-zt[e]));
+      __syncwarp();
+      if (p.keep < p.groups) {
+        float* gs = zt + E * TB;   // scores of the groups, -inf once kept
+        const int size = E / p.groups;
+        for (int g = lane; g < p.groups; g += 32) {
+          float a = -INFINITY, b = -INFINITY;   // the two best
+          for (int e = g * size; e < (g + 1) * size; ++e) {
+            b = fmaxf(b, fminf(a, zt[e]));
+            a = fmaxf(a, zt[e]);
+          }
+          gs[g] = size > 1 ? a + b : a;
+        }
+        __syncwarp();
+        for (int k = 0; k < p.keep; ++k) {
+          float best;
+          const int g = warp_argmax(gs, p.groups, best);
+          __syncwarp();
+          if (lane == 0) gs[g] = -INFINITY;
+          __syncwarp();
+        }
+        for (int e = lane; e < E; e += 32)
+          if (gs[e / size] != -INFINITY) zt[e] = -INFINITY;
+        __syncwarp();
+      }
+    }
+    if (p.mode == kRouteAll) {   // logits -> scores plus correction
       float mx = -INFINITY;
       for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zt[e]);
       mx = warp_max(mx);
@@ -217,28 +279,14 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
     int* my_ids = p.ids + (t0 + t) * top;
     float* my_w = p.weights + (t0 + t) * top;
     for (int j = 0; j < top; ++j) {
-      float best = -INFINITY;
-      int bi = 0x7fffffff;
-      for (int e = lane; e < E; e += 32) {
-        const float v = zt[e];
-        if (v > best || bi == 0x7fffffff) {
-          best = v;
-          bi = e;
-        }
-      }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-        if (ov > best || (ov == best && oi < bi)) {
-          best = ov;
-          bi = oi;
-        }
-      }
-      bi = min(bi, E - 1);   // (a row of NaNs must still name an expert)
+      float best;
+      const int bi = warp_argmax(zt, E, best);
       if (j == 0) first = best;
-      const float ex = p.all ? zt[E * TB + bi] * p.scale : expf(best - first);
+      const float ex = p.mode == kRouteAll       ? zt[E * TB + bi] * p.scale
+                       : p.mode == kRouteSigmoid ? best
+                                                 : expf(best - first);
       sum += ex;
+      __syncwarp();
       if (lane == 0) {
         my_ids[j] = bi;
         my_w[j] = ex;
@@ -247,8 +295,8 @@ __global__ void __launch_bounds__(kRouteThreads) moe_route_kernel(const RouteArg
       }
       __syncwarp();
     }
-    if (p.all) continue;
-    const float inv = 1.f / sum;
+    if (p.mode == kRouteAll) continue;
+    const float inv = p.mode == kRouteSigmoid ? p.scale / (sum + 1e-20f) : 1.f / sum;
     for (int j = lane; j < top; j += 32) my_w[j] *= inv;
   }
   // every block counts itself done after its counts are visible; the last one plans
@@ -299,7 +347,7 @@ moe_permute_kernel(const T* __restrict__ x, const int* __restrict__ ids, int* __
 
 template <typename T, int TB>
 static int launch_route(const RouteArgs& a, cudaStream_t stream) {
-  size_t smem = ((size_t)TB * a.W + (size_t)TB * a.E * (a.all ? 2 : 1)) * sizeof(float);
+  size_t smem = ((size_t)TB * a.W + (size_t)TB * a.E * (a.mode == kRouteChosen ? 1 : 2)) * sizeof(float);
   if (smem < (size_t)3 * a.E * sizeof(int)) smem = (size_t)3 * a.E * sizeof(int);
   if (smem > 220 * 1024) return -6;
   // few tokens: more warps per block, so that each has few experts to go through
@@ -321,17 +369,24 @@ typedef __nv_bfloat16 bf16;
 
 extern "C" {
 
-// x fp32 [T, W]; w [E, W] (dtype 0 = bf16, 1 = fp32); b fp32 [E] or null; the first `experts` of the
-// E outputs are experts, the others the identity; all, scale: see RouteArgs. ids int32 and weights fp32
+// x [T, W] (x_dtype 0 = bf16, 1 = fp32: fp32, or what w has); w [E, W] (dtype likewise); b fp32 [E] or
+// null; the first `experts` of the E outputs are experts, the others the identity; mode, scale, groups,
+// keep: see RouteArgs. ids int32 and weights fp32
 // [T, top]; state int32 [experts + 1], zero; cursor int32 [experts]; tiles int32 x 4 [T * top / 128 +
 // experts at most]; num_tiles int32 [1]
-int ab200_moe_route(const void* x, const void* w, const void* b, long long T, int W, int E,
-                    int experts, int top, int all, float scale, void* ids, void* weights, void* state, void* cursor, void* tiles,
-                    void* num_tiles, int dtype, cudaStream_t stream) {
+int ab200_moe_route(const void* x, int x_dtype, const void* w, const void* b, long long T, int W, int E,
+                    int experts, int top, int mode, float scale, int groups, int keep, void* ids,
+                    void* weights, void* state, void* cursor, void* tiles, void* num_tiles, int dtype,
+                    cudaStream_t stream) {
   if (T <= 0) return 0;
   if (top < 1 || top > E || experts < 1 || experts > E) return -2;
+  if (mode < kRouteChosen || mode > kRouteSigmoid || (x_dtype != 1 && x_dtype != dtype)) return -2;
+  if (mode == kRouteSigmoid && (groups < 1 || E % groups || keep < 1 || keep > groups ||
+                                top > keep * (E / groups) || experts != E || b != nullptr))
+    return -2;
   RouteArgs a;
-  a.x = reinterpret_cast<const float*>(x);
+  a.x = x;
+  a.x_act = x_dtype != 1;
   a.w = w;
   a.b = reinterpret_cast<const float*>(b);
   a.n = T;
@@ -339,8 +394,10 @@ int ab200_moe_route(const void* x, const void* w, const void* b, long long T, in
   a.E = E;
   a.top = top;
   a.experts = experts;
-  a.all = all;
+  a.mode = mode;
   a.scale = scale;
+  a.groups = groups;
+  a.keep = keep;
   a.ids = reinterpret_cast<int*>(ids);
   a.weights = reinterpret_cast<float*>(weights);
   a.state = reinterpret_cast<int*>(state);

@@ -8,8 +8,11 @@
 //                       o = S^T q / (max(|z . q|, exp(-m')) + 1e-6)
 //                   z is kept as one more column of S, whose value is always 1.
 //
-// Both are followed by the RMS norm of each head's o, a weight and an output gate. Everything that
-// enters the recurrence is fp32, and so is its arithmetic (FMAs on pairs of rows).
+//   forget scan     (HGRN2) a forget gate f per channel, which also decides what is written:
+//                       S <- f * S + (1 - f) v^T;  o = S^T q,  q through silu
+//
+// They are followed by the RMS norm of each head's o, a weight and (but for the forget scan) an output
+// gate. Everything that enters the recurrence is fp32, and so is its arithmetic (FMAs on pairs of rows).
 //
 // Steps of one token per sequence run in one kernel (step_kernel): a block owns a sequence's head, or
 // some of the head's columns, which do not depend on one another.
@@ -24,7 +27,8 @@
 // and a group of tokens needs no exchange but its scalar products: with a = G k, b = k / G, c = G q
 //     u_i = beta_i (v_i - Z^T a_i - sum_{j<i} (a_i . b_j) u_j),  o_i = Z^T c_i + sum_{j<=i} (c_i . b_j) u_j
 // where Z is the one before the group. G goes back to 1 at a tile's end, and after every group when a
-// channel decays so much within the tile that 1 / G would leave fp32's range.
+// channel decays so much within the tile that 1 / G would leave fp32's range. (Without the delta rule u is
+// the value; the forget scan's k is 1 - f, its decays f.)
 //
 // For 16-bit models the products of a tile run on the tensor cores (recurrent_mma.cu); 32-bit models use
 // fp32 multiply-adds.
@@ -166,14 +170,15 @@ __device__ __forceinline__ int reduce_columns(const float2 (&acc)[KINDS][COLS][N
 template <int DP>
 struct StepShape {
   static constexpr int kGroups = DP <= 128 ? 8 : 16, kRows = DP / kGroups;
-  static constexpr int max_threads(bool delta) { return kGroups * max_warps(delta) * 4; }
+  static constexpr int max_threads(int rule) { return kGroups * max_warps(rule) * 4; }
   static constexpr int smem_floats(int nc) { return 3 * DP + nc + 2 * kGroups * nc; }
 };
 
-template <typename T, int DP, bool DELTA>
-__global__ void __launch_bounds__(StepShape<DP>::max_threads(DELTA), DP <= 128 ? 2 : 1)
+template <typename T, int DP, int RULE>
+__global__ void __launch_bounds__(StepShape<DP>::max_threads(RULE), DP <= 128 ? 2 : 1)
 step_kernel(const ScanArgs p) {
   using Sh = StepShape<DP>;
+  constexpr bool DELTA = RULE == kDelta, MEMORY = RULE == kMemory, FORGET = RULE == kForget;
   constexpr int kRows = Sh::kRows;
   extern __shared__ __align__(16) float sm[];
   float* sQ = sm;              // query, key (before their norms), decay, values / outputs
@@ -188,7 +193,7 @@ step_kernel(const ScanArgs p) {
   const Seq s(p.steps + (long long)(blockIdx.x / p.slices / p.heads) * kStepInts);
   if (s.n <= 0) return;
   if (s.slot <= 0 || s.slot >= p.num_slots) {
-    put_zeros<T, DELTA>(p, s, h, slice);
+    put_zeros<T, RULE>(p, s, h, slice);
     return;
   }
   const int tid = threadIdx.x, threads = blockDim.x, lane = tid & 31;
@@ -210,7 +215,7 @@ step_kernel(const ScanArgs p) {
   if (DELTA) {
     a_exp = p.a_exp[h];
     beta = sigmoid_f(to_f32<T>(in.proj[p.b_at + h]));
-  } else {
+  } else if (MEMORY) {
     const float2 g = memory_log_gates(to_f32<T>(in.proj[p.i_at + h]) + p.i_bias[h],
                                       to_f32<T>(in.proj[p.f_at + h]) + p.f_bias[h], p.cap);
     const float m = s.start > 0 ? p.max_state[((long long)s.slot * 2 + s.phase) * p.heads + h] : 0.f;
@@ -224,11 +229,11 @@ step_kernel(const ScanArgs p) {
   T gate0 = from_f32<T>(0.f);
   float norm0 = 0.f;
   if (p.raw == nullptr && tid < p.vdim) {
-    gate0 = gate[tid];
+    if (!FORGET) gate0 = gate[tid];
     norm0 = norm[tid];
   }
   // a channel a thread and turn, two turns' loads at once
-  const bool qk_block = slice == 0 && h % p.group == 0;   // saves the queries' and keys' inputs
+  const bool qk_block = DELTA && slice == 0 && h % p.group == 0;   // saves the queries' and keys' inputs
   T* next = reinterpret_cast<T*>(p.conv_state) + ((long long)s.slot * 2 + (s.phase ^ 1)) * in.back * p.channels;
   struct Channel {   // the inputs as they lie in memory: earlier ones, the token's own
     T old[kTaps - 1], x, z;
@@ -236,10 +241,11 @@ step_kernel(const ScanArgs p) {
   };
   const T* decay = reinterpret_cast<const T*>(p.decay) + s.first * p.ld_decay + h * p.dim;
   const long long last_tap = (long long)in.back * p.channels;
-  const int channels = 2 * DP + p.nc;
+  constexpr int kKeyed = FORGET ? DP : 2 * DP;   // (the forget scan's keys come with the queries)
+  const int channels = kKeyed + p.nc;
   auto place = [&](int x, int& part, int& d) {
-    part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
-    d = x - part * DP + (part == 2 ? c_first : 0);
+    part = x < DP ? 0 : x < kKeyed ? 1 : 2;
+    d = part == 2 ? x - kKeyed + c_first : x - part * DP;
     return x < channels && (part == 2 ? d < c_first + nv : d < p.dim);
   };
   auto fetch = [&](int x, Channel& c) {
@@ -261,6 +267,11 @@ step_kernel(const ScanArgs p) {
       }
     } else {
       c.x = in.proj[in.col(part) + d];
+      if (FORGET && part == 0) {
+        c.z = decay[d];
+        c.bias = p.dt_bias[h * p.dim + d];
+        c.w[0] = p.lower[h * p.dim + d];
+      }
     }
   };
   auto finish = [&](int x, const Channel& c) {
@@ -283,8 +294,16 @@ step_kernel(const ScanArgs p) {
           if (j < in.back) *o = j == in.back - 1 ? c.x : c.old[j + 1 < kTaps - 1 ? j + 1 : j];
       }
       y = silu_f(y);
-    } else if (!DELTA) {
+    } else if (MEMORY) {
       y = ok ? to_f32<T>(c.x) : part == 2 && d == p.vdim ? 1.f : 0.f;
+    } else if (FORGET) {
+      y = ok ? to_f32<T>(c.x) : 0.f;
+      if (part == 0) {
+        const float z = ok ? to_f32<T>(c.z) + c.bias : 0.f;
+        y = silu_f(y);
+        sG[d] = ok ? forget_keep(z, c.w[0]) : 1.f;
+        sK[d] = ok ? forget_put(z, c.w[0]) : 0.f;
+      }
     }
     if (DELTA && part == 0) sG[d] = ok ? exp2_fast(-kLog2e * a_exp * softplus_f(to_f32<T>(c.z) + c.bias)) : 1.f;
     (part == 0 ? sQ : part == 1 ? sK : sV)[part == 2 ? d - c_first : d] = y;
@@ -311,16 +330,16 @@ step_kernel(const ScanArgs p) {
     fq /= sqrtf(warp_sum(qq) + 1e-6f);
     fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
   }
-  qk *= fq * fk * (DELTA ? 1.f : put);
+  qk *= fq * fk * (MEMORY ? put : 1.f);
   float4 P = make_float4(0.f, 0.f, 0.f, 0.f), Q = P;
 #pragma unroll
   for (int i = 0; i < kRows; i += 4) {
-    const float4 q = load4(sQ + r0 + i), k = load4(sK + r0 + i), g = load4(sG + r0 + i);
+    const float4 q = load4(sQ + r0 + i), k = load4(sK + r0 + i), g = load4(sG + r0 + i);   // (g: not memory)
     const float qs[4] = {q.x, q.y, q.z, q.w}, ks[4] = {k.x, k.y, k.z, k.w}, gs[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
     for (int e = 0; e < 4; ++e) {   // S <- g * S; S^T k, S^T q
       float4& x = S[i + e];
-      const float f = DELTA ? gs[e] : keep;
+      const float f = MEMORY ? keep : gs[e];
       x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
       if (DELTA) axpy4(P, make_float4(ks[e], ks[e], ks[e], ks[e]), x);
       axpy4(Q, make_float4(qs[e], qs[e], qs[e], qs[e]), x);
@@ -338,7 +357,7 @@ step_kernel(const ScanArgs p) {
     }
     if (DELTA) u = beta * (u - fk * pk);
     sV[c] = fmaf(qk, u, fq * o);
-    sP[c] = u * (DELTA ? fk : put);   // what the rows' keys are multiplied by
+    sP[c] = u * (MEMORY ? put : fk);   // what the rows' keys are multiplied by
   }
   __syncthreads();
   const float4 u = load4(sP + c_local);
@@ -357,9 +376,9 @@ step_kernel(const ScanArgs p) {
   if (p.raw != nullptr) {
     float* dst = p.raw + (s.first * p.heads + h) * p.raw_cols + c_first;
     for (int c = tid; c < min(p.nc, p.ncols - c_first); c += threads) dst[c] = sV[c];
-    if (!DELTA && slice == 0 && tid == 0) dst[p.ncols] = expf(-m_new);
+    if (MEMORY && slice == 0 && tid == 0) dst[p.ncols] = expf(-m_new);
   } else {   // every warp the norm, then its own columns
-    float scale = DELTA ? 1.f : 1.f / (fmaxf(fabsf(sV[p.vdim]), expf(-m_new)) + 1e-6f), ss = 0.f;
+    float scale = !MEMORY ? 1.f : 1.f / (fmaxf(fabsf(sV[p.vdim]), expf(-m_new)) + 1e-6f), ss = 0.f;
     for (int c = lane; c < p.vdim; c += 32) {
       const float x = sV[c] * scale;
       ss = fmaf(x, x, ss);
@@ -368,11 +387,11 @@ step_kernel(const ScanArgs p) {
     T* dst = reinterpret_cast<T*>(p.out) + s.first * p.ldo + (long long)h * p.vdim;
     for (int c = tid; c < p.vdim; c += threads)
       dst[c] = from_f32<T>(sV[c] * scale * (c == tid ? norm0 : norm[c]) *
-                           sigmoid_f(to_f32<T>(c == tid ? gate0 : gate[c])));
+                           (FORGET ? 1.f : sigmoid_f(to_f32<T>(c == tid ? gate0 : gate[c]))));
   }
   if (DELTA) {
     if (p.taps > kTaps) save_inputs<T>(p, s, in, qk_block, c_first, max(0, nv));
-  } else if (slice == 0 && tid == 0)
+  } else if (MEMORY && slice == 0 && tid == 0)
     p.max_state[((long long)s.slot * 2 + (s.phase ^ 1)) * p.heads + h] = m_new;
 }
 
@@ -428,8 +447,9 @@ __global__ void __launch_bounds__(1024) memory_gates_kernel(const ScanArgs p) {
 }
 
 // A tile's records of a head: queries, keys, values (convolved), unit lengths, decays, products.
-template <typename T, int DP, bool DELTA>
+template <typename T, int DP, int RULE>
 __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanArgs p) {
+  constexpr bool DELTA = RULE == kDelta, MEMORY = RULE == kMemory, FORGET = RULE == kForget;
   using R = Record<DP, DELTA>;
   constexpr int kThreads = DP <= 128 ? 128 : 256, kWarps = kThreads / 32;
   constexpr int kOwn = (DP + kThreads - 1) / kThreads;
@@ -454,7 +474,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanA
 
   // this thread's channel of the decays, on its way
   float z[kTT];
-  if (DELTA) {
+  if (!MEMORY) {
     const T* src = reinterpret_cast<const T*>(p.decay) + (s.first + t0) * p.ld_decay + h * p.dim + tid;
 #pragma unroll
     for (int t = 0; t < kTT; ++t)
@@ -477,6 +497,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanA
   };
   for (int x = tid * 4; x < 2 * DP + vcols; x += kThreads * 4) {
     const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
+    if (FORGET && part == 1) continue;   // (keys: with the decays)
     const int d = x - part * DP, limit = part == 2 ? p.vdim : p.dim;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.vec && (!DELTA || p.taps <= kTaps)) {
@@ -507,10 +528,11 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanA
           for (int j = 0; j < kTaps - 1; ++j) v[j] = v[4 + j];
         }
       } else {
-        const int one = part == 2 ? p.vdim - d : -1;   // the normaliser's column
+        const int one = MEMORY && part == 2 ? p.vdim - d : -1;   // the normaliser's column
 #pragma unroll
         for (int t = 0; t < kTT; ++t) {
           float4 y = ok && t < nt ? in.four(part, d, t0 + t) : zero;
+          if (FORGET && part == 0) y = silu4(y);
           if (one == 0) y.x = 1.f;
           if (one == 1) y.y = 1.f;
           if (one == 2) y.z = 1.f;
@@ -533,9 +555,10 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanA
             y[e] = silu_f(y[e]);
           } else {
             y[e] = in.one(part, d + e, t0 + t);
+            if (FORGET && part == 0) y[e] = silu_f(y[e]);
           }
         }
-        if (!DELTA && part == 2 && d + e == p.vdim) y[e] = 1.f;
+        if (MEMORY && part == 2 && d + e == p.vdim) y[e] = 1.f;
       }
       put(part, d, t, make_float4(y[0], y[1], y[2], y[3]));
     }
@@ -569,6 +592,19 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanA
       if (t < nt) cum += fmaxf(-ae * softplus_f(z[t] + bias), kMinLogDecay);
       z[t] = cum;
     }
+  } else if (FORGET) {
+    if (tid < DP) {
+      const bool ok = tid < p.dim;
+      const float bias = ok ? p.dt_bias[h * p.dim + tid] : 0.f, lower = ok ? p.lower[h * p.dim + tid] : 0.f;
+#pragma unroll
+      for (int t = 0; t < kTT; ++t) {
+        const float k = ok && t < nt ? (1.f - lower) / (1.f + expf(z[t] + bias)) : 0.f;
+        const float f = lower + (1.f - lower) / (1.f + expf(-z[t] - bias));
+        if (ok && t < nt) cum += fmaxf(k < 0.5f ? log1pf(-k) : logf(f), kMinLogDecay);
+        sB[t * DP + tid] = k;
+        z[t] = cum;
+      }
+    }
   } else {
 #pragma unroll
     for (int t = 0; t < kTT; ++t) {
@@ -585,7 +621,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256) tile_kernel(const ScanA
       const float l = z[t] - base, g = __expf(l);
       const float k = sB[t * DP + tid], q = sC[t * DP + tid];
       const float kn = DELTA ? k * invK[t] : k;
-      const float b = kn * __expf((DELTA ? 0.f : invK[t]) - l);
+      const float b = kn * __expf((MEMORY ? invK[t] : 0.f) - l);
       const float c = q * g * (DELTA ? invQ[t] : p.q_scale);
       sB[t * DP + tid] = b;
       sC[t * DP + tid] = c;
@@ -646,8 +682,9 @@ __host__ __device__ constexpr int stage_floats(int nc) {
   return Record<DP, DELTA>::kV + kTT * nc;
 }
 
-template <typename T, int DP, bool DELTA, int STAGES>
-__global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const ScanArgs p) {
+template <typename T, int DP, int RULE, int STAGES>
+__global__ void __launch_bounds__(max_warps(RULE) * 32, 1) scan_kernel(const ScanArgs p) {
+  constexpr bool DELTA = RULE == kDelta;
   using Sh = ScanShape<DP>;
   using R = Record<DP, DELTA>;
   constexpr int kCols = Sh::kCols, kChunks = Sh::kRows / 4, kKinds = DELTA ? 2 : 1;
@@ -659,7 +696,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
   const Seq s(p.steps + (long long)seq * kStepInts);
   if (s.n <= 0) return;
   if (s.slot <= 0 || s.slot >= p.num_slots) {
-    put_zeros<T, DELTA>(p, s, h, slice);
+    put_zeros<T, RULE>(p, s, h, slice);
     return;
   }
   const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31, rl = lane & 7;
@@ -712,7 +749,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
     float* sV = st + R::kV;
     const bool strong = st[R::kStrong] != 0.f;
     Raw8<T> gates = {};
-    if (p.vec_out && o_t < nt)   // the first outputs' gates, ahead
+    if (RULE != kForget && p.vec_out && o_t < nt)   // the first outputs' gates, ahead
       gates.load(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
     for (int q0 = 0; q0 < nt; q0 += kB) {
       float2 acc[kKinds][kCols][kB];
@@ -810,14 +847,14 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
       for (int t = warp; t < nt; t += threads / 32) {
         float* dst = p.raw + ((s.first + t0 + t) * p.heads + h) * p.raw_cols + c_first;
         for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = sV[t * nc + c];
-        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = st[R::kBeta + t];
+        if (RULE == kMemory && slice == 0 && lane == 0) dst[p.ncols] = st[R::kBeta + t];
       }
     } else if (p.vec_out) {
-      vector_outputs<T, DELTA>(p, sV, nc, st + R::kBeta, nt, lanes, gate + (long long)t0 * p.ld_gate,
+      vector_outputs<T, RULE>(p, sV, nc, st + R::kBeta, nt, lanes, gate + (long long)t0 * p.ld_gate,
                                out + (long long)t0 * p.ldo, w, gates, wa, wb);
     } else {
       for (int t = warp; t < nt; t += threads / 32)
-        head_output<T, DELTA>(p, sV + t * nc, s.first + t0 + t, h, st[R::kBeta + t]);
+        head_output<T, RULE>(p, sV + t * nc, s.first + t0 + t, h, st[R::kBeta + t]);
     }
   }
   copies_wait<0>();
@@ -826,21 +863,22 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 32, 1) scan_kernel(const Sc
 
 // Heads whose columns several blocks share: norm, weight and gate of the raw outputs. A warp per
 // (token, head).
-template <typename T, bool DELTA>
+template <typename T, int RULE>
 __global__ void __launch_bounds__(256) scan_output_kernel(const ScanArgs p, long long n) {
   pdl_wait();
   pdl_trigger();
   const long long k = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (k >= n) return;
   const float* o = p.raw + k * p.raw_cols;
-  head_output<T, DELTA>(p, o, k / p.heads, (int)(k % p.heads), DELTA ? 0.f : o[p.vdim + 1]);
+  head_output<T, RULE>(p, o, k / p.heads, (int)(k % p.heads), RULE == kMemory ? o[p.vdim + 1] : 0.f);
 }
 
-template <typename T, int DP, bool DELTA>
+template <typename T, int DP, int RULE>
 static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, cudaStream_t stream) {
+  constexpr bool DELTA = RULE == kDelta;
   // (one-token steps and 32-bit models; on tensor cores a warp has 16 columns)
   const int wc = a.warp_cols;
-  if (a.nc % wc || a.nc / wc > max_warps(DELTA) || (long long)a.nc * (a.slices - 1) >= a.ncols ||
+  if (a.nc % wc || a.nc / wc > max_warps(RULE) || (long long)a.nc * (a.slices - 1) >= a.ncols ||
       (long long)a.nc * a.slices < a.ncols)
     return -2;
   const long long blocks = (long long)n_seq * a.heads * a.slices;
@@ -850,9 +888,9 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
     using Sh = StepShape<DP>;
     const size_t smem = (size_t)Sh::smem_floats(a.nc) * sizeof(float);
     const dim3 step_threads(a.nc / 4 * Sh::kGroups);
-    if (step_threads.x > Sh::max_threads(DELTA)) return -2;
-    if (!set_smem(step_kernel<T, DP, DELTA>, smem)) return -3;
-    return launch_pdl(step_kernel<T, DP, DELTA>, dim3((unsigned)blocks), step_threads, smem, stream, a) ==
+    if (step_threads.x > Sh::max_threads(RULE)) return -2;
+    if (!set_smem(step_kernel<T, DP, RULE>, smem)) return -3;
+    return launch_pdl(step_kernel<T, DP, RULE>, dim3((unsigned)blocks), step_threads, smem, stream, a) ==
                    cudaSuccess
                ? 0
                : -5;
@@ -861,21 +899,21 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
       a.record < (sizeof(T) == 2 ? MmaRecord<DP, DELTA>::bytes(a.nc * a.slices) / 4
                                  : stage_floats<DP, DELTA>(a.nc * a.slices)))
     return -2;
-  if (!DELTA && launch_pdl(memory_gates_kernel<T>, dim3((unsigned)(n_seq * a.heads)),
+  if (RULE == kMemory && launch_pdl(memory_gates_kernel<T>, dim3((unsigned)(n_seq * a.heads)),
                            dim3(max_rows <= 128 ? 128 : max_rows <= 512 ? 512 : 1024), 0, stream,
                            a) != cudaSuccess)
     return -5;
   if constexpr (sizeof(T) == 2) {
-    return launch_tiles_mma(a, DELTA, n_seq, n_tiles, stream);
+    return launch_tiles_mma(a, RULE, n_seq, n_tiles, stream);
   } else {
     const dim3 tile_grid((unsigned)(n_tiles * a.heads)), tile_threads(DP <= 128 ? 128 : 256);
     const size_t tile_smem = (size_t)(DELTA ? 3 : 2) * kTT * DP * sizeof(float);
-    if (!set_smem(tile_kernel<T, DP, DELTA>, tile_smem)) return -3;
-    if (launch_pdl(tile_kernel<T, DP, DELTA>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
+    if (!set_smem(tile_kernel<T, DP, RULE>, tile_smem)) return -3;
+    if (launch_pdl(tile_kernel<T, DP, RULE>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
       return -5;
     const size_t stage = (size_t)stage_floats<DP, DELTA>(a.nc) * sizeof(float);
     const bool three = 3 * stage <= 220 * 1024;
-    auto k = three ? scan_kernel<T, DP, DELTA, 3> : scan_kernel<T, DP, DELTA, 2>;
+    auto k = three ? scan_kernel<T, DP, RULE, 3> : scan_kernel<T, DP, RULE, 2>;
     const size_t smem = (three ? 3 : 2) * stage;
     if (smem > 220 * 1024) return -6;
     if (!set_smem(k, smem)) return -3;
@@ -883,17 +921,17 @@ static int launch_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, 
   }
 }
 
-template <typename T, bool DELTA>
+template <typename T, int RULE>
 static int run_scan(const ScanArgs& a, int n_seq, int n_tiles, int max_rows, long long rows,
                     cudaStream_t stream) {
-  const int rc = a.dim <= 32    ? launch_scan<T, 32, DELTA>(a, n_seq, n_tiles, max_rows, stream)
-                 : a.dim <= 64  ? launch_scan<T, 64, DELTA>(a, n_seq, n_tiles, max_rows, stream)
-                 : a.dim <= 128 ? launch_scan<T, 128, DELTA>(a, n_seq, n_tiles, max_rows, stream)
-                 : a.dim <= 256 ? launch_scan<T, 256, DELTA>(a, n_seq, n_tiles, max_rows, stream)
+  const int rc = a.dim <= 32    ? launch_scan<T, 32, RULE>(a, n_seq, n_tiles, max_rows, stream)
+                 : a.dim <= 64  ? launch_scan<T, 64, RULE>(a, n_seq, n_tiles, max_rows, stream)
+                 : a.dim <= 128 ? launch_scan<T, 128, RULE>(a, n_seq, n_tiles, max_rows, stream)
+                 : a.dim <= 256 ? launch_scan<T, 256, RULE>(a, n_seq, n_tiles, max_rows, stream)
                                 : -6;
   if (rc != 0 || a.raw == nullptr) return rc;
   const long long n = rows * a.heads;
-  return launch_pdl(scan_output_kernel<T, DELTA>, dim3((unsigned)((n + 7) / 8)), dim3(256), 0, stream, a,
+  return launch_pdl(scan_output_kernel<T, RULE>, dim3((unsigned)((n + 7) / 8)), dim3(256), 0, stream, a,
                     n) == cudaSuccess
              ? 0
              : -5;
@@ -908,7 +946,7 @@ static int warp_cols(int dim, int dtype, bool several) {
   return dim <= 128 || (several && dtype == 0) ? 16 : 8;
 }
 
-// The common part of both entry points
+// The common part of the entry points
 static void finish_args(ScanArgs& a, int slices, int ncols, int raw_cols, void* raw, int dtype,
                         bool several) {
   a.slices = slices;
@@ -936,14 +974,15 @@ typedef __nv_bfloat16 bf16;
 extern "C" {
 
 // Blocks per head so that each block's columns fit: 0 if dim is beyond the kernel's.
-int ab200_scan_min_slices(int dim, int ncols, int delta, int dtype, int several) {
+int ab200_scan_min_slices(int dim, int ncols, int rule, int dtype, int several) {
   if (dim < 1 || dim > 256) return 0;
-  const int most = max_warps(delta != 0) * warp_cols(dim, dtype, several != 0);
+  const int most = max_warps(rule) * warp_cols(dim, dtype, several != 0);
   return (ncols + most - 1) / most;
 }
 
 // Floats of a tile's record of a head (portions of more than one token).
-long long ab200_scan_record(int dim, int ncols, int slices, int delta, int dtype) {
+long long ab200_scan_record(int dim, int ncols, int slices, int rule, int dtype) {
+  const bool delta = rule == kDelta;
   const int wc = warp_cols(dim, dtype, true), nc = ((ncols + slices - 1) / slices + wc - 1) / wc * wc;
   const int dp = dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256;
   if (dtype == 0) {
@@ -995,7 +1034,7 @@ int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_a
   a.tiles = reinterpret_cast<const int*>(tiles);
   a.first_tile = reinterpret_cast<const int*>(first_tile);
   a.records = reinterpret_cast<float*>(records);
-  a.record = ab200_scan_record(dim, vdim, slices, 1, dtype);
+  a.record = ab200_scan_record(dim, vdim, slices, kDelta, dtype);
   a.heads = heads; a.group = heads / kv_heads; a.dim = dim; a.vdim = vdim;
   a.taps = taps;
   a.channels = 2 * kv_heads * dim + heads * vdim;
@@ -1003,8 +1042,8 @@ int ab200_delta_scan(const void* proj, long long ld, int q_at, int k_at, int v_a
   a.out = out; a.ldo = ldo;
   a.status = status;
   finish_args(a, slices, vdim, vdim, raw, dtype, max_rows > 1);
-  return dtype == 0 ? run_scan<bf16, true>(a, n_seq, n_tiles, max_rows, T, stream)
-                    : run_scan<float, true>(a, n_seq, n_tiles, max_rows, T, stream);
+  return dtype == 0 ? run_scan<bf16, kDelta>(a, n_seq, n_tiles, max_rows, T, stream)
+                    : run_scan<float, kDelta>(a, n_seq, n_tiles, max_rows, T, stream);
 }
 
 // Matrix memory: query and key heads of dim, value heads of vdim, gates at i_at and f_at; state
@@ -1038,7 +1077,7 @@ int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_
   a.tiles = reinterpret_cast<const int*>(tiles);
   a.first_tile = reinterpret_cast<const int*>(first_tile);
   a.records = reinterpret_cast<float*>(records);
-  a.record = ab200_scan_record(dim, vdim + 1, slices, 0, dtype);
+  a.record = ab200_scan_record(dim, vdim + 1, slices, kMemory, dtype);
   a.gates = reinterpret_cast<float*>(gates);
   a.heads = heads; a.group = 1; a.dim = dim; a.vdim = vdim;
   a.taps = 1;
@@ -1046,8 +1085,48 @@ int ab200_memory_scan(const void* proj, long long ld, int q_at, int k_at, int v_
   a.out = out; a.ldo = ldo;
   a.status = status;
   finish_args(a, slices, vdim + 1, vdim + 2, raw, dtype, max_rows > 1);
-  return dtype == 0 ? run_scan<bf16, false>(a, n_seq, n_tiles, max_rows, T, stream)
-                    : run_scan<float, false>(a, n_seq, n_tiles, max_rows, T, stream);
+  return dtype == 0 ? run_scan<bf16, kMemory>(a, n_seq, n_tiles, max_rows, T, stream)
+                    : run_scan<float, kMemory>(a, n_seq, n_tiles, max_rows, T, stream);
+}
+
+// Forget scan: query heads of dim at q_at (before silu), forget gates [heads][dim] at f_at (before bias and
+// sigmoid), value heads of vdim at v_at; f_bias and lower fp32 [heads, dim], norm fp32 [vdim]; state
+// [slots, heads, dim, state_cols]; the rest as for ab200_delta_scan, without an output gate.
+int ab200_forget_scan(const void* proj, long long ld, int q_at, int f_at, int v_at, const void* f_bias,
+                      const void* lower, const void* norm, void* state, int state_cols, int num_slots,
+                      const void* steps, int n_seq, int max_rows, const void* tiles,
+                      const void* first_tile, int n_tiles, void* records, long long T, int heads, int dim,
+                      int vdim, int slices, float eps, void* raw, void* out, long long ldo, int dtype,
+                      int* status, cudaStream_t stream) {
+  if (T <= 0 || n_seq <= 0) return 0;
+  if (heads < 1 || dim < 1 || vdim < 1 || slices < 1 || state_cols < vdim || state_cols % 4 ||
+      (slices > 1 && raw == nullptr))
+    return -2;
+  ScanArgs a = {};
+  a.proj = proj; a.ld = ld;
+  a.q_at = q_at; a.k_at = f_at; a.v_at = v_at;
+  a.decay = reinterpret_cast<const char*>(proj) + (long long)f_at * (dtype == 0 ? 2 : 4);
+  a.ld_decay = ld;
+  a.dt_bias = reinterpret_cast<const float*>(f_bias);
+  a.lower = reinterpret_cast<const float*>(lower);
+  a.norm = reinterpret_cast<const float*>(norm);
+  a.state = reinterpret_cast<float*>(state);
+  a.state_cols = state_cols;
+  a.num_slots = num_slots;
+  a.steps = reinterpret_cast<const int*>(steps);
+  a.tiles = reinterpret_cast<const int*>(tiles);
+  a.first_tile = reinterpret_cast<const int*>(first_tile);
+  a.records = reinterpret_cast<float*>(records);
+  a.record = ab200_scan_record(dim, vdim, slices, kForget, dtype);
+  a.heads = heads; a.group = 1; a.dim = dim; a.vdim = vdim;
+  a.taps = 1;
+  a.eps = eps;
+  a.out = out; a.ldo = ldo;
+  a.status = status;
+  finish_args(a, slices, vdim, vdim, raw, dtype, max_rows > 1);
+  a.q_scale = 1.f;
+  return dtype == 0 ? run_scan<bf16, kForget>(a, n_seq, n_tiles, max_rows, T, stream)
+                    : run_scan<float, kForget>(a, n_seq, n_tiles, max_rows, T, stream);
 }
 
 }  // extern "C"

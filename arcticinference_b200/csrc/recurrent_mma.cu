@@ -50,9 +50,11 @@ __device__ __forceinline__ void mma_split(float (&d)[2][4], const uint32_t (&hi)
     mma_bf16(d[n], hi, bh[2 * n], bh[2 * n + 1]);
   }
 }
-template <int DP, bool DELTA>
-__global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 4 : 6) tile_mma_kernel(const ScanArgs p) {
+template <int DP, int RULE>
+__global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : RULE == kMemory ? 6 : 4)
+tile_mma_kernel(const ScanArgs p) {
   typedef __nv_bfloat16 T;
+  constexpr bool DELTA = RULE == kDelta, MEMORY = RULE == kMemory, FORGET = RULE == kForget;
   using R = MmaRecord<DP, DELTA>;
   constexpr int kThreads = DP <= 128 ? 128 : 256, kWarps = kThreads / 32, kLd = R::kLd;
   extern __shared__ __align__(16) float sm[];
@@ -80,13 +82,17 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
   const int d0 = 2 * ((tid & 15) + (tid >> 5) * 16), half = (tid >> 4) & 1;
   uint32_t zr[8] = {};
   float2 z[8];
-  float2 bias = make_float2(0.f, 0.f);
+  float2 bias = make_float2(0.f, 0.f), lower = bias;
   float ae = 0.f;
-  if (DELTA) {
+  if (!MEMORY) {
     if (d0 < p.dim) {
       const T* src = reinterpret_cast<const T*>(p.decay) + (s.first + t0 + half * 8) * p.ld_decay + h * p.dim + d0;
       const bool two = d0 + 1 < p.dim;
-      ae = -kLog2e * p.a_exp[h];     // (logs are to base 2 from here on)
+      if (DELTA) ae = -kLog2e * p.a_exp[h];     // (logs are to base 2 from here on)
+      if (FORGET) {
+        lower.x = p.lower[h * p.dim + d0];
+        if (two) lower.y = p.lower[h * p.dim + d0 + 1];
+      }
       bias.x = p.dt_bias[h * p.dim + d0];
       if (two) bias.y = p.dt_bias[h * p.dim + d0 + 1];
       const int mine = nt - half * 8;
@@ -101,7 +107,9 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
             zr[t] = pack_bf16x2(to_f32<T>(src[t * p.ld_decay]), two ? to_f32<T>(src[t * p.ld_decay + 1]) : 0.f);
       }
     }
-    if (tid < kTT)
+    if (FORGET) {
+      if (tid < kTT) beta[tid] = 1.f;
+    } else if (tid < kTT)
       beta[tid] = tid < nt ? sigmoid_f(to_f32<T>(in.proj[(long long)(t0 + tid) * p.ld + p.b_at + h])) : 0.f;
   } else if (tid < kTT) {
     const float* g = p.gates + ((s.first + t0 + tid) * p.heads + h) * 3;
@@ -115,6 +123,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int x = tid * 4; x < 2 * DP + vcols; x += kThreads * 4) {
     const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
+    if (FORGET && part == 1) continue;   // (keys: with the decays)
     const int d = x - part * DP, limit = part == 2 ? p.vdim : p.dim;
     float* dst = part == 2 ? rec_v + d : (part == 0 ? sC : sB) + d;
     const int dst_ld = part == 2 ? vld : DP;
@@ -156,10 +165,11 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
           for (int j = 0; j < kTaps - 1; ++j) v[j] = v[4 + j];
         }
       } else {
-        const int one = part == 2 ? p.vdim - d : -1;   // the normaliser's column
+        const int one = MEMORY && part == 2 ? p.vdim - d : -1;   // the normaliser's column
 #pragma unroll
         for (int t = 0; t < kTT; ++t, src += p.ld, dst += dst_ld) {
           float4 y = ok && t < nt ? load4(src) : zero;
+          if (FORGET && part == 0) y = silu4(y);
           if (one == 0) y.x = 1.f;
           if (one == 1) y.y = 1.f;
           if (one == 2) y.z = 1.f;
@@ -182,20 +192,28 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
             y[e] = silu_f(y[e]);
           } else {
             y[e] = in.one(part, d + e, t0 + t);
+            if (FORGET && part == 0) y[e] = silu_f(y[e]);
           }
         }
-        if (!DELTA && part == 2 && d + e == p.vdim) y[e] = 1.f;
+        if (MEMORY && part == 2 && d + e == p.vdim) y[e] = 1.f;
       }
       store4(dst + t * dst_ld, make_float4(y[0], y[1], y[2], y[3]));
     }
   }
   // cumulative log decays
   float2 cum = make_float2(0.f, 0.f);
-  if (DELTA) {
+  if (!MEMORY) {
 #pragma unroll
     for (int t = 0; t < 8; ++t) {
-      if (half * 8 + t < nt) {
-        const float zx = __uint_as_float(zr[t] << 16), zy = __uint_as_float(zr[t] & 0xffff0000u);
+      const float zx = __uint_as_float(zr[t] << 16), zy = __uint_as_float(zr[t] & 0xffff0000u);
+      if (FORGET && tid < DP) {   // and the keys
+        const bool x_in = d0 < p.dim && half * 8 + t < nt, y_in = d0 + 1 < p.dim && half * 8 + t < nt;
+        const float kx = x_in ? forget_put(zx + bias.x, lower.x) : 0.f;
+        const float ky = y_in ? forget_put(zy + bias.y, lower.y) : 0.f;
+        *reinterpret_cast<float2*>(sB + (half * 8 + t) * DP + d0) = make_float2(kx, ky);
+        if (x_in) cum.x += fmaxf(forget_log2(forget_keep(zx + bias.x, lower.x), kx), kMinLogDecay * kLog2e);
+        if (y_in) cum.y += fmaxf(forget_log2(forget_keep(zy + bias.y, lower.y), ky), kMinLogDecay * kLog2e);
+      } else if (DELTA && half * 8 + t < nt) {
         cum.x += fmaxf(ae * softplus_f(zx + bias.x), kMinLogDecay * kLog2e);
         cum.y += fmaxf(ae * softplus_f(zy + bias.y), kMinLogDecay * kLog2e);
       }
@@ -224,7 +242,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
         invK[t] = 1.f / sqrtf(b + 1e-6f);
       }
     }
-  } else {
+  } else if (MEMORY) {
     float c = 0.f;
     for (int t = 0; t < half * 8; ++t) c += invQ[t];
 #pragma unroll
@@ -254,7 +272,7 @@ __global__ void __launch_bounds__(DP <= 128 ? 128 : 256, DP > 128 ? 2 : DELTA ? 
       const float2 k = *reinterpret_cast<const float2*>(sB + tok * DP + d0);
       const float2 q = *reinterpret_cast<const float2*>(sC + tok * DP + d0);
       const float fk = DELTA ? invK[tok] : 1.f, fq = DELTA ? invQ[tok] : p.q_scale;
-      const float put = DELTA ? 0.f : invK[tok];
+      const float put = MEMORY ? invK[tok] : 0.f;
       const float kx = k.x * fk, ky = k.y * fk;
       auto split_to = [&](int at, float x, float y) {
         uint32_t hi, lo;
@@ -352,9 +370,10 @@ __device__ __forceinline__ void pair_sync(int pair) {
 // floats a lane of a pair swaps: both halves of P, one of O
 __host__ __device__ constexpr int swap_floats(bool delta) { return delta ? 24 : 8; }
 
-template <int DP, bool DELTA, int STAGES>
-__global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(const ScanArgs p) {
+template <int DP, int RULE, int STAGES>
+__global__ void __launch_bounds__(max_warps(RULE) * 64, 1) scan_mma_kernel(const ScanArgs p) {
   typedef __nv_bfloat16 T;
+  constexpr bool DELTA = RULE == kDelta;
   using R = MmaRecord<DP, DELTA>;
   constexpr int kSwap = swap_floats(DELTA);
   constexpr int kN = DP / 16, kSteps = DP / 32, kLd = R::kLd;   // of a warp's half of the rows
@@ -366,7 +385,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
   const Seq s(p.steps + (long long)seq * kStepInts);
   if (s.n <= 0) return;
   if (s.slot <= 0 || s.slot >= p.num_slots) {
-    put_zeros<T, DELTA>(p, s, h, slice);
+    put_zeros<T, RULE>(p, s, h, slice);
     return;
   }
   const int tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31;
@@ -435,14 +454,14 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
       for (int t = warp; t < nt; t += threads / 32) {
         float* dst = p.raw + ((s.first + t0 + t) * p.heads + h) * p.raw_cols + c_first;
         for (int c = lane; c < min(nc, p.ncols - c_first); c += 32) dst[c] = sV[t * vld + c];
-        if (!DELTA && slice == 0 && lane == 0) dst[p.ncols] = beta[t];
+        if (RULE == kMemory && slice == 0 && lane == 0) dst[p.ncols] = beta[t];
       }
     } else if (p.vec_out) {
-      vector_outputs<T, DELTA>(p, sV, vld, beta, nt, lanes, gate + (long long)t0 * p.ld_gate,
+      vector_outputs<T, RULE>(p, sV, vld, beta, nt, lanes, gate + (long long)t0 * p.ld_gate,
                                out + (long long)t0 * p.ldo, w, gates, wa, wb);
     } else {
       for (int t = warp; t < nt; t += threads / 32)
-        head_output<T, DELTA>(p, sV + t * vld, s.first + t0 + t, h, beta[t]);
+        head_output<T, RULE>(p, sV + t * vld, s.first + t0 + t, h, beta[t]);
     }
   };
 
@@ -457,7 +476,7 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
     float* sV = reinterpret_cast<float*>(st + R::kV);
     const int groups = (int)*reinterpret_cast<const float*>(st + R::kGroups);
     if (it > 0) put_out(it - 1);
-    if (p.vec_out && o_t < nt)   // the first outputs' gates, ahead
+    if (RULE != kForget && p.vec_out && o_t < nt)   // the first outputs' gates, ahead
       gates.load(gate + (long long)(t0 + o_t) * p.ld_gate + o_c);
     for (int grp = 0; grp < groups; ++grp) {
       // read-outs [16 columns x 16 tokens]: P, what is put (U = beta (v - P), solved), O
@@ -559,28 +578,31 @@ __global__ void __launch_bounds__(max_warps(DELTA) * 64, 1) scan_mma_kernel(cons
     }
 }
 
-template <int DP, bool DELTA>
+template <int DP, int RULE>
 static int launch_tiles(const ScanArgs& a, int n_seq, int n_tiles, cudaStream_t stream) {
   const dim3 tile_grid((unsigned)(n_tiles * a.heads)), tile_threads(DP <= 128 ? 128 : 256);
   const long long blocks = (long long)n_seq * a.heads * a.slices;
+  constexpr bool DELTA = RULE == kDelta;
   using R = MmaRecord<DP, DELTA>;
   const size_t tile_smem = (size_t)2 * kTT * DP * 4 + R::kV + kTT * (kTT + 4) * 4;
-  if (!set_smem(tile_mma_kernel<DP, DELTA>, tile_smem)) return -3;
-  if (launch_pdl(tile_mma_kernel<DP, DELTA>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
+  if (!set_smem(tile_mma_kernel<DP, RULE>, tile_smem)) return -3;
+  if (launch_pdl(tile_mma_kernel<DP, RULE>, tile_grid, tile_threads, tile_smem, stream, a) != cudaSuccess)
     return -5;
   const size_t stage = R::bytes(a.nc);
   const size_t swap = (size_t)a.nc / 16 * swap_floats(DELTA) * 32 * 4;
   const bool four = 4 * stage + swap <= 220 * 1024;
-  auto k = four ? scan_mma_kernel<DP, DELTA, 4> : scan_mma_kernel<DP, DELTA, 3>;
+  auto k = four ? scan_mma_kernel<DP, RULE, 4> : scan_mma_kernel<DP, RULE, 3>;
   const size_t smem = (four ? 4 : 3) * stage + swap;
   if (smem > 220 * 1024) return -6;
   if (!set_smem(k, smem)) return -3;
   return launch_pdl(k, dim3((unsigned)blocks), dim3(a.nc / 16 * 64), smem, stream, a) == cudaSuccess ? 0 : -5;
 }
 
-int launch_tiles_mma(const ScanArgs& a, bool delta, int n_seq, int n_tiles, cudaStream_t stream) {
-#define AB200_TILES(DP) \
-  (delta ? launch_tiles<DP, true>(a, n_seq, n_tiles, stream) : launch_tiles<DP, false>(a, n_seq, n_tiles, stream))
+int launch_tiles_mma(const ScanArgs& a, int rule, int n_seq, int n_tiles, cudaStream_t stream) {
+#define AB200_TILES(DP)                                                    \
+  (rule == kDelta    ? launch_tiles<DP, kDelta>(a, n_seq, n_tiles, stream)  \
+   : rule == kForget ? launch_tiles<DP, kForget>(a, n_seq, n_tiles, stream) \
+                     : launch_tiles<DP, kMemory>(a, n_seq, n_tiles, stream))
   return a.dim <= 32    ? AB200_TILES(32)
          : a.dim <= 64  ? AB200_TILES(64)
          : a.dim <= 128 ? AB200_TILES(128)

@@ -1,6 +1,7 @@
 // Kernels around a 32-bit residual stream (decoders that list their layers):
 //
-//   embedding          x (fp32, scaled) and its 16-bit copy that the projections read
+//   embedding          x (fp32, scaled) and its 16-bit copy that the projections read; optionally plus
+//                      a second table's row, looked up by the token and the one before it
 //   stream_norm        x <- norm(alpha * x + y) * (1 + w), in place, plus the 16-bit copy; y is a
 //                      sublayer's output or, for a mixture of experts, the weighted sum of the
 //                      chosen experts' rows, gathered here so that it never exists in memory;
@@ -10,6 +11,12 @@
 //   stream_add         x <- x + norm(y) * w, in place, and the 16-bit copy; y is a sublayer's output,
 //                      half the sum of two normed ones, or a mixture of experts' weighted sum with
 //                      identity experts and a shared expert, formed here in fp32
+//   stream_pre         x <- x + m * y (+ the embedding) (+ a vector), in place, and the next sublayer's
+//                      input act = norm(x) * w, in one pass over the row; y is a sublayer's output plus
+//                      a bias, or a mixture of experts' weighted sum plus a shared expert's rows
+//   poly_norm          a N(z) + b N(z^2) + c N(z^3) + e over the rows of an up projection, N dividing
+//                      by the row's root mean square; the projection's bias is added here
+//   soft_cap           fp32 logits cap * tanh(z / cap)
 //   latent_norm_cache  RMS norm of the compressed K/V projection and its write into the paged
 //                      latent cache
 //   gated_act          act(gate) * up on the interleaved gate / up layout
@@ -22,11 +29,19 @@
 
 namespace ab200 {
 
+// The second embedding: row (prev * mul_prev + id * mul_cur) mod buckets of `table`, the last row where
+// there is no previous token
+struct PairArgs {
+  const long long* prev;   // [T], negative: none; null: no second embedding
+  const void* table;       // [buckets + 1][W]
+  long long buckets, mul_prev, mul_cur;
+};
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 stream_embedding_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
-                        float* __restrict__ x, T* __restrict__ act, float scale, int W,
-                        long long vocab, int* status) {
+                        float* __restrict__ x, T* __restrict__ act, float* __restrict__ keep, float scale,
+                        int W, long long vocab, const PairArgs pairs, int* status) {
   pdl_wait();
   pdl_trigger();
   const long long t = blockIdx.x;
@@ -35,19 +50,37 @@ stream_embedding_kernel(const long long* __restrict__ ids, const T* __restrict__
   // (-1 stands for a token that is not known yet, when a decode step is captured)
   if (id >= vocab && threadIdx.x == 0) report_error(status, kErrBounds, 40, (int)t);
   const T* src = table + (ok ? id : 0) * W;
+  const T* second = nullptr;
+  if (pairs.prev != nullptr) {
+    const long long before = pairs.prev[t];
+    long long row = pairs.buckets;
+    if (before >= 0 && ok) {
+      row = (before * pairs.mul_prev + id * pairs.mul_cur) % pairs.buckets;
+      if (row < 0) row += pairs.buckets;
+    }
+    second = reinterpret_cast<const T*>(pairs.table) + row * W;
+  }
   if (W % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(x) |
-                      reinterpret_cast<uintptr_t>(act)) & 15) == 0) {
+                      reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(keep) |
+                      reinterpret_cast<uintptr_t>(pairs.table)) & 15) == 0) {
     for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
       float4 v = ok ? load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
       v = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+      if (second != nullptr) {
+        const float4 u = load4(second + i);
+        v = make_float4(v.x + u.x, v.y + u.y, v.z + u.z, v.w + u.w);
+      }
       store4(x + t * W + i, v);
+      if (keep != nullptr) store4(keep + t * W + i, v);
       if (act != nullptr) store4(act + t * W + i, v);
     }
     return;
   }
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
-    const float v = ok ? to_f32<T>(src[i]) * scale : 0.f;
+    float v = ok ? to_f32<T>(src[i]) * scale : 0.f;
+    if (second != nullptr) v += to_f32<T>(second[i]);
     x[t * W + i] = v;
+    if (keep != nullptr) keep[t * W + i] = v;
     if (act != nullptr) act[t * W + i] = from_f32<T>(v);
   }
 }
@@ -404,6 +437,262 @@ static int launch_stream_add(const StreamAddArgs& a, long long T_rows, cudaStrea
   return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), smem, stream, a) == cudaSuccess ? 0 : -5;
 }
 
+struct StreamPreArgs {
+  float* x;
+  const void* y;           // optional sublayer output (a mixture: the experts' rows)
+  long long ldy;
+  const float* bias;       // optional [W], added to y
+  const int* y_rows;       // mixture: [T][top] rows of y
+  const float* y_weights;
+  int top;
+  const void* shared;      // optional further rows to add
+  long long ld_shared;
+  float mult;              // of all that
+  const float* base;       // optional [T][W], added to the stream after it
+  const float* step;       // optional [W], likewise
+  const float* w_in;       // with act: weight of the new stream's norm, [W] or (w_scalar) one number
+  int w_scalar;
+  void* act;
+  float eps;
+  int W;
+};
+
+// N4: four-element pieces of the row a thread holds in registers (0: any width, through memory)
+template <typename T, int N4>
+__global__ void __launch_bounds__(256) stream_pre_kernel(const StreamPreArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  float* xr = p.x + t * p.W;
+  const T* yb = reinterpret_cast<const T*>(p.y);
+  const T* sh = p.shared ? reinterpret_cast<const T*>(p.shared) + t * p.ld_shared : nullptr;
+  const float* base = p.base ? p.base + t * p.W : nullptr;
+  T* act = p.act ? reinterpret_cast<T*>(p.act) + t * p.W : nullptr;
+  const bool moved = yb != nullptr || base != nullptr || p.step != nullptr;
+  const float gain = p.w_scalar ? p.w_in[0] : 1.f;
+  const float rw = 1.f / (float)p.W;
+  if constexpr (N4 > 0) {
+    float4 x[N4], f[N4];
+    auto add = [](float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; };
+    auto axpy = [](float4& a, float m, const float4& b) {
+      a.x = fmaf(m, b.x, a.x); a.y = fmaf(m, b.y, a.y);
+      a.z = fmaf(m, b.z, a.z); a.w = fmaf(m, b.w, a.w);
+    };
+    auto each = [&](auto g) {
+#pragma unroll
+      for (int j = 0; j < N4; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * 4;
+        if (i < p.W) g(i, x[j], f[j]);
+      }
+    };
+    each([&](int i, float4& xv, float4& fv) {
+      xv = load4(xr + i);
+      fv = sh != nullptr ? load4(sh + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    });
+    if (p.y_rows != nullptr) {
+      for (int k = 0; k < p.top; ++k) {
+        const float w = p.y_weights[t * p.top + k];
+        const T* yr = yb + (long long)p.y_rows[t * p.top + k] * p.ldy;
+        each([&](int i, float4&, float4& fv) { axpy(fv, w, load4(yr + i)); });
+      }
+    } else if (yb != nullptr) {
+      each([&](int i, float4&, float4& fv) { add(fv, load4(yb + t * p.ldy + i)); });
+    }
+    if (p.bias != nullptr) each([&](int i, float4&, float4& fv) { add(fv, load4(p.bias + i)); });
+    float ss = 0.f;
+    each([&](int i, float4& xv, float4& fv) {
+      axpy(xv, p.mult, fv);
+      if (base != nullptr) add(xv, load4(base + i));
+      if (p.step != nullptr) add(xv, load4(p.step + i));
+      if (moved) store4(xr + i, xv);
+      ss += xv.x * xv.x + xv.y * xv.y + xv.z * xv.z + xv.w * xv.w;
+    });
+    if (act == nullptr) return;
+    const float inv = gain / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+    each([&](int i, float4& xv, float4&) {
+      float4 w = make_float4(inv, inv, inv, inv);
+      if (!p.w_scalar) {
+        const float4 v = load4(p.w_in + i);
+        w = make_float4(inv * v.x, inv * v.y, inv * v.z, inv * v.w);
+      }
+      store4(act + i, make_float4(xv.x * w.x, xv.y * w.y, xv.z * w.z, xv.w * w.w));
+    });
+  } else {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x) {   // a thread re-reads only its own columns
+      float f = sh != nullptr ? to_f32<T>(sh[i]) : 0.f;
+      if (p.y_rows != nullptr) {
+        for (int k = 0; k < p.top; ++k)
+          f = fmaf(p.y_weights[t * p.top + k],
+                   to_f32<T>(yb[(long long)p.y_rows[t * p.top + k] * p.ldy + i]), f);
+      } else if (yb != nullptr) {
+        f += to_f32<T>(yb[t * p.ldy + i]);
+      }
+      if (p.bias != nullptr) f += p.bias[i];
+      float v = fmaf(p.mult, f, xr[i]);
+      if (base != nullptr) v += base[i];
+      if (p.step != nullptr) v += p.step[i];
+      if (moved) xr[i] = v;
+      ss += v * v;
+    }
+    if (act == nullptr) return;
+    const float inv = gain / sqrtf(block_sum_all(ss, red) * rw + p.eps);
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x)
+      act[i] = from_f32<T>(xr[i] * (p.w_scalar ? inv : inv * p.w_in[i]));
+  }
+}
+
+template <typename T>
+static int launch_stream_pre(const StreamPreArgs& a, long long T_rows, cudaStream_t stream) {
+  const bool vec = a.W % 4 == 0 && a.ldy % 4 == 0 && a.ld_shared % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.x) |
+                     reinterpret_cast<uintptr_t>(a.shared) | reinterpret_cast<uintptr_t>(a.bias) |
+                     reinterpret_cast<uintptr_t>(a.base) | reinterpret_cast<uintptr_t>(a.step) |
+                     (a.w_scalar ? 0 : reinterpret_cast<uintptr_t>(a.w_in)) |
+                     reinterpret_cast<uintptr_t>(a.act)) & 15) == 0;
+  const int n4 = (a.W + 3) / 4;
+  auto k = stream_pre_kernel<T, 0>;
+  int threads = 256;
+  if (vec && n4 <= 256 * 8) {
+    while (threads > 64 && n4 <= threads) threads /= 2;
+    const int per = (n4 + threads - 1) / threads;
+    k = per <= 1   ? stream_pre_kernel<T, 1>
+        : per <= 2 ? stream_pre_kernel<T, 2>
+        : per <= 4 ? stream_pre_kernel<T, 4>
+                   : stream_pre_kernel<T, 8>;
+  }
+  return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), 0, stream, a) == cudaSuccess ? 0 : -5;
+}
+
+// Rows of n columns of which the first ff count; a block per row. N4: four-element pieces a thread holds
+// in registers (0: any width, read twice).
+struct PolyArgs {
+  const void* z;
+  const float* bias;   // [ff]
+  const float* coef;   // a, b, c, e
+  void* out;
+  int n, ff;
+  float eps;
+};
+
+// sums of z^2, z^4, z^6 over the block
+__device__ __forceinline__ float3 block_sum3(float3 v, float* red) {
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  v.z = warp_sum(v.z);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = (blockDim.x + 31) >> 5;
+  if (lane == 0) {
+    red[warp] = v.x;
+    red[32 + warp] = v.y;
+    red[64 + warp] = v.z;
+  }
+  __syncthreads();
+  const bool in = lane < warps;
+  return make_float3(warp_sum(in ? red[lane] : 0.f), warp_sum(in ? red[32 + lane] : 0.f),
+                     warp_sum(in ? red[64 + lane] : 0.f));
+}
+
+template <typename T, int N4>
+__global__ void __launch_bounds__(512) poly_norm_kernel(const PolyArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[96];
+  const T* z = reinterpret_cast<const T*>(p.z) + (long long)blockIdx.x * p.n;
+  T* out = reinterpret_cast<T*>(p.out) + (long long)blockIdx.x * p.n;
+  const float a = p.coef[0], b = p.coef[1], c = p.coef[2], e = p.coef[3];
+  const float rf = 1.f / (float)p.ff;
+  float3 s = make_float3(0.f, 0.f, 0.f);
+  auto count = [&](float v) {
+    const float q = v * v, r = q * q;
+    s.x += q;
+    s.y += r;
+    s.z = fmaf(r, q, s.z);
+  };
+  float fa = 0.f, fb = 0.f, fc = 0.f;
+  auto factors = [&]() {
+    s = block_sum3(s, red);
+    fa = a / sqrtf(s.x * rf + p.eps);
+    fb = b / sqrtf(s.y * rf + p.eps);
+    fc = c / sqrtf(s.z * rf + p.eps);
+  };
+  auto poly = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, fc, fb), fa), e); };
+  if constexpr (N4 > 0) {
+    float4 v[N4];
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (threadIdx.x + j * blockDim.x) * 4;
+      v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < p.ff) {
+        const float4 x = load4(z + i), y = load4(p.bias + i);
+        v[j] = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      count(v[j].x);
+      count(v[j].y);
+      count(v[j].z);
+      count(v[j].w);
+    }
+    factors();
+#pragma unroll
+    for (int j = 0; j < N4; ++j) {
+      const int i = (threadIdx.x + j * blockDim.x) * 4;
+      if (i < p.ff)
+        store4(out + i, make_float4(poly(v[j].x), poly(v[j].y), poly(v[j].z), poly(v[j].w)));
+      else if (i < p.n)
+        store4(out + i, make_float4(0.f, 0.f, 0.f, 0.f));
+    }
+  } else {
+    for (int i = threadIdx.x; i < p.ff; i += blockDim.x) count(to_f32<T>(z[i]) + p.bias[i]);
+    factors();
+    for (int i = threadIdx.x; i < p.n; i += blockDim.x)
+      out[i] = from_f32<T>(i < p.ff ? poly(to_f32<T>(z[i]) + p.bias[i]) : 0.f);
+  }
+}
+
+template <typename T>
+static int launch_poly_norm(const PolyArgs& a, long long T_rows, cudaStream_t stream) {
+  const bool vec = a.n % 4 == 0 && a.ff % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.z) | reinterpret_cast<uintptr_t>(a.bias) |
+                     reinterpret_cast<uintptr_t>(a.out)) & 15) == 0;
+  const int n4 = (a.n + 3) / 4;
+  auto k = poly_norm_kernel<T, 0>;
+  int threads = 512;
+  if (vec && n4 <= 512 * 16) {
+    while (threads > 64 && n4 <= threads) threads /= 2;
+    const int per = (n4 + threads - 1) / threads;
+    k = per <= 1   ? poly_norm_kernel<T, 1>
+        : per <= 2 ? poly_norm_kernel<T, 2>
+        : per <= 4 ? poly_norm_kernel<T, 4>
+        : per <= 8 ? poly_norm_kernel<T, 8>
+                   : poly_norm_kernel<T, 16>;
+  }
+  return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), 0, stream, a) == cudaSuccess ? 0 : -5;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+soft_cap_kernel(const T* __restrict__ z, long long ld, float* __restrict__ out, int V, float cap, int vec) {
+  pdl_wait();
+  pdl_trigger();
+  const long long t = blockIdx.y;
+  const T* src = z + t * ld;
+  float* dst = out + t * V;
+  const float inv = 1.f / cap;
+  const int at = blockIdx.x * blockDim.x + threadIdx.x, step = gridDim.x * blockDim.x;
+  if (vec) {
+    for (int i = at * 4; i < V; i += step * 4) {
+      const float4 v = load4(src + i);
+      store4(dst + i, make_float4(cap * tanhf(v.x * inv), cap * tanhf(v.y * inv), cap * tanhf(v.z * inv),
+                                  cap * tanhf(v.w * inv)));
+    }
+  } else {
+    for (int i = at; i < V; i += step) dst[i] = cap * tanhf(to_f32<T>(src[i]) * inv);
+  }
+}
+
 // c = ckv / rms(ckv) * w over R columns -> cache row `slot` of Rp columns (the rest stays zero).
 // One warp per token.
 template <typename T>
@@ -502,18 +791,85 @@ typedef __nv_bfloat16 bf16;
 extern "C" {
 
 // dtype: 0 = bf16, 1 = fp32 (element type of weights, activations and caches)
-int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, float scale,
-                           long long T, int W, long long vocab, int dtype, int* status, cudaStream_t stream) {
+// x fp32 [T, W] = table[ids] * scale, plus, with `prev` int64 [T], the row of `second` [buckets + 1, W]
+// that (prev * mul_prev + id * mul_cur) mod buckets names (prev < 0: the last one). act (may be null): x in
+// the element type; keep (may be null): another copy of x.
+int ab200_stream_embedding(const void* ids, const void* table, void* x, void* act, void* keep, float scale,
+                           long long T, int W, long long vocab, const void* prev, const void* second,
+                           long long buckets, long long mul_prev, long long mul_cur, int dtype,
+                           int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (prev != nullptr && (second == nullptr || buckets < 1)) return -2;
+  const PairArgs pairs = {reinterpret_cast<const long long*>(prev), second, buckets, mul_prev, mul_cur};
   cudaError_t e;
   if (dtype == 0)
     e = launch_pdl(stream_embedding_kernel<bf16>, dim3((unsigned)T), dim3(256), 0, stream,
                    reinterpret_cast<const long long*>(ids), reinterpret_cast<const bf16*>(table),
-                   reinterpret_cast<float*>(x), reinterpret_cast<bf16*>(act), scale, W, vocab, status);
+                   reinterpret_cast<float*>(x), reinterpret_cast<bf16*>(act),
+                   reinterpret_cast<float*>(keep), scale, W, vocab, pairs, status);
   else
     e = launch_pdl(stream_embedding_kernel<float>, dim3((unsigned)T), dim3(256), 0, stream,
                    reinterpret_cast<const long long*>(ids), reinterpret_cast<const float*>(table),
-                   reinterpret_cast<float*>(x), reinterpret_cast<float*>(act), scale, W, vocab, status);
+                   reinterpret_cast<float*>(x), reinterpret_cast<float*>(act),
+                   reinterpret_cast<float*>(keep), scale, W, vocab, pairs, status);
+  return e == cudaSuccess ? 0 : -5;
+}
+
+// In place on x [T, W]: x += mult * f, where f is y + bias (bias may be null) or, with y_rows int32 and
+// y_weights fp32 [T, top], the weighted sum of these rows of y, plus `shared`'s rows (may be null);
+// x += base (fp32 [T, W]) and += step (fp32 [W]) if given; act = norm(x) * w_in if act. All may be null.
+int ab200_stream_pre(void* x, const void* y, long long ldy, const void* bias, const void* y_rows,
+                     const void* y_weights, int top, const void* shared, long long ld_shared,
+                     float mult, const void* base, const void* step, const void* w_in, int w_scalar,
+                     void* act, float eps, long long T, int W, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if ((y_rows != nullptr && (y_weights == nullptr || y == nullptr)) || (act != nullptr && w_in == nullptr) ||
+      (y == nullptr && (bias != nullptr || shared != nullptr)))
+    return -2;
+  StreamPreArgs a;
+  a.x = reinterpret_cast<float*>(x);
+  a.y = y; a.ldy = ldy;
+  a.bias = reinterpret_cast<const float*>(bias);
+  a.y_rows = reinterpret_cast<const int*>(y_rows);
+  a.y_weights = reinterpret_cast<const float*>(y_weights);
+  a.top = top;
+  a.shared = shared; a.ld_shared = ld_shared;
+  a.mult = mult;
+  a.base = reinterpret_cast<const float*>(base);
+  a.step = reinterpret_cast<const float*>(step);
+  a.w_in = reinterpret_cast<const float*>(w_in);
+  a.w_scalar = w_scalar && w_in != nullptr;
+  a.act = act;
+  a.eps = eps;
+  a.W = W;
+  return dtype == 0 ? launch_stream_pre<bf16>(a, T, stream) : launch_stream_pre<float>(a, T, stream);
+}
+
+// z, out [T, n] (element type by dtype), of whose columns the first ff count (the others become zero):
+// a N(z') + b N(z'^2) + c N(z'^3) + e with z' = z + bias; bias fp32 [ff], coef fp32 [4] (a, b, c, e)
+int ab200_poly_norm(const void* z, const void* bias, const void* coef, void* out, long long T, int n,
+                    int ff, float eps, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (ff < 1 || ff > n) return -2;
+  const PolyArgs a = {z, reinterpret_cast<const float*>(bias), reinterpret_cast<const float*>(coef), out,
+                      n, ff, eps};
+  return dtype == 0 ? launch_poly_norm<bf16>(a, T, stream) : launch_poly_norm<float>(a, T, stream);
+}
+
+// out fp32 [T, V] = cap * tanh(z / cap), z [T, ld]
+int ab200_soft_cap(const void* z, long long ld, void* out, long long T, int V, float cap, int dtype,
+                   cudaStream_t stream) {
+  if (T <= 0 || V <= 0) return 0;
+  if (!(cap > 0.f) || T > 65535) return -2;
+  const int vec = V % 4 == 0 && ld % 4 == 0 &&
+                  ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const int per = (V + 1023) / 1024;
+  const dim3 grid((unsigned)(per < 64 ? per : 64), (unsigned)T);
+  const cudaError_t e =
+      dtype == 0 ? launch_pdl(soft_cap_kernel<bf16>, grid, dim3(256), 0, stream,
+                              reinterpret_cast<const bf16*>(z), ld, reinterpret_cast<float*>(out), V, cap, vec)
+                 : launch_pdl(soft_cap_kernel<float>, grid, dim3(256), 0, stream,
+                              reinterpret_cast<const float*>(z), ld, reinterpret_cast<float*>(out), V, cap, vec);
   return e == cudaSuccess ? 0 : -5;
 }
 

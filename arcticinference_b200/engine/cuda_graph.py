@@ -48,7 +48,9 @@ class DecodeGraph:
         self.max_blocks = (cfg.scheduler.max_model_len + runner.block_size - 1) // runner.block_size
         max_q = 1 + (cfg.speculative.max_draft_tokens if cfg.speculative else 0)
         self.plans = m.decode_plans(bucket, max_q, runner.block_size)
-        n64 = 4 * bucket      # ids | positions | slots | source rows of run-ahead tokens
+        # ids | positions | slots | source rows of run-ahead tokens | tokens before them, if asked for
+        self.pairs = cfg.model.bigram is not None
+        n64 = (5 if self.pairs else 4) * bucket
         self.state_plan = StateDecodePlan(bucket) if runner.num_state_slots else None
         n32 = bucket * self.max_blocks + sum(p.int32_words for p in self.plans)
         if self.state_plan is not None:
@@ -71,6 +73,8 @@ class DecodeGraph:
         self.batch = ForwardBatch(input_ids=self.d64[:B], positions=self.d64[B:2 * B],
                                   slots=self.d64[2 * B:3 * B], attn_meta=self.meta,
                                   logits_indices=self.logits_indices, num_tokens=B, mode=mode)
+        if self.pairs:
+            self.batch.prev_ids = self.d64[4 * B:5 * B]
         if self.state_plan is not None:
             self.batch.state = self.state_plan.step
         if cfg.model.is_swiftkv:
@@ -105,7 +109,8 @@ class DecodeGraph:
             src[:len(src_rows)] = src_rows
         bt = h32[:B * MB].reshape(B, MB)
         from .model_runner import pack_tokens
-        q_lens, kv_lens, offs = pack_tokens(out.scheduled, bs, ids, pos, slots, bt)
+        prev = h64[4 * B:5 * B] if self.pairs else None
+        q_lens, kv_lens, offs = pack_tokens(out.scheduled, bs, ids, pos, slots, bt, prev)
         rows = [[t] if n == 1 else list(range(t, t + n)) for t, n in zip(offs, q_lens)]
         t = offs[-1] + q_lens[-1] if offs else 0
         N = t
@@ -113,6 +118,8 @@ class DecodeGraph:
             ids[N:] = 0
             pos[N:] = 0
             slots[N:] = -1
+            if self.pairs:
+                prev[N:] = -1
             bt[len(q_lens), :] = 0
             q_lens.append(B - N)
             kv_lens.append(B - N)

@@ -32,12 +32,14 @@ from .sampler import row_seed
 from .scheduler import SchedulerOutput
 
 
-def pack_tokens(sched, bs: int, ids, pos, slots, bt):
+def pack_tokens(sched, bs: int, ids, pos, slots, bt, prev=None):
     """Write token ids, positions, cache slots and block-table rows of the scheduled requests
     into the staging arrays. Single-token requests (the bulk of a serving step) are gathered
     in Python lists and written with three vector assignments; only multi-token chunks touch
-    numpy per request. Returns (q_lens, kv_lens, token offset of each request)."""
-    one_t, one_tok, one_pos, one_slot = [], [], [], []
+    numpy per request. ``prev`` (optional) receives the token before each one, -1 at a sequence's
+    start; it is always known here: of a request, only the newest token can be a placeholder.
+    Returns (q_lens, kv_lens, token offset of each request)."""
+    one_t, one_tok, one_pos, one_slot, one_prev = [], [], [], [], []
     q_lens, kv_lens, offs = [], [], []
     t = 0
     for i, s in enumerate(sched):
@@ -50,12 +52,17 @@ def pack_tokens(sched, bs: int, ids, pos, slots, bt):
             one_tok.append(r.token_at(st))
             one_pos.append(st)
             one_slot.append(r.block_ids[st // bs] * bs + st % bs)
+            if prev is not None:
+                one_prev.append(r.token_at(st - 1) if st else -1)
         else:
             known = r.num_tokens
             seq = r.tokens_slice(st, min(st + n, known))
             if len(seq) < n:
                 seq = seq + list(r.spec_token_ids[:n - len(seq)])
             ids[t:t + n] = seq
+            if prev is not None:
+                prev[t] = r.token_at(st - 1) if st else -1
+                prev[t + 1:t + n] = seq[:-1]
             p = np.arange(st, st + n, dtype=np.int64)
             pos[t:t + n] = p
             blocks = r.block_array().astype(np.int64)
@@ -69,6 +76,8 @@ def pack_tokens(sched, bs: int, ids, pos, slots, bt):
         ids[one_t] = one_tok
         pos[one_t] = one_pos
         slots[one_t] = one_slot
+        if prev is not None:
+            prev[one_t] = one_prev
     return q_lens, kv_lens, offs
 
 
@@ -267,13 +276,15 @@ class ModelRunner:
                     prompt_spans.append((s, s.start, hi - s.start))
         n_sel = n_smp + sum(c for _, _, c in prompt_spans)
         max_blocks = max(len(s.request.block_ids) for s in sched)
-        stage = self._stage(3 * Np + n_sel + n_sel)
+        pairs = self.config.model.bigram is not None
+        stage = self._stage(3 * Np + n_sel + n_sel + (Np if pairs else 0))
         h = stage.numpy()
         ids, pos, slots = h[:Np], h[Np:2 * Np], h[2 * Np:3 * Np]
         sel = h[3 * Np:3 * Np + n_sel]
         sel_pos = h[3 * Np + n_sel:3 * Np + 2 * n_sel]
         bt = np.zeros((len(sched), max_blocks), dtype=np.int32)
-        q_lens, kv_lens, offs = pack_tokens(sched, bs, ids, pos, slots, bt)
+        prev = h[3 * Np + 2 * n_sel:] if pairs else None
+        q_lens, kv_lens, offs = pack_tokens(sched, bs, ids, pos, slots, bt, prev)
         k = 0
         rows = []
         sel_q_lens = []
@@ -317,6 +328,8 @@ class ModelRunner:
             ids[N:] = 0
             pos[N:] = 0
             slots[N:] = -1
+            if pairs:
+                prev[N:] = -1
         dev = self.device
         d = stage.to(dev, non_blocking=True)
         self._stage_done()
@@ -355,6 +368,8 @@ class ModelRunner:
                              attn_meta=meta, logits_indices=d[3 * Np:3 * Np + n_sel],
                              num_tokens=Np, mode=mode)
         batch.num_sampled = n_smp
+        if pairs:
+            batch.prev_ids = d[3 * Np + 2 * n_sel:]
         if self.num_state_slots:
             batch.state = StateStep.of(sched, q_lens, Np - N, dev)
             self.h2d_bytes += batch.state.uploaded_bytes

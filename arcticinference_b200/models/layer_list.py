@@ -1,6 +1,6 @@
 """Decoders whose config.json lists their layers one by one, each with its own mixer and
-feed-forward: Taralix, Zatirax and Pererax. ``config.LAYER_LIST_DESIGNS`` says what each name stands for;
-``mixers.py`` has the mixers.
+feed-forward: Taralix, Zatirax, Pererax and Pefivik. ``config.LAYER_LIST_DESIGNS`` says what each name
+stands for; ``mixers.py`` has the mixers.
 
 Taralix: norms after the residual sum.
 
@@ -15,11 +15,19 @@ that use other layers' weights.
 
     x <- x + norm1(mixer(x)) * ls1;   x <- x + norm2(feed_forward(x)) * ls2
 
+Pefivik: a norm before each sublayer, whose output enters with a constant factor; layers that run
+several times, the embedding entering again ahead of every further pass; a second embedding of token
+pairs; softly capped logits.
+
+    x <- x + m * mixer(norm1(x));   x <- x + m * feed_forward(norm2(x))
+
 The residual stream ``x`` is fp32 from the embedding to the final norm; the projections read the
 model's element type, written by the same kernel that updates the stream. Per layer: one input
 projection, norms and rotation with the cache write, attention, output projection, stream update;
 then gate / up with the activation in the product's epilogue, down, stream update (for experts
-that kernel also takes the weighted sum of the chosen experts' rows). Routing stays on the device.
+that kernel also takes the weighted sum of the chosen experts' rows). An activation that needs a
+token's whole row (PolyNorm) is a kernel of its own, which adds the up projection's bias; the down
+projection's is added by the stream update. Routing stays on the device.
 
 A *run* is one execution of a layer: a layer inside the loop has one per pass, and a layer whose
 weights others use one for each of them, each with a cache and state of its own
@@ -61,8 +69,8 @@ def scale_names(cfg: ModelConfig, spec) -> list:
 
 
 def router_vector(f) -> str:
-    """The vector beside the router's matrix: a bias, or a correction of the choice."""
-    return "mlp.correction" if f.scoring == "all" else "mlp.router.b"
+    """The vector beside the router's matrix: a bias, a correction of the choice, or none."""
+    return {"chosen": "mlp.router.b", "all": "mlp.correction", "sigmoid": None}[f.scoring]
 
 
 def required_tensors(cfg: ModelConfig, spec) -> list:
@@ -75,8 +83,10 @@ def required_tensors(cfg: ModelConfig, spec) -> list:
     if f is not None and f.shared is not None:
         names += ["mlp.shared." + n for n in ("gate", "up", "down")]
     if f is not None and f.experts:
-        names += ["mlp.router", router_vector(f)]
+        names += [n for n in ("mlp.router", router_vector(f)) if n is not None]
         names += ["mlp.e%d.%s" % (e, n) for e in range(f.experts) for n in ("gate", "up", "down")]
+    elif f is not None and f.act == "poly_norm":
+        names += ["mlp.up", "mlp.up.b", "mlp.down", "mlp.down.b", "mlp.act"]
     elif f is not None:
         names += ["mlp.gate", "mlp.up", "mlp.down"]
     return names
@@ -99,7 +109,10 @@ def random_state(cfg: ModelConfig, seed: int, device, dtype) -> Iterable:
     yield "embed", rnd(cfg.vocab_size, W, std=1.0)
     if not cfg.tie_word_embeddings:
         yield "head", rnd(cfg.vocab_size, W)
-    yield "final.norm", one + rnd(W, std=0.1)
+    gains = () if cfg.design.scalar_norms else (W,)
+    yield "final.norm", one + rnd(*gains, std=0.1)
+    if cfg.bigram is not None:
+        yield "bigram", rnd(cfg.bigram.buckets + 1, W, std=0.5)
     if cfg.loop is not None:
         yield "loop.step", rnd(cfg.loop.times, W, std=0.1)
     for i, l in enumerate(cfg.layer_specs):
@@ -107,7 +120,7 @@ def random_state(cfg: ModelConfig, seed: int, device, dtype) -> Iterable:
         if l.weights_of is not None:
             continue
         for n in norm_names(cfg, l):
-            yield p + n, one + rnd(W, std=0.1)
+            yield p + n, one + rnd(*gains, std=0.1)
         for n in scale_names(cfg, l):
             yield p + n, 1.0 + rnd(W, std=0.1)
         for n, t in mixer_class(l.mixer).random(l.mixer, W, rnd):
@@ -117,7 +130,15 @@ def random_state(cfg: ModelConfig, seed: int, device, dtype) -> Iterable:
         if f.experts:
             outputs = f.experts + f.identity
             yield p + "mlp.router", rnd(outputs, W)
-            yield p + router_vector(f), rnd(outputs, std=0.1 if f.scoring == "chosen" else 0.1 / outputs)
+            if router_vector(f) is not None:
+                yield p + router_vector(f), rnd(outputs, std=0.1 if f.scoring == "chosen" else 0.1 / outputs)
+        elif f.act == "poly_norm":
+            yield p + "mlp.up", rnd(f.ff, W)
+            yield p + "mlp.up.b", rnd(f.ff, std=0.1)
+            yield p + "mlp.down", rnd(W, f.ff)
+            yield p + "mlp.down.b", rnd(W, std=0.1)
+            yield p + "mlp.act", 0.5 + rnd(4, std=0.1)
+            continue
         ffs = {"mlp.e%d." % e: f.ff for e in range(f.experts)} if f.experts else {"mlp.": f.ff}
         if f.shared is not None:
             ffs["mlp.shared."] = f.shared.ff
@@ -142,7 +163,7 @@ class LayerListForCausalLM:
         self.h, self.hkv = cfg.num_attention_heads, 1
         self.D = cfg.head_dim
         self.layers: list = [None] * cfg.num_hidden_layers
-        self.embed = self.norm = self.lm_head = None
+        self.embed = self.norm = self.lm_head = self.bigram = None
         if cfg.loop is not None:
             self.loop_step = None
         self._lay_out()
@@ -160,7 +181,7 @@ class LayerListForCausalLM:
                 self.mixers.append(LatentMixer(l.mixer, sharing, self.dtype, self.device))
             else:
                 self.mixers.append(mixer_class(l.mixer)(l.mixer, self.dtype, self.device))
-        gate = lambda f: None if f is None else st.Gate(f.act, f.limit)
+        gate = lambda f: None if f is None or f.act == "poly_norm" else st.Gate(f.act, f.limit)
         self.gates = [gate(l.mlp) for l in specs]
         self.shared_gates = [gate(l.mlp and l.mlp.shared) for l in specs]
         self.runs = self.cfg.layer_runs
@@ -196,7 +217,9 @@ class LayerListForCausalLM:
         V, W = cfg.vocab_size, cfg.hidden_size
         pending: dict = {}
         need = [set(required_tensors(cfg, l)) for l in cfg.layer_specs]
-        top = {"embed": (V, W), "final.norm": (W,)}
+        top = {"embed": (V, W), "final.norm": () if cfg.design.scalar_norms else (W,)}
+        if cfg.bigram is not None:
+            top["bigram"] = (cfg.bigram.buckets + 1, W)
         if not cfg.tie_word_embeddings:
             top["head"] = (V, W)
         if cfg.loop is not None:
@@ -212,7 +235,9 @@ class LayerListForCausalLM:
                 elif name == "embed":
                     self.embed = t
                 elif name == "final.norm":
-                    self.norm = t.float()
+                    self.norm = t.float().expand(W).contiguous()
+                elif name == "bigram":
+                    self.bigram = t
                 elif name == "loop.step":
                     self.loop_step = t.float()
                 else:
@@ -241,6 +266,9 @@ class LayerListForCausalLM:
         self.mixers[l].pack(c, lw, W)
         scales = dict(zip(("norm1", "norm2"), scale_names(self.cfg, spec)))
         for n in norm_names(self.cfg, spec):
+            if self.design.scalar_norms:
+                lw.put(**{n: c.take(n).float().reshape(1)})
+                continue
             v = c.vector(n, W)
             if n in scales:      # norm and layer scale are factors of the same vector
                 v = v * c.vector(scales[n], W)
@@ -255,11 +283,20 @@ class LayerListForCausalLM:
                    shared_down=padded(down, W, round_up(ff, st.GATE_BLOCK)).contiguous())
         if f.experts:
             outputs = f.experts + f.identity
-            lw.put(router=c.take("mlp.router", outputs, W),
-                   router_b=c.vector(router_vector(f), outputs))
+            b = router_vector(f)
+            lw.put(router=c.take("mlp.router", outputs, W))
+            if b is not None:
+                lw.put(router_b=c.vector(b, outputs))
             stack = lambda n, *s: torch.stack(
                 [c.take("mlp.e%d.%s" % (e, n), *s) for e in range(f.experts)])
             gate, up, down = stack("gate", f.ff, W), stack("up", f.ff, W), stack("down", W, f.ff)
+        elif f.act == "poly_norm":
+            n = round_up(f.ff, 8) if self.dtype == torch.bfloat16 else f.ff
+            lw.put(w_up=padded(c.take("mlp.up", f.ff, W), n).contiguous(),
+                   w_down=padded(c.take("mlp.down", W, f.ff), W, n).contiguous(),
+                   up_bias=c.vector("mlp.up.b", f.ff), down_bias=c.vector("mlp.down.b", W),
+                   act=c.vector("mlp.act", 4))
+            return lw
         else:
             gate, up, down = (c.take("mlp.gate", f.ff, W), c.take("mlp.up", f.ff, W),
                               c.take("mlp.down", W, f.ff))
@@ -274,6 +311,8 @@ class LayerListForCausalLM:
         yield "embed", self.embed
         yield "norm", self.norm
         yield "lm_head", self.lm_head
+        if self.bigram is not None:
+            yield "bigram", self.bigram
         if self.cfg.loop is not None:
             yield "loop_step", self.loop_step
         for i, lw in enumerate(self.layers):
@@ -365,14 +404,26 @@ class LayerListForCausalLM:
 
     # ------------------------------------------------------------------ forward
     def _feed_forward(self, l: int, x, act):
-        """(output rows, routing): with a routing the rows are the experts', still to be summed."""
+        """(output rows, routing): with a routing the rows are the experts', still to be summed, and
+        with a bias on the down projection it is still to be added. ``x``: what the router reads."""
         lw, f, gate = self.layers[l], self.cfg.layer_specs[l].mlp, self.gates[l]
+        if f.act == "poly_norm":
+            h = st.poly_norm(ops.linear(act, lw.w_up), lw.up_bias, lw.act, f.ff, self.cfg.rms_norm_eps)
+            return ops.linear(h, lw.w_down), None
         if not f.experts:
             return ops.linear(st.gated_linear(act, lw.w_gu, gate), lw.w_down), None
-        routing, rows = st.route(x, act, lw.router, lw.router_b, f.top, f.identity,
-                                 f.router_scale if f.scoring == "all" else None)
+        routing, rows = st.route(x, act, lw.router, getattr(lw, "router_b", None), f.top, f.identity,
+                                 f.router_scale if f.scoring != "chosen" else None,
+                                 (f.groups, f.keep_groups) if f.scoring == "sigmoid" else None)
         h = st.grouped_linear(rows, lw.w_gu, routing, act=gate)
         return st.grouped_linear(h, lw.w_down, routing), routing
+
+    def _shared_expert(self, l: int, act):
+        """Rows of the expert that every token uses, None where there is none."""
+        lw, gate = self.layers[l], self.shared_gates[l]
+        if gate is None:
+            return None
+        return ops.linear(st.gated_linear(act, lw.shared_gu, gate), lw.shared_down)
 
     def forward(self, batch: ForwardBatch, kv, layers_out: list = None) -> torch.Tensor:
         """Final-norm states of the sampled rows [B, W]. ``layers_out`` receives a copy of the
@@ -382,7 +433,7 @@ class LayerListForCausalLM:
         mix = lambda r, l, act: self.mixers[l].run(act, self.layers[l], batch, kv.of(r),
                                                    kv.state_of(r), step, shared, eps)
         body = {"post": self._post_norm_body, "sandwich": self._sandwich_body,
-                "output": self._output_norm_body}[self.design.residual]
+                "output": self._output_norm_body, "pre": self._pre_norm_body}[self.design.residual]
         x = body(batch, mix, layers_out)
         return st.stream_final_norm(x, batch.logits_indices, self.norm, eps, self.dtype,
                                     self.design.norm_offset)
@@ -440,17 +491,54 @@ class LayerListForCausalLM:
             st.stream_add(x, act, lw.norm1, eps, y, pair=pair)
             if self.cfg.layer_specs[l].mlp is not None:
                 y, routing = self._feed_forward(l, x, act)
-                shared = None
-                if self.shared_gates[l] is not None:
-                    shared = ops.linear(st.gated_linear(act, lw.shared_gu, self.shared_gates[l]),
-                                        lw.shared_down)
-                st.stream_add(x, act, lw.norm2, eps, y, experts=routing, shared=shared)
+                st.stream_add(x, act, lw.norm2, eps, y, experts=routing,
+                              shared=self._shared_expert(l, act))
             if layers_out is not None:
                 layers_out.append(x.clone())
         return x
 
+    def _pre_norm_body(self, batch, mix, layers_out):
+        cfg, loop = self.cfg, self.cfg.loop
+        eps, mult = cfg.rms_norm_eps, cfg.residual_mult
+        T, W, dev = batch.input_ids.numel(), cfg.hidden_size, self.device
+        x0 = None       # the embedding, where later passes of the loop add it
+        if loop is not None and loop.reenter and loop.times > 1:
+            x0 = torch.empty(T, W, dtype=torch.float32, device=dev)
+        pairs = None if cfg.bigram is None else (batch.prev_ids, self.bigram, cfg.bigram)
+        x, _ = st.stream_embedding(batch.input_ids, self.embed, cfg.embedding_scale, rounded=False,
+                                   pairs=pairs, keep=x0)
+        act = torch.empty(T, W, dtype=self.dtype, device=dev)
+        update = lambda **kw: st.stream_pre(x, mult, eps, **kw)
+
+        def enter(r, out):
+            """The stream after a sublayer's output and what run ``r`` reads of it."""
+            if r == len(self.runs):
+                if out:
+                    update(**out)
+                return
+            l, t = self.runs[r]
+            update(**out, base=x0 if t else None, step=None if t is None else self.loop_step[t],
+                   w_in=self.layers[l].norm1, act=act)
+
+        enter(0, {})
+        for r, (l, _) in enumerate(self.runs):
+            lw, out = self.layers[l], {"y": mix(r, l, act)}
+            if cfg.layer_specs[l].mlp is not None:
+                update(**out, w_in=lw.norm2, act=act)
+                y, routing = self._feed_forward(l, act, act)
+                out = {"y": y, "bias": getattr(lw, "down_bias", None), "experts": routing,
+                       "shared": self._shared_expert(l, act)}
+            if layers_out is not None:
+                update(**out)
+                layers_out.append(x.clone())
+                out = {}
+            enter(r + 1, out)
+        return x
+
     def compute_logits(self, hidden: torch.Tensor, fp32: bool = False) -> torch.Tensor:
-        V = self.cfg.vocab_size
+        V, cap = self.cfg.vocab_size, self.cfg.logit_softcap
         if fp32 and self.dtype != torch.float32:
-            return hidden.float() @ self.lm_head[:V].float().t()
-        return ops.linear(hidden, self.lm_head)[:, :V]
+            logits = hidden.float() @ self.lm_head[:V].float().t()
+        else:
+            logits = ops.linear(hidden, self.lm_head)[:, :V]
+        return st.soft_cap(logits, cap) if cap else logits

@@ -294,6 +294,8 @@ class ForwardBatch:
     sel_positions: Optional[torch.Tensor] = None
     # models with recurrent layers: the step's sequences and their state slots (ops.state_ops)
     state: object = None
+    # models that embed pairs of tokens: the token before each one, -1 at a sequence's start
+    prev_ids: Optional[torch.Tensor] = None
     # the first ``num_sampled`` selected rows are sampled; further rows are prompt positions
     # whose log-probabilities were asked for: (request, first position, count) per span and
     # the token that follows each such position

@@ -3,10 +3,12 @@ attention is planned and how it runs. A mixer object belongs to a layer and hold
 weights lie in the layer's :class:`LayerWeights`.
 
 * :class:`LatentMixer`: keys and values from one cached latent per token, optionally with a rotated
-  key part that the heads share (``ops/latent_ops.py``);
+  key part that the heads share, a sink and an output gate per head (``ops/latent_ops.py``);
 * :class:`HeadMixer`: cached keys and values, with norms, rotation, soft cap, sink and output gate as
   its spec asks (``ops/head_ops.py``);
 * :class:`DeltaMixer`: gated delta rule, a state per head instead of a cache (``ops/state_ops.py``);
+* :class:`ForgetMixer`: linear attention whose forget gate also decides what is written, a state per
+  head (``ops/state_ops.py``);
 * :class:`ParallelMixer`: attention and a matrix memory (:class:`MemoryMixer`) side by side.
 
 Sizes that the tensor-core kernels tile by are padded with zeros, which changes no value.
@@ -17,8 +19,8 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from ..config import (AttentionSpec, DeltaRuleSpec, LatentAttentionSpec, MatrixMemorySpec,
-                      ParallelSpec)
+from ..config import (AttentionSpec, DeltaRuleSpec, ForgetScanSpec, LatentAttentionSpec,
+                      MatrixMemorySpec, ParallelSpec)
 from ..ops import head_ops as heads
 from ..ops import latent_ops as lat
 from ..ops import state_ops as states
@@ -126,7 +128,8 @@ class LatentMixer:
     @staticmethod
     def names(m: LatentAttentionSpec) -> list:
         own = [] if m.kv_from is not None else ["mix.dkv", "mix.dkv.norm"]
-        return ["mix.q", "mix.uk", "mix.uv", "mix.o"] + own
+        return ["mix.q", "mix.uk", "mix.uv", "mix.o"] + own + \
+            (["mix.sink"] if m.sink == "learned" else []) + (["mix.g"] if m.head_gate else [])
 
     @staticmethod
     def random(m: LatentAttentionSpec, W: int, rnd):
@@ -136,6 +139,10 @@ class LatentMixer:
             yield "mix.dkv.norm", 1.0 + rnd(m.kv_rank, std=0.1)
         yield "mix.uk", rnd(m.heads * m.dim, m.kv_rank)
         yield "mix.uv", rnd(m.heads * m.vdim, m.kv_rank)
+        if m.sink == "learned":
+            yield "mix.sink", rnd(m.heads, std=1.0)
+        if m.head_gate:
+            yield "mix.g", rnd(m.heads, W)
         yield "mix.o", rnd(W, m.heads * m.vdim)
 
     def pack(self, c: Checkpoint, lw: LayerWeights, W: int) -> None:
@@ -146,13 +153,16 @@ class LatentMixer:
         self.scale = m.scale
         if m.scale <= 0:
             q, self.scale = (-q, -m.scale) if m.scale < 0 else (torch.zeros_like(q), 1.0)
-        rows = [q.reshape(H * dq, W)]
+        cols = Columns(self.dtype)
+        cols.add(q.reshape(H * dq, W))
         if m.kv_from is None:
-            n = R + m.rot_dim
-            cols = round_up(n, 8) if self.dtype == torch.bfloat16 else n
-            rows.append(padded(c.take("mix.dkv", n, W), cols))
+            cols.add(c.take("mix.dkv", R + m.rot_dim, W))
             lw.put(ckv_norm=c.vector("mix.dkv.norm", R))
-        lw.put(wq=torch.cat(rows, 0).contiguous())
+        if m.head_gate:
+            self.gate_at = cols.add(c.take("mix.g", H, W))
+        if m.sink == "learned":
+            lw.put(sink=c.vector("mix.sink", H))
+        lw.put(wq=cols.weight())
         uk = padded(c.take("mix.uk", H * m.dim, R).view(H, m.dim, R), H, dq, lo.width)
         for i in range(m.rot_dim):      # the shared rotated part passes through
             uk[:, m.dim + i, lo.rot_at + i] = 1.0
@@ -191,12 +201,15 @@ class LatentMixer:
                                   cache, self.layout.rot_at)
         elif m.kv_from is None:
             lat.latent_norm_cache(proj[:, nq:], lw.ckv_norm, m.kv_rank, eps, batch.slots, cache)
+        sink = lw.sink if m.sink is not None else None
+        gate = proj[:, self.gate_at:self.gate_at + H] if m.head_gate else None
         n = T if self.expand is None else step.n_absorbed
         out = torch.empty(T, H * self.dv, dtype=self.dtype, device=act.device)
         if n:
             q = st.head_linear(proj[:n, :nq], lw.wuk_t)
             o = lat.latent_attention(q, cache, step.absorbed[(self.shape, n == T)], self.shape,
-                                     self.scale, step.tok_seq, batch.positions)
+                                     self.scale, step.tok_seq, batch.positions, sink,
+                                     gate if gate is None else gate[:n])
             st.head_linear(o, lw.wuv, out=out[:n])
         if n < T:
             key = (cache.data_ptr(), m.mask)
@@ -206,7 +219,8 @@ class LatentMixer:
                                                     step.ctx[m.mask][0])
             kvs = ops.linear(c, lw.wukv)
             lat.expanded_attention(proj[n:, :nq], kvs[:, :nq], kvs[:, nq:], step, H, self.expand,
-                                   self.scale, out[n:], m.mask)
+                                   self.scale, out[n:], m.mask, sink,
+                                   gate if gate is None else gate[n:])
         return ops.linear(out, lw.wo)
 
 
@@ -422,6 +436,43 @@ class DeltaMixer(StatefulMixer):
         return ops.linear(out, lw.wo)
 
 
+class ForgetMixer(StatefulMixer):
+    def __init__(self, spec: ForgetScanSpec, dtype: torch.dtype, device):
+        self.spec, self.dtype = spec, dtype
+
+    @property
+    def state_rows(self) -> list:
+        m = self.spec
+        return [((m.heads, m.dim, round_up(m.vdim, 4)), torch.float32)]
+
+    @staticmethod
+    def names(m: ForgetScanSpec) -> list:
+        return ["mix." + n for n in ("q", "f", "f.b", "lower", "v", "norm", "o")]
+
+    @staticmethod
+    def random(m: ForgetScanSpec, W: int, rnd):
+        nk, nv = m.heads * m.dim, m.heads * m.vdim
+        for x, n in (("q", nk), ("f", nk), ("v", nv)):
+            yield "mix." + x, rnd(n, W)
+        yield "mix.f.b", rnd(nk, std=0.5) + 2.0
+        yield "mix.lower", torch.sigmoid(rnd(nk, std=1.0))
+        yield "mix.norm", 1.0 + rnd(m.vdim, std=0.1)
+        yield "mix.o", rnd(W, nv)
+
+    def pack(self, c: Checkpoint, lw: LayerWeights, W: int) -> None:
+        m, cols = self.spec, Columns(self.dtype)
+        nk, nv = m.heads * m.dim, m.heads * m.vdim
+        at = [cols.add(c.take("mix." + x, n, W)) for x, n in (("q", nk), ("f", nk), ("v", nv))]
+        lw.put(win=cols.weight(), f_bias=c.vector("mix.f.b", nk), lower=c.vector("mix.lower", nk),
+               norm=c.vector("mix.norm", m.vdim), wo=c.take("mix.o", W, nv))
+        self.scan = states.ForgetShape(m.heads, m.dim, m.vdim, *at)
+
+    def run(self, act, lw: LayerWeights, batch, cache, state, step, shared: dict, eps: float):
+        out = states.forget_scan(ops.linear(act, lw.win), lw.f_bias, lw.lower, lw.norm, self.scan,
+                                 *state, batch.state, eps)
+        return ops.linear(out, lw.wo)
+
+
 class MemoryMixer(StatefulMixer):
     def __init__(self, spec: MatrixMemorySpec, dtype: torch.dtype, device, at: str = ""):
         self.spec, self.dtype, self.at = spec, dtype, at
@@ -515,7 +566,7 @@ class ParallelMixer:
 
 
 MIXERS = {LatentAttentionSpec: LatentMixer, AttentionSpec: HeadMixer, DeltaRuleSpec: DeltaMixer,
-          ParallelSpec: ParallelMixer}
+          ForgetScanSpec: ForgetMixer, ParallelSpec: ParallelMixer}
 
 
 def mixer_class(spec):

@@ -1064,7 +1064,8 @@ def attention_masked(q, k, v, meta: AttentionMetadata, Hq: int, Hkv: int, D: int
                      Dk: int | None = None, softcap: float = 0.0) -> torch.Tensor:
     """Causal attention with a lower bound on the keys (``mask``, a MaskSpec), an optional sink
     (fp32 [Hq]: a further term of the softmax denominator), an optional output gate (rows
-    [T, Hq * D]; the output is multiplied by their sigmoid) and, with ``softcap`` > 0, scores
+    [T, Hq * D], or [T, Hq] with one number per head; the output is multiplied by their sigmoid) and, with
+    ``softcap`` > 0, scores
     softcap * tanh(score / softcap). CUDA tensors only. Keys and values:
     caches [num_blocks, Hkv, block_size, D], or with ``paged`` false rows [n, Hkv * D] (of queries
     and keys Hkv * Dk, where given: 192 with D = 128). ``meta`` must have been planned with the
@@ -1079,12 +1080,15 @@ def attention_masked(q, k, v, meta: AttentionMetadata, Hq: int, Hkv: int, D: int
         assert k.is_contiguous() and v.is_contiguous()
     else:
         assert k.stride(0) == v.stride(0)
+    per_head = gate is not None and gate.shape[1] == Hq
+    assert gate is None or gate.stride(1) == 1
     rc = nat.lib().ab200_attention_ext(
         q.data_ptr(), q.stride(0), k.data_ptr(), v.data_ptr(), 0 if paged else k.stride(0),
         k.shape[0], k.shape[2] if paged else 0, nat.ptr(bt), bt.shape[1] if paged else 0,
         meta.work.data_ptr(), meta.num_work, nat.ptr(meta.tok_splits) if meta.max_splits > 1 else None,
         meta.max_splits, T, Hq, Hkv, Dk or D, D, mask.code, mask.size, nat.ptr(sink), nat.ptr(gate),
-        gate.stride(0) if gate is not None else 0, float(scale), float(softcap), out.data_ptr(),
+        gate.stride(0) if gate is not None else 0, int(per_head), float(scale), float(softcap),
+        out.data_ptr(),
         out.stride(0), nat.ptr(meta.o_part), nat.ptr(meta.lse_part), meta.tile_keys if paged else 128,
         nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "attention_masked")

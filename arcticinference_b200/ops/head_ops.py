@@ -140,16 +140,19 @@ def attention_exact(q, k_cache, v_cache, block_tables, tok_seq, positions, H: in
                     Dv: int, scale: float, mask: MaskSpec, sink=None, gate=None,
                     softcap: float = 0.0) -> torch.Tensor:
     """fp32-accumulating attention without tensor cores; q [T, H * Dk], caches [num_blocks, Hkv,
-    block_size, >= Dk / Dv] (they may be one tensor). Returns [T, H * Dv]."""
+    block_size, >= Dk / Dv] (they may be one tensor); ``gate`` [T, H * Dv], or [T, H]: one per head.
+    Returns [T, H * Dv]."""
     nat = _nat()
     T = q.shape[0]
+    assert gate is None or gate.stride(1) == 1
     out = torch.empty(T, H * Dv, dtype=q.dtype, device=q.device)
     assert q.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
     rc = nat.lib().ab200_attention_exact(
         q.data_ptr(), q.stride(0), k_cache.data_ptr(), k_cache.shape[3], v_cache.data_ptr(),
         v_cache.shape[3], k_cache.shape[0], k_cache.shape[2], block_tables.data_ptr(),
         block_tables.shape[1], tok_seq.data_ptr(), positions.data_ptr(), nat.ptr(sink),
-        nat.ptr(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), T, H,
+        nat.ptr(gate), gate.stride(0) if gate is not None else 0,
+        int(gate is not None and gate.shape[1] == H), out.data_ptr(), out.stride(0), T, H,
         Hkv, Dk, Dv, mask.code, mask.size, float(scale), float(softcap), dtype_code(q.dtype),
         nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "attention_exact")

@@ -302,7 +302,20 @@ def latent_rope_cache(q, ckv, heads: int, dq: int, dim: int, weight, rank: int, 
     launch_counter.add(1)
 
 
-def latent_attention_ref(q, cache, meta, shape: LatentShape, scale):
+def sink_softmax(s, sink):
+    """Softmax of scores [H, n, k] over their last dimension, with exp(sink[h]) in the denominator."""
+    if sink is None:
+        return torch.softmax(s, -1)
+    s = torch.cat([s, sink.view(-1, 1, 1).expand(*s.shape[:2], 1)], -1)
+    return torch.softmax(s, -1)[..., :-1]
+
+
+def gated_heads(o, gate):
+    """o [n, H, d] times the sigmoid of gate [n, H]."""
+    return o if gate is None else o * torch.sigmoid(gate.float()).unsqueeze(-1)
+
+
+def latent_attention_ref(q, cache, meta, shape: LatentShape, scale, sink=None, gate=None):
     nb, _, bs, W = cache.shape
     H, R = shape.heads, shape.rank
     flat = cache.view(nb * bs, W)
@@ -316,37 +329,42 @@ def latent_attention_ref(q, cache, meta, shape: LatentShape, scale):
         s = torch.einsum("thr,kr->htk", q[t:t + n].reshape(n, H, W).float(), c) * scale
         at = torch.arange(kl - n, kl).view(n, 1)
         s = s.masked_fill((pos > at) | (pos < shape.mask.first_key(at)), float("-inf"))
-        o = torch.einsum("htk,kr->thr", torch.softmax(s, -1), c[:, :R])
+        o = torch.einsum("htk,kr->thr", sink_softmax(s, sink), c[:, :R])
+        o = gated_heads(o, None if gate is None else gate[t:t + n])
         out[t:t + n] = o.reshape(n, H * R).to(q.dtype)
         t += n
     return out
 
 
 def latent_attention(q: torch.Tensor, cache: torch.Tensor, meta: AttentionMetadata,
-                     shape: LatentShape, scale: float, tok_seq=None, positions=None):
+                     shape: LatentShape, scale: float, tok_seq=None, positions=None, sink=None,
+                     gate=None):
     """q [T, H * width] in latent space; cache [num_blocks, 1, block_size, width]. Softmax over the
-    keys the shape's mask shows; returns [T, H * rank]. ``tok_seq`` and ``positions`` (per token)
-    are read by the "exact" kernel only."""
+    keys the shape's mask shows; returns [T, H * rank]. ``sink`` fp32 [H]: a further term of the
+    denominator, as its logarithm; ``gate`` [T, H] (row stride free): heads' outputs are multiplied
+    by its sigmoid. ``tok_seq`` and ``positions`` (per token) are read by the "exact" kernel only."""
     H, R, W = shape.heads, shape.rank, shape.width
     bt = meta.block_tables
     if not q.is_cuda:
-        return latent_attention_ref(q, cache, meta, shape, scale)
+        return latent_attention_ref(q, cache, meta, shape, scale, sink, gate)
     nat = _nat()
     T = q.shape[0]
     assert q.is_contiguous() and cache.is_contiguous() and cache.shape[3] == W
     if shape.kernel == "packed":
-        if shape.mask.kind == "causal":
+        if shape.mask.kind == "causal" and sink is None and gate is None:
             return attention(q, cache, cache, meta, H, 1, R, scale)
-        return attention_masked(q, cache, cache, meta, H, 1, R, scale, shape.mask)
+        return attention_masked(q, cache, cache, meta, H, 1, R, scale, shape.mask, sink, gate)
     if shape.kernel == "exact":
         return attention_exact(q, cache, cache, bt, tok_seq, positions, H, 1, W, R, scale,
-                               shape.mask)
+                               shape.mask, sink, gate)
+    assert gate is None or gate.stride(1) == 1
     out = torch.empty(T, H * R, dtype=q.dtype, device=q.device)
     rc = nat.lib().ab200_latent_attention(
         q.data_ptr(), T * H, cache.data_ptr(), cache.shape[0], cache.shape[2], bt.data_ptr(),
         bt.shape[1], meta.work.data_ptr(), meta.num_work, nat.ptr(meta.tok_splits),
         meta.max_splits, T, H, R, shape.key_extra, shape.mask.code, shape.mask.size,
-        shape.tile_rows, float(scale), out.data_ptr(), nat.ptr(meta.o_part), nat.ptr(meta.lse_part),
+        shape.tile_rows, float(scale), nat.ptr(sink), nat.ptr(gate),
+        gate.stride(0) if gate is not None else 0, out.data_ptr(), nat.ptr(meta.o_part), nat.ptr(meta.lse_part),
         nat.status_buffer(q.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "latent_attention")
     launch_counter.add(2 if meta.max_splits > 1 else 1)
@@ -364,17 +382,18 @@ def expanded_widths(dq: int, dv: int):
 
 
 def expanded_attention(q, k, v, step: AttentionStep, H: int, widths: tuple, scale: float, out,
-                       mask: MaskSpec = CAUSAL) -> None:
+                       mask: MaskSpec = CAUSAL, sink=None, gate=None) -> None:
     """Attention of the step's long chunks over expanded keys and values (rows of ``k`` and ``v``:
     the keys those sequences see, one sequence after the other, as ``step.ctx[mask]`` names them;
-    ``widths``: columns of a head of each)."""
+    ``widths``: columns of a head of each). ``sink`` and ``gate``: see latent_attention."""
     Dk, D = widths
     if q.is_cuda:
         meta = step.exp_plans[(H, widths, mask)]
-        if mask.kind == "causal" and Dk == D:
+        if mask.kind == "causal" and Dk == D and sink is None and gate is None:
             attention_contiguous(q, k, v, None, H, D, scale, causal=True, meta=meta, out=out)
         else:
-            attention_masked(q, k, v, meta, H, H, D, scale, mask, out=out, paged=False, Dk=Dk)
+            attention_masked(q, k, v, meta, H, H, D, scale, mask, sink, gate, out=out, paged=False,
+                             Dk=Dk)
         return
     t = r = 0
     for n, kl, lo in zip(step.exp_q_lens, step.exp_kv_lens, step.ctx[mask][1]):
@@ -383,6 +402,7 @@ def expanded_attention(q, k, v, step: AttentionStep, H: int, widths: tuple, scal
         s = torch.einsum("thd,khd->htk", qs, ks) * scale
         at, pos = torch.arange(kl - n, kl).view(n, 1), torch.arange(lo, kl)
         s = s.masked_fill((pos > at) | (pos < mask.first_key(at)), float("-inf"))
-        out[t:t + n] = torch.einsum("htk,khd->thd", torch.softmax(s, -1), vs) \
-            .reshape(n, H * D).to(out.dtype)
+        o = torch.einsum("htk,khd->thd", sink_softmax(s, sink), vs)
+        o = gated_heads(o, None if gate is None else gate[t:t + n])
+        out[t:t + n] = o.reshape(n, H * D).to(out.dtype)
         t, r = t + n, r + kl - lo

@@ -123,7 +123,10 @@ def _declare(L: ctypes.CDLL) -> None:
         "ab200_mlp_spec_step": (I, [P, LL, P, P, F, P, P, P, LL, LL, I, F, I, P]),
         "ab200_sum_lstm": (I, [P, LL, P, I, P, F, P, LL, P, P, P, P, P, P, LL, LL, I, F, I, P]),
         "ab200_verify_greedy": (I, [P, P, P, P, I, I, P, P, P, P, P]),
-        "ab200_stream_embedding": (I, [P, P, P, P, F, LL, I, LL, I, P, P]),
+        "ab200_stream_embedding": (I, [P, P, P, P, P, F, LL, I, LL, P, P, LL, LL, LL, I, P, P]),
+        "ab200_stream_pre": (I, [P, P, LL, P, P, P, I, P, LL, F, P, P, P, I, P, F, LL, I, I, P]),
+        "ab200_poly_norm": (I, [P, P, P, P, LL, I, I, F, I, P]),
+        "ab200_soft_cap": (I, [P, LL, P, LL, I, F, I, P]),
         "ab200_stream_norm": (I, [P, P, P, LL, P, P, I, P, F, F, F, P, P, LL, I, I, P]),
         "ab200_stream_sandwich": (I, [P, P, LL, P, P, P, P, F, F, LL, I, I, P]),
         "ab200_stream_add": (I, [P, P, P, P, LL, P, P, LL, P, P, P, I, P, LL, F, LL, I, I, P]),
@@ -133,24 +136,26 @@ def _declare(L: ctypes.CDLL) -> None:
                                  I, P, LL, I, I, I, I, I, F, P, P, LL, I, P, P]),
         "ab200_memory_scan": (I, [P, LL, I, I, I, I, I, P, LL, P, P, F, P, P, I, P, I, P, I, I, P, P, I, P,
                                   P, LL, I, I, I, I, F, P, P, LL, I, P, P]),
+        "ab200_forget_scan": (I, [P, LL, I, I, I, P, P, P, P, I, I, P, I, I, P, P, I, P, LL, I, I, I, I, F, P,
+                                  P, LL, I, P, P]),
         "ab200_latent_norm_cache": (I, [P, LL, P, I, I, F, P, P, LL, LL, I, P, P]),
         "ab200_gated_act": (I, [P, P, LL, I, I, F, F, I, P]),
         "ab200_linear_exact": (I, [P, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, P]),
-        "ab200_attention_exact": (I, [P, LL, P, I, P, I, I, I, P, I, P, P, P, P, LL, P, LL, LL, I,
+        "ab200_attention_exact": (I, [P, LL, P, I, P, I, I, I, P, I, P, P, P, P, LL, I, P, LL, LL, I,
                                       I, I, I, I, I, F, F, I, P, P]),
         "ab200_rotary_table": (I, [P, P, P, LL, I, P]),
         "ab200_head_rope_cache": (I, [P, LL, P, I, P, P, P, P, P, LL, I, I, I, I, I, I, LL, F, I, I, I,
                                       P, P]),
         "ab200_latent_rope_cache": (I, [P, P, LL, P, I, P, P, P, LL, I, I, I, I, I, I, LL, F, I, P,
                                         P]),
-        "ab200_moe_route": (I, [P, P, P, LL, I, I, I, I, I, F, P, P, P, P, P, P, I, P]),
+        "ab200_moe_route": (I, [P, I, P, P, LL, I, I, I, I, I, F, I, I, P, P, P, P, P, P, I, P]),
         "ab200_moe_permute": (I, [P, P, P, P, P, LL, I, I, I, I, P]),
         "ab200_grouped_gemm": (I, [P, LL, LL, LL, P, LL, LL, P, LL, LL, I, I, I, I, P, P, I, I, F,
                                    F, P, P]),
-        "ab200_latent_attention": (I, [P, LL, P, I, I, P, I, P, I, P, I, LL, I, I, I, I, I, I, F, P,
-                                       P, P, P, P]),
+        "ab200_latent_attention": (I, [P, LL, P, I, I, P, I, P, I, P, I, LL, I, I, I, I, I, I, F, P, P,
+                                       LL, P, P, P, P, P]),
         "ab200_attention_ext": (I, [P, LL, P, P, LL, LL, I, P, I, P, I, P, I, LL, I, I, I, I, I, I, P,
-                                    P, LL, F, F, P, LL, P, P, I, P, P]),
+                                    P, LL, I, F, F, P, LL, P, P, I, P, P]),
         "ab200_attention": (I, [P, LL, P, P, LL, LL, I, P, I, P, I, P, I, LL, I, I, I, I, F, P,
                                 LL, P, P, P, I, P, P]),
     }

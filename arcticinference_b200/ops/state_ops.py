@@ -98,10 +98,13 @@ class StateDecodePlan:
         self._host[:, 2] = 0
 
 
-def slices_for(dim: int, ncols: int, delta: bool, dtype: torch.dtype, blocks: int, long: bool) -> int:
+MEMORY, DELTA, FORGET = 0, 1, 2     # recurrences (csrc/common/recurrent.cuh)
+
+
+def slices_for(dim: int, ncols: int, rule: int, dtype: torch.dtype, blocks: int, long: bool) -> int:
     """Blocks that share a head's columns: as few as hold them, more where a prompt's few heads
     would leave most of the GPU idle."""
-    least = _nat().lib().ab200_scan_min_slices(dim, ncols, int(delta), dtype_code(dtype), int(long))
+    least = _nat().lib().ab200_scan_min_slices(dim, ncols, rule, dtype_code(dtype), int(long))
     if least == 0:
         raise NotImplementedError("recurrent layers with keys of more than 256 dimensions")
     width = 16 if dim <= 128 or (long and dtype == torch.bfloat16) else 8     # of a warp
@@ -113,15 +116,15 @@ def slices_for(dim: int, ncols: int, delta: bool, dtype: torch.dtype, blocks: in
     return -(-ncols // cols)
 
 
-def _scratch(s, ncols: int, delta: bool, steps: StateStep, proj: torch.Tensor):
+def _scratch(s, ncols: int, rule: int, steps: StateStep, proj: torch.Tensor):
     """(slices, raw outputs or None, tile records or None) of a scan."""
-    slices = slices_for(s.dim, ncols, delta, proj.dtype, steps.table.shape[0] * s.heads,
+    slices = slices_for(s.dim, ncols, rule, proj.dtype, steps.table.shape[0] * s.heads,
                         steps.max_rows > 1)
     f32 = dict(dtype=torch.float32, device=proj.device)
-    raw = torch.empty(proj.shape[0], s.heads, ncols + (not delta), **f32) if slices > 1 else None
+    raw = torch.empty(proj.shape[0], s.heads, ncols + (rule == MEMORY), **f32) if slices > 1 else None
     records = None
     if steps.max_rows > 1:
-        size = _nat().lib().ab200_scan_record(s.dim, ncols, slices, int(delta), dtype_code(proj.dtype))
+        size = _nat().lib().ab200_scan_record(s.dim, ncols, slices, rule, dtype_code(proj.dtype))
         records = torch.empty(steps.tiles.shape[0], s.heads, size, **f32)
     return slices, raw, records
 
@@ -154,7 +157,8 @@ def _head_output(o, norm, gate, eps):
     """o fp32 [n, heads, vdim] -> [n, heads * vdim]."""
     n = o.shape[0]
     o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps)
-    return (o * norm).reshape(n, -1) * torch.sigmoid(gate.float())
+    o = (o * norm).reshape(n, -1)
+    return o if gate is None else o * torch.sigmoid(gate.float())
 
 
 def delta_scan_ref(proj, decay, gate, conv, a_exp, dt_bias, norm, s: DeltaShape, state, conv_state,
@@ -205,7 +209,7 @@ def delta_scan(proj, decay, gate, conv, a_exp, dt_bias, norm, s: DeltaShape, sta
     nat = _nat()
     T, n = proj.shape[0], steps.table.shape[0]
     out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
-    slices, raw, records = _scratch(s, s.vdim, True, steps, proj)
+    slices, raw, records = _scratch(s, s.vdim, DELTA, steps, proj)
     assert proj.stride(1) == decay.stride(1) == gate.stride(1) == 1
     assert state.is_contiguous() and conv_state.is_contiguous() and steps.table.is_contiguous()
     rc = nat.lib().ab200_delta_scan(
@@ -218,6 +222,70 @@ def delta_scan(proj, decay, gate, conv, a_exp, dt_bias, norm, s: DeltaShape, sta
         out.stride(0), dtype_code(proj.dtype), nat.status_buffer(proj.device).data_ptr(),
         nat.stream_ptr())
     nat.check(rc, "delta_scan")
+    launch_counter.add(1 + (slices > 1) + (records is not None))
+    return out
+
+
+# ------------------------------------------------------------------------------ forget scan
+@dataclass(frozen=True)
+class ForgetShape:
+    heads: int
+    dim: int
+    vdim: int
+    # columns of the input projection
+    q_at: int
+    f_at: int
+    v_at: int
+
+    @property
+    def state_cols(self) -> int:
+        return -(-self.vdim // 4) * 4
+
+
+def forget_scan_ref(proj, f_bias, lower, norm, s: ForgetShape, state, steps: StateStep, eps: float):
+    H, d, dv = s.heads, s.dim, s.vdim
+    out = torch.zeros(proj.shape[0], H * dv, dtype=proj.dtype)
+    for first, n, slot, start, _ in steps.table.tolist():
+        if slot <= 0:
+            continue
+        rows = slice(first, first + n)
+        p = proj[rows].float()
+        q = F.silu(p[:, s.q_at:s.q_at + H * d]).view(n, H, d)
+        z = p[:, s.f_at:s.f_at + H * d] + f_bias
+        k = ((1.0 - lower) * torch.sigmoid(-z)).view(n, H, d)      # 1 - f
+        f = (lower + (1.0 - lower) * torch.sigmoid(z)).view(n, H, d)
+        v = p[:, s.v_at:s.v_at + H * dv].view(n, H, dv)
+        S = state[slot, :, :, :dv].clone() if start > 0 else torch.zeros(H, d, dv)
+        o = torch.empty(n, H, dv)
+        for t in range(n):
+            S = f[t].unsqueeze(-1) * S + k[t].unsqueeze(-1) * v[t].unsqueeze(1)
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        state[slot, :, :, :dv] = S
+        out[rows] = _head_output(o, norm, None, eps).to(out.dtype)
+    return out
+
+
+def forget_scan(proj, f_bias, lower, norm, s: ForgetShape, state, steps: StateStep,
+                eps: float) -> torch.Tensor:
+    """Linear attention with a forget gate f per channel and 1 - f in the key's place, over a step's
+    sequences: from the input projection (queries before their silu, gates before bias and sigmoid,
+    values) to the normed heads [T, heads * vdim]. ``f_bias`` and ``lower`` (the gates' lower bound)
+    fp32 [heads * dim]; ``norm`` fp32 [vdim]; ``state`` fp32 [slots, heads, dim, state_cols]."""
+    if not proj.is_cuda:
+        return forget_scan_ref(proj, f_bias, lower, norm, s, state, steps, eps)
+    nat = _nat()
+    T, n = proj.shape[0], steps.table.shape[0]
+    out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
+    slices, raw, records = _scratch(s, s.vdim, FORGET, steps, proj)
+    assert proj.stride(1) == 1 and state.is_contiguous() and steps.table.is_contiguous()
+    rc = nat.lib().ab200_forget_scan(
+        proj.data_ptr(), proj.stride(0), s.q_at, s.f_at, s.v_at, f_bias.data_ptr(), lower.data_ptr(),
+        norm.data_ptr(), state.data_ptr(), state.shape[3], state.shape[0], steps.table.data_ptr(), n,
+        steps.max_rows, nat.ptr(steps.tiles), nat.ptr(steps.first_tile),
+        steps.tiles.shape[0] if records is not None else 0, nat.ptr(records), T, s.heads, s.dim,
+        s.vdim, slices, float(eps), nat.ptr(raw), out.data_ptr(), out.stride(0),
+        dtype_code(proj.dtype), nat.status_buffer(proj.device).data_ptr(), nat.stream_ptr())
+    nat.check(rc, "forget_scan")
     launch_counter.add(1 + (slices > 1) + (records is not None))
     return out
 
@@ -284,7 +352,7 @@ def memory_scan(proj, gate, i_bias, f_bias, norm, s: MemoryShape, state, max_sta
     nat = _nat()
     T, n = proj.shape[0], steps.table.shape[0]
     out = torch.empty(T, s.heads * s.vdim, dtype=proj.dtype, device=proj.device)
-    slices, raw, records = _scratch(s, s.vdim + 1, False, steps, proj)
+    slices, raw, records = _scratch(s, s.vdim + 1, MEMORY, steps, proj)
     gates = torch.empty(T, s.heads, 3, dtype=torch.float32, device=proj.device) \
         if records is not None else None
     assert proj.stride(1) == gate.stride(1) == 1

@@ -60,11 +60,23 @@ def dtype_code(dt: torch.dtype) -> int:
 
 
 # ------------------------------------------------------------------------ residual stream
+def bigram_rows(ids, prev, bigram) -> torch.Tensor:
+    rows = (prev * bigram.mul_prev + ids * bigram.mul_cur) % bigram.buckets
+    return torch.where(prev < 0, bigram.buckets, rows)
+
+
 def stream_embedding(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0,
-                     rounded: bool = True):
-    """(x, act) of the token embeddings times ``scale``; act is None unless ``rounded``."""
+                     rounded: bool = True, pairs: tuple = None, keep: torch.Tensor = None):
+    """(x, act) of the token embeddings times ``scale``; act is None unless ``rounded``. ``pairs``:
+    (previous token of every token, negative where there is none, the table of a bigram embedding
+    [buckets + 1, W], its BigramSpec), added in fp32. ``keep`` fp32 [T, W] receives a copy of x."""
     if not table.is_cuda:
         x = table[ids].float() * scale
+        if pairs is not None:
+            prev, second, bigram = pairs
+            x = x + second[bigram_rows(ids, prev, bigram)].float()
+        if keep is not None:
+            keep.copy_(x)
         if not rounded:
             return x, None
         return (x, x) if table.dtype == torch.float32 else (x, x.to(table.dtype))
@@ -75,10 +87,15 @@ def stream_embedding(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0,
     if rounded:
         act = x if table.dtype == torch.float32 else torch.empty(T, W, dtype=table.dtype,
                                                                  device=table.device)
+    prev, second, bigram = pairs or (None, None, None)
+    assert ids.is_contiguous() and (prev is None or (
+        prev.dtype == ids.dtype and prev.is_contiguous() and second.dtype == table.dtype and
+        second.shape[0] == bigram.buckets + 1))
     rc = nat.lib().ab200_stream_embedding(
         ids.data_ptr(), table.data_ptr(), x.data_ptr(), None if act is x else nat.ptr(act),
-        float(scale), T, W, table.shape[0], dtype_code(table.dtype), nat.status_buffer(table.device).data_ptr(),
-        nat.stream_ptr())
+        nat.ptr(keep), float(scale), T, W, table.shape[0], nat.ptr(prev), nat.ptr(second),
+        *((bigram.buckets, bigram.mul_prev, bigram.mul_cur) if bigram else (0, 0, 0)),
+        dtype_code(table.dtype), nat.status_buffer(table.device).data_ptr(), nat.stream_ptr())
     nat.check(rc, "stream_embedding")
     launch_counter.add(1)
     return x, act
@@ -179,6 +196,61 @@ def stream_add(x, act, w, eps: float, y=None, pair=None, experts: "Routing" = No
     launch_counter.add(1)
 
 
+def stream_pre(x, mult: float, eps: float, y=None, bias=None, experts: "Routing" = None, shared=None,
+               base=None, step=None, w_in=None, act=None) -> None:
+    """In place, in one pass over the rows of the stream: ``x += mult * f`` if a sublayer's output is
+    given, ``x += base`` (fp32 [T, W]) and ``x += step`` (fp32 [W]) if they are; then ``act = norm(x) *
+    w_in`` if ``act`` is given: what the next sublayer reads. f is ``y`` + ``bias`` (fp32 [W], or None)
+    or, with ``experts`` (``y``: the experts' rows), each token's weighted sum plus the rows of
+    ``shared``. ``w_in`` fp32: [W], or one number for all coordinates."""
+    T, W = x.shape
+    if not x.is_cuda:
+        if y is not None:
+            f = y.float()
+            if experts is not None:
+                f = (f[experts.rows.long()] * experts.weights.unsqueeze(-1)).sum(1)
+            if shared is not None:
+                f = f + shared.float()
+            x += mult * (f if bias is None else f + bias)
+        if base is not None:
+            x += base
+        if step is not None:
+            x += step
+        if act is not None:
+            act.copy_(_scaled_norm_ref(x, w_in, eps, 0.0))
+        return
+    nat = _nat()
+    dt = act.dtype if act is not None else y.dtype if y is not None else torch.float32
+    assert x.is_contiguous() and act is not x and (act is None or act.is_contiguous())
+    assert all(t is None or (t.stride(1) == 1 and t.dtype == dt) for t in (y, shared))
+    assert base is None or base.is_contiguous()
+    rc = nat.lib().ab200_stream_pre(
+        x.data_ptr(), nat.ptr(y), y.stride(0) if y is not None else 0, nat.ptr(bias),
+        experts.rows.data_ptr() if experts is not None else None,
+        experts.weights.data_ptr() if experts is not None else None,
+        experts.top if experts is not None else 0, nat.ptr(shared),
+        shared.stride(0) if shared is not None else 0, float(mult), nat.ptr(base), nat.ptr(step),
+        nat.ptr(w_in), int(w_in is not None and w_in.numel() == 1), nat.ptr(act), float(eps), T, W,
+        dtype_code(dt), nat.stream_ptr())
+    nat.check(rc, "stream_pre")
+    launch_counter.add(1)
+
+
+def soft_cap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """fp32 [T, V]: cap * tanh(logits / cap). (In 16 bits logits near the cap would tie.)"""
+    if not logits.is_cuda:
+        return cap * torch.tanh(logits.float() / cap)
+    nat = _nat()
+    T, V = logits.shape
+    assert logits.stride(1) == 1 and cap > 0
+    out = torch.empty(T, V, dtype=torch.float32, device=logits.device)
+    rc = nat.lib().ab200_soft_cap(logits.data_ptr(), logits.stride(0), out.data_ptr(), T, V,
+                                  float(cap), dtype_code(logits.dtype), nat.stream_ptr())
+    nat.check(rc, "soft_cap")
+    launch_counter.add(1)
+    return out
+
+
 def stream_final_norm(x, rows, weight, eps: float, dtype: torch.dtype,
                       offset: float = 1.0) -> torch.Tensor:
     """norm(x[rows]) * (offset + weight), rounded to ``dtype``: the state the LM head reads."""
@@ -232,6 +304,28 @@ def gated_act(gu: torch.Tensor, act) -> torch.Tensor:
     return out
 
 
+# ------------------------------------------------------------------------ feed-forward without a gate
+def poly_norm(z: torch.Tensor, bias, coef, ff: int, eps: float) -> torch.Tensor:
+    """a N(z') + b N(z'^2) + c N(z'^3) + e of z' = z + bias over the first ``ff`` columns of z [T, n],
+    powers element by element, N dividing by the root mean square over the token's ff values;
+    zeros in the columns beyond. ``bias`` fp32 [ff], ``coef`` fp32 [4]: a, b, c, e."""
+    T, n = z.shape
+    if not z.is_cuda:
+        v = z[:, :ff].float() + bias
+        unit = lambda t: t / torch.sqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+        out = torch.zeros(T, n, dtype=z.dtype)
+        out[:, :ff] = coef[0] * unit(v) + coef[1] * unit(v * v) + coef[2] * unit(v * v * v) + coef[3]
+        return out
+    nat = _nat()
+    assert z.is_contiguous() and bias.numel() == ff and coef.numel() == 4
+    out = torch.empty_like(z)
+    rc = nat.lib().ab200_poly_norm(z.data_ptr(), bias.data_ptr(), coef.data_ptr(), out.data_ptr(), T, n,
+                                   ff, float(eps), dtype_code(z.dtype), nat.stream_ptr())
+    nat.check(rc, "poly_norm")
+    launch_counter.add(1)
+    return out
+
+
 # ------------------------------------------------------------------------ grouped products
 @dataclass
 class Routing:
@@ -246,8 +340,18 @@ class Routing:
     counts: list = None               # CPU path: rows per expert
 
 
-def route_ref(x, w, b, top: int, scale=None):
+def route_ref(x, w, b, top: int, scale=None, groups=None):
     z = x.float() @ w.float().t()
+    if groups is not None:     # sigmoids, among the experts of the best groups
+        s, (count, keep) = torch.sigmoid(z), groups
+        best = s.view(*s.shape[:-1], count, -1).sort(-1, descending=True).values[..., :2].sum(-1)
+        kept = torch.argsort(best, dim=-1, descending=True, stable=True)[:, :keep]
+        open_ = torch.zeros_like(best, dtype=torch.bool).scatter_(1, kept, True)
+        open_ = open_.repeat_interleave(s.shape[-1] // count, 1)
+        order = torch.argsort(s.masked_fill(~open_, float("-inf")), dim=-1, descending=True,
+                              stable=True)[:, :top]
+        own = s.gather(1, order)
+        return order, own / (own.sum(-1, keepdim=True) + 1e-20) * scale
     if scale is not None:      # softmax over all outputs, b: correction of the choice
         s = torch.softmax(z, -1)
         order = torch.argsort(s if b is None else s + b, dim=-1, descending=True, stable=True)[:, :top]
@@ -271,16 +375,18 @@ def _route_state(E: int, device) -> torch.Tensor:
 
 
 def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, top: int,
-          identity: int = 0, scale: float = None):
-    """Router of a mixture of experts. ``x`` fp32 [T, W] stream, ``act`` its rounding (what the
-    experts read), ``w`` [outputs, W], ``b`` fp32 [outputs] or None. The weights are the softmax over
+          identity: int = 0, scale: float = None, groups: tuple = None):
+    """Router of a mixture of experts. ``x`` [T, W]: fp32 stream, or ``act``; ``act`` what the
+    experts read, ``w`` [outputs, W], ``b`` fp32 [outputs] or None. The weights are the softmax over
     the chosen logits (with the bias ``b``) or, with a ``scale``, the chosen ones of the softmax over
-    all outputs times it (``b`` then corrects the choice only). The last ``identity`` outputs are
+    all outputs times it (``b`` then corrects the choice only). With ``groups`` = (count, kept) they
+    are the chosen sigmoids, normalised to the sum ``scale``; only experts of the best groups are
+    chosen, a group's score being the sum of its two best. The last ``identity`` outputs are
     identity experts. Returns (Routing, act rows sorted by expert)."""
     T, W = x.shape
     E = w.shape[0] - identity
     if not x.is_cuda:
-        ids, weights = route_ref(x, w, b, top, scale)
+        ids, weights = route_ref(x, w, b, top, scale, groups)
         order = torch.argsort(ids.reshape(-1), stable=True)
         rows = torch.empty_like(order)
         rows[order] = torch.arange(order.numel())
@@ -300,8 +406,11 @@ def route(x: torch.Tensor, act: torch.Tensor, w: torch.Tensor, b: torch.Tensor, 
     num_tiles = plan[4 * max_tiles:4 * max_tiles + 1]
     cursor = plan[4 * max_tiles + 4:4 * max_tiles + 4 + E]
     rows = plan[4 * max_tiles + 4 + E:].view(T, top)
-    rc = L.ab200_moe_route(x.data_ptr(), w.data_ptr(), nat.ptr(b), T, W, E + identity, E, top,
-                           int(scale is not None), scale or 0.0, ids.data_ptr(), weights.data_ptr(),
+    assert x.dtype in (torch.float32, act.dtype) and (groups is None or (b is None and not identity))
+    mode = 2 if groups is not None else int(scale is not None)
+    rc = L.ab200_moe_route(x.data_ptr(), dtype_code(x.dtype), w.data_ptr(), nat.ptr(b), T, W,
+                           E + identity, E, top, mode, scale or 0.0, *(groups or (1, 1)),
+                           ids.data_ptr(), weights.data_ptr(),
                            _route_state(E, dev).data_ptr(), cursor.data_ptr(), tiles.data_ptr(),
                            num_tiles.data_ptr(), dc, nat.stream_ptr())
     nat.check(rc, "moe_route")

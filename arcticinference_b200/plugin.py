@@ -83,6 +83,10 @@ def _ensure_registered() -> None:
                                "windowed attention; experts with identity and shared ones; layers "
                                "that use others' weights")
     register_model("Pererax", _layer_list)
+    register_config("pefivik", "layer list: latent attention with sinks and head gates, HGRN2; grouped "
+                               "experts and PolyNorm feed-forwards; a loop that the embedding enters "
+                               "again; token pair embedding")
+    register_model("Pefivik", _layer_list)
     for arch in ("ArcticMLPSpeculatorPreTrainedModel", "ArcticLSTMSpeculatorPreTrainedModel",
                  "MLPVariantSpeculatorPreTrainedModel", "MLPSpeculatorPreTrainedModel"):
         register_model(arch, _speculator)
