@@ -103,7 +103,7 @@ def random_state(cfg: ModelConfig, seed: int, device, dtype) -> Iterable:
         count += 1
         gen.manual_seed(seed * 1000003 + count)
         std = shape[-1] ** -0.5 if std is None else std
-        return (torch.randn(*shape, generator=gen, device=device) * std).to(dtype)
+        return (torch.randn(shape, generator=gen, device=device) * std).to(dtype)
 
     W, one = cfg.hidden_size, 1.0 - cfg.design.norm_offset
     yield "embed", rnd(cfg.vocab_size, W, std=1.0)

@@ -158,7 +158,7 @@ def mixture(h, f, w, p, margins=None):
     chosen, weight, lead = route(h, w[p + "router"], f["router"])
     if margins is not None:
         margins.append(lead)
-    out = expert(h, w, p + "shared.")
+    out = expert(h, w, p + "shared.") if f.get("shared") else torch.zeros_like(h)
     for e in range(f["router"]["experts"]):
         t, j = torch.nonzero(chosen == e, as_tuple=True)
         if t.numel():
