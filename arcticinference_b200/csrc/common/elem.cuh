@@ -35,6 +35,24 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
   *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
+// Packed fp32 pairs
+__device__ __forceinline__ void fma2(float2& d, const float2& a, const float2& b) {
+  asm("fma.rn.f32x2 %0, %1, %2, %0;"
+      : "+l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<const unsigned long long&>(a)),
+        "l"(reinterpret_cast<const unsigned long long&>(b)));
+}
+__device__ __forceinline__ void mul2(float2& d, const float2& a) {
+  asm("mul.rn.f32x2 %0, %0, %1;"
+      : "+l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<const unsigned long long&>(a)));
+}
+__device__ __forceinline__ void add2(float2& d, const float2& a) {
+  asm("add.rn.f32x2 %0, %0, %1;"
+      : "+l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<const unsigned long long&>(a)));
+}
+
 // Block-wide sum; `red` is 32 floats of shared memory. Every thread gets the sum.
 __device__ __forceinline__ float block_sum_all(float v, float* red) {
   v = warp_sum(v);

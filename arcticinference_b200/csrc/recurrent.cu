@@ -42,18 +42,6 @@
 
 namespace ab200 {
 
-// Packed fp32 pairs
-__device__ __forceinline__ void fma2(float2& d, const float2& a, const float2& b) {
-  asm("fma.rn.f32x2 %0, %1, %2, %0;"
-      : "+l"(reinterpret_cast<unsigned long long&>(d))
-      : "l"(reinterpret_cast<const unsigned long long&>(a)),
-        "l"(reinterpret_cast<const unsigned long long&>(b)));
-}
-__device__ __forceinline__ void mul2(float2& d, const float2& a) {
-  asm("mul.rn.f32x2 %0, %0, %1;"
-      : "+l"(reinterpret_cast<unsigned long long&>(d))
-      : "l"(reinterpret_cast<const unsigned long long&>(a)));
-}
 // DP: rows (dim, zero-padded)
 template <int DP>
 struct ScanShape {

@@ -565,18 +565,19 @@ static int launch_stream_pre(const StreamPreArgs& a, long long T_rows, cudaStrea
   return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), 0, stream, a) == cudaSuccess ? 0 : -5;
 }
 
-// Rows of n columns of which the first ff count; a block per row. N4: four-element pieces a thread holds
-// in registers (0: any width, read twice).
+// Rows of n columns of which the first ff count; a block takes rows gridDim apart, the next one on its way
+// while it computes.
 struct PolyArgs {
   const void* z;
-  const float* bias;   // [ff]
+  const void* bias;    // [n]
   const float* coef;   // a, b, c, e
   void* out;
+  long long rows;
   int n, ff;
   float eps;
 };
 
-// sums of z^2, z^4, z^6 over the block
+// sums over the block, in every thread
 __device__ __forceinline__ float3 block_sum3(float3 v, float* red) {
   v.x = warp_sum(v.x);
   v.y = warp_sum(v.y);
@@ -593,83 +594,162 @@ __device__ __forceinline__ float3 block_sum3(float3 v, float* red) {
                      warp_sum(in ? red[64 + lane] : 0.f));
 }
 
-template <typename T, int N4>
-__global__ void __launch_bounds__(512) poly_norm_kernel(const PolyArgs p) {
+// 16 bytes as pairs of floats, and back
+__device__ __forceinline__ void widen16(const uint4& q, float2 (&f)[4]) {
+  const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    f[i] = make_float2(__uint_as_float(w[i] << 16), __uint_as_float(w[i] & 0xffff0000u));
+}
+__device__ __forceinline__ void widen16(const uint4& q, float2 (&f)[2]) {
+  f[0] = make_float2(__uint_as_float(q.x), __uint_as_float(q.y));
+  f[1] = make_float2(__uint_as_float(q.z), __uint_as_float(q.w));
+}
+__device__ __forceinline__ uint4 narrow16(const float2 (&f)[4]) {
+  return make_uint4(pack_bf16x2(f[0].x, f[0].y), pack_bf16x2(f[1].x, f[1].y), pack_bf16x2(f[2].x, f[2].y),
+                    pack_bf16x2(f[3].x, f[3].y));
+}
+__device__ __forceinline__ uint4 narrow16(const float2 (&f)[2]) {
+  return make_uint4(__float_as_uint(f[0].x), __float_as_uint(f[0].y), __float_as_uint(f[1].x),
+                    __float_as_uint(f[1].y));
+}
+
+// N: 16-byte pieces of the row a thread holds, widened; 0: any width and alignment, read twice
+template <typename T, int N>
+__global__ void __launch_bounds__(1024) poly_norm_kernel(const PolyArgs p) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[96];
-  const T* z = reinterpret_cast<const T*>(p.z) + (long long)blockIdx.x * p.n;
-  T* out = reinterpret_cast<T*>(p.out) + (long long)blockIdx.x * p.n;
-  const float a = p.coef[0], b = p.coef[1], c = p.coef[2], e = p.coef[3];
+  __shared__ float red[2][96];
+  const T* z = reinterpret_cast<const T*>(p.z);
+  const T* bias = reinterpret_cast<const T*>(p.bias);
+  T* out = reinterpret_cast<T*>(p.out);
   const float rf = 1.f / (float)p.ff;
-  float3 s = make_float3(0.f, 0.f, 0.f);
-  auto count = [&](float v) {
-    const float q = v * v, r = q * q;
-    s.x += q;
-    s.y += r;
-    s.z = fmaf(r, q, s.z);
-  };
+  const float ca = p.coef[0], cb = p.coef[1], cc = p.coef[2], e = p.coef[3];
   float fa = 0.f, fb = 0.f, fc = 0.f;
-  auto factors = [&]() {
-    s = block_sum3(s, red);
-    fa = a / sqrtf(s.x * rf + p.eps);
-    fb = b / sqrtf(s.y * rf + p.eps);
-    fc = c / sqrtf(s.z * rf + p.eps);
+  int turn = 0;
+  auto factors = [&](float3 s) {   // from the thread's sums of z^2, z^4, z^6
+    s = block_sum3(s, red[turn]);  // (what the row before left is still being read)
+    turn ^= 1;
+    fa = ca / sqrtf(s.x * rf + p.eps);
+    fb = cb / sqrtf(s.y * rf + p.eps);
+    fc = cc / sqrtf(s.z * rf + p.eps);
   };
-  auto poly = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, fc, fb), fa), e); };
-  if constexpr (N4 > 0) {
-    float4 v[N4];
+  if constexpr (N > 0) {
+    constexpr int V = 16 / sizeof(T);
+    uint4 raw[N];
+    float2 v[N][V / 2];
+    const float2 zero = make_float2(0.f, 0.f);
+    auto fetch = [&](long long row) {
 #pragma unroll
-    for (int j = 0; j < N4; ++j) {
-      const int i = (threadIdx.x + j * blockDim.x) * 4;
-      v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (i < p.ff) {
-        const float4 x = load4(z + i), y = load4(p.bias + i);
-        v[j] = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
+      for (int j = 0; j < N; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * V;
+        raw[j] = make_uint4(0, 0, 0, 0);
+        if (row < p.rows && i < p.n) raw[j] = *reinterpret_cast<const uint4*>(z + row * p.n + i);
+      }
+    };
+    fetch(blockIdx.x);
+    for (long long row = blockIdx.x; row < p.rows; row += gridDim.x) {
+      float2 s2 = zero, s4 = zero, s6 = zero;
+#pragma unroll
+      for (int j = 0; j < N; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * V;
+        widen16(raw[j], v[j]);
+        if (i < p.n) {
+          float2 w[V / 2];
+          widen16(*reinterpret_cast<const uint4*>(bias + i), w);
+#pragma unroll
+          for (int k = 0; k < V / 2; ++k) add2(v[j][k], w[k]);
+          if (i + V > p.ff) {   // the columns beyond count nothing
+#pragma unroll
+            for (int k = 0; k < V / 2; ++k) {
+              if (i + 2 * k >= p.ff) v[j][k].x = 0.f;
+              if (i + 2 * k + 1 >= p.ff) v[j][k].y = 0.f;
+            }
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < V / 2; ++k) {
+          const float2 x = v[j][k];
+          float2 q = x, r;
+          fma2(s2, x, x);
+          mul2(q, x);
+          r = q;
+          mul2(r, q);
+          add2(s4, r);
+          fma2(s6, r, q);
+        }
+      }
+      fetch(row + gridDim.x);
+      factors(make_float3(s2.x + s2.y, s4.x + s4.y, s6.x + s6.y));
+      const float2 A = make_float2(fa, fa), B = make_float2(fb, fb), C = make_float2(fc, fc),
+                   E = make_float2(e, e);
+#pragma unroll
+      for (int j = 0; j < N; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * V;
+        if (i >= p.n) continue;
+#pragma unroll
+        for (int k = 0; k < V / 2; ++k) {   // ((c v + b) v + a) v + e
+          float2 y = B, u = A, x = v[j][k];
+          fma2(y, C, x);
+          fma2(u, y, x);
+          y = E;
+          fma2(y, u, x);
+          v[j][k] = y;
+        }
+        if (i + V > p.ff) {
+#pragma unroll
+          for (int k = 0; k < V / 2; ++k) {
+            if (i + 2 * k >= p.ff) v[j][k].x = 0.f;
+            if (i + 2 * k + 1 >= p.ff) v[j][k].y = 0.f;
+          }
+        }
+        *reinterpret_cast<uint4*>(out + row * p.n + i) = narrow16(v[j]);
       }
     }
-#pragma unroll
-    for (int j = 0; j < N4; ++j) {
-      count(v[j].x);
-      count(v[j].y);
-      count(v[j].z);
-      count(v[j].w);
-    }
-    factors();
-#pragma unroll
-    for (int j = 0; j < N4; ++j) {
-      const int i = (threadIdx.x + j * blockDim.x) * 4;
-      if (i < p.ff)
-        store4(out + i, make_float4(poly(v[j].x), poly(v[j].y), poly(v[j].z), poly(v[j].w)));
-      else if (i < p.n)
-        store4(out + i, make_float4(0.f, 0.f, 0.f, 0.f));
-    }
   } else {
-    for (int i = threadIdx.x; i < p.ff; i += blockDim.x) count(to_f32<T>(z[i]) + p.bias[i]);
-    factors();
-    for (int i = threadIdx.x; i < p.n; i += blockDim.x)
-      out[i] = from_f32<T>(i < p.ff ? poly(to_f32<T>(z[i]) + p.bias[i]) : 0.f);
+    for (long long row = blockIdx.x; row < p.rows; row += gridDim.x) {
+      const T* z_row = z + row * p.n;
+      auto at = [&](int i) { return to_f32<T>(z_row[i]) + to_f32<T>(bias[i]); };
+      float3 s = make_float3(0.f, 0.f, 0.f);
+      for (int i = threadIdx.x; i < p.ff; i += blockDim.x) {
+        const float x = at(i), q = x * x, r = q * q;
+        s.x += q;
+        s.y += r;
+        s.z = fmaf(r, q, s.z);
+      }
+      factors(s);
+      for (int i = threadIdx.x; i < p.n; i += blockDim.x) {
+        const float x = i < p.ff ? at(i) : 0.f;
+        out[row * p.n + i] = from_f32<T>(i < p.ff ? fmaf(x, fmaf(x, fmaf(x, fc, fb), fa), e) : 0.f);
+      }
+    }
   }
 }
 
 template <typename T>
 static int launch_poly_norm(const PolyArgs& a, long long T_rows, cudaStream_t stream) {
-  const bool vec = a.n % 4 == 0 && a.ff % 4 == 0 &&
+  constexpr int V = 16 / sizeof(T);
+  const bool vec = a.n % V == 0 &&
                    ((reinterpret_cast<uintptr_t>(a.z) | reinterpret_cast<uintptr_t>(a.bias) |
                      reinterpret_cast<uintptr_t>(a.out)) & 15) == 0;
-  const int n4 = (a.n + 3) / 4;
+  const int pieces = a.n / V;
   auto k = poly_norm_kernel<T, 0>;
   int threads = 512;
-  if (vec && n4 <= 512 * 16) {
-    while (threads > 64 && n4 <= threads) threads /= 2;
-    const int per = (n4 + threads - 1) / threads;
+  if (vec && pieces <= 1024 * 4) {
+    const int most = T_rows <= 148 ? 1 : 4;   // few rows: more threads on each
+    threads = 64;
+    while (threads < 1024 && pieces > threads * most) threads *= 2;
+    const int per = (pieces + threads - 1) / threads;
     k = per <= 1   ? poly_norm_kernel<T, 1>
         : per <= 2 ? poly_norm_kernel<T, 2>
-        : per <= 4 ? poly_norm_kernel<T, 4>
-        : per <= 8 ? poly_norm_kernel<T, 8>
-                   : poly_norm_kernel<T, 16>;
+        : per <= 3 ? poly_norm_kernel<T, 3>
+                   : poly_norm_kernel<T, 4>;
   }
-  return launch_pdl(k, dim3((unsigned)T_rows), dim3(threads), 0, stream, a) == cudaSuccess ? 0 : -5;
+  const long long blocks = 148 * (threads >= 1024 ? 1 : threads >= 512 ? 2 : 1024 / threads);
+  return launch_pdl(k, dim3((unsigned)(T_rows < blocks ? T_rows : blocks)), dim3(threads), 0, stream, a) ==
+                 cudaSuccess
+             ? 0
+             : -5;
 }
 
 template <typename T>
@@ -846,13 +926,12 @@ int ab200_stream_pre(void* x, const void* y, long long ldy, const void* bias, co
 }
 
 // z, out [T, n] (element type by dtype), of whose columns the first ff count (the others become zero):
-// a N(z') + b N(z'^2) + c N(z'^3) + e with z' = z + bias; bias fp32 [ff], coef fp32 [4] (a, b, c, e)
+// a N(z') + b N(z'^2) + c N(z'^3) + e with z' = z + bias; bias [n], coef fp32 [4] (a, b, c, e)
 int ab200_poly_norm(const void* z, const void* bias, const void* coef, void* out, long long T, int n,
                     int ff, float eps, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (ff < 1 || ff > n) return -2;
-  const PolyArgs a = {z, reinterpret_cast<const float*>(bias), reinterpret_cast<const float*>(coef), out,
-                      n, ff, eps};
+  const PolyArgs a = {z, bias, reinterpret_cast<const float*>(coef), out, T, n, ff, eps};
   return dtype == 0 ? launch_poly_norm<bf16>(a, T, stream) : launch_poly_norm<float>(a, T, stream);
 }
 

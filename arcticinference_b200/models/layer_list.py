@@ -294,7 +294,7 @@ class LayerListForCausalLM:
             n = round_up(f.ff, 8) if self.dtype == torch.bfloat16 else f.ff
             lw.put(w_up=padded(c.take("mlp.up", f.ff, W), n).contiguous(),
                    w_down=padded(c.take("mlp.down", W, f.ff), W, n).contiguous(),
-                   up_bias=c.vector("mlp.up.b", f.ff), down_bias=c.vector("mlp.down.b", W),
+                   up_bias=padded(c.take("mlp.up.b", f.ff), n), down_bias=c.vector("mlp.down.b", W),
                    act=c.vector("mlp.act", 4))
             return lw
         else:

@@ -308,16 +308,16 @@ def gated_act(gu: torch.Tensor, act) -> torch.Tensor:
 def poly_norm(z: torch.Tensor, bias, coef, ff: int, eps: float) -> torch.Tensor:
     """a N(z') + b N(z'^2) + c N(z'^3) + e of z' = z + bias over the first ``ff`` columns of z [T, n],
     powers element by element, N dividing by the root mean square over the token's ff values;
-    zeros in the columns beyond. ``bias`` fp32 [ff], ``coef`` fp32 [4]: a, b, c, e."""
+    zeros in the columns beyond. ``bias`` [n] of z's element type, ``coef`` fp32 [4]: a, b, c, e."""
     T, n = z.shape
     if not z.is_cuda:
-        v = z[:, :ff].float() + bias
+        v = z[:, :ff].float() + bias[:ff].float()
         unit = lambda t: t / torch.sqrt(t.pow(2).mean(-1, keepdim=True) + eps)
         out = torch.zeros(T, n, dtype=z.dtype)
         out[:, :ff] = coef[0] * unit(v) + coef[1] * unit(v * v) + coef[2] * unit(v * v * v) + coef[3]
         return out
     nat = _nat()
-    assert z.is_contiguous() and bias.numel() == ff and coef.numel() == 4
+    assert z.is_contiguous() and bias.numel() == n and bias.dtype == z.dtype and coef.numel() == 4
     out = torch.empty_like(z)
     rc = nat.lib().ab200_poly_norm(z.data_ptr(), bias.data_ptr(), coef.data_ptr(), out.data_ptr(), T, n,
                                    ff, float(eps), dtype_code(z.dtype), nat.stream_ptr())

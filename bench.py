@@ -56,7 +56,7 @@ def parse_args():
     ap.add_argument("--no-clocks", action="store_true")
     ap.add_argument("--workload", default="serving", choices=["serving", "layers"],
                     help="serving: the headline benchmark; layers: prefill and decode of "
-                         "Pererax, Zatirax and Taralix layers beside Llama layers of equal size "
+                         "Pefivik, Pererax, Zatirax and Taralix layers beside Llama layers of equal size "
                          "(benchmarks/layer_bench.py)")
     ap.add_argument("--layer-case", default=None)
     return ap.parse_args()

@@ -157,6 +157,14 @@ CASES = {
     "delta_prefill_4x256": ("delta", (32, 4, 256)),
     "delta_decode_128": ("delta", (32, 128, 1)),
     "delta_decode_64": ("delta", (32, 64, 1)),
+    "forget_prefill_4x2048": ("forget", (32, 4, 2048)),
+    "forget_prefill_4x256": ("forget", (32, 4, 256)),
+    "forget_decode_128": ("forget", (32, 128, 1)),
+    "poly_norm_prefill": ("poly", (8192, 21504)),
+    "poly_norm_prefill_9600": ("poly", (8192, 9600)),
+    "poly_norm_decode": ("poly", (128, 21504)),
+    "soft_cap_decode": ("soft_cap", (128, 128256)),
+    "stream_pre": ("pre", (8192, 4096)),
     "memory_prefill_4x2048": ("memory", (16, 4, 2048)),
     "memory_decode_128": ("memory", (16, 128, 1)),
 }
@@ -332,6 +340,42 @@ def run_case(a, case):
             sets = [(R(T, 2 * nk + nv + 2 * H), R(T, nv), rnd(nseq + 1, H, d, cols), rnd(nseq + 1, 2, H))
                     for _ in range(nc)]
             fn = lambda i=0: states.memory_scan(*sets[i][:2], *w, sh, *sets[i][2:], step, 1e-6)
+    elif kind == "forget":
+        import numpy as np
+        from arcticinference_b200.ops import state_ops as states
+        H, nseq, n = prm
+        T, d = nseq * n, 128
+        step = states.StateStep.build(np.asarray([(i * n, n, i + 1, 0 if n > 1 else 5, 0)
+                                                  for i in range(nseq)], dtype=np.int32), DEV)
+        byts = 2.0 * T * H * 4 * d + 4.0 * nseq * H * d * d * (1 if n > 1 else 2)
+        flops = 4.0 * T * H * d * d
+        nc = copies_for(byts)
+        sh = states.ForgetShape(H, d, d, 0, H * d, 2 * H * d)
+        w = (torch.rand(H * d, device=DEV) * 4, torch.rand(H * d, device=DEV) * 0.9, torch.ones(d, device=DEV))
+        sets = [(R(T, 3 * H * d), torch.randn(nseq + 1, H, d, d, device=DEV)) for _ in range(nc)]
+        fn = lambda i=0: states.forget_scan(sets[i][0], *w, sh, sets[i][1], step, 1e-6)
+    elif kind == "poly":
+        from arcticinference_b200.ops import stream_ops as st
+        T, ff = prm
+        nc = copies_for(4 * T * ff)
+        zs, bias, coef = [R(T, ff) for _ in range(nc)], R(ff), torch.ones(4, device=DEV)
+        fn = lambda i=0: st.poly_norm(zs[i], bias, coef, ff, 1e-6)
+        flops, byts = 0.0, 4.0 * T * ff
+    elif kind == "soft_cap":
+        from arcticinference_b200.ops import stream_ops as st
+        T, V = prm
+        nc = copies_for(6 * T * V)
+        zs = [R(T, V) for _ in range(nc)]
+        fn = lambda i=0: st.soft_cap(zs[i], 30.0)
+        flops, byts = 0.0, 6.0 * T * V
+    elif kind == "pre":
+        from arcticinference_b200.ops import stream_ops as st
+        T, W = prm
+        nc = copies_for(8 * T * W)
+        sets = [(torch.randn(T, W, device=DEV), R(T, W), R(T, W)) for _ in range(nc)]
+        w = torch.ones(1, device=DEV)
+        fn = lambda i=0: st.stream_pre(sets[i][0], 0.5, 1e-6, y=sets[i][1], w_in=w, act=sets[i][2])
+        flops, byts = 0.0, 12.0 * T * W
     elif kind == "sandwich":
         from arcticinference_b200.ops import stream_ops as st
         T, W = prm

@@ -1,14 +1,14 @@
-"""Prefill and decode throughput of layer-list decoders (Taralix, Zatirax, Pererax) beside Llama layers
-of equal size (random weights), with the device time of every op and the time its roofline allows.
+"""Prefill and decode throughput of layer-list decoders (Taralix, Zatirax, Pererax, Pefivik) beside Llama
+layers of equal size (random weights), with the device time of every op and the time its roofline allows.
 
     python bench.py --workload layers [--layer-case NAME]       (or: python benchmarks/layer_bench.py)
 
 Cases (width, heads x (dim, vdim), kv_rank, feed-forward):
 
-    moe-2048     2048, 16 x (128, 128), 512, 64 experts of 1408, 6 per token   (Taralix, Pererax)
-    moe-4096     4096, 32 x (128, 128), 512, 64 experts of 2048, 6 per token   (Taralix, Pererax)
-    dense-2560   2560, 40 x (64, 64),   256, 6400
-    dense-4096   4096, 32 x (128, 128), 512, 14336
+    moe-2048     2048, 16 x (128, 128), 512, 64 experts of 1408, 6 per token   (Taralix, Pererax, Pefivik)
+    moe-4096     4096, 32 x (128, 128), 512, 64 experts of 2048, 6 per token   (Taralix, Pererax, Pefivik)
+    dense-2560   2560, 40 x (64, 64),   256, 6400                      (Taralix, Zatirax, Pefivik)
+    dense-4096   4096, 32 x (128, 128), 512, 14336                     (Taralix, Zatirax, Pefivik)
     masks-4096   dense-4096 with windows and chunks of 1024 positions          (Zatirax)
 
 Taralix: every second layer shares the latents of the one before it. Zatirax: attention layers with
@@ -16,12 +16,15 @@ Taralix: every second layer shares the latents of the one before it. Zatirax: at
 key part of 64; windows and chunks of 4096 positions, which hold every context here, but in
 masks-4096. Pererax: delta-rule layers (every head with keys of its own), attention beside a matrix
 memory, and windowed attention (1024 positions), the attentions with 8 K/V heads; of the experts per
-token one is the shared expert and 8 identity experts take part in the choice. The Llama beside them has the same width, query heads, head dimension and active feed-forward width, and 8
+token one is the shared expert and 8 identity experts take part in the choice. Pefivik: latent layers
+with sinks and head gates alternate with HGRN2 layers; of the experts per token one is the shared expert,
+the others come from 4 of 8 groups; the dense feed-forwards, which have two matrices, are 3/2 as wide. The
+Llama beside them has the same width, query heads, head dimension and active feed-forward width, and 8
 K/V heads. Prefill: four prompts of 2048 tokens in one step. Decode: 128 sequences at 2000 tokens of
 context, captured step. Both are one forward pass without the LM head, timed with CUDA events; the
 weights of a pass exceed L2. The roofline of an op is the larger of its algorithmic bytes over the
 measured copy bandwidth and its flops over the measured bf16 rate; only visible keys count. The
-recurrences compute in fp32: three (delta rule) or two (matrix memory) multiply-adds per state element
+recurrences compute in fp32: three (delta rule) or two (the others) multiply-adds per state element
 and token over the fp32 rate (128 per SM and cycle) are a third bound of theirs; ``of_bytes`` leaves it
 out.
 """
@@ -104,6 +107,24 @@ def pererax_config(c):
         "layers": [{**l, "mlp": mlp} for l in (delta, both, window, delta)]})
 
 
+def pefivik_config(c):
+    from arcticinference_b200.config import ModelConfig
+    H, d = c["heads"], c["dim"]
+    latent = {"type": "latent_attention", "mixer": {
+        "heads": H, "dim": d, "vdim": d, "kv_rank": c["rank"], "scale": d ** -0.5}}
+    scan = {"type": "hgrn2", "mixer": {"heads": H, "dim": d, "vdim": d}}
+    mlp = {"kind": "dense", "ff": c["ff"] * 3 // 2}
+    if c["experts"]:
+        mlp = {"kind": "moe", "expert": {"ff": c["ff"]}, "shared": {"ff": c["ff"]},
+               "router": {"experts": c["experts"], "top": c["top"] - 1, "scale": 2.5,
+                          "groups": {"count": 8, "keep": 4}}}
+    return ModelConfig.from_layer_list({
+        "architecture": "Pefivik", "width": c["width"], "vocab": VOCAB, "norm": {"eps": 1e-6},
+        "embedding": {"bigram": {"buckets": 50021, "mul_prev": 10007, "mul_cur": 3}},
+        "residual_mult": 0.5, "logit_softcap": 30.0, "loop": None,
+        "layers": [{**l, "mlp": mlp} for l in (latent, scan, latent, scan)]})
+
+
 def model_configs(c):
     from arcticinference_b200.config import ModelConfig
     llama = ModelConfig(hidden_size=c["width"], num_hidden_layers=LAYERS,
@@ -116,6 +137,7 @@ def model_configs(c):
     else:
         out["zatirax"] = zatirax_config(c)
     if "mask" not in c:
+        out["pefivik"] = pefivik_config(c)
         out["taralix"] = taralix_config(c)
         out["llama"] = llama
     return out
@@ -147,7 +169,8 @@ FP32_FMAS = 148 * 128 * 1.965e9      # per second, every SM at its highest clock
 def rooflines(model, q_lens, kv_lens, fp32: bool = True):
     """op -> seconds the layers' algorithmic bytes and flops allow (2 bytes per element; ``fp32``: and
     the fp32 multiply-adds of recurrences)."""
-    from arcticinference_b200.config import AttentionSpec, DeltaRuleSpec, MaskSpec, ParallelSpec
+    from arcticinference_b200.config import (AttentionSpec, DeltaRuleSpec, ForgetScanSpec, MaskSpec,
+                                             ParallelSpec)
     cfg = model.cfg
     hbm, flops, _ = peaks()
     T, S = sum(q_lens), len(q_lens)
@@ -176,6 +199,12 @@ def rooflines(model, q_lens, kv_lens, fp32: bool = True):
             fmas=3.0 * T * H * d * dv)
         linear(W, H * dv)
 
+    def forget(m):
+        H, d, dv = m.heads, m.dim, m.vdim
+        linear(H * (2 * d + dv), W)
+        add("forget_scan", 2.0 * T * H * (2 * d + 2 * dv) + state(H, d, dv), fmas=2.0 * T * H * d * dv)
+        linear(W, H * dv)
+
     def parallel(m):
         l, r = m.left, m.right
         linear(l.heads * l.dim + l.kv_heads * (l.dim + l.vdim) + 2 * r.heads * (r.dim + r.vdim + 1), W)
@@ -202,13 +231,15 @@ def rooflines(model, q_lens, kv_lens, fp32: bool = True):
             linear(W, I)
             add("rmsnorm", 2 * 2.0 * T * 4 * W)
         return out
-    norm = {"sandwich": "stream_sandwich", "post": "stream_norm", "output": "stream_add"}[
-        cfg.design.residual]
+    norm = {"sandwich": "stream_sandwich", "post": "stream_norm", "output": "stream_add",
+            "pre": "stream_pre"}[cfg.design.residual]
     for i, _ in cfg.layer_runs:
         l = cfg.layer_specs[i]
         m, f = l.mixer, l.mlp
         if isinstance(m, DeltaRuleSpec):
             delta(m)
+        elif isinstance(m, ForgetScanSpec):
+            forget(m)
         elif isinstance(m, ParallelSpec):
             parallel(m)
         elif isinstance(m, AttentionSpec):
@@ -218,12 +249,12 @@ def rooflines(model, q_lens, kv_lens, fp32: bool = True):
             attention(m)
         else:
             H, d, dv = m.heads, m.dim, m.vdim
-            masked = m.mask.kind != "causal"
+            masked = m.mask.kind != "causal" or m.sink is not None or m.head_gate
             pairs, ctx = visible_pairs(m.mask, q_lens, kv_lens)
             R, rot = m.kv_rank, m.rot_dim
             own = R + rot if m.kv_from is None else 0
             dq = d + rot
-            linear(H * dq + own, W)
+            linear(H * dq + own + (H if m.head_gate else 0), W)
             if rot:
                 add("latent_rope_cache", 2.0 * T * 2 * (R + rot + H * rot))
             elif own:
@@ -258,6 +289,11 @@ def rooflines(model, q_lens, kv_lens, fp32: bool = True):
             if f.shared is not None:
                 dense(f.shared.ff)
             add(norm, T * W * (12.0 if f.shared is not None else 10.0) + 2.0 * n * W)
+        elif f.act == "poly_norm":
+            linear(f.ff, W)
+            add("poly_norm", 2.0 * T * 2 * f.ff)
+            linear(W, f.ff)
+            add(norm, T * W * 12.0)
         else:
             dense(f.ff)
             add(norm, T * W * 12.0)
@@ -371,7 +407,7 @@ def fwd_graph(r, g):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("--layer-case", choices=sorted(CASES), default=None)
-    ap.add_argument("--model", choices=["pererax", "zatirax", "taralix", "llama"], default=None)
+    ap.add_argument("--model", choices=["pefivik", "pererax", "zatirax", "taralix", "llama"], default=None)
     ns = ap.parse_args(argv)
     import torch
     torch.cuda.set_device(0)

@@ -239,9 +239,9 @@ def test_stream_pre():
 
 
 def test_poly_norm_and_soft_cap():
-    z, bias, coef = torch.randn(5, 24) * 3, torch.randn(21), torch.tensor([0.6, -0.5, 0.4, 0.3])
+    z, bias, coef = torch.randn(5, 24) * 3, torch.randn(24), torch.tensor([0.6, -0.5, 0.4, 0.3])
     got = st.poly_norm(z, bias, coef, 21, 0.02)
-    want = oracle.poly_norm(z[:, :21].double() + bias.double(), coef, 0.02)
+    want = oracle.poly_norm(z[:, :21].double() + bias[:21].double(), coef, 0.02)
     assert float((got[:, :21] - want).abs().max()) < 1e-5 and float(got[:, 21:].abs().max()) == 0
     cap = st.soft_cap(torch.tensor([[1.0, -50.0, 0.0]]), 4.0)
     assert cap.dtype == torch.float32
