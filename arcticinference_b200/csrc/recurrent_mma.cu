@@ -121,13 +121,37 @@ tile_mma_kernel(const ScanArgs p) {
 
   // ---- 1. queries, keys, values: four channels and all of the tile's tokens a thread
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int x = tid * 4; x < 2 * DP + vcols; x += kThreads * 4) {
+  const bool halves = FORGET && p.vec;
+  if (halves) {   // (the keys come with the decays: enough threads for half of the tokens each)
+    const int quads = (DP + vcols) / 4;
+    for (int x = tid; x < 2 * quads; x += kThreads) {
+      const int late = x >= quads, d_all = (x - late * quads) * 4;
+      const bool query = d_all < DP;
+      const int d = query ? d_all : d_all - DP;
+      const bool ok = d < (query ? p.dim : p.vdim);
+      const T* src = in.proj + (long long)(t0 + late * 8) * p.ld + (query ? in.q_col : in.v_col) + (ok ? d : 0);
+      float* dst = query ? sC + late * 8 * DP + d : rec_v + late * 8 * vld + d;
+      const int dst_ld = query ? DP : vld;
+      uint2 raw[8];
+#pragma unroll
+      for (int t = 0; t < 8; ++t, src += p.ld) {
+        raw[t] = make_uint2(0u, 0u);
+        if (ok && late * 8 + t < nt) raw[t] = *reinterpret_cast<const uint2*>(src);
+      }
+#pragma unroll
+      for (int t = 0; t < 8; ++t, dst += dst_ld) {
+        const float4 y = widen(raw[t].x, raw[t].y);
+        store4(dst, query ? silu4(y) : y);
+      }
+    }
+  }
+  for (int x = halves ? 2 * DP + vcols : tid * 4; x < 2 * DP + vcols; x += kThreads * 4) {
     const int part = x < DP ? 0 : x < 2 * DP ? 1 : 2;
     if (FORGET && part == 1) continue;   // (keys: with the decays)
     const int d = x - part * DP, limit = part == 2 ? p.vdim : p.dim;
     float* dst = part == 2 ? rec_v + d : (part == 0 ? sC : sB) + d;
     const int dst_ld = part == 2 ? vld : DP;
-    if (p.vec && (!DELTA || p.taps <= kTaps)) {
+    if (!FORGET && p.vec && (!DELTA || p.taps <= kTaps)) {
       const bool ok = d < limit;
       const T* src = in.proj + (long long)t0 * p.ld + in.col(part) + (ok ? d : 0);
       if constexpr (DELTA) {
@@ -169,7 +193,6 @@ tile_mma_kernel(const ScanArgs p) {
 #pragma unroll
         for (int t = 0; t < kTT; ++t, src += p.ld, dst += dst_ld) {
           float4 y = ok && t < nt ? load4(src) : zero;
-          if (FORGET && part == 0) y = silu4(y);
           if (one == 0) y.x = 1.f;
           if (one == 1) y.y = 1.f;
           if (one == 2) y.z = 1.f;
