@@ -55,15 +55,20 @@ struct LatentArgs {
   int x_bufs;              // buffers of the key-only piece (0: none)
   int mask_kind, mask_size;
   float scale, scale_log2;
-  const float* sink;           // [H] or null
-  const __nv_bfloat16* gate;   // [T][ldg], one per head, or null
-  long long ldg;
   uint32_t tmem_cols;
   __nv_bfloat16* out;      // [T * H][R]
   float* o_part;           // [pieces of keys][T * H][R]
   float* lse_part;         // [pieces of keys][T * H]
   long long rows_total;    // T * H
   int* status;
+};
+
+// What acts on finished rows. (A parameter of its own: as part of LatentArgs it costs the 48-row kernel
+// spilled registers.)
+struct LatentExt {
+  const float* sink;           // [H] or null
+  const __nv_bfloat16* gate;   // [T][ldg], one per head, or null
+  long long ldg;
 };
 
 __device__ __forceinline__ void bar_softmax() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
@@ -113,7 +118,8 @@ __device__ __forceinline__ int reduce16_index(int lane) {
 template <int NR>
 __global__ void __launch_bounds__(kLatThreads, 1)
 latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
-                        const __grid_constant__ CUtensorMap tmap_c, const LatentArgs p) {
+                        const __grid_constant__ CUtensorMap tmap_c, const LatentArgs p,
+                        const LatentExt x) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
@@ -512,14 +518,14 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
       if (n_pieces > 1 && tid < n_rows)
         p.lse_part[(long long)piece * p.rows_total + row0 + tid] =
             sum > 0.f ? m_s[tid] * p.scale + logf(sum) : -INFINITY;
-      const bool last = n_pieces <= 1 && tid < n_rows && sum > 0.f;   // (else the merge does it)
-      const int tok = (row0 + tid) / p.H, head = row0 + tid - tok * p.H;
-      if (last && p.sink != nullptr)
-        sum += ex2_approx(fmaf(p.sink[head], 1.4426950408889634f, neg_s[tid]));
-      float inv = sum > 0.f ? 1.f / sum : 0.f;
-      if (last && p.gate != nullptr)
-        inv *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[tok * p.ldg + head])));
-      inv_s[tid] = inv;
+      float factor = 1.f;
+      if (n_pieces <= 1 && tid < n_rows && sum > 0.f) {   // (else the merge does it)
+        const int tok = (row0 + tid) / p.H, head = row0 + tid - tok * p.H;
+        if (x.sink != nullptr) sum += ex2_approx(fmaf(x.sink[head], 1.4426950408889634f, neg_s[tid]));
+        if (x.gate != nullptr)
+          factor = __fdividef(1.f, 1.f + __expf(-__bfloat162float(x.gate[tok * x.ldg + head])));
+      }
+      inv_s[tid] = sum > 0.f ? factor / sum : 0.f;
     }
     bar_softmax();
     if (n_tiles > 0) {
@@ -567,8 +573,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_q,
 }
 
 template <int NR>
-static int launch_latent(const CUtensorMap& tq, const CUtensorMap& tc, LatentArgs a, int num_work,
-                         cudaStream_t stream) {
+static int launch_latent(const CUtensorMap& tq, const CUtensorMap& tc, LatentArgs a, const LatentExt& x,
+                         int num_work, cudaStream_t stream) {
   const int NC = a.pieces;
   const size_t limit = 227 * 1024 - 4096;   // static shared memory and alignment aside
   const int NX = a.x_bufs;   // (wanted: 0 or 1)
@@ -608,7 +614,7 @@ static int launch_latent(const CUtensorMap& tq, const CUtensorMap& tc, LatentArg
     attr_set[dev] = true;
   }
   return launch_pdl(latent_attention_kernel<NR>, dim3((unsigned)num_work), dim3(kLatThreads), smem,
-                    stream, tq, tc, a) == cudaSuccess
+                    stream, tq, tc, a, x) == cudaSuccess
              ? 0
              : -5;
 }
@@ -646,6 +652,7 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
   if (make_tmap_2d(&tc, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)num_blocks * block_size,
                    (uint64_t)W, (uint64_t)W * 2, (uint32_t)block_size, 64) != 0)
     return -4;
+  const LatentExt x = {reinterpret_cast<const float*>(sink), reinterpret_cast<const __nv_bfloat16*>(gate), ldg};
   LatentArgs a;
   memset(&a, 0, sizeof(a));
   a.work = reinterpret_cast<const int*>(work);
@@ -657,9 +664,6 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
   a.x_bufs = key_extra / 64;
   a.mask_kind = mask_kind;
   a.mask_size = mask_size;
-  a.sink = reinterpret_cast<const float*>(sink);
-  a.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
-  a.ldg = ldg;
   a.scale = scale;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
@@ -669,10 +673,10 @@ int ab200_latent_attention(const void* q, long long q_rows, const void* cache, i
   a.status = status;
   int rc;
   switch (tile_rows) {
-    case 16: rc = launch_latent<16>(tq, tc, a, num_work, stream); break;
-    case 32: rc = launch_latent<32>(tq, tc, a, num_work, stream); break;
-    case 48: rc = launch_latent<48>(tq, tc, a, num_work, stream); break;
-    case 64: rc = launch_latent<64>(tq, tc, a, num_work, stream); break;
+    case 16: rc = launch_latent<16>(tq, tc, a, x, num_work, stream); break;
+    case 32: rc = launch_latent<32>(tq, tc, a, x, num_work, stream); break;
+    case 48: rc = launch_latent<48>(tq, tc, a, x, num_work, stream); break;
+    case 64: rc = launch_latent<64>(tq, tc, a, x, num_work, stream); break;
     default: return -2;
   }
   if (rc != 0 || max_splits <= 1) return rc;
